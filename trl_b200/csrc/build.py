@@ -24,6 +24,8 @@ OBJ = os.path.join(LIB, "obj")
 
 NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17", "--use_fast_math",
               "-Xcompiler", "-fPIC,-fvisibility=hidden", "-Xptxas", "-v", "--expt-relaxed-constexpr"]
+# sources whose results the fast approximations of exp, tanh, erf, division and square root would show in
+EXACT_MATH = {"mixers.cu"}
 # every source here builds into the one library used at any GPU count (no loads shared across a thread-block cluster)
 
 
@@ -47,7 +49,7 @@ def _digest(path: str, extra: str) -> str:
 
 def _compile(src: str, force: bool, verbose: bool) -> str:
     is_cu = src.endswith(".cu")
-    flags = NVCC_FLAGS if is_cu else ["-O3", "-std=c++17", "-fPIC", "-fvisibility=hidden", "-pthread"]
+    flags = [f for f in NVCC_FLAGS if not (f == "--use_fast_math" and os.path.basename(src) in EXACT_MATH)] if is_cu else ["-O3", "-std=c++17", "-fPIC", "-fvisibility=hidden", "-pthread"]
     tag = _digest(src, " ".join(flags))
     obj = os.path.join(OBJ, f"{os.path.basename(src)}.{tag}.o")
     if os.path.exists(obj) and not force:

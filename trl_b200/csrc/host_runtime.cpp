@@ -173,6 +173,28 @@ API int trlb_sched_admit(void* h, int max_admit, int64_t* out_ids, int32_t* out_
   return n;
 }
 
+// Makes room for `total_tokens` tokens of the request in `slot`, taking blocks from the pool as needed; its row of
+// block_table is extended.  Returns the number of blocks added, -1 when the slot is idle or the sequence would exceed
+// its table row, -2 when the pool is empty (what was taken before stays with the request).
+API int trlb_sched_grow(void* h, int slot, int total_tokens, int32_t* block_table) {
+  auto* s = static_cast<Scheduler*>(h);
+  std::lock_guard<std::mutex> g(s->mu);
+  if (slot < 0 || slot >= s->max_slots || s->slots[slot].id < 0) return -1;
+  Running& run = s->slots[slot];
+  const int need = (total_tokens + s->block_size - 1) / s->block_size;
+  if (need > s->max_blocks_per_seq) return -1;
+  int32_t* row = block_table + (size_t)slot * s->max_blocks_per_seq;
+  int added = 0;
+  while ((int)run.blocks.size() < need) {
+    const int b = s->pool.alloc();
+    if (b < 0) return -2;
+    row[run.blocks.size()] = b;
+    run.blocks.push_back(b);
+    ++added;
+  }
+  return added;
+}
+
 // Retire the request in `slot`; its blocks are released (shared prompt blocks survive while the
 // group still has members).  Returns the request id or -1.
 API int64_t trlb_sched_retire(void* h, int slot, int64_t group) {

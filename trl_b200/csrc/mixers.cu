@@ -1,0 +1,752 @@
+// Element-wise, cache and recurrence kernels of the layered decoders (models/layered.py): embedding scale, Dynamic-Tanh
+// norm fused with the residual addition, latent-attention preparation / absorption, mLSTM gates, steps and outputs.
+//
+// T is the model dtype (bf16 or fp32).  The residual stream, norm statistics, gates, attention scores and recurrent
+// states are fp32 in both.  This file is compiled without fast-math (csrc/build.py: EXACT_MATH).
+//
+// Decode kernels work on one row per sequence slot; seq_lens[slot] is the position of the slot's new token and a
+// negative value marks an idle slot.  fp32 sums of the stream-K decode GEMM are cleared by their last reader
+// (`clear`), so no memset runs between two steps.
+//
+// The latent-attention prompt kernel here covers every size and dtype; bf16 prompts with 8-element aligned head
+// sizes run the tcgen05 kernel of latent_attn_tcgen05.cu.
+#include "mixers.cuh"
+
+namespace trlb {
+
+// ------------------------------------------------------------------------------------------------------------
+// embedding and norm
+// ------------------------------------------------------------------------------------------------------------
+template <typename T>
+__global__ void __launch_bounds__(256)
+embed_scaled_kernel(const long long* __restrict__ ids, const T* __restrict__ emb, float* __restrict__ x, int H, int V,
+                    float scale) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const long long id = ids[blockIdx.x];
+  for (int j = threadIdx.x; j < H; j += blockDim.x)
+    x[(size_t)blockIdx.x * H + j] = (id >= 0 && id < V) ? to_f(emb[(size_t)id * H + j]) * scale : 0.f;
+}
+
+// x (+= delta) ; out = tanh(alpha x) w + b.  VEC elements per thread along H (H % VEC == 0).
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256)
+dynamic_tanh_kernel(float* __restrict__ x, float* __restrict__ delta, const float* __restrict__ alpha_p,
+                    const float* __restrict__ w, const float* __restrict__ b, T* __restrict__ out, long long n_vec,
+                    int H, int clear) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const float alpha = *alpha_p;
+  for (long long v = blockIdx.x * (long long)blockDim.x + threadIdx.x; v < n_vec; v += (long long)gridDim.x * blockDim.x) {
+    const long long e = v * VEC;
+    const int j = (int)(e % H);
+    float a[VEC];
+    if (VEC == 4) {
+      const float4 t = *reinterpret_cast<const float4*>(x + e);
+      a[0] = t.x; a[1 % VEC] = t.y; a[2 % VEC] = t.z; a[3 % VEC] = t.w;
+    } else {
+      a[0] = x[e];
+    }
+    if (delta != nullptr) {
+      if (VEC == 4) {
+        const float4 d = *reinterpret_cast<const float4*>(delta + e);
+        a[0] += d.x; a[1 % VEC] += d.y; a[2 % VEC] += d.z; a[3 % VEC] += d.w;
+        *reinterpret_cast<float4*>(x + e) = make_float4(a[0], a[1 % VEC], a[2 % VEC], a[3 % VEC]);
+        if (clear) *reinterpret_cast<float4*>(delta + e) = make_float4(0.f, 0.f, 0.f, 0.f);
+      } else {
+        a[0] += delta[e];
+        x[e] = a[0];
+        if (clear) delta[e] = 0.f;
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) out[e + i] = from_f<T>(tanhf(alpha * a[i]) * w[j + i] + b[j + i]);
+  }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256)
+gelu_erf_kernel(const T* __restrict__ z, T* __restrict__ out, long long n) {
+  for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x) {
+    const float v = to_f(z[i]);
+    out[i] = from_f<T>(0.5f * v * (1.f + erff(v * 0.70710678118654752f)));
+  }
+}
+
+// ------------------------------------------------------------------------------------------------------------
+// latent attention
+// ------------------------------------------------------------------------------------------------------------
+struct LatentPrep {
+  float* acc;           // [rows, ld]: query latent | key/value latent | rotated key | gate logits
+  long long ld;
+  int q_rank, kv_rank, rot, heads, clear;
+  const float* q_norm;
+  const float* kv_norm;
+  float eps;
+  const int* positions;  // [rows] position of every row (prompt) or of every slot (decode); negative: idle
+  const int* tok_slot;   // [rows] or null (slot = row)
+  const float2* table;   // [table_len, rot / 2] (cos, sin) with the rotation's magnitude folded in
+  int table_len;
+  float* gate;           // [rows, heads] sigmoid of the gate logits
+  int kr_off, lat_w;     // a latent row: [kv_rank | pad to kr_off | rot | pad to lat_w]
+  const int* block_table;  // null: no cache
+  int max_blocks, block_size;
+};
+
+template <typename T>
+__global__ void __launch_bounds__(256)
+latent_prep_kernel(const LatentPrep p, T* __restrict__ cq, T* __restrict__ lat, T* __restrict__ cache) {
+  __shared__ float red[64];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int row = blockIdx.x;
+  float* a = p.acc + (size_t)row * p.ld;
+  const float* akv = a + p.q_rank;
+  const float* ar = akv + p.kv_rank;
+  const float* ag = ar + p.rot;
+  float sq = 0.f, sk = 0.f;
+  for (int j = threadIdx.x; j < p.q_rank; j += blockDim.x) sq += a[j] * a[j];
+  for (int j = threadIdx.x; j < p.kv_rank; j += blockDim.x) sk += akv[j] * akv[j];
+  const float2 s = block_sum2(sq, sk, red);
+  const float rq = 1.f / sqrtf(s.x / (float)p.q_rank + p.eps), rk = 1.f / sqrtf(s.y / (float)p.kv_rank + p.eps);
+  for (int j = threadIdx.x; j < p.q_rank; j += blockDim.x)
+    cq[(size_t)row * p.q_rank + j] = from_f<T>(a[j] * rq * p.q_norm[j]);
+  for (int h = threadIdx.x; h < p.heads; h += blockDim.x) p.gate[(size_t)row * p.heads + h] = sigmoid_f(ag[h]);
+  const int pos = p.positions[row];
+  const bool live = pos >= 0 && pos < p.table_len;
+  T* dense = lat == nullptr ? nullptr : lat + (size_t)row * p.lat_w;
+  T* paged = nullptr;
+  if (live && p.block_table != nullptr) {
+    const int slot = p.tok_slot ? p.tok_slot[row] : row;
+    if (slot >= 0 && pos / p.block_size < p.max_blocks) {
+      const int blk = p.block_table[(size_t)slot * p.max_blocks + pos / p.block_size];
+      paged = cache + ((size_t)blk * p.block_size + pos % p.block_size) * p.lat_w;
+    }
+  }
+  for (int j = threadIdx.x; j < p.kv_rank; j += blockDim.x) {
+    const T v = from_f<T>(akv[j] * rk * p.kv_norm[j]);
+    if (dense) dense[j] = v;
+    if (paged) paged[j] = v;
+  }
+  for (int i = threadIdx.x; i < p.rot / 2; i += blockDim.x) {
+    const float2 cs = live ? p.table[(size_t)pos * (p.rot / 2) + i] : make_float2(1.f, 0.f);
+    const float u = ar[2 * i], v = ar[2 * i + 1];
+    const T x0 = from_f<T>(u * cs.x - v * cs.y), x1 = from_f<T>(v * cs.x + u * cs.y);
+    if (dense) { dense[p.kr_off + 2 * i] = x0; dense[p.kr_off + 2 * i + 1] = x1; }
+    if (paged) { paged[p.kr_off + 2 * i] = x0; paged[p.kr_off + 2 * i + 1] = x1; }
+  }
+  if (p.clear) {
+    __syncthreads();
+    const int n = p.q_rank + p.kv_rank + p.rot + p.heads;
+    for (int j = threadIdx.x; j < n; j += blockDim.x) a[j] = 0.f;
+  }
+}
+
+// q [rows, heads, dim + rot]: the rot part of every head turned in place.
+template <typename T>
+__global__ void __launch_bounds__(256)
+rotate_q_kernel(T* __restrict__ q, int heads, int dim, int rot, const int* __restrict__ positions,
+                const float2* __restrict__ table, int table_len, long long n) {
+  const int half = rot / 2;
+  for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x) {
+    const int f = (int)(i % half);
+    const long long th = i / half;
+    const int pos = positions[th / heads];
+    if (pos < 0 || pos >= table_len) continue;
+    T* d = q + (size_t)th * (dim + rot) + dim + 2 * f;
+    const float2 cs = table[(size_t)pos * half + f];
+    const float u = to_f(d[0]), v = to_f(d[1]);
+    d[0] = from_f<T>(u * cs.x - v * cs.y);
+    d[1] = from_f<T>(v * cs.x + u * cs.y);
+  }
+}
+
+// Prompt attention, any size: one warp per (token, head).  Keys of token t are rows t - min(pos, window - 1) .. t of
+// the packed stream (pos counts from the token's own sequence start), so no sequence table is needed.
+struct LatentPrompt {
+  int T, heads, dim, rot, vdim, kr_off, lat_w, window;
+  long long kv_ld;  // kv row: [heads * dim keys | heads * vdim values]
+  float scale;
+  const int* positions;
+  const float* sink;
+  const float* gate;  // [T, heads]
+};
+
+template <typename T>
+__global__ void __launch_bounds__(128)
+latent_prompt_kernel(const LatentPrompt p, const T* __restrict__ q, const T* __restrict__ kv, const T* __restrict__ lat,
+                     T* __restrict__ out) {
+  extern __shared__ float sm[];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const long long item = (long long)blockIdx.x * 4 + warp;
+  if (item >= (long long)p.T * p.heads) return;
+  const int t = (int)(item / p.heads), h = (int)(item % p.heads);
+  const int dq = p.dim + p.rot;
+  float* qs = sm + (size_t)warp * (dq + p.vdim);
+  float* os = qs + dq;
+  for (int d = lane; d < dq; d += 32) qs[d] = to_f(q[((size_t)t * p.heads + h) * dq + d]);
+  for (int e = lane; e < p.vdim; e += 32) os[e] = 0.f;
+  __syncwarp();
+  const int pos = p.positions[t];
+  const int back = p.window > 0 ? min(pos, p.window - 1) : pos;
+  const int k0 = t - back;
+  float m = -INFINITY, l = 0.f;
+  for (int base = k0; base <= t; base += 32) {
+    const int key = base + lane;
+    float s = -INFINITY;
+    if (key <= t) {
+      const T* kn = kv + (size_t)key * p.kv_ld + (size_t)h * p.dim;
+      const T* kr = lat + (size_t)key * p.lat_w + p.kr_off;
+      float acc = 0.f;
+      for (int d = 0; d < p.dim; ++d) acc += qs[d] * to_f(kn[d]);
+      for (int d = 0; d < p.rot; ++d) acc += qs[p.dim + d] * to_f(kr[d]);
+      s = acc * p.scale;
+    }
+    const float mn = fmaxf(m, warp_max(s));
+    const float corr = m == -INFINITY ? 0.f : expf(m - mn);
+    const float pr = key <= t ? expf(s - mn) : 0.f;
+    l = l * corr + warp_sum(pr);
+    m = mn;
+    const int nk = min(32, t - base + 1);
+    const int e_end = (p.vdim + 31) & ~31;
+    for (int e = lane; e < e_end; e += 32) {
+      float acc = e < p.vdim ? os[e] * corr : 0.f;
+      for (int j = 0; j < nk; ++j) {
+        const float w = __shfl_sync(0xffffffffu, pr, j);
+        if (e < p.vdim)
+          acc += w * to_f(kv[(size_t)(base + j) * p.kv_ld + (size_t)p.heads * p.dim + (size_t)h * p.vdim + e]);
+      }
+      if (e < p.vdim) os[e] = acc;
+    }
+    __syncwarp();
+  }
+  const float sk = p.sink[h], mt = fmaxf(m, sk);
+  const float f = expf(m - mt) / (l * expf(m - mt) + expf(sk - mt)) * p.gate[(size_t)t * p.heads + h];
+  for (int e = lane; e < p.vdim; e += 32) out[((size_t)t * p.heads + h) * p.vdim + e] = from_f<T>(os[e] * f);
+}
+
+// Decode, any size.  Absorption: q_lat[b, h] = [ W_uk[h]^T q_nope | rotated q_rot ] in the layout of a latent row.
+template <typename T>
+__global__ void __launch_bounds__(128)
+latent_absorb_kernel(float* __restrict__ qacc, long long ld, const T* __restrict__ uk, T* __restrict__ q_lat, int heads,
+                     int dim, int rot, int kv_rank, int kr_off, int lat_w, const int* __restrict__ positions,
+                     const float2* __restrict__ table, int table_len, int clear) {
+  extern __shared__ float sm[];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int h = blockIdx.x, b = blockIdx.y;
+  float* q = qacc + (size_t)b * ld + (size_t)h * (dim + rot);
+  for (int d = threadIdx.x; d < dim + rot; d += blockDim.x) {
+    // the query has the precision of the model dtype, as in a prompt
+    sm[d] = to_f(from_f<T>(q[d]));
+    if (clear) q[d] = 0.f;
+  }
+  __syncthreads();
+  const int pos = positions[b];
+  if (pos < 0 || pos >= table_len) return;
+  T* dst = q_lat + ((size_t)b * heads + h) * lat_w;
+  for (int r = threadIdx.x; r < lat_w; r += blockDim.x) {
+    float v = 0.f;
+    if (r < kv_rank) {
+      const T* w = uk + (size_t)h * dim * kv_rank + r;
+      for (int d = 0; d < dim; ++d) v += sm[d] * to_f(w[(size_t)d * kv_rank]);
+    } else if (r >= kr_off && r < kr_off + rot) {
+      const int i = (r - kr_off) >> 1;
+      const float2 cs = table[(size_t)pos * (rot / 2) + i];
+      const float a = sm[dim + 2 * i], c = sm[dim + 2 * i + 1];
+      v = ((r - kr_off) & 1) ? c * cs.x + a * cs.y : a * cs.x - c * cs.y;
+    }
+    dst[r] = from_f<T>(v);
+  }
+}
+
+struct LatentDecode {
+  int B, heads, kv_rank, lat_w, window, max_blocks, block_size, splits;
+  float scale;
+  const int* seq_lens;
+  const int* block_table;
+  const float* sink;
+};
+
+// One block per (slot, head, split): the four warps take keys in turn, lanes own dimensions of the latent row.
+constexpr int LD_MAX_REG = 32;  // lat_w <= 1024
+template <typename T>
+__global__ void __launch_bounds__(128)
+latent_decode_kernel(const LatentDecode p, const T* __restrict__ q_lat, const T* __restrict__ cache, T* __restrict__ o_lat) {
+  extern __shared__ float sm[];  // [lat_w] query, [4][kv_rank] partial outputs, [8] max / sum
+  pdl_launch_dependents();
+  pdl_wait();
+  const int b = blockIdx.y, h = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int pos = p.seq_lens[b];
+  if (pos < 0 || pos >= p.max_blocks * p.block_size) return;
+  float* qs = sm;
+  float* po = sm + p.lat_w;
+  float* ml = po + 4 * p.kv_rank;
+  for (int d = threadIdx.x; d < p.lat_w; d += 128) qs[d] = to_f(q_lat[((size_t)b * p.heads + h) * p.lat_w + d]);
+  __syncthreads();
+  const int first = p.window > 0 ? max(0, pos - p.window + 1) : 0;
+  const int* bt = p.block_table + (size_t)b * p.max_blocks;
+  float m = -INFINITY, l = 0.f, acc[LD_MAX_REG];
+#pragma unroll
+  for (int i = 0; i < LD_MAX_REG; ++i) acc[i] = 0.f;
+  for (int j = first + warp; j <= pos; j += 4) {
+    const T* row = cache + ((size_t)bt[j / p.block_size] * p.block_size + j % p.block_size) * p.lat_w;
+    float c[LD_MAX_REG], s = 0.f;
+#pragma unroll
+    for (int i = 0; i < LD_MAX_REG; ++i) {
+      const int d = lane + 32 * i;
+      c[i] = d < p.lat_w ? to_f(row[d]) : 0.f;
+      if (d < p.lat_w) s += c[i] * qs[d];
+    }
+    s = warp_sum(s) * p.scale;
+    const float mn = fmaxf(m, s), corr = m == -INFINITY ? 0.f : expf(m - mn), w = expf(s - mn);
+    l = l * corr + w;
+    m = mn;
+#pragma unroll
+    for (int i = 0; i < LD_MAX_REG; ++i) acc[i] = acc[i] * corr + w * c[i];
+  }
+#pragma unroll
+  for (int i = 0; i < LD_MAX_REG; ++i) {
+    const int d = lane + 32 * i;
+    if (d < p.kv_rank) po[(size_t)warp * p.kv_rank + d] = acc[i];
+  }
+  if (lane == 0) { ml[warp] = m; ml[4 + warp] = l; }
+  __syncthreads();
+  const float sk = p.sink[h];
+  float mt = sk;
+  for (int w = 0; w < 4; ++w) mt = fmaxf(mt, ml[w]);
+  float den = expf(sk - mt), f[4];
+  for (int w = 0; w < 4; ++w) {
+    f[w] = ml[w] == -INFINITY ? 0.f : expf(ml[w] - mt);
+    den += f[w] * ml[4 + w];
+  }
+  for (int d = threadIdx.x; d < p.kv_rank; d += 128) {
+    float v = 0.f;
+    for (int w = 0; w < 4; ++w) v += f[w] * po[(size_t)w * p.kv_rank + d];
+    o_lat[((size_t)b * p.heads + h) * p.kv_rank + d] = from_f<T>(v / den);
+  }
+}
+
+// out[b, h, e] = gate[b, h] * sum_r uv[h, e, r] o_lat[b, h, r]
+template <typename T>
+__global__ void __launch_bounds__(128)
+latent_expand_kernel(const T* __restrict__ o_lat, const T* __restrict__ uv, const float* __restrict__ gate,
+                     T* __restrict__ out, int heads, int vdim, int kv_rank, const int* __restrict__ positions) {
+  extern __shared__ float sm[];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int h = blockIdx.x, b = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const bool live = positions[b] >= 0;
+  for (int r = threadIdx.x; r < kv_rank; r += 128) sm[r] = live ? to_f(o_lat[((size_t)b * heads + h) * kv_rank + r]) : 0.f;
+  __syncthreads();
+  const float g = gate[(size_t)b * heads + h];
+  for (int e = warp; e < vdim; e += 4) {
+    const T* w = uv + ((size_t)h * vdim + e) * kv_rank;
+    float v = 0.f;
+    for (int r = lane; r < kv_rank; r += 32) v += sm[r] * to_f(w[r]);
+    v = warp_sum(v);
+    if (lane == 0) out[((size_t)b * heads + h) * vdim + e] = from_f<T>(v * g);
+  }
+}
+
+// ------------------------------------------------------------------------------------------------------------
+// mLSTM.  State of a slot and head: S [dim, vdim], n [dim], m, all fp32.  n and m are kept twice, indexed by the parity
+// of the number of tokens consumed, so that the blocks that share a head can all read the old values.
+// ------------------------------------------------------------------------------------------------------------
+__device__ __forceinline__ void mlstm_log_gates(float zi, float zf, float cap, float& ig, float& fg) {
+  ig = cap * tanhf(zi / cap);
+  fg = log_sigmoid_f(cap * tanhf(zf / cap));
+}
+
+// z [T, 2 heads] -> log input gates and log forget gates, both [T, heads]
+__global__ void __launch_bounds__(256)
+mlstm_gates_kernel(const float* __restrict__ z, const float* __restrict__ bias, float cap, int heads, long long n,
+                   float* __restrict__ ig, float* __restrict__ fg) {
+  for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x) {
+    const long long t = i / heads;
+    const int h = (int)(i % heads);
+    mlstm_log_gates(z[t * 2 * heads + h] + bias[h], z[t * 2 * heads + heads + h] + bias[heads + h], cap, ig[i], fg[i]);
+  }
+}
+
+struct MlstmState {
+  float* S;   // [slots, heads, dim, vdim]
+  float* n;   // [2, slots, heads, dim]
+  float* m;   // [2, slots, heads]
+  int slots;
+};
+
+// Prompts token by token: grid (sequence, head, 32-column tile of vdim), 256 threads.  Every size and dtype.
+template <typename T>
+__global__ void __launch_bounds__(256)
+mlstm_prompt_kernel(const T* __restrict__ qkv, long long ld, int k_off, int v_off, const float* __restrict__ ig,
+                    const float* __restrict__ fg, const int* __restrict__ cu, const int* __restrict__ seq_slot, MlstmState st,
+                    int heads, int dim, int vdim, float qscale, float* __restrict__ out) {
+  extern __shared__ float sm[];
+  __shared__ float red[64];
+  float* S = sm;               // [dim][32]
+  float* n = S + (size_t)dim * 32;
+  float* qs = n + dim;
+  float* ks = qs + dim;
+  float* part = ks + dim;      // [8][32]
+  const int seq = blockIdx.x, h = blockIdx.y, e0 = blockIdx.z * 32, tid = threadIdx.x;
+  const int ec = tid & 31, g = tid >> 5, e = e0 + ec;
+  for (int i = tid; i < dim * 32; i += 256) S[i] = 0.f;
+  for (int i = tid; i < dim; i += 256) n[i] = 0.f;
+  float m = 0.f;
+  const int t0 = cu[seq], t1 = cu[seq + 1];
+  for (int t = t0; t < t1; ++t) {
+    __syncthreads();
+    const T* row = qkv + (size_t)t * ld;
+    for (int d = tid; d < dim; d += 256) {
+      qs[d] = to_f(row[(size_t)h * dim + d]) * qscale;
+      ks[d] = to_f(row[k_off + (size_t)h * dim + d]);
+    }
+    const float li = ig[(size_t)t * heads + h], lf = fg[(size_t)t * heads + h];
+    const float mn = fmaxf(lf + m, li), keep = expf(lf + m - mn), wr = expf(li - mn);
+    m = mn;
+    const float v = e < vdim ? to_f(row[v_off + (size_t)h * vdim + e]) : 0.f;
+    __syncthreads();
+    float nq = 0.f;
+    for (int d = tid; d < dim; d += 256) {
+      const float nn = keep * n[d] + wr * ks[d];
+      n[d] = nn;
+      nq += nn * qs[d];
+    }
+    float acc = 0.f;
+    for (int d = g; d < dim; d += 8) {
+      const float s = keep * S[d * 32 + ec] + wr * ks[d] * v;
+      S[d * 32 + ec] = s;
+      acc += s * qs[d];
+    }
+    part[g * 32 + ec] = acc;
+    nq = block_sum2(nq, 0.f, red).x;
+    if (tid < 32 && e < vdim) {
+      float o = 0.f;
+#pragma unroll
+      for (int w = 0; w < 8; ++w) o += part[w * 32 + tid];
+      out[((size_t)t * heads + h) * vdim + e] = o / (fmaxf(fabsf(nq), expf(-m)) + 1e-6f);
+    }
+  }
+  __syncthreads();
+  if (seq_slot == nullptr) return;
+  const int slot = seq_slot[seq];
+  if (slot < 0 || slot >= st.slots) return;
+  const int par = (t1 - t0) & 1;
+  for (int i = tid; i < dim * 32; i += 256) {
+    const int d = i >> 5, c = e0 + (i & 31);
+    if (c < vdim) st.S[(((size_t)slot * heads + h) * dim + d) * vdim + c] = S[i];
+  }
+  if (blockIdx.z == 0) {
+    for (int d = tid; d < dim; d += 256) st.n[(((size_t)par * st.slots + slot) * heads + h) * dim + d] = n[d];
+    if (tid == 0) st.m[((size_t)par * st.slots + slot) * heads + h] = m;
+  }
+}
+
+// One token per slot: grid (head, slot, 16 * VEC-column tile of vdim), 256 threads = 16 column groups x 16 row groups.
+// acc [rows, ld] fp32: q | k | v | output gate | input gate | forget gate.  It is read by several blocks, so the
+// output kernel clears it.
+template <int VEC>
+__global__ void __launch_bounds__(256)
+mlstm_step_kernel(const float* __restrict__ acc, long long ld, const float* __restrict__ gate_bias, float cap,
+                  const int* __restrict__ seq_lens, MlstmState st, int heads, int dim, int vdim, float qscale,
+                  float* __restrict__ out) {
+  extern __shared__ float sm[];  // q [dim], k [dim], partial sums [16][16 VEC]
+  __shared__ float red[64];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int h = blockIdx.x, b = blockIdx.y, tid = threadIdx.x, cg = tid & 15, rg = tid >> 4;
+  const int pos = seq_lens[b];
+  if (pos < 0) return;
+  float* qs = sm;
+  float* ks = sm + dim;
+  float* part = ks + dim;
+  const float* row = acc + (size_t)b * ld;
+  const int qd = heads * dim, vd = heads * vdim;
+  const int par = pos & 1;
+  const size_t bh = (size_t)b * heads + h;
+  const float* n_old = st.n + ((size_t)par * st.slots * heads + bh) * dim;
+  float* n_new = st.n + ((size_t)(par ^ 1) * st.slots * heads + bh) * dim;
+  const float m_old = st.m[(size_t)par * st.slots * heads + bh];
+  float li, lf;
+  const int gr = 2 * qd + 2 * vd;
+  mlstm_log_gates(row[gr + h] + gate_bias[h], row[gr + heads + h] + gate_bias[heads + h], cap, li, lf);
+  const float m = fmaxf(lf + m_old, li), keep = expf(lf + m_old - m), wr = expf(li - m);
+  float nq = 0.f;
+  for (int d = tid; d < dim; d += 256) {
+    const float q = row[h * dim + d] * qscale, k = row[qd + h * dim + d];
+    qs[d] = q;
+    ks[d] = k * wr;
+    const float nn = keep * n_old[d] + wr * k;
+    if (blockIdx.z == 0) n_new[d] = nn;
+    nq += nn * q;
+  }
+  if (blockIdx.z == 0 && tid == 0) st.m[(size_t)(par ^ 1) * st.slots * heads + bh] = m;
+  nq = block_sum2(nq, 0.f, red).x;  // also orders the shared q and k
+  const int e = blockIdx.z * 16 * VEC + cg * VEC;
+  float o[VEC];
+#pragma unroll
+  for (int i = 0; i < VEC; ++i) o[i] = 0.f;
+  if (e < vdim) {
+    float v[VEC];
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) v[i] = row[2 * qd + h * vdim + e + i];
+    float* S = st.S + bh * dim * vdim + e;
+#pragma unroll 4
+    for (int d = rg; d < dim; d += 16) {
+      float s[VEC];
+      if (VEC == 4) {
+        const float4 t = *reinterpret_cast<const float4*>(S + (size_t)d * vdim);
+        s[0] = t.x; s[1 % VEC] = t.y; s[2 % VEC] = t.z; s[3 % VEC] = t.w;
+      } else {
+        s[0] = S[(size_t)d * vdim];
+      }
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) {
+        s[i] = keep * s[i] + ks[d] * v[i];
+        o[i] += s[i] * qs[d];
+      }
+      if (VEC == 4)
+        *reinterpret_cast<float4*>(S + (size_t)d * vdim) = make_float4(s[0], s[1 % VEC], s[2 % VEC], s[3 % VEC]);
+      else
+        S[(size_t)d * vdim] = s[0];
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < VEC; ++i) part[rg * 16 * VEC + cg * VEC + i] = o[i];
+  __syncthreads();
+  const float inv = 1.f / (fmaxf(fabsf(nq), expf(-m)) + 1e-6f);
+  for (int c = tid; c < 16 * VEC; c += 256) {
+    const int ee = blockIdx.z * 16 * VEC + c;
+    if (ee < vdim) {
+      float s = 0.f;
+#pragma unroll
+      for (int w = 0; w < 16; ++w) s += part[w * 16 * VEC + c];
+      out[bh * vdim + ee] = s * inv;
+    }
+  }
+}
+
+// y = unit_rms(o per head) * norm * sigmoid(g).  G: dtype of the gate logits (g_ld elements between rows).  With
+// `clear_row` the block also zeroes its share of the fp32 sums the step kernel has read.
+template <typename T, typename G>
+__global__ void __launch_bounds__(128)
+mlstm_out_kernel(const float* __restrict__ o, const G* __restrict__ gl, long long g_ld, const float* __restrict__ norm,
+                 float eps, int heads, int vdim, T* __restrict__ y, float* __restrict__ clear_row, long long clear_ld,
+                 int clear_n) {
+  __shared__ float red[64];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int h = blockIdx.x;
+  const size_t row = blockIdx.y, base = (row * heads + h) * vdim;
+  float ss = 0.f;
+  for (int e = threadIdx.x; e < vdim; e += 128) ss += o[base + e] * o[base + e];
+  const float r = 1.f / sqrtf(block_sum2(ss, 0.f, red).x / (float)vdim + eps);
+  for (int e = threadIdx.x; e < vdim; e += 128)
+    y[base + e] = from_f<T>(o[base + e] * r * norm[h * vdim + e] * sigmoid_f(to_f(gl[row * g_ld + (size_t)h * vdim + e])));
+  if (clear_row != nullptr) {
+    // every head's gate logits belong to this block alone; the rest of the row (q, k, v, input and forget gates) has
+    // been consumed by the step kernel.  clear_n = elements before / after the gates, dealt over the heads' blocks
+    float* c = clear_row + row * clear_ld;
+    __syncthreads();
+    const int g0 = clear_n, vd = heads * vdim;
+    for (int i = h * 128 + threadIdx.x; i < g0; i += heads * 128) c[i] = 0.f;
+    for (int e = threadIdx.x; e < vdim; e += 128) c[g0 + h * vdim + e] = 0.f;
+    for (int i = h * 128 + threadIdx.x; i < 2 * heads; i += heads * 128) c[g0 + vd + i] = 0.f;
+  }
+}
+
+}  // namespace trlb
+
+using namespace trlb;
+
+namespace {
+
+int grid_for(long long work, int per_block) {
+  long long g = (work + per_block - 1) / per_block;
+  const long long cap = (long long)trlb_host::sm_count() * 16;
+  return (int)(g < 1 ? 1 : (g > cap ? cap : g));
+}
+
+// dynamic shared memory above the default limit has to be announced once per kernel
+template <typename K>
+bool allow_smem(K kern, size_t bytes) {
+  if (bytes <= 48 * 1024) return true;
+  if (bytes > 227 * 1024) return false;
+  return cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes) == cudaSuccess;
+}
+
+using bf16 = __nv_bfloat16;
+
+}  // namespace
+
+#define PDL trlb_host::pdl_enabled()
+
+TRLB_API int trlb_embed_scaled(const long long* ids, const void* emb, float* x, int T, int H, int V, float scale, int is_bf16,
+                               cudaStream_t st) {
+  if (T <= 0) return 0;
+  if (is_bf16) return (int)trlb_host::launch_kernel(embed_scaled_kernel<bf16>, dim3(T), dim3(256), 0, st, PDL, ids, (const bf16*)emb, x, H, V, scale);
+  return (int)trlb_host::launch_kernel(embed_scaled_kernel<float>, dim3(T), dim3(256), 0, st, PDL, ids, (const float*)emb, x, H, V, scale);
+}
+
+TRLB_API int trlb_dynamic_tanh(float* x, float* delta, const float* alpha, const float* w, const float* b, void* out, int T,
+                               int H, int clear, int is_bf16, cudaStream_t st) {
+  if (T <= 0) return 0;
+  const bool v4 = (H % 4) == 0;
+  const long long n = (long long)T * H / (v4 ? 4 : 1);
+  const dim3 grid(grid_for(n, 256)), blk(256);
+#define GO(TT, VV) (int)trlb_host::launch_kernel(dynamic_tanh_kernel<TT, VV>, grid, blk, 0, st, PDL, x, delta, alpha, w, b, (TT*)out, n, H, clear)
+  if (is_bf16) return v4 ? GO(bf16, 4) : GO(bf16, 1);
+  return v4 ? GO(float, 4) : GO(float, 1);
+#undef GO
+}
+
+TRLB_API int trlb_gelu_erf(const void* z, void* out, long long n, int is_bf16, cudaStream_t st) {
+  if (n <= 0) return 0;
+  if (is_bf16) gelu_erf_kernel<bf16><<<grid_for(n, 256), 256, 0, st>>>((const bf16*)z, (bf16*)out, n);
+  else gelu_erf_kernel<float><<<grid_for(n, 256), 256, 0, st>>>((const float*)z, (float*)out, n);
+  return (int)cudaGetLastError();
+}
+
+TRLB_API int trlb_latent_prep(float* acc, long long ld, int rows, int q_rank, int kv_rank, int rot, int heads, int clear,
+                              const float* q_norm, const float* kv_norm, float eps, const int* positions,
+                              const int* tok_slot, const float* table, int table_len, void* cq, void* lat, float* gate,
+                              int kr_off, int lat_w, void* cache, const int* block_table, int max_blocks, int block_size,
+                              int is_bf16, cudaStream_t st) {
+  if (rows <= 0) return 0;
+  if ((rot & 1) || kr_off < kv_rank || lat_w < kr_off + rot || (cache != nullptr && block_table == nullptr)) return -200;
+  LatentPrep p = {acc, ld, q_rank, kv_rank, rot, heads, clear, q_norm, kv_norm, eps, positions, tok_slot,
+                  (const float2*)table, table_len, gate, kr_off, lat_w, cache ? block_table : nullptr, max_blocks, block_size};
+  if (is_bf16)
+    return (int)trlb_host::launch_kernel(latent_prep_kernel<bf16>, dim3(rows), dim3(256), 0, st, PDL, p, (bf16*)cq, (bf16*)lat, (bf16*)cache);
+  return (int)trlb_host::launch_kernel(latent_prep_kernel<float>, dim3(rows), dim3(256), 0, st, PDL, p, (float*)cq, (float*)lat, (float*)cache);
+}
+
+TRLB_API int trlb_rotate_q(void* q, int rows, int heads, int dim, int rot, const int* positions, const float* table,
+                           int table_len, int is_bf16, cudaStream_t st) {
+  const long long n = (long long)rows * heads * (rot / 2);
+  if (n <= 0) return 0;
+  if (is_bf16) rotate_q_kernel<bf16><<<grid_for(n, 256), 256, 0, st>>>((bf16*)q, heads, dim, rot, positions, (const float2*)table, table_len, n);
+  else rotate_q_kernel<float><<<grid_for(n, 256), 256, 0, st>>>((float*)q, heads, dim, rot, positions, (const float2*)table, table_len, n);
+  return (int)cudaGetLastError();
+}
+
+// window <= 0: unlimited
+TRLB_API int trlb_latent_prompt(const void* q, const void* kv, long long kv_ld, const void* lat, int T, int heads, int dim,
+                                int rot, int vdim, int kr_off, int lat_w, int window, float scale, const int* positions,
+                                const float* sink, const float* gate, void* out, int is_bf16, cudaStream_t st) {
+  if (T <= 0) return 0;
+  LatentPrompt p = {T, heads, dim, rot, vdim, kr_off, lat_w, window, kv_ld, scale, positions, sink, gate};
+  const long long items = (long long)T * heads;
+  const int grid = (int)((items + 3) / 4);
+  const size_t smem = (size_t)4 * (dim + rot + vdim) * 4;
+  if (is_bf16) {
+    if (!allow_smem(latent_prompt_kernel<bf16>, smem)) return -201;
+    latent_prompt_kernel<bf16><<<grid, 128, smem, st>>>(p, (const bf16*)q, (const bf16*)kv, (const bf16*)lat, (bf16*)out);
+  } else {
+    if (!allow_smem(latent_prompt_kernel<float>, smem)) return -201;
+    latent_prompt_kernel<float><<<grid, 128, smem, st>>>(p, (const float*)q, (const float*)kv, (const float*)lat, (float*)out);
+  }
+  return (int)cudaGetLastError();
+}
+
+TRLB_API int trlb_latent_absorb(float* qacc, long long ld, const void* uk, void* q_lat, int B, int heads, int dim, int rot,
+                                int kv_rank, int kr_off, int lat_w, const int* positions, const float* table,
+                                int table_len, int clear, int is_bf16, cudaStream_t st) {
+  if (B <= 0) return 0;
+  const size_t smem = (size_t)(dim + rot) * 4;
+  const dim3 grid(heads, B), blk(128);
+  if (smem > 48 * 1024) return -202;
+  if (is_bf16)
+    return (int)trlb_host::launch_kernel(latent_absorb_kernel<bf16>, grid, blk, smem, st, PDL, qacc, ld, (const bf16*)uk, (bf16*)q_lat,
+                                         heads, dim, rot, kv_rank, kr_off, lat_w, positions, (const float2*)table, table_len, clear);
+  return (int)trlb_host::launch_kernel(latent_absorb_kernel<float>, grid, blk, smem, st, PDL, qacc, ld, (const float*)uk, (float*)q_lat,
+                                       heads, dim, rot, kv_rank, kr_off, lat_w, positions, (const float2*)table, table_len, clear);
+}
+
+TRLB_API int trlb_latent_decode(const void* q_lat, const void* cache, void* o_lat, int B, int heads, int kv_rank, int lat_w,
+                                int window, float scale, const int* seq_lens, const int* block_table, int max_blocks,
+                                int block_size, const float* sink, int is_bf16, cudaStream_t st) {
+  if (B <= 0) return 0;
+  if (lat_w > 32 * LD_MAX_REG) return -203;
+  LatentDecode p = {B, heads, kv_rank, lat_w, window, max_blocks, block_size, 1, scale, seq_lens, block_table, sink};
+  const size_t smem = (size_t)(lat_w + 4 * kv_rank + 8) * 4;
+  const dim3 grid(heads, B), blk(128);
+  if (smem > 48 * 1024) return -203;
+  if (is_bf16)
+    return (int)trlb_host::launch_kernel(latent_decode_kernel<bf16>, grid, blk, smem, st, PDL, p, (const bf16*)q_lat, (const bf16*)cache, (bf16*)o_lat);
+  return (int)trlb_host::launch_kernel(latent_decode_kernel<float>, grid, blk, smem, st, PDL, p, (const float*)q_lat, (const float*)cache, (float*)o_lat);
+}
+
+TRLB_API int trlb_latent_expand(const void* o_lat, const void* uv, const float* gate, void* out, int B, int heads, int vdim,
+                                int kv_rank, const int* positions, int is_bf16, cudaStream_t st) {
+  if (B <= 0) return 0;
+  const size_t smem = (size_t)kv_rank * 4;
+  const dim3 grid(heads, B), blk(128);
+  if (smem > 48 * 1024) return -204;
+  if (is_bf16)
+    return (int)trlb_host::launch_kernel(latent_expand_kernel<bf16>, grid, blk, smem, st, PDL, (const bf16*)o_lat, (const bf16*)uv, gate, (bf16*)out, heads, vdim, kv_rank, positions);
+  return (int)trlb_host::launch_kernel(latent_expand_kernel<float>, grid, blk, smem, st, PDL, (const float*)o_lat, (const float*)uv, gate, (float*)out, heads, vdim, kv_rank, positions);
+}
+
+TRLB_API int trlb_mlstm_gates(const float* z, const float* bias, float cap, int T, int heads, float* ig, float* fg, cudaStream_t st) {
+  const long long n = (long long)T * heads;
+  if (n <= 0) return 0;
+  mlstm_gates_kernel<<<grid_for(n, 256), 256, 0, st>>>(z, bias, cap, heads, n, ig, fg);
+  return (int)cudaGetLastError();
+}
+
+// qkv [T, ld]: q at 0, k at k_off, v at v_off (elements).  Sequences by cu [n_seq + 1]; seq_slot null: no state is kept.
+TRLB_API int trlb_mlstm_prompt(const void* qkv, long long ld, int k_off, int v_off, const float* ig, const float* fg,
+                               const int* cu, int n_seq, const int* seq_slot, float* S, float* n, float* m, int slots,
+                               int heads, int dim, int vdim, float qscale, float* out, int is_bf16, cudaStream_t st) {
+  if (n_seq <= 0) return 0;
+  const size_t smem = (size_t)(dim * 32 + 3 * dim + 256) * 4;
+  const dim3 grid(n_seq, heads, (vdim + 31) / 32);
+  MlstmState s = {S, n, m, slots};
+  if (is_bf16) {
+    if (!allow_smem(mlstm_prompt_kernel<bf16>, smem)) return -205;
+    mlstm_prompt_kernel<bf16><<<grid, 256, smem, st>>>((const bf16*)qkv, ld, k_off, v_off, ig, fg, cu, seq_slot, s, heads, dim, vdim, qscale, out);
+  } else {
+    if (!allow_smem(mlstm_prompt_kernel<float>, smem)) return -205;
+    mlstm_prompt_kernel<float><<<grid, 256, smem, st>>>((const float*)qkv, ld, k_off, v_off, ig, fg, cu, seq_slot, s, heads, dim, vdim, qscale, out);
+  }
+  return (int)cudaGetLastError();
+}
+
+TRLB_API int trlb_mlstm_step(const float* acc, long long ld, const float* gate_bias, float cap, const int* seq_lens, float* S,
+                             float* n, float* m, int slots, int B, int heads, int dim, int vdim, float qscale, float* out,
+                             cudaStream_t st) {
+  if (B <= 0) return 0;
+  if (B > slots) return -206;
+  MlstmState s = {S, n, m, slots};
+  const bool v4 = (vdim % 4) == 0;
+  const int tile = v4 ? 64 : 16;
+  const dim3 grid(heads, B, (vdim + tile - 1) / tile), blk(256);
+  const size_t smem = (size_t)(2 * dim + 16 * tile) * 4;
+  if (smem > 48 * 1024) return -206;
+  if (v4) return (int)trlb_host::launch_kernel(mlstm_step_kernel<4>, grid, blk, smem, st, PDL, acc, ld, gate_bias, cap, seq_lens, s, heads, dim, vdim, qscale, out);
+  return (int)trlb_host::launch_kernel(mlstm_step_kernel<1>, grid, blk, smem, st, PDL, acc, ld, gate_bias, cap, seq_lens, s, heads, dim, vdim, qscale, out);
+}
+
+// g_bf16 / y_bf16: dtypes of the gate logits and of the output (bf16 else fp32).  clear_row (fp32 sums, gates at clear_n) may be null.
+TRLB_API int trlb_mlstm_out(const float* o, const void* gl, long long g_ld, int g_bf16, const float* norm, float eps, int rows,
+                            int heads, int vdim, void* y, int y_bf16, float* clear_row, long long clear_ld, int clear_n,
+                            cudaStream_t st) {
+  if (rows <= 0) return 0;
+  const dim3 blk(128);
+  // rows on y: prompts can be longer than 65535 tokens, so they are launched in slices
+  for (int r0 = 0; r0 < rows; r0 += 32768) {
+    const int nr = rows - r0 < 32768 ? rows - r0 : 32768;
+    const dim3 grid(heads, nr);
+    const size_t off = (size_t)r0 * heads * vdim;
+    int rc;
+#define GO(TT, GG) (int)trlb_host::launch_kernel(mlstm_out_kernel<TT, GG>, grid, blk, 0, st, PDL, o + off, (const GG*)gl + (size_t)r0 * g_ld, g_ld, \
+                                                norm, eps, heads, vdim, (TT*)y + off, clear_row ? clear_row + (size_t)r0 * clear_ld : nullptr, clear_ld, clear_n)
+    if (y_bf16) rc = g_bf16 ? GO(bf16, bf16) : GO(bf16, float);
+    else rc = g_bf16 ? GO(float, bf16) : GO(float, float);
+#undef GO
+    if (rc) return rc;
+  }
+  return 0;
+}

@@ -1,0 +1,32 @@
+// Device helpers shared by the kernels of the layered decoders (mixers.cu, latent_attn_*.cu, mlstm_chunk_*.cu).
+#pragma once
+#include "common.cuh"
+
+namespace trlb {
+
+__device__ __forceinline__ float to_f(float v) { return v; }
+__device__ __forceinline__ float to_f(__nv_bfloat16 v) { return __bfloat162float(v); }
+template <typename T>
+__device__ __forceinline__ T from_f(float v);
+template <>
+__device__ __forceinline__ float from_f<float>(float v) { return v; }
+template <>
+__device__ __forceinline__ __nv_bfloat16 from_f<__nv_bfloat16>(float v) { return __float2bfloat16(v); }
+
+__device__ __forceinline__ float sigmoid_f(float z) { return 1.f / (1.f + expf(-z)); }
+__device__ __forceinline__ float log_sigmoid_f(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); }
+
+// Sums `a` and `b` over the block (at most 32 warps); `red` is 64 floats of shared memory.  All threads get the result.
+__device__ __forceinline__ float2 block_sum2(float a, float b, float* red) {
+  const int lane = threadIdx.x & 31, wid = threadIdx.x >> 5, nw = blockDim.x >> 5;
+  a = warp_sum(a);
+  b = warp_sum(b);
+  __syncthreads();
+  if (lane == 0) { red[wid] = a; red[32 + wid] = b; }
+  __syncthreads();
+  a = b = 0.f;
+  for (int w = 0; w < nw; ++w) { a += red[w]; b += red[32 + w]; }
+  return make_float2(a, b);
+}
+
+}  // namespace trlb

@@ -75,13 +75,13 @@ def sample_completions(model, prompts, max_new_tokens, temperature=1.0, top_p=1.
     sp = SamplingParams(n=1, max_tokens=max_new_tokens, temperature=temperature, top_p=top_p, top_k=top_k,
                         eos_token_id=eos_token_id, seed=seed)
     if model.device.type == "cuda":
-        from ..rollout.engine import RolloutEngine
+        from ..rollout.engine import make_engine
 
         cache = engine_cache if engine_cache is not None else _GENERATORS
         need = max(len(p) for p in prompts) + max_new_tokens + 8
         eng = cache.get(("engine", id(model)))
         if eng is None or eng.max_len < need or eng.max_seqs < len(prompts):
-            eng = RolloutEngine(model, max_num_seqs=max(len(prompts), 8), max_model_len=(need + 63) // 64 * 64)
+            eng = make_engine(model, max_num_seqs=max(len(prompts), 8), max_model_len=(need + 63) // 64 * 64)
             cache[("engine", id(model))] = eng
         outs = eng.generate(prompts, sp)
     else:

@@ -36,9 +36,9 @@ class RolloutGeneration:
             if D.world_size() % tensor_parallel_size != 0:
                 raise ValueError(f"tensor_parallel_size ({tensor_parallel_size}) must divide world size ({D.world_size()})")
             if model.device.type == "cuda":
-                from ..rollout.engine import RolloutEngine
+                from ..rollout.engine import make_engine
 
-                self.engine = RolloutEngine(model, max_num_seqs, max_model_len)
+                self.engine = make_engine(model, max_num_seqs, max_model_len)
             else:
                 from ..rollout.engine import EagerGenerator
 

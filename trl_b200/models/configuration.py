@@ -159,6 +159,10 @@ class ModelArch:
     def from_hf_dict(cls, d: dict[str, Any]) -> "ModelArch":
         if hasattr(d, "to_dict"):
             d = d.to_dict()
+        if "architecture" in d and "layers" in d:  # a design that lists its layers
+            from .layered import LayeredArch
+
+            return LayeredArch.from_dict(d)
         mt = d.get("model_type", "llama")
         if mt not in _FAMILY_ARCH:
             raise ValueError(
@@ -258,10 +262,18 @@ PRESETS: dict[str, dict] = {
                           num_hidden_layers=48, num_attention_heads=32, num_key_value_heads=4, head_dim=128,
                           num_experts=128, num_experts_per_tok=8, moe_intermediate_size=768,
                           rope_theta=1e6, rms_norm_eps=1e-6),
+    "tiny-zorelorn": dict(
+        architecture="Zorelorn", vocab=1024, width=64, norm=dict(eps=1e-6), embedding=dict(scale=8.0),
+        layers=[dict(type="mlstm", mixer=dict(heads=2, dim=16, vdim=32, gate_cap=10.0), mlp=None),
+                dict(type="latent_attention", mlp=dict(kind="dense", ff=192),
+                     mixer=dict(heads=4, dim=16, rot_dim=8, vdim=16, q_rank=24, kv_rank=32, scale=0.2, mask=dict(size=20),
+                                rot=dict(base=1e4, dims=8, scaling=dict(factor=4.0, original=256, fast=16.0, slow=1.0))))]),
 }
 
 
 def preset(name: str, **overrides) -> ModelArch:
     cfg = dict(PRESETS[name])
     cfg.update(overrides)
+    if "architecture" in cfg:
+        return ModelArch.from_hf_dict(cfg)
     return ModelArch(**cfg)

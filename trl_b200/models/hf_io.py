@@ -33,6 +33,8 @@ def to_hf_state_dict(model, include_lora: bool = False, before_layer=None, copy_
     makes a copy of every layer's tensors right after: the streamed full-shard engine holds one layer at a time.  With
     ``before_layer`` set and ``copy_to`` None the layers are visited (the gathers are collective) but not kept."""
     c = model.config
+    if getattr(model, "is_layered", False):
+        return {k: v.detach() for k, v in model.named_tensors().items()}
     sd = {"model.embed_tokens.weight": model.embed_tokens.detach()}
     for i, l in enumerate(model.layers):
         p = f"model.layers.{i}."
@@ -94,6 +96,8 @@ def load_hf_state_dict(model, sd: dict[str, torch.Tensor], strict: bool = True, 
     """Copy tensors named the HF way into the fused native parameters.  ``after_layer(i)`` runs once layer i is
     complete (the streamed full-shard engine re-slices its shard there, before the slot is reused)."""
     c = model.config
+    if getattr(model, "is_layered", False):
+        return model.load_named_tensors(sd, strict)
     used = set()
 
     def take(name, required=True):
@@ -226,11 +230,19 @@ def save_model(model, path: str, state_dict=None):
         json.dump(gen, f, indent=2)
 
 
+def build_model(config: ModelArch, dtype=torch.float32, device=None, init: bool = True):
+    """Decoder of the class that ``config`` describes."""
+    if getattr(config, "design", ""):
+        from .layered import LayeredLM as cls
+    else:
+        from .decoder import CausalLM as cls
+
+    return cls(config, dtype=dtype, device=device, init=init)
+
+
 def load_model(path_or_name, dtype=None, device=None, num_labels: int | None = None, config: ModelArch | None = None,
                seed: int | None = None, **unused):
     """Load from a local HF directory, or random-init a named preset (``"preset:qwen2.5-7b"``)."""
-    from .decoder import CausalLM
-
     dtype = resolve_dtype(dtype) or torch.float32
     if isinstance(path_or_name, ModelArch):
         config, path_or_name = path_or_name, ""
@@ -262,7 +274,7 @@ def load_model(path_or_name, dtype=None, device=None, num_labels: int | None = N
         config.num_labels = num_labels
     if seed is not None:
         torch.manual_seed(seed)
-    model = CausalLM(config, dtype=dtype, device=device)
+    model = build_model(config, dtype=dtype, device=device)
     if is_dir:
         has_weights = any(re.match(r"(model.*\.safetensors.*|pytorch_model\.bin)$", f) for f in os.listdir(name))
         if has_weights:

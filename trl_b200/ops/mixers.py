@@ -1,0 +1,140 @@
+"""Mechanisms of the layered decoders (models/layered.py) on packed prompts.
+
+CUDA tensors run the kernels of ``csrc/mixers.cu`` and the tensor-core mixer kernels, in bf16 or fp32; CPU tensors run
+:mod:`trl_b200.oracle.mixers`.  On CUDA the kernels are inference only (prompts, log-probs, generation).
+
+A serving engine passes itself through ``ctx.kv``: ``latent_cache(li)`` and ``recurrent_state(li)`` say where layer
+``li`` leaves what decoding continues from."""
+from __future__ import annotations
+
+import contextlib
+import math
+
+import torch
+import torch.nn.functional as F
+
+from ..oracle import mixers as _ref
+
+
+def _k():
+    from . import cuda_mixers
+
+    return cuda_mixers
+
+
+class RotarySpec:
+    """Interleaved rotary positions with optional YaRN scaling.  ``table(n)``: fp32 [n, dims / 2, 2] (cos, sin), the
+    magnitude of the scaling folded in; angles are evaluated in fp64 before they are rounded."""
+
+    def __init__(self, dims: int, base: float, scaling: dict | None = None):
+        self.dims, self.base, self.scaling = dims, base, dict(scaling) if scaling else None
+        self._tables: dict = {}
+
+    def frequencies(self) -> torch.Tensor:
+        i = torch.arange(self.dims // 2, dtype=torch.float64)
+        f = torch.pow(torch.tensor(self.base, dtype=torch.float64), -2.0 * i / self.dims)
+        if self.scaling is None:
+            return f
+        s = self.scaling
+
+        def turns_to_dim(t):
+            return self.dims * math.log(s["original"] / (2.0 * math.pi * t)) / (2.0 * math.log(self.base))
+
+        lo = max(math.floor(turns_to_dim(s["fast"])), 0)
+        hi = min(math.ceil(turns_to_dim(s["slow"])), self.dims - 1)
+        ramp = ((i - lo) / max(hi - lo, 0.001)).clamp(0.0, 1.0)
+        return f / s["factor"] * ramp + f * (1.0 - ramp)
+
+    @property
+    def magnitude(self) -> float:
+        return 1.0 if self.scaling is None else 0.1 * math.log(self.scaling["factor"]) + 1.0
+
+    def table(self, n: int, device) -> torch.Tensor:
+        key = str(device)
+        t = self._tables.get(key)
+        if t is None or t.shape[0] < n:
+            size = max(256, 1 << (n - 1).bit_length())
+            ang = torch.arange(size, dtype=torch.float64, device=device)[:, None] * self.frequencies().to(device)
+            t = (torch.stack([ang.cos(), ang.sin()], -1) * self.magnitude).float().contiguous()
+            self._tables[key] = t
+        return t
+
+
+def check_can_run(w: torch.Tensor):
+    if w.is_cuda and torch.is_grad_enabled() and w.requires_grad:
+        raise NotImplementedError("the CUDA kernels of the layered decoders are inference only: run them under "
+                                  "torch.no_grad(), or train on CPU tensors")
+
+
+@contextlib.contextmanager
+def _ieee_fp32():
+    """fp32 matrix products in fp32 (no TF32), whatever the process default is."""
+    was = torch.backends.cuda.matmul.allow_tf32
+    torch.backends.cuda.matmul.allow_tf32 = False
+    try:
+        yield
+    finally:
+        torch.backends.cuda.matmul.allow_tf32 = was
+
+
+def linear(x, w):
+    """``x W^T`` in the dtype of the inputs."""
+    if x.is_cuda and x.dtype == torch.float32:
+        with _ieee_fp32():
+            return F.linear(x, w)
+    return F.linear(x, w.to(x.dtype))
+
+
+def linear_f32(x, w):
+    """``x W^T`` with the fp32 accumulators as the result."""
+    if x.is_cuda and x.dtype == torch.bfloat16:
+        return torch.mm(x, w.t(), out_dtype=torch.float32)
+    return linear(x, w)
+
+
+def embed_scaled(ids, emb, scale):
+    if emb.is_cuda:
+        return _k().embed_scaled(ids, emb, scale)
+    return F.embedding(ids, emb).float() * scale
+
+
+def dynamic_tanh(x, delta, alpha, w, b, out_dtype):
+    """(norm of ``x + delta`` in ``out_dtype``, ``x + delta``); on CUDA the sum is formed in place."""
+    if x.is_cuda:
+        return _k().dynamic_tanh(x, delta, alpha, w, b, out_dtype), x
+    x = x if delta is None else x + delta
+    return _ref.dynamic_tanh(x, alpha, w, b).to(out_dtype), x
+
+
+def gelu_linear(h, up):
+    z = linear(h, up)
+    return _k().gelu_erf(z) if z.is_cuda else F.gelu(z)
+
+
+def latent_attention(m, h, ctx, li):
+    if not h.is_cuda:
+        return _ref.latent_attention(m, h.float(), ctx.positions, ctx.cu_seqlens)
+    K = _k()
+    pos = ctx.positions if ctx.positions.dtype == torch.int32 else ctx.positions.to(torch.int32)
+    table = m.rope.table(ctx.max_seqlen, h.device)
+    kr, width = K.latent_row(m.kv_rank, m.rot_dim)
+    lat = torch.zeros(h.shape[0], width, dtype=h.dtype, device=h.device)
+    cache = ctx.kv.latent_cache(li) if ctx.kv is not None else {}
+    cq, gate = K.latent_prep(linear_f32(h, m.w_in), m, pos, table, lat=lat, **cache)
+    q = linear(cq, m.uq)
+    K.rotate_q(q, m, pos, table)
+    kv = linear(lat[:, : m.kv_rank], m.ukv)
+    return linear_f32(K.latent_prompt(q, kv, lat, m, pos, gate), m.o)
+
+
+def mlstm(m, h, ctx, li):
+    if not h.is_cuda:
+        return _ref.mlstm(m, h.float(), ctx.cu_seqlens)
+    K = _k()
+    y = linear(h, m.w_in[: m.gate_row])
+    ig, fg = K.mlstm_gates(linear_f32(h, m.w_in[m.gate_row:]), m.gate_bias, m.cap, m.heads)
+    where = ctx.kv.recurrent_state(li) if ctx.kv is not None else {}
+    o = K.mlstm_prompt(y, m, ig, fg, ctx.cu_seqlens, **where)
+    out = torch.empty(h.shape[0], m.heads * m.vdim, dtype=h.dtype, device=h.device)
+    K.mlstm_out(o, y[:, m.heads * (2 * m.dim + m.vdim):], m, out)
+    return linear_f32(out, m.o)

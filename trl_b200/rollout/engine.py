@@ -119,6 +119,8 @@ class _PrefillKV:
 
 
 class RolloutEngine:
+    stateful = False  # True: slots hold state that a decode step replaces (not only pages that it extends)
+
     def _decode_attention(self, li: int, scale: float):
         """q_buf x paged KV of layer ``li`` -> attn_buf (tcgen05 kernel when the cache layout allows it)."""
         from ..ops import cuda as K
@@ -139,41 +141,21 @@ class RolloutEngine:
         if self.vlm is not None:
             model = model.language_model
         cfg = model.config
-        if cfg.num_attention_heads % tp or cfg.num_key_value_heads % tp:
-            raise ValueError(f"tensor parallel size {tp} must divide the head counts")
         self.tp, self.tp_rank = tp, tp_rank
-        self.hq_local, self.hk_local = cfg.num_attention_heads // tp, cfg.num_key_value_heads // tp
         self.model, self.cfg = model, cfg
         self.dev = model.device
         if self.dev.type != "cuda":
             raise RuntimeError("RolloutEngine needs a CUDA device; use EagerGenerator on CPU")
-        if cfg.hidden_act != "silu" or cfg.norm_plus_one or cfg.embed_scale != 1.0 or cfg.head_dim not in (64, 128):
-            raise NotImplementedError("the decode kernels cover SwiGLU models with head_dim 64 or 128; use EagerGenerator "
-                                      f"for model_type={cfg.model_type!r}")
-        if cfg.sliding_window and max_model_len > cfg.sliding_window:
-            raise NotImplementedError(f"the paged decode attention attends over the whole context: sliding_window="
-                                      f"{cfg.sliding_window} < max_model_len={max_model_len}; use EagerGenerator")
+        block_size = self._check_model(max_model_len, block_size)
         from .._native import host_runtime
 
         rt = host_runtime()
         if rt is None:
             raise RuntimeError("libtrl_b200_host.so missing: run python -m trl_b200.csrc.build")
-        # head_dim 128 with at most 8 query heads per KV head: tensor-core decode attention, which wants 64-token
-        # pages and V transposed inside a page; anything else keeps 16-token pages and the CUDA-core kernel
-        tc_ok = cfg.head_dim == 128 and self.hq_local // self.hk_local <= 8
-        if not block_size:
-            block_size = 64 if tc_ok else 16
-        self.attn_tc = tc_ok and block_size == 64
-        self.attn_groups = int(os.environ.get("TRL_B200_DECODE_ATTN_GROUPS", "1"))  # 2: two softmax groups per CTA
         self.max_seqs, self.max_len, self.block_size = max_num_seqs, max_model_len, block_size
         self.max_blocks = (max_model_len + block_size - 1) // block_size
         self.num_blocks = num_blocks or max_num_seqs * self.max_blocks
         self.sched = rt.scheduler(max_num_seqs, self.num_blocks, block_size, self.max_blocks)
-        L, Hk, D = cfg.num_hidden_layers, self.hk_local, cfg.head_dim
-        dt = torch.bfloat16
-        self.k_cache = [torch.zeros(self.num_blocks, block_size, Hk, D, dtype=dt, device=self.dev) for _ in range(L)]
-        v_shape = (self.num_blocks, Hk, D, block_size) if self.attn_tc else (self.num_blocks, block_size, Hk, D)
-        self.v_cache = [torch.zeros(*v_shape, dtype=dt, device=self.dev) for _ in range(L)]
         i32 = dict(dtype=torch.int32, device=self.dev)
         self.block_table = torch.zeros(max_num_seqs, self.max_blocks, **i32)
         self.block_table_host = torch.zeros(max_num_seqs, self.max_blocks, dtype=torch.int32).pin_memory()
@@ -188,6 +170,44 @@ class RolloutEngine:
         self.tok = torch.zeros(max_num_seqs, **i32)
         self.logp = torch.zeros(max_num_seqs, dtype=torch.float32, device=self.dev)
         self.poll_every, self.use_graph = poll_every, use_cuda_graph
+        self._pdl = os.environ.get("TRL_B200_PDL", "1") == "1"
+        self._alloc_layers(kv_splits)
+        self.seen = None
+        self.out_tokens = self.out_logps = None
+        self._graph = None
+        self._graph_key = None
+        self.stats = {"decode_steps": 0, "prefill_tokens": 0, "generated_tokens": 0}
+
+    # ---- what depends on the kind of decoder (rollout/layered_engine.py overrides these) -----------------
+    def _check_model(self, max_model_len: int, block_size: int | None) -> int:
+        """Raises if the decode kernels do not cover the model; returns the page size of its cache."""
+        cfg = self.cfg
+        if cfg.num_attention_heads % self.tp or cfg.num_key_value_heads % self.tp:
+            raise ValueError(f"tensor parallel size {self.tp} must divide the head counts")
+        self.hq_local, self.hk_local = cfg.num_attention_heads // self.tp, cfg.num_key_value_heads // self.tp
+        if cfg.hidden_act != "silu" or cfg.norm_plus_one or cfg.embed_scale != 1.0 or cfg.head_dim not in (64, 128):
+            raise NotImplementedError("the decode kernels cover SwiGLU models with head_dim 64 or 128; use EagerGenerator "
+                                      f"for model_type={cfg.model_type!r}")
+        if cfg.sliding_window and max_model_len > cfg.sliding_window:
+            raise NotImplementedError(f"the paged decode attention attends over the whole context: sliding_window="
+                                      f"{cfg.sliding_window} < max_model_len={max_model_len}; use EagerGenerator")
+        # head_dim 128 with at most 8 query heads per KV head: tensor-core decode attention, which wants 64-token
+        # pages and V transposed inside a page; anything else keeps 16-token pages and the CUDA-core kernel
+        tc_ok = cfg.head_dim == 128 and self.hq_local // self.hk_local <= 8
+        if not block_size:
+            block_size = 64 if tc_ok else 16
+        self.attn_tc = tc_ok and block_size == 64
+        self.attn_groups = int(os.environ.get("TRL_B200_DECODE_ATTN_GROUPS", "1"))  # 2: two softmax groups per CTA
+        return block_size
+
+    def _alloc_layers(self, kv_splits: int):
+        """Caches and activation buffers of the decoder stack."""
+        cfg, tp, max_num_seqs, block_size = self.cfg, self.tp, self.max_seqs, self.block_size
+        L, Hk, D = cfg.num_hidden_layers, self.hk_local, cfg.head_dim
+        dt = torch.bfloat16
+        self.k_cache = [torch.zeros(self.num_blocks, block_size, Hk, D, dtype=dt, device=self.dev) for _ in range(L)]
+        v_shape = (self.num_blocks, Hk, D, block_size) if self.attn_tc else (self.num_blocks, block_size, Hk, D)
+        self.v_cache = [torch.zeros(*v_shape, dtype=dt, device=self.dev) for _ in range(L)]
         # enough CTAs for ~4 per SM: the kernel is latency-bound on KV loads, occupancy hides it
         self.kv_splits = kv_splits or max(1, min(8, -(-(4 * 148) // max(1, max_num_seqs * Hk))))
         if self.attn_tc and not kv_splits:  # persistent CTAs, one per SM: split only to give every SM an item
@@ -202,7 +222,6 @@ class RolloutEngine:
         self._own_gemm = (os.environ.get("TRL_B200_DECODE_GEMM", "own") != "cublas" and tp == 1 and max_num_seqs <= 128
                           and cfg.hidden_size <= 8192 and cfg.hidden_size % 8 == 0 and cfg.head_dim <= 128
                           and (cfg.is_moe or cfg.intermediate_size % 8 == 0))
-        self._pdl = os.environ.get("TRL_B200_PDL", "1") == "1"
         if self._own_gemm:  # fp32 accumulators; their consumers clear them after reading
             f32 = dict(dtype=torch.float32, device=self.dev)
             qkv_out = (self.hq_local + 2 * self.hk_local) * cfg.head_dim
@@ -216,11 +235,28 @@ class RolloutEngine:
             self._one_group = torch.tensor([0, max_num_seqs], dtype=torch.int32, device=self.dev)
             self._act_buf = torch.empty(max_num_seqs, cfg.intermediate_size, dtype=dt, device=self.dev)
         self.attn_buf = torch.empty(max_num_seqs, self.hq_local, D, dtype=dt, device=self.dev)
-        self.seen = None
-        self.out_tokens = self.out_logps = None
-        self._graph = None
-        self._graph_key = None
-        self.stats = {"decode_steps": 0, "prefill_tokens": 0, "generated_tokens": 0}
+
+    def _reset_sums(self):
+        """A step that raised half-way may have left partial sums behind."""
+        if self._own_gemm:
+            self._acc_qkv.zero_()
+            self._acc_o.zero_()
+            self._acc_d.zero_()
+
+    def _copy_pages(self, dst: torch.Tensor, src: torch.Tensor):
+        for li in range(self.cfg.num_hidden_layers):
+            self.k_cache[li].index_copy_(0, dst, self.k_cache[li].index_select(0, src))
+            self.v_cache[li].index_copy_(0, dst, self.v_cache[li].index_select(0, src))
+
+    def _copy_slots(self, dst: torch.Tensor, src: torch.Tensor):
+        """Per-slot state a sequence takes over from another one with the same prompt (a paged cache has none)."""
+
+    def _head(self, hidden: torch.Tensor) -> torch.Tensor:
+        return torch.nn.functional.linear(hidden, self.model.lm_head_weight)
+
+    def _page_writer(self, tok_slot, ctx: SeqCtx, slots: torch.Tensor):
+        """What the model's prompt forward hands its keys and values (or states) to."""
+        return _PrefillKV(self, tok_slot, ctx.positions.to(torch.int32))
 
     # ---- weights ------------------------------------------------------------------------------
     def sync_weights(self, model: CausalLM | None = None):
@@ -238,19 +274,24 @@ class RolloutEngine:
     def _decode_step(self, sp: SamplingParams, max_total_len: int):
         from ..ops import cuda as K
 
-        if self._own_gemm:
-            was = K.set_pdl(self._pdl)
-            try:
-                logits = self._decode_layers_own()
-            finally:
-                K.set_pdl(was)
-        else:
-            logits = self._decode_layers_lib()
-        self._sample(logits, sp)
+        self._sample(self._decode_logits(), sp)
         K.advance(self.tok, self.logp, None, self.seq_lens, self.n_gen, self.finished, self.out_tokens, self.out_logps,
                   sp.eos_token_id, max_total_len, self.next_input, self.step_counter, 1)
         if self.seen is not None:
             self.seen.scatter_(1, self.next_input[:, None], 1)
+
+    def _decode_logits(self):
+        """Logits [max_seqs, V] after the tokens in ``next_input`` (one per slot; rows of idle slots mean nothing); their
+        keys and values, or states, are stored at position ``seq_lens[slot]``."""
+        from ..ops import cuda as K
+
+        if not self._own_gemm:
+            return self._decode_layers_lib()
+        was = K.set_pdl(self._pdl)
+        try:
+            return self._decode_layers_own()
+        finally:
+            K.set_pdl(was)
 
     def _decode_layers_own(self):
         """Decoder stack of one decode step on this library's kernels only: every linear is the weight-streaming
@@ -373,11 +414,18 @@ class RolloutEngine:
     def _prefill(self, owners: list[tuple[int, list]], pixels: list | None = None) -> torch.Tensor:
         """owners: [(slot, prompt_ids)]; pixels: per owner the pixel tensor of its images (vision-language models).
         Returns last-token hidden states [len(owners), H]."""
+        hidden, ctx = self._prefill_all(owners, pixels)
+        return hidden[(ctx.cu_seqlens[1:] - 1).long()]
+
+    @torch.no_grad()
+    def _prefill_all(self, owners: list[tuple[int, list]], pixels: list | None = None):
+        """Runs whole prompts into the cache of their slots; returns the hidden states of all their tokens (packed) and
+        the geometry."""
         lens = [len(p) for _, p in owners]
         flat = torch.tensor([t for _, p in owners for t in p], dtype=torch.long).pin_memory().to(self.dev, non_blocking=True)
         tok_slot = torch.tensor([s for (s, p) in owners for _ in p], dtype=torch.int32).to(self.dev, non_blocking=True)
         ctx = SeqCtx.from_lengths(lens, self.dev)
-        ctx.kv = _PrefillKV(self, tok_slot, ctx.positions.to(torch.int32))
+        ctx.kv = self._page_writer(tok_slot, ctx, torch.tensor([s for s, _ in owners], dtype=torch.int32, device=self.dev))
         self.stats["prefill_tokens"] += int(flat.numel())
         was = self.model.training
         self.model.eval()
@@ -385,7 +433,7 @@ class RolloutEngine:
         hidden = self.model.forward_hidden(flat, ctx, inputs_embeds=embeds)
         if was:
             self.model.train()
-        return hidden[(ctx.cu_seqlens[1:] - 1).long()]
+        return hidden, ctx
 
     # ---- public API -----------------------------------------------------------------------------------
     @torch.no_grad()
@@ -421,10 +469,7 @@ class RolloutEngine:
         self.seq_lens.fill_(-1)
         self.finished.zero_()
         self.n_gen.zero_()
-        if self._own_gemm:  # a step that raised half-way may have left partial sums behind
-            self._acc_qkv.zero_()
-            self._acc_o.zero_()
-            self._acc_d.zero_()
+        self._reset_sums()
         bt_np = self.block_table_host.numpy()
         timing = os.environ.get("TRL_B200_ROLLOUT_TIMING", "0") == "1"  # wall-clock sections in self.stats (adds syncs)
         graph_key = (sp.temperature, sp.top_p, sp.top_k, sp.min_p, sp.repetition_penalty, sp.eos_token_id,
@@ -462,9 +507,7 @@ class RolloutEngine:
                 if pairs:
                     dst_t = torch.tensor([p[0] for p in pairs], dtype=torch.long, device=dev)
                     src_t = torch.tensor([p[1] for p in pairs], dtype=torch.long, device=dev)
-                    for li in range(self.cfg.num_hidden_layers):
-                        self.k_cache[li].index_copy_(0, dst_t, self.k_cache[li].index_select(0, src_t))
-                        self.v_cache[li].index_copy_(0, dst_t, self.v_cache[li].index_select(0, src_t))
+                    self._copy_pages(dst_t, src_t)
                 slots = torch.tensor([a[1] for a in admitted], dtype=torch.int32, device=dev)
                 plen_t = torch.tensor([len(reqs[a[0]][0]) for a in admitted], dtype=torch.int32, device=dev)
                 self.seq_lens[slots.long()] = plen_t
@@ -475,6 +518,7 @@ class RolloutEngine:
                     for a in admitted:
                         self.seen[a[1], torch.tensor(reqs[a[0]][0], device=dev)] = 1
                 # first token of every admitted request from its group's last-prompt-token logits
+                source_slot = {reqs[a[0]][1]: a[1] for a in admitted if a[2]}
                 if last_h is not None and len(group_row) == len(set(reqs[a[0]][1] for a in admitted)):
                     rows = torch.tensor([group_row[reqs[a[0]][1]] for a in admitted], device=dev)
                     h_rows = last_h[rows]
@@ -482,11 +526,16 @@ class RolloutEngine:
                     need = {}
                     for a in admitted:
                         need.setdefault(reqs[a[0]][1], a)
-                    tmp = self._prefill_hidden_only([reqs[a[0]][0] for a in need.values()],
-                                                    None if images is None else [images[g] for g in need])
+                    tmp = self._prefill_again([(a[1], reqs[a[0]][0]) for a in need.values()],
+                                              None if images is None else [images[g] for g in need])
+                    source_slot = {g: a[1] for g, a in need.items()}
                     gi = {g: i for i, g in enumerate(need)}
                     h_rows = tmp[torch.tensor([gi[reqs[a[0]][1]] for a in admitted], device=dev)]
-                logits = torch.nn.functional.linear(h_rows, self.model.lm_head_weight)
+                # sequences of one prompt start from the state its prefill left in one of their slots
+                takes = [(a[1], source_slot[reqs[a[0]][1]]) for a in admitted if source_slot[reqs[a[0]][1]] != a[1]]
+                if takes:
+                    self._copy_slots(*torch.tensor(takes, dtype=torch.long, device=dev).t())
+                logits = self._head(h_rows)
                 tok = torch.empty(len(admitted), dtype=torch.int32, device=dev)
                 lp = torch.empty(len(admitted), dtype=torch.float32, device=dev)
                 self._sample(logits, sp, rows=slots.long(), tok=tok, logp=lp)
@@ -544,6 +593,10 @@ class RolloutEngine:
         self._tmp_next = torch.zeros(self.max_seqs, dtype=torch.int64, device=self.dev)
         return self._tmp_next
 
+    def _prefill_again(self, owners: list[tuple[int, list]], pixels: list | None = None):
+        """Last hidden states of prompts whose pages were already written by an earlier admission."""
+        return self._prefill_hidden_only([p for _, p in owners], pixels)
+
     def _prefill_hidden_only(self, prompts, pixels: list | None = None):
         lens = [len(p) for p in prompts]
         flat = torch.tensor([t for p in prompts for t in p], dtype=torch.long, device=self.dev)
@@ -585,6 +638,8 @@ class RolloutEngine:
                                      self.out_tokens, self.out_logps)]
         s = torch.cuda.Stream()
         s.wait_stream(torch.cuda.current_stream())
+        if self.stateful:  # a recurrent state must not take the same token twice: warm up with every slot idle
+            self.seq_lens.fill_(-1)
         with torch.cuda.stream(s):
             self._decode_step(sp, max_total)
         torch.cuda.current_stream().wait_stream(s)
@@ -599,3 +654,12 @@ class RolloutEngine:
                          self.out_logps), state):
             t.copy_(o)
         self._graph, self._graph_key = g, key
+
+
+def make_engine(model, *args, **kw) -> RolloutEngine:
+    """Rollout engine of the class that serves ``model`` on one GPU."""
+    if getattr(model, "is_layered", False):
+        from .layered_engine import LayeredRolloutEngine as cls
+    else:
+        cls = RolloutEngine
+    return cls(model, *args, **kw)

@@ -72,7 +72,7 @@ class EngineHolder:
         import torch
 
         from ..models.hf_io import load_model
-        from ..rollout.engine import EagerGenerator, RolloutEngine
+        from ..rollout.engine import EagerGenerator, make_engine
 
         cuda = torch.cuda.is_available()
         if cuda:
@@ -91,7 +91,7 @@ class EngineHolder:
 
             self.engine = TPRolloutEngine(self.model, tp_group, max_num_seqs=a.max_num_seqs, max_model_len=a.max_model_len or 2048)
         elif cuda:
-            self.engine = RolloutEngine(self.model, a.max_num_seqs, a.max_model_len or 2048)
+            self.engine = make_engine(self.model, a.max_num_seqs, a.max_model_len or 2048)
         else:
             self.engine = EagerGenerator(self.model)
         self.world_size = a.tensor_parallel_size * a.data_parallel_size

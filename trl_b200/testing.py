@@ -11,6 +11,7 @@ import torch
 
 from .models.configuration import ModelArch, preset
 from .models.decoder import CausalLM
+from .models.hf_io import build_model
 
 CHATML_TEMPLATE = (
     "{% for message in messages %}"
@@ -64,7 +65,7 @@ def make_tiny_tokenizer(vocab_size: int = 1024):
 def make_tiny_model(name: str = "tiny-qwen2", dtype=torch.float32, device=None, seed: int = 0, **overrides) -> CausalLM:
     torch.manual_seed(seed)
     cfg = preset(name, **overrides)
-    return CausalLM(cfg, dtype=dtype, device=device)
+    return build_model(cfg, dtype=dtype, device=device)
 
 
 def _sentence(rng: random.Random, lo=3, hi=12) -> str:

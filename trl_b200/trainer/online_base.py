@@ -23,7 +23,8 @@ import torch.nn as nn
 
 from ..data_utils import apply_chat_template, is_conversational, maybe_apply_chat_template
 from ..loop.trainer import Trainer
-from ..models.decoder import CausalLM, SeqCtx
+from ..models.decoder import SeqCtx
+from ..models.hf_io import build_model
 from ..models.vision import merge_vision_entries, same_vision_entry
 from ..ops import functional as ops
 from ..parallel import dist as D
@@ -220,7 +221,7 @@ class OnlineTrainer(Trainer):
             if getattr(self.model, "is_vlm", False):
                 raise NotImplementedError("streamed full shard with a vision-language generation replica")
             if getattr(self, "_gen_model", None) is None:
-                self._gen_model = CausalLM(self.model.config, dtype=self.model.dtype, device=self.args.device, init=False)
+                self._gen_model = build_model(self.model.config, dtype=self.model.dtype, device=self.args.device, init=False)
                 self._gen_model.eval().requires_grad_(False)
             gen_model = self._gen_model
         elif (getattr(self.model, "peft_config", None) is not None and self.args.device.type == "cuda"
@@ -231,13 +232,13 @@ class OnlineTrainer(Trainer):
             if getattr(self.model, "is_vlm", False):
                 raise NotImplementedError("adapters with a vision-language generation replica")
             if getattr(self, "_gen_model", None) is None:
-                self._gen_model = CausalLM(self.model.config, dtype=self.model.dtype, device=self.args.device, init=False)
+                self._gen_model = build_model(self.model.config, dtype=self.model.dtype, device=self.args.device, init=False)
                 self._gen_model.eval().requires_grad_(False)
                 self._gen_merged = True
             gen_model = self._gen_model
         if self._rollout is None:
             if self.args.device.type == "cuda":
-                from ..rollout.engine import RolloutEngine
+                from ..rollout.engine import make_engine
 
                 a = self.args
                 max_len = a.vllm_max_model_length or (self._max_prompt_len_seen + self.max_completion_length + 8)
@@ -256,7 +257,7 @@ class OnlineTrainer(Trainer):
                                                     block_size=bs, poll_every=a.rollout_poll_every)
                 else:
                     try:
-                        self._rollout = RolloutEngine(gen_model, max_num_seqs=nseq, max_model_len=max_len, block_size=bs,
+                        self._rollout = make_engine(gen_model, max_num_seqs=nseq, max_model_len=max_len, block_size=bs,
                                                       poll_every=a.rollout_poll_every)
                     except NotImplementedError as e:  # e.g. GeGLU models: correct but slow eager generation
                         import warnings

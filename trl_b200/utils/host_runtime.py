@@ -21,6 +21,8 @@ class HostRuntime:
         lib.trlb_sched_admit.restype = c_int
         lib.trlb_sched_retire.argtypes = [c_void_p, c_int, c_int64]
         lib.trlb_sched_retire.restype = c_int64
+        lib.trlb_sched_grow.argtypes = [c_void_p, c_int, c_int, c_void_p]
+        lib.trlb_sched_grow.restype = c_int
         lib.trlb_bfd_assign.argtypes = [c_void_p, c_int, c_int, c_void_p]
         lib.trlb_bfd_assign.restype = c_int
 
@@ -69,6 +71,15 @@ class Scheduler:
 
     def retire(self, slot: int, group: int) -> int:
         return int(self.lib.trlb_sched_retire(self.h, slot, group))
+
+    def grow(self, slot: int, total_tokens: int, block_table_np: np.ndarray) -> int:
+        """Blocks for ``total_tokens`` tokens of the running request in ``slot``; returns how many were added."""
+        n = int(self.lib.trlb_sched_grow(self.h, slot, total_tokens, block_table_np.ctypes.data))
+        if n == -2:
+            raise RuntimeError("the paged cache is full")
+        if n < 0:
+            raise ValueError(f"slot {slot} cannot hold {total_tokens} tokens")
+        return n
 
     num_waiting = property(lambda s: s.lib.trlb_sched_num_waiting(s.h))
     num_running = property(lambda s: s.lib.trlb_sched_num_running(s.h))
