@@ -124,7 +124,19 @@ def latent_attention(m, h, ctx, li):
     q = linear(cq, m.uq)
     K.rotate_q(q, m, pos, table)
     kv = linear(lat[:, : m.kv_rank], m.ukv)
-    return linear_f32(K.latent_prompt(q, kv, lat, m, pos, gate), m.o)
+    return linear_f32(latent_prompt_attention(q, kv, lat, m, ctx, gate), m.o)
+
+
+def latent_prompt_attention(q, kv, lat, m, ctx, gate):
+    """Windowed sink attention of packed prompts, times the output gates.  q [T, heads (dim | rot)] rotated, kv [T, heads
+    dim | heads vdim], lat [T, latent row], gate [T, heads] -> [T, heads vdim]."""
+    return _k().latent_prompt(q, kv, lat, m, ctx.positions.to(torch.int32), gate)
+
+
+def mlstm_prompt_scan(y, m, ig, fg, ctx, where):
+    """The recurrence over packed prompts.  y [T, q | k | v | ...] in the model dtype, log gates [T, heads] ->
+    [T, heads, vdim] fp32; ``where`` (may be empty) says which slots get the final states."""
+    return _k().mlstm_prompt(y, m, ig, fg, ctx.cu_seqlens, **where)
 
 
 def mlstm(m, h, ctx, li):
@@ -134,7 +146,7 @@ def mlstm(m, h, ctx, li):
     y = linear(h, m.w_in[: m.gate_row])
     ig, fg = K.mlstm_gates(linear_f32(h, m.w_in[m.gate_row:]), m.gate_bias, m.cap, m.heads)
     where = ctx.kv.recurrent_state(li) if ctx.kv is not None else {}
-    o = K.mlstm_prompt(y, m, ig, fg, ctx.cu_seqlens, **where)
+    o = mlstm_prompt_scan(y, m, ig, fg, ctx, where)
     out = torch.empty(h.shape[0], m.heads * m.vdim, dtype=h.dtype, device=h.device)
     K.mlstm_out(o, y[:, m.heads * (2 * m.dim + m.vdim):], m, out)
     return linear_f32(out, m.o)
