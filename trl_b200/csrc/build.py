@@ -25,7 +25,7 @@ OBJ = os.path.join(LIB, "obj")
 NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17", "--use_fast_math",
               "-Xcompiler", "-fPIC,-fvisibility=hidden", "-Xptxas", "-v", "--expt-relaxed-constexpr"]
 # sources whose results the fast approximations of exp, tanh, erf, division and square root would show in
-EXACT_MATH = {"mixers.cu"}
+EXACT_MATH = {"mixers.cu", "mlstm_chunk_tcgen05.cu"}
 # every source here builds into the one library used at any GPU count (no loads shared across a thread-block cluster)
 
 

@@ -1,0 +1,375 @@
+// Prompt attention of the latent-attention mixer on the 5th-generation tensor cores (bf16, packed sequences).
+//
+// The structure is that of fa_varlen_tcgen05.cu (one CTA per 128-query tile and head; TMA warp, MMA warp, one softmax
+// thread per query row; S double-buffered in TMEM, O accumulated in TMEM and rescaled only when a row's reference
+// maximum moves by more than 2^8).  What differs:
+//
+//   * a query / key vector has two parts that live in different tensors: `dim` elements per head (queries in q, keys in
+//     the up-projected kv rows) and `rot` rotated elements (in q behind the first part; keys in the latent rows, ONE
+//     for all heads).  Each part is loaded as 64-column TMA boxes of its own, zero-filled past its end, so nothing is
+//     concatenated or expanded in memory; Q.K^T runs over the 16-column steps that hold data;
+//   * sizes are launch parameters: dim, rot, vdim any multiples of 8 (vdim <= 256) that leave room for one stage;
+//   * probabilities keep 32-bit precision into P.V: each is split into two bf16 (value and remainder), both halves of
+//     the S buffer are reused for them (64 columns each), and P.V accumulates both products;
+//   * the softmax denominator contains exp(sink[head]) and the output is multiplied by a per-token, per-head gate;
+//   * keys are those of the same sequence at distance < window.
+#include "common.cuh"
+
+namespace trlb {
+
+constexpr int LA_BM = 128, LA_BN = 128;
+constexpr int LA_THREADS = 192;
+constexpr uint32_t LA_BOX = 128 * 64 * 2;  // one TMA box: 128 rows x 64 bf16, 128-byte swizzle
+
+struct LatentTcParams {
+  const int* cu;
+  int n_seq, heads, dim, rot, vdim, window;
+  int nn, nr, nv;      // boxes of the unrotated part, the rotated part and the value
+  int k_stages, v_stages;
+  float scale_log2;
+  const float* sink;
+  const float* gate;   // [T, heads]
+  __nv_bfloat16* out;  // [T, heads, vdim]
+  int* status;
+};
+
+__device__ __forceinline__ bool la_find_tile(const int* cu, int n_seq, int slot, int& seq, int& tile) {
+  for (int s = 0; s < n_seq; ++s) {
+    const int nt = (cu[s + 1] - cu[s] + LA_BM - 1) / LA_BM;
+    if (slot < nt) { seq = s; tile = nt - 1 - slot; return true; }
+    slot -= nt;
+  }
+  return false;
+}
+
+__global__ void __launch_bounds__(LA_THREADS, 1)
+latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_constant__ CUtensorMap tm_qr,
+                      const __grid_constant__ CUtensorMap tm_kn, const __grid_constant__ CUtensorMap tm_kr,
+                      const __grid_constant__ CUtensorMap tm_v, const LatentTcParams p) {
+  int seq, tile;
+  if (!la_find_tile(p.cu, p.n_seq, (int)blockIdx.x, seq, tile)) return;  // uniform: before any barrier or TMEM use
+  extern __shared__ uint8_t smem_raw[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
+  const uint32_t k_bytes = (uint32_t)(p.nn + p.nr) * LA_BOX, v_bytes = (uint32_t)p.nv * LA_BOX;
+  uint8_t* q_s = smem;
+  uint8_t* k_s = q_s + k_bytes;
+  uint8_t* v_s = k_s + (size_t)p.k_stages * k_bytes;
+  uint64_t* bars = reinterpret_cast<uint64_t*>(v_s + (size_t)p.v_stages * v_bytes);
+  uint64_t* q_full = bars;
+  uint64_t* k_full = bars + 1;        // [<= 3]
+  uint64_t* k_empty = bars + 4;
+  uint64_t* v_full = bars + 7;
+  uint64_t* v_empty = bars + 10;
+  uint64_t* s_full = bars + 13;       // [2]
+  uint64_t* p_full = bars + 15;       // [2]
+  uint64_t* o_full = bars + 17;
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 18);
+  volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
+
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int h = blockIdx.y;
+  const int beg = p.cu[seq], len = p.cu[seq + 1] - beg;
+  const int q_first = tile * LA_BM;
+  const int q_last = min(len, q_first + LA_BM) - 1;
+  const int hi = q_last / LA_BN;
+  const int lo = p.window > 0 ? max(0, q_first - p.window + 1) / LA_BN : 0;
+  const int n_kv = hi - lo + 1;  // >= 1: a token sees itself
+
+  if (threadIdx.x == 0) {
+    mbar_init(q_full, 1);
+    for (int s = 0; s < 3; ++s) {
+      mbar_init(&k_full[s], 1);
+      mbar_init(&k_empty[s], 1);
+      mbar_init(&v_full[s], 1);
+      mbar_init(&v_empty[s], 1);
+    }
+    for (int s = 0; s < 2; ++s) {
+      mbar_init(&s_full[s], 1);
+      mbar_init(&p_full[s], 128);
+    }
+    mbar_init(o_full, 1);
+    *abort_flag = 0;
+    mbar_fence_init();
+    tma_prefetch_desc(&tm_qn);
+    tma_prefetch_desc(&tm_kn);
+    tma_prefetch_desc(&tm_v);
+  }
+  if (warp == 1) {
+    tmem_alloc(tmem_slot, 512);
+    tmem_relinquish();
+    tc_fence_before();
+  }
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem_base = *tmem_slot;
+
+  if (warp == 0) {
+    // ---------------- TMA producer ----------------
+    if (lane == 0) {
+      mbar_expect_tx(q_full, k_bytes);
+      for (int i = 0; i < p.nn; ++i) tma_load_3d(q_s + i * LA_BOX, &tm_qn, q_full, 64 * i, h, beg + q_first);
+      for (int i = 0; i < p.nr; ++i) tma_load_3d(q_s + (p.nn + i) * LA_BOX, &tm_qr, q_full, 64 * i, h, beg + q_first);
+      auto load_k = [&](int j) {
+        const int s = j % p.k_stages;
+        if (!mbar_wait(&k_empty[s], (uint32_t)(((j / p.k_stages) & 1) ^ 1), abort_flag, p.status, 1200 + s)) return false;
+        uint8_t* ks = k_s + (size_t)s * k_bytes;
+        const int row = beg + (lo + j) * LA_BN;
+        mbar_expect_tx(&k_full[s], k_bytes);
+        for (int i = 0; i < p.nn; ++i) tma_load_3d(ks + i * LA_BOX, &tm_kn, &k_full[s], 64 * i, h, row);
+        for (int i = 0; i < p.nr; ++i) tma_load_2d(ks + (p.nn + i) * LA_BOX, &tm_kr, &k_full[s], 64 * i, row);
+        return true;
+      };
+      bool ok = load_k(0);
+      for (int j = 0; j < n_kv && ok; ++j) {
+        if (j + 1 < n_kv) ok = load_k(j + 1);
+        if (!ok) break;
+        const int s = j % p.v_stages;
+        if (!mbar_wait(&v_empty[s], (uint32_t)(((j / p.v_stages) & 1) ^ 1), abort_flag, p.status, 1205 + s)) break;
+        uint8_t* vs = v_s + (size_t)s * v_bytes;
+        mbar_expect_tx(&v_full[s], v_bytes);
+        for (int i = 0; i < p.nv; ++i) tma_load_3d(vs + i * LA_BOX, &tm_v, &v_full[s], 64 * i, h, beg + (lo + j) * LA_BN);
+      }
+    }
+    __syncwarp();
+  } else if (warp == 1) {
+    // ---------------- MMA issuer ----------------
+    if (lane == 0) {
+      const uint32_t idesc_s = umma_idesc_bf16_major(LA_BM, LA_BN, false, false);
+      const uint32_t idesc_o = umma_idesc_bf16_major(LA_BM, (p.vdim + 15) & ~15, false, true);  // V is MN-major
+      const uint32_t q_u = smem_u32(q_s), ks_u = smem_u32(k_s), vs_u = smem_u32(v_s);
+      bool ok = mbar_wait(q_full, 0, abort_flag, p.status, 1210);
+      auto issue_s = [&](int j) {
+        const int s = j & 1, kst = j % p.k_stages;
+        // buffer s is free: its P.V product (tile j - 2) was issued before this call
+        if (!mbar_wait(&k_full[kst], (uint32_t)((j / p.k_stages) & 1), abort_flag, p.status, 1220 + kst)) return false;
+        tc_fence_after();
+        const uint32_t k_u = ks_u + (uint32_t)kst * k_bytes;
+        uint32_t acc = 0;
+        for (int i = 0; i < p.nn + p.nr; ++i) {
+          const int left = i < p.nn ? p.dim - 64 * i : p.rot - 64 * (i - p.nn);
+          const int steps = min(4, (left + 15) >> 4);
+          const uint64_t da = umma_desc_kmajor_sw128(q_u + (uint32_t)i * LA_BOX), db = umma_desc_kmajor_sw128(k_u + (uint32_t)i * LA_BOX);
+          for (int kk = 0; kk < steps; ++kk) {
+            umma_bf16_ss(tmem_base + (uint32_t)s * LA_BN, da + 2 * kk, db + 2 * kk, idesc_s, acc);
+            acc = 1;
+          }
+        }
+        umma_commit(&s_full[s]);
+        umma_commit(&k_empty[kst]);
+        return true;
+      };
+      if (ok) ok = issue_s(0);
+      for (int j = 0; j < n_kv && ok; ++j) {
+        if (j + 1 < n_kv) ok = issue_s(j + 1);
+        if (!ok) break;
+        const int sb = j & 1, s = j % p.v_stages;
+        if (!mbar_wait(&p_full[sb], (uint32_t)((j >> 1) & 1), abort_flag, p.status, 1240 + sb)) break;
+        if (!mbar_wait(&v_full[s], (uint32_t)((j / p.v_stages) & 1), abort_flag, p.status, 1250 + s)) break;
+        tc_fence_after();
+        const uint32_t v_u = vs_u + (uint32_t)s * v_bytes;
+        // the S buffer holds P as bf16 pairs: leading parts in its first 64 columns, remainders in the other 64
+        for (int half = 0; half < 2; ++half)
+#pragma unroll
+          for (int kk = 0; kk < LA_BN / 16; ++kk)
+            umma_bf16_ts(tmem_base + 256, tmem_base + (uint32_t)(sb * LA_BN + half * 64 + kk * 8),
+                         umma_desc_mnmajor_sw128(v_u + (uint32_t)kk * 2048, LA_BOX), idesc_o, (j | half | kk) != 0);
+        umma_commit(o_full);
+        umma_commit(&v_empty[s]);
+      }
+    }
+    __syncwarp();
+  } else {
+    // ---------------- softmax: one thread per query row ----------------
+    const int quarter = warp & 3;
+    const int r = quarter * 32 + lane;
+    const uint32_t lane_off = (uint32_t)(quarter * 32) << 16;
+    const int q_pos = q_first + r;
+    const bool row_ok = q_pos < len;
+    const int k_max = row_ok ? q_pos : -1;
+    const int k_min = p.window > 0 ? max(0, q_pos - p.window + 1) : 0;
+    const uint32_t to = tmem_base + lane_off + 256;
+    float m_ref = -INFINITY, l_run = 0.f;
+    bool ok = true;
+    for (int j = 0; j < n_kv && ok; ++j) {
+      const int s = j & 1;
+      const int key0 = (lo + j) * LA_BN;
+      const bool full = q_first + LA_BM <= len && key0 + LA_BN - 1 <= q_first &&
+                        (p.window <= 0 || key0 >= q_first + LA_BM - p.window);
+      ok = __all_sync(0xffffffffu, mbar_wait(&s_full[s], (uint32_t)((j >> 1) & 1), abort_flag, p.status, 1270 + s));
+      if (!ok) break;
+      tc_fence_after();
+      const uint32_t ts = tmem_base + lane_off + (uint32_t)s * LA_BN;
+      float v[4][32];
+#pragma unroll
+      for (int c = 0; c < 4; ++c) tmem_ld_32x32(ts + 32 * c, v[c]);
+      tmem_ld_wait();
+      if (!full) {
+#pragma unroll
+        for (int c = 0; c < 4; ++c)
+#pragma unroll
+          for (int i = 0; i < 32; ++i) {
+            const int key = key0 + 32 * c + i;
+            if (key < k_min || key > k_max) v[c][i] = -INFINITY;
+          }
+      }
+      float mx = -INFINITY;
+#pragma unroll
+      for (int c = 0; c < 4; ++c)
+#pragma unroll
+        for (int i = 0; i < 32; ++i) mx = fmaxf(mx, v[c][i]);
+      const float m_tile = mx * p.scale_log2;
+      float alpha = 1.f;
+      bool moved = false;
+      if (m_ref == -INFINITY) {
+        m_ref = m_tile;  // nothing seen so far: the row of O is zero (or meaningless only through zero weights)
+      } else if (m_tile > m_ref + 8.f) {
+        alpha = fast_exp2(m_ref - m_tile);
+        m_ref = m_tile;
+        moved = true;
+      }
+      if (j > 0 && __any_sync(0xffffffffu, moved)) {
+        ok = __all_sync(0xffffffffu, mbar_wait(o_full, (uint32_t)((j - 1) & 1), abort_flag, p.status, 1290));
+        if (!ok) break;
+        tc_fence_after();
+#pragma unroll 1
+        for (int c = 0; c < p.vdim; c += 16) {
+          float o[16];
+          tmem_ld_32x16(to + c, o);
+          tmem_ld_wait();
+          uint32_t w[16];
+#pragma unroll
+          for (int i = 0; i < 16; ++i) w[i] = __float_as_uint(o[i] * alpha);
+          tmem_st_32x16(to + c, w);
+        }
+      }
+      l_run *= alpha;
+      const float neg_m = m_ref == -INFINITY ? 0.f : -m_ref;
+      float sum = 0.f;
+#pragma unroll
+      for (int c = 0; c < 4; ++c) {
+        uint32_t a[16], b[16];
+#pragma unroll
+        for (int i = 0; i < 16; ++i) {
+          const float p0 = fast_exp2(fmaf(v[c][2 * i], p.scale_log2, neg_m));  // masked scores: exp2(-inf) = 0
+          const float p1 = fast_exp2(fmaf(v[c][2 * i + 1], p.scale_log2, neg_m));
+          sum += p0 + p1;
+          a[i] = pack_bf16(p0, p1);
+          const float2 f = unpack_bf16(a[i]);
+          b[i] = pack_bf16(p0 - f.x, p1 - f.y);
+        }
+        tmem_st_32x16(ts + 16 * c, a);
+        tmem_st_32x16(ts + 64 + 16 * c, b);
+      }
+      tmem_st_wait();
+      tc_fence_before();
+      mbar_arrive(&p_full[s]);
+      l_run += sum;
+    }
+    if (ok) {
+      const int last = n_kv - 1;
+      if (last >= 1)
+        ok = __all_sync(0xffffffffu, mbar_wait(o_full, (uint32_t)((last - 1) & 1), abort_flag, p.status, 1294));
+      if (ok) ok = __all_sync(0xffffffffu, mbar_wait(o_full, (uint32_t)(last & 1), abort_flag, p.status, 1295));
+      if (ok) {
+        tc_fence_after();
+        float f = 0.f;
+        __nv_bfloat16* dst = nullptr;
+        if (row_ok) {
+          const float sk = p.sink[h] * 1.4426950408889634f, mt = fmaxf(m_ref, sk);
+          const float wm = fast_exp2(m_ref - mt);
+          const size_t th = (size_t)(beg + q_pos) * p.heads + h;
+          f = wm / (l_run * wm + fast_exp2(sk - mt)) * p.gate[th];
+          dst = p.out + th * p.vdim;
+        }
+#pragma unroll 1
+        for (int c = 0; c < p.vdim; c += 16) {
+          float o[16];
+          tmem_ld_32x16(to + c, o);
+          tmem_ld_wait();
+          if (row_ok) {
+#pragma unroll
+            for (int i = 0; i < 16; i += 8)
+              if (c + i < p.vdim)
+                *reinterpret_cast<uint4*>(dst + c + i) =
+                    make_uint4(pack_bf16(o[i] * f, o[i + 1] * f), pack_bf16(o[i + 2] * f, o[i + 3] * f),
+                               pack_bf16(o[i + 4] * f, o[i + 5] * f), pack_bf16(o[i + 6] * f, o[i + 7] * f));
+          }
+        }
+        tc_fence_before();
+      }
+    }
+  }
+  __syncthreads();
+  if (*abort_flag) {
+    const uint64_t t0 = globaltimer_ns();
+    while (globaltimer_ns() - t0 < 200000ull) __nanosleep(1000);
+    __syncthreads();
+  }
+  if (warp == 1) {
+    tc_fence_after();
+    tmem_dealloc(tmem_base, 512);
+  }
+}
+
+}  // namespace trlb
+
+using namespace trlb;
+
+namespace {
+
+size_t la_smem(int nk, int nv, int ks, int vs) { return (size_t)(nk + ks * nk + vs * nv) * LA_BOX + 1024 + 256; }
+
+// Deepest rings that fit shared memory; false: not even one stage each.
+bool la_stages(int nk, int nv, int& ks, int& vs) {
+  constexpr int opt[6][2] = {{3, 3}, {3, 2}, {2, 2}, {2, 1}, {1, 1}, {0, 0}};
+  for (int i = 0; opt[i][0]; ++i)
+    if (la_smem(nk, nv, opt[i][0], opt[i][1]) <= 227 * 1024) { ks = opt[i][0]; vs = opt[i][1]; return true; }
+  return false;
+}
+
+int la_boxes(int n) { return (n + 63) / 64; }
+
+}  // namespace
+
+// 1 when trlb_latent_attn_tc takes these sizes.
+TRLB_API int trlb_latent_attn_tc_ok(int heads, int dim, int rot, int vdim) {
+  int ks, vs;
+  return dim > 0 && rot > 0 && vdim > 0 && dim % 8 == 0 && rot % 8 == 0 && vdim % 8 == 0 && vdim <= 256 && heads > 0 &&
+         la_stages(la_boxes(dim) + la_boxes(rot), la_boxes(vdim), ks, vs);
+}
+
+// q [T, heads, dim + rot] (rotated part last), kv [T, kv_ld]: heads * dim keys then heads * vdim values, krot [T, krot_ld]:
+// the shared rotated keys; all bf16, 16-byte aligned rows.  window <= 0: unlimited.  scale > 0.
+TRLB_API int trlb_latent_attn_tc(const void* q, const void* kv, long long kv_ld, const void* krot, long long krot_ld,
+                                 const int* cu, int n_seq, int T, int heads, int dim, int rot, int vdim, int window,
+                                 float scale, const float* sink, const float* gate, void* out, int* status,
+                                 cudaStream_t st) {
+  if (T <= 0 || n_seq <= 0) return 0;
+  if (!trlb_latent_attn_tc_ok(heads, dim, rot, vdim) || (kv_ld % 8) || (krot_ld % 8) || !(scale > 0.f)) return -210;
+  LatentTcParams p = {};
+  p.cu = cu; p.n_seq = n_seq; p.heads = heads; p.dim = dim; p.rot = rot; p.vdim = vdim; p.window = window;
+  p.nn = la_boxes(dim); p.nr = la_boxes(rot); p.nv = la_boxes(vdim);
+  la_stages(p.nn + p.nr, p.nv, p.k_stages, p.v_stages);
+  p.scale_log2 = scale * 1.4426950408889634f;
+  p.sink = sink; p.gate = gate; p.out = (__nv_bfloat16*)out; p.status = status;
+  const __nv_bfloat16* qb = (const __nv_bfloat16*)q;
+  const __nv_bfloat16* kb = (const __nv_bfloat16*)kv;
+  const int dq = dim + rot;
+  CUtensorMap tqn, tqr, tkn, tkr, tv;
+  using trlb_host::make_tmap_3d_bf16;
+  if (make_tmap_3d_bf16(&tqn, qb, dim, heads, T, dq, (uint64_t)heads * dq, 64, 1, 128)) return -211;
+  if (make_tmap_3d_bf16(&tqr, qb + dim, rot, heads, T, dq, (uint64_t)heads * dq, 64, 1, 128)) return -212;
+  if (make_tmap_3d_bf16(&tkn, kb, dim, heads, T, dim, (uint64_t)kv_ld, 64, 1, 128)) return -213;
+  if (trlb_host::make_tmap_2d_bf16(&tkr, krot, T, rot, (uint64_t)krot_ld, 128, 64)) return -214;
+  if (make_tmap_3d_bf16(&tv, kb + (size_t)heads * dim, vdim, heads, T, vdim, (uint64_t)kv_ld, 64, 1, 128)) return -215;
+  static bool attr_set = false;
+  if (!attr_set) {
+    if (cudaFuncSetAttribute(latent_attn_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024) != cudaSuccess)
+      return -216;
+    attr_set = true;
+  }
+  const int max_tiles = (T + LA_BM - 1) / LA_BM + n_seq;
+  latent_attn_tc_kernel<<<dim3(max_tiles, heads), LA_THREADS, la_smem(p.nn + p.nr, p.nv, p.k_stages, p.v_stages), st>>>(
+      tqn, tqr, tkn, tkr, tv, p);
+  return (int)cudaGetLastError();
+}

@@ -91,6 +91,23 @@ def latent_prompt(q, kv, lat, m, positions, gate):
     return out
 
 
+def latent_prompt_tc_ok(m) -> bool:
+    return m.scale > 0 and bool(lib().trlb_latent_attn_tc_ok(c_int(m.heads), c_int(m.dim), c_int(m.rot_dim), c_int(m.vdim)))
+
+
+def latent_prompt_tc(q, kv, lat, m, cu, gate):
+    """:func:`latent_prompt` on the tensor cores (bf16; see ``latent_prompt_tc_ok``); ``cu`` int32 sequence starts."""
+    T = q.shape[0]
+    kr, w = latent_row(m.kv_rank, m.rot_dim)
+    out = torch.empty(T, m.heads * m.vdim, dtype=q.dtype, device=q.device)
+    assert q.dtype == torch.bfloat16 and q.is_contiguous() and kv.stride(1) == 1 and lat.is_contiguous() and cu.dtype == torch.int32
+    _chk(lib().trlb_latent_attn_tc(_p(q), _p(kv), c_longlong(kv.stride(0)), _p(lat[:, kr:]), c_longlong(w), _p(cu),
+                                   c_int(cu.numel() - 1), c_int(T), c_int(m.heads), c_int(m.dim), c_int(m.rot_dim),
+                                   c_int(m.vdim), c_int(m.window or 0), c_float(m.scale), _p(m.sink), _p(gate), _p(out),
+                                   _p(status_buffer(q.device)), _s()), "latent_attn_tc")
+    return out
+
+
 def latent_absorb(qacc, m, positions, table, q_lat, clear):
     B = qacc.shape[0]
     kr, w = latent_row(m.kv_rank, m.rot_dim)
@@ -133,6 +150,29 @@ def mlstm_prompt(y, m, ig, fg, cu, seq_slot=None, state=None):
                                  c_int(cu.numel() - 1), _p(seq_slot if state is not None else None), _p(S), _p(n), _p(mm),
                                  c_int(0 if S is None else S.shape[0]), c_int(m.heads), c_int(m.dim), c_int(m.vdim),
                                  c_float(m.dim ** -0.5), _p(out), _b(y), _s()), "mlstm_prompt")
+    return out
+
+
+def mlstm_chunk_ok(m) -> bool:
+    return bool(lib().trlb_mlstm_chunk_ok(c_int(m.heads), c_int(m.dim), c_int(m.vdim)))
+
+
+def mlstm_chunk(y, m, ig, fg, cu, seq_slot=None, state=None):
+    """:func:`mlstm_prompt` in 128-token chunks on the tensor cores (bf16; see ``mlstm_chunk_ok``)."""
+    T, H, n_seq = y.shape[0], m.heads, cu.numel() - 1
+    assert y.dtype == torch.bfloat16 and y.stride(1) == 1 and cu.dtype == torch.int32
+    chunks = int(lib().trlb_mlstm_chunks(c_int(T), c_int(n_seq)))
+    f32 = dict(dtype=torch.float32, device=y.device)
+    out = torch.empty(T, H, m.vdim, **f32)
+    bgm, n_in = torch.empty(3, H, T, **f32), torch.empty(chunks, H, m.dim, **f32)
+    parts = torch.empty(2, chunks, H, m.dim, m.vdim, dtype=torch.bfloat16, device=y.device)
+    S, n, mm = state if state is not None else (None, None, None)
+    qd = H * m.dim
+    _chk(lib().trlb_mlstm_chunk(_p(y), c_longlong(y.stride(0)), c_int(qd), c_int(2 * qd), _p(ig), _p(fg), _p(cu), c_int(n_seq),
+                                c_int(T), _p(seq_slot if state is not None else None), _p(S), _p(n), _p(mm),
+                                c_int(0 if S is None else S.shape[0]), c_int(H), c_int(m.dim), c_int(m.vdim),
+                                c_float(m.dim ** -0.5), _p(bgm[0]), _p(bgm[1]), _p(bgm[2]), _p(n_in), _p(parts[0]),
+                                _p(parts[1]), _p(out), _p(status_buffer(y.device)), _s()), "mlstm_chunk")
     return out
 
 

@@ -130,13 +130,19 @@ def latent_attention(m, h, ctx, li):
 def latent_prompt_attention(q, kv, lat, m, ctx, gate):
     """Windowed sink attention of packed prompts, times the output gates.  q [T, heads (dim | rot)] rotated, kv [T, heads
     dim | heads vdim], lat [T, latent row], gate [T, heads] -> [T, heads vdim]."""
-    return _k().latent_prompt(q, kv, lat, m, ctx.positions.to(torch.int32), gate)
+    K = _k()
+    if q.dtype == torch.bfloat16 and K.latent_prompt_tc_ok(m):
+        return K.latent_prompt_tc(q, kv, lat, m, ctx.cu_seqlens, gate)
+    return K.latent_prompt(q, kv, lat, m, ctx.positions.to(torch.int32), gate)
 
 
 def mlstm_prompt_scan(y, m, ig, fg, ctx, where):
     """The recurrence over packed prompts.  y [T, q | k | v | ...] in the model dtype, log gates [T, heads] ->
     [T, heads, vdim] fp32; ``where`` (may be empty) says which slots get the final states."""
-    return _k().mlstm_prompt(y, m, ig, fg, ctx.cu_seqlens, **where)
+    K = _k()
+    if y.dtype == torch.bfloat16 and K.mlstm_chunk_ok(m):
+        return K.mlstm_chunk(y, m, ig, fg, ctx.cu_seqlens, **where)
+    return K.mlstm_prompt(y, m, ig, fg, ctx.cu_seqlens, **where)
 
 
 def mlstm(m, h, ctx, li):
