@@ -1,0 +1,281 @@
+"""Prompt and decode throughput of a layered design beside the closest flat decoder of the same width, depth and
+parameter count (random weights, bf16, one GPU), through the serving engine.
+
+    python -m trl_b200.benchmarks.layered_throughput [--sizes small,base] [--kernels]
+
+Prompt: packed prompts through the engine's prompt forward into its cache.  Decode: replays of the captured step (CUDA
+graph, sampler included) with every slot at the given context.  CUDA events after warm-up; the weights of a step are
+larger than L2.  ``--kernels`` times the mixers' kernels alone, L2 flushed in between, against the measured peaks."""
+from __future__ import annotations
+
+import argparse
+import json
+import os
+
+import torch
+
+# width, heads (latent attention and flat attention), query latent, ff, mLSTM heads
+SIZES = {"small": dict(width=2048, heads=16, q_rank=768, ff=8192, mheads=4, pairs=4),
+         "base": dict(width=4096, heads=32, q_rank=1536, ff=16384, mheads=8, pairs=4)}
+VOCAB = 32768
+
+
+def layered_config(width, heads, q_rank, ff, mheads, pairs, window=1024):
+    att = dict(type="latent_attention", mlp=dict(kind="dense", ff=ff),
+               mixer=dict(heads=heads, dim=128, rot_dim=64, vdim=128, q_rank=q_rank, kv_rank=512, scale=192 ** -0.5,
+                          mask=dict(size=window), rot=dict(base=1e4, dims=64, scaling=dict(factor=4.0, original=4096,
+                                                                                          fast=32.0, slow=1.0))))
+    rec = dict(type="mlstm", mlp=dict(kind="dense", ff=ff), mixer=dict(heads=mheads, dim=256, vdim=512, gate_cap=15.0))
+    return dict(architecture="Zorelorn", vocab=VOCAB, width=width, norm=dict(eps=1e-6), embedding=dict(scale=1.0),
+                layers=[att, rec] * pairs)
+
+
+def flat_config(s, target):
+    """Llama-type decoder of the same width and depth whose feed-forward width brings it to ``target`` parameters."""
+    from ..models.configuration import ModelArch
+
+    kw = dict(model_type="llama", vocab_size=VOCAB, hidden_size=s["width"], num_hidden_layers=2 * s["pairs"],
+              num_attention_heads=s["width"] // 128, num_key_value_heads=max(1, s["width"] // 512), head_dim=128,
+              rope_theta=5e5)
+    rest = target - ModelArch(intermediate_size=0, **kw).num_parameters()
+    return ModelArch(intermediate_size=max(256, rest // (kw["num_hidden_layers"] * 3 * s["width"]) // 256 * 256), **kw)
+
+
+def timed(fn, iters, warmup=3):
+    for _ in range(warmup):
+        fn()
+    torch.cuda.synchronize()
+    a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    a.record()
+    for _ in range(iters):
+        fn()
+    b.record()
+    torch.cuda.synchronize()
+    return a.elapsed_time(b) / iters
+
+
+@torch.no_grad()
+def measure(model, batch, prompt, n_prompts, iters=10):
+    from ..ops import cuda as K
+    from ..rollout.engine import make_engine
+    from ..rollout.sampling import SamplingParams
+
+    eng = make_engine(model, max_num_seqs=batch, max_model_len=prompt + 192)
+    toks = [torch.randint(2, VOCAB, (prompt,)).tolist() for _ in range(n_prompts)]
+    sp = SamplingParams(n=max(1, batch // n_prompts), max_tokens=64, seed=1)
+    eng.generate(toks, sp)  # fills the cache and captures the decode graph
+    bt = eng.block_table_host.numpy()
+    for i, t in enumerate(toks):
+        eng.sched.add(i, len(t), 64, i)
+    owners = [(slot, toks[rid]) for rid, slot, _, _ in eng.sched.admit(bt)]
+    eng.block_table.copy_(eng.block_table_host)
+    n0 = K.LAUNCHES[0]
+    ms_prompt = timed(lambda: eng._prefill_all(owners), iters)
+    launches = K.LAUNCHES[0] - n0
+    for slot, _ in owners:
+        eng.sched.retire(slot, slot)
+    eng.block_table.copy_(torch.arange(eng.block_table.numel(), device=eng.dev).view_as(eng.block_table).remainder(eng.num_blocks))
+
+    def step():
+        eng._graph.replay()
+
+    eng.n_gen.zero_()
+    eng.finished.zero_()
+    eng.seq_lens.fill_(prompt)
+    ms_step = timed(step, 40)
+    K.check_status()
+    return dict(prompt_tok_s=round(n_prompts * prompt / ms_prompt * 1e3), prompt_ms=round(ms_prompt, 3),
+                decode_tok_s=round(batch / ms_step * 1e3), decode_ms=round(ms_step, 4), own_prompt_launches=launches)
+
+
+def run(sizes=("small", "base"), batch=64, prompt=1024, n_prompts=8):
+    from ..models.configuration import ModelArch
+    from ..models.hf_io import build_model
+
+    out = []
+    for name in sizes:
+        s = SIZES[name]
+        arch = ModelArch.from_hf_dict(layered_config(**s))
+        n = arch.num_parameters()
+        flat = flat_config(s, n)
+        row = dict(size=name, layers=2 * s["pairs"], width=s["width"], batch=batch, prompt=f"{n_prompts}x{prompt}",
+                   decode_context=prompt)
+        for key, cfg in (("layered", arch), ("flat", flat)):
+            torch.manual_seed(0)
+            model = build_model(cfg, dtype=torch.bfloat16, device="cuda").eval().requires_grad_(False)
+            row[key] = dict(params_m=round(sum(p.numel() for p in model.parameters()) / 1e6), **measure(model, batch, prompt, n_prompts))
+            del model
+            torch.cuda.empty_cache()
+        row["prompt_ratio"] = round(row["layered"]["prompt_tok_s"] / row["flat"]["prompt_tok_s"], 3)
+        row["decode_ratio"] = round(row["layered"]["decode_tok_s"] / row["flat"]["decode_tok_s"], 3)
+        out.append(row)
+    return out
+
+
+def peaks():
+    p = os.path.join(os.path.dirname(os.path.dirname(os.path.dirname(os.path.abspath(__file__)))), "MEASURED_PEAKS.json")
+    if os.path.exists(p):
+        with open(p) as f:
+            d = json.load(f)
+        return d["hbm_gbs"] * 1e9, d["bf16_tflops"] * 1e12
+    return 6.65e12, 1.59e15
+
+
+@torch.no_grad()
+def kernel_table(size="base", batch=64, prompt=1024, n_prompts=8, iters=20):
+    """Time of every mixer kernel alone (cold L2) and the fraction of its roofline: the larger of bytes / measured copy
+    bandwidth and operations / measured bf16 GEMM throughput, over the time."""
+    from ..models.configuration import ModelArch
+    from ..models.decoder import SeqCtx
+    from ..models.hf_io import build_model
+    from ..ops import cuda as K
+    from ..ops import cuda_mixers as KM
+    from ..ops import mixers as mx
+    from ..rollout.engine import make_engine
+
+    bw, fl = peaks()
+    s = dict(SIZES[size], pairs=1)
+    model = build_model(ModelArch.from_hf_dict(layered_config(**s)), dtype=torch.bfloat16, device="cuda").eval().requires_grad_(False)
+    eng = make_engine(model, max_num_seqs=batch, max_model_len=prompt + 64)
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device="cuda")
+    rows = []
+
+    def row(name, fn, nbytes, flops=0.0):
+        for _ in range(3):
+            fn()
+        ev = []
+        for _ in range(iters):
+            flush.zero_()
+            a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            a.record()
+            fn()
+            b.record()
+            ev.append((a, b))
+        torch.cuda.synchronize()
+        us = sorted(a.elapsed_time(b) * 1e3 for a, b in ev)[iters // 2]
+        roof = max(nbytes / bw, flops / fl) * 1e6
+        rows.append(dict(kernel=name, us=round(us, 1), roof_us=round(roof, 2), frac=round(roof / us, 3)))
+
+    la, ml = model.layers[0].mixer, model.layers[1].mixer
+    T, W, dev, bf = n_prompts * prompt, s["width"], "cuda", torch.bfloat16
+    ctx = SeqCtx.from_lengths([prompt] * n_prompts, dev)
+    h = torch.randn(T, W, device=dev, dtype=bf)
+    x, d = torch.randn(T, W, device=dev), torch.randn(T, W, device=dev)
+    nrm = model.norm
+    row("prompt dynamic_tanh + residual", lambda: KM.dynamic_tanh(x, d, nrm.alpha, nrm.weight, nrm.bias, bf), T * W * 14)
+    acc = mx.linear_f32(h, la.w_in)
+    kr, lw = KM.latent_row(la.kv_rank, la.rot_dim)
+    lat = torch.zeros(T, lw, device=dev, dtype=bf)
+    table = la.rope.table(prompt, dev)
+    row("prompt latent_prep", lambda: KM.latent_prep(acc, la, ctx.positions, table, lat=lat),
+        T * (acc.shape[1] * 4 + (la.q_rank + lw) * 2 + la.heads * 4))
+    cq, gate = KM.latent_prep(acc, la, ctx.positions, table, lat=lat)
+    q, kv = mx.linear(cq, la.uq), mx.linear(lat[:, : la.kv_rank], la.ukv)
+    row("prompt rotate_q", lambda: KM.rotate_q(q, la, ctx.positions, table), T * la.heads * la.rot_dim * 4)
+    win = min(la.window or prompt, prompt)
+    pairs = n_prompts * (win * (win + 1) / 2 + (prompt - win) * win)
+    row("prompt latent attention", lambda: KM.latent_prompt_tc(q, kv, lat, la, ctx.cu_seqlens, gate),
+        (q.numel() + kv.numel() + lat.numel() + T * la.heads * la.vdim) * 2,
+        2 * pairs * la.heads * (la.dim + la.rot_dim + la.vdim))
+    y = mx.linear(h, ml.w_in[: ml.gate_row])
+    z = mx.linear_f32(h, ml.w_in[ml.gate_row:])
+    ig, fg = KM.mlstm_gates(z, ml.gate_bias, ml.cap, ml.heads)
+    row("prompt mlstm_gates", lambda: KM.mlstm_gates(z, ml.gate_bias, ml.cap, ml.heads), z.numel() * 8)
+    qkv = ml.heads * (2 * ml.dim + ml.vdim)
+    chunks = T // 128
+    row("prompt mlstm chunk (scan + states + outputs)", lambda: KM.mlstm_chunk(y, ml, ig, fg, ctx.cu_seqlens),
+        T * (qkv * 2 + ml.heads * ml.vdim * 4),
+        2 * T * ml.heads * (2 * ml.dim * ml.vdim + 64 * (ml.dim + ml.vdim)))
+    o32 = KM.mlstm_chunk(y, ml, ig, fg, ctx.cu_seqlens)
+    yo = torch.empty(T, ml.heads * ml.vdim, device=dev, dtype=bf)
+    row("prompt mlstm_out", lambda: KM.mlstm_out(o32, y[:, qkv:], ml, yo), o32.numel() * 8)
+    up = torch.randn(T, s["ff"], device=dev, dtype=bf)
+    row("prompt gelu", lambda: KM.gelu_erf(up), up.numel() * 4)
+    del up, y, q, kv, o32
+
+    eng.seq_lens.fill_(prompt)
+    eng.block_table.copy_(torch.arange(eng.block_table.numel(), device=dev).view_as(eng.block_table).remainder(eng.num_blocks))
+    a, r, B = eng.slots[0], eng.slots[1], batch
+    hb = torch.randn(B, W, device=dev, dtype=bf)
+    xb, db = torch.randn(B, W, device=dev), torch.randn(B, W, device=dev)
+    row("decode dynamic_tanh + residual", lambda: KM.dynamic_tanh(xb, db, nrm.alpha, nrm.weight, nrm.bias, bf, clear=True, out=hb), B * W * 18)
+    row("decode gemm input latent", lambda: K.decode_gemm(hb, la.w_in, y32=a.acc_in), la.w_in.numel() * 2)
+    row("decode latent_prep", lambda: KM.latent_prep(a.acc_in, la, eng.seq_lens, a.table, clear=True, cq=a.cq, gate=a.gate,
+                                                     cache=a.cache, block_table=eng.block_table, block_size=eng.block_size),
+        B * la.w_in.shape[0] * 8)
+    row("decode gemm query up", lambda: K.decode_gemm(a.cq, la.uq, y32=a.acc_q), la.uq.numel() * 2)
+    row("decode absorb", lambda: KM.latent_absorb(a.acc_q, la, eng.seq_lens, a.table, a.q_lat, True),
+        la.uk.numel() * 2 + a.acc_q.numel() * 8 + a.q_lat.numel() * 2, 2 * B * la.heads * la.dim * la.kv_rank)
+    n = min(prompt + 1, la.window or prompt + 1)
+    row("decode latent attention", lambda: a.attend(),
+        B * n * lw * 2 + (a.q_lat.numel() + a.o_lat.numel()) * 2, 2 * B * n * la.heads * (lw + la.kv_rank))
+    row("decode expand", lambda: KM.latent_expand(a.o_lat, la, a.gate, eng.seq_lens, a.o), la.uv.numel() * 2 + (a.o_lat.numel() + a.o.numel()) * 2,
+        2 * B * la.heads * la.vdim * la.kv_rank)
+    row("decode gemm input mlstm", lambda: K.decode_gemm(hb, ml.w_in, y32=r.acc_in), ml.w_in.numel() * 2)
+    row("decode mlstm_step", lambda: KM.mlstm_step(r.acc_in, ml, eng.seq_lens, r.state, r.o32),
+        r.state[0].numel() * 8 + r.acc_in.numel() * 4 + r.o32.numel() * 4)
+    row("decode mlstm_out", lambda: KM.mlstm_out(r.o32, r.acc_in[:, qkv:], ml, r.y, clear=r.acc_in), r.acc_in.numel() * 4 + r.o32.numel() * 8)
+    mlp = model.layers[0].mlp
+    row("decode up + gelu", lambda: eng._up_gelu(hb, mlp), mlp.up.numel() * 2)
+    K.check_status()
+    rows += flat_kernels(s, batch, prompt, n_prompts, row, rows)
+    return rows
+
+
+def flat_kernels(s, batch, prompt, n_prompts, row, rows):
+    """The like kernels of the flat decoder, timed the same way."""
+    from ..ops import cuda as K
+
+    dev, bf, T, W = "cuda", torch.bfloat16, n_prompts * prompt, s["width"]
+    Hq, Hk, D = W // 128, max(1, W // 512), 128
+    q, k, v = (torch.randn(T, n, D, device=dev, dtype=bf) for n in (Hq, Hk, Hk))
+    cu = torch.arange(0, T + 1, prompt, dtype=torch.int32, device=dev)
+    pairs = n_prompts * prompt * (prompt + 1) / 2
+    row("flat: prompt flash attention", lambda: K.fa_varlen_fwd(q, k, v, cu, cu), (2 * q.numel() + 2 * k.numel()) * 2, 4 * pairs * Hq * D)
+    res, dl, w = (torch.randn(T, W, device=dev, dtype=bf), torch.randn(T, W, device=dev, dtype=bf), torch.ones(W, device=dev, dtype=bf))
+    row("flat: prompt add + rmsnorm", lambda: K.add_rmsnorm_infer(res, dl, w, 1e-5), T * W * 8)
+    gu = torch.randn(T, 2 * s["ff"], device=dev, dtype=bf)
+    row("flat: prompt swiglu", lambda: K.swiglu_infer(gu), gu.numel() * 3)
+    pages = batch * (prompt // 64 + 1)
+    kc = torch.randn(pages, 64, Hk, D, device=dev, dtype=bf)
+    vc = torch.randn(pages, Hk, D, 64, device=dev, dtype=bf)
+    bt = torch.arange(pages, dtype=torch.int32, device=dev).view(batch, -1)
+    sl = torch.full((batch,), prompt - 1, dtype=torch.int32, device=dev)
+    splits = max(1, min(8, 148 // (batch * Hk)))
+    po = torch.empty(batch * Hq * splits * D, device=dev)
+    pm = torch.empty(batch * Hq * splits * 2, device=dev)
+    qd, od = torch.randn(batch, Hq, D, device=dev, dtype=bf), torch.empty(batch, Hq, D, device=dev, dtype=bf)
+    row("flat: decode attention", lambda: K.paged_decode_attn_tc(qd, kc, vc, sl, None, bt, D ** -0.5, splits, po, pm, od),
+        batch * prompt * Hk * D * 4, 4 * batch * prompt * Hq * D)
+    x, acc = torch.randn(batch, W, device=dev, dtype=bf), torch.zeros(batch, W, device=dev)
+    row("flat: decode add + rmsnorm", lambda: K.add_rmsnorm_f32_infer(x, acc, w, 1e-5), batch * W * 14)
+    qkv_w = torch.randn((Hq + 2 * Hk) * D, W, device=dev, dtype=bf)
+    aq = torch.zeros(batch, qkv_w.shape[0], device=dev)
+    row("flat: decode gemm qkv", lambda: K.decode_gemm(x, qkv_w, y32=aq), qkv_w.numel() * 2)
+    row("flat: decode rope + kv write", lambda: K.rope_kv_write_f32(aq, None, None, None, 1e-5, sl, None, bt, 64, qd, kc, vc, Hq, Hk, D, 5e5,
+                                                                    v_transposed=True), aq.numel() * 10)
+    gw = torch.randn(2 * s["ff"], W, device=dev, dtype=bf)
+    act = torch.empty(batch, s["ff"], device=dev, dtype=bf)
+    row("flat: decode gate/up + swiglu", lambda: K.decode_gemm(x, gw, out=act, swiglu=True), gw.numel() * 2)
+    K.check_status()
+    return []
+
+
+def main():
+    ap = argparse.ArgumentParser()
+    ap.add_argument("--sizes", default="small,base")
+    ap.add_argument("--batch", type=int, default=64)
+    ap.add_argument("--prompt", type=int, default=1024)
+    ap.add_argument("--prompts", type=int, default=8)
+    ap.add_argument("--kernels", action="store_true")
+    a = ap.parse_args()
+    if a.kernels:
+        for r in kernel_table(a.sizes.split(",")[-1], a.batch, a.prompt, a.prompts):
+            print(json.dumps(r))
+        return
+    for r in run(a.sizes.split(","), a.batch, a.prompt, a.prompts):
+        print(json.dumps(r))
+
+
+if __name__ == "__main__":
+    main()

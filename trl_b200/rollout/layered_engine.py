@@ -51,6 +51,13 @@ class _LatentSlots:
     def copy_slots(self, dst, src):
         pass
 
+    def attend(self):
+        """Absorbed queries against the cached latent rows -> ``o_lat``."""
+        from ..ops import cuda_mixers as K
+
+        e = self.e
+        K.latent_decode(self.q_lat, self.cache, self.m, e.seq_lens, e.block_table, e.block_size, self.o_lat)
+
     def step(self, h, out):
         from ..ops import cuda_mixers as K
 
@@ -60,7 +67,7 @@ class _LatentSlots:
                       block_table=e.block_table, block_size=e.block_size)
         e.gemm(self.cq, m.uq, self.acc_q)
         K.latent_absorb(self.acc_q, m, e.seq_lens, self.table, self.q_lat, True)
-        K.latent_decode(self.q_lat, self.cache, m, e.seq_lens, e.block_table, e.block_size, self.o_lat)
+        self.attend()
         K.latent_expand(self.o_lat, m, self.gate, e.seq_lens, self.o)
         e.gemm(self.o, m.o, out)
 
