@@ -320,16 +320,82 @@ def test_far_key_and_window_edge_in_decode():
             cache[:, :, r:off] = 0
             cache[:, :, off + dr:] = 0
             out = torch.full((2, heads, r), 9.0, dtype=dtype, device="cuda")
-            K.latent_decode(dev(q, dtype), dev(cache, dtype), m, torch.tensor([-1, pos], dtype=torch.int32, device="cuda"),
-                            table.cuda(), bs, out)
+            args = (dev(q, dtype), dev(cache, dtype), m, torch.tensor([-1, pos], dtype=torch.int32, device="cuda"), table.cuda(), bs)
+            K.latent_decode(*args, out)
+            outs = [out]
+            m.dim, m.vdim = 8, 8
+            hg = K.latent_decode_tc_heads(m, bs)
+            assert hg == (64 if heads > 32 else 32)
+            for splits in (1, 2, 3) if dtype == torch.bfloat16 else ():
+                outs.append(torch.full((2, heads, r), 9.0, dtype=dtype, device="cuda"))
+                scratch = torch.full((2, heads * splits * r), 5.0, device="cuda")
+                K.latent_decode_tc(*args, outs[-1], scratch, torch.full((2, heads * splits * 2), 5.0, device="cuda"), hg, splits)
             a = max(0, pos - window + 1)
             s = q[1] @ lat[a:].T
             p = s.exp() / (s.exp().sum(-1, keepdim=True) + torch.exp(torch.tensor(-4.0, dtype=torch.float64)))
             want = p @ lat[a:, :r]
-            got = out[1].double().cpu()
-            assert (got - want).abs().max() < (1e-5 if dtype == torch.float32 else 1e-2) * want.abs().max(), (heads, pos, target)
-            near = (got - lat[pos - target, :r]).abs().max() < 0.1 * lat[pos - target, :r].abs().max()
-            assert bool(near) == (target < window)
+            for out in outs:
+                got = out[1].double().cpu()
+                assert (got - want).abs().max() < (1e-5 if dtype == torch.float32 else 1e-2) * want.abs().max(), (heads, pos, target)
+                near = (got - lat[pos - target, :r]).abs().max() < 0.1 * lat[pos - target, :r].abs().max()
+                assert bool(near) == (target < window)
+
+
+@pytest.mark.parametrize("heads,r,dr,bs,window", [(5, 128, 64, 64, None), (32, 512, 64, 64, 300), (40, 96, 8, 16, 129), (64, 72, 40, 32, 128),
+                                                  (100, 256, 32, 128, None), (2, 8, 8, 8, 1)])
+def test_tensor_core_decode_attention(heads, r, dr, bs, window):
+    """Ragged slots (idle ones included), several tiles and splits, scores large enough to move the reference maximum."""
+    from trl_b200.ops import cuda_mixers as K
+
+    lens = [0, 700, -1, 127, 128, 5, 300]
+    B, off = len(lens), K.latent_row(r, dr)[0]
+    w = K.latent_row(r, dr)[1]
+    g = torch.Generator().manual_seed(heads)
+    m = types.SimpleNamespace(heads=heads, kv_rank=r, rot_dim=dr, dim=8, vdim=8, window=window, scale=0.3,
+                              sink=torch.randn(heads, generator=g).cuda())
+    pages = -(-701 // bs)
+    table = (torch.randperm(B * pages, generator=g) + 1).view(B, pages).int()
+    cache = torch.randn(B * pages + 1, bs, w, generator=g, dtype=torch.float64)
+    cache[:, :, r:off] = 0
+    cache[:, :, off + dr:] = 0
+    q = torch.randn(B, heads, w, generator=g, dtype=torch.float64) * (2.0 / w ** 0.5) * 8
+    q[:, :, r:off] = 0
+    q[:, :, off + dr:] = 0
+    cache, q = cache.bfloat16().double(), q.bfloat16().double()
+    hg = K.latent_decode_tc_heads(m, bs)
+    assert hg
+    for splits in (1, 3):
+        out = torch.zeros(B, heads, r, dtype=torch.bfloat16, device="cuda")
+        K.latent_decode_tc(dev(q, torch.bfloat16), dev(cache, torch.bfloat16), m, torch.tensor(lens, dtype=torch.int32, device="cuda"),
+                           table.cuda(), bs, out, torch.full((B, heads * splits * r), 5.0, device="cuda"),
+                           torch.full((B, heads * splits * 2), 5.0, device="cuda"), hg, splits)
+        for b, pos in enumerate(lens):
+            if pos < 0:
+                assert not out[b].any()
+                continue
+            rows = torch.cat([cache[int(x)] for x in table[b]])[max(0, pos - window + 1) if window else 0:pos + 1]
+            s = q[b] @ rows.T * m.scale
+            top = torch.maximum(s.amax(-1), m.sink.double().cpu())
+            e = (s - top[:, None]).exp()
+            want = e @ rows[:, :r] / (e.sum(-1) + (m.sink.double().cpu() - top).exp())[:, None]
+            assert (out[b].double().cpu() - want).abs().max() < 1e-2 * max(1.0, float(want.abs().max())), (b, splits)
+
+
+@pytest.mark.parametrize("B", [1, 17, 64, 128, 130])
+@pytest.mark.parametrize("H,M,Kd", [(3, 128, 64), (2, 200, 40), (1, 16, 520)])
+@pytest.mark.parametrize("w_mn", [False, True])
+def test_head_gemm(B, H, M, Kd, w_mn):
+    from trl_b200.ops import cuda_mixers as K
+
+    g = torch.Generator().manual_seed(B + M)
+    x = torch.randn(B, H, Kd + 8, generator=g).bfloat16().cuda()
+    w = torch.randn(*((H, Kd, M) if w_mn else (H, M, Kd)), generator=g).bfloat16().cuda()
+    sc = torch.rand(B, H, generator=g).cuda()
+    y = torch.zeros(B, H, M + 24, dtype=torch.bfloat16, device="cuda")
+    K.head_gemm(x, w, y, w_mn=w_mn, scale=sc)
+    want = torch.einsum("bhk,hkm->bhm" if w_mn else "bhk,hmk->bhm", x[..., :Kd].double(), w.double()) * sc.double()[..., None]
+    assert torch.allclose(y[..., :M].double(), want, rtol=1e-2, atol=1e-2 * Kd ** 0.5)
+    assert not y[..., M:].any()
 
 
 @pytest.mark.parametrize("graph", [True, False])

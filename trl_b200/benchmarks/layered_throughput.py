@@ -204,12 +204,12 @@ def kernel_table(size="base", batch=64, prompt=1024, n_prompts=8, iters=20):
                                                      cache=a.cache, block_table=eng.block_table, block_size=eng.block_size),
         B * la.w_in.shape[0] * 8)
     row("decode gemm query up", lambda: K.decode_gemm(a.cq, la.uq, y32=a.acc_q), la.uq.numel() * 2)
-    row("decode absorb", lambda: KM.latent_absorb(a.acc_q, la, eng.seq_lens, a.table, a.q_lat, True),
+    row("decode absorb", a.absorb,
         la.uk.numel() * 2 + a.acc_q.numel() * 8 + a.q_lat.numel() * 2, 2 * B * la.heads * la.dim * la.kv_rank)
     n = min(prompt + 1, la.window or prompt + 1)
-    row("decode latent attention", lambda: a.attend(),
+    row("decode latent attention", a.attend,
         B * n * lw * 2 + (a.q_lat.numel() + a.o_lat.numel()) * 2, 2 * B * n * la.heads * (lw + la.kv_rank))
-    row("decode expand", lambda: KM.latent_expand(a.o_lat, la, a.gate, eng.seq_lens, a.o), la.uv.numel() * 2 + (a.o_lat.numel() + a.o.numel()) * 2,
+    row("decode expand", a.expand, la.uv.numel() * 2 + (a.o_lat.numel() + a.o.numel()) * 2,
         2 * B * la.heads * la.vdim * la.kv_rank)
     row("decode gemm input mlstm", lambda: K.decode_gemm(hb, ml.w_in, y32=r.acc_in), ml.w_in.numel() * 2)
     row("decode mlstm_step", lambda: KM.mlstm_step(r.acc_in, ml, eng.seq_lens, r.state, r.o32),

@@ -131,6 +131,51 @@ def latent_expand(o_lat, m, gate, positions, out):
                                   c_int(m.kv_rank), _p(positions), _b(out), _s()), "latent_expand")
 
 
+def latent_decode_tc_heads(m, block_size: int) -> int:
+    """Heads per CTA of :func:`latent_decode_tc` for a mixer's sizes; 0: the CUDA-core kernels serve it."""
+    _, w = latent_row(m.kv_rank, m.rot_dim)
+    if m.scale <= 0:
+        return 0
+    return int(lib().trlb_latent_decode_tc_heads(c_int(m.heads), c_int(m.dim), c_int(m.rot_dim), c_int(m.vdim),
+                                                 c_int(m.kv_rank), c_int(w), c_int(block_size)))
+
+
+def latent_decode_tc(q_lat, cache, m, seq_lens, block_table, block_size, o_lat, part_o, part_ml, hg, splits):
+    """:func:`latent_decode` on the tensor cores (bf16).  ``part_o`` [>= B heads splits kv_rank] and ``part_ml`` [>= 2 B heads
+    splits] fp32 scratch."""
+    B = q_lat.shape[0]
+    _, w = latent_row(m.kv_rank, m.rot_dim)
+    assert q_lat.dtype == torch.bfloat16 and cache.is_contiguous() and cache.shape[1] == block_size and cache.shape[2] == w
+    assert part_o.numel() >= B * m.heads * splits * m.kv_rank and part_ml.numel() >= 2 * B * m.heads * splits
+    _chk(lib().trlb_latent_decode_tc(_p(q_lat), _p(cache), c_int(cache.shape[0]), c_int(B), c_int(m.heads), c_int(m.kv_rank),
+                                     c_int(w), c_int(hg), c_int(m.window or 0), c_float(m.scale), _p(seq_lens),
+                                     _p(block_table), c_int(block_table.shape[1]), c_int(block_size), _p(m.sink),
+                                     c_int(splits), _p(part_o), _p(part_ml), _p(o_lat), _p(status_buffer(q_lat.device)), _s()),
+         "latent_decode_tc")
+
+
+def latent_query(qacc, m, positions, table, q, q_lat):
+    """fp32 query sums (cleared) -> bf16 ``q`` and the rotated part of ``q_lat``."""
+    B = qacc.shape[0]
+    kr, w = latent_row(m.kv_rank, m.rot_dim)
+    _chk(lib().trlb_latent_query(_p(qacc), c_longlong(qacc.stride(0)), _p(q), _p(q_lat), c_int(B), c_int(m.heads), c_int(m.dim),
+                                 c_int(m.rot_dim), c_int(kr), c_int(w), _p(positions), _p(table), c_int(table.shape[0]), _s()),
+         "latent_query")
+
+
+def head_gemm(x, w, y, *, w_mn: bool = False, scale=None):
+    """``y[b, h] = scale[b, h] * x[b, h] w[h]^T`` per head: x [B, heads, >= K] (last dim dense), w [heads, M, K], or [heads, K,
+    M] with ``w_mn`` (read MN-major, nothing is transposed in memory); y [B, heads, >= M] bf16."""
+    (B, H), (_, a, b) = x.shape[:2], w.shape
+    M, Kd = (b, a) if w_mn else (a, b)
+    assert x.dtype == y.dtype == w.dtype == torch.bfloat16 and w.is_contiguous() and x.stride(2) == 1 and y.stride(2) == 1
+    assert x.shape[2] >= Kd and y.shape[2] >= M and (scale is None or (scale.is_contiguous() and scale.shape == (B, H)))
+    _chk(lib().trlb_head_gemm(_p(x), c_longlong(x.stride(0)), c_longlong(x.stride(1)), _p(w), c_int(int(w_mn)), _p(y),
+                              c_longlong(y.stride(0)), c_longlong(y.stride(1)), _p(scale), c_int(B), c_int(H), c_int(M),
+                              c_int(Kd), _p(status_buffer(x.device)), _s()), "head_gemm")
+    return y
+
+
 def mlstm_gates(z, bias, cap, heads):
     T = z.shape[0]
     assert z.is_contiguous()

@@ -41,6 +41,15 @@ class _LatentSlots:
         self.q_lat = eng.scratch("q_lat", B, m.heads, self.width)
         self.o_lat = eng.scratch("o_lat", B, m.heads, m.kv_rank)
         self.o = eng.scratch("o", B, m.heads * m.vdim)
+        # tensor-core decode: heads per CTA (0: sizes or dtype that only the CUDA-core kernels take)
+        self.hg = K.latent_decode_tc_heads(m, eng.block_size) if eng.dtype == torch.bfloat16 else 0
+        if self.hg:
+            tiles = -(-(m.window or eng.max_len) // 128) + 1
+            ctas = B * -(-m.heads // self.hg)
+            self.splits = max(1, min(8, tiles, 148 // ctas))
+            self.q = eng.scratch("q", B, m.heads, m.dim + m.rot_dim)
+            self.part_o = eng.scratch("part_o", B, m.heads * self.splits * m.kv_rank, dtype=torch.float32)
+            self.part_ml = eng.scratch("part_ml", B, m.heads * self.splits * 2, dtype=torch.float32)
 
     def prompt_target(self, pages: "_Pages") -> dict:
         return dict(cache=self.cache, tok_slot=pages.tok_slot, block_table=self.e.block_table, block_size=self.e.block_size)
@@ -56,7 +65,32 @@ class _LatentSlots:
         from ..ops import cuda_mixers as K
 
         e = self.e
-        K.latent_decode(self.q_lat, self.cache, self.m, e.seq_lens, e.block_table, e.block_size, self.o_lat)
+        if self.hg:
+            K.latent_decode_tc(self.q_lat, self.cache, self.m, e.seq_lens, e.block_table, e.block_size, self.o_lat,
+                               self.part_o, self.part_ml, self.hg, self.splits)
+        else:
+            K.latent_decode(self.q_lat, self.cache, self.m, e.seq_lens, e.block_table, e.block_size, self.o_lat)
+
+    def absorb(self):
+        """``acc_q`` -> queries in the latent basis, ``q_lat``."""
+        from ..ops import cuda_mixers as K
+
+        e, m = self.e, self.m
+        if self.hg:
+            K.latent_query(self.acc_q, m, e.seq_lens, self.table, self.q, self.q_lat)
+            K.head_gemm(self.q, m.uk.view(m.heads, m.dim, m.kv_rank), self.q_lat, w_mn=True)
+        else:
+            K.latent_absorb(self.acc_q, m, e.seq_lens, self.table, self.q_lat, True)
+
+    def expand(self):
+        """``o_lat`` -> gated head outputs, ``o``."""
+        from ..ops import cuda_mixers as K
+
+        m = self.m
+        if self.hg:
+            K.head_gemm(self.o_lat, m.uv.view(m.heads, m.vdim, m.kv_rank), self.o.view(-1, m.heads, m.vdim), scale=self.gate)
+        else:
+            K.latent_expand(self.o_lat, m, self.gate, self.e.seq_lens, self.o)
 
     def step(self, h, out):
         from ..ops import cuda_mixers as K
@@ -66,9 +100,9 @@ class _LatentSlots:
         K.latent_prep(self.acc_in, m, e.seq_lens, self.table, clear=True, cq=self.cq, gate=self.gate, cache=self.cache,
                       block_table=e.block_table, block_size=e.block_size)
         e.gemm(self.cq, m.uq, self.acc_q)
-        K.latent_absorb(self.acc_q, m, e.seq_lens, self.table, self.q_lat, True)
+        self.absorb()
         self.attend()
-        K.latent_expand(self.o_lat, m, self.gate, e.seq_lens, self.o)
+        self.expand()
         e.gemm(self.o, m.o, out)
 
 
