@@ -324,12 +324,11 @@ def test_far_key_and_window_edge_in_decode():
             K.latent_decode(*args, out)
             outs = [out]
             m.dim, m.vdim = 8, 8
-            hg = K.latent_decode_tc_heads(m, bs)
-            assert hg == (64 if heads > 32 else 32)
+            assert K.latent_decode_tc_ok(m, bs)
             for splits in (1, 2, 3) if dtype == torch.bfloat16 else ():
                 outs.append(torch.full((2, heads, r), 9.0, dtype=dtype, device="cuda"))
                 scratch = torch.full((2, heads * splits * r), 5.0, device="cuda")
-                K.latent_decode_tc(*args, outs[-1], scratch, torch.full((2, heads * splits * 2), 5.0, device="cuda"), hg, splits)
+                K.latent_decode_tc(*args, outs[-1], scratch, torch.full((2, heads * splits * 2), 5.0, device="cuda"), splits)
             a = max(0, pos - window + 1)
             s = q[1] @ lat[a:].T
             p = s.exp() / (s.exp().sum(-1, keepdim=True) + torch.exp(torch.tensor(-4.0, dtype=torch.float64)))
@@ -362,13 +361,12 @@ def test_tensor_core_decode_attention(heads, r, dr, bs, window):
     q[:, :, r:off] = 0
     q[:, :, off + dr:] = 0
     cache, q = cache.bfloat16().double(), q.bfloat16().double()
-    hg = K.latent_decode_tc_heads(m, bs)
-    assert hg
+    assert K.latent_decode_tc_ok(m, bs)
     for splits in (1, 3):
         out = torch.zeros(B, heads, r, dtype=torch.bfloat16, device="cuda")
         K.latent_decode_tc(dev(q, torch.bfloat16), dev(cache, torch.bfloat16), m, torch.tensor(lens, dtype=torch.int32, device="cuda"),
                            table.cuda(), bs, out, torch.full((B, heads * splits * r), 5.0, device="cuda"),
-                           torch.full((B, heads * splits * 2), 5.0, device="cuda"), hg, splits)
+                           torch.full((B, heads * splits * 2), 5.0, device="cuda"), splits)
         for b, pos in enumerate(lens):
             if pos < 0:
                 assert not out[b].any()

@@ -137,7 +137,8 @@ def kernel_table(size="base", batch=64, prompt=1024, n_prompts=8, iters=20):
     s = dict(SIZES[size], pairs=1)
     model = build_model(ModelArch.from_hf_dict(layered_config(**s)), dtype=torch.bfloat16, device="cuda").eval().requires_grad_(False)
     eng = make_engine(model, max_num_seqs=batch, max_model_len=prompt + 64)
-    flush = torch.empty(256 << 20, dtype=torch.uint8, device="cuda")
+    # larger than L2, and long enough that the host has launched everything of an iteration before the first event
+    flush = torch.empty(2 << 30, dtype=torch.uint8, device="cuda")
     rows = []
 
     def row(name, fn, nbytes, flops=0.0):

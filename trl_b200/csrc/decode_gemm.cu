@@ -32,7 +32,7 @@
 //
 // Stands where the reference's rollout backend (vLLM, trl/generation/vllm_generation.py:351-368,636-699) runs its
 // decode linears; the reference tree itself has no such kernel.
-#include "common.cuh"
+#include "mixers.cuh"
 
 namespace trlb {
 
@@ -41,7 +41,7 @@ constexpr int DG_THREADS = 192;
 constexpr uint32_t DG_W_BYTES = DG_BM * DG_BK * 2;
 constexpr int DG_MAX_PEERS = 7;
 
-enum { DG_ACCUM_F32 = 0, DG_STORE_BF16 = 1, DG_SWIGLU = 2 };
+enum { DG_ACCUM_F32 = 0, DG_STORE_BF16 = 1, DG_SWIGLU = 2, DG_GELU = 3 };
 
 struct DecodeGemmParams {
   int B, N, K;
@@ -51,7 +51,7 @@ struct DecodeGemmParams {
   int steps_per_slab;  // k_blocks (x 2 with SwiGLU: gate step, up step)
   int up_slab_offset;  // SwiGLU: the up slab of features [128 j, 128 j + 128) is slab j + up_slab_offset of W
   float* Y32;          // DG_ACCUM_F32: [B, ldy] fp32, added to
-  __nv_bfloat16* Yb;   // DG_STORE_BF16 / DG_SWIGLU: [B, ldy] bf16
+  __nv_bfloat16* Yb;   // DG_STORE_BF16 / DG_SWIGLU / DG_GELU: [B, ldy] bf16
   long long ldy;
   const __nv_bfloat16* bias;  // [N] or null (not with SwiGLU)
   int* status;
@@ -296,7 +296,7 @@ decode_gemm_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_cons
           __nv_bfloat16* dst = p.Yb + off;
 #pragma unroll
           for (int i = 0; i < 16; ++i) {
-            if (i < rows) *dst = __float2bfloat16(v[i] + bias);
+            if (i < rows) *dst = __float2bfloat16(p.mode == DG_GELU ? gelu_erf_f(v[i] + bias) : v[i] + bias);
             dst += p.ldy;
           }
         }
@@ -381,6 +381,7 @@ int dg_launch(const CUtensorMap& tw, const CUtensorMap& tx, const DecodeGemmPara
 }
 
 int dg_ctas_per_sm(int B, int mode) {
+  if (mode == DG_GELU) return 1;
   if (B > 64) return (mode == DG_SWIGLU || g_ctas_per_sm < 2) ? 1 : 2;  // 128-row tiles: 256 / 512 TMEM columns each
   if (mode == DG_SWIGLU) return 1;  // SwiGLU slabs cannot be split along K: one CTA per SM with a deep ring
   return g_ctas_per_sm;
@@ -420,6 +421,7 @@ TRLB_API int trlb_decode_gemm_arrivals(int N) { return 4 * ((N + DG_BM - 1) / DG
 // [ceil(rows/128)][ceil(K/64)][128][64] as written by trlb_tile_weights.
 //   mode 0  W [N, K];  Y32 [B, N] fp32 (row stride ldy) is added to (+ bias once): the caller provides zeros
 //   mode 1  W [N, K];  Yb  [B, N] bf16 = X W^T (+ bias)
+//   mode 3  like mode 1 with the exact GELU of the sum stored
 //   mode 2  W [2N, K] (gate rows, then up rows; N a multiple of 128);  Yb [B, N] bf16 = silu(X Wg^T) * (X Wu^T)
 // max_ctas: 0 = every SM with its resident CTAs, else an upper bound on the grid.
 // Fused all-reduce (mode 0, n_peers > 0): peer_y32[i] is the same buffer on peer i; arrive[0] is this rank's arrival
@@ -432,7 +434,7 @@ TRLB_API int trlb_decode_gemm(const void* X, const void* W, const void* bias, fl
                               float* const* peer_y32, uint32_t* const* arrive, float* stage, uint32_t* slab_ctr,
                               int* status, cudaStream_t st) {
   if (B <= 0 || N <= 0 || K <= 0) return 0;
-  if (B > 128 || (K % 8) != 0 || (ldx % 8) != 0 || mode < 0 || mode > 2) return -150;
+  if (B > 128 || (K % 8) != 0 || (ldx % 8) != 0 || mode < 0 || mode > 3) return -150;
   if (!tiled && (ldw % 8) != 0) return -150;
   if (mode == DG_SWIGLU && (bias != nullptr || (N % DG_BM) != 0)) return -150;
   if (n_peers < 0 || n_peers > DG_MAX_PEERS || (n_peers > 0 && (mode != DG_ACCUM_F32 || !peer_y32 || !arrive))) return -150;
@@ -462,10 +464,12 @@ TRLB_API int trlb_decode_gemm(const void* X, const void* W, const void* bias, fl
   const int ctas = trlb_decode_gemm_ctas(B, N, K, mode, max_ctas);
   if (BN == 64) {
     if (mode == DG_SWIGLU) return dg_launch<64, true, 8, 1>(tw, tx, p, ctas, st);
+    if (mode == DG_GELU) return dg_launch<64, false, 8, 1>(tw, tx, p, ctas, st);  // one slab per CTA: a deep ring
     if (g_ctas_per_sm == 3) return dg_launch<64, false, 3, 3>(tw, tx, p, ctas, st);
     return dg_launch<64, false, 4, 2>(tw, tx, p, ctas, st);
   }
   if (mode == DG_SWIGLU) return dg_launch<128, true, 6, 1>(tw, tx, p, ctas, st);
+  if (mode == DG_GELU) return dg_launch<128, false, 6, 1>(tw, tx, p, ctas, st);
   if (g_ctas_per_sm < 2) return dg_launch<128, false, 6, 1>(tw, tx, p, ctas, st);
   return dg_launch<128, false, 3, 2>(tw, tx, p, ctas, st);
 }

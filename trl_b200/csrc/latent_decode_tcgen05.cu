@@ -2,7 +2,7 @@
 //
 // In absorbed form all heads of a slot attend to ONE row per token, [latent | rotated key], which is also the value (its
 // latent part).  The operands are swapped so that the tokens and the latent dimensions fill the 128 rows of an MMA and
-// the heads (32 or 64 per CTA) are its columns:
+// the heads (32 per CTA) are its columns:
 //
 //     S^T [128 tokens x heads]      = C [tokens x row]  Q^T            both K-major, straight from their TMA tiles
 //     O^T [128 dims x heads] (+)=     C^T [dims x tokens] P^T          the same tile of C read MN-major
@@ -11,8 +11,8 @@
 // when there are few heads.  One CTA per (slot, head group, split of the visible pages), 192 threads: TMA warp, MMA warp,
 // and one softmax thread per token of the 128-token tile.  Per-head maxima are formed with a shuffle reduce-scatter and
 // exchanged between the four warps; the reference maximum of a head moves (and O^T is rescaled) only when it is exceeded
-// by 2^8.  Probabilities keep 32-bit precision: they go to shared memory as two bf16 (value and remainder), and both
-// products accumulate.  A tile's 64-column boxes are released slab by slab as O^T consumes them, so the next tile streams
+// by 2^8.  Probabilities keep 32-bit precision: they go to shared memory as two bf16 (value and remainder) that are
+// separate columns of the second product, so the tile of C is read once for both.  A tile's 64-column boxes are released slab by slab as O^T consumes them, so the next tile streams
 // in behind it.  Splits leave fp32 partial sums; latent_combine_kernel merges them with the softmax sink.
 #include "mixers.cuh"
 
@@ -48,17 +48,16 @@ __device__ __forceinline__ float reduce_scatter32(float (&x)[32], int lane) {
   return x[0];
 }
 
-template <int HG>
 __global__ void __launch_bounds__(192, 1)
 latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_c,
                         const LatentDecodeTc p) {
-  constexpr int HC = HG / 32;  // 32-head chunks
+  constexpr int HG = 32;  // heads per CTA
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   uint8_t* c_s = smem;                                            // [boxes] 128 tokens x 64 columns
   uint8_t* q_s = c_s + (size_t)p.boxes * LD_BOX;                  // [boxes] HG heads x 64 columns
-  uint8_t* p_s = q_s + (size_t)p.boxes * HG * 128;                // value and remainder: 128 tokens x 64 columns each
-  uint64_t* bars = reinterpret_cast<uint64_t*>(p_s + 2 * LD_BOX);
+  uint8_t* p_s = q_s + (size_t)p.boxes * HG * 128;                // 128 tokens x (32 values | 32 remainders)
+  uint64_t* bars = reinterpret_cast<uint64_t*>(p_s + LD_BOX);
   uint64_t* full = bars;                   // [LD_MAX_BOX]
   uint64_t* empty = full + LD_MAX_BOX;     // [LD_MAX_BOX]
   uint64_t* q_full = empty + LD_MAX_BOX;
@@ -113,14 +112,17 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
       for (int i = 0; i < p.boxes; ++i) tma_load_3d(q_s + (size_t)i * HG * 128, &tm_q, q_full, 64 * i, h0, b);
       bool ok = true;
       for (int j = 0; j < n_t && ok; ++j) {
+        int rows[16];  // pages past the sequence's last one are masked: any page that exists will do
+#pragma unroll
+        for (int g = 0; g < 16; ++g)
+          rows[g] = g < ppt ? bt[min(page0 + (t_beg + j) * ppt + g, pos / p.block_size)] * p.block_size : 0;
         for (int i = 0; i < p.boxes; ++i) {
           if (!mbar_wait(&empty[i], (uint32_t)((j & 1) ^ 1), abort_flag, p.status, 1500 + i)) { ok = false; break; }
           mbar_expect_tx(&full[i], LD_BOX);
-          for (int g = 0; g < ppt; ++g) {
-            // pages past the sequence's last one are masked: any page that exists will do
-            const int blk = bt[min(page0 + (t_beg + j) * ppt + g, pos / p.block_size)];
-            tma_load_2d(c_s + (size_t)i * LD_BOX + (size_t)g * p.block_size * 128, &tm_c, &full[i], 64 * i, blk * p.block_size);
-          }
+#pragma unroll
+          for (int g = 0; g < 16; ++g)
+            if (g < ppt)
+              tma_load_2d(c_s + (size_t)i * LD_BOX + (size_t)g * p.block_size * 128, &tm_c, &full[i], 64 * i, rows[g]);
         }
       }
     }
@@ -128,7 +130,7 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
   } else if (warp == 1) {
     if (lane == 0 && n_t > 0) {
       constexpr uint32_t idesc_s = umma_idesc_bf16_major(128, HG, false, false);
-      constexpr uint32_t idesc_o = umma_idesc_bf16_major(128, HG, true, true);
+      constexpr uint32_t idesc_o = umma_idesc_bf16_major(128, 2 * HG, true, true);
       const uint32_t c_u = smem_u32(c_s), q_u = smem_u32(q_s), p_u = smem_u32(p_s);
       bool ok = mbar_wait(q_full, 0, abort_flag, p.status, 1520);
       for (int j = 0; j < n_t && ok; ++j) {
@@ -146,13 +148,11 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
         if (!mbar_wait(p_full, (uint32_t)(j & 1), abort_flag, p.status, 1550)) break;
         tc_fence_after();
         for (int s = 0; s < p.slabs; ++s) {
-          for (int half = 0; half < 2; ++half)
 #pragma unroll
-            for (int kk = 0; kk < LD_TOK / 16; ++kk)
-              umma_bf16_ss(tmem_base + 64 + (uint32_t)(s * HG),
-                           umma_desc_mnmajor_sw128(c_u + (uint32_t)(2 * s) * LD_BOX + (uint32_t)kk * 2048, LD_BOX),
-                           umma_desc_mnmajor_sw128(p_u + (uint32_t)half * LD_BOX + (uint32_t)kk * 2048, LD_BOX), idesc_o,
-                           (j | half | kk) != 0);
+          for (int kk = 0; kk < LD_TOK / 16; ++kk)
+            umma_bf16_ss(tmem_base + 64 + (uint32_t)(s * 2 * HG),
+                         umma_desc_mnmajor_sw128(c_u + (uint32_t)(2 * s) * LD_BOX + (uint32_t)kk * 2048, LD_BOX),
+                         umma_desc_mnmajor_sw128(p_u + (uint32_t)kk * 2048, LD_BOX), idesc_o, (j | kk) != 0);
           umma_commit(&empty[2 * s]);
           umma_commit(&empty[2 * s + 1]);
         }
@@ -163,9 +163,7 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
   } else if (n_t > 0) {
     const int w4 = warp & 3, r = w4 * 32 + lane;
     const uint32_t ts = tmem_base + ((uint32_t)(w4 * 32) << 16), to = ts + 64;
-    float m_ref[HC], l[HG];
-#pragma unroll
-    for (int c = 0; c < HC; ++c) m_ref[c] = -INFINITY;
+    float m_ref = -INFINITY, l[HG];  // the reference maximum of head `lane`; per-head sums over this thread's tokens
 #pragma unroll
     for (int i = 0; i < HG; ++i) l[i] = 0.f;
     bool ok = true;
@@ -176,79 +174,62 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
       ok = __all_sync(0xffffffffu, mbar_wait(s_full, (uint32_t)(j & 1), abort_flag, p.status, 1560));
       if (!ok) break;
       tc_fence_after();
-      float v[HC][32];
-#pragma unroll
-      for (int c = 0; c < HC; ++c) tmem_ld_32x32(ts + 32 * c, v[c]);
+      float v[32], x[32];
+      tmem_ld_32x32(ts, v);
       tmem_ld_wait();
-      float* mine = red + (size_t)(j & 1) * 4 * HG;
 #pragma unroll
-      for (int c = 0; c < HC; ++c) {
-        float x[32];
-#pragma unroll
-        for (int i = 0; i < 32; ++i) {
-          v[c][i] = seen ? v[c][i] * p.scale_log2 : -INFINITY;
-          x[i] = v[c][i];
-        }
-        mine[w4 * HG + 32 * c + lane] = reduce_scatter32<true>(x, lane);
-      }
+      for (int i = 0; i < 32; ++i) x[i] = v[i] = seen ? v[i] * p.scale_log2 : -INFINITY;
+      float* mine = red + (j & 1) * 4 * HG;
+      mine[w4 * HG + lane] = reduce_scatter32<true>(x, lane);
       mbar_arrive(red_full);
       ok = __all_sync(0xffffffffu, mbar_wait(red_full, (uint32_t)(j & 1), abort_flag, p.status, 1570));
       if (!ok) break;
-      float alpha[HC], neg_m[HC];
+      const float mt = fmaxf(fmaxf(mine[lane], mine[HG + lane]), fmaxf(mine[2 * HG + lane], mine[3 * HG + lane]));
+      float alpha = 1.f;
       bool moved = false;
-#pragma unroll
-      for (int c = 0; c < HC; ++c) {
-        const int i = 32 * c + lane;
-        const float mt = fmaxf(fmaxf(mine[i], mine[HG + i]), fmaxf(mine[2 * HG + i], mine[3 * HG + i]));
-        alpha[c] = 1.f;
-        if (m_ref[c] == -INFINITY) {
-          m_ref[c] = mt;
-        } else if (mt > m_ref[c] + 8.f) {
-          alpha[c] = exp2f(m_ref[c] - mt);
-          m_ref[c] = mt;
-          moved = true;
-        }
-        neg_m[c] = m_ref[c] == -INFINITY ? 0.f : -m_ref[c];
+      if (m_ref == -INFINITY) {
+        m_ref = mt;
+      } else if (mt > m_ref + 8.f) {
+        alpha = exp2f(m_ref - mt);
+        m_ref = mt;
+        moved = true;
       }
+      const float neg_m = m_ref == -INFINITY ? 0.f : -m_ref;
       if (__any_sync(0xffffffffu, moved)) {  // the same in all four warps
 #pragma unroll
-        for (int i = 0; i < HG; ++i) l[i] *= __shfl_sync(0xffffffffu, alpha[i / 32], i & 31);
+        for (int i = 0; i < HG; ++i) l[i] *= __shfl_sync(0xffffffffu, alpha, i);
         if (j > 0) {
 #pragma unroll 1
-          for (int s = 0; s < p.slabs; ++s) {
+          for (int y = 0; y < p.slabs * 2 * HG; y += 16) {
+            float o[16];
+            tmem_ld_32x16(to + (uint32_t)y, o);
+            tmem_ld_wait();
+            uint32_t w[16];
 #pragma unroll
-            for (int x = 0; x < HG; x += 16) {
-              float o[16];
-              tmem_ld_32x16(to + (uint32_t)(s * HG + x), o);
-              tmem_ld_wait();
-              uint32_t w[16];
-#pragma unroll
-              for (int i = 0; i < 16; ++i)
-                w[i] = __float_as_uint(o[i] * __shfl_sync(0xffffffffu, alpha[x / 32], (x & 31) + i));
-              tmem_st_32x16(to + (uint32_t)(s * HG + x), w);
-            }
+            for (int i = 0; i < 16; ++i) w[i] = __float_as_uint(o[i] * __shfl_sync(0xffffffffu, alpha, (y & 31) + i));
+            tmem_st_32x16(to + (uint32_t)y, w);
           }
           tmem_st_wait();
         }
       }
-      // token r's weights: one 128-byte row (heads) of each of the two P tiles
+      // token r's weights: one 128-byte row of the P tile
 #pragma unroll
       for (int c8 = 0; c8 < HG / 8; ++c8) {
         uint32_t a[4], bb[4];
 #pragma unroll
         for (int q = 0; q < 4; ++q) {
           const int i = c8 * 8 + 2 * q;
-          const float p0 = exp2f(v[i / 32][i & 31] + __shfl_sync(0xffffffffu, neg_m[i / 32], i & 31));
-          const float p1 = exp2f(v[i / 32][(i & 31) + 1] + __shfl_sync(0xffffffffu, neg_m[i / 32], (i & 31) + 1));
+          const float p0 = exp2f(v[i] + __shfl_sync(0xffffffffu, neg_m, i));
+          const float p1 = exp2f(v[i + 1] + __shfl_sync(0xffffffffu, neg_m, i + 1));
           l[i] += p0;
           l[i + 1] += p1;
           a[q] = pack_bf16(p0, p1);
           const float2 back = unpack_bf16(a[q]);
           bb[q] = pack_bf16(p0 - back.x, p1 - back.y);
         }
-        const size_t off = (size_t)r * 128 + (size_t)((c8 ^ (r & 7)) << 4);
-        *reinterpret_cast<uint4*>(p_s + off) = make_uint4(a[0], a[1], a[2], a[3]);
-        *reinterpret_cast<uint4*>(p_s + LD_BOX + off) = make_uint4(bb[0], bb[1], bb[2], bb[3]);
+        uint8_t* row = p_s + (size_t)r * 128;
+        *reinterpret_cast<uint4*>(row + ((c8 ^ (r & 7)) << 4)) = make_uint4(a[0], a[1], a[2], a[3]);
+        *reinterpret_cast<uint4*>(row + (((c8 + 4) ^ (r & 7)) << 4)) = make_uint4(bb[0], bb[1], bb[2], bb[3]);
       }
       fence_proxy_async_smem();
       tc_fence_before();
@@ -256,42 +237,29 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
     }
     if (ok) {
       // sums over the tokens; then O^T
-      float* mine = red + (size_t)(n_t & 1) * 4 * HG;
-#pragma unroll
-      for (int c = 0; c < HC; ++c) {
-        float x[32];
-#pragma unroll
-        for (int i = 0; i < 32; ++i) x[i] = l[32 * c + i];
-        mine[w4 * HG + 32 * c + lane] = reduce_scatter32<false>(x, lane);
-      }
+      float* mine = red + (n_t & 1) * 4 * HG;
+      mine[w4 * HG + lane] = reduce_scatter32<false>(l, lane);
       mbar_arrive(red_full);
       ok = __all_sync(0xffffffffu, mbar_wait(red_full, (uint32_t)(n_t & 1), abort_flag, p.status, 1580));
       if (ok) ok = __all_sync(0xffffffffu, mbar_wait(o_full, (uint32_t)((n_t - 1) & 1), abort_flag, p.status, 1590));
       if (ok) {
         tc_fence_after();
-        if (w4 == 0) {
-#pragma unroll
-          for (int c = 0; c < HC; ++c) {
-            const int i = 32 * c + lane;
-            if (h0 + i < p.heads)
-              p.part_ml[((size_t)b * p.heads + h0 + i) * p.splits + split] =
-                  make_float2(m_ref[c], mine[i] + mine[HG + i] + mine[2 * HG + i] + mine[3 * HG + i]);
-          }
-        }
-#pragma unroll 1
+        const size_t bh0 = (size_t)b * p.heads + h0;
+        if (w4 == 0 && h0 + lane < p.heads)
+          p.part_ml[(bh0 + lane) * p.splits + split] =
+              make_float2(m_ref, mine[lane] + mine[HG + lane] + mine[2 * HG + lane] + mine[3 * HG + lane]);
+        const int nh = min(HG, p.heads - h0);
         for (int s = 0; s < p.slabs; ++s) {
           const int d = s * 128 + r;
-#pragma unroll 1
-          for (int x = 0; x < HG; x += 16) {
-            float o[16];
-            tmem_ld_32x16(to + (uint32_t)(s * HG + x), o);
-            tmem_ld_wait();
-            if (d < p.kv_rank) {
+          float o[32], e[32];
+          tmem_ld_32x32(to + (uint32_t)(s * 2 * HG), o);
+          tmem_ld_32x32(to + (uint32_t)(s * 2 * HG + HG), e);
+          tmem_ld_wait();
+          if (d < p.kv_rank) {
+            float* dst = p.part_o + (bh0 * p.splits + split) * p.kv_rank + d;
 #pragma unroll
-              for (int i = 0; i < 16; ++i)
-                if (h0 + x + i < p.heads)
-                  p.part_o[(((size_t)b * p.heads + h0 + x + i) * p.splits + split) * p.kv_rank + d] = o[i];
-            }
+            for (int i = 0; i < 32; ++i)
+              if (i < nh) dst[(size_t)i * p.splits * p.kv_rank] = o[i] + e[i];
           }
         }
         tc_fence_before();
@@ -331,13 +299,17 @@ latent_combine_kernel(const float* __restrict__ part_o, const float2* __restrict
     den += ml.y * exp2f(ml.x - m);
   }
   const float inv = 1.f / den;
-  for (int d = threadIdx.x; d < kv_rank; d += 128) {
-    float v = 0.f;
+  for (int d = threadIdx.x * 4; d < kv_rank; d += 512) {  // kv_rank is a multiple of 8
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
     for (int s = 0; s < splits; ++s) {
       const float2 ml = part_ml[bh * splits + s];
-      if (ml.y > 0.f) v = fmaf(part_o[(bh * splits + s) * kv_rank + d], exp2f(ml.x - m), v);
+      if (ml.y > 0.f) {
+        const float w = exp2f(ml.x - m) * inv;
+        const float4 x = *reinterpret_cast<const float4*>(part_o + (bh * splits + s) * kv_rank + d);
+        v.x = fmaf(x.x, w, v.x); v.y = fmaf(x.y, w, v.y); v.z = fmaf(x.z, w, v.z); v.w = fmaf(x.w, w, v.w);
+      }
     }
-    o_lat[bh * kv_rank + d] = __float2bfloat16(v * inv);
+    *reinterpret_cast<uint2*>(o_lat + bh * kv_rank + d) = make_uint2(pack_bf16(v.x, v.y), pack_bf16(v.z, v.w));
   }
 }
 
@@ -467,19 +439,25 @@ head_gemm_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant
   } else {
     pdl_wait();
     const int r = (warp & 3) * 32 + lane, m = m0 + r;
+    float sc[4];  // the scale of slot b0 + 32 i + lane
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int b = b0 + 32 * i + lane;
+      sc[i] = (p.scale != nullptr && b < p.B) ? p.scale[(size_t)b * p.heads + h] : 1.f;
+    }
     if (__all_sync(0xffffffffu, mbar_wait(done, 0, abort_flag, p.status, 1620))) {
       tc_fence_after();
-#pragma unroll 1
-      for (int x = 0; x < p.n_cols; x += 16) {
-        float o[16];
-        tmem_ld_32x16(tmem_base + ((uint32_t)((warp & 3) * 32) << 16) + x, o);
-        tmem_ld_wait();
-        if (m < p.M) {
+#pragma unroll
+      for (int x = 0; x < 128; x += 16) {
+        if (x < p.n_cols) {
+          float o[16];
+          tmem_ld_32x16(tmem_base + ((uint32_t)((warp & 3) * 32) << 16) + x, o);
+          tmem_ld_wait();
 #pragma unroll
           for (int i = 0; i < 16; ++i) {
+            const float y = o[i] * __shfl_sync(0xffffffffu, sc[x / 32], (x & 31) + i);
             const int b = b0 + x + i;
-            if (b < p.B)
-              p.Y[b * p.y_b + h * p.y_h + m] = __float2bfloat16(p.scale ? o[i] * p.scale[(size_t)b * p.heads + h] : o[i]);
+            if (m < p.M && b < p.B) p.Y[b * p.y_b + h * p.y_h + m] = __float2bfloat16(y);
           }
         }
       }
@@ -506,45 +484,41 @@ namespace {
 
 int ld_slabs(int kv_rank) { return (kv_rank + 127) / 128; }
 int ld_boxes(int kv_rank, int lat_w) { return max((lat_w + 63) / 64, 2 * ld_slabs(kv_rank)); }
-size_t ld_smem(int boxes, int hg) { return (size_t)boxes * (LD_BOX + hg * 128) + 2 * LD_BOX + 1024 + 320 + 2 * 4 * 64 * 4; }
+size_t ld_smem(int boxes) { return (size_t)boxes * (LD_BOX + 32 * 128) + LD_BOX + 1024 + 320 + 2 * 4 * 32 * 4; }
 
 }  // namespace
 
-// Heads per CTA (64 or 32) of trlb_latent_decode_tc for these sizes, 0 when it does not take them.
-TRLB_API int trlb_latent_decode_tc_heads(int heads, int dim, int rot, int vdim, int kv_rank, int lat_w, int block_size) {
-  const int boxes = ld_boxes(kv_rank, lat_w), slabs = ld_slabs(kv_rank);
+// 1 when trlb_latent_decode_tc (and with it trlb_head_gemm for the absorption and expansion) takes these sizes.
+TRLB_API int trlb_latent_decode_tc_ok(int heads, int dim, int rot, int vdim, int kv_rank, int lat_w, int block_size) {
+  const int boxes = ld_boxes(kv_rank, lat_w);
   if (heads <= 0 || dim % 8 || rot % 8 || vdim <= 0 || kv_rank % 8 || lat_w % 8 || boxes > LD_MAX_BOX) return 0;
   if (block_size < 8 || block_size > 128 || 128 % block_size) return 0;
-  for (int hg = heads > 32 ? 64 : 32; hg >= 32; hg -= 32)
-    if (64 + slabs * hg <= 512 && ld_smem(boxes, hg) <= 227 * 1024) return hg;
-  return 0;
+  return 64 + ld_slabs(kv_rank) * 64 <= 512 && ld_smem(boxes) <= 227 * 1024;
 }
 
 // q_lat [B, heads, lat_w], cache [num_blocks, block_size, lat_w] bf16 (lat_w as in csrc/mixers.cu), one new token per slot at
 // seq_lens[slot]; part_o [B, heads, splits, kv_rank] and part_ml [B, heads, splits, 2] fp32 scratch; o_lat [B, heads, kv_rank].
 TRLB_API int trlb_latent_decode_tc(const void* q_lat, const void* cache, int num_blocks, int B, int heads, int kv_rank, int lat_w,
-                                   int hg, int window, float scale, const int* seq_lens, const int* block_table, int max_blocks,
+                                   int window, float scale, const int* seq_lens, const int* block_table, int max_blocks,
                                    int block_size, const float* sink, int splits, float* part_o, float* part_ml, void* o_lat,
                                    int* status, cudaStream_t st) {
   if (B <= 0) return 0;
   const int boxes = ld_boxes(kv_rank, lat_w);
-  if ((hg != 32 && hg != 64) || !(scale > 0.f) || splits < 1 || ld_smem(boxes, hg) > 227 * 1024 || boxes > LD_MAX_BOX) return -230;
+  if (!(scale > 0.f) || splits < 1 || !trlb_latent_decode_tc_ok(heads, 8, 8, 8, kv_rank, lat_w, block_size)) return -230;
   CUtensorMap tq, tc;
-  if (trlb_host::make_tmap_3d_bf16(&tq, q_lat, lat_w, heads, B, lat_w, (uint64_t)heads * lat_w, 64, hg, 1)) return -231;
+  if (trlb_host::make_tmap_3d_bf16(&tq, q_lat, lat_w, heads, B, lat_w, (uint64_t)heads * lat_w, 64, 32, 1)) return -231;
   if (trlb_host::make_tmap_2d_bf16(&tc, cache, (uint64_t)num_blocks * block_size, lat_w, lat_w, block_size, 64)) return -232;
   LatentDecodeTc p = {heads, kv_rank, boxes, ld_slabs(kv_rank), lat_w, window, max_blocks, block_size, splits,
                       scale * 1.4426950408889634f, seq_lens, block_table, part_o, (float2*)part_ml, status};
   static bool attr_set = false;
   if (!attr_set) {
-    if (cudaFuncSetAttribute(latent_decode_tc_kernel<32>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024) != cudaSuccess ||
-        cudaFuncSetAttribute(latent_decode_tc_kernel<64>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024) != cudaSuccess)
+    if (cudaFuncSetAttribute(latent_decode_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024) != cudaSuccess)
       return -233;
     attr_set = true;
   }
-  const dim3 grid((heads + hg - 1) / hg, splits, B), blk(192);
   const bool pdl = trlb_host::pdl_enabled();
-  const int rc = hg == 64 ? (int)trlb_host::launch_kernel(latent_decode_tc_kernel<64>, grid, blk, ld_smem(boxes, hg), st, pdl, tq, tc, p)
-                          : (int)trlb_host::launch_kernel(latent_decode_tc_kernel<32>, grid, blk, ld_smem(boxes, hg), st, pdl, tq, tc, p);
+  const int rc = (int)trlb_host::launch_kernel(latent_decode_tc_kernel, dim3((heads + 31) / 32, splits, B), dim3(192), ld_smem(boxes),
+                                               st, pdl, tq, tc, p);
   if (rc) return rc;
   return (int)trlb_host::launch_kernel(latent_combine_kernel, dim3(heads, B), dim3(128), 0, st, pdl, (const float*)part_o,
                                        (const float2*)part_ml, sink, seq_lens, heads, kv_rank, splits, (__nv_bfloat16*)o_lat);

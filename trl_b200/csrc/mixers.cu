@@ -24,6 +24,13 @@ embed_scaled_kernel(const long long* __restrict__ ids, const T* __restrict__ emb
   pdl_launch_dependents();
   pdl_wait();
   const long long id = ids[blockIdx.x];
+  if ((H & 3) == 0 && id >= 0 && id < V) {
+    for (int j = 4 * threadIdx.x; j < H; j += 4 * blockDim.x) {
+      const float4 e = load4(emb + (size_t)id * H + j);
+      store4(x + (size_t)blockIdx.x * H + j, make_float4(e.x * scale, e.y * scale, e.z * scale, e.w * scale));
+    }
+    return;
+  }
   for (int j = threadIdx.x; j < H; j += blockDim.x)
     x[(size_t)blockIdx.x * H + j] = (id >= 0 && id < V) ? to_f(emb[(size_t)id * H + j]) * scale : 0.f;
 }
@@ -67,10 +74,13 @@ dynamic_tanh_kernel(float* __restrict__ x, float* __restrict__ delta, const floa
 template <typename T>
 __global__ void __launch_bounds__(256)
 gelu_erf_kernel(const T* __restrict__ z, T* __restrict__ out, long long n) {
-  for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x) {
-    const float v = to_f(z[i]);
-    out[i] = from_f<T>(0.5f * v * (1.f + erff(v * 0.70710678118654752f)));
+  const long long stride = (long long)gridDim.x * blockDim.x, first = blockIdx.x * (long long)blockDim.x + threadIdx.x;
+#pragma unroll 2
+  for (long long i = first; i < n / 4; i += stride) {
+    const float4 v = load4(z + 4 * i);
+    store4(out + 4 * i, make_float4(gelu_erf_f(v.x), gelu_erf_f(v.y), gelu_erf_f(v.z), gelu_erf_f(v.w)));
   }
+  for (long long i = n / 4 * 4 + first; i < n; i += stride) out[i] = from_f<T>(gelu_erf_f(to_f(z[i])));
 }
 
 // ------------------------------------------------------------------------------------------------------------
@@ -105,13 +115,41 @@ latent_prep_kernel(const LatentPrep p, T* __restrict__ cq, T* __restrict__ lat, 
   const float* ar = akv + p.kv_rank;
   const float* ag = ar + p.rot;
   float sq = 0.f, sk = 0.f;
-  for (int j = threadIdx.x; j < p.q_rank; j += blockDim.x) sq += a[j] * a[j];
-  for (int j = threadIdx.x; j < p.kv_rank; j += blockDim.x) sk += akv[j] * akv[j];
+  const bool vec = ((p.q_rank | p.kv_rank | (int)p.ld) & 3) == 0;
+  if (vec) {
+#pragma unroll 2
+    for (int j = 4 * threadIdx.x; j < p.q_rank; j += 4 * blockDim.x) {
+      const float4 v = load4(a + j);
+      sq += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+    }
+    for (int j = 4 * threadIdx.x; j < p.kv_rank; j += 4 * blockDim.x) {
+      const float4 v = load4(akv + j);
+      sk += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+    }
+  } else {
+    for (int j = threadIdx.x; j < p.q_rank; j += blockDim.x) sq += a[j] * a[j];
+    for (int j = threadIdx.x; j < p.kv_rank; j += blockDim.x) sk += akv[j] * akv[j];
+  }
   const float2 s = block_sum2(sq, sk, red);
   const float rq = 1.f / sqrtf(s.x / (float)p.q_rank + p.eps), rk = 1.f / sqrtf(s.y / (float)p.kv_rank + p.eps);
-  for (int j = threadIdx.x; j < p.q_rank; j += blockDim.x)
-    cq[(size_t)row * p.q_rank + j] = from_f<T>(a[j] * rq * p.q_norm[j]);
-  for (int h = threadIdx.x; h < p.heads; h += blockDim.x) p.gate[(size_t)row * p.heads + h] = sigmoid_f(ag[h]);
+  const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+  if (vec) {
+#pragma unroll 2
+    for (int j = 4 * threadIdx.x; j < p.q_rank; j += 4 * blockDim.x) {
+      const float4 v = load4(a + j), w = load4(p.q_norm + j);
+      store4(cq + (size_t)row * p.q_rank + j, make_float4(v.x * rq * w.x, v.y * rq * w.y, v.z * rq * w.z, v.w * rq * w.w));
+      if (p.clear) store4(a + j, zero);
+    }
+  } else {
+    for (int j = threadIdx.x; j < p.q_rank; j += blockDim.x) {
+      cq[(size_t)row * p.q_rank + j] = from_f<T>(a[j] * rq * p.q_norm[j]);
+      if (p.clear) a[j] = 0.f;
+    }
+  }
+  for (int h = threadIdx.x; h < p.heads; h += blockDim.x) {
+    p.gate[(size_t)row * p.heads + h] = sigmoid_f(ag[h]);
+    if (p.clear) a[p.q_rank + p.kv_rank + p.rot + h] = 0.f;
+  }
   const int pos = p.positions[row];
   const bool live = pos >= 0 && pos < p.table_len;
   T* dense = lat == nullptr ? nullptr : lat + (size_t)row * p.lat_w;
@@ -123,10 +161,22 @@ latent_prep_kernel(const LatentPrep p, T* __restrict__ cq, T* __restrict__ lat, 
       paged = cache + ((size_t)blk * p.block_size + pos % p.block_size) * p.lat_w;
     }
   }
-  for (int j = threadIdx.x; j < p.kv_rank; j += blockDim.x) {
-    const T v = from_f<T>(akv[j] * rk * p.kv_norm[j]);
-    if (dense) dense[j] = v;
-    if (paged) paged[j] = v;
+  float* akw = a + p.q_rank;
+  if (vec) {
+    for (int j = 4 * threadIdx.x; j < p.kv_rank; j += 4 * blockDim.x) {
+      const float4 v = load4(akv + j), w = load4(p.kv_norm + j);
+      const float4 y = make_float4(v.x * rk * w.x, v.y * rk * w.y, v.z * rk * w.z, v.w * rk * w.w);
+      if (dense) store4(dense + j, y);
+      if (paged) store4(paged + j, y);
+      if (p.clear) store4(akw + j, zero);
+    }
+  } else {
+    for (int j = threadIdx.x; j < p.kv_rank; j += blockDim.x) {
+      const T v = from_f<T>(akv[j] * rk * p.kv_norm[j]);
+      if (dense) dense[j] = v;
+      if (paged) paged[j] = v;
+      if (p.clear) akw[j] = 0.f;
+    }
   }
   for (int i = threadIdx.x; i < p.rot / 2; i += blockDim.x) {
     const float2 cs = live ? p.table[(size_t)pos * (p.rot / 2) + i] : make_float2(1.f, 0.f);
@@ -134,26 +184,30 @@ latent_prep_kernel(const LatentPrep p, T* __restrict__ cq, T* __restrict__ lat, 
     const T x0 = from_f<T>(u * cs.x - v * cs.y), x1 = from_f<T>(v * cs.x + u * cs.y);
     if (dense) { dense[p.kr_off + 2 * i] = x0; dense[p.kr_off + 2 * i + 1] = x1; }
     if (paged) { paged[p.kr_off + 2 * i] = x0; paged[p.kr_off + 2 * i + 1] = x1; }
-  }
-  if (p.clear) {
-    __syncthreads();
-    const int n = p.q_rank + p.kv_rank + p.rot + p.heads;
-    for (int j = threadIdx.x; j < n; j += blockDim.x) a[j] = 0.f;
+    if (p.clear) {
+      akw[p.kv_rank + 2 * i] = 0.f;
+      akw[p.kv_rank + 2 * i + 1] = 0.f;
+    }
   }
 }
 
 // q [rows, heads, dim + rot]: the rot part of every head turned in place.
-template <typename T>
+template <typename T, int PAIRS>  // pairs per thread: 2 needs dim and rot to be multiples of 4
 __global__ void __launch_bounds__(256)
 rotate_q_kernel(T* __restrict__ q, int heads, int dim, int rot, const int* __restrict__ positions,
                 const float2* __restrict__ table, int table_len, long long n) {
-  const int half = rot / 2;
+  const int half = rot / 2, groups = half / PAIRS;
   for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x) {
-    const int f = (int)(i % half);
-    const long long th = i / half;
+    const int f = (int)(i % groups) * PAIRS;
+    const long long th = i / groups;
     const int pos = positions[th / heads];
     if (pos < 0 || pos >= table_len) continue;
     T* d = q + (size_t)th * (dim + rot) + dim + 2 * f;
+    if (PAIRS == 2) {
+      const float4 cs = *reinterpret_cast<const float4*>(table + (size_t)pos * half + f), v = load4(d);
+      store4(d, make_float4(v.x * cs.x - v.y * cs.y, v.y * cs.x + v.x * cs.y, v.z * cs.z - v.w * cs.w, v.w * cs.z + v.z * cs.w));
+      continue;
+    }
     const float2 cs = table[(size_t)pos * half + f];
     const float u = to_f(d[0]), v = to_f(d[1]);
     d[0] = from_f<T>(u * cs.x - v * cs.y);
@@ -540,9 +594,23 @@ mlstm_out_kernel(const float* __restrict__ o, const G* __restrict__ gl, long lon
   const int h = blockIdx.x;
   const size_t row = blockIdx.y, base = (row * heads + h) * vdim;
   float ss = 0.f;
-  for (int e = threadIdx.x; e < vdim; e += 128) ss += o[base + e] * o[base + e];
+  const bool vec = ((vdim | (int)g_ld) & 3) == 0 && (reinterpret_cast<uintptr_t>(gl) & (4 * sizeof(G) - 1)) == 0;
+  if (vec) {
+    for (int e = 4 * threadIdx.x; e < vdim; e += 512) {
+      const float4 v = load4(o + base + e);
+      ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+    }
+  } else {
+    for (int e = threadIdx.x; e < vdim; e += 128) ss += o[base + e] * o[base + e];
+  }
   const float r = 1.f / sqrtf(block_sum2(ss, 0.f, red).x / (float)vdim + eps);
-  for (int e = threadIdx.x; e < vdim; e += 128)
+  if (vec) {
+    for (int e = 4 * threadIdx.x; e < vdim; e += 512) {
+      const float4 v = load4(o + base + e), w = load4(norm + h * vdim + e), g = load4(gl + row * g_ld + (size_t)h * vdim + e);
+      store4(y + base + e, make_float4(v.x * r * w.x * sigmoid_f(g.x), v.y * r * w.y * sigmoid_f(g.y),
+                                       v.z * r * w.z * sigmoid_f(g.z), v.w * r * w.w * sigmoid_f(g.w)));
+    }
+  } else for (int e = threadIdx.x; e < vdim; e += 128)
     y[base + e] = from_f<T>(o[base + e] * r * norm[h * vdim + e] * sigmoid_f(to_f(gl[row * g_ld + (size_t)h * vdim + e])));
   if (clear_row != nullptr) {
     // every head's gate logits belong to this block alone; the rest of the row (q, k, v, input and forget gates) has
@@ -624,10 +692,13 @@ TRLB_API int trlb_latent_prep(float* acc, long long ld, int rows, int q_rank, in
 
 TRLB_API int trlb_rotate_q(void* q, int rows, int heads, int dim, int rot, const int* positions, const float* table,
                            int table_len, int is_bf16, cudaStream_t st) {
-  const long long n = (long long)rows * heads * (rot / 2);
+  const bool two = dim % 4 == 0 && rot % 4 == 0;
+  const long long n = (long long)rows * heads * (rot / 2) / (two ? 2 : 1);
   if (n <= 0) return 0;
-  if (is_bf16) rotate_q_kernel<bf16><<<grid_for(n, 256), 256, 0, st>>>((bf16*)q, heads, dim, rot, positions, (const float2*)table, table_len, n);
-  else rotate_q_kernel<float><<<grid_for(n, 256), 256, 0, st>>>((float*)q, heads, dim, rot, positions, (const float2*)table, table_len, n);
+#define GO(TT, PP) rotate_q_kernel<TT, PP><<<grid_for(n, 256), 256, 0, st>>>((TT*)q, heads, dim, rot, positions, (const float2*)table, table_len, n)
+  if (is_bf16) { if (two) GO(bf16, 2); else GO(bf16, 1); }
+  else { if (two) GO(float, 2); else GO(float, 1); }
+#undef GO
   return (int)cudaGetLastError();
 }
 

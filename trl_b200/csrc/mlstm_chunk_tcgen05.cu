@@ -111,11 +111,11 @@ mlstm_scan_kernel(const float* __restrict__ ig, const float* __restrict__ fg, co
 // ------------------------------------------------------------------------------------------------------------
 // State pass.  Warp 0: TMA; warp 1: MMA; warps 2-5: thread r scales token r of a chunk's v, and owns row r (of the
 // CTA's 128 rows of S) in registers.
-constexpr int MS_STAGES = 3;
+constexpr int MS_STAGES = 1;  // 64 KB: two CTAs per SM hide each other's loads; the work per chunk is in the row threads
 constexpr uint32_t MS_STAGE_BYTES = 4 * ML_BOX;  // k (two boxes), v scaled in place, v remainder
 constexpr size_t MS_SMEM = MS_STAGES * (size_t)MS_STAGE_BYTES + 1024 + 2048;
 
-__global__ void __launch_bounds__(192, 1)
+__global__ void __launch_bounds__(192, 2)
 mlstm_state_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_constant__ CUtensorMap tm_v, const MlstmChunk p) {
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
@@ -325,15 +325,14 @@ mlstm_state_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_consta
 
 // ------------------------------------------------------------------------------------------------------------
 // Output pass.  Warp 0: TMA; warp 1: MMA; warps 2-5: one thread per token of the chunk.  Q stays in shared memory; K
-// boxes, 64-row pieces of S (both halves) and finally V travel through one ring of 32 KB stages.
-// TMEM: scores / weights [0, 128), output [128, 256).
-constexpr int MO_STAGES = 2;
-constexpr uint32_t MO_STAGE_BYTES = 2 * ML_BOX;
+// boxes, 64-row pieces of S (leading part, remainder) and finally the halves of V travel through one ring of 16 KB boxes.
+// TMEM: scores / weights [0, 128), output [128, 256): two CTAs fit an SM when the ring is short enough.
+constexpr int MO_MAX_STAGES = 6;
 
-__global__ void __launch_bounds__(192)
+__global__ void __launch_bounds__(192, 2)
 mlstm_output_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_k,
                     const __grid_constant__ CUtensorMap tm_v, const __grid_constant__ CUtensorMap tm_sh,
-                    const __grid_constant__ CUtensorMap tm_sl, const MlstmChunk p) {
+                    const __grid_constant__ CUtensorMap tm_sl, const MlstmChunk p, const int stages) {
   int seq = -1, c = (int)blockIdx.x;
   for (int s = 0; s < p.n_seq; ++s) {
     const int n = ml_chunks(p.cu[s + 1] - p.cu[s]);
@@ -346,11 +345,11 @@ mlstm_output_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
   const int nd = (p.dim + 63) / 64;
   uint8_t* q_s = smem;
   uint8_t* ring = q_s + (size_t)nd * ML_BOX;
-  uint64_t* bars = reinterpret_cast<uint64_t*>(ring + MO_STAGES * MO_STAGE_BYTES);
+  uint64_t* bars = reinterpret_cast<uint64_t*>(ring + (size_t)stages * ML_BOX);
   uint64_t* q_full = bars;
-  uint64_t* full = bars + 1;               // [MO_STAGES]
-  uint64_t* empty = full + MO_STAGES;      // [MO_STAGES]
-  uint64_t* s_full = empty + MO_STAGES;    // scores done
+  uint64_t* full = bars + 1;                  // [MO_MAX_STAGES]
+  uint64_t* empty = full + MO_MAX_STAGES;     // [MO_MAX_STAGES]
+  uint64_t* s_full = empty + MO_MAX_STAGES;   // scores done
   uint64_t* x_full = s_full + 1;           // Q S done
   uint64_t* p_full = x_full + 1;           // weights in TMEM, output rescaled
   uint64_t* o_full = p_full + 1;
@@ -358,6 +357,7 @@ mlstm_output_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(g_full + 1);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
   float* g_s = reinterpret_cast<float*>(bars + 32);  // [128] g_j log2(e)
+  float* n_s = g_s + 128;                            // [dim] n in front of the chunk
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int h = blockIdx.y, e0 = (int)blockIdx.z * 128;
@@ -369,7 +369,7 @@ mlstm_output_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
 
   if (threadIdx.x == 0) {
     mbar_init(q_full, 1);
-    for (int s = 0; s < MO_STAGES; ++s) {
+    for (int s = 0; s < MO_MAX_STAGES; ++s) {
       mbar_init(&full[s], 1);
       mbar_init(&empty[s], 1);
     }
@@ -392,31 +392,28 @@ mlstm_output_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
   __syncthreads();
   tc_fence_after();
   const uint32_t tmem_base = *tmem_slot;
-  const int n_items = nd + (carried ? nd : 0) + 1;  // K boxes, state pieces, V
+  const int nv = (n_cols + 63) / 64, n_state = carried ? 2 * nd : 0;
+  const int n_items = nd + n_state + nv;  // K boxes, state pieces, halves of V
 
   if (warp == 0) {
     if (lane == 0) {
       mbar_expect_tx(q_full, (uint32_t)nd * ML_BOX);
       for (int i = 0; i < nd; ++i) tma_load_3d(q_s + (size_t)i * ML_BOX, &tm_q, q_full, 64 * i, h, row0);
       for (int it = 0; it < n_items; ++it) {
-        const int s = it % MO_STAGES;
-        if (!mbar_wait(&empty[s], (uint32_t)(((it / MO_STAGES) & 1) ^ 1), abort_flag, p.status, 1400 + s)) break;
-        uint8_t* st = ring + (size_t)s * MO_STAGE_BYTES;
+        const int s = it % stages;
+        if (!mbar_wait(&empty[s], (uint32_t)(((it / stages) & 1) ^ 1), abort_flag, p.status, 1400 + s)) break;
+        uint8_t* st = ring + (size_t)s * ML_BOX;
+        mbar_expect_tx(&full[s], ML_BOX);
         if (it < nd) {
-          mbar_expect_tx(&full[s], ML_BOX);
           tma_load_3d(st, &tm_k, &full[s], 64 * it, h, row0);
-        } else if (it < n_items - 1) {
-          // rows 64 (it - nd) .. of S: two 64-column boxes of 8 KB of each half
-          mbar_expect_tx(&full[s], 2 * ML_BOX);
-          const int d = 64 * (it - nd), z = chunk * p.heads + h;
-          tma_load_3d(st, &tm_sh, &full[s], e0, d, z);
-          tma_load_3d(st + 8192, &tm_sh, &full[s], e0 + 64, d, z);
-          tma_load_3d(st + 16384, &tm_sl, &full[s], e0, d, z);
-          tma_load_3d(st + 24576, &tm_sl, &full[s], e0 + 64, d, z);
+        } else if (it < nd + n_state) {
+          // rows 64 i .. of S as two 64-column boxes of 8 KB
+          const CUtensorMap* tm = ((it - nd) & 1) ? &tm_sl : &tm_sh;
+          const int d = 64 * ((it - nd) >> 1), z = chunk * p.heads + h;
+          tma_load_3d(st, tm, &full[s], e0, d, z);
+          tma_load_3d(st + 8192, tm, &full[s], e0 + 64, d, z);
         } else {
-          mbar_expect_tx(&full[s], 2 * ML_BOX);
-          tma_load_3d(st, &tm_v, &full[s], e0, h, row0);
-          tma_load_3d(st + ML_BOX, &tm_v, &full[s], e0 + 64, h, row0);
+          tma_load_3d(st, &tm_v, &full[s], e0 + 64 * (it - nd - n_state), h, row0);
         }
       }
     }
@@ -428,35 +425,34 @@ mlstm_output_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
       const uint32_t q_u = smem_u32(q_s), r_u = smem_u32(ring);
       bool ok = mbar_wait(q_full, 0, abort_flag, p.status, 1410);
       for (int it = 0; it < n_items && ok; ++it) {
-        const int s = it % MO_STAGES;
-        if (it == n_items - 1) ok = mbar_wait(p_full, 0, abort_flag, p.status, 1412);
-        if (ok) ok = mbar_wait(&full[s], (uint32_t)((it / MO_STAGES) & 1), abort_flag, p.status, 1420 + s);
+        const int s = it % stages;
+        if (it == nd + n_state) ok = mbar_wait(p_full, 0, abort_flag, p.status, 1412);
+        if (ok) ok = mbar_wait(&full[s], (uint32_t)((it / stages) & 1), abort_flag, p.status, 1420 + s);
         if (!ok) break;
         tc_fence_after();
-        const uint32_t st = r_u + (uint32_t)s * MO_STAGE_BYTES;
+        const uint32_t st = r_u + (uint32_t)s * ML_BOX;
         if (it < nd) {
           const int steps = min(4, (p.dim - 64 * it + 15) >> 4);
           const uint64_t da = umma_desc_kmajor_sw128(q_u + (uint32_t)it * ML_BOX), db = umma_desc_kmajor_sw128(st);
           for (int kk = 0; kk < steps; ++kk) umma_bf16_ss(tmem_base, da + 2 * kk, db + 2 * kk, idesc_s, (it | kk) != 0);
           if (it == nd - 1) umma_commit(s_full);
-        } else if (it < n_items - 1) {
-          const int i = it - nd;
+        } else if (it < nd + n_state) {
+          const int i = (it - nd) >> 1;
           const int steps = min(4, (p.dim - 64 * i + 15) >> 4);
           const uint64_t da = umma_desc_kmajor_sw128(q_u + (uint32_t)i * ML_BOX);
-          for (int half = 0; half < 2; ++half)
-            for (int kk = 0; kk < steps; ++kk)
-              umma_bf16_ss(tmem_base + 128, da + 2 * kk,
-                           umma_desc_mnmajor_sw128(st + (uint32_t)(half * 16384 + kk * 2048), 8192), idesc_o,
-                           (i | half | kk) != 0);
-          if (i == nd - 1) umma_commit(x_full);
+          for (int kk = 0; kk < steps; ++kk)
+            umma_bf16_ss(tmem_base + 128, da + 2 * kk, umma_desc_mnmajor_sw128(st + (uint32_t)kk * 2048, 8192), idesc_o,
+                         (it > nd) || kk != 0);
+          if (it == nd + n_state - 1) umma_commit(x_full);
         } else {
+          const int i = it - nd - n_state;
+          const uint32_t idesc_v = umma_idesc_bf16_major(128, min(64, n_cols - 64 * i), false, true);
           for (int half = 0; half < 2; ++half)
 #pragma unroll
             for (int kk = 0; kk < ML_L / 16; ++kk)
-              umma_bf16_ts(tmem_base + 128, tmem_base + (uint32_t)(half * 64 + kk * 8),
-                           umma_desc_mnmajor_sw128(st + (uint32_t)kk * 2048, ML_BOX), idesc_o,
-                           carried || (half | kk) != 0);
-          umma_commit(o_full);
+              umma_bf16_ts(tmem_base + 128 + 64 * i, tmem_base + (uint32_t)(half * 64 + kk * 8),
+                           umma_desc_mnmajor_sw128(st + (uint32_t)kk * 2048, ML_BOX), idesc_v, carried || (half | kk) != 0);
+          if (it == n_items - 1) umma_commit(o_full);
         }
         umma_commit(&empty[s]);
       }
@@ -469,6 +465,8 @@ mlstm_output_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
     const bool row_ok = t < len;
     const size_t at = (size_t)h * p.T + beg;
     g_s[r] = row_ok ? p.g[at + t] * ML_LOG2E : -INFINITY;
+    if (carried)
+      for (int d = r; d < p.dim; d += 128) n_s[d] = p.n_in[((size_t)chunk * p.heads + h) * p.dim + d];
     mbar_arrive(g_full);
     const float bt = row_ok ? p.b[at + t] : 0.f, mt = row_ok ? p.m[at + t] : 0.f;
     const float m_in = carried ? p.m[at + c * ML_L - 1] : 0.f;
@@ -476,28 +474,29 @@ mlstm_output_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
     const float c2 = (bt - mt) * ML_LOG2E;
     float nq = 0.f;
     bool ok = __all_sync(0xffffffffu, mbar_wait(q_full, 0, abort_flag, p.status, 1430));
+    if (ok) ok = __all_sync(0xffffffffu, mbar_wait(g_full, 0, abort_flag, p.status, 1432));
     if (ok && carried) {
-      const float* n_in = p.n_in + ((size_t)chunk * p.heads + h) * p.dim;
       for (int d = 0; d < p.dim; d += 8) {
         const int box = d >> 6, cc = (d & 63) >> 3;
         const uint4 x = *reinterpret_cast<const uint4*>(q_s + (size_t)box * ML_BOX + (size_t)r * 128 + ((cc ^ (r & 7)) << 4));
-        const float4 n0 = *reinterpret_cast<const float4*>(n_in + d), n1 = *reinterpret_cast<const float4*>(n_in + d + 4);
+        const float4 n0 = *reinterpret_cast<const float4*>(n_s + d), n1 = *reinterpret_cast<const float4*>(n_s + d + 4);
         const float2 a = unpack_bf16(x.x), b = unpack_bf16(x.y), e = unpack_bf16(x.z), f = unpack_bf16(x.w);
         nq += a.x * n0.x + a.y * n0.y + b.x * n0.z + b.y * n0.w + e.x * n1.x + e.y * n1.y + f.x * n1.z + f.y * n1.w;
       }
       nq *= carry;
     }
-    if (ok) ok = __all_sync(0xffffffffu, mbar_wait(g_full, 0, abort_flag, p.status, 1432));
     if (ok) ok = __all_sync(0xffffffffu, mbar_wait(s_full, 0, abort_flag, p.status, 1434));
     if (ok) {
       tc_fence_after();
       const uint32_t ts = tmem_base + lane_off, to = ts + 128;
-      float v[4][32];
+      // the last 64 keys first: their packed weights wait in registers until the first 64 scores have been read too
+      uint32_t late[2][32];
 #pragma unroll
-      for (int x = 0; x < 4; ++x) tmem_ld_32x32(ts + 32 * x, v[x]);
-      tmem_ld_wait();
-#pragma unroll
-      for (int x = 0; x < 4; ++x) {
+      for (int y = 0; y < 4; ++y) {
+        const int x = y ^ 2;  // 2, 3, 0, 1
+        float v[32];
+        tmem_ld_32x32(ts + 32 * x, v);
+        tmem_ld_wait();
         uint32_t a[16], b[16];
 #pragma unroll
         for (int i = 0; i < 16; ++i) {
@@ -505,15 +504,29 @@ mlstm_output_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
 #pragma unroll
           for (int k = 0; k < 2; ++k) {
             const int j = 32 * x + 2 * i + k;
-            w[k] = (row_ok && j <= r) ? fast_exp2(c2 + g_s[j]) * p.qscale * v[x][2 * i + k] : 0.f;
+            w[k] = (row_ok && j <= r) ? fast_exp2(c2 + g_s[j]) * p.qscale * v[2 * i + k] : 0.f;
             nq += w[k];
           }
           a[i] = pack_bf16(w[0], w[1]);
           const float2 back = unpack_bf16(a[i]);
           b[i] = pack_bf16(w[0] - back.x, w[1] - back.y);
         }
-        tmem_st_32x16(ts + 16 * x, a);
-        tmem_st_32x16(ts + 64 + 16 * x, b);
+        if (y < 2) {
+#pragma unroll
+          for (int i = 0; i < 16; ++i) { late[y][i] = a[i]; late[y][16 + i] = b[i]; }
+        } else {
+          // columns [64, 128) have been read, and of [0, 64) those up to here
+          tmem_st_32x16(ts + 16 * x, a);
+          tmem_st_32x16(ts + 64 + 16 * x, b);
+        }
+      }
+#pragma unroll
+      for (int y = 0; y < 2; ++y) {
+        uint32_t a[16], b[16];
+#pragma unroll
+        for (int i = 0; i < 16; ++i) { a[i] = late[y][i]; b[i] = late[y][16 + i]; }
+        tmem_st_32x16(ts + 32 + 16 * y, a);
+        tmem_st_32x16(ts + 96 + 16 * y, b);
       }
       if (carried) {
         ok = __all_sync(0xffffffffu, mbar_wait(x_full, 0, abort_flag, p.status, 1436));
@@ -573,13 +586,23 @@ using namespace trlb;
 
 namespace {
 
-size_t mo_smem(int dim) { return (size_t)((dim + 63) / 64) * ML_BOX + MO_STAGES * (size_t)MO_STAGE_BYTES + 1024 + 1024; }
+size_t mo_smem(int dim, int stages) {
+  return ((size_t)((dim + 63) / 64) + stages) * ML_BOX + 1024 + 256 + 512 + (size_t)dim * 4;
+}
+
+// Ring length: what lets two CTAs share an SM if that is at least two boxes, else what one CTA can have.
+int mo_stages(int dim) {
+  for (int limit : {113 * 1024, 227 * 1024})
+    for (int n = MO_MAX_STAGES; n >= 2; --n)
+      if (mo_smem(dim, n) <= (size_t)limit) return n;
+  return 0;
+}
 
 }  // namespace
 
 // 1 when trlb_mlstm_chunk takes these sizes.
 TRLB_API int trlb_mlstm_chunk_ok(int heads, int dim, int vdim) {
-  return heads > 0 && dim > 0 && vdim > 0 && dim % 8 == 0 && vdim % 8 == 0 && mo_smem(dim) <= 227 * 1024;
+  return heads > 0 && dim > 0 && vdim > 0 && dim % 8 == 0 && vdim % 8 == 0 && mo_stages(dim) > 0;
 }
 
 // Chunks (upper bound) of T packed tokens in n_seq sequences: the leading size of s_hi, s_lo [chunks, heads, dim, vdim] bf16
@@ -618,6 +641,7 @@ TRLB_API int trlb_mlstm_chunk(const void* qkv, long long ld, int k_off, int v_of
   mlstm_scan_kernel<<<dim3(n_seq, heads), 256, 0, st>>>(ig, fg, cu, T, heads, b, g, m);
   const int tiles = ((dim + 127) / 128) * ((vdim + 63) / 64);
   mlstm_state_kernel<<<dim3(n_seq, heads, tiles), 192, MS_SMEM, st>>>(tk, tv, p);
-  mlstm_output_kernel<<<dim3(chunks, heads, (vdim + 127) / 128), 192, mo_smem(dim), st>>>(tq, tk, tv, tsh, tsl, p);
+  mlstm_output_kernel<<<dim3(chunks, heads, (vdim + 127) / 128), 192, mo_smem(dim, mo_stages(dim)), st>>>(tq, tk, tv, tsh, tsl, p,
+                                                                                                                  mo_stages(dim));
   return (int)cudaGetLastError();
 }

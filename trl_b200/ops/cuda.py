@@ -840,13 +840,14 @@ def set_pdl(on: bool) -> bool:
     return bool(lib().trlb_set_pdl(c_int(int(bool(on)))))
 
 
-def decode_gemm(x, w, bias=None, *, y32=None, out=None, swiglu=False, max_ctas: int = 0, tiled_shape=None,
+def decode_gemm(x, w, bias=None, *, y32=None, out=None, swiglu=False, gelu=False, max_ctas: int = 0, tiled_shape=None,
                 peers=None):
     """Weight-streaming tcgen05 GEMM for decode batches (at most 128 rows of ``x``).
 
     ``y32`` given: ``y32[B, N] (fp32) += x @ w^T (+ bias)``, work split stream-K style over every SM; the caller passes
     zeros (the consumer kernels clear the buffer after reading it).  Otherwise bf16 ``out[B, N] = x @ w^T (+ bias)``;
-    with ``swiglu`` ``w`` is ``[2N, K]`` (gate rows, then up rows) and ``out = silu(x Wg^T) * (x Wu^T)``.
+    with ``swiglu`` ``w`` is ``[2N, K]`` (gate rows, then up rows) and ``out = silu(x Wg^T) * (x Wu^T)``; with ``gelu`` the
+    exact GELU of the sum is stored.
 
     ``tiled_shape=(rows, K)``: ``w`` is the flat tile-major copy made by :func:`tile_weights` of a ``[rows, K]`` weight.
     ``peers=(peer_y32_ptrs, arrive_ptrs, stage, slab_ctr)``: row-parallel GEMM fused with its all-reduce: partial sums
@@ -871,7 +872,7 @@ def decode_gemm(x, w, bias=None, *, y32=None, out=None, swiglu=False, max_ctas: 
         if out is None:
             out = torch.empty(B, N, dtype=torch.bfloat16, device=x.device)
         assert out.dtype == torch.bfloat16 and out.stride(1) == 1 and tuple(out.shape) == (B, N)
-        mode, ldy, dst32, dstb, ret = (2 if swiglu else 1), out.stride(0), None, out, out
+        mode, ldy, dst32, dstb, ret = (2 if swiglu else 3 if gelu else 1), out.stride(0), None, out, out
     n_peers, peer_arr, arrive_arr, stage, slab_ctr = 0, None, None, None, None
     if peers is not None:
         peer_ptrs, arrive_ptrs, stage, slab_ctr = peers

@@ -131,16 +131,14 @@ def latent_expand(o_lat, m, gate, positions, out):
                                   c_int(m.kv_rank), _p(positions), _b(out), _s()), "latent_expand")
 
 
-def latent_decode_tc_heads(m, block_size: int) -> int:
-    """Heads per CTA of :func:`latent_decode_tc` for a mixer's sizes; 0: the CUDA-core kernels serve it."""
+def latent_decode_tc_ok(m, block_size: int) -> bool:
+    """Whether :func:`latent_decode_tc` and :func:`head_gemm` serve a mixer's sizes (else the CUDA-core kernels do)."""
     _, w = latent_row(m.kv_rank, m.rot_dim)
-    if m.scale <= 0:
-        return 0
-    return int(lib().trlb_latent_decode_tc_heads(c_int(m.heads), c_int(m.dim), c_int(m.rot_dim), c_int(m.vdim),
+    return m.scale > 0 and bool(lib().trlb_latent_decode_tc_ok(c_int(m.heads), c_int(m.dim), c_int(m.rot_dim), c_int(m.vdim),
                                                  c_int(m.kv_rank), c_int(w), c_int(block_size)))
 
 
-def latent_decode_tc(q_lat, cache, m, seq_lens, block_table, block_size, o_lat, part_o, part_ml, hg, splits):
+def latent_decode_tc(q_lat, cache, m, seq_lens, block_table, block_size, o_lat, part_o, part_ml, splits):
     """:func:`latent_decode` on the tensor cores (bf16).  ``part_o`` [>= B heads splits kv_rank] and ``part_ml`` [>= 2 B heads
     splits] fp32 scratch."""
     B = q_lat.shape[0]
@@ -148,7 +146,7 @@ def latent_decode_tc(q_lat, cache, m, seq_lens, block_table, block_size, o_lat, 
     assert q_lat.dtype == torch.bfloat16 and cache.is_contiguous() and cache.shape[1] == block_size and cache.shape[2] == w
     assert part_o.numel() >= B * m.heads * splits * m.kv_rank and part_ml.numel() >= 2 * B * m.heads * splits
     _chk(lib().trlb_latent_decode_tc(_p(q_lat), _p(cache), c_int(cache.shape[0]), c_int(B), c_int(m.heads), c_int(m.kv_rank),
-                                     c_int(w), c_int(hg), c_int(m.window or 0), c_float(m.scale), _p(seq_lens),
+                                     c_int(w), c_int(m.window or 0), c_float(m.scale), _p(seq_lens),
                                      _p(block_table), c_int(block_table.shape[1]), c_int(block_size), _p(m.sink),
                                      c_int(splits), _p(part_o), _p(part_ml), _p(o_lat), _p(status_buffer(q_lat.device)), _s()),
          "latent_decode_tc")

@@ -41,11 +41,11 @@ class _LatentSlots:
         self.q_lat = eng.scratch("q_lat", B, m.heads, self.width)
         self.o_lat = eng.scratch("o_lat", B, m.heads, m.kv_rank)
         self.o = eng.scratch("o", B, m.heads * m.vdim)
-        # tensor-core decode: heads per CTA (0: sizes or dtype that only the CUDA-core kernels take)
-        self.hg = K.latent_decode_tc_heads(m, eng.block_size) if eng.dtype == torch.bfloat16 else 0
-        if self.hg:
+        # tensor-core decode; other sizes and fp32 run the CUDA-core kernels
+        self.tc = eng.dtype == torch.bfloat16 and K.latent_decode_tc_ok(m, eng.block_size)
+        if self.tc:
             tiles = -(-(m.window or eng.max_len) // 128) + 1
-            ctas = B * -(-m.heads // self.hg)
+            ctas = B * -(-m.heads // 32)
             self.splits = max(1, min(8, tiles, 148 // ctas))
             self.q = eng.scratch("q", B, m.heads, m.dim + m.rot_dim)
             self.part_o = eng.scratch("part_o", B, m.heads * self.splits * m.kv_rank, dtype=torch.float32)
@@ -65,9 +65,9 @@ class _LatentSlots:
         from ..ops import cuda_mixers as K
 
         e = self.e
-        if self.hg:
+        if self.tc:
             K.latent_decode_tc(self.q_lat, self.cache, self.m, e.seq_lens, e.block_table, e.block_size, self.o_lat,
-                               self.part_o, self.part_ml, self.hg, self.splits)
+                               self.part_o, self.part_ml, self.splits)
         else:
             K.latent_decode(self.q_lat, self.cache, self.m, e.seq_lens, e.block_table, e.block_size, self.o_lat)
 
@@ -76,7 +76,7 @@ class _LatentSlots:
         from ..ops import cuda_mixers as K
 
         e, m = self.e, self.m
-        if self.hg:
+        if self.tc:
             K.latent_query(self.acc_q, m, e.seq_lens, self.table, self.q, self.q_lat)
             K.head_gemm(self.q, m.uk.view(m.heads, m.dim, m.kv_rank), self.q_lat, w_mn=True)
         else:
@@ -87,7 +87,7 @@ class _LatentSlots:
         from ..ops import cuda_mixers as K
 
         m = self.m
-        if self.hg:
+        if self.tc:
             K.head_gemm(self.o_lat, m.uv.view(m.heads, m.vdim, m.kv_rank), self.o.view(-1, m.heads, m.vdim), scale=self.gate)
         else:
             K.latent_expand(self.o_lat, m, self.gate, self.e.seq_lens, self.o)
@@ -264,4 +264,9 @@ class LayeredRolloutEngine(RolloutEngine):
     def _up_gelu(self, h, mlp):
         from ..ops import cuda_mixers as KM
 
-        return KM.gelu_erf(mx.linear(h, mlp.up), out=self.scratch("act", self.max_seqs, mlp.up.shape[0]))
+        act = self.scratch("act", self.max_seqs, mlp.up.shape[0])
+        if self._own_gemm and h.shape[1] % 8 == 0:
+            from ..ops import cuda as K
+
+            return K.decode_gemm(h, mlp.up, out=act, gelu=True)
+        return KM.gelu_erf(mx.linear(h, mlp.up), out=act)
