@@ -13,7 +13,7 @@
 //     the S buffer are reused for them (64 columns each), and P.V accumulates both products;
 //   * the softmax denominator contains exp(sink[head]) and the output is multiplied by a per-token, per-head gate;
 //   * keys are those of the same sequence at distance < window.
-#include "common.cuh"
+#include "mixers.cuh"
 
 namespace trlb {
 
@@ -136,19 +136,20 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_co
     if (lane == 0) {
       const uint32_t idesc_s = umma_idesc_bf16_major(LA_BM, LA_BN, false, false);
       const uint32_t idesc_o = umma_idesc_bf16_major(LA_BM, (p.vdim + 15) & ~15, false, true);  // V is MN-major
-      const uint32_t q_u = smem_u32(q_s), ks_u = smem_u32(k_s), vs_u = smem_u32(v_s);
+      const uint64_t q_d = umma_desc_kmajor_sw128(smem_u32(q_s)), k_d = umma_desc_kmajor_sw128(smem_u32(k_s));
+      const uint64_t v_d = umma_desc_mnmajor_sw128(smem_u32(v_s), LA_BOX);
       bool ok = mbar_wait(q_full, 0, abort_flag, p.status, 1210);
       auto issue_s = [&](int j) {
         const int s = j & 1, kst = j % p.k_stages;
         // buffer s is free: its P.V product (tile j - 2) was issued before this call
         if (!mbar_wait(&k_full[kst], (uint32_t)((j / p.k_stages) & 1), abort_flag, p.status, 1220 + kst)) return false;
         tc_fence_after();
-        const uint32_t k_u = ks_u + (uint32_t)kst * k_bytes;
+        const uint64_t k_t = desc_at(k_d, (uint32_t)kst * k_bytes);
         uint32_t acc = 0;
         for (int i = 0; i < p.nn + p.nr; ++i) {
           const int left = i < p.nn ? p.dim - 64 * i : p.rot - 64 * (i - p.nn);
           const int steps = min(4, (left + 15) >> 4);
-          const uint64_t da = umma_desc_kmajor_sw128(q_u + (uint32_t)i * LA_BOX), db = umma_desc_kmajor_sw128(k_u + (uint32_t)i * LA_BOX);
+          const uint64_t da = desc_at(q_d, (uint32_t)i * LA_BOX), db = desc_at(k_t, (uint32_t)i * LA_BOX);
           for (int kk = 0; kk < steps; ++kk) {
             umma_bf16_ss(tmem_base + (uint32_t)s * LA_BN, da + 2 * kk, db + 2 * kk, idesc_s, acc);
             acc = 1;
@@ -166,13 +167,13 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_co
         if (!mbar_wait(&p_full[sb], (uint32_t)((j >> 1) & 1), abort_flag, p.status, 1240 + sb)) break;
         if (!mbar_wait(&v_full[s], (uint32_t)((j / p.v_stages) & 1), abort_flag, p.status, 1250 + s)) break;
         tc_fence_after();
-        const uint32_t v_u = vs_u + (uint32_t)s * v_bytes;
+        const uint64_t v_t = desc_at(v_d, (uint32_t)s * v_bytes);
         // the S buffer holds P as bf16 pairs: leading parts in its first 64 columns, remainders in the other 64
         for (int half = 0; half < 2; ++half)
 #pragma unroll
           for (int kk = 0; kk < LA_BN / 16; ++kk)
             umma_bf16_ts(tmem_base + 256, tmem_base + (uint32_t)(sb * LA_BN + half * 64 + kk * 8),
-                         umma_desc_mnmajor_sw128(v_u + (uint32_t)kk * 2048, LA_BOX), idesc_o, (j | half | kk) != 0);
+                         desc_at(v_t, kk * 2048), idesc_o, (j | half | kk) != 0);
         umma_commit(o_full);
         umma_commit(&v_empty[s]);
       }

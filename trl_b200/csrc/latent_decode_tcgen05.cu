@@ -131,16 +131,19 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
     if (lane == 0 && n_t > 0) {
       constexpr uint32_t idesc_s = umma_idesc_bf16_major(128, HG, false, false);
       constexpr uint32_t idesc_o = umma_idesc_bf16_major(128, 2 * HG, true, true);
-      const uint32_t c_u = smem_u32(c_s), q_u = smem_u32(q_s), p_u = smem_u32(p_s);
+      const uint64_t c_k = umma_desc_kmajor_sw128(smem_u32(c_s)), q_k = umma_desc_kmajor_sw128(smem_u32(q_s));
+      const uint64_t c_mn = umma_desc_mnmajor_sw128(smem_u32(c_s), LD_BOX), p_mn = umma_desc_mnmajor_sw128(smem_u32(p_s), LD_BOX);
       bool ok = mbar_wait(q_full, 0, abort_flag, p.status, 1520);
       for (int j = 0; j < n_t && ok; ++j) {
+        uint64_t da = c_k, db = q_k;
         for (int i = 0; i < p.boxes && ok; ++i) {
           ok = mbar_wait(&full[i], (uint32_t)(j & 1), abort_flag, p.status, 1530 + i);
           if (!ok) break;
           tc_fence_after();
           const int steps = min(4, (p.lat_w - 64 * i + 15) >> 4);  // none for a box that only completes a slab
-          const uint64_t da = umma_desc_kmajor_sw128(c_u + (uint32_t)i * LD_BOX), db = umma_desc_kmajor_sw128(q_u + (uint32_t)(i * HG * 128));
           for (int kk = 0; kk < steps; ++kk) umma_bf16_ss(tmem_base, da + 2 * kk, db + 2 * kk, idesc_s, (i | kk) != 0);
+          da += LD_BOX >> 4;
+          db += (HG * 128) >> 4;
           if (i >= 2 * p.slabs) umma_commit(&empty[i]);
         }
         if (!ok) break;
@@ -148,11 +151,10 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
         if (!mbar_wait(p_full, (uint32_t)(j & 1), abort_flag, p.status, 1550)) break;
         tc_fence_after();
         for (int s = 0; s < p.slabs; ++s) {
+          const uint64_t ds = desc_at(c_mn, (uint32_t)(2 * s) * LD_BOX);
 #pragma unroll
           for (int kk = 0; kk < LD_TOK / 16; ++kk)
-            umma_bf16_ss(tmem_base + 64 + (uint32_t)(s * 2 * HG),
-                         umma_desc_mnmajor_sw128(c_u + (uint32_t)(2 * s) * LD_BOX + (uint32_t)kk * 2048, LD_BOX),
-                         umma_desc_mnmajor_sw128(p_u + (uint32_t)kk * 2048, LD_BOX), idesc_o, (j | kk) != 0);
+            umma_bf16_ss(tmem_base + 64 + (uint32_t)(s * 2 * HG), desc_at(ds, kk * 2048), desc_at(p_mn, kk * 2048), idesc_o, (j | kk) != 0);
           umma_commit(&empty[2 * s]);
           umma_commit(&empty[2 * s + 1]);
         }

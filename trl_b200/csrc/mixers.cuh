@@ -30,6 +30,10 @@ __device__ __forceinline__ float gelu_erf_f(float v) { return 0.5f * v * (1.f + 
 __device__ __forceinline__ float sigmoid_f(float z) { return 1.f / (1.f + expf(-z)); }
 __device__ __forceinline__ float log_sigmoid_f(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); }
 
+// A shared-memory matrix descriptor moved on by a multiple of 16 bytes (the address field cannot overflow inside 228 KB).  The
+// thread that issues MMAs runs alone, so what it computes per MMA is paid in full: descriptors are built once.
+__device__ __forceinline__ uint64_t desc_at(uint64_t desc, uint32_t bytes) { return desc + (bytes >> 4); }
+
 // Sums `a` and `b` over the block (at most 32 warps); `red` is 64 floats of shared memory.  All threads get the result.
 __device__ __forceinline__ float2 block_sum2(float a, float b, float* red) {
   const int lane = threadIdx.x & 31, wid = threadIdx.x >> 5, nw = blockDim.x >> 5;

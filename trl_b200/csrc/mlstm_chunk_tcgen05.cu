@@ -184,12 +184,12 @@ mlstm_state_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_consta
         if (!mbar_wait(&acc_empty[a], (uint32_t)(((c >> 1) & 1) ^ 1), abort_flag, p.status, 1310 + a)) break;
         if (!mbar_wait(&ready[s], (uint32_t)((c / MS_STAGES) & 1), abort_flag, p.status, 1320 + s)) break;
         tc_fence_after();
-        const uint32_t st = smem_u32(smem + (size_t)s * MS_STAGE_BYTES);
+        const uint64_t st = umma_desc_mnmajor_sw128(smem_u32(smem + (size_t)s * MS_STAGE_BYTES), ML_BOX);
+#pragma unroll
         for (int half = 0; half < 2; ++half)
 #pragma unroll
           for (int kk = 0; kk < ML_L / 16; ++kk)
-            umma_bf16_ss(tmem_base + (uint32_t)a * 64, umma_desc_mnmajor_sw128(st + (uint32_t)kk * 2048, ML_BOX),
-                         umma_desc_mnmajor_sw128(st + (uint32_t)(2 + half) * ML_BOX + (uint32_t)kk * 2048, ML_BOX), idesc,
+            umma_bf16_ss(tmem_base + (uint32_t)a * 64, desc_at(st, kk * 2048), desc_at(st, (2 + half) * ML_BOX + kk * 2048), idesc,
                          (half | kk) != 0);
         umma_commit(&acc_full[a]);
         umma_commit(&empty[s]);
@@ -422,7 +422,8 @@ mlstm_output_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
     if (lane == 0) {
       const uint32_t idesc_s = umma_idesc_bf16_major(128, 128, false, false);
       const uint32_t idesc_o = umma_idesc_bf16_major(128, n_cols, false, true);
-      const uint32_t q_u = smem_u32(q_s), r_u = smem_u32(ring);
+      const uint64_t q_k = umma_desc_kmajor_sw128(smem_u32(q_s)), r_k = umma_desc_kmajor_sw128(smem_u32(ring));
+      const uint64_t r_s = umma_desc_mnmajor_sw128(smem_u32(ring), 8192), r_v = umma_desc_mnmajor_sw128(smem_u32(ring), ML_BOX);
       bool ok = mbar_wait(q_full, 0, abort_flag, p.status, 1410);
       for (int it = 0; it < n_items && ok; ++it) {
         const int s = it % stages;
@@ -430,28 +431,32 @@ mlstm_output_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
         if (ok) ok = mbar_wait(&full[s], (uint32_t)((it / stages) & 1), abort_flag, p.status, 1420 + s);
         if (!ok) break;
         tc_fence_after();
-        const uint32_t st = r_u + (uint32_t)s * ML_BOX;
+        const uint32_t st = (uint32_t)s * ML_BOX;
         if (it < nd) {
           const int steps = min(4, (p.dim - 64 * it + 15) >> 4);
-          const uint64_t da = umma_desc_kmajor_sw128(q_u + (uint32_t)it * ML_BOX), db = umma_desc_kmajor_sw128(st);
-          for (int kk = 0; kk < steps; ++kk) umma_bf16_ss(tmem_base, da + 2 * kk, db + 2 * kk, idesc_s, (it | kk) != 0);
+          const uint64_t da = desc_at(q_k, (uint32_t)it * ML_BOX), db = desc_at(r_k, st);
+#pragma unroll
+          for (int kk = 0; kk < 4; ++kk)
+            if (kk < steps) umma_bf16_ss(tmem_base, da + 2 * kk, db + 2 * kk, idesc_s, (it | kk) != 0);
           if (it == nd - 1) umma_commit(s_full);
         } else if (it < nd + n_state) {
           const int i = (it - nd) >> 1;
           const int steps = min(4, (p.dim - 64 * i + 15) >> 4);
-          const uint64_t da = umma_desc_kmajor_sw128(q_u + (uint32_t)i * ML_BOX);
-          for (int kk = 0; kk < steps; ++kk)
-            umma_bf16_ss(tmem_base + 128, da + 2 * kk, umma_desc_mnmajor_sw128(st + (uint32_t)kk * 2048, 8192), idesc_o,
-                         (it > nd) || kk != 0);
+          const uint64_t da = desc_at(q_k, (uint32_t)i * ML_BOX), db = desc_at(r_s, st);
+#pragma unroll
+          for (int kk = 0; kk < 4; ++kk)
+            if (kk < steps) umma_bf16_ss(tmem_base + 128, da + 2 * kk, desc_at(db, kk * 2048), idesc_o, (it > nd) || kk != 0);
           if (it == nd + n_state - 1) umma_commit(x_full);
         } else {
           const int i = it - nd - n_state;
           const uint32_t idesc_v = umma_idesc_bf16_major(128, min(64, n_cols - 64 * i), false, true);
+          const uint64_t db = desc_at(r_v, st);
+#pragma unroll
           for (int half = 0; half < 2; ++half)
 #pragma unroll
             for (int kk = 0; kk < ML_L / 16; ++kk)
               umma_bf16_ts(tmem_base + 128 + 64 * i, tmem_base + (uint32_t)(half * 64 + kk * 8),
-                           umma_desc_mnmajor_sw128(st + (uint32_t)kk * 2048, ML_BOX), idesc_v, carried || (half | kk) != 0);
+                           desc_at(db, kk * 2048), idesc_v, carried || (half | kk) != 0);
           if (it == n_items - 1) umma_commit(o_full);
         }
         umma_commit(&empty[s]);
