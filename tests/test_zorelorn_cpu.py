@@ -166,3 +166,28 @@ def test_scheduler_grows_and_reuses_pages():
     assert s.grow(b, 24, bt) == 3 and len(set(bt[b, :6])) == 6
     with pytest.raises(ValueError):
         s.grow(b, 33, bt)
+
+
+def test_server_serves_a_checkpoint_without_tokenizer(tmp_path):
+    from trl_b200.scripts.rollout_serve import ServeArguments, WorkerPool
+
+    m, t = U.make(U.ODD)
+    m.save_pretrained(str(tmp_path))
+    pool = WorkerPool(ServeArguments(model=str(tmp_path), max_model_len=64))
+    try:
+        assert pool.tok is None
+        prompt = U.tokens(7, 203, 9)
+        out = pool.generate([prompt], {"max_tokens": 3, "generation_kwargs": {"greedy": True}})
+        seq = list(prompt)
+        for _ in range(3):
+            seq.append(int(U.logits(U.ODD, t, seq)[-1].argmax()))
+        assert out[0][1] == seq[7:]
+    finally:
+        pool.close()
+
+
+def test_replay_command_needs_the_documented_arguments():
+    from trl_b200.scripts.trace_run import main
+
+    with pytest.raises(SystemExit):
+        main(["--model", "x"])

@@ -444,3 +444,35 @@ def test_gradients_are_refused():
     m.requires_grad_(True)
     with pytest.raises(NotImplementedError, match="inference only"):
         m(torch.tensor([[1, 2, 3]], device="cuda"))
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_replay_command(tmp_path, dtype):
+    """bin/trace_run in a process of its own: unequal requests, requests that end, logits written in the order asked for."""
+    import json
+    import os
+    import subprocess
+    import sys
+
+    import numpy as np
+
+    m, t = U.make(U.ODD, torch.bfloat16)
+    m.save_pretrained(str(tmp_path / "m"))
+    (tmp_path / "out").mkdir()
+    a, wa = wanted("odd", 70, 1)
+    b, wb = wanted("odd", 70, 2)
+    steps = [{"step": 0, "entries": [{"id": "b", "tokens": b[:5], "want": [4, 0]}, {"id": "a", "tokens": a[:60], "want": [59]}], "end": []},
+             {"step": 1, "entries": [{"id": "a", "tokens": [a[60]], "want": []}, {"id": "b", "tokens": [b[5]], "want": []}], "end": ["b"]},
+             {"step": 2, "entries": [{"id": "a", "tokens": [a[61]], "want": [0]}], "end": ["a"]},
+             {"step": 3, "entries": [{"id": "b", "tokens": b[:9], "want": [8]}], "end": ["b"]}]
+    root = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
+    r = subprocess.run([sys.executable, os.path.join(root, "bin", "trace_run"), "--model", str(tmp_path / "m"), "--dtype", dtype,
+                        "--out", str(tmp_path / "out"), "--max-tokens", "80"], input="\n".join(map(json.dumps, steps)) + "\n",
+                       capture_output=True, text=True, timeout=300)
+    assert r.returncode == 0, r.stderr[-2000:]
+    assert [x for x in r.stdout.splitlines() if x.startswith("done")] == [f"done {i}" for i in range(4)]
+    want = {0: torch.stack([wb[4], wb[0], wa[59]]), 2: wa[61:62], 3: wb[8:9]}
+    assert sorted(os.listdir(tmp_path / "out")) == ["0.f32", "2.f32", "3.f32"]
+    for i, w in want.items():
+        got = torch.from_numpy(np.fromfile(tmp_path / "out" / f"{i}.f32", dtype="<f4").copy()).view(-1, 203)
+        assert U.rel(got, w) < TOL[getattr(torch, dtype)]

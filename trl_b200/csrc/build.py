@@ -1,9 +1,11 @@
 """Builds the in-tree native libraries.
 
-    python -m trl_b200.csrc.build [--force] [--verbose]
+    python -m trl_b200.csrc.build [--force] [--verbose] [--part layered]
 
 * ``trl_b200/_lib/libtrl_b200_kernels.so``  every ``*.cu`` here, compiled by nvcc for sm_100a only
   (``-gencode arch=compute_100a,code=sm_100a``); works without a GPU (cross-compile).
+* ``trl_b200/_lib/libtrl_b200_layered.so``  with ``--part layered``: only the sources that serving a layered decoder needs
+  (used when the whole kernel library has not been built).
 * ``trl_b200/_lib/libtrl_b200_host.so``     ``*.cpp`` host runtime (scheduler, packing), g++ -O3.
 
 Objects are cached next to the sources' hashes, so unchanged files are not recompiled.
@@ -27,6 +29,11 @@ NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", 
 # sources whose results the fast approximations of exp, tanh, erf, division and square root would show in
 EXACT_MATH = {"mixers.cu", "mlstm_chunk_tcgen05.cu"}
 # every source here builds into the one library used at any GPU count (no loads shared across a thread-block cluster)
+
+
+# parts of the kernel library that can be built alone
+PARTS = {"layered": ("decode.cu", "decode_gemm.cu", "latent_attn_tcgen05.cu", "latent_decode_tcgen05.cu", "mixers.cu",
+                     "mlstm_chunk_tcgen05.cu", "tensormap.cu")}
 
 
 def _nvcc() -> str:
@@ -69,16 +76,17 @@ def _compile(src: str, force: bool, verbose: bool) -> str:
     return obj
 
 
-def build(force: bool = False, verbose: bool = False) -> dict[str, str]:
+def build(force: bool = False, verbose: bool = False, part: str | None = None) -> dict[str, str]:
     os.makedirs(OBJ, exist_ok=True)
-    cus = sorted(os.path.join(HERE, f) for f in os.listdir(HERE) if f.endswith(".cu"))
+    cus = sorted(os.path.join(HERE, f) for f in os.listdir(HERE)
+                 if f.endswith(".cu") and (part is None or f in PARTS[part]))
     cpps = sorted(os.path.join(HERE, f) for f in os.listdir(HERE) if f.endswith(".cpp"))
     with cf.ThreadPoolExecutor(max_workers=min(8, os.cpu_count() or 2)) as ex:
         cu_objs = list(ex.map(lambda s: _compile(s, force, verbose), cus))
         cpp_objs = list(ex.map(lambda s: _compile(s, force, verbose), cpps))
     out = {}
     if cu_objs:
-        so = os.path.join(LIB, "libtrl_b200_kernels.so")
+        so = os.path.join(LIB, f"libtrl_b200_{part or 'kernels'}.so")
         if force or not os.path.exists(so) or any(os.path.getmtime(o) > os.path.getmtime(so) for o in cu_objs):
             cmd = [_nvcc(), "-shared", "-o", so] + cu_objs + ["-gencode", "arch=compute_100a,code=sm_100a",
                                                               "-Xcompiler", "-fPIC", "-cudart", "shared"]
@@ -100,8 +108,9 @@ def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--force", action="store_true")
     ap.add_argument("--verbose", action="store_true")
+    ap.add_argument("--part", choices=sorted(PARTS))
     a = ap.parse_args()
-    for k, v in build(a.force, a.verbose).items():
+    for k, v in build(a.force, a.verbose, a.part).items():
         print(f"{k}: {v}")
 
 

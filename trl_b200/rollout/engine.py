@@ -182,6 +182,8 @@ class RolloutEngine:
     def _check_model(self, max_model_len: int, block_size: int | None) -> int:
         """Raises if the decode kernels do not cover the model; returns the page size of its cache."""
         cfg = self.cfg
+        if getattr(self.model, "is_layered", False):
+            raise NotImplementedError("layered decoders are served by LayeredRolloutEngine (make_engine), on one GPU each")
         if cfg.num_attention_heads % self.tp or cfg.num_key_value_heads % self.tp:
             raise ValueError(f"tensor parallel size {self.tp} must divide the head counts")
         self.hq_local, self.hk_local = cfg.num_attention_heads // self.tp, cfg.num_key_value_heads // self.tp

@@ -67,6 +67,19 @@ def pack_tensors(named: list) -> tuple[dict, list]:
     return {"tensors": meta, "total": off}, parts
 
 
+def load_tokenizer(path: str):
+    """Tokenizer of a checkpoint directory; None for presets and for directories that hold none (prompts are then token
+    ids)."""
+    import os
+
+    if not any(os.path.exists(os.path.join(path, f)) for f in ("tokenizer.json", "tokenizer_config.json", "tokenizer.model",
+                                                               "vocab.json")):
+        return None
+    from transformers import AutoTokenizer
+
+    return AutoTokenizer.from_pretrained(path)
+
+
 class EngineHolder:
     def __init__(self, a: ServeArguments, device_index: int = 0, tp_group=None):
         import torch
@@ -79,13 +92,7 @@ class EngineHolder:
             torch.cuda.set_device(device_index)
         dt = (torch.bfloat16 if cuda else torch.float32) if a.dtype == "auto" else a.dtype
         self.model = load_model(a.model, dtype=dt, device=f"cuda:{device_index}" if cuda else None).eval()
-        self.tok = None
-        import os
-
-        if os.path.isdir(a.model):
-            from transformers import AutoTokenizer
-
-            self.tok = AutoTokenizer.from_pretrained(a.model)
+        self.tok = load_tokenizer(a.model)
         if cuda and tp_group is not None:
             from ..rollout.tp_engine import TPRolloutEngine
 
@@ -296,13 +303,7 @@ class WorkerPool:
         ready = [c.recv() for row in self.conns for c in row]  # blocks until every engine is built
         self.eos = ready[0]["eos"]
         self.world_size = self.dp * self.tp
-        self.tok = None
-        import os
-
-        if os.path.isdir(a.model):
-            from transformers import AutoTokenizer
-
-            self.tok = AutoTokenizer.from_pretrained(a.model)
+        self.tok = load_tokenizer(a.model)
 
     @staticmethod
     def _result(msg):
@@ -502,6 +503,8 @@ def build_app(holder_or_pool):
 
     @app.post("/generate/")
     async def generate(r: GenerateRequest):
+        if pool.tok is None and not all(isinstance(p, list) for p in r.prompts):
+            return {"error": "text prompts need a tokenizer (the served model has none): send token ids"}
         ids = [p if isinstance(p, list) else pool.tok(text=p)["input_ids"] for p in r.prompts]
         return _run(ids, r)
 

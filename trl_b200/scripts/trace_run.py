@@ -27,9 +27,12 @@ def main(argv=None) -> int:
     ap.add_argument("--max-seqs", type=int, default=16, help="slots of the engine (a larger first batch raises it)")
     a = ap.parse_args(argv)
 
+    from .._native import lib_path
     from ..csrc.build import build
+    from ..models.layered import is_layered_dir
 
-    build()
+    # a fresh checkout compiles what the model needs; an existing complete library is kept up to date
+    build(part="layered" if is_layered_dir(a.model) and not os.path.exists(lib_path("libtrl_b200_kernels.so")) else None)
     import torch
 
     from ..models.hf_io import load_model
