@@ -112,17 +112,17 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
       for (int i = 0; i < p.boxes; ++i) tma_load_3d(q_s + (size_t)i * HG * 128, &tm_q, q_full, 64 * i, h0, b);
       bool ok = true;
       for (int j = 0; j < n_t && ok; ++j) {
-        int rows[16];  // pages past the sequence's last one are masked: any page that exists will do
-#pragma unroll
-        for (int g = 0; g < 16; ++g)
-          rows[g] = g < ppt ? bt[min(page0 + (t_beg + j) * ppt + g, pos / p.block_size)] * p.block_size : 0;
+        // first cache row of page g of the tile (pages past the sequence's last one are masked: any page will do)
+        auto row_of = [&](int g) { return bt[min(page0 + (t_beg + j) * ppt + g, pos / p.block_size)] * p.block_size; };
+        const int row0 = row_of(0), row1 = row_of(ppt > 1 ? 1 : 0);
         for (int i = 0; i < p.boxes; ++i) {
           if (!mbar_wait(&empty[i], (uint32_t)((j & 1) ^ 1), abort_flag, p.status, 1500 + i)) { ok = false; break; }
           mbar_expect_tx(&full[i], LD_BOX);
-#pragma unroll
-          for (int g = 0; g < 16; ++g)
-            if (g < ppt)
-              tma_load_2d(c_s + (size_t)i * LD_BOX + (size_t)g * p.block_size * 128, &tm_c, &full[i], 64 * i, rows[g]);
+          uint8_t* dst = c_s + (size_t)i * LD_BOX;
+          tma_load_2d(dst, &tm_c, &full[i], 64 * i, row0);
+          if (ppt > 1) tma_load_2d(dst + p.block_size * 128, &tm_c, &full[i], 64 * i, row1);
+          for (int g = 2; g < ppt; ++g)  // pages shorter than 64 tokens
+            tma_load_2d(dst + g * p.block_size * 128, &tm_c, &full[i], 64 * i, row_of(g));
         }
       }
     }
@@ -141,7 +141,13 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
           if (!ok) break;
           tc_fence_after();
           const int steps = min(4, (p.lat_w - 64 * i + 15) >> 4);  // none for a box that only completes a slab
-          for (int kk = 0; kk < steps; ++kk) umma_bf16_ss(tmem_base, da + 2 * kk, db + 2 * kk, idesc_s, (i | kk) != 0);
+          // each step has an accumulator of its own (with so few columns the latency of one would show)
+          if (steps == 4) {
+#pragma unroll
+            for (int kk = 0; kk < 4; ++kk) umma_bf16_ss(tmem_base + kk * HG, da + 2 * kk, db + 2 * kk, idesc_s, i);
+          } else {
+            for (int kk = 0; kk < steps; ++kk) umma_bf16_ss(tmem_base + kk * HG, da + 2 * kk, db + 2 * kk, idesc_s, i);
+          }
           da += LD_BOX >> 4;
           db += (HG * 128) >> 4;
           if (i >= 2 * p.slabs) umma_commit(&empty[i]);
@@ -154,7 +160,7 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
           const uint64_t ds = desc_at(c_mn, (uint32_t)(2 * s) * LD_BOX);
 #pragma unroll
           for (int kk = 0; kk < LD_TOK / 16; ++kk)
-            umma_bf16_ss(tmem_base + 64 + (uint32_t)(s * 2 * HG), desc_at(ds, kk * 2048), desc_at(p_mn, kk * 2048), idesc_o, (j | kk) != 0);
+            umma_bf16_ss(tmem_base + 4 * HG + (uint32_t)(s * 2 * HG), desc_at(ds, kk * 2048), desc_at(p_mn, kk * 2048), idesc_o, (j | kk) != 0);
           umma_commit(&empty[2 * s]);
           umma_commit(&empty[2 * s + 1]);
         }
@@ -164,7 +170,7 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
     __syncwarp();
   } else if (n_t > 0) {
     const int w4 = warp & 3, r = w4 * 32 + lane;
-    const uint32_t ts = tmem_base + ((uint32_t)(w4 * 32) << 16), to = ts + 64;
+    const uint32_t ts = tmem_base + ((uint32_t)(w4 * 32) << 16), to = ts + 4 * HG;
     float m_ref = -INFINITY, l[HG];  // the reference maximum of head `lane`; per-head sums over this thread's tokens
 #pragma unroll
     for (int i = 0; i < HG; ++i) l[i] = 0.f;
@@ -179,6 +185,13 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
       float v[32], x[32];
       tmem_ld_32x32(ts, v);
       tmem_ld_wait();
+      const int parts = min(4, (p.lat_w + 15) >> 4);  // partial sums of S^T that hold something
+      for (int c = 1; c < parts; ++c) {
+        tmem_ld_32x32(ts + (uint32_t)(c * HG), x);
+        tmem_ld_wait();
+#pragma unroll
+        for (int i = 0; i < 32; ++i) v[i] += x[i];
+      }
 #pragma unroll
       for (int i = 0; i < 32; ++i) x[i] = v[i] = seen ? v[i] * p.scale_log2 : -INFINITY;
       float* mine = red + (j & 1) * 4 * HG;
@@ -495,7 +508,7 @@ TRLB_API int trlb_latent_decode_tc_ok(int heads, int dim, int rot, int vdim, int
   const int boxes = ld_boxes(kv_rank, lat_w);
   if (heads <= 0 || dim % 8 || rot % 8 || vdim <= 0 || kv_rank % 8 || lat_w % 8 || boxes > LD_MAX_BOX) return 0;
   if (block_size < 8 || block_size > 128 || 128 % block_size) return 0;
-  return 64 + ld_slabs(kv_rank) * 64 <= 512 && ld_smem(boxes) <= 227 * 1024;
+  return 4 * 32 + ld_slabs(kv_rank) * 64 <= 512 && ld_smem(boxes) <= 227 * 1024;
 }
 
 // q_lat [B, heads, lat_w], cache [num_blocks, block_size, lat_w] bf16 (lat_w as in csrc/mixers.cu), one new token per slot at
