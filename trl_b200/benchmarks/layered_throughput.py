@@ -175,7 +175,7 @@ def kernel_table(size="base", batch=64, prompt=1024, n_prompts=8, iters=20):
     row("prompt rotate_q", lambda: KM.rotate_q(q, la, ctx.positions, table), T * la.heads * la.rot_dim * 4)
     win = min(la.window or prompt, prompt)
     pairs = n_prompts * (win * (win + 1) / 2 + (prompt - win) * win)
-    row("prompt latent attention", lambda: KM.latent_prompt_tc(q, kv, lat, la, ctx.cu_seqlens, gate),
+    row("prompt latent attention", lambda: mx.latent_prompt_attention(q, kv, lat, la, ctx, gate),
         (q.numel() + kv.numel() + lat.numel() + T * la.heads * la.vdim) * 2,
         2 * pairs * la.heads * (la.dim + la.rot_dim + la.vdim))
     y = mx.linear(h, ml.w_in[: ml.gate_row])
@@ -217,7 +217,7 @@ def kernel_table(size="base", batch=64, prompt=1024, n_prompts=8, iters=20):
         r.state[0].numel() * 8 + r.acc_in.numel() * 4 + r.o32.numel() * 4)
     row("decode mlstm_out", lambda: KM.mlstm_out(r.o32, r.acc_in[:, qkv:], ml, r.y, clear=r.acc_in), r.acc_in.numel() * 4 + r.o32.numel() * 8)
     mlp = model.layers[0].mlp
-    row("decode up + gelu", lambda: eng._up_gelu(hb, mlp), mlp.up.numel() * 2)
+    row("decode up + gelu", lambda: eng.mlp_act(hb, mlp), mlp.up.numel() * 2)
     K.check_status()
     rows += flat_kernels(s, batch, prompt, n_prompts, row, rows)
     return rows

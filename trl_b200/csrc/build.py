@@ -27,13 +27,14 @@ OBJ = os.path.join(LIB, "obj")
 NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17", "--use_fast_math",
               "-Xcompiler", "-fPIC,-fvisibility=hidden", "-Xptxas", "-v", "--expt-relaxed-constexpr"]
 # sources whose results the fast approximations of exp, tanh, erf, division and square root would show in
-EXACT_MATH = {"mixers.cu", "mlstm_chunk_tcgen05.cu"}
+EXACT_MATH = {"grouped_attn.cu", "mixers.cu", "mlstm_chunk_tcgen05.cu", "rglru.cu", "rglru_tcgen05.cu"}
 # every source here builds into the one library used at any GPU count (no loads shared across a thread-block cluster)
 
 
 # parts of the kernel library that can be built alone
-PARTS = {"layered": ("decode.cu", "decode_gemm.cu", "latent_attn_tcgen05.cu", "latent_decode_tcgen05.cu", "mixers.cu",
-                     "mlstm_chunk_tcgen05.cu", "tensormap.cu")}
+PARTS = {"layered": ("decode.cu", "decode_gemm.cu", "grouped_attn.cu", "grouped_decode_tcgen05.cu", "latent_decode_tcgen05.cu",
+                     "mixer_attn_tcgen05.cu", "mixers.cu", "mlstm_chunk_tcgen05.cu", "rglru.cu", "rglru_tcgen05.cu",
+                     "tensormap.cu")}
 
 
 def _nvcc() -> str:

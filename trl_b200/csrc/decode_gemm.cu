@@ -23,7 +23,8 @@
 //     counter.  So each sum crosses NVLink once per peer whatever the stream-K split is, finished quarters go out
 //     while other SMs still stream weights, and the consumer waits only on its own counter;
 //   * whole-slab schedules store bf16 directly (+ bias), or apply SwiGLU: gate and up slabs of the same features go
-//     to two accumulators through alternate pipeline stages and the epilogue writes silu(gate) * up;
+//     to two accumulators through alternate pipeline stages and the epilogue writes silu(gate) * up (or the clamped
+//     gated unit g sigmoid(alpha g) (u + shift) of g = min(gate, limit), u = up clamped to [-limit, limit]);
 //   * W may be stored tile-major ([slab][K block][128][64], each 16 KB tile contiguous), which turns the weight
 //     stream into sequential DRAM bursts; tensor-parallel engines repack their weight slices anyway and use it;
 //   * the kernel is launched with programmatic stream serialization: barrier set-up, TMEM allocation and the first
@@ -41,7 +42,7 @@ constexpr int DG_THREADS = 192;
 constexpr uint32_t DG_W_BYTES = DG_BM * DG_BK * 2;
 constexpr int DG_MAX_PEERS = 7;
 
-enum { DG_ACCUM_F32 = 0, DG_STORE_BF16 = 1, DG_SWIGLU = 2, DG_GELU = 3 };
+enum { DG_ACCUM_F32 = 0, DG_STORE_BF16 = 1, DG_SWIGLU = 2, DG_GELU = 3, DG_CLAMPED_GLU = 4 };
 
 struct DecodeGemmParams {
   int B, N, K;
@@ -49,7 +50,8 @@ struct DecodeGemmParams {
   int mode;
   int tiled;           // W is tile-major
   int steps_per_slab;  // k_blocks (x 2 with SwiGLU: gate step, up step)
-  int up_slab_offset;  // SwiGLU: the up slab of features [128 j, 128 j + 128) is slab j + up_slab_offset of W
+  int up_slab_offset;  // SwiGLU, tile-major: the up slab of features [128 j, 128 j + 128) is slab j + up_slab_offset of W
+  float glu_limit, glu_alpha, glu_shift;  // DG_CLAMPED_GLU
   float* Y32;          // DG_ACCUM_F32: [B, ldy] fp32, added to
   __nv_bfloat16* Yb;   // DG_STORE_BF16 / DG_SWIGLU / DG_GELU: [B, ldy] bf16
   long long ldy;
@@ -187,10 +189,10 @@ decode_gemm_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_cons
       };
       auto load_w = [&](uint8_t* sa, uint64_t* bar, int t) {
         const int s = t % sps;
-        const int slab = t / sps + ((SWIGLU && (s & 1)) ? p.up_slab_offset : 0);
+        const bool up = SWIGLU && (s & 1);
         const int kb = SWIGLU ? (s >> 1) : s;
-        if (p.tiled) tma_load_2d(sa, &tmap_w, bar, 0, (slab * kbs + kb) * DG_BM);
-        else tma_load_2d(sa, &tmap_w, bar, kb * DG_BK, slab * DG_BM);
+        if (p.tiled) tma_load_2d(sa, &tmap_w, bar, 0, ((t / sps + (up ? p.up_slab_offset : 0)) * kbs + kb) * DG_BM);
+        else tma_load_2d(sa, &tmap_w, bar, kb * DG_BK, t / sps * DG_BM + (up ? p.N : 0));
       };
       // the first ring of weight tiles does not depend on the previous kernel
       for (int i = 0; i < n_pro; ++i) {
@@ -277,8 +279,16 @@ decode_gemm_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_cons
           float u[16];
           tmem_ld_32x16(tacc + BN + c, u);
           tmem_ld_wait();
+          if (p.mode == DG_CLAMPED_GLU) {
 #pragma unroll
-          for (int i = 0; i < 16; ++i) v[i] = v[i] / (1.f + __expf(-v[i])) * u[i];
+            for (int i = 0; i < 16; ++i) {
+              const float g = fminf(v[i], p.glu_limit), w = fminf(fmaxf(u[i], -p.glu_limit), p.glu_limit);
+              v[i] = g * fast_sigmoid(p.glu_alpha * g) * (w + p.glu_shift);
+            }
+          } else {
+#pragma unroll
+            for (int i = 0; i < 16; ++i) v[i] = v[i] / (1.f + __expf(-v[i])) * u[i];
+          }
         } else {
           tmem_ld_wait();
         }
@@ -380,8 +390,10 @@ int dg_launch(const CUtensorMap& tw, const CUtensorMap& tx, const DecodeGemmPara
   return (int)trlb_host::launch_kernel(kern, dim3(ctas), dim3(DG_THREADS), C::SMEM, st, trlb_host::pdl_enabled(), tw, tx, p);
 }
 
+bool dg_glu(int mode) { return mode == DG_SWIGLU || mode == DG_CLAMPED_GLU; }
+
 int dg_ctas_per_sm(int B, int mode) {
-  if (mode == DG_GELU) return 1;
+  if (mode == DG_GELU || mode == DG_CLAMPED_GLU) return 1;
   if (B > 64) return (mode == DG_SWIGLU || g_ctas_per_sm < 2) ? 1 : 2;  // 128-row tiles: 256 / 512 TMEM columns each
   if (mode == DG_SWIGLU) return 1;  // SwiGLU slabs cannot be split along K: one CTA per SM with a deep ring
   return g_ctas_per_sm;
@@ -423,6 +435,7 @@ TRLB_API int trlb_decode_gemm_arrivals(int N) { return 4 * ((N + DG_BM - 1) / DG
 //   mode 1  W [N, K];  Yb  [B, N] bf16 = X W^T (+ bias)
 //   mode 3  like mode 1 with the exact GELU of the sum stored
 //   mode 2  W [2N, K] (gate rows, then up rows; N a multiple of 128);  Yb [B, N] bf16 = silu(X Wg^T) * (X Wu^T)
+//   mode 4  W [2N, K] row-major, any N;  Yb [B, N] bf16 = clamped gated unit of both (glu = {limit, alpha, shift})
 // max_ctas: 0 = every SM with its resident CTAs, else an upper bound on the grid.
 // Fused all-reduce (mode 0, n_peers > 0): peer_y32[i] is the same buffer on peer i; arrive[0] is this rank's arrival
 // counter and arrive[1 + i] peer i's; stage is a local zeroed fp32 buffer shaped like Y32 and slab_ctr a local zeroed
@@ -432,9 +445,10 @@ TRLB_API int trlb_decode_gemm_arrivals(int N) { return 4 * ((N + DG_BM - 1) / DG
 TRLB_API int trlb_decode_gemm(const void* X, const void* W, const void* bias, float* Y32, void* Yb, int B, int N, int K,
                               long long ldx, long long ldw, long long ldy, int mode, int tiled, int max_ctas, int n_peers,
                               float* const* peer_y32, uint32_t* const* arrive, float* stage, uint32_t* slab_ctr,
-                              int* status, cudaStream_t st) {
+                              const float* glu, int* status, cudaStream_t st) {
   if (B <= 0 || N <= 0 || K <= 0) return 0;
-  if (B > 128 || (K % 8) != 0 || (ldx % 8) != 0 || mode < 0 || mode > 3) return -150;
+  if (B > 128 || (K % 8) != 0 || (ldx % 8) != 0 || mode < 0 || mode > 4) return -150;
+  if (mode == DG_CLAMPED_GLU && (bias != nullptr || tiled || glu == nullptr)) return -150;
   if (!tiled && (ldw % 8) != 0) return -150;
   if (mode == DG_SWIGLU && (bias != nullptr || (N % DG_BM) != 0)) return -150;
   if (n_peers < 0 || n_peers > DG_MAX_PEERS || (n_peers > 0 && (mode != DG_ACCUM_F32 || !peer_y32 || !arrive))) return -150;
@@ -442,12 +456,13 @@ TRLB_API int trlb_decode_gemm(const void* X, const void* W, const void* bias, fl
                       (reinterpret_cast<uintptr_t>(stage) & 15)))
     return -150;
   const int BN = B <= 64 ? 64 : 128;
-  const long long w_rows = mode == DG_SWIGLU ? 2LL * N : N;
+  const long long w_rows = dg_glu(mode) ? 2LL * N : N;
   DecodeGemmParams p = {};
   p.B = B; p.N = N; p.K = K; p.mode = mode; p.tiled = tiled ? 1 : 0;
   p.k_blocks = (K + DG_BK - 1) / DG_BK;
   p.slabs = (N + DG_BM - 1) / DG_BM;
-  p.steps_per_slab = p.k_blocks * (mode == DG_SWIGLU ? 2 : 1);
+  p.steps_per_slab = p.k_blocks * (dg_glu(mode) ? 2 : 1);
+  if (mode == DG_CLAMPED_GLU) { p.glu_limit = glu[0]; p.glu_alpha = glu[1]; p.glu_shift = glu[2]; }
   p.up_slab_offset = p.slabs;
   CUtensorMap tw, tx;
   if (tiled) {
@@ -463,12 +478,12 @@ TRLB_API int trlb_decode_gemm(const void* X, const void* W, const void* bias, fl
   for (int i = 0; i < n_peers; ++i) { p.peer_Y32[i] = peer_y32[i]; p.arrive[1 + i] = arrive[1 + i]; }
   const int ctas = trlb_decode_gemm_ctas(B, N, K, mode, max_ctas);
   if (BN == 64) {
-    if (mode == DG_SWIGLU) return dg_launch<64, true, 8, 1>(tw, tx, p, ctas, st);
+    if (dg_glu(mode)) return dg_launch<64, true, 8, 1>(tw, tx, p, ctas, st);
     if (mode == DG_GELU) return dg_launch<64, false, 8, 1>(tw, tx, p, ctas, st);  // one slab per CTA: a deep ring
     if (g_ctas_per_sm == 3) return dg_launch<64, false, 3, 3>(tw, tx, p, ctas, st);
     return dg_launch<64, false, 4, 2>(tw, tx, p, ctas, st);
   }
-  if (mode == DG_SWIGLU) return dg_launch<128, true, 6, 1>(tw, tx, p, ctas, st);
+  if (dg_glu(mode)) return dg_launch<128, true, 6, 1>(tw, tx, p, ctas, st);
   if (mode == DG_GELU) return dg_launch<128, false, 6, 1>(tw, tx, p, ctas, st);
   if (g_ctas_per_sm < 2) return dg_launch<128, false, 6, 1>(tw, tx, p, ctas, st);
   return dg_launch<128, false, 3, 2>(tw, tx, p, ctas, st);

@@ -1,0 +1,333 @@
+// Grouped-query attention of the layered decoders: preparation of queries, keys and values, and attention on the CUDA
+// cores for every size and dtype (tcgen05 forms: mixer_attn_tcgen05.cu for prompts, grouped_decode_tcgen05.cu for decode).
+//
+// T is the model dtype (bf16 or fp32); norms, scores, softmax and its sums are fp32 in both.  Compiled without fast-math
+// (csrc/build.py: EXACT_MATH).  In decode kernels seq_lens[slot] is the position of the slot's new token, negative: idle.
+#include "mixers.cuh"
+
+namespace trlb {
+
+// ------------------------------------------------------------------------------------------------------------
+// From the projections of a layer's input, rows [q | k | v | g] (no k and v in a layer that reads another one's cache):
+// queries divided by their rms per head and multiplied by the temperature of their position, keys divided by their rms,
+// keys and values to the paged cache.  S is the dtype of the rows: T (prompt: q and k are replaced in place, v and g stay
+// where they are) or fp32 sums (decode: q and the gate logits go to buffers, everything read is zeroed).
+// One warp per (row, head of q / k / v / g).
+// ------------------------------------------------------------------------------------------------------------
+struct AttnPrep {
+  long long ld;
+  int rows, heads, kv_heads, dim, vdim, has_kv, has_gate;
+  float eps;
+  const int* positions;   // [rows]
+  const int* tok_slot;    // [rows] or null (slot = row)
+  const float* temp;      // [temp_len] factor of the query by position, or null
+  int temp_len;
+  const int* block_table;  // null: no cache
+  int max_blocks, block_size;
+};
+
+template <typename T, typename S>
+__global__ void __launch_bounds__(256)
+attn_prep_kernel(const AttnPrep p, S* __restrict__ src, T* __restrict__ q_out, T* __restrict__ g_out, T* __restrict__ k_cache,
+                 T* __restrict__ v_cache) {
+  constexpr bool SUMS = !(sizeof(T) == 2 && sizeof(S) == 2);  // fp32 models: q_out tells (null: in place)
+  pdl_launch_dependents();
+  pdl_wait();
+  const int lane = threadIdx.x & 31;
+  const int kv = p.has_kv ? p.kv_heads : 0, units = p.heads + 2 * kv + (p.has_gate && g_out != nullptr ? p.heads : 0);
+  const long long item = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
+  if (item >= (long long)p.rows * units) return;
+  const int row = (int)(item / units), u = (int)(item % units);
+  const int pos = p.positions[row];
+  const bool in_place = !SUMS || q_out == nullptr;
+  S* r = src + (size_t)row * p.ld;
+  const int q_n = p.heads * p.dim, k_n = kv * p.dim, v_n = kv * p.vdim;
+  S* x;
+  int n;
+  bool normed = false;
+  T* dst = nullptr;    // besides the cache
+  T* paged = nullptr;
+  float mul = 1.f;
+  long long at = -1;   // token's row in the cache
+  if (pos >= 0 && p.block_table != nullptr && u >= p.heads && u < p.heads + 2 * kv) {
+    const int slot = p.tok_slot ? p.tok_slot[row] : row;
+    if (slot >= 0 && pos / p.block_size < p.max_blocks)
+      at = (long long)p.block_table[(size_t)slot * p.max_blocks + pos / p.block_size] * p.block_size + pos % p.block_size;
+  }
+  if (u < p.heads) {
+    x = r + (size_t)u * p.dim;
+    n = p.dim;
+    normed = true;
+    if (p.temp != nullptr && pos >= 0 && pos < p.temp_len) mul = p.temp[pos];
+    if (!in_place) dst = q_out + ((size_t)row * p.heads + u) * p.dim;
+  } else if (u < p.heads + kv) {
+    const int h = u - p.heads;
+    x = r + q_n + (size_t)h * p.dim;
+    n = p.dim;
+    normed = true;
+    if (at >= 0) paged = k_cache + (size_t)(at * kv + h) * p.dim;
+  } else if (u < p.heads + 2 * kv) {
+    const int h = u - p.heads - kv;
+    x = r + q_n + k_n + (size_t)h * p.vdim;
+    n = p.vdim;
+    if (at >= 0) paged = v_cache + (size_t)(at * kv + h) * p.vdim;
+  } else {
+    const int h = u - p.heads - 2 * kv;
+    x = r + q_n + k_n + v_n + (size_t)h * p.vdim;
+    n = p.vdim;
+    dst = g_out + ((size_t)row * p.heads + h) * p.vdim;
+  }
+  const bool vec = ((n | (int)p.ld | (int)(x - r)) & 3) == 0 && (reinterpret_cast<uintptr_t>(src) & (4 * sizeof(S) - 1)) == 0;
+  float s = 1.f;
+  if (normed) {
+    float ss = 0.f;
+    if (vec) {
+      for (int j = 4 * lane; j < n; j += 128) {
+        const float4 v = load4(x + j);
+        ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+      }
+    } else {
+      for (int j = lane; j < n; j += 32) ss += to_f(x[j]) * to_f(x[j]);
+    }
+    s = mul / sqrtf(warp_sum(ss) / (float)n + p.eps);
+  }
+  if (vec) {
+    for (int j = 4 * lane; j < n; j += 128) {
+      float4 v = load4(x + j);
+      v = make_float4(v.x * s, v.y * s, v.z * s, v.w * s);
+      if (dst) store4(dst + j, v);
+      if (paged) store4(paged + j, v);
+      if (!in_place) store4(x + j, make_float4(0.f, 0.f, 0.f, 0.f));
+      else if (normed) store4(x + j, v);
+    }
+  } else {
+    for (int j = lane; j < n; j += 32) {
+      const float v = to_f(x[j]) * s;
+      if (dst) dst[j] = from_f<T>(v);
+      if (paged) paged[j] = from_f<T>(v);
+      if (!in_place) x[j] = from_f<S>(0.f);
+      else if (normed) x[j] = from_f<S>(v);
+    }
+  }
+}
+
+// ------------------------------------------------------------------------------------------------------------
+// Prompt attention, any size: one warp per (token, head).  Keys of token t are rows t - min(pos, window - 1) .. t of the
+// packed stream (pos counts from the token's own sequence start), so no sequence table is needed.  Keys may have a second
+// part of `rot` elements shared by the heads; scores may be capped; sink and gate may be null.
+// ------------------------------------------------------------------------------------------------------------
+struct MixerAttn {
+  int T, heads, group, dim, rot, vdim, window;
+  long long q_ld, k_ld, v_ld, kr_ld, gate_ld;
+  float scale, cap;
+  const int* positions;
+  const float* sink;       // [heads] or null
+  int gate_mode;           // 0 none, 1 fp32 [T, heads], 2 logits of T [T rows of gate_ld]
+  const float* head_gate;
+};
+
+__device__ __forceinline__ float capped(float s, float cap) { return cap > 0.f ? cap * tanhf(s / cap) : s; }
+
+template <typename T>
+__global__ void __launch_bounds__(128)
+mixer_attn_kernel(const MixerAttn p, const T* __restrict__ q, const T* __restrict__ k, const T* __restrict__ v,
+                  const T* __restrict__ krot, const T* __restrict__ gate, T* __restrict__ out) {
+  extern __shared__ float sm[];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const long long item = (long long)blockIdx.x * 4 + warp;
+  if (item >= (long long)p.T * p.heads) return;
+  const int t = (int)(item / p.heads), h = (int)(item % p.heads), hk = h / p.group;
+  const int dq = p.dim + p.rot;
+  float* qs = sm + (size_t)warp * (dq + p.vdim);
+  float* os = qs + dq;
+  for (int d = lane; d < dq; d += 32) qs[d] = to_f(q[(size_t)t * p.q_ld + (size_t)h * dq + d]);
+  for (int e = lane; e < p.vdim; e += 32) os[e] = 0.f;
+  __syncwarp();
+  const int pos = p.positions[t];
+  const int back = p.window > 0 ? min(pos, p.window - 1) : pos;
+  const int k0 = t - back;
+  float m = -INFINITY, l = 0.f;
+  for (int base = k0; base <= t; base += 32) {
+    const int key = base + lane;
+    float s = -INFINITY;
+    if (key <= t) {
+      const T* kn = k + (size_t)key * p.k_ld + (size_t)hk * p.dim;
+      float acc = 0.f;
+      for (int d = 0; d < p.dim; ++d) acc += qs[d] * to_f(kn[d]);
+      if (p.rot > 0) {
+        const T* kr = krot + (size_t)key * p.kr_ld;
+        for (int d = 0; d < p.rot; ++d) acc += qs[p.dim + d] * to_f(kr[d]);
+      }
+      s = capped(acc * p.scale, p.cap);
+    }
+    const float mn = fmaxf(m, warp_max(s));
+    const float corr = m == -INFINITY ? 0.f : expf(m - mn);
+    const float pr = key <= t ? expf(s - mn) : 0.f;
+    l = l * corr + warp_sum(pr);
+    m = mn;
+    const int nk = min(32, t - base + 1);
+    const int e_end = (p.vdim + 31) & ~31;
+    for (int e = lane; e < e_end; e += 32) {
+      float acc = e < p.vdim ? os[e] * corr : 0.f;
+      for (int j = 0; j < nk; ++j) {
+        const float w = __shfl_sync(0xffffffffu, pr, j);
+        if (e < p.vdim) acc += w * to_f(v[(size_t)(base + j) * p.v_ld + (size_t)hk * p.vdim + e]);
+      }
+      if (e < p.vdim) os[e] = acc;
+    }
+    __syncwarp();
+  }
+  const float sk = p.sink != nullptr ? p.sink[h] : -INFINITY, mt = fmaxf(m, sk);
+  float f = expf(m - mt) / (l * expf(m - mt) + expf(sk - mt));
+  if (p.gate_mode == 1) f *= p.head_gate[(size_t)t * p.heads + h];
+  for (int e = lane; e < p.vdim; e += 32) {
+    float o = os[e] * f;
+    if (p.gate_mode == 2) o *= sigmoid_f(to_f(gate[(size_t)t * p.gate_ld + (size_t)h * p.vdim + e]));
+    out[((size_t)t * p.heads + h) * p.vdim + e] = from_f<T>(o);
+  }
+}
+
+// ------------------------------------------------------------------------------------------------------------
+// Decode attention over the paged cache, any size with dim, vdim <= 1024: one block per (slot, head), the four warps take
+// keys in turn, lanes own dimensions.
+// ------------------------------------------------------------------------------------------------------------
+struct GroupedDecode {
+  int B, heads, kv_heads, dim, vdim, max_blocks, block_size;
+  float scale, cap;
+  const int* seq_lens;
+  const int* block_table;
+};
+
+constexpr int GD_MAX_REG = 32;
+template <typename T>
+__global__ void __launch_bounds__(128)
+grouped_decode_kernel(const GroupedDecode p, const T* __restrict__ q, const T* __restrict__ k_cache, const T* __restrict__ v_cache,
+                      const T* __restrict__ gate, T* __restrict__ out) {
+  extern __shared__ float sm[];  // [dim] query, [4][vdim] partial outputs, [8] max / sum
+  pdl_launch_dependents();
+  pdl_wait();
+  const int b = blockIdx.y, h = blockIdx.x, hk = h / (p.heads / p.kv_heads), warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int pos = p.seq_lens[b];
+  if (pos < 0 || pos >= p.max_blocks * p.block_size) return;
+  float* qs = sm;
+  float* po = sm + p.dim;
+  float* ml = po + 4 * p.vdim;
+  for (int d = threadIdx.x; d < p.dim; d += 128) qs[d] = to_f(q[((size_t)b * p.heads + h) * p.dim + d]);
+  __syncthreads();
+  const int* bt = p.block_table + (size_t)b * p.max_blocks;
+  float m = -INFINITY, l = 0.f, acc[GD_MAX_REG];
+#pragma unroll
+  for (int i = 0; i < GD_MAX_REG; ++i) acc[i] = 0.f;
+  for (int j = warp; j <= pos; j += 4) {
+    const size_t row = ((size_t)bt[j / p.block_size] * p.block_size + j % p.block_size) * p.kv_heads + hk;
+    const T* kr = k_cache + row * p.dim;
+    const T* vr = v_cache + row * p.vdim;
+    float s = 0.f;
+    for (int d = lane; d < p.dim; d += 32) s += to_f(kr[d]) * qs[d];
+    s = capped(warp_sum(s) * p.scale, p.cap);
+    const float mn = fmaxf(m, s), corr = m == -INFINITY ? 0.f : expf(m - mn), w = expf(s - mn);
+    l = l * corr + w;
+    m = mn;
+#pragma unroll
+    for (int i = 0; i < GD_MAX_REG; ++i) {
+      const int e = lane + 32 * i;
+      if (e < p.vdim) acc[i] = acc[i] * corr + w * to_f(vr[e]);
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < GD_MAX_REG; ++i) {
+    const int e = lane + 32 * i;
+    if (e < p.vdim) po[(size_t)warp * p.vdim + e] = acc[i];
+  }
+  if (lane == 0) { ml[warp] = m; ml[4 + warp] = l; }
+  __syncthreads();
+  float mt = ml[0], den = 0.f, f[4];  // warp 0 always has a key
+  for (int w = 1; w < 4; ++w) mt = fmaxf(mt, ml[w]);
+  for (int w = 0; w < 4; ++w) {
+    f[w] = ml[w] == -INFINITY ? 0.f : expf(ml[w] - mt);
+    den += f[w] * ml[4 + w];
+  }
+  for (int e = threadIdx.x; e < p.vdim; e += 128) {
+    float o = 0.f;
+    for (int w = 0; w < 4; ++w) o += f[w] * po[(size_t)w * p.vdim + e];
+    o /= den;
+    const size_t i = ((size_t)b * p.heads + h) * p.vdim + e;
+    if (gate != nullptr) o *= sigmoid_f(to_f(gate[i]));
+    out[i] = from_f<T>(o);
+  }
+}
+
+}  // namespace trlb
+
+using namespace trlb;
+
+namespace {
+
+template <typename K>
+bool allow_smem(K kern, size_t bytes) {
+  if (bytes <= 48 * 1024) return true;
+  if (bytes > 227 * 1024) return false;
+  return cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes) == cudaSuccess;
+}
+
+using bf16 = __nv_bfloat16;
+
+}  // namespace
+
+#define PDL trlb_host::pdl_enabled()
+
+// rows [q | k | v | g] of ld elements; src_f32: fp32 sums (decode: q_out and g_out given), else the model dtype.  temp, tok_slot,
+// block_table may be null.
+TRLB_API int trlb_attn_prep(void* src, int src_f32, long long ld, int rows, int heads, int kv_heads, int dim, int vdim, int has_kv,
+                            int has_gate, float eps, const int* positions, const int* tok_slot, const float* temp, int temp_len,
+                            void* q_out, void* g_out, void* k_cache, void* v_cache, const int* block_table, int max_blocks,
+                            int block_size, int is_bf16, cudaStream_t st) {
+  if (rows <= 0) return 0;
+  if (heads <= 0 || kv_heads <= 0 || heads % kv_heads || (is_bf16 && src_f32 && q_out == nullptr)) return -250;
+  AttnPrep p = {ld, rows, heads, kv_heads, dim, vdim, has_kv, has_gate, eps, positions, tok_slot, temp, temp_len,
+                k_cache ? block_table : nullptr, max_blocks, block_size};
+  const int units = heads + (has_kv ? 2 * kv_heads : 0) + (has_gate && g_out != nullptr ? heads : 0);
+  const dim3 grid((unsigned)(((long long)rows * units + 7) / 8)), blk(256);
+#define GO(TT, SS) (int)trlb_host::launch_kernel(attn_prep_kernel<TT, SS>, grid, blk, 0, st, PDL, p, (SS*)src, (TT*)q_out, (TT*)g_out, (TT*)k_cache, (TT*)v_cache)
+  if (is_bf16) return src_f32 ? GO(bf16, float) : GO(bf16, bf16);
+  return GO(float, float);
+#undef GO
+}
+
+// Arguments as trlb_mixer_attn_tc (mixer_attn_tcgen05.cu), in either dtype and any size; positions instead of sequence starts.
+TRLB_API int trlb_mixer_attn(const void* q, long long q_ld, const void* k, long long k_ld, const void* v, long long v_ld,
+                             const void* krot, long long krot_ld, const int* positions, int T, int heads, int kv_heads, int dim,
+                             int rot, int vdim, int window, float scale, float cap, const float* sink, int gate_mode,
+                             const void* gate, long long gate_ld, void* out, int is_bf16, cudaStream_t st) {
+  if (T <= 0) return 0;
+  if (heads <= 0 || kv_heads <= 0 || heads % kv_heads) return -251;
+  MixerAttn p = {T, heads, heads / kv_heads, dim, rot, vdim, window, q_ld, k_ld, v_ld, krot_ld, gate_ld, scale, cap, positions,
+                 sink, gate_mode, gate_mode == 1 ? (const float*)gate : nullptr};
+  const int grid = (int)(((long long)T * heads + 3) / 4);
+  const size_t smem = (size_t)4 * (dim + rot + vdim) * 4;
+  if (is_bf16) {
+    if (!allow_smem(mixer_attn_kernel<bf16>, smem)) return -252;
+    mixer_attn_kernel<bf16><<<grid, 128, smem, st>>>(p, (const bf16*)q, (const bf16*)k, (const bf16*)v, (const bf16*)krot,
+                                                     gate_mode == 2 ? (const bf16*)gate : nullptr, (bf16*)out);
+  } else {
+    if (!allow_smem(mixer_attn_kernel<float>, smem)) return -252;
+    mixer_attn_kernel<float><<<grid, 128, smem, st>>>(p, (const float*)q, (const float*)k, (const float*)v, (const float*)krot,
+                                                      gate_mode == 2 ? (const float*)gate : nullptr, (float*)out);
+  }
+  return (int)cudaGetLastError();
+}
+
+// q [B, heads, dim], k_cache [blocks, block_size, kv_heads, dim], v_cache [.., vdim], gate logits [B, heads, vdim] or null.
+TRLB_API int trlb_grouped_decode(const void* q, const void* k_cache, const void* v_cache, const void* gate, void* out, int B,
+                                 int heads, int kv_heads, int dim, int vdim, float scale, float cap, const int* seq_lens,
+                                 const int* block_table, int max_blocks, int block_size, int is_bf16, cudaStream_t st) {
+  if (B <= 0) return 0;
+  if (heads <= 0 || kv_heads <= 0 || heads % kv_heads || vdim > 32 * GD_MAX_REG) return -253;
+  GroupedDecode p = {B, heads, kv_heads, dim, vdim, max_blocks, block_size, scale, cap, seq_lens, block_table};
+  const size_t smem = (size_t)(dim + 4 * vdim + 8) * 4;
+  if (smem > 48 * 1024) return -253;
+  const dim3 grid(heads, B), blk(128);
+#define GO(TT) (int)trlb_host::launch_kernel(grouped_decode_kernel<TT>, grid, blk, smem, st, PDL, p, (const TT*)q, (const TT*)k_cache, (const TT*)v_cache, (const TT*)gate, (TT*)out)
+  return is_bf16 ? GO(bf16) : GO(float);
+#undef GO
+}

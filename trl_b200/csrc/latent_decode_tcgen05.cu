@@ -296,7 +296,7 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
   }
 }
 
-// o_lat[b, h] = (sum over splits) / (sum of exponentials + exp(sink)).  One block per (head, slot).
+// o_lat[b, h] = (sum over splits) / (sum of exponentials + exp(sink), no such term when sink is null).  One block per (head, slot).
 __global__ void __launch_bounds__(128)
 latent_combine_kernel(const float* __restrict__ part_o, const float2* __restrict__ part_ml, const float* __restrict__ sink,
                       const int* __restrict__ seq_lens, int heads, int kv_rank, int splits, __nv_bfloat16* __restrict__ o_lat) {
@@ -305,7 +305,7 @@ latent_combine_kernel(const float* __restrict__ part_o, const float2* __restrict
   const int h = blockIdx.x, b = blockIdx.y;
   if (seq_lens[b] < 0) return;
   const size_t bh = (size_t)b * heads + h;
-  const float sk = sink[h] * 1.4426950408889634f;
+  const float sk = sink != nullptr ? sink[h] * 1.4426950408889634f : -INFINITY;
   float m = sk;
   for (int s = 0; s < splits; ++s) m = fmaxf(m, part_ml[bh * splits + s].x);
   float den = exp2f(sk - m);

@@ -1,18 +1,23 @@
-// Prompt attention of the latent-attention mixer on the 5th-generation tensor cores (bf16, packed sequences).
+// Prompt attention of the layered decoders' mixers on the 5th-generation tensor cores (bf16, packed sequences).
 //
 // The structure is that of fa_varlen_tcgen05.cu (one CTA per 128-query tile and head; TMA warp, MMA warp, one softmax
 // thread per query row; S double-buffered in TMEM, O accumulated in TMEM and rescaled only when a row's reference
 // maximum moves by more than 2^8).  What differs:
 //
-//   * a query / key vector has two parts that live in different tensors: `dim` elements per head (queries in q, keys in
-//     the up-projected kv rows) and `rot` rotated elements (in q behind the first part; keys in the latent rows, ONE
-//     for all heads).  Each part is loaded as 64-column TMA boxes of its own, zero-filled past its end, so nothing is
-//     concatenated or expanded in memory; Q.K^T runs over the 16-column steps that hold data;
+//   * a query / key vector may have two parts that live in different tensors: `dim` elements per head and `rot` rotated
+//     elements (in q behind the first part; keys in rows of their own, ONE for all heads).  Each part is loaded as
+//     64-column TMA boxes, zero-filled past its end, so nothing is concatenated or expanded in memory; Q.K^T runs over
+//     the 16-column steps that hold data.  rot = 0: no such part;
+//   * groups of heads / kv_heads query heads read one key / value head;
 //   * sizes are launch parameters: dim, rot, vdim any multiples of 8 (vdim <= 256) that leave room for one stage;
 //   * probabilities keep 32-bit precision into P.V: each is split into two bf16 (value and remainder), both halves of
 //     the S buffer are reused for them (64 columns each), and P.V accumulates both products;
-//   * the softmax denominator contains exp(sink[head]) and the output is multiplied by a per-token, per-head gate;
-//   * keys are those of the same sequence at distance < window.
+//   * scores may be capped, cap tanh(s / cap) (CAP): a series near zero, where scores of normed queries and keys lie, so
+//     that the special-function units are left to the exponentials;
+//   * the softmax denominator may contain exp(sink[head]);
+//   * the output may be multiplied by a gate: one fp32 factor per token and head, or the sigmoid of bf16 logits per
+//     element;
+//   * keys are those of the same sequence, with a window those at distance < window.
 #include "mixers.cuh"
 
 namespace trlb {
@@ -21,14 +26,19 @@ constexpr int LA_BM = 128, LA_BN = 128;
 constexpr int LA_THREADS = 192;
 constexpr uint32_t LA_BOX = 128 * 64 * 2;  // one TMA box: 128 rows x 64 bf16, 128-byte swizzle
 
-struct LatentTcParams {
+enum { GATE_NONE = 0, GATE_HEAD = 1, GATE_LOGITS = 2 };
+
+struct MixerAttnTc {
   const int* cu;
-  int n_seq, heads, dim, rot, vdim, window;
+  int n_seq, heads, group, dim, rot, vdim, window;
   int nn, nr, nv;      // boxes of the unrotated part, the rotated part and the value
   int k_stages, v_stages;
-  float scale_log2;
-  const float* sink;
-  const float* gate;   // [T, heads]
+  float scale_log2;    // CAP: 1 (capped scores are in log2 units already)
+  float cap_in, cap_out;  // CAP: scale / cap, cap log2(e)
+  const float* sink;   // [heads] or null
+  int gate_mode;
+  const void* gate;    // GATE_HEAD: fp32 [T, heads]; GATE_LOGITS: bf16 [T, gate_ld >= heads vdim]
+  long long gate_ld;
   __nv_bfloat16* out;  // [T, heads, vdim]
   int* status;
 };
@@ -42,10 +52,11 @@ __device__ __forceinline__ bool la_find_tile(const int* cu, int n_seq, int slot,
   return false;
 }
 
+template <bool CAP>
 __global__ void __launch_bounds__(LA_THREADS, 1)
-latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_constant__ CUtensorMap tm_qr,
+mixer_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_constant__ CUtensorMap tm_qr,
                       const __grid_constant__ CUtensorMap tm_kn, const __grid_constant__ CUtensorMap tm_kr,
-                      const __grid_constant__ CUtensorMap tm_v, const LatentTcParams p) {
+                      const __grid_constant__ CUtensorMap tm_v, const MixerAttnTc p) {
   int seq, tile;
   if (!la_find_tile(p.cu, p.n_seq, (int)blockIdx.x, seq, tile)) return;  // uniform: before any barrier or TMEM use
   extern __shared__ uint8_t smem_raw[];
@@ -67,7 +78,7 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_co
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int h = blockIdx.y;
+  const int h = blockIdx.y, hk = h / p.group;
   const int beg = p.cu[seq], len = p.cu[seq + 1] - beg;
   const int q_first = tile * LA_BM;
   const int q_last = min(len, q_first + LA_BM) - 1;
@@ -115,7 +126,7 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_co
         uint8_t* ks = k_s + (size_t)s * k_bytes;
         const int row = beg + (lo + j) * LA_BN;
         mbar_expect_tx(&k_full[s], k_bytes);
-        for (int i = 0; i < p.nn; ++i) tma_load_3d(ks + i * LA_BOX, &tm_kn, &k_full[s], 64 * i, h, row);
+        for (int i = 0; i < p.nn; ++i) tma_load_3d(ks + i * LA_BOX, &tm_kn, &k_full[s], 64 * i, hk, row);
         for (int i = 0; i < p.nr; ++i) tma_load_2d(ks + (p.nn + i) * LA_BOX, &tm_kr, &k_full[s], 64 * i, row);
         return true;
       };
@@ -127,7 +138,7 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_co
         if (!mbar_wait(&v_empty[s], (uint32_t)(((j / p.v_stages) & 1) ^ 1), abort_flag, p.status, 1205 + s)) break;
         uint8_t* vs = v_s + (size_t)s * v_bytes;
         mbar_expect_tx(&v_full[s], v_bytes);
-        for (int i = 0; i < p.nv; ++i) tma_load_3d(vs + i * LA_BOX, &tm_v, &v_full[s], 64 * i, h, beg + (lo + j) * LA_BN);
+        for (int i = 0; i < p.nv; ++i) tma_load_3d(vs + i * LA_BOX, &tm_v, &v_full[s], 64 * i, hk, beg + (lo + j) * LA_BN);
       }
     }
     __syncwarp();
@@ -204,6 +215,27 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_co
 #pragma unroll
       for (int c = 0; c < 4; ++c) tmem_ld_32x32(ts + 32 * c, v[c]);
       tmem_ld_wait();
+      if (CAP) {
+        float top = 0.f;
+#pragma unroll
+        for (int c = 0; c < 4; ++c)
+#pragma unroll
+          for (int i = 0; i < 32; ++i) {
+            v[c][i] *= p.cap_in;
+            top = fmaxf(top, fabsf(v[c][i]));
+          }
+        if (__any_sync(0xffffffffu, top > CAP_SERIES)) {
+#pragma unroll
+          for (int c = 0; c < 4; ++c)
+#pragma unroll
+            for (int i = 0; i < 32; ++i) v[c][i] = p.cap_out * tanh_exp(v[c][i]);
+        } else {
+#pragma unroll
+          for (int c = 0; c < 4; ++c)
+#pragma unroll
+            for (int i = 0; i < 32; ++i) v[c][i] = p.cap_out * tanh_series(v[c][i]);
+        }
+      }
       if (!full) {
 #pragma unroll
         for (int c = 0; c < 4; ++c)
@@ -275,11 +307,14 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_co
         tc_fence_after();
         float f = 0.f;
         __nv_bfloat16* dst = nullptr;
+        const __nv_bfloat16* gl = nullptr;
         if (row_ok) {
-          const float sk = p.sink[h] * 1.4426950408889634f, mt = fmaxf(m_ref, sk);
+          const size_t t = (size_t)(beg + q_pos), th = t * p.heads + h;
+          const float sk = p.sink != nullptr ? p.sink[h] * 1.4426950408889634f : -INFINITY, mt = fmaxf(m_ref, sk);
           const float wm = fast_exp2(m_ref - mt);
-          const size_t th = (size_t)(beg + q_pos) * p.heads + h;
-          f = wm / (l_run * wm + fast_exp2(sk - mt)) * p.gate[th];
+          f = wm / (l_run * wm + fast_exp2(sk - mt));
+          if (p.gate_mode == GATE_HEAD) f *= reinterpret_cast<const float*>(p.gate)[th];
+          if (p.gate_mode == GATE_LOGITS) gl = reinterpret_cast<const __nv_bfloat16*>(p.gate) + t * p.gate_ld + (size_t)h * p.vdim;
           dst = p.out + th * p.vdim;
         }
 #pragma unroll 1
@@ -290,10 +325,23 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_co
           if (row_ok) {
 #pragma unroll
             for (int i = 0; i < 16; i += 8)
-              if (c + i < p.vdim)
+              if (c + i < p.vdim) {
+#pragma unroll
+                for (int q = 0; q < 8; ++q) o[i + q] *= f;
+                if (gl != nullptr) {
+                  const uint4 g = *reinterpret_cast<const uint4*>(gl + c + i);
+                  const uint32_t w[4] = {g.x, g.y, g.z, g.w};
+#pragma unroll
+                  for (int q = 0; q < 4; ++q) {
+                    const float2 z = unpack_bf16(w[q]);
+                    o[i + 2 * q] *= fast_sigmoid(z.x);
+                    o[i + 2 * q + 1] *= fast_sigmoid(z.y);
+                  }
+                }
                 *reinterpret_cast<uint4*>(dst + c + i) =
-                    make_uint4(pack_bf16(o[i] * f, o[i + 1] * f), pack_bf16(o[i + 2] * f, o[i + 3] * f),
-                               pack_bf16(o[i + 4] * f, o[i + 5] * f), pack_bf16(o[i + 6] * f, o[i + 7] * f));
+                    make_uint4(pack_bf16(o[i], o[i + 1]), pack_bf16(o[i + 2], o[i + 3]), pack_bf16(o[i + 4], o[i + 5]),
+                               pack_bf16(o[i + 6], o[i + 7]));
+              }
           }
         }
         tc_fence_before();
@@ -332,45 +380,55 @@ int la_boxes(int n) { return (n + 63) / 64; }
 
 }  // namespace
 
-// 1 when trlb_latent_attn_tc takes these sizes.
-TRLB_API int trlb_latent_attn_tc_ok(int heads, int dim, int rot, int vdim) {
+// 1 when trlb_mixer_attn_tc takes these sizes.
+TRLB_API int trlb_mixer_attn_tc_ok(int heads, int kv_heads, int dim, int rot, int vdim) {
   int ks, vs;
-  return dim > 0 && rot > 0 && vdim > 0 && dim % 8 == 0 && rot % 8 == 0 && vdim % 8 == 0 && vdim <= 256 && heads > 0 &&
-         la_stages(la_boxes(dim) + la_boxes(rot), la_boxes(vdim), ks, vs);
+  return dim > 0 && rot >= 0 && vdim > 0 && dim % 8 == 0 && rot % 8 == 0 && vdim % 8 == 0 && vdim <= 256 && heads > 0 &&
+         kv_heads > 0 && heads % kv_heads == 0 && la_stages(la_boxes(dim) + la_boxes(rot), la_boxes(vdim), ks, vs);
 }
 
-// q [T, heads, dim + rot] (rotated part last), kv [T, kv_ld]: heads * dim keys then heads * vdim values, krot [T, krot_ld]:
-// the shared rotated keys; all bf16, 16-byte aligned rows.  window <= 0: unlimited.  scale > 0.
-TRLB_API int trlb_latent_attn_tc(const void* q, const void* kv, long long kv_ld, const void* krot, long long krot_ld,
-                                 const int* cu, int n_seq, int T, int heads, int dim, int rot, int vdim, int window,
-                                 float scale, const float* sink, const float* gate, void* out, int* status,
-                                 cudaStream_t st) {
+// q [T rows of q_ld]: heads x (dim + rot), rotated part last; k, v [T rows of k_ld / v_ld]: kv_heads x dim / vdim; krot [T rows
+// of krot_ld]: the shared rotated keys (rot > 0).  All bf16, rows on 16 bytes.  window <= 0: unlimited; cap <= 0: none; scale > 0;
+// sink may be null; gate by gate_mode (0 none, 1 fp32 [T, heads], 2 bf16 logits [T rows of gate_ld]).
+TRLB_API int trlb_mixer_attn_tc(const void* q, long long q_ld, const void* k, long long k_ld, const void* v, long long v_ld,
+                                const void* krot, long long krot_ld, const int* cu, int n_seq, int T, int heads, int kv_heads,
+                                int dim, int rot, int vdim, int window, float scale, float cap, const float* sink,
+                                int gate_mode, const void* gate, long long gate_ld, void* out, int* status, cudaStream_t st) {
   if (T <= 0 || n_seq <= 0) return 0;
-  if (!trlb_latent_attn_tc_ok(heads, dim, rot, vdim) || (kv_ld % 8) || (krot_ld % 8) || !(scale > 0.f)) return -210;
-  LatentTcParams p = {};
-  p.cu = cu; p.n_seq = n_seq; p.heads = heads; p.dim = dim; p.rot = rot; p.vdim = vdim; p.window = window;
+  if (!trlb_mixer_attn_tc_ok(heads, kv_heads, dim, rot, vdim) || (q_ld % 8) || (k_ld % 8) || (v_ld % 8) || !(scale > 0.f)) return -210;
+  if (rot > 0 && (krot_ld % 8)) return -210;
+  if (gate_mode == GATE_LOGITS && ((gate_ld % 8) || (reinterpret_cast<uintptr_t>(gate) & 15))) return -210;
+  MixerAttnTc p = {};
+  p.cu = cu; p.n_seq = n_seq; p.heads = heads; p.group = heads / kv_heads; p.dim = dim; p.rot = rot; p.vdim = vdim; p.window = window;
   p.nn = la_boxes(dim); p.nr = la_boxes(rot); p.nv = la_boxes(vdim);
   la_stages(p.nn + p.nr, p.nv, p.k_stages, p.v_stages);
-  p.scale_log2 = scale * 1.4426950408889634f;
-  p.sink = sink; p.gate = gate; p.out = (__nv_bfloat16*)out; p.status = status;
+  p.scale_log2 = cap > 0.f ? 1.f : scale * 1.4426950408889634f;
+  p.cap_in = cap > 0.f ? scale / cap : 0.f;
+  p.cap_out = cap * 1.4426950408889634f;
+  p.sink = sink; p.gate_mode = gate_mode; p.gate = gate; p.gate_ld = gate_ld; p.out = (__nv_bfloat16*)out; p.status = status;
   const __nv_bfloat16* qb = (const __nv_bfloat16*)q;
-  const __nv_bfloat16* kb = (const __nv_bfloat16*)kv;
   const int dq = dim + rot;
   CUtensorMap tqn, tqr, tkn, tkr, tv;
   using trlb_host::make_tmap_3d_bf16;
-  if (make_tmap_3d_bf16(&tqn, qb, dim, heads, T, dq, (uint64_t)heads * dq, 64, 1, 128)) return -211;
-  if (make_tmap_3d_bf16(&tqr, qb + dim, rot, heads, T, dq, (uint64_t)heads * dq, 64, 1, 128)) return -212;
-  if (make_tmap_3d_bf16(&tkn, kb, dim, heads, T, dim, (uint64_t)kv_ld, 64, 1, 128)) return -213;
-  if (trlb_host::make_tmap_2d_bf16(&tkr, krot, T, rot, (uint64_t)krot_ld, 128, 64)) return -214;
-  if (make_tmap_3d_bf16(&tv, kb + (size_t)heads * dim, vdim, heads, T, vdim, (uint64_t)kv_ld, 64, 1, 128)) return -215;
+  if (make_tmap_3d_bf16(&tqn, qb, dim, heads, T, dq, (uint64_t)q_ld, 64, 1, 128)) return -211;
+  if (make_tmap_3d_bf16(&tkn, k, dim, kv_heads, T, dim, (uint64_t)k_ld, 64, 1, 128)) return -213;
+  if (make_tmap_3d_bf16(&tv, v, vdim, kv_heads, T, vdim, (uint64_t)v_ld, 64, 1, 128)) return -215;
+  tqr = tqn;
+  tkr = tkn;
+  if (rot > 0) {
+    if (make_tmap_3d_bf16(&tqr, qb + dim, rot, heads, T, dq, (uint64_t)q_ld, 64, 1, 128)) return -212;
+    if (trlb_host::make_tmap_2d_bf16(&tkr, krot, T, rot, (uint64_t)krot_ld, 128, 64)) return -214;
+  }
   static bool attr_set = false;
   if (!attr_set) {
-    if (cudaFuncSetAttribute(latent_attn_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024) != cudaSuccess)
+    if (cudaFuncSetAttribute(mixer_attn_tc_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024) != cudaSuccess ||
+        cudaFuncSetAttribute(mixer_attn_tc_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024) != cudaSuccess)
       return -216;
     attr_set = true;
   }
-  const int max_tiles = (T + LA_BM - 1) / LA_BM + n_seq;
-  latent_attn_tc_kernel<<<dim3(max_tiles, heads), LA_THREADS, la_smem(p.nn + p.nr, p.nv, p.k_stages, p.v_stages), st>>>(
-      tqn, tqr, tkn, tkr, tv, p);
+  const dim3 grid((T + LA_BM - 1) / LA_BM + n_seq, heads);
+  const size_t smem = la_smem(p.nn + p.nr, p.nv, p.k_stages, p.v_stages);
+  if (cap > 0.f) mixer_attn_tc_kernel<true><<<grid, LA_THREADS, smem, st>>>(tqn, tqr, tkn, tkr, tv, p);
+  else mixer_attn_tc_kernel<false><<<grid, LA_THREADS, smem, st>>>(tqn, tqr, tkn, tkr, tv, p);
   return (int)cudaGetLastError();
 }

@@ -1,5 +1,7 @@
-// Element-wise, cache and recurrence kernels of the layered decoders (models/layered.py): embedding scale, Dynamic-Tanh
-// norm fused with the residual addition, latent-attention preparation / absorption, mLSTM gates, steps and outputs.
+// Element-wise, cache and recurrence kernels of the layered decoders (models/layered.py): embedding scale, Dynamic-Tanh and
+// RMS norms fused with the residual addition, clamped gated linear unit, per-token side inputs, latent-attention
+// preparation / absorption, mLSTM gates, steps and outputs.  Grouped-query attention is in grouped_attn.cu, the real-gated
+// linear recurrent unit in rglru.cu.
 //
 // T is the model dtype (bf16 or fp32).  The residual stream, norm statistics, gates, attention scores and recurrent
 // states are fp32 in both.  This file is compiled without fast-math (csrc/build.py: EXACT_MATH).
@@ -7,9 +9,6 @@
 // Decode kernels work on one row per sequence slot; seq_lens[slot] is the position of the slot's new token and a
 // negative value marks an idle slot.  fp32 sums of the stream-K decode GEMM are cleared by their last reader
 // (`clear`), so no memset runs between two steps.
-//
-// The latent-attention prompt kernel here covers every size and dtype; bf16 prompts with 8-element aligned head
-// sizes run the tcgen05 kernel of latent_attn_tcgen05.cu.
 #include "mixers.cuh"
 
 namespace trlb {
@@ -84,6 +83,144 @@ gelu_erf_kernel(const T* __restrict__ z, T* __restrict__ out, long long n) {
 }
 
 // ------------------------------------------------------------------------------------------------------------
+// RMS norms around the residual stream, in one pass over a row:
+//     x += delta                      or, with `post`,   x += delta / rms(delta) * post
+//     out = x / rms(x) * w            or, without `w`,   out = x
+// `clear` zeroes delta behind itself.  One block per row; NV float4 of the row live in each thread's registers.
+// ------------------------------------------------------------------------------------------------------------
+struct RmsResidual {
+  float* x;
+  float* delta;        // null: nothing is added
+  const float* post;   // null: delta is added as it is
+  const float* w;      // null: the sum itself is the output
+  int H, clear;
+  float eps;
+};
+
+template <typename T, int NV>
+__global__ void __launch_bounds__(256)
+rms_residual_kernel(const RmsResidual p, T* __restrict__ out) {
+  __shared__ float red[64];
+  pdl_launch_dependents();
+  pdl_wait();
+  const size_t row = (size_t)blockIdx.x * p.H;
+  const int n4 = p.H / 4, nt = blockDim.x;
+  float4 a[NV], d[NV];
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int j = threadIdx.x + i * nt;
+    a[i] = j < n4 ? load4(p.x + row + 4 * j) : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+  if (p.delta != nullptr) {
+    float sd = 0.f;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int j = threadIdx.x + i * nt;
+      d[i] = j < n4 ? load4(p.delta + row + 4 * j) : make_float4(0.f, 0.f, 0.f, 0.f);
+      sd += d[i].x * d[i].x + d[i].y * d[i].y + d[i].z * d[i].z + d[i].w * d[i].w;
+    }
+    float r = 1.f;
+    if (p.post != nullptr) r = 1.f / sqrtf(block_sum2(sd, 0.f, red).x / (float)p.H + p.eps);
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int j = threadIdx.x + i * nt;
+      if (j < n4) {
+        const float4 g = p.post != nullptr ? load4(p.post + 4 * j) : make_float4(1.f, 1.f, 1.f, 1.f);
+        a[i].x += d[i].x * r * g.x; a[i].y += d[i].y * r * g.y; a[i].z += d[i].z * r * g.z; a[i].w += d[i].w * r * g.w;
+        store4(p.x + row + 4 * j, a[i]);
+        if (p.clear) store4(p.delta + row + 4 * j, make_float4(0.f, 0.f, 0.f, 0.f));
+      }
+    }
+  }
+  float r = 1.f;
+  if (p.w != nullptr) {
+    float s = 0.f;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) s += a[i].x * a[i].x + a[i].y * a[i].y + a[i].z * a[i].z + a[i].w * a[i].w;
+    r = 1.f / sqrtf(block_sum2(s, 0.f, red).x / (float)p.H + p.eps);
+  }
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int j = threadIdx.x + i * nt;
+    if (j < n4) {
+      const float4 g = p.w != nullptr ? load4(p.w + 4 * j) : make_float4(1.f, 1.f, 1.f, 1.f);
+      store4(out + row + 4 * j, make_float4(a[i].x * r * g.x, a[i].y * r * g.y, a[i].z * r * g.z, a[i].w * r * g.w));
+    }
+  }
+}
+
+// The same for any row length.
+template <typename T>
+__global__ void __launch_bounds__(256)
+rms_residual_any_kernel(const RmsResidual p, T* __restrict__ out) {
+  __shared__ float red[64];
+  pdl_launch_dependents();
+  pdl_wait();
+  const size_t row = (size_t)blockIdx.x * p.H;
+  float* x = p.x + row;
+  float* d = p.delta == nullptr ? nullptr : p.delta + row;
+  float r = 1.f, s = 0.f;
+  if (d != nullptr && p.post != nullptr) {
+    for (int j = threadIdx.x; j < p.H; j += 256) s += d[j] * d[j];
+    r = 1.f / sqrtf(block_sum2(s, 0.f, red).x / (float)p.H + p.eps);
+  }
+  s = 0.f;
+  for (int j = threadIdx.x; j < p.H; j += 256) {
+    float a = x[j];
+    if (d != nullptr) {
+      a += p.post != nullptr ? d[j] * r * p.post[j] : d[j];
+      x[j] = a;
+      if (p.clear) d[j] = 0.f;
+    }
+    s += a * a;
+  }
+  float rx = 1.f;
+  if (p.w != nullptr) rx = 1.f / sqrtf(block_sum2(s, 0.f, red).x / (float)p.H + p.eps);
+  for (int j = threadIdx.x; j < p.H; j += 256) out[row + j] = from_f<T>(p.w != nullptr ? x[j] * rx * p.w[j] : x[j]);
+}
+
+// Clamped gated linear unit: z [rows, 2 n] = gate | up -> g sigmoid(alpha g) (u + shift), g = min(gate, limit), u = up clamped
+// to [-limit, limit].
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256)
+clamped_glu_kernel(const T* __restrict__ z, T* __restrict__ out, long long total, int n, float limit, float alpha, float shift) {
+  const int per = n / VEC;
+  for (long long v = blockIdx.x * (long long)blockDim.x + threadIdx.x; v < total; v += (long long)gridDim.x * blockDim.x) {
+    const long long row = v / per;
+    const int j = (int)(v % per) * VEC;
+    const T* zr = z + row * 2 * n + j;
+    auto act = [&](float g, float u) {
+      g = fminf(g, limit);
+      u = fminf(fmaxf(u, -limit), limit);
+      return g * sigmoid_t<T>(alpha * g) * (u + shift);
+    };
+    if (VEC == 4) {
+      const float4 g = load4(zr), u = load4(zr + n);
+      store4(out + row * n + j, make_float4(act(g.x, u.x), act(g.y, u.y), act(g.z, u.z), act(g.w, u.w)));
+    } else {
+      out[row * n + j] = from_f<T>(act(to_f(zr[0]), to_f(zr[n])));
+    }
+  }
+}
+
+// Side input of a layer: out[row] = gelu_tanh(z[row]) * table[ids[row], off : off + n].  Z: dtype of z; `clear` zeroes it.
+template <typename T, typename Z>
+__global__ void __launch_bounds__(128)
+side_gate_kernel(Z* __restrict__ z, const long long* __restrict__ ids, const T* __restrict__ table, long long table_ld, int off,
+                 int n, int V, int clear, T* __restrict__ out) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const size_t row = blockIdx.x;
+  const long long id = ids[row];
+  const bool ok = id >= 0 && id < V;
+  for (int j = threadIdx.x; j < n; j += blockDim.x) {
+    const float e = ok ? to_f(table[(size_t)id * table_ld + off + j]) : 0.f;
+    out[row * n + j] = from_f<T>(gelu_tanh_t<T>(to_f(z[row * n + j])) * e);
+    if (clear) z[row * n + j] = from_f<Z>(0.f);
+  }
+}
+
+// ------------------------------------------------------------------------------------------------------------
 // latent attention
 // ------------------------------------------------------------------------------------------------------------
 struct LatentPrep {
@@ -95,7 +232,7 @@ struct LatentPrep {
   float eps;
   const int* positions;  // [rows] position of every row (prompt) or of every slot (decode); negative: idle
   const int* tok_slot;   // [rows] or null (slot = row)
-  const float2* table;   // [table_len, rot / 2] (cos, sin) with the rotation's magnitude folded in
+  const float2* table;   // [table_len, rot / 2] (cos, sin) with the rotation's magnitude folded in; unused if rot == 0
   int table_len;
   float* gate;           // [rows, heads] sigmoid of the gate logits
   int kr_off, lat_w;     // a latent row: [kv_rank | pad to kr_off | rot | pad to lat_w]
@@ -115,7 +252,7 @@ latent_prep_kernel(const LatentPrep p, T* __restrict__ cq, T* __restrict__ lat, 
   const float* ar = akv + p.kv_rank;
   const float* ag = ar + p.rot;
   float sq = 0.f, sk = 0.f;
-  const bool vec = ((p.q_rank | p.kv_rank | (int)p.ld) & 3) == 0;
+  const bool vec = ((p.q_rank | p.kv_rank | (int)p.ld) & 3) == 0 && (reinterpret_cast<uintptr_t>(p.acc) & 15) == 0;
   if (vec) {
 #pragma unroll 2
     for (int j = 4 * threadIdx.x; j < p.q_rank; j += 4 * blockDim.x) {
@@ -131,7 +268,7 @@ latent_prep_kernel(const LatentPrep p, T* __restrict__ cq, T* __restrict__ lat, 
     for (int j = threadIdx.x; j < p.kv_rank; j += blockDim.x) sk += akv[j] * akv[j];
   }
   const float2 s = block_sum2(sq, sk, red);
-  const float rq = 1.f / sqrtf(s.x / (float)p.q_rank + p.eps), rk = 1.f / sqrtf(s.y / (float)p.kv_rank + p.eps);
+  const float rq = p.q_rank > 0 ? 1.f / sqrtf(s.x / (float)p.q_rank + p.eps) : 0.f, rk = 1.f / sqrtf(s.y / (float)p.kv_rank + p.eps);
   const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
   if (vec) {
 #pragma unroll 2
@@ -151,7 +288,7 @@ latent_prep_kernel(const LatentPrep p, T* __restrict__ cq, T* __restrict__ lat, 
     if (p.clear) a[p.q_rank + p.kv_rank + p.rot + h] = 0.f;
   }
   const int pos = p.positions[row];
-  const bool live = pos >= 0 && pos < p.table_len;
+  const bool live = pos >= 0 && (p.rot == 0 || pos < p.table_len);
   T* dense = lat == nullptr ? nullptr : lat + (size_t)row * p.lat_w;
   T* paged = nullptr;
   if (live && p.block_table != nullptr) {
@@ -215,70 +352,6 @@ rotate_q_kernel(T* __restrict__ q, int heads, int dim, int rot, const int* __res
   }
 }
 
-// Prompt attention, any size: one warp per (token, head).  Keys of token t are rows t - min(pos, window - 1) .. t of
-// the packed stream (pos counts from the token's own sequence start), so no sequence table is needed.
-struct LatentPrompt {
-  int T, heads, dim, rot, vdim, kr_off, lat_w, window;
-  long long kv_ld;  // kv row: [heads * dim keys | heads * vdim values]
-  float scale;
-  const int* positions;
-  const float* sink;
-  const float* gate;  // [T, heads]
-};
-
-template <typename T>
-__global__ void __launch_bounds__(128)
-latent_prompt_kernel(const LatentPrompt p, const T* __restrict__ q, const T* __restrict__ kv, const T* __restrict__ lat,
-                     T* __restrict__ out) {
-  extern __shared__ float sm[];
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const long long item = (long long)blockIdx.x * 4 + warp;
-  if (item >= (long long)p.T * p.heads) return;
-  const int t = (int)(item / p.heads), h = (int)(item % p.heads);
-  const int dq = p.dim + p.rot;
-  float* qs = sm + (size_t)warp * (dq + p.vdim);
-  float* os = qs + dq;
-  for (int d = lane; d < dq; d += 32) qs[d] = to_f(q[((size_t)t * p.heads + h) * dq + d]);
-  for (int e = lane; e < p.vdim; e += 32) os[e] = 0.f;
-  __syncwarp();
-  const int pos = p.positions[t];
-  const int back = p.window > 0 ? min(pos, p.window - 1) : pos;
-  const int k0 = t - back;
-  float m = -INFINITY, l = 0.f;
-  for (int base = k0; base <= t; base += 32) {
-    const int key = base + lane;
-    float s = -INFINITY;
-    if (key <= t) {
-      const T* kn = kv + (size_t)key * p.kv_ld + (size_t)h * p.dim;
-      const T* kr = lat + (size_t)key * p.lat_w + p.kr_off;
-      float acc = 0.f;
-      for (int d = 0; d < p.dim; ++d) acc += qs[d] * to_f(kn[d]);
-      for (int d = 0; d < p.rot; ++d) acc += qs[p.dim + d] * to_f(kr[d]);
-      s = acc * p.scale;
-    }
-    const float mn = fmaxf(m, warp_max(s));
-    const float corr = m == -INFINITY ? 0.f : expf(m - mn);
-    const float pr = key <= t ? expf(s - mn) : 0.f;
-    l = l * corr + warp_sum(pr);
-    m = mn;
-    const int nk = min(32, t - base + 1);
-    const int e_end = (p.vdim + 31) & ~31;
-    for (int e = lane; e < e_end; e += 32) {
-      float acc = e < p.vdim ? os[e] * corr : 0.f;
-      for (int j = 0; j < nk; ++j) {
-        const float w = __shfl_sync(0xffffffffu, pr, j);
-        if (e < p.vdim)
-          acc += w * to_f(kv[(size_t)(base + j) * p.kv_ld + (size_t)p.heads * p.dim + (size_t)h * p.vdim + e]);
-      }
-      if (e < p.vdim) os[e] = acc;
-    }
-    __syncwarp();
-  }
-  const float sk = p.sink[h], mt = fmaxf(m, sk);
-  const float f = expf(m - mt) / (l * expf(m - mt) + expf(sk - mt)) * p.gate[(size_t)t * p.heads + h];
-  for (int e = lane; e < p.vdim; e += 32) out[((size_t)t * p.heads + h) * p.vdim + e] = from_f<T>(os[e] * f);
-}
-
 // Decode, any size.  Absorption: q_lat[b, h] = [ W_uk[h]^T q_nope | rotated q_rot ] in the layout of a latent row.
 template <typename T>
 __global__ void __launch_bounds__(128)
@@ -297,7 +370,7 @@ latent_absorb_kernel(float* __restrict__ qacc, long long ld, const T* __restrict
   }
   __syncthreads();
   const int pos = positions[b];
-  if (pos < 0 || pos >= table_len) return;
+  if (pos < 0 || (rot > 0 && pos >= table_len)) return;
   T* dst = q_lat + ((size_t)b * heads + h) * lat_w;
   for (int r = threadIdx.x; r < lat_w; r += blockDim.x) {
     float v = 0.f;
@@ -319,7 +392,7 @@ struct LatentDecode {
   float scale;
   const int* seq_lens;
   const int* block_table;
-  const float* sink;
+  const float* sink;  // [heads] or null
 };
 
 // One block per (slot, head, split): the four warps take keys in turn, lanes own dimensions of the latent row.
@@ -366,7 +439,7 @@ latent_decode_kernel(const LatentDecode p, const T* __restrict__ q_lat, const T*
   }
   if (lane == 0) { ml[warp] = m; ml[4 + warp] = l; }
   __syncthreads();
-  const float sk = p.sink[h];
+  const float sk = p.sink != nullptr ? p.sink[h] : -INFINITY;
   float mt = sk;
   for (int w = 0; w < 4; ++w) mt = fmaxf(mt, ml[w]);
   float den = expf(sk - mt), f[4];
@@ -381,7 +454,7 @@ latent_decode_kernel(const LatentDecode p, const T* __restrict__ q_lat, const T*
   }
 }
 
-// out[b, h, e] = gate[b, h] * sum_r uv[h, e, r] o_lat[b, h, r]
+// out[b, h, e] = gate[b, h] (1 without gates) * sum_r uv[h, e, r] o_lat[b, h, r]
 template <typename T>
 __global__ void __launch_bounds__(128)
 latent_expand_kernel(const T* __restrict__ o_lat, const T* __restrict__ uv, const float* __restrict__ gate,
@@ -393,7 +466,7 @@ latent_expand_kernel(const T* __restrict__ o_lat, const T* __restrict__ uv, cons
   const bool live = positions[b] >= 0;
   for (int r = threadIdx.x; r < kv_rank; r += 128) sm[r] = live ? to_f(o_lat[((size_t)b * heads + h) * kv_rank + r]) : 0.f;
   __syncthreads();
-  const float g = gate[(size_t)b * heads + h];
+  const float g = gate != nullptr ? gate[(size_t)b * heads + h] : 1.f;
   for (int e = warp; e < vdim; e += 4) {
     const T* w = uv + ((size_t)h * vdim + e) * kv_rank;
     float v = 0.f;
@@ -669,6 +742,45 @@ TRLB_API int trlb_dynamic_tanh(float* x, float* delta, const float* alpha, const
 #undef GO
 }
 
+// post, w, delta may be null (see RmsResidual); H: row length
+TRLB_API int trlb_rms_residual(float* x, float* delta, const float* post, const float* w, void* out, int T, int H, float eps,
+                               int clear, int is_bf16, cudaStream_t st) {
+  if (T <= 0) return 0;
+  const RmsResidual p = {x, delta, post, w, H, clear, eps};
+  const int n4 = H / 4;
+  const bool regs = H % 4 == 0 && n4 <= 256 * 8;
+#define GO(TT, NN) (int)trlb_host::launch_kernel(rms_residual_kernel<TT, NN>, dim3(T), dim3(n4 >= 256 ? 256 : (n4 + 31) / 32 * 32), 0, st, PDL, p, (TT*)out)
+#define PICK(TT) (n4 <= 256 ? GO(TT, 1) : n4 <= 512 ? GO(TT, 2) : n4 <= 1024 ? GO(TT, 4) : GO(TT, 8))
+  if (regs) return is_bf16 ? PICK(bf16) : PICK(float);
+#undef PICK
+#undef GO
+  if (is_bf16) return (int)trlb_host::launch_kernel(rms_residual_any_kernel<bf16>, dim3(T), dim3(256), 0, st, PDL, p, (bf16*)out);
+  return (int)trlb_host::launch_kernel(rms_residual_any_kernel<float>, dim3(T), dim3(256), 0, st, PDL, p, (float*)out);
+}
+
+TRLB_API int trlb_clamped_glu(const void* z, void* out, int rows, int n, float limit, float alpha, float shift, int is_bf16,
+                              cudaStream_t st) {
+  if (rows <= 0 || n <= 0) return 0;
+  const bool v4 = n % 4 == 0;
+  const long long total = (long long)rows * n / (v4 ? 4 : 1);
+#define GO(TT, VV) clamped_glu_kernel<TT, VV><<<grid_for(total, 256), 256, 0, st>>>((const TT*)z, (TT*)out, total, n, limit, alpha, shift)
+  if (is_bf16) { if (v4) GO(bf16, 4); else GO(bf16, 1); }
+  else { if (v4) GO(float, 4); else GO(float, 1); }
+#undef GO
+  return (int)cudaGetLastError();
+}
+
+// z [rows, n] (fp32 if z_f32, else the dtype of the table), table [V, table_ld]
+TRLB_API int trlb_side_gate(void* z, int z_f32, const long long* ids, const void* table, long long table_ld, int off, int rows,
+                            int n, int V, int clear, void* out, int is_bf16, cudaStream_t st) {
+  if (rows <= 0 || n <= 0) return 0;
+  const dim3 grid(rows), blk(n >= 128 ? 128 : (n + 31) / 32 * 32);
+#define GO(TT, ZZ) (int)trlb_host::launch_kernel(side_gate_kernel<TT, ZZ>, grid, blk, 0, st, PDL, (ZZ*)z, ids, (const TT*)table, table_ld, off, n, V, clear, (TT*)out)
+  if (is_bf16) return z_f32 ? GO(bf16, float) : GO(bf16, bf16);
+  return GO(float, float);
+#undef GO
+}
+
 TRLB_API int trlb_gelu_erf(const void* z, void* out, long long n, int is_bf16, cudaStream_t st) {
   if (n <= 0) return 0;
   if (is_bf16) gelu_erf_kernel<bf16><<<grid_for(n, 256), 256, 0, st>>>((const bf16*)z, (bf16*)out, n);
@@ -699,25 +811,6 @@ TRLB_API int trlb_rotate_q(void* q, int rows, int heads, int dim, int rot, const
   if (is_bf16) { if (two) GO(bf16, 2); else GO(bf16, 1); }
   else { if (two) GO(float, 2); else GO(float, 1); }
 #undef GO
-  return (int)cudaGetLastError();
-}
-
-// window <= 0: unlimited
-TRLB_API int trlb_latent_prompt(const void* q, const void* kv, long long kv_ld, const void* lat, int T, int heads, int dim,
-                                int rot, int vdim, int kr_off, int lat_w, int window, float scale, const int* positions,
-                                const float* sink, const float* gate, void* out, int is_bf16, cudaStream_t st) {
-  if (T <= 0) return 0;
-  LatentPrompt p = {T, heads, dim, rot, vdim, kr_off, lat_w, window, kv_ld, scale, positions, sink, gate};
-  const long long items = (long long)T * heads;
-  const int grid = (int)((items + 3) / 4);
-  const size_t smem = (size_t)4 * (dim + rot + vdim) * 4;
-  if (is_bf16) {
-    if (!allow_smem(latent_prompt_kernel<bf16>, smem)) return -201;
-    latent_prompt_kernel<bf16><<<grid, 128, smem, st>>>(p, (const bf16*)q, (const bf16*)kv, (const bf16*)lat, (bf16*)out);
-  } else {
-    if (!allow_smem(latent_prompt_kernel<float>, smem)) return -201;
-    latent_prompt_kernel<float><<<grid, 128, smem, st>>>(p, (const float*)q, (const float*)kv, (const float*)lat, (float*)out);
-  }
   return (int)cudaGetLastError();
 }
 

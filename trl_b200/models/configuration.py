@@ -268,6 +268,16 @@ PRESETS: dict[str, dict] = {
                 dict(type="latent_attention", mlp=dict(kind="dense", ff=192),
                      mixer=dict(heads=4, dim=16, rot_dim=8, vdim=16, q_rank=24, kv_rank=32, scale=0.2, mask=dict(size=20),
                                 rot=dict(base=1e4, dims=8, scaling=dict(factor=4.0, original=256, fast=16.0, slow=1.0))))]),
+    "tiny-povusun": dict(
+        architecture="Povusun", vocab=1024, width=64, norm=dict(eps=1e-6), token_side=dict(dim=16),
+        layers=[dict(type="attention", mlp=dict(kind="dense", ff=96, limit=6.0),
+                     mixer=dict(heads=4, kv_heads=2, dim=16, vdim=16, scale=0.25, softcap=30.0, q_temp=dict(coef=0.1, every=128))),
+                dict(type="rglru", mlp=None, mixer=dict(width=48, blocks=3, conv=4)),
+                dict(type="latent_attention", mlp=dict(kind="dense", ff=96, limit=6.0),
+                     mixer=dict(heads=4, dim=16, vdim=24, kv_rank=32, scale=0.25)),
+                dict(type="attention", mlp=dict(kind="dense", ff=96, limit=6.0),
+                     mixer=dict(heads=4, kv_heads=2, dim=16, vdim=16, scale=0.25, softcap=30.0, q_temp=dict(coef=0.1, every=128),
+                                kv_from=0))]),
 }
 
 

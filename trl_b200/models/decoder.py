@@ -37,6 +37,8 @@ class SeqCtx:
     sp: Any = None
     # multimodal rotary positions [3, T] (temporal, height, width; models/vision_qwen.py); None = ordinary RoPE
     mrope_positions: Any = None
+    # keys and values of the layers that later layers borrow them from (models/layered.py), by layer
+    shared: dict = field(default_factory=dict)
 
     @staticmethod
     def from_lengths(lengths, device) -> "SeqCtx":

@@ -1,22 +1,28 @@
 """Decoders described layer by layer.
 
 The flat families of :mod:`trl_b200.models.configuration` repeat one block.  A *layered* design instead lists its
-layers in ``config.json``, each with a mixer (kind and sizes) and a feed-forward (or none), and a layer may run with
-another layer's weights.  :data:`DESIGNS` registers what a design fixes (norm, activation); everything else is read
-from the file.  A mixer is a module here (parameters, tensor names, prompt forward) with its kernels in
-``csrc/mixers.cu`` and its decode state in ``rollout/layered_engine.py``; registering another kind in :data:`MIXERS`
-makes it available to every layered design.
+layers in ``config.json``, each with a mixer (kind and sizes) and a feed-forward (or none); a layer may run with
+another layer's weights, or attend to another layer's keys and values.  :data:`DESIGNS` registers what a design fixes
+(norm and where it stands, feed-forward, head); everything else is read from the file.  A mixer is a module here
+(parameters, tensor names, prompt forward) with its kernels in ``csrc/`` and its decode state in
+``rollout/layered_engine.py``; registering another kind in :data:`MIXERS` makes it available to every layered design.
 
 Designs
     Zorelorn    embeddings times a constant, Dynamic-Tanh norms, ``latent_attention`` (multi-head latent attention with
                 YaRN rotary part, sliding window, softmax sink, per-head output gate) and ``mlstm`` (matrix memory with
                 exponential gates) mixers, erf-GELU feed-forward.
+    Povusun     RMS norms before and after every sublayer, ``attention`` (grouped queries, unit-rms queries and keys, query
+                temperature by position, capped scores, per-element output gate; a layer may read another one's cache),
+                ``latent_attention`` (without positions, queries straight from the input) and ``rglru`` (short convolution
+                and real-gated linear recurrence) mixers, clamped gated feed-forward, a per-token input of every layer,
+                tied head.
 
 The residual stream, norms, gates and recurrent states are fp32 whatever the model dtype.
 """
 from __future__ import annotations
 
 import copy
+import dataclasses
 import json
 import os
 from dataclasses import dataclass, field
@@ -34,11 +40,18 @@ from .decoder import CausalLM, SeqCtx
 class Design:
     """What a design fixes for all its models."""
 
-    norm: str = "dynamic_tanh"
-    mlp_act: str = "gelu"
+    norm: str
+    mlp: str
+    post_norm: bool = False      # a norm on the output of every sublayer, before it is added
+    latent_sink: bool = False    # latent_attention: exp(sink) in the softmax denominator
+    latent_gate: bool = False    # latent_attention: sigmoid gate per head
+    tied_head: bool = False
 
 
-DESIGNS: dict[str, Design] = {"Zorelorn": Design()}
+DESIGNS: dict[str, Design] = {
+    "Zorelorn": Design(norm="dynamic_tanh", mlp="gelu", latent_sink=True, latent_gate=True),
+    "Povusun": Design(norm="rms", mlp="clamped_glu", post_norm=True, tied_head=True),
+}
 
 
 @dataclass
@@ -47,18 +60,23 @@ class LayerSpec:
 
     kind: str
     mixer: dict
-    ff: int | None
+    mlp: dict | None
     owner: int
 
     @property
+    def ff(self) -> int:
+        return 0 if self.mlp is None else int(self.mlp["ff"])
+
+    @property
     def key(self):
-        return (self.kind, json.dumps(self.mixer, sort_keys=True), self.ff)
+        return (self.kind, json.dumps(self.mixer, sort_keys=True), json.dumps(self.mlp, sort_keys=True))
 
 
 @dataclass
 class LayeredArch(ModelArch):
     design: str = ""
     layers: list = field(default_factory=list)  # [LayerSpec]
+    side_dim: int = 0  # per-token input of every layer: elements per layer (0: none)
     source: dict = field(default_factory=dict)  # the config.json this came from
 
     @classmethod
@@ -79,15 +97,18 @@ class LayeredArch(ModelArch):
                 if not 0 <= j < i:
                     raise ValueError(f"layer {i}: weights_of={j} must name an earlier layer")
                 owner = specs[j].owner
-            s = LayerSpec(e["type"], dict(e["mixer"]), None if mlp is None else int(mlp["ff"]), owner)
+            s = LayerSpec(e["type"], dict(e["mixer"]), None if mlp is None else dict(mlp), owner)
+            _check_lender(specs, s, i)
             if owner != i and s.key != specs[owner].key:
                 raise ValueError(f"layer {i} runs with the weights of layer {owner} but is described differently")
             specs.append(s)
+        design = DESIGNS[name]
         heads = max((s.mixer.get("heads", 1) for s in specs), default=1)
         return cls(model_type=name.lower(), design=name, vocab_size=d["vocab"], hidden_size=d["width"],
-                   intermediate_size=max((s.ff or 0 for s in specs), default=0), num_hidden_layers=len(specs),
+                   intermediate_size=max((s.ff for s in specs), default=0), num_hidden_layers=len(specs),
                    num_attention_heads=heads, num_key_value_heads=heads, rms_norm_eps=float(d["norm"]["eps"]),
                    embed_scale=float((d.get("embedding") or {}).get("scale", 1.0)), layers=specs, source=copy.deepcopy(d),
+                   side_dim=int((d.get("token_side") or {}).get("dim", 0)), tie_word_embeddings=design.tied_head,
                    attention_bias=False, qk_norm=False, pad_token_id=d.get("pad_token_id"),
                    bos_token_id=d.get("bos_token_id"), eos_token_id=d.get("eos_token_id"))
 
@@ -106,7 +127,23 @@ class LayeredArch(ModelArch):
     def num_parameters(self, exclude_embeddings: bool = False) -> int:
         m = LayeredLM(self, device="meta", init=False)
         n = sum(p.numel() for p in m.parameters())
-        return n - (2 * self.vocab_size * self.hidden_size if exclude_embeddings else 0)
+        return n - ((1 if self.tie_word_embeddings else 2) * self.vocab_size * self.hidden_size if exclude_embeddings else 0)
+
+    @property
+    def lenders(self) -> set:
+        """Layers whose keys and values others borrow."""
+        return {s.mixer["kv_from"] for s in self.layers if s.mixer.get("kv_from") is not None}
+
+
+def _check_lender(specs: list, s: LayerSpec, i: int):
+    j = s.mixer.get("kv_from")
+    if j is None:
+        return
+    if not 0 <= j < i or specs[j].kind != s.kind or specs[j].mixer.get("kv_from") is not None:
+        raise ValueError(f"layer {i}: kv_from={j} must name an earlier layer of the same kind with keys and values of its own")
+    for k in ("heads", "kv_heads", "dim", "vdim"):
+        if specs[j].mixer[k] != s.mixer[k]:
+            raise ValueError(f"layer {i}: {k} differs from that of layer {j}, whose keys and values it reads")
 
 
 def _vec(n=None, fill=0.0, device=None):
@@ -118,48 +155,73 @@ def _vec(n=None, fill=0.0, device=None):
 class DynamicTanh(nn.Module):
     """``tanh(alpha x) w + b``: a norm without statistics."""
 
-    def __init__(self, n, device=None):
+    def __init__(self, cfg: LayeredArch, device=None):
         super().__init__()
+        n = cfg.hidden_size
         self.weight, self.bias, self.alpha = _vec(n, 1.0, device), _vec(n, 0.0, device), _vec(None, 0.5, device)
 
     def tensors(self, name):
         return {name: self.weight, name + ".b": self.bias, name + ".alpha": self.alpha}
 
-    def forward(self, x, out_dtype, delta=None):
-        """x [T, H] fp32 (``delta``, when given, is added to it in place first) -> [T, H] ``out_dtype``."""
-        return mx.dynamic_tanh(x, delta, self.alpha, self.weight, self.bias, out_dtype)
+    def forward(self, x, out_dtype, delta=None, post=None, **kw):
+        """x [T, H] fp32 -> (norm of the stream in ``out_dtype``, the stream).  ``delta``, when given, is added to the stream
+        first (in place on CUDA), normalised by ``post`` when that is given.  ``clear`` (delta is zeroed) and ``out`` are for
+        the decode step."""
+        if post is not None:
+            raise NotImplementedError("Dynamic Tanh around a sublayer's output")
+        return mx.dynamic_tanh(x, delta, self.alpha, self.weight, self.bias, out_dtype, **kw)
 
 
-NORMS = {"dynamic_tanh": DynamicTanh}
+class RmsNorm(nn.Module):
+    """``x / sqrt(mean(x^2) + eps) w``."""
+
+    def __init__(self, cfg: LayeredArch, device=None):
+        super().__init__()
+        self.weight, self.eps = _vec(cfg.hidden_size, 1.0, device), cfg.rms_norm_eps
+
+    def tensors(self, name):
+        return {name: self.weight}
+
+    def forward(self, x, out_dtype, delta=None, post=None, **kw):
+        return mx.rms_residual(x, delta, None if post is None else post.weight, self.weight, self.eps, out_dtype, **kw)
+
+
+NORMS = {"dynamic_tanh": DynamicTanh, "rms": RmsNorm}
 
 
 class LatentAttention(nn.Module):
     """Multi-head latent attention: keys and values of all heads are linear in one latent per token (plus one rotated
-    key part shared by the heads), and only those are cached.  In memory the projections that read the layer input are
-    one matrix (query latent | key/value latent | rotated key | gate), as are the key and value up-projections."""
+    key part shared by the heads), and only those are cached.  Queries come through a latent of their own (``q_rank``) or
+    straight from the layer input.  In memory the projections that read the layer input are one matrix (query latent or
+    queries | key/value latent | rotated key | gate), as are the key and value up-projections."""
 
     kind = "latent_attention"
 
     def __init__(self, cfg: LayeredArch, m: dict, dtype, device):
         super().__init__()
         kw = dict(dtype=dtype, device=device)
-        self.eps = cfg.rms_norm_eps
-        self.heads, self.dim, self.rot_dim, self.vdim = m["heads"], m["dim"], m["rot_dim"], m["vdim"]
-        self.q_rank, self.kv_rank = m["q_rank"], m["kv_rank"]
+        design = DESIGNS[cfg.design]
+        self.eps, self.gated = cfg.rms_norm_eps, design.latent_gate
+        self.heads, self.dim, self.rot_dim, self.vdim = m["heads"], m["dim"], m.get("rot_dim", 0), m["vdim"]
+        self.q_rank, self.kv_rank = m.get("q_rank", 0), m["kv_rank"]
         self.scale = float(m["scale"])
         mask = m.get("mask") or {}
         self.window = int(mask["size"]) if mask.get("size") else None
-        rot = m["rot"]
-        if rot["dims"] != self.rot_dim or self.rot_dim % 2:
-            raise ValueError("latent_attention rotates its whole rot_dim part, in pairs")
-        self.rope = mx.RotarySpec(self.rot_dim, float(rot["base"]), rot.get("scaling"))
-        h = cfg.hidden_size
-        self.w_in = nn.Parameter(torch.empty(self.q_rank + self.kv_rank + self.rot_dim + self.heads, h, **kw))
-        self.uq = nn.Parameter(torch.empty(self.heads * (self.dim + self.rot_dim), self.q_rank, **kw))
+        self.rope = None
+        if self.rot_dim:
+            rot = m["rot"]
+            if rot["dims"] != self.rot_dim or self.rot_dim % 2:
+                raise ValueError("latent_attention rotates its whole rot_dim part, in pairs")
+            self.rope = mx.RotarySpec(self.rot_dim, float(rot["base"]), rot.get("scaling"))
+        h, q = cfg.hidden_size, self.heads * (self.dim + self.rot_dim)
+        self.q_rows = self.q_rank or q  # first rows of w_in
+        self.w_in = nn.Parameter(torch.empty(self.q_rows + self.kv_rank + self.rot_dim + (self.heads if self.gated else 0), h, **kw))
+        self.uq = nn.Parameter(torch.empty(q, self.q_rank, **kw)) if self.q_rank else None
         self.ukv = nn.Parameter(torch.empty(self.heads * (self.dim + self.vdim), self.kv_rank, **kw))
         self.o = nn.Parameter(torch.empty(h, self.heads * self.vdim, **kw))
-        self.q_norm, self.kv_norm = _vec(self.q_rank, 1.0, device), _vec(self.kv_rank, 1.0, device)
-        self.sink = _vec(self.heads, 0.0, device)
+        self.q_norm = _vec(self.q_rank, 1.0, device) if self.q_rank else None
+        self.kv_norm = _vec(self.kv_rank, 1.0, device)
+        self.sink = _vec(self.heads, 0.0, device) if design.latent_sink else None
 
     @property
     def uk(self):
@@ -170,10 +232,15 @@ class LatentAttention(nn.Module):
         return self.ukv[self.heads * self.dim:]
 
     def tensors(self, p):
-        a, b = self.q_rank, self.q_rank + self.kv_rank + self.rot_dim
-        return {p + "dq": self.w_in[:a], p + "dq.norm": self.q_norm, p + "uq": self.uq, p + "dkv": self.w_in[a:b],
-                p + "dkv.norm": self.kv_norm, p + "uk": self.uk, p + "uv": self.uv, p + "sink": self.sink,
-                p + "g": self.w_in[b:], p + "o": self.o}
+        a, b = self.q_rows, self.q_rows + self.kv_rank + self.rot_dim
+        out = ({p + "dq": self.w_in[:a], p + "dq.norm": self.q_norm, p + "uq": self.uq} if self.q_rank else {p + "q": self.w_in[:a]})
+        out.update({p + "dkv": self.w_in[a:b], p + "dkv.norm": self.kv_norm, p + "uk": self.uk, p + "uv": self.uv})
+        if self.sink is not None:
+            out[p + "sink"] = self.sink
+        if self.gated:
+            out[p + "g"] = self.w_in[b:]
+        out[p + "o"] = self.o
+        return out
 
     def forward(self, h, ctx: SeqCtx, li: int):
         """[T, H] normed input -> [T, H] fp32 block output (packed prompts)."""
@@ -215,14 +282,87 @@ class MLstm(nn.Module):
         return mx.mlstm(self, h, ctx, li)
 
 
-MIXERS = {c.kind: c for c in (LatentAttention, MLstm)}
+class GroupedAttention(nn.Module):
+    """Grouped-query attention without rotation: queries and keys over their rms per head, queries times a temperature that
+    grows with the position, scores capped by tanh, heads times the sigmoid of gates that read the layer input.  With
+    ``kv_from`` the layer has no keys and values of its own and reads those of another layer.  The projections are one
+    matrix (query | key | value | gate)."""
+
+    kind = "attention"
+
+    def __init__(self, cfg: LayeredArch, m: dict, dtype, device):
+        super().__init__()
+        kw = dict(dtype=dtype, device=device)
+        self.eps = cfg.rms_norm_eps
+        self.heads, self.kv_heads, self.dim, self.vdim = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+        if self.heads % self.kv_heads:
+            raise ValueError(f"{self.heads} query heads over {self.kv_heads} key/value heads")
+        self.scale = float(m["scale"])
+        self.cap = float(m["softcap"]) if m.get("softcap") else None
+        t = m.get("q_temp")
+        self.temperature = mx.TemperatureSpec(t["coef"], t["every"]) if t else None
+        self.kv_from = m.get("kv_from")
+        own = self.kv_heads if self.kv_from is None else 0
+        self.parts = [self.heads * self.dim, own * self.dim, own * self.vdim, self.heads * self.vdim]  # rows of w_in
+        h = cfg.hidden_size
+        self.w_in = nn.Parameter(torch.empty(sum(self.parts), h, **kw))
+        self.o = nn.Parameter(torch.empty(h, self.heads * self.vdim, **kw))
+
+    def tensors(self, p):
+        q, k, v, g = self.w_in.split(self.parts)
+        out = {p + "q": q, p + "g": g, p + "o": self.o}
+        if self.kv_from is None:
+            out.update({p + "k": k, p + "v": v})
+        return out
+
+    def forward(self, h, ctx: SeqCtx, li: int):
+        return mx.attention(self, h, ctx, li)
+
+
+class RgLru(nn.Module):
+    """Griffin's recurrent block: a GELU branch times a branch of a short causal convolution and a linear recurrence per
+    channel whose decay and input gates are block-diagonal in the convolved input.  The projections are one matrix (GELU
+    branch | recurrent branch), the gates' weights one tensor (recurrence gate, input gate)."""
+
+    kind = "rglru"
+    decay = 8.0  # log a = -decay * gate * softplus(lam)
+
+    def __init__(self, cfg: LayeredArch, m: dict, dtype, device):
+        super().__init__()
+        kw = dict(dtype=dtype, device=device)
+        self.eps = cfg.rms_norm_eps
+        self.width, self.blocks, self.taps = m["width"], m["blocks"], m["conv"]
+        if self.width % self.blocks:
+            raise ValueError(f"{self.width} channels in {self.blocks} blocks")
+        h, w, wb = cfg.hidden_size, self.width, self.width // self.blocks
+        self.w_in = nn.Parameter(torch.empty(2 * w, h, **kw))
+        self.gates = nn.Parameter(torch.empty(2, self.blocks, wb, wb, **kw))
+        self.o = nn.Parameter(torch.empty(h, w, **kw))
+        self.y_bias, self.x_bias, self.conv_bias, self.lam = (_vec(w, 0.0, device) for _ in range(4))
+        f32 = dict(dtype=torch.float32, device=device)
+        self.gate_bias = nn.Parameter(torch.zeros(2, w, **f32))
+        self.conv = nn.Parameter(torch.zeros(w, self.taps, **f32))
+
+    def tensors(self, p):
+        w = self.width
+        b = self.gate_bias.view(2, self.blocks, -1)
+        return {p + "y": self.w_in[:w], p + "y.b": self.y_bias, p + "x": self.w_in[w:], p + "x.b": self.x_bias, p + "conv": self.conv,
+                p + "conv.b": self.conv_bias, p + "ra": self.gates[0], p + "ra.b": b[0], p + "ri": self.gates[1], p + "ri.b": b[1],
+                p + "lam": self.lam, p + "o": self.o}
+
+    def forward(self, h, ctx: SeqCtx, li: int):
+        return mx.rglru(self, h, ctx, li)
+
+
+MIXERS = {c.kind: c for c in (LatentAttention, MLstm, GroupedAttention, RgLru)}
 
 
 class DenseMlp(nn.Module):
     """``down(act(up x))`` with the exact GELU."""
 
-    def __init__(self, cfg: LayeredArch, ff: int, dtype, device):
+    def __init__(self, cfg: LayeredArch, spec: dict, dtype, device):
         super().__init__()
+        ff = int(spec["ff"])
         self.up = nn.Parameter(torch.empty(ff, cfg.hidden_size, dtype=dtype, device=device))
         self.down = nn.Parameter(torch.empty(cfg.hidden_size, ff, dtype=dtype, device=device))
 
@@ -233,16 +373,70 @@ class DenseMlp(nn.Module):
         return mx.linear_f32(mx.gelu_linear(h, self.up), self.down)
 
 
+class ClampedGluMlp(nn.Module):
+    """``down(g sigmoid(alpha g) (u + shift))`` with ``g = min(gate x, limit)`` and ``u = up x`` within +- limit.  Gate and up
+    projections are one matrix."""
+
+    alpha, shift = 1.702, 1.0
+
+    def __init__(self, cfg: LayeredArch, spec: dict, dtype, device):
+        super().__init__()
+        self.ff, self.limit = int(spec["ff"]), float(spec["limit"])
+        self.gate_up = nn.Parameter(torch.empty(2 * self.ff, cfg.hidden_size, dtype=dtype, device=device))
+        self.down = nn.Parameter(torch.empty(cfg.hidden_size, self.ff, dtype=dtype, device=device))
+
+    @property
+    def glu(self):
+        return self.limit, self.alpha, self.shift
+
+    def tensors(self, p):
+        return {p + "gate": self.gate_up[: self.ff], p + "up": self.gate_up[self.ff:], p + "down": self.down}
+
+    def forward(self, h):
+        return mx.linear_f32(mx.clamped_glu_linear(h, self.gate_up, *self.glu), self.down)
+
+
+MLPS = {"gelu": DenseMlp, "clamped_glu": ClampedGluMlp}
+
+
+class TokenSide(nn.Module):
+    """A layer's own input from the token: ``proj(gelu_tanh(gate x) * e)``, e the layer's part of the token's row in a table
+    shared by the layers; its output is normed before it is added."""
+
+    def __init__(self, cfg: LayeredArch, dtype, device):
+        super().__init__()
+        self.dim = cfg.side_dim
+        self.gate = nn.Parameter(torch.empty(self.dim, cfg.hidden_size, dtype=dtype, device=device))
+        self.proj = nn.Parameter(torch.empty(cfg.hidden_size, self.dim, dtype=dtype, device=device))
+        self.norm = RmsNorm(cfg, device)
+
+    def tensors(self, p):
+        return {p + "gate": self.gate, p + "proj": self.proj, **self.norm.tensors(p + "norm")}
+
+    def stream(self, x, out_dtype, delta, post, **kw):
+        """The stream itself after the addition of ``delta`` (normed by ``post``), in ``out_dtype``, and in fp32."""
+        return mx.rms_residual(x, delta, None if post is None else post.weight, None, self.norm.eps, out_dtype, **kw)
+
+    def forward(self, h, ids, table, li: int):
+        return mx.side_input(h, ids, table, li * self.dim, self.gate, self.proj)
+
+
 class LayeredBlock(nn.Module):
-    """Pre-norm mixer and (optional) feed-forward around an fp32 residual stream."""
+    """Pre-norm mixer and (optional) feed-forward around an fp32 residual stream; depending on the design with a norm on each
+    sublayer's output and a per-token input after them."""
 
     def __init__(self, cfg: LayeredArch, spec: LayerSpec, dtype, device):
         super().__init__()
-        norm = NORMS[DESIGNS[cfg.design].norm]
-        self.norm1 = norm(cfg.hidden_size, device)
+        design = DESIGNS[cfg.design]
+        norm = NORMS[design.norm]
+        post = norm if design.post_norm else lambda *_: None
+        self.norm1, self.norm1b = norm(cfg, device), post(cfg, device)
         self.mixer = MIXERS[spec.kind](cfg, spec.mixer, dtype, device)
-        self.norm2 = norm(cfg.hidden_size, device) if spec.ff is not None else None
-        self.mlp = DenseMlp(cfg, spec.ff, dtype, device) if spec.ff is not None else None
+        self.norm2 = self.norm2b = self.mlp = None
+        if spec.mlp is not None:
+            self.norm2, self.norm2b = norm(cfg, device), post(cfg, device)
+            self.mlp = MLPS[design.mlp](cfg, spec.mlp, dtype, device)
+        self.side = TokenSide(cfg, dtype, device) if cfg.side_dim else None
         self.dtype = dtype
         self.lora = nn.ModuleDict()
         self.lora_enabled = True
@@ -252,19 +446,28 @@ class LayeredBlock(nn.Module):
 
     def tensors(self, p):
         out = {**self.norm1.tensors(p + "norm1"), **self.mixer.tensors(p + "mix.")}
+        if self.norm1b is not None:
+            out.update(self.norm1b.tensors(p + "norm1b"))
         if self.mlp is not None:
             out.update({**self.norm2.tensors(p + "norm2"), **self.mlp.tensors(p + "mlp.")})
+            if self.norm2b is not None:
+                out.update(self.norm2b.tensors(p + "norm2b"))
+        if self.side is not None:
+            out.update(self.side.tensors(p + "side."))
         return out
 
-    def forward(self, x, delta, ctx: SeqCtx, li: int):
-        """(residual, block output not yet added to it) -> the same pair after this layer: every addition rides on the
-        norm that follows it."""
-        h, x = self.norm1(x, self.dtype, delta)
-        delta = self.mixer(h, ctx, li)
+    def forward(self, x, delta, post, ctx: SeqCtx, li: int, ids=None, side_table=None):
+        """(residual, sublayer output not yet added to it, norm of that output) -> the same triple after this layer: every
+        addition rides on the norm that follows it."""
+        h, x = self.norm1(x, self.dtype, delta, post)
+        delta, post = self.mixer(h, ctx, li), self.norm1b
         if self.mlp is not None:
-            h, x = self.norm2(x, self.dtype, delta)
-            delta = self.mlp(h)
-        return x, delta
+            h, x = self.norm2(x, self.dtype, delta, post)
+            delta, post = self.mlp(h), self.norm2b
+        if self.side is not None:
+            h, x = self.side.stream(x, self.dtype, delta, post)
+            delta, post = self.side(h, ids, side_table, li), self.side.norm
+        return x, delta, post
 
 
 class LayeredLM(CausalLM):
@@ -283,8 +486,10 @@ class LayeredLM(CausalLM):
         for i, s in enumerate(cfg.layers):  # a layer that borrows weights IS its owner's block at another place
             blocks.append(blocks[s.owner] if s.owner != i else LayeredBlock(cfg, s, dtype, device))
         self.layers = nn.ModuleList(blocks)
-        self.norm = NORMS[DESIGNS[cfg.design].norm](cfg.hidden_size, device)
-        self.lm_head = nn.Parameter(torch.empty(cfg.vocab_size, cfg.hidden_size, dtype=dtype, device=device))
+        self.norm = NORMS[DESIGNS[cfg.design].norm](cfg, device)
+        self.lm_head = None if cfg.tie_word_embeddings else nn.Parameter(torch.empty(cfg.vocab_size, cfg.hidden_size, dtype=dtype, device=device))
+        self.side_embed = (nn.Parameter(torch.empty(cfg.vocab_size, cfg.side_dim * cfg.num_hidden_layers, dtype=dtype, device=device))
+                           if cfg.side_dim else None)
         self.gradient_checkpointing = False
         self.name_or_path = ""
         self.generation_config = None
@@ -301,12 +506,23 @@ class LayeredLM(CausalLM):
     def named_tensors(self) -> dict[str, torch.Tensor]:
         """Checkpoint name -> parameter or view into a fused parameter."""
         out = {"embed": self.embed_tokens}
+        if self.side_embed is not None:
+            out["side.embed"] = self.side_embed
         for i, (s, b) in enumerate(zip(self.config.layers, self.layers)):
             if s.owner == i:
                 out.update(b.tensors(f"l{i}."))
         out.update(self.norm.tensors("final.norm"))
-        out["head"] = self.lm_head
+        if self.lm_head is not None:
+            out["head"] = self.lm_head
         return out
+
+    def resize_token_embeddings(self, new_size: int, pad_to_multiple_of: int | None = None):
+        super().resize_token_embeddings(new_size, pad_to_multiple_of)
+        if self.side_embed is not None and self.side_embed.shape[0] != self.config.vocab_size:
+            old, n = self.side_embed, min(self.side_embed.shape[0], self.config.vocab_size)
+            w = torch.empty(self.config.vocab_size, old.shape[1], dtype=old.dtype, device=old.device).normal_(0, 0.02)
+            w[:n] = old.data[:n]
+            self.side_embed = nn.Parameter(w)
 
     @torch.no_grad()
     def load_named_tensors(self, sd: dict[str, torch.Tensor], strict: bool = True) -> list[str]:
@@ -324,15 +540,17 @@ class LayeredLM(CausalLM):
     def embed(self, input_ids):
         return mx.embed_scaled(input_ids, self.embed_tokens, self.config.embed_scale)
 
-    def final_norm(self, x, delta=None):
-        return self.norm(x, self.dtype, delta)[0]
+    def final_norm(self, x, delta=None, post=None):
+        return self.norm(x, self.dtype, delta, post)[0]
 
     def forward_hidden(self, input_ids, ctx: SeqCtx, inputs_embeds=None):
         mx.check_can_run(self.embed_tokens)
-        x, delta = (self.embed(input_ids) if inputs_embeds is None else inputs_embeds.float()), None
+        ctx = dataclasses.replace(ctx, shared=dict.fromkeys(self.config.lenders))
+        ids = input_ids.reshape(-1)
+        x, delta, post = (self.embed(input_ids) if inputs_embeds is None else inputs_embeds.float()), None, None
         for li, layer in enumerate(self.layers):
-            x, delta = layer(x, delta, ctx, li)
-        return self.final_norm(x, delta)
+            x, delta, post = layer(x, delta, post, ctx, li, ids, self.side_embed)
+        return self.final_norm(x, delta, post)
 
 
 def is_layered_dir(path: str) -> bool:

@@ -840,14 +840,15 @@ def set_pdl(on: bool) -> bool:
     return bool(lib().trlb_set_pdl(c_int(int(bool(on)))))
 
 
-def decode_gemm(x, w, bias=None, *, y32=None, out=None, swiglu=False, gelu=False, max_ctas: int = 0, tiled_shape=None,
-                peers=None):
+def decode_gemm(x, w, bias=None, *, y32=None, out=None, swiglu=False, gelu=False, clamped_glu=None, max_ctas: int = 0,
+                tiled_shape=None, peers=None):
     """Weight-streaming tcgen05 GEMM for decode batches (at most 128 rows of ``x``).
 
     ``y32`` given: ``y32[B, N] (fp32) += x @ w^T (+ bias)``, work split stream-K style over every SM; the caller passes
     zeros (the consumer kernels clear the buffer after reading it).  Otherwise bf16 ``out[B, N] = x @ w^T (+ bias)``;
     with ``swiglu`` ``w`` is ``[2N, K]`` (gate rows, then up rows) and ``out = silu(x Wg^T) * (x Wu^T)``; with ``gelu`` the
-    exact GELU of the sum is stored.
+    exact GELU of the sum is stored; ``clamped_glu=(limit, alpha, shift)`` is the clamped gated unit of a ``[2N, K]``
+    weight (:func:`~trl_b200.ops.cuda_mixers.clamped_glu`).
 
     ``tiled_shape=(rows, K)``: ``w`` is the flat tile-major copy made by :func:`tile_weights` of a ``[rows, K]`` weight.
     ``peers=(peer_y32_ptrs, arrive_ptrs, stage, slab_ctr)``: row-parallel GEMM fused with its all-reduce: partial sums
@@ -864,15 +865,15 @@ def decode_gemm(x, w, bias=None, *, y32=None, out=None, swiglu=False, gelu=False
     else:
         assert w.stride(1) == 1 and w.shape[1] == Kd
         rows, ldw = w.shape[0], w.stride(0)
-    N = rows // 2 if swiglu else rows
+    N = rows // 2 if swiglu or clamped_glu else rows
     if y32 is not None:
-        assert y32.dtype == torch.float32 and y32.stride(1) == 1 and tuple(y32.shape) == (B, N) and not swiglu
+        assert y32.dtype == torch.float32 and y32.stride(1) == 1 and tuple(y32.shape) == (B, N) and not swiglu and not clamped_glu
         mode, ldy, dst32, dstb, ret = 0, y32.stride(0), y32, None, y32
     else:
         if out is None:
             out = torch.empty(B, N, dtype=torch.bfloat16, device=x.device)
         assert out.dtype == torch.bfloat16 and out.stride(1) == 1 and tuple(out.shape) == (B, N)
-        mode, ldy, dst32, dstb, ret = (2 if swiglu else 3 if gelu else 1), out.stride(0), None, out, out
+        mode, ldy, dst32, dstb, ret = (2 if swiglu else 3 if gelu else 4 if clamped_glu else 1), out.stride(0), None, out, out
     n_peers, peer_arr, arrive_arr, stage, slab_ctr = 0, None, None, None, None
     if peers is not None:
         peer_ptrs, arrive_ptrs, stage, slab_ctr = peers
@@ -885,7 +886,8 @@ def decode_gemm(x, w, bias=None, *, y32=None, out=None, swiglu=False, gelu=False
     _chk(lib().trlb_decode_gemm(_p(x), _p(w), _p(bias), _p(dst32), _p(dstb), c_int(B), c_int(N), c_int(Kd),
                                 c_longlong(x.stride(0)), c_longlong(ldw), c_longlong(ldy), c_int(mode),
                                 c_int(int(tiled_shape is not None)), c_int(max_ctas), c_int(n_peers), peer_arr, arrive_arr,
-                                _p(stage), _p(slab_ctr), _p(status_buffer(x.device)), _s()), "decode_gemm")
+                                _p(stage), _p(slab_ctr), (ctypes.c_float * 3)(*clamped_glu) if clamped_glu else None,
+                                _p(status_buffer(x.device)), _s()), "decode_gemm")
     return ret
 
 

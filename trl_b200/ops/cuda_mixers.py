@@ -1,4 +1,5 @@
-"""ctypes bindings of ``csrc/mixers.cu`` and of the tensor-core mixer kernels (inference only).
+"""ctypes bindings of ``csrc/mixers.cu``, ``csrc/grouped_attn.cu``, ``csrc/rglru.cu`` and of the tensor-core mixer kernels
+(inference only).
 
 ``model dtype`` below is bf16 or fp32; accumulators, gates, states and norms are fp32 in both."""
 from __future__ import annotations
@@ -14,6 +15,11 @@ def _b(t) -> c_int:
     if t.dtype not in (torch.bfloat16, torch.float32):
         raise TypeError(f"layered decoders run in bfloat16 or float32, not {t.dtype}")
     return c_int(int(t.dtype == torch.bfloat16))
+
+
+def _len(table) -> c_int:
+    """Entries of a table by position (none: a mixer without one)."""
+    return c_int(0 if table is None else table.shape[0])
 
 
 def round8(n: int) -> int:
@@ -45,6 +51,39 @@ def dynamic_tanh(x, delta, alpha, w, b, dtype, clear=False, out=None):
     return out
 
 
+def rms_residual(x, delta, post, w, eps, dtype, clear=False, out=None):
+    """``x += delta`` or, with ``post``, ``x += delta / rms(delta) * post`` (in place; with ``clear`` delta is zeroed); returns
+    ``x / rms(x) * w`` in ``dtype``, or ``x`` itself without ``w``."""
+    T, H = x.shape
+    assert x.dtype == torch.float32 and x.is_contiguous() and (delta is None or (delta.dtype == torch.float32
+                                                                               and delta.is_contiguous()))
+    out = torch.empty(T, H, dtype=dtype, device=x.device) if out is None else out
+    _chk(lib().trlb_rms_residual(_p(x), _p(delta), _p(post), _p(w), _p(out), c_int(T), c_int(H), c_float(eps),
+                                 c_int(int(clear)), _b(out), _s()), "rms_residual")
+    return out
+
+
+def clamped_glu(z, limit, alpha, shift, out=None):
+    """z [rows, 2n] = gate | up -> ``g sigmoid(alpha g) (u + shift)``, ``g = min(gate, limit)``, u = up within +- limit."""
+    rows, n = z.shape[0], z.shape[1] // 2
+    assert z.is_contiguous()
+    out = torch.empty(rows, n, dtype=z.dtype, device=z.device) if out is None else out
+    _chk(lib().trlb_clamped_glu(_p(z), _p(out), c_int(rows), c_int(n), c_float(limit), c_float(alpha), c_float(shift), _b(z), _s()),
+         "clamped_glu")
+    return out
+
+
+def side_gate(z, ids, table, off, clear=False, out=None):
+    """``gelu_tanh(z) * table[ids, off : off + n]`` in the dtype of the table; z [rows, n] fp32 or of that dtype."""
+    rows, n = z.shape
+    assert z.is_contiguous() and ids.dtype == torch.int64 and ids.is_contiguous() and table.is_contiguous() and off + n <= table.shape[1]
+    assert z.dtype in (torch.float32, table.dtype)
+    out = torch.empty(rows, n, dtype=table.dtype, device=z.device) if out is None else out
+    _chk(lib().trlb_side_gate(_p(z), c_int(int(z.dtype == torch.float32)), _p(ids), _p(table), c_longlong(table.shape[1]), c_int(off),
+                              c_int(rows), c_int(n), c_int(table.shape[0]), c_int(int(clear)), _p(out), _b(table), _s()), "side_gate")
+    return out
+
+
 def gelu_erf(z, out=None):
     assert z.is_contiguous()
     out = torch.empty_like(z) if out is None else out
@@ -54,20 +93,21 @@ def gelu_erf(z, out=None):
 
 def latent_prep(acc, m, positions, table, *, clear=False, tok_slot=None, cq=None, lat=None, gate=None, cache=None,
                 block_table=None, block_size=0):
-    """From the sums of a layer's input projection: normed query latent, latent row (dense and / or appended to the
-    paged cache), sigmoid gates."""
+    """From the sums of a layer's input projection (without the query rows of a mixer that has no query latent): normed query
+    latent, latent row (dense and / or appended to the paged cache), sigmoid gates; the first and the last may be absent."""
     rows = acc.shape[0]
+    gates = m.heads if m.gated else 0
     kr, w = latent_row(m.kv_rank, m.rot_dim)
     dt = m.o.dtype
     assert acc.dtype == torch.float32 and acc.stride(1) == 1 and positions.dtype == torch.int32
-    cq = torch.empty(rows, m.q_rank, dtype=dt, device=acc.device) if cq is None else cq
-    gate = torch.empty(rows, m.heads, dtype=torch.float32, device=acc.device) if gate is None else gate
+    cq = torch.empty(rows, m.q_rank, dtype=dt, device=acc.device) if cq is None and m.q_rank else cq
+    gate = torch.empty(rows, gates, dtype=torch.float32, device=acc.device) if gate is None and gates else gate
     mb = 0 if block_table is None else block_table.shape[1]
     _chk(lib().trlb_latent_prep(_p(acc), c_longlong(acc.stride(0)), c_int(rows), c_int(m.q_rank), c_int(m.kv_rank),
-                                c_int(m.rot_dim), c_int(m.heads), c_int(int(clear)), _p(m.q_norm), _p(m.kv_norm),
-                                c_float(m.eps), _p(positions), _p(tok_slot), _p(table), c_int(table.shape[0]), _p(cq),
+                                c_int(m.rot_dim), c_int(gates), c_int(int(clear)), _p(m.q_norm), _p(m.kv_norm),
+                                c_float(m.eps), _p(positions), _p(tok_slot), _p(table), _len(table), _p(cq),
                                 _p(lat), _p(gate), c_int(kr), c_int(w), _p(cache), _p(block_table), c_int(mb),
-                                c_int(block_size), _b(cq), _s()), "latent_prep")
+                                c_int(block_size), _b(m.o), _s()), "latent_prep")
     return cq, gate
 
 
@@ -78,34 +118,147 @@ def rotate_q(q, m, positions, table):
                              c_int(table.shape[0]), _b(q), _s()), "rotate_q")
 
 
-def latent_prompt(q, kv, lat, m, positions, gate):
-    """Windowed sink attention of packed prompts on the CUDA cores: any size, bf16 or fp32."""
-    T = q.shape[0]
-    kr, w = latent_row(m.kv_rank, m.rot_dim)
-    out = torch.empty(T, m.heads * m.vdim, dtype=q.dtype, device=q.device)
-    assert q.is_contiguous() and kv.stride(1) == 1 and lat.is_contiguous()
-    _chk(lib().trlb_latent_prompt(_p(q), _p(kv), c_longlong(kv.stride(0)), _p(lat), c_int(T), c_int(m.heads), c_int(m.dim),
-                                  c_int(m.rot_dim), c_int(m.vdim), c_int(kr), c_int(w), c_int(m.window or 0),
-                                  c_float(m.scale), _p(positions), _p(m.sink), _p(gate), _p(out), _b(q), _s()),
-         "latent_prompt")
+def mixer_attn_tc_ok(heads, kv_heads, dim, rot, vdim) -> bool:
+    """Whether :func:`mixer_attn` runs bf16 prompts of these sizes on the tensor cores."""
+    return bool(lib().trlb_mixer_attn_tc_ok(c_int(heads), c_int(kv_heads), c_int(dim), c_int(rot), c_int(vdim)))
+
+
+def mixer_attn(q, k, v, *, heads, kv_heads, scale, ctx, rot=0, krot=None, window=None, cap=None, sink=None, gate=None,
+               gate_logits=None, tensor_cores=True):
+    """Causal attention of packed prompts.  Rows of q: heads x (dim | rot), of k and v: kv_heads x dim / vdim, of krot: the rot
+    elements that all heads' keys share (rows may be strided, their elements are dense) -> [T, heads vdim].  Keys at distance <
+    ``window``; scores ``cap tanh(s / cap)``; ``exp(sink)`` in the denominator; ``gate`` (fp32 [T, heads]) or the sigmoid of
+    ``gate_logits`` ([T, heads vdim] in the model dtype) multiplies the result."""
+    T, dim, vdim = q.shape[0], k.shape[1] // kv_heads, v.shape[1] // kv_heads
+    out = torch.empty(T, heads * vdim, dtype=q.dtype, device=q.device)
+    assert q.shape[1] == heads * (dim + rot) and all(t.stride(1) == 1 for t in (q, k, v)) and (rot == 0 or krot.stride(1) == 1)
+    mode = 1 if gate is not None else 2 if gate_logits is not None else 0
+    assert mode != 1 or (gate.shape == (T, heads) and gate.dtype == torch.float32 and gate.is_contiguous())
+    assert mode != 2 or (gate_logits.shape == out.shape and gate_logits.dtype == q.dtype and gate_logits.stride(1) == 1)
+    gate = gate_logits if mode == 2 else gate
+    rows = [c for t in (q, k, v, krot) for c in (_p(t), c_longlong(0 if t is None else t.stride(0)))]
+    sizes = [c_int(x) for x in (T, heads, kv_heads, dim, rot, vdim, window or 0)] + [c_float(scale), c_float(cap or 0.0)]
+    tail = [_p(sink), c_int(mode), _p(gate), c_longlong(0 if gate is None else gate.stride(0)), _p(out)]
+    aligned = all(t is None or (t.data_ptr() % 16 == 0 and t.stride(0) % 8 == 0) for t in (q, k, v, krot)) and (
+        mode != 2 or (gate.data_ptr() % 16 == 0 and gate.stride(0) % 8 == 0))
+    if q.dtype == torch.bfloat16 and tensor_cores and aligned and scale > 0 and mixer_attn_tc_ok(heads, kv_heads, dim, rot, vdim):
+        cu = ctx.cu_seqlens
+        assert cu.dtype == torch.int32
+        _chk(lib().trlb_mixer_attn_tc(*rows, _p(cu), c_int(cu.numel() - 1), *sizes, *tail, _p(status_buffer(q.device)), _s()),
+             "mixer_attn_tc")
+    else:
+        _chk(lib().trlb_mixer_attn(*rows, _p(ctx.positions.to(torch.int32)), *sizes, *tail, _b(q), _s()), "mixer_attn")
     return out
 
 
-def latent_prompt_tc_ok(m) -> bool:
-    return m.scale > 0 and bool(lib().trlb_latent_attn_tc_ok(c_int(m.heads), c_int(m.dim), c_int(m.rot_dim), c_int(m.vdim)))
+def attn_prep(y, m, positions, temp, *, tok_slot=None, q=None, g=None, k_cache=None, v_cache=None, block_table=None, block_size=0):
+    """Rows ``y`` [q | k | v | g] of an attention mixer's input projection: unit-rms queries (times ``temp`` by position) and
+    keys, keys and values to the paged cache.  Without ``q`` queries and keys are replaced in place; with ``q`` (and ``g`` for
+    the gate logits) ``y`` is fp32 sums, and they are zeroed."""
+    rows = y.shape[0]
+    assert y.stride(1) == 1 and positions.dtype == torch.int32 and (q is None or y.dtype == torch.float32)
+    mb = 0 if block_table is None else block_table.shape[1]
+    _chk(lib().trlb_attn_prep(_p(y), c_int(int(y.dtype == torch.float32)), c_longlong(y.stride(0)), c_int(rows), c_int(m.heads),
+                              c_int(m.kv_heads), c_int(m.dim), c_int(m.vdim), c_int(int(m.kv_from is None)), c_int(1), c_float(m.eps),
+                              _p(positions), _p(tok_slot), _p(temp), _len(temp), _p(q), _p(g), _p(k_cache), _p(v_cache),
+                              _p(block_table), c_int(mb), c_int(block_size), _b(m.o), _s()), "attn_prep")
 
 
-def latent_prompt_tc(q, kv, lat, m, cu, gate):
-    """:func:`latent_prompt` on the tensor cores (bf16; see ``latent_prompt_tc_ok``); ``cu`` int32 sequence starts."""
-    T = q.shape[0]
-    kr, w = latent_row(m.kv_rank, m.rot_dim)
-    out = torch.empty(T, m.heads * m.vdim, dtype=q.dtype, device=q.device)
-    assert q.dtype == torch.bfloat16 and q.is_contiguous() and kv.stride(1) == 1 and lat.is_contiguous() and cu.dtype == torch.int32
-    _chk(lib().trlb_latent_attn_tc(_p(q), _p(kv), c_longlong(kv.stride(0)), _p(lat[:, kr:]), c_longlong(w), _p(cu),
-                                   c_int(cu.numel() - 1), c_int(T), c_int(m.heads), c_int(m.dim), c_int(m.rot_dim),
-                                   c_int(m.vdim), c_int(m.window or 0), c_float(m.scale), _p(m.sink), _p(gate), _p(out),
-                                   _p(status_buffer(q.device)), _s()), "latent_attn_tc")
+def grouped_decode(q, k_cache, v_cache, m, seq_lens, block_table, block_size, out, gate=None):
+    """One token per slot on the CUDA cores: any size, bf16 or fp32.  q [B, heads, dim], gate logits [B, heads vdim]."""
+    B = q.shape[0]
+    _chk(lib().trlb_grouped_decode(_p(q), _p(k_cache), _p(v_cache), _p(gate), _p(out), c_int(B), c_int(m.heads), c_int(m.kv_heads),
+                                   c_int(m.dim), c_int(m.vdim), c_float(m.scale), c_float(m.cap or 0.0), _p(seq_lens), _p(block_table),
+                                   c_int(block_table.shape[1]), c_int(block_size), _b(q), _s()), "grouped_decode")
+
+
+def grouped_decode_tc_ok(m, block_size: int) -> bool:
+    return m.scale > 0 and bool(lib().trlb_grouped_decode_tc_ok(c_int(m.heads), c_int(m.kv_heads), c_int(m.dim), c_int(m.vdim),
+                                                                c_int(block_size)))
+
+
+def grouped_decode_tc_items(B: int, m) -> int:
+    return int(lib().trlb_grouped_decode_tc_items(c_int(B), c_int(m.heads), c_int(m.kv_heads)))
+
+
+def grouped_decode_tc(q, k_cache, v_cache, m, seq_lens, block_table, block_size, out, gate=None, splits=1, part_o=None, part_ml=None):
+    """:func:`grouped_decode` on the tensor cores (bf16).  With ``splits`` > 1: ``part_o`` [>= B heads splits vdim] and
+    ``part_ml`` [>= 2 B heads splits] fp32 scratch."""
+    B = q.shape[0]
+    assert q.dtype == torch.bfloat16 and q.is_contiguous() and k_cache.is_contiguous() and v_cache.is_contiguous()
+    assert k_cache.shape[1] == block_size and out.is_contiguous() and (gate is None or gate.is_contiguous())
+    if splits > 1:
+        assert part_o.numel() >= B * m.heads * splits * m.vdim and part_ml.numel() >= 2 * B * m.heads * splits
+    _chk(lib().trlb_grouped_decode_tc(_p(q), _p(k_cache), _p(v_cache), _p(gate), _p(out), c_int(k_cache.shape[0]), c_int(B), c_int(m.heads),
+                                      c_int(m.kv_heads), c_int(m.dim), c_int(m.vdim), c_float(m.scale), c_float(m.cap or 0.0), _p(seq_lens),
+                                      _p(block_table), c_int(block_table.shape[1]), c_int(block_size), c_int(splits), _p(part_o), _p(part_ml),
+                                      _p(status_buffer(q.device)), _s()), "grouped_decode_tc")
+
+
+def conv_prompt(x, m, ctx, seq_slot=None, conv_state=None):
+    """Causal per-channel convolution of packed prompts: x [T, width] (rows may be strided) -> [T, width]; ``conv_state`` [slots,
+    taps - 1, width] of ``seq_slot`` gets the last inputs of every sequence."""
+    T, C = x.shape
+    assert x.stride(1) == 1
+    u = torch.empty(T, C, dtype=x.dtype, device=x.device)
+    cu = ctx.cu_seqlens
+    _chk(lib().trlb_conv_prompt(_p(x), c_longlong(x.stride(0)), _p(m.x_bias), _p(m.conv), _p(m.conv_bias), _p(ctx.positions.to(torch.int32)),
+                                c_int(T), c_int(C), c_int(m.taps), _p(cu), c_int(cu.numel() - 1), _p(seq_slot),
+                                c_int(0 if conv_state is None else conv_state.shape[0]), _p(conv_state), _p(u), _b(x), _s()), "conv_prompt")
+    return u
+
+
+def conv_step(x, m, seq_lens, state, u):
+    """One token per slot: x fp32 sums [B, width] (zeroed), state [B, taps - 1, width] moves on."""
+    B, C = x.shape
+    assert x.dtype == torch.float32 and x.stride(1) == 1
+    _chk(lib().trlb_conv_step(_p(x), c_longlong(x.stride(0)), _p(m.x_bias), _p(m.conv), _p(m.conv_bias), _p(seq_lens), c_int(B), c_int(C),
+                              c_int(m.taps), _p(state), _p(u), _b(u), _s()), "conv_step")
+
+
+def rglru_tc_ok(m) -> bool:
+    return bool(lib().trlb_rglru_tc_ok(c_int(m.width), c_int(m.blocks)))
+
+
+def rglru_scan(z, u, y, m, ctx, seq_slot=None, state=None):
+    """Recurrence of packed prompts on the CUDA cores.  z [T, 2, width] fp32 gate logits without their biases, u [T, width], y
+    [T, width] GELU branch without its bias (rows may be strided); ``state`` [slots, width] of ``seq_slot`` gets the final one."""
+    T, C = u.shape
+    out = torch.empty(T, C, dtype=u.dtype, device=u.device)
+    cu = ctx.cu_seqlens
+    _chk(lib().trlb_rglru_scan(_p(z), _p(u), _p(y), c_longlong(y.stride(0)), _p(m.lam), _p(m.gate_bias), _p(m.y_bias), _p(cu),
+                               c_int(cu.numel() - 1), _p(seq_slot), c_int(0 if state is None else state.shape[0]), _p(state),
+                               c_float(m.decay), c_int(C), _p(out), _b(u), _s()), "rglru_scan")
     return out
+
+
+def rglru_prompt_tc(u, y, m, ctx, seq_slot=None, state=None):
+    """Gate products and :func:`rglru_scan` in one tensor-core kernel (bf16; see ``rglru_tc_ok``)."""
+    T, C = u.shape
+    assert u.dtype == y.dtype == m.gates.dtype == torch.bfloat16 and u.is_contiguous() and m.gates.is_contiguous() and y.stride(1) == 1
+    out = torch.empty(T, C, dtype=u.dtype, device=u.device)
+    cu = ctx.cu_seqlens
+    _chk(lib().trlb_rglru_prompt_tc(_p(u), _p(y), c_longlong(y.stride(0)), _p(m.gates), _p(m.lam), _p(m.gate_bias), _p(m.y_bias), _p(cu),
+                                    c_int(cu.numel() - 1), c_int(T), _p(seq_slot), c_int(0 if state is None else state.shape[0]),
+                                    _p(state), c_float(m.decay), c_int(C), c_int(m.blocks), _p(out), _p(status_buffer(u.device)), _s()),
+         "rglru_prompt_tc")
+    return out
+
+
+def rglru_step(z, u, y, m, seq_lens, state, out):
+    """One token per slot; y: fp32 sums of the GELU branch (zeroed)."""
+    B, C = u.shape
+    _chk(lib().trlb_rglru_step(_p(z), _p(u), _p(y), c_longlong(y.stride(0)), _p(m.lam), _p(m.gate_bias), _p(m.y_bias), _p(seq_lens),
+                               c_int(B), _p(state), c_float(m.decay), c_int(C), _p(out), _b(u), _s()), "rglru_step")
+
+
+def rglru_step_tc(u, y, m, seq_lens, state, out):
+    """Gate products and :func:`rglru_step` in one tensor-core kernel (bf16)."""
+    B, C = u.shape
+    assert u.dtype == torch.bfloat16 and u.is_contiguous() and m.gates.is_contiguous() and state.shape[0] >= B
+    _chk(lib().trlb_rglru_step_tc(_p(u), _p(y), c_longlong(y.stride(0)), _p(m.gates), _p(m.lam), _p(m.gate_bias), _p(m.y_bias), _p(seq_lens),
+                                  c_int(B), _p(state), c_float(m.decay), c_int(C), c_int(m.blocks), _p(out), _p(status_buffer(u.device)),
+                                  _s()), "rglru_step_tc")
 
 
 def latent_absorb(qacc, m, positions, table, q_lat, clear):
@@ -113,7 +266,7 @@ def latent_absorb(qacc, m, positions, table, q_lat, clear):
     kr, w = latent_row(m.kv_rank, m.rot_dim)
     _chk(lib().trlb_latent_absorb(_p(qacc), c_longlong(qacc.stride(0)), _p(m.uk), _p(q_lat), c_int(B), c_int(m.heads),
                                   c_int(m.dim), c_int(m.rot_dim), c_int(m.kv_rank), c_int(kr), c_int(w), _p(positions),
-                                  _p(table), c_int(table.shape[0]), c_int(int(clear)), _b(q_lat), _s()), "latent_absorb")
+                                  _p(table), _len(table), c_int(int(clear)), _b(q_lat), _s()), "latent_absorb")
 
 
 def latent_decode(q_lat, cache, m, seq_lens, block_table, block_size, o_lat):
@@ -157,7 +310,7 @@ def latent_query(qacc, m, positions, table, q, q_lat):
     B = qacc.shape[0]
     kr, w = latent_row(m.kv_rank, m.rot_dim)
     _chk(lib().trlb_latent_query(_p(qacc), c_longlong(qacc.stride(0)), _p(q), _p(q_lat), c_int(B), c_int(m.heads), c_int(m.dim),
-                                 c_int(m.rot_dim), c_int(kr), c_int(w), _p(positions), _p(table), c_int(table.shape[0]), _s()),
+                                 c_int(m.rot_dim), c_int(kr), c_int(w), _p(positions), _p(table), _len(table), _s()),
          "latent_query")
 
 

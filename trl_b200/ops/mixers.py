@@ -1,10 +1,11 @@
 """Mechanisms of the layered decoders (models/layered.py) on packed prompts.
 
-CUDA tensors run the kernels of ``csrc/mixers.cu`` and the tensor-core mixer kernels, in bf16 or fp32; CPU tensors run
-:mod:`trl_b200.oracle.mixers`.  On CUDA the kernels are inference only (prompts, log-probs, generation).
+CUDA tensors run the kernels of ``csrc/mixers.cu``, ``csrc/grouped_attn.cu``, ``csrc/rglru.cu`` and the tensor-core mixer
+kernels, in bf16 or fp32; CPU tensors run :mod:`trl_b200.oracle.mixers`.  On CUDA the kernels are inference only (prompts,
+log-probs, generation).
 
-A serving engine passes itself through ``ctx.kv``: ``latent_cache(li)`` and ``recurrent_state(li)`` say where layer
-``li`` leaves what decoding continues from."""
+A serving engine passes itself through ``ctx.kv``: ``paged_cache(li)`` and ``recurrent_state(li)`` say where layer ``li``
+leaves what decoding continues from.  ``ctx.shared`` holds the keys and values that later layers of the same forward borrow."""
 from __future__ import annotations
 
 import contextlib
@@ -60,6 +61,24 @@ class RotarySpec:
         return t
 
 
+class TemperatureSpec:
+    """Factor of the query by position: ``1 + coef ln(floor((p + 1) / every) + 1)``, fp32 values of fp64 arithmetic."""
+
+    def __init__(self, coef: float, every: float):
+        self.coef, self.every = float(coef), every
+        self._tables: dict = {}
+
+    def table(self, n: int, device) -> torch.Tensor:
+        key = str(device)
+        t = self._tables.get(key)
+        if t is None or t.shape[0] < n:
+            size = max(256, 1 << (n - 1).bit_length())
+            p = torch.arange(1, size + 1, dtype=torch.float64)
+            t = (1.0 + self.coef * torch.log(torch.floor(p / self.every) + 1.0)).float().to(device)
+            self._tables[key] = t
+        return t
+
+
 def check_can_run(w: torch.Tensor):
     if w.is_cuda and torch.is_grad_enabled() and w.requires_grad:
         raise NotImplementedError("the CUDA kernels of the layered decoders are inference only: run them under "
@@ -98,12 +117,34 @@ def embed_scaled(ids, emb, scale):
     return F.embedding(ids, emb).float() * scale
 
 
-def dynamic_tanh(x, delta, alpha, w, b, out_dtype):
+def dynamic_tanh(x, delta, alpha, w, b, out_dtype, clear=False, out=None):
     """(norm of ``x + delta`` in ``out_dtype``, ``x + delta``); on CUDA the sum is formed in place."""
     if x.is_cuda:
-        return _k().dynamic_tanh(x, delta, alpha, w, b, out_dtype), x
+        return _k().dynamic_tanh(x, delta, alpha, w, b, out_dtype, clear=clear, out=out), x
     x = x if delta is None else x + delta
     return _ref.dynamic_tanh(x, alpha, w, b).to(out_dtype), x
+
+
+def rms_residual(x, delta, post, w, eps, out_dtype, clear=False, out=None):
+    """(``s / rms(s) * w`` in ``out_dtype``, s) of ``s = x + delta``, where delta over its rms times ``post`` is added when
+    ``post`` is given and s itself is the output when ``w`` is None; on CUDA the sum is formed in place."""
+    if x.is_cuda:
+        return _k().rms_residual(x, delta, post, w, eps, out_dtype, clear=clear, out=out), x
+    y, x = _ref.rms_residual(x, delta, post, w, eps)
+    return y.to(out_dtype), x
+
+
+def clamped_glu_linear(h, gate_up, limit, alpha, shift):
+    z = linear(h, gate_up)
+    return _k().clamped_glu(z, limit, alpha, shift) if z.is_cuda else _ref.clamped_glu(z, limit, alpha, shift)
+
+
+def side_input(h, ids, table, off, gate, proj):
+    """``proj (gelu_tanh(gate h) * table[ids, off : off + n])`` with fp32 sums."""
+    z = linear(h, gate)
+    if z.is_cuda:
+        return linear_f32(_k().side_gate(z, ids, table, off), proj)
+    return linear(F.gelu(z, approximate="tanh") * F.embedding(ids, table)[:, off:off + z.shape[1]].to(z.dtype), proj).float()
 
 
 def gelu_linear(h, up):
@@ -116,24 +157,77 @@ def latent_attention(m, h, ctx, li):
         return _ref.latent_attention(m, h.float(), ctx.positions, ctx.cu_seqlens)
     K = _k()
     pos = ctx.positions if ctx.positions.dtype == torch.int32 else ctx.positions.to(torch.int32)
-    table = m.rope.table(ctx.max_seqlen, h.device)
+    table = m.rope.table(ctx.max_seqlen, h.device) if m.rot_dim else None
     kr, width = K.latent_row(m.kv_rank, m.rot_dim)
     lat = torch.zeros(h.shape[0], width, dtype=h.dtype, device=h.device)
-    cache = ctx.kv.latent_cache(li) if ctx.kv is not None else {}
-    cq, gate = K.latent_prep(linear_f32(h, m.w_in), m, pos, table, lat=lat, **cache)
-    q = linear(cq, m.uq)
-    K.rotate_q(q, m, pos, table)
+    cache = ctx.kv.paged_cache(li) if ctx.kv is not None else {}
+    if m.q_rank:
+        cq, gate = K.latent_prep(linear_f32(h, m.w_in), m, pos, table, lat=lat, **cache)
+        q = linear(cq, m.uq)
+    else:
+        q = linear(h, m.w_in[: m.q_rows])
+        _, gate = K.latent_prep(linear_f32(h, m.w_in[m.q_rows:]), m, pos, table, lat=lat, **cache)
+    if m.rot_dim:
+        K.rotate_q(q, m, pos, table)
     kv = linear(lat[:, : m.kv_rank], m.ukv)
     return linear_f32(latent_prompt_attention(q, kv, lat, m, ctx, gate), m.o)
 
 
-def latent_prompt_attention(q, kv, lat, m, ctx, gate):
-    """Windowed sink attention of packed prompts, times the output gates.  q [T, heads (dim | rot)] rotated, kv [T, heads
-    dim | heads vdim], lat [T, latent row], gate [T, heads] -> [T, heads vdim]."""
+def latent_prompt_attention(q, kv, lat, m, ctx, gate, tensor_cores=True):
+    """Attention of packed prompts with latent keys and values, times the output gates (if any).  q [T, heads (dim | rot)]
+    rotated, kv [T, heads dim | heads vdim], lat [T, latent row], gate [T, heads] -> [T, heads vdim]."""
     K = _k()
-    if q.dtype == torch.bfloat16 and K.latent_prompt_tc_ok(m):
-        return K.latent_prompt_tc(q, kv, lat, m, ctx.cu_seqlens, gate)
-    return K.latent_prompt(q, kv, lat, m, ctx.positions.to(torch.int32), gate)
+    kr, _ = K.latent_row(m.kv_rank, m.rot_dim)
+    n = m.heads * m.dim
+    return K.mixer_attn(q, kv[:, :n], kv[:, n:], heads=m.heads, kv_heads=m.heads, rot=m.rot_dim, krot=lat[:, kr:] if m.rot_dim else None,
+                        scale=m.scale, window=m.window, sink=m.sink, gate=gate, ctx=ctx, tensor_cores=tensor_cores)
+
+
+def attention(m, h, ctx, li):
+    kept = ctx.shared[m.kv_from] if m.kv_from is not None else None
+    if not h.is_cuda:
+        out, kept = _ref.attention(m, h.float(), ctx.positions, ctx.cu_seqlens, kept)
+    else:
+        K = _k()
+        pos = ctx.positions if ctx.positions.dtype == torch.int32 else ctx.positions.to(torch.int32)
+        temp = m.temperature.table(ctx.max_seqlen, h.device) if m.temperature is not None else None
+        y = linear(h, m.w_in)
+        K.attn_prep(y, m, pos, temp, **(ctx.kv.paged_cache(li) if ctx.kv is not None else {}))
+        q, k, v, g = y.split(m.parts, 1)
+        kept = (k, v) if kept is None else kept
+        o = K.mixer_attn(q, *kept, heads=m.heads, kv_heads=m.kv_heads, scale=m.scale, cap=m.cap, gate_logits=g, ctx=ctx)
+        out = linear_f32(o, m.o)
+    if li in ctx.shared:
+        ctx.shared[li] = kept
+    return out
+
+
+def block_gates(u, gates):
+    """Block-diagonal products in fp32: u [T, C], gates [2, blocks, C / blocks (out), C / blocks (in)] -> [T, 2, C]."""
+    T, C = u.shape
+    n, blocks, w, _ = gates.shape
+    with _ieee_fp32():
+        z = torch.matmul(u.float().view(T, blocks, w).transpose(0, 1), gates.float().transpose(2, 3))  # [2, blocks, T, w]
+    return z.permute(2, 0, 1, 3).reshape(T, n, C)
+
+
+def rglru(m, h, ctx, li):
+    if not h.is_cuda:
+        return _ref.rglru(m, h.float(), ctx.cu_seqlens)
+    K = _k()
+    y, x = linear(h, m.w_in).chunk(2, 1)
+    where = ctx.kv.recurrent_state(li) if ctx.kv is not None else {}
+    slot, state = where.get("seq_slot"), where.get("state")
+    u = K.conv_prompt(x, m, ctx, slot, where.get("conv_state"))
+    return linear_f32(rglru_prompt_scan(u, y, m, ctx, slot, state), m.o)
+
+
+def rglru_prompt_scan(u, y, m, ctx, seq_slot=None, state=None, tensor_cores=True):
+    """Gates, recurrence and multiplication by the GELU branch over packed prompts: u, y [T, width] -> [T, width]."""
+    K = _k()
+    if u.dtype == torch.bfloat16 and tensor_cores and K.rglru_tc_ok(m):
+        return K.rglru_prompt_tc(u, y, m, ctx, seq_slot, state)
+    return K.rglru_scan(block_gates(u, m.gates), u, y, m, ctx, seq_slot, state)
 
 
 def mlstm_prompt_scan(y, m, ig, fg, ctx, where):

@@ -14,6 +14,19 @@ def unit_rms(x, eps):
     return x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps)
 
 
+def rms_residual(x, delta, post, w, eps):
+    """(``x + delta`` (delta over its rms times ``post``, when given)) over its rms times ``w`` (when given), and the sum."""
+    if delta is not None:
+        x = x + (delta if post is None else unit_rms(delta, eps) * post)
+    return (x if w is None else unit_rms(x, eps) * w), x
+
+
+def clamped_glu(z, limit, alpha, shift):
+    g, u = z.chunk(2, -1)
+    g, u = g.clamp(max=limit), u.clamp(-limit, limit)
+    return g * torch.sigmoid(alpha * g) * (u + shift)
+
+
 def rotate_pairs(x, cos, sin):
     """x [T, ..., n] with pairs (2i, 2i + 1); cos / sin [T, n / 2]."""
     shape = (x.shape[0],) + (1,) * (x.ndim - 2) + (x.shape[-1] // 2,)
@@ -22,18 +35,24 @@ def rotate_pairs(x, cos, sin):
     return torch.stack([u * c - v * s, v * c + u * s], -1).flatten(-2)
 
 
-def sink_window_attention(q, k, v, scale, window, sink, cu):
-    """q, k [T, H, D], v [T, H, E], packed sequences by ``cu``; softmax with ``exp(sink)`` added to the denominator."""
-    outs = []
+def sink_window_attention(q, k, v, scale, window, sink, cu, cap=None):
+    """q [T, H, D], k [T, G, D], v [T, G, E] (H / G query heads read one key head), packed sequences by ``cu``; scores
+    ``cap tanh(s / cap)``; softmax with ``exp(sink)`` added to the denominator (no such term without a sink)."""
+    outs, per = [], q.shape[1] // k.shape[1]
+    if per > 1:
+        k, v = k.repeat_interleave(per, 1), v.repeat_interleave(per, 1)
     for a, b in zip(cu[:-1].tolist(), cu[1:].tolist()):
         n = b - a
         s = torch.einsum("qhd,khd->hqk", q[a:b], k[a:b]) * scale
-        i = torch.arange(n)
+        if cap is not None:
+            s = cap * torch.tanh(s / cap)
+        i = torch.arange(n, device=s.device)
         gap = i[:, None] - i[None, :]
         seen = (gap >= 0) if window is None else (gap >= 0) & (gap < window)
         s = s.masked_fill(~seen, float("-inf"))
-        full = torch.cat([s, sink.to(s.dtype)[:, None, None].expand(-1, n, 1)], -1)
-        outs.append(torch.einsum("hqk,khe->qhe", torch.softmax(full, -1)[..., :-1], v[a:b]))
+        if sink is not None:
+            s = torch.cat([s, sink.to(s.dtype)[:, None, None].expand(-1, n, 1)], -1)
+        outs.append(torch.einsum("hqk,khe->qhe", torch.softmax(s, -1)[..., :n], v[a:b]))
     return torch.cat(outs)
 
 
@@ -57,19 +76,74 @@ def latent_attention(m, h, positions, cu):
     """``m``: a models.layered.LatentAttention; h [T, width] -> [T, width]."""
     T, H = h.shape[0], m.heads
     y = F.linear(h, m.w_in.to(h.dtype))
-    ql, kl, kr, g = y.split([m.q_rank, m.kv_rank, m.rot_dim, H], -1)
-    table = m.rope.table(int(positions.max()) + 1 if T else 1, h.device).to(h.dtype)[positions.long()]
-    cos, sin = table[..., 0], table[..., 1]
-    q = F.linear(unit_rms(ql, m.eps) * m.q_norm.to(h.dtype), m.uq.to(h.dtype)).view(T, H, m.dim + m.rot_dim)
-    q = torch.cat([q[..., : m.dim], rotate_pairs(q[..., m.dim:], cos, sin)], -1)
+    q, kl, kr, g = y.split([m.q_rows, m.kv_rank, m.rot_dim, H if m.gated else 0], -1)
+    if m.q_rank:
+        q = F.linear(unit_rms(q, m.eps) * m.q_norm.to(h.dtype), m.uq.to(h.dtype))
+    q = q.view(T, H, m.dim + m.rot_dim)
     lat = unit_rms(kl, m.eps) * m.kv_norm.to(h.dtype)
-    kr = rotate_pairs(kr, cos, sin)
     k = F.linear(lat, m.uk.to(h.dtype)).view(T, H, m.dim)
-    k = torch.cat([k, kr[:, None].expand(T, H, m.rot_dim)], -1)
+    if m.rot_dim:
+        table = m.rope.table(int(positions.max()) + 1 if T else 1, h.device).to(h.dtype)[positions.long()]
+        cos, sin = table[..., 0], table[..., 1]
+        q = torch.cat([q[..., : m.dim], rotate_pairs(q[..., m.dim:], cos, sin)], -1)
+        k = torch.cat([k, rotate_pairs(kr, cos, sin)[:, None].expand(T, H, m.rot_dim)], -1)
     v = F.linear(lat, m.uv.to(h.dtype)).view(T, H, m.vdim)
     o = sink_window_attention(q, k, v, m.scale, m.window, m.sink, cu)
-    o = o * torch.sigmoid(g)[..., None]
+    if m.gated:
+        o = o * torch.sigmoid(g)[..., None]
     return F.linear(o.reshape(T, H * m.vdim), m.o.to(h.dtype))
+
+
+def attention(m, h, positions, cu, kept=None):
+    """``m``: a models.layered.GroupedAttention; ``kept``: keys and values of the layer it borrows from.  Returns ([T, width],
+    (keys, values))."""
+    T, H, G = h.shape[0], m.heads, m.kv_heads
+    y = F.linear(h, m.w_in.to(h.dtype))
+    own = 0 if m.kv_from is not None else G
+    q, k, v, g = y.split([H * m.dim, own * m.dim, own * m.vdim, H * m.vdim], -1)
+    q = unit_rms(q.view(T, H, m.dim), m.eps)
+    if m.temperature is not None:
+        q = q * m.temperature.table(int(positions.max()) + 1 if T else 1, h.device).to(h.dtype)[positions.long()][:, None, None]
+    if kept is None:
+        kept = unit_rms(k.view(T, G, m.dim), m.eps), v.view(T, G, m.vdim)
+    o = sink_window_attention(q, *kept, m.scale, None, None, cu, m.cap).reshape(T, H * m.vdim)
+    return F.linear(o * torch.sigmoid(g), m.o.to(h.dtype)), kept
+
+
+def causal_conv(x, w, bias, cu):
+    """x [T, C], w [C, taps] (last column: the current token), zeros before the start of every sequence."""
+    taps = w.shape[1]
+    outs = []
+    for a, b in zip(cu[:-1].tolist(), cu[1:].tolist()):
+        padded = F.pad(x[a:b].T[None], (taps - 1, 0))
+        outs.append(F.conv1d(padded, w.to(x.dtype)[:, None], bias.to(x.dtype), groups=x.shape[1])[0].T)
+    return torch.cat(outs)
+
+
+def linear_recurrence(a, b, cu):
+    """S_t = a_t S_(t-1) + b_t from S = 0, per channel.  Doubling: after step s an entry covers 2^s tokens."""
+    outs = []
+    for i, j in zip(cu[:-1].tolist(), cu[1:].tolist()):
+        x, y, d = a[i:j], b[i:j], 1
+        while d < j - i:
+            y = torch.cat([y[:d], x[d:] * y[:-d] + y[d:]])
+            x = torch.cat([x[:d], x[d:] * x[:-d]])
+            d *= 2
+        outs.append(y)
+    return torch.cat(outs)
+
+
+def rglru(m, h, cu):
+    """``m``: a models.layered.RgLru."""
+    T = h.shape[0]
+    y, x = F.linear(h, m.w_in.to(h.dtype)).chunk(2, -1)
+    y = F.gelu(y + m.y_bias.to(h.dtype), approximate="tanh")
+    u = causal_conv(x + m.x_bias.to(h.dtype), m.conv, m.conv_bias, cu)
+    z = torch.einsum("tbi,gboi->tgbo", u.view(T, m.blocks, -1), m.gates.to(h.dtype)).reshape(T, 2, -1)
+    r, i = torch.sigmoid(z + m.gate_bias.to(h.dtype)).unbind(1)
+    log_a = -m.decay * r * F.softplus(m.lam.to(h.dtype))
+    b = torch.sqrt(-torch.expm1(2 * log_a)) * i * u
+    return F.linear(linear_recurrence(torch.exp(log_a), b, cu) * y, m.o.to(h.dtype))
 
 
 def mlstm(m, h, cu):

@@ -2,16 +2,20 @@
 :class:`~trl_b200.rollout.engine.RolloutEngine`'s; this module adds what a layer keeps between tokens and how it takes
 one token further.
 
-Every layer of the list has a cache of its own, also one that runs with another layer's weights:
+Every layer of the list has a cache of its own, also one that runs with another layer's weights (a layer with ``kv_from``
+reads that layer's instead):
 
     latent_attention   pages of latent rows ``[kv_rank | rotated key]`` behind the engine's block table (the window is a
                        mask: pages stay until the sequence ends)
+    attention          pages of keys (over their rms) and pages of values
     mlstm              per slot an fp32 matrix state, its normaliser and running maximum
+    rglru              per slot an fp32 state vector and the last inputs of the convolution
 
 A decode step is one graph: embed, then per layer norm (+ residual) -> input projection -> mixer -> output projection
--> norm (+ residual) -> up / GELU -> down, then final norm, head and sampler.  With bf16 weights the projections are
-the weight-streaming tcgen05 kernel; their fp32 sums are consumed and cleared by the next kernel.  fp32 models run the
-same kernels' fp32 forms with library fp32 matrix products."""
+-> norm (+ residual) -> up / activation -> down (-> stream -> side gate -> side projection), then final norm, head and
+sampler.  Norms on a sublayer's output ride on the norm kernel that follows.  With bf16 weights the projections are the
+weight-streaming tcgen05 kernel; their fp32 sums are consumed and cleared by the next kernel.  fp32 models run the same
+kernels' fp32 forms with library fp32 matrix products."""
 from __future__ import annotations
 
 import os
@@ -19,6 +23,7 @@ import os
 import torch
 
 from ..models.decoder import SeqCtx
+from ..models.layered import ClampedGluMlp
 from ..ops import mixers as mx
 from .engine import RolloutEngine
 
@@ -26,18 +31,21 @@ from .engine import RolloutEngine
 class _LatentSlots:
     """Decode side of one ``latent_attention`` layer."""
 
-    def __init__(self, eng: "LayeredRolloutEngine", m):
+    def __init__(self, eng: "LayeredRolloutEngine", m, li):
         from ..ops import cuda_mixers as K
 
         self.e, self.m = eng, m
         self.kr, self.width = K.latent_row(m.kv_rank, m.rot_dim)
         self.cache = torch.zeros(eng.num_blocks, eng.block_size, self.width, dtype=eng.dtype, device=eng.dev)
-        self.table = m.rope.table(eng.max_len + 1, eng.dev)
+        self.table = m.rope.table(eng.max_len + 1, eng.dev) if m.rot_dim else None
         B = eng.max_seqs
         self.acc_in = eng.sums("in", m.w_in.shape[0])
-        self.acc_q = eng.sums("q", m.uq.shape[0])
-        self.cq = eng.scratch("cq", B, m.q_rank)
-        self.gate = eng.scratch("gate", B, m.heads, dtype=torch.float32)
+        if m.q_rank:  # queries through a latent: prepared with the rest of the row
+            self.acc_q, self.acc_prep = eng.sums("q", m.uq.shape[0]), self.acc_in
+            self.cq = eng.scratch("cq", B, m.q_rank)
+        else:
+            self.acc_q, self.acc_prep, self.cq = self.acc_in[:, : m.q_rows], self.acc_in[:, m.q_rows:], None
+        self.gate = eng.scratch("gate", B, m.heads, dtype=torch.float32) if m.gated else None
         self.q_lat = eng.scratch("q_lat", B, m.heads, self.width)
         self.o_lat = eng.scratch("o_lat", B, m.heads, m.kv_rank)
         self.o = eng.scratch("o", B, m.heads * m.vdim)
@@ -97,9 +105,10 @@ class _LatentSlots:
 
         e, m = self.e, self.m
         e.gemm(h, m.w_in, self.acc_in)
-        K.latent_prep(self.acc_in, m, e.seq_lens, self.table, clear=True, cq=self.cq, gate=self.gate, cache=self.cache,
+        K.latent_prep(self.acc_prep, m, e.seq_lens, self.table, clear=True, cq=self.cq, gate=self.gate, cache=self.cache,
                       block_table=e.block_table, block_size=e.block_size)
-        e.gemm(self.cq, m.uq, self.acc_q)
+        if m.q_rank:
+            e.gemm(self.cq, m.uq, self.acc_q)
         self.absorb()
         self.attend()
         self.expand()
@@ -109,7 +118,7 @@ class _LatentSlots:
 class _MLstmSlots:
     """Decode side of one ``mlstm`` layer."""
 
-    def __init__(self, eng: "LayeredRolloutEngine", m):
+    def __init__(self, eng: "LayeredRolloutEngine", m, li):
         self.e, self.m = eng, m
         B, f32 = eng.max_seqs, dict(dtype=torch.float32, device=eng.dev)
         # the normaliser and the maximum are double-buffered by the parity of the token count (csrc/mixers.cu)
@@ -141,19 +150,133 @@ class _MLstmSlots:
         e.gemm(self.y, m.o, out)
 
 
-SLOTS = {"latent_attention": _LatentSlots, "mlstm": _MLstmSlots}
+class _AttentionSlots:
+    """Decode side of one ``attention`` layer."""
+
+    def __init__(self, eng: "LayeredRolloutEngine", m, li):
+        from ..ops import cuda_mixers as K
+
+        self.e, self.m = eng, m
+        self.own = m.kv_from is None
+        if self.own:
+            shape = (eng.num_blocks, eng.block_size, m.kv_heads)
+            self.k_cache = torch.zeros(*shape, m.dim, dtype=eng.dtype, device=eng.dev)
+            self.v_cache = torch.zeros(*shape, m.vdim, dtype=eng.dtype, device=eng.dev)
+        else:
+            lender = eng.slots[m.kv_from]
+            self.k_cache, self.v_cache = lender.k_cache, lender.v_cache
+        self.temp = m.temperature.table(eng.max_len + 1, eng.dev) if m.temperature is not None else None
+        B = eng.max_seqs
+        self.acc_in = eng.sums("in", m.w_in.shape[0])
+        self.q = eng.scratch("q", B, m.heads, m.dim)
+        self.g = eng.scratch("g", B, m.heads * m.vdim)
+        self.o = eng.scratch("o", B, m.heads * m.vdim)
+        # tensor-core decode; other sizes and fp32 run the CUDA-core kernel
+        self.tc = eng.dtype == torch.bfloat16 and K.grouped_decode_tc_ok(m, eng.block_size)
+        self.splits, self.part_o, self.part_ml = 1, None, None
+        if self.tc:
+            self.splits = max(1, min(8, -(-eng.max_len // 128), 148 // K.grouped_decode_tc_items(B, m)))
+            if self.splits > 1:
+                self.part_o = eng.scratch("part_o", B, m.heads * self.splits * m.vdim, dtype=torch.float32)
+                self.part_ml = eng.scratch("part_ml", B, m.heads * self.splits * 2, dtype=torch.float32)
+
+    def prompt_target(self, pages: "_Pages") -> dict:
+        if not self.own:
+            return {}
+        return dict(k_cache=self.k_cache, v_cache=self.v_cache, tok_slot=pages.tok_slot, block_table=self.e.block_table,
+                    block_size=self.e.block_size)
+
+    def copy_pages(self, dst, src):
+        for c in (self.k_cache, self.v_cache) if self.own else ():
+            c.index_copy_(0, dst, c.index_select(0, src))
+
+    def copy_slots(self, dst, src):
+        pass
+
+    def prepare(self):
+        """``acc_in`` -> queries, gate logits, the new rows of the cache."""
+        from ..ops import cuda_mixers as K
+
+        e = self.e
+        where = dict(k_cache=self.k_cache, v_cache=self.v_cache, block_table=e.block_table, block_size=e.block_size) if self.own else {}
+        K.attn_prep(self.acc_in, self.m, e.seq_lens, self.temp, q=self.q, g=self.g, **where)
+
+    def attend(self):
+        from ..ops import cuda_mixers as K
+
+        e = self.e
+        args = (self.q, self.k_cache, self.v_cache, self.m, e.seq_lens, e.block_table, e.block_size, self.o, self.g)
+        if self.tc:
+            K.grouped_decode_tc(*args, self.splits, self.part_o, self.part_ml)
+        else:
+            K.grouped_decode(*args)
+
+    def step(self, h, out):
+        self.e.gemm(h, self.m.w_in, self.acc_in)
+        self.prepare()
+        self.attend()
+        self.e.gemm(self.o, self.m.o, out)
+
+
+class _RgLruSlots:
+    """Decode side of one ``rglru`` layer."""
+
+    def __init__(self, eng: "LayeredRolloutEngine", m, li):
+        from ..ops import cuda_mixers as K
+
+        self.e, self.m = eng, m
+        B, f32 = eng.max_seqs, dict(dtype=torch.float32, device=eng.dev)
+        self.state = torch.zeros(B, m.width, **f32)
+        self.conv_state = torch.zeros(B, m.taps - 1, m.width, **f32)
+        self.acc_in = eng.sums("in", 2 * m.width)
+        self.u = eng.scratch("u", B, m.width)
+        self.y = eng.scratch("o", B, m.width)
+        self.tc = eng.dtype == torch.bfloat16 and K.rglru_tc_ok(m)
+
+    def prompt_target(self, pages: "_Pages") -> dict:
+        return dict(seq_slot=pages.slots, state=self.state, conv_state=self.conv_state)
+
+    def copy_pages(self, dst, src):
+        pass
+
+    def copy_slots(self, dst, src):
+        for t in (self.state, self.conv_state):
+            t.index_copy_(0, dst, t.index_select(0, src))
+
+    def convolve(self):
+        from ..ops import cuda_mixers as K
+
+        K.conv_step(self.acc_in[:, self.m.width:], self.m, self.e.seq_lens, self.conv_state, self.u)
+
+    def recur(self):
+        from ..ops import cuda_mixers as K
+
+        args = (self.u, self.acc_in[:, : self.m.width], self.m, self.e.seq_lens, self.state, self.y)
+        if self.tc:
+            K.rglru_step_tc(*args)
+        else:
+            K.rglru_step(mx.block_gates(self.u, self.m.gates), *args)
+
+    def step(self, h, out):
+        self.e.gemm(h, self.m.w_in, self.acc_in)
+        self.convolve()
+        self.recur()
+        self.e.gemm(self.y, self.m.o, out)
+
+
+SLOTS = {"latent_attention": _LatentSlots, "mlstm": _MLstmSlots, "attention": _AttentionSlots, "rglru": _RgLruSlots}
 
 
 class _Pages:
-    """``ctx.kv`` of a prompt forward: where layer ``li`` leaves its latents or its final state."""
+    """``ctx.kv`` of a prompt forward: where layer ``li`` leaves its keys and values or its final state."""
 
     def __init__(self, eng, tok_slot, slots):
         self.e, self.tok_slot, self.slots = eng, tok_slot, slots
 
-    def latent_cache(self, li):
+    def paged_cache(self, li):
         return self.e.slots[li].prompt_target(self)
 
-    recurrent_state = latent_cache
+    recurrent_state = paged_cache
 
 
 class LayeredRolloutEngine(RolloutEngine):
@@ -190,7 +313,9 @@ class LayeredRolloutEngine(RolloutEngine):
         # weight-streaming GEMM: bf16, at most 128 rows, rows of 16 bytes; other shapes and fp32 use the library
         self._own_gemm = (os.environ.get("TRL_B200_DECODE_GEMM", "own") != "cublas" and self.dtype == torch.bfloat16
                           and B <= 128)
-        self.slots = [SLOTS[s.kind](self, l.mixer) for s, l in zip(cfg.layers, self.model.layers)]
+        self.slots: list = []  # a layer may look up an earlier one
+        for li, (s, l) in enumerate(zip(cfg.layers, self.model.layers)):
+            self.slots.append(SLOTS[s.kind](self, l.mixer, li))
         self._x = torch.zeros(B, H, dtype=torch.float32, device=self.dev)
         self._acc = self.sums("out", H)
         self._h = self.scratch("h", B, H)
@@ -242,31 +367,45 @@ class LayeredRolloutEngine(RolloutEngine):
         from ..ops import cuda as K
         from ..ops import cuda_mixers as KM
 
-        m, x, h, acc = self.model, self._x, self._h, self._acc
+        m, x, h, acc, dt = self.model, self._x, self._h, self._acc, self.dtype
         KM.embed_scaled(self.next_input, m.embed_tokens, self.cfg.embed_scale, out=x)
-
-        def norm(n, delta):
-            KM.dynamic_tanh(x, delta, n.alpha, n.weight, n.bias, self.dtype, clear=True, out=h)
-
-        delta = None
-        for layer, slots in zip(m.layers, self.slots):
-            norm(layer.norm1, delta)
+        delta = post = None  # sums not yet added to the stream, and the norm they pass first
+        for li, (layer, slots) in enumerate(zip(m.layers, self.slots)):
+            layer.norm1(x, dt, delta, post, clear=True, out=h)
             slots.step(h, acc)
-            delta = acc
+            delta, post = acc, layer.norm1b
             if layer.mlp is not None:
-                norm(layer.norm2, delta)
-                self.gemm(self._up_gelu(h, layer.mlp), layer.mlp.down, acc)
-        norm(m.norm, delta)
+                layer.norm2(x, dt, delta, post, clear=True, out=h)
+                self.gemm(self.mlp_act(h, layer.mlp), layer.mlp.down, acc)
+                post = layer.norm2b
+            if layer.side is not None:
+                layer.side.stream(x, dt, delta, post, clear=True, out=h)
+                self.gemm(self.side_act(h, layer.side, li), layer.side.proj, acc)
+                post = layer.side.norm
+        m.norm(x, dt, delta, post, clear=True, out=h)
         if self._own_gemm and h.shape[1] % 8 == 0:
             return K.decode_gemm(h, m.lm_head_weight, out=self._logits_buf)
         return mx.linear(h, m.lm_head_weight)
 
-    def _up_gelu(self, h, mlp):
+    def mlp_act(self, h, mlp):
+        """Activation of a feed-forward: fused into the product where the weight-streaming kernel runs."""
+        from ..ops import cuda as K
         from ..ops import cuda_mixers as KM
 
-        act = self.scratch("act", self.max_seqs, mlp.up.shape[0])
-        if self._own_gemm and h.shape[1] % 8 == 0:
-            from ..ops import cuda as K
-
+        act = self.scratch("act", self.max_seqs, mlp.down.shape[1])
+        own = self._own_gemm and h.shape[1] % 8 == 0
+        if isinstance(mlp, ClampedGluMlp):
+            if own:
+                return K.decode_gemm(h, mlp.gate_up, out=act, clamped_glu=mlp.glu)
+            return KM.clamped_glu(mx.linear(h, mlp.gate_up), *mlp.glu, out=act)
+        if own:
             return K.decode_gemm(h, mlp.up, out=act, gelu=True)
         return KM.gelu_erf(mx.linear(h, mlp.up), out=act)
+
+    def side_act(self, h, side, li):
+        from ..ops import cuda_mixers as KM
+
+        z = self.sums("side", side.dim)
+        self.gemm(h, side.gate, z)
+        return KM.side_gate(z, self.next_input, self.model.side_embed, li * side.dim, clear=True,
+                            out=self.scratch("side_act", self.max_seqs, side.dim))
