@@ -65,13 +65,13 @@ def parse():
                          "warm-up steps how many layers fit (gradient_checkpointing_kwargs={'num_layers': 'auto'}).  With "
                          "micro-batches of varying length keeping activations did not pay here: the allocator's "
                          "remapping cost what the recomputation saved")
-    ap.add_argument("--layered", action="store_true",
-                    help="instead of the GRPO workload: prompt and decode throughput of the layered design (Zorelorn) beside a "
-                         "flat decoder of equal width, depth and parameter count, and the mixers' kernels alone (one GPU)")
+    ap.add_argument("--layered", nargs="?", const="zorelorn", choices=["zorelorn", "povusun"],
+                    help="instead of the GRPO workload: prompt and decode throughput of a layered design (default Zorelorn) beside "
+                         "a flat decoder of equal width, depth and parameter count, and the mixers' kernels alone (one GPU)")
     return ap.parse_args()
 
 
-def layered_arm():
+def layered_arm(design):
     """One JSON line: throughput at two sizes and the kernel table of the larger one."""
     import torch
 
@@ -79,11 +79,11 @@ def layered_arm():
 
     clk = ClockSampler(torch.cuda.current_device())
     clk.start()
-    rows = run()
+    rows = run(design=design)
     clocks = clk.stop()
     print(json.dumps({"metric": "layered_decoder_throughput", "unit": "tok/s", "n_gpus": 1, "dtype": "bf16", "data": "synthetic",
                       "config": {"timing": "CUDA events; weights of a step larger than L2; kernels alone: L2 flushed"},
-                      "sizes": rows, "kernels": kernel_table(), "clocks": clocks}))
+                      "sizes": rows, "kernels": kernel_table(design=design), "clocks": clocks}))
     return 0
 
 
@@ -172,7 +172,7 @@ def main():
     if a.impl == "reference":
         return reference_arm()
     if a.layered:
-        return layered_arm()
+        return layered_arm(a.layered)
     import torch
 
     from trl_b200.models.configuration import preset

@@ -1,7 +1,7 @@
 """Prompt and decode throughput of a layered design beside the closest flat decoder of the same width, depth and
 parameter count (random weights, bf16, one GPU), through the serving engine.
 
-    python -m trl_b200.benchmarks.layered_throughput [--sizes small,base] [--kernels]
+    python -m trl_b200.benchmarks.layered_throughput [--design zorelorn|povusun] [--sizes small,base] [--kernels]
 
 Prompt: packed prompts through the engine's prompt forward into its cache.  Decode: replays of the captured step (CUDA
 graph, sampler included) with every slot at the given context.  CUDA events after warm-up; the weights of a step are
@@ -14,13 +14,15 @@ import os
 
 import torch
 
-# width, heads (latent attention and flat attention), query latent, ff, mLSTM heads
-SIZES = {"small": dict(width=2048, heads=16, q_rank=768, ff=8192, mheads=4, pairs=4),
-         "base": dict(width=4096, heads=32, q_rank=1536, ff=16384, mheads=8, pairs=4)}
+# width, heads (attention of every kind), ff; Zorelorn: query latent, mLSTM heads, pairs of layers; Povusun: side input, quads
+SIZES = {"zorelorn": {"small": dict(width=2048, heads=16, q_rank=768, ff=8192, mheads=4, pairs=4),
+                      "base": dict(width=4096, heads=32, q_rank=1536, ff=16384, mheads=8, pairs=4)},
+         "povusun": {"small": dict(width=2048, heads=16, ff=6144, side=256, quads=2),
+                     "base": dict(width=4096, heads=32, ff=12288, side=256, quads=2)}}
 VOCAB = 32768
 
 
-def layered_config(width, heads, q_rank, ff, mheads, pairs, window=1024):
+def zorelorn_config(width, heads, q_rank, ff, mheads, pairs, window=1024):
     att = dict(type="latent_attention", mlp=dict(kind="dense", ff=ff),
                mixer=dict(heads=heads, dim=128, rot_dim=64, vdim=128, q_rank=q_rank, kv_rank=512, scale=192 ** -0.5,
                           mask=dict(size=window), rot=dict(base=1e4, dims=64, scaling=dict(factor=4.0, original=4096,
@@ -30,13 +32,29 @@ def layered_config(width, heads, q_rank, ff, mheads, pairs, window=1024):
                 layers=[att, rec] * pairs)
 
 
-def flat_config(s, target):
+def povusun_config(width, heads, ff, side, quads):
+    mlp = dict(kind="dense", ff=ff, limit=7.0)
+    att = dict(heads=heads, kv_heads=heads // 4, dim=128, vdim=128, scale=128 ** -0.5, softcap=50.0, q_temp=dict(coef=0.1, every=1024))
+    lat = dict(type="latent_attention", mlp=mlp, mixer=dict(heads=heads, dim=128, vdim=128, kv_rank=512, scale=128 ** -0.5))
+    rec = dict(type="rglru", mlp=mlp, mixer=dict(width=width, blocks=width // 256, conv=4))
+    layers = []
+    for i in range(quads):  # every second attention layer reads the cache of the one before
+        own = dict(att, kv_from=4 * (i - 1)) if i % 2 else att
+        layers += [dict(type="attention", mlp=mlp, mixer=own), rec, lat, rec]
+    return dict(architecture="Povusun", vocab=VOCAB, width=width, norm=dict(eps=1e-6), token_side=dict(dim=side), layers=layers)
+
+
+def layered_config(design, s):
+    return zorelorn_config(**s) if design == "zorelorn" else povusun_config(**s)
+
+
+def flat_config(s, depth, target, tied):
     """Llama-type decoder of the same width and depth whose feed-forward width brings it to ``target`` parameters."""
     from ..models.configuration import ModelArch
 
-    kw = dict(model_type="llama", vocab_size=VOCAB, hidden_size=s["width"], num_hidden_layers=2 * s["pairs"],
+    kw = dict(model_type="llama", vocab_size=VOCAB, hidden_size=s["width"], num_hidden_layers=depth,
               num_attention_heads=s["width"] // 128, num_key_value_heads=max(1, s["width"] // 512), head_dim=128,
-              rope_theta=5e5)
+              rope_theta=5e5, tie_word_embeddings=tied)
     rest = target - ModelArch(intermediate_size=0, **kw).num_parameters()
     return ModelArch(intermediate_size=max(256, rest // (kw["num_hidden_layers"] * 3 * s["width"]) // 256 * 256), **kw)
 
@@ -88,22 +106,25 @@ def measure(model, batch, prompt, n_prompts, iters=10):
                 decode_tok_s=round(batch / ms_step * 1e3), decode_ms=round(ms_step, 4), own_prompt_launches=launches)
 
 
-def run(sizes=("small", "base"), batch=64, prompt=1024, n_prompts=8):
+def run(sizes=("small", "base"), batch=64, prompt=1024, n_prompts=8, design="zorelorn"):
     from ..models.configuration import ModelArch
     from ..models.hf_io import build_model
 
     out = []
     for name in sizes:
-        s = SIZES[name]
-        arch = ModelArch.from_hf_dict(layered_config(**s))
-        n = arch.num_parameters()
-        flat = flat_config(s, n)
-        row = dict(size=name, layers=2 * s["pairs"], width=s["width"], batch=batch, prompt=f"{n_prompts}x{prompt}",
+        s = SIZES[design][name]
+        arch = ModelArch.from_hf_dict(layered_config(design, s))
+        depth = arch.num_hidden_layers
+        # the per-token table of a side input is looked up, not multiplied with: it does not count as size
+        n = arch.num_parameters() - VOCAB * depth * arch.side_dim
+        flat = flat_config(s, depth, n, arch.tie_word_embeddings)
+        row = dict(design=design, size=name, layers=depth, width=s["width"], batch=batch, prompt=f"{n_prompts}x{prompt}",
                    decode_context=prompt)
         for key, cfg in (("layered", arch), ("flat", flat)):
             torch.manual_seed(0)
             model = build_model(cfg, dtype=torch.bfloat16, device="cuda").eval().requires_grad_(False)
-            row[key] = dict(params_m=round(sum(p.numel() for p in model.parameters()) / 1e6), **measure(model, batch, prompt, n_prompts))
+            params = sum(p.numel() for p in model.parameters()) - (VOCAB * depth * arch.side_dim if key == "layered" else 0)
+            row[key] = dict(params_m=round(params / 1e6), **measure(model, batch, prompt, n_prompts))
             del model
             torch.cuda.empty_cache()
         row["prompt_ratio"] = round(row["layered"]["prompt_tok_s"] / row["flat"]["prompt_tok_s"], 3)
@@ -121,41 +142,134 @@ def peaks():
     return 6.65e12, 1.59e15
 
 
-@torch.no_grad()
-def kernel_table(size="base", batch=64, prompt=1024, n_prompts=8, iters=20):
-    """Time of every mixer kernel alone (cold L2) and the fraction of its roofline: the larger of bytes / measured copy
-    bandwidth and operations / measured bf16 GEMM throughput, over the time."""
-    from ..models.configuration import ModelArch
-    from ..models.decoder import SeqCtx
-    from ..models.hf_io import build_model
-    from ..ops import cuda as K
-    from ..ops import cuda_mixers as KM
-    from ..ops import mixers as mx
-    from ..rollout.engine import make_engine
+class KernelTimer:
+    """Times kernels alone (cold L2): median time and the fraction of the roofline, which is the larger of bytes / measured
+    copy bandwidth and operations / measured bf16 GEMM throughput."""
 
-    bw, fl = peaks()
-    s = dict(SIZES[size], pairs=1)
-    model = build_model(ModelArch.from_hf_dict(layered_config(**s)), dtype=torch.bfloat16, device="cuda").eval().requires_grad_(False)
-    eng = make_engine(model, max_num_seqs=batch, max_model_len=prompt + 64)
-    # larger than L2, and long enough that the host has launched everything of an iteration before the first event
-    flush = torch.empty(2 << 30, dtype=torch.uint8, device="cuda")
-    rows = []
+    def __init__(self, iters=20):
+        self.iters, self.rows = iters, []
+        self.bw, self.fl = peaks()
+        # larger than L2, and long enough that the host has launched everything of an iteration before the first event
+        self.flush = torch.empty(2 << 30, dtype=torch.uint8, device="cuda")
 
-    def row(name, fn, nbytes, flops=0.0):
+    def __call__(self, name, fn, nbytes, flops=0.0):
         for _ in range(3):
             fn()
         ev = []
-        for _ in range(iters):
-            flush.zero_()
+        for _ in range(self.iters):
+            self.flush.zero_()
             a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
             a.record()
             fn()
             b.record()
             ev.append((a, b))
         torch.cuda.synchronize()
-        us = sorted(a.elapsed_time(b) * 1e3 for a, b in ev)[iters // 2]
-        roof = max(nbytes / bw, flops / fl) * 1e6
-        rows.append(dict(kernel=name, us=round(us, 1), roof_us=round(roof, 2), frac=round(roof / us, 3)))
+        us = sorted(a.elapsed_time(b) * 1e3 for a, b in ev)[self.iters // 2]
+        roof = max(nbytes / self.bw, flops / self.fl) * 1e6
+        self.rows.append(dict(kernel=name, us=round(us, 1), roof_us=round(roof, 2), frac=round(roof / us, 3)))
+
+
+def kernel_table(size="base", batch=64, prompt=1024, n_prompts=8, iters=20, design="zorelorn"):
+    """Time of every mixer kernel alone beside the like kernels of the flat decoder."""
+    from ..models.configuration import ModelArch
+    from ..models.hf_io import build_model
+    from ..ops import cuda as K
+    from ..rollout.engine import make_engine
+
+    s = dict(SIZES[design][size], **(dict(pairs=1) if design == "zorelorn" else dict(quads=1)))
+    model = build_model(ModelArch.from_hf_dict(layered_config(design, s)), dtype=torch.bfloat16, device="cuda").eval().requires_grad_(False)
+    eng = make_engine(model, max_num_seqs=batch, max_model_len=prompt + 64)
+    row = KernelTimer(iters)
+    (zorelorn_kernels if design == "zorelorn" else povusun_kernels)(s, model, eng, batch, prompt, n_prompts, row)
+    flat_kernels(s, batch, prompt, n_prompts, row)
+    K.check_status()
+    return row.rows
+
+
+def paged_context(eng, prompt):
+    """Every slot at the given context, its pages spread over the cache."""
+    eng.seq_lens.fill_(prompt)
+    eng.block_table.copy_(torch.arange(eng.block_table.numel(), device=eng.dev).view_as(eng.block_table).remainder(eng.num_blocks))
+
+
+@torch.no_grad()
+def povusun_kernels(s, model, eng, batch, prompt, n_prompts, row):
+    from ..models.decoder import SeqCtx
+    from ..ops import cuda as K
+    from ..ops import cuda_mixers as KM
+    from ..ops import mixers as mx
+
+    at, rg, la = (model.layers[i].mixer for i in range(3))
+    T, W, dev, bf, B = n_prompts * prompt, s["width"], "cuda", torch.bfloat16, batch
+    ctx = SeqCtx.from_lengths([prompt] * n_prompts, dev)
+    h = torch.randn(T, W, device=dev, dtype=bf)
+    x, d, nrm = torch.randn(T, W, device=dev), torch.randn(T, W, device=dev), model.norm
+    pairs = n_prompts * prompt * (prompt + 1) / 2
+    row("prompt norm of output + residual + norm", lambda: KM.rms_residual(x, d, nrm.weight, nrm.weight, nrm.eps, bf), T * W * 14)
+    y = mx.linear(h, at.w_in)
+    temp = at.temperature.table(prompt, dev)
+    kv = at.kv_heads * (at.dim + at.vdim)
+    where = eng.slots[0].prompt_target(eng._page_writer(torch.arange(n_prompts, device=dev, dtype=torch.int32).repeat_interleave(prompt), ctx, None))
+    paged_context(eng, prompt)
+    row("prompt attention preparation + cache", lambda: KM.attn_prep(y, at, ctx.positions, temp, **where),
+        T * 2 * (2 * (at.heads + at.kv_heads) * at.dim + at.kv_heads * at.vdim + kv))
+    q, k, v, g = y.split(at.parts, 1)
+    row("prompt grouped attention (capped, gated)", lambda: KM.mixer_attn(q, k, v, heads=at.heads, kv_heads=at.kv_heads, scale=at.scale, cap=at.cap,
+                                                                          gate_logits=g, ctx=ctx),
+        T * 2 * (y.shape[1] + at.heads * at.vdim), 2 * pairs * at.heads * (at.dim + at.vdim))
+    row("prompt grouped attention without cap", lambda: KM.mixer_attn(q, k, v, heads=at.heads, kv_heads=at.kv_heads, scale=at.scale,
+                                                                      gate_logits=g, ctx=ctx),
+        T * 2 * (y.shape[1] + at.heads * at.vdim), 2 * pairs * at.heads * (at.dim + at.vdim))
+    del y, q, k, v, g
+    acc = mx.linear_f32(h, la.w_in[la.q_rows:])
+    lw = KM.latent_row(la.kv_rank, 0)[1]
+    lat = torch.zeros(T, lw, device=dev, dtype=bf)
+    row("prompt latent preparation", lambda: KM.latent_prep(acc, la, ctx.positions, None, lat=lat), T * (acc.shape[1] * 4 + lw * 2))
+    KM.latent_prep(acc, la, ctx.positions, None, lat=lat)
+    q, ukv = mx.linear(h, la.w_in[: la.q_rows]), mx.linear(lat[:, : la.kv_rank], la.ukv)
+    row("prompt latent attention", lambda: mx.latent_prompt_attention(q, ukv, lat, la, ctx, None),
+        (q.numel() + ukv.numel() + T * la.heads * la.vdim) * 2, 2 * pairs * la.heads * (la.dim + la.vdim))
+    del q, ukv, acc
+    yx = mx.linear(h, rg.w_in)
+    gy, gx = yx.chunk(2, 1)
+    C, wb = rg.width, rg.width // rg.blocks
+    row("prompt convolution", lambda: KM.conv_prompt(gx, rg, ctx), T * C * 4)
+    u = KM.conv_prompt(gx, rg, ctx)
+    row("prompt rglru (gates + scan + output)", lambda: KM.rglru_prompt_tc(u, gy, rg, ctx), T * C * 6 + rg.gates.numel() * 2, 4 * T * C * wb)
+    del yx, gy, gx, u
+    z = torch.randn(T, 2 * s["ff"], device=dev, dtype=bf)
+    mlp, side = model.layers[0].mlp, model.layers[0].side
+    row("prompt clamped unit", lambda: KM.clamped_glu(z, *mlp.glu), z.numel() * 3)
+    del z
+    zs, ids = torch.randn(T, side.dim, device=dev, dtype=bf), torch.randint(0, VOCAB, (T,), device=dev)
+    row("prompt side gate", lambda: KM.side_gate(zs, ids, model.side_embed, 0), T * side.dim * 6)
+
+    a, r, l = eng.slots[0], eng.slots[1], eng.slots[2]
+    hb, xb, db = torch.randn(B, W, device=dev, dtype=bf), torch.randn(B, W, device=dev), torch.randn(B, W, device=dev)
+    row("decode norm of output + residual + norm", lambda: KM.rms_residual(xb, db, nrm.weight, nrm.weight, nrm.eps, bf, clear=True, out=hb), B * W * 18)
+    row("decode gemm input attention", lambda: K.decode_gemm(hb, at.w_in, y32=a.acc_in), at.w_in.numel() * 2)
+    row("decode attention preparation + cache", a.prepare, a.acc_in.numel() * 10)
+    row("decode grouped attention (capped, gated)", a.attend,
+        B * (prompt + 1) * kv * 2 + (a.q.numel() + 2 * a.o.numel()) * 2, 2 * B * (prompt + 1) * at.heads * (at.dim + at.vdim))
+    row("decode latent preparation", lambda: KM.latent_prep(l.acc_prep, la, eng.seq_lens, None, clear=True, cache=l.cache,
+                                                            block_table=eng.block_table, block_size=eng.block_size), B * la.kv_rank * 10)
+    row("decode absorb", l.absorb, la.uk.numel() * 2 + l.acc_q.numel() * 8 + l.q_lat.numel() * 2, 2 * B * la.heads * la.dim * la.kv_rank)
+    row("decode latent attention", l.attend, B * (prompt + 1) * lw * 2 + (l.q_lat.numel() + l.o_lat.numel()) * 2,
+        2 * B * (prompt + 1) * la.heads * (lw + la.kv_rank))
+    row("decode expand", l.expand, la.uv.numel() * 2 + (l.o_lat.numel() + l.o.numel()) * 2, 2 * B * la.heads * la.vdim * la.kv_rank)
+    row("decode convolution", r.convolve, B * C * (8 + 8 * (rg.taps - 1) + 2))
+    row("decode rglru (gates + step + output)", r.recur, B * C * (2 + 8 + 8 + 2) + rg.gates.numel() * 2, 4 * B * C * wb)
+    row("decode gate/up + clamped unit", lambda: eng.mlp_act(hb, mlp), mlp.gate_up.numel() * 2)
+    row("decode side gate gemm", lambda: eng.gemm(hb, side.gate, eng.sums("side", side.dim)), side.gate.numel() * 2)
+    row("decode side gate", lambda: KM.side_gate(eng.sums("side", side.dim), eng.next_input, model.side_embed, 0, clear=True), B * side.dim * 12)
+
+
+@torch.no_grad()
+def zorelorn_kernels(s, model, eng, batch, prompt, n_prompts, row):
+    from ..models.decoder import SeqCtx
+    from ..ops import cuda as K
+    from ..ops import cuda_mixers as KM
+    from ..ops import mixers as mx
 
     la, ml = model.layers[0].mixer, model.layers[1].mixer
     T, W, dev, bf = n_prompts * prompt, s["width"], "cuda", torch.bfloat16
@@ -194,8 +308,7 @@ def kernel_table(size="base", batch=64, prompt=1024, n_prompts=8, iters=20):
     row("prompt gelu", lambda: KM.gelu_erf(up), up.numel() * 4)
     del up, y, q, kv, o32
 
-    eng.seq_lens.fill_(prompt)
-    eng.block_table.copy_(torch.arange(eng.block_table.numel(), device=dev).view_as(eng.block_table).remainder(eng.num_blocks))
+    paged_context(eng, prompt)
     a, r, B = eng.slots[0], eng.slots[1], batch
     hb = torch.randn(B, W, device=dev, dtype=bf)
     xb, db = torch.randn(B, W, device=dev), torch.randn(B, W, device=dev)
@@ -218,12 +331,9 @@ def kernel_table(size="base", batch=64, prompt=1024, n_prompts=8, iters=20):
     row("decode mlstm_out", lambda: KM.mlstm_out(r.o32, r.acc_in[:, qkv:], ml, r.y, clear=r.acc_in), r.acc_in.numel() * 4 + r.o32.numel() * 8)
     mlp = model.layers[0].mlp
     row("decode up + gelu", lambda: eng.mlp_act(hb, mlp), mlp.up.numel() * 2)
-    K.check_status()
-    rows += flat_kernels(s, batch, prompt, n_prompts, row, rows)
-    return rows
 
 
-def flat_kernels(s, batch, prompt, n_prompts, row, rows):
+def flat_kernels(s, batch, prompt, n_prompts, row):
     """The like kernels of the flat decoder, timed the same way."""
     from ..ops import cuda as K
 
@@ -258,12 +368,11 @@ def flat_kernels(s, batch, prompt, n_prompts, row, rows):
     gw = torch.randn(2 * s["ff"], W, device=dev, dtype=bf)
     act = torch.empty(batch, s["ff"], device=dev, dtype=bf)
     row("flat: decode gate/up + swiglu", lambda: K.decode_gemm(x, gw, out=act, swiglu=True), gw.numel() * 2)
-    K.check_status()
-    return []
 
 
 def main():
     ap = argparse.ArgumentParser()
+    ap.add_argument("--design", choices=sorted(SIZES), default="zorelorn")
     ap.add_argument("--sizes", default="small,base")
     ap.add_argument("--batch", type=int, default=64)
     ap.add_argument("--prompt", type=int, default=1024)
@@ -271,10 +380,10 @@ def main():
     ap.add_argument("--kernels", action="store_true")
     a = ap.parse_args()
     if a.kernels:
-        for r in kernel_table(a.sizes.split(",")[-1], a.batch, a.prompt, a.prompts):
+        for r in kernel_table(a.sizes.split(",")[-1], a.batch, a.prompt, a.prompts, design=a.design):
             print(json.dumps(r))
         return
-    for r in run(a.sizes.split(","), a.batch, a.prompt, a.prompts):
+    for r in run(a.sizes.split(","), a.batch, a.prompt, a.prompts, a.design):
         print(json.dumps(r))
 
 

@@ -325,16 +325,15 @@ fa_fwd_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant_
           tmem_st_32x16(ts + (c >> 1), w);
         }
         tmem_st_wait();
+        // P.V(last) completes phase `last` of o_full, possibly before this thread looks: see phase last - 1 first
+        if (j > 0 && j == n_kv - 1)
+          ok = __all_sync(0xffffffffu, mbar_wait(o_full, (uint32_t)((j - 1) & 1), abort_flag, p.status, 1094));
         tc_fence_before();
         mbar_arrive(&p_full[s]);
         l_run += sum;
       }
       if (ok) {
-        // the last P.V product: wait for the one before it first, so that the parity of the last wait is unambiguous
-        const int last = n_kv - 1;
-        if (last >= 1)
-          ok = __all_sync(0xffffffffu, mbar_wait(o_full, (uint32_t)((last - 1) & 1), abort_flag, p.status, 1094));
-        if (ok) ok = __all_sync(0xffffffffu, mbar_wait(o_full, (uint32_t)(last & 1), abort_flag, p.status, 1095));
+        ok = __all_sync(0xffffffffu, mbar_wait(o_full, (uint32_t)((n_kv - 1) & 1), abort_flag, p.status, 1095));
         if (ok) {
           tc_fence_after();
           const float inv = l_run > 0.f ? 1.f / l_run : 0.f;

@@ -10,10 +10,14 @@
 //     the 16-column steps that hold data.  rot = 0: no such part;
 //   * groups of heads / kv_heads query heads read one key / value head;
 //   * sizes are launch parameters: dim, rot, vdim any multiples of 8 (vdim <= 256) that leave room for one stage;
-//   * probabilities keep 32-bit precision into P.V: each is split into two bf16 (value and remainder), both halves of
-//     the S buffer are reused for them (64 columns each), and P.V accumulates both products;
-//   * scores may be capped, cap tanh(s / cap) (CAP): a series near zero, where scores of normed queries and keys lie, so
-//     that the special-function units are left to the exponentials;
+//   * probabilities keep 32-bit precision into P.V: each is split into two bf16 (value and remainder) that replace the scores
+//     in TMEM, 32 keys at a time (16 columns of values, 16 of remainders), and P.V accumulates both products;
+//   * scores may be capped, cap tanh(s / cap) (CAP): an odd polynomial (the Taylor series of tanh, its length by the largest
+//     score of the tile) near zero, where scores of normed queries and keys lie, so that the special-function units are left
+//     to the exponentials; exp2 and a division further out;
+//   * NB = 1 when two CTAs fit an SM (vdim <= 128, at most 6 boxes of Q, K and V together): one S buffer of 128 columns and O
+//     in 256 columns of TMEM; the softmax of one CTA runs beside the products of the other.  NB = 2 otherwise: one CTA, S
+//     double-buffered;
 //   * the softmax denominator may contain exp(sink[head]);
 //   * the output may be multiplied by a gate: one fp32 factor per token and head, or the sigmoid of bf16 logits per
 //     element;
@@ -35,6 +39,8 @@ struct MixerAttnTc {
   int k_stages, v_stages;
   float scale_log2;    // CAP: 1 (capped scores are in log2 units already)
   float cap_in, cap_out;  // CAP: scale / cap, cap log2(e)
+  float poly[6];          // CAP: cap_out tanh(cap_in v) = v (poly[0] + poly[1] v^2 + ...)
+  float near7, near11;    // CAP: |v| up to which the polynomial through v^7, v^11 serves
   const float* sink;   // [heads] or null
   int gate_mode;
   const void* gate;    // GATE_HEAD: fp32 [T, heads]; GATE_LOGITS: bf16 [T, gate_ld >= heads vdim]
@@ -52,8 +58,56 @@ __device__ __forceinline__ bool la_find_tile(const int* cu, int n_seq, int slot,
   return false;
 }
 
-template <bool CAP>
-__global__ void __launch_bounds__(LA_THREADS, 1)
+// cap_out tanh(cap_in v); LEVEL 0, 1: the polynomial through v^7, v^11, 2: any v
+template <int LEVEL>
+__device__ __forceinline__ float la_capped(const MixerAttnTc& p, float v) {
+  if (LEVEL == 2) return p.cap_out * tanh_exp(p.cap_in * v);
+  const float z = v * v;
+  float t = p.poly[3];
+  if (LEVEL == 1) t = fmaf(z, fmaf(z, p.poly[5], p.poly[4]), t);
+  t = fmaf(z, t, p.poly[2]);
+  t = fmaf(z, t, p.poly[1]);
+  return v * fmaf(z, t, p.poly[0]);
+}
+
+// Second pass over a row of scores: probabilities, as value and remainder, in place.  LEVEL -1: no cap.  Returns their sum.
+template <int LEVEL>
+__device__ __forceinline__ float la_probs(const MixerAttnTc& p, uint32_t ts, float neg_m, bool full, int key0, int k_min, int k_max) {
+  float sum = 0.f;
+#pragma unroll
+  for (int c = 0; c < 4; ++c) {
+    float v[32];
+    tmem_ld_32x32(ts + 32 * c, v);
+    tmem_ld_wait();
+#pragma unroll
+    for (int i = 0; i < 32; ++i) {
+      if (LEVEL < 0) v[i] = fast_exp2(fmaf(v[i], p.scale_log2, neg_m));
+      else v[i] = fast_exp2(la_capped<LEVEL < 0 ? 0 : LEVEL>(p, v[i]) + neg_m);
+    }
+    if (!full) {
+#pragma unroll
+      for (int i = 0; i < 32; ++i) {
+        const int key = key0 + 32 * c + i;
+        if (key < k_min || key > k_max) v[i] = 0.f;
+      }
+    }
+    uint32_t a[16], b[16];
+#pragma unroll
+    for (int i = 0; i < 16; ++i) {
+      sum += v[2 * i] + v[2 * i + 1];
+      a[i] = pack_bf16(v[2 * i], v[2 * i + 1]);
+      const float2 f = unpack_bf16(a[i]);
+      b[i] = pack_bf16(v[2 * i] - f.x, v[2 * i + 1] - f.y);
+    }
+    tmem_st_32x16(ts + 32 * c, a);
+    tmem_st_32x16(ts + 32 * c + 16, b);
+  }
+  tmem_st_wait();
+  return sum;
+}
+
+template <bool CAP, int NB>
+__global__ void __launch_bounds__(LA_THREADS, 3 - NB)
 mixer_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_constant__ CUtensorMap tm_qr,
                       const __grid_constant__ CUtensorMap tm_kn, const __grid_constant__ CUtensorMap tm_kr,
                       const __grid_constant__ CUtensorMap tm_v, const MixerAttnTc p) {
@@ -106,7 +160,7 @@ mixer_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_con
     tma_prefetch_desc(&tm_v);
   }
   if (warp == 1) {
-    tmem_alloc(tmem_slot, 512);
+    tmem_alloc(tmem_slot, NB * 256);
     tmem_relinquish();
     tc_fence_before();
   }
@@ -132,13 +186,14 @@ mixer_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_con
       };
       bool ok = load_k(0);
       for (int j = 0; j < n_kv && ok; ++j) {
-        if (j + 1 < n_kv) ok = load_k(j + 1);
+        if (NB == 2 && j + 1 < n_kv) ok = load_k(j + 1);
         if (!ok) break;
         const int s = j % p.v_stages;
         if (!mbar_wait(&v_empty[s], (uint32_t)(((j / p.v_stages) & 1) ^ 1), abort_flag, p.status, 1205 + s)) break;
         uint8_t* vs = v_s + (size_t)s * v_bytes;
         mbar_expect_tx(&v_full[s], v_bytes);
         for (int i = 0; i < p.nv; ++i) tma_load_3d(vs + i * LA_BOX, &tm_v, &v_full[s], 64 * i, hk, beg + (lo + j) * LA_BN);
+        if (NB == 1 && j + 1 < n_kv) ok = load_k(j + 1);  // one stage: free only after S(j)
       }
     }
     __syncwarp();
@@ -151,8 +206,8 @@ mixer_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_con
       const uint64_t v_d = umma_desc_mnmajor_sw128(smem_u32(v_s), LA_BOX);
       bool ok = mbar_wait(q_full, 0, abort_flag, p.status, 1210);
       auto issue_s = [&](int j) {
-        const int s = j & 1, kst = j % p.k_stages;
-        // buffer s is free: its P.V product (tile j - 2) was issued before this call
+        const int s = j % NB, kst = j % p.k_stages;
+        // buffer s is free: its P.V product (tile j - NB) was issued before this call
         if (!mbar_wait(&k_full[kst], (uint32_t)((j / p.k_stages) & 1), abort_flag, p.status, 1220 + kst)) return false;
         tc_fence_after();
         const uint64_t k_t = desc_at(k_d, (uint32_t)kst * k_bytes);
@@ -172,21 +227,22 @@ mixer_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_con
       };
       if (ok) ok = issue_s(0);
       for (int j = 0; j < n_kv && ok; ++j) {
-        if (j + 1 < n_kv) ok = issue_s(j + 1);
+        if (NB == 2 && j + 1 < n_kv) ok = issue_s(j + 1);
         if (!ok) break;
-        const int sb = j & 1, s = j % p.v_stages;
-        if (!mbar_wait(&p_full[sb], (uint32_t)((j >> 1) & 1), abort_flag, p.status, 1240 + sb)) break;
+        const int sb = j % NB, s = j % p.v_stages;
+        if (!mbar_wait(&p_full[sb], (uint32_t)((j / NB) & 1), abort_flag, p.status, 1240 + sb)) break;
         if (!mbar_wait(&v_full[s], (uint32_t)((j / p.v_stages) & 1), abort_flag, p.status, 1250 + s)) break;
         tc_fence_after();
         const uint64_t v_t = desc_at(v_d, (uint32_t)s * v_bytes);
-        // the S buffer holds P as bf16 pairs: leading parts in its first 64 columns, remainders in the other 64
+        // 32 keys are 16 columns of values and 16 of remainders, 16 keys an MMA step
         for (int half = 0; half < 2; ++half)
 #pragma unroll
           for (int kk = 0; kk < LA_BN / 16; ++kk)
-            umma_bf16_ts(tmem_base + 256, tmem_base + (uint32_t)(sb * LA_BN + half * 64 + kk * 8),
+            umma_bf16_ts(tmem_base + NB * 128, tmem_base + (uint32_t)(sb * LA_BN + (kk >> 1) * 32 + half * 16 + (kk & 1) * 8),
                          desc_at(v_t, kk * 2048), idesc_o, (j | half | kk) != 0);
         umma_commit(o_full);
         umma_commit(&v_empty[s]);
+        if (NB == 1 && j + 1 < n_kv) ok = issue_s(j + 1);  // takes the place of the probabilities just consumed
       }
     }
     __syncwarp();
@@ -199,58 +255,46 @@ mixer_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_con
     const bool row_ok = q_pos < len;
     const int k_max = row_ok ? q_pos : -1;
     const int k_min = p.window > 0 ? max(0, q_pos - p.window + 1) : 0;
-    const uint32_t to = tmem_base + lane_off + 256;
+    const uint32_t to = tmem_base + lane_off + NB * 128;
     float m_ref = -INFINITY, l_run = 0.f;
     bool ok = true;
     for (int j = 0; j < n_kv && ok; ++j) {
-      const int s = j & 1;
+      const int s = j % NB;
       const int key0 = (lo + j) * LA_BN;
       const bool full = q_first + LA_BM <= len && key0 + LA_BN - 1 <= q_first &&
                         (p.window <= 0 || key0 >= q_first + LA_BM - p.window);
-      ok = __all_sync(0xffffffffu, mbar_wait(&s_full[s], (uint32_t)((j >> 1) & 1), abort_flag, p.status, 1270 + s));
+      ok = __all_sync(0xffffffffu, mbar_wait(&s_full[s], (uint32_t)((j / NB) & 1), abort_flag, p.status, 1270 + s));
       if (!ok) break;
       tc_fence_after();
       const uint32_t ts = tmem_base + lane_off + (uint32_t)s * LA_BN;
-      float v[4][32];
+      // first pass: the row's largest score (and with a cap the largest magnitude)
+      float mx = -INFINITY, mn = INFINITY;
 #pragma unroll
-      for (int c = 0; c < 4; ++c) tmem_ld_32x32(ts + 32 * c, v[c]);
-      tmem_ld_wait();
+      for (int c = 0; c < 4; c += 2) {
+        float v[2][32];
+        tmem_ld_32x32(ts + 32 * c, v[0]);
+        tmem_ld_32x32(ts + 32 * c + 32, v[1]);
+        tmem_ld_wait();
+#pragma unroll
+        for (int h2 = 0; h2 < 2; ++h2)
+#pragma unroll
+          for (int i = 0; i < 32; ++i) {
+            const int key = key0 + 32 * (c + h2) + i;
+            if (CAP) mn = fminf(mn, v[h2][i]);
+            if (full) mx = fmaxf(mx, v[h2][i]);
+            else {
+              if (CAP) mn = fminf(mn, -v[h2][i]);  // masked scores count for the magnitude
+              if (key >= k_min && key <= k_max) mx = fmaxf(mx, v[h2][i]);
+            }
+          }
+      }
+      int level = -1;
+      float m_tile = mx * p.scale_log2;
       if (CAP) {
-        float top = 0.f;
-#pragma unroll
-        for (int c = 0; c < 4; ++c)
-#pragma unroll
-          for (int i = 0; i < 32; ++i) {
-            v[c][i] *= p.cap_in;
-            top = fmaxf(top, fabsf(v[c][i]));
-          }
-        if (__any_sync(0xffffffffu, top > CAP_SERIES)) {
-#pragma unroll
-          for (int c = 0; c < 4; ++c)
-#pragma unroll
-            for (int i = 0; i < 32; ++i) v[c][i] = p.cap_out * tanh_exp(v[c][i]);
-        } else {
-#pragma unroll
-          for (int c = 0; c < 4; ++c)
-#pragma unroll
-            for (int i = 0; i < 32; ++i) v[c][i] = p.cap_out * tanh_series(v[c][i]);
-        }
+        const float top = fmaxf(mx, -mn);
+        level = !__any_sync(0xffffffffu, top > p.near7) ? 0 : !__any_sync(0xffffffffu, top > p.near11) ? 1 : 2;
+        m_tile = mx == -INFINITY ? mx : level == 0 ? la_capped<0>(p, mx) : level == 1 ? la_capped<1>(p, mx) : la_capped<2>(p, mx);
       }
-      if (!full) {
-#pragma unroll
-        for (int c = 0; c < 4; ++c)
-#pragma unroll
-          for (int i = 0; i < 32; ++i) {
-            const int key = key0 + 32 * c + i;
-            if (key < k_min || key > k_max) v[c][i] = -INFINITY;
-          }
-      }
-      float mx = -INFINITY;
-#pragma unroll
-      for (int c = 0; c < 4; ++c)
-#pragma unroll
-        for (int i = 0; i < 32; ++i) mx = fmaxf(mx, v[c][i]);
-      const float m_tile = mx * p.scale_log2;
       float alpha = 1.f;
       bool moved = false;
       if (m_ref == -INFINITY) {
@@ -277,32 +321,22 @@ mixer_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_con
       }
       l_run *= alpha;
       const float neg_m = m_ref == -INFINITY ? 0.f : -m_ref;
-      float sum = 0.f;
-#pragma unroll
-      for (int c = 0; c < 4; ++c) {
-        uint32_t a[16], b[16];
-#pragma unroll
-        for (int i = 0; i < 16; ++i) {
-          const float p0 = fast_exp2(fmaf(v[c][2 * i], p.scale_log2, neg_m));  // masked scores: exp2(-inf) = 0
-          const float p1 = fast_exp2(fmaf(v[c][2 * i + 1], p.scale_log2, neg_m));
-          sum += p0 + p1;
-          a[i] = pack_bf16(p0, p1);
-          const float2 f = unpack_bf16(a[i]);
-          b[i] = pack_bf16(p0 - f.x, p1 - f.y);
-        }
-        tmem_st_32x16(ts + 16 * c, a);
-        tmem_st_32x16(ts + 64 + 16 * c, b);
-      }
-      tmem_st_wait();
+      float sum;
+      if (!CAP) sum = la_probs<-1>(p, ts, neg_m, full, key0, k_min, k_max);
+      else if (level == 0) sum = la_probs<0>(p, ts, neg_m, full, key0, k_min, k_max);
+      else if (level == 1) sum = la_probs<1>(p, ts, neg_m, full, key0, k_min, k_max);
+      else sum = la_probs<2>(p, ts, neg_m, full, key0, k_min, k_max);
+      // P.V(last) completes phase `last` of o_full, and may do so before this thread looks: phase last - 1 has to be seen
+      // first.  (With one S buffer the last S was issued after P.V(last - 1), so s_full has shown it.)
+      if (NB == 2 && j > 0 && j == n_kv - 1)
+        ok = __all_sync(0xffffffffu, mbar_wait(o_full, (uint32_t)((j - 1) & 1), abort_flag, p.status, 1294));
       tc_fence_before();
       mbar_arrive(&p_full[s]);
       l_run += sum;
     }
     if (ok) {
       const int last = n_kv - 1;
-      if (last >= 1)
-        ok = __all_sync(0xffffffffu, mbar_wait(o_full, (uint32_t)((last - 1) & 1), abort_flag, p.status, 1294));
-      if (ok) ok = __all_sync(0xffffffffu, mbar_wait(o_full, (uint32_t)(last & 1), abort_flag, p.status, 1295));
+      ok = __all_sync(0xffffffffu, mbar_wait(o_full, (uint32_t)(last & 1), abort_flag, p.status, 1295));
       if (ok) {
         tc_fence_after();
         float f = 0.f;
@@ -318,30 +352,36 @@ mixer_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_con
           dst = p.out + th * p.vdim;
         }
 #pragma unroll 1
-        for (int c = 0; c < p.vdim; c += 16) {
-          float o[16];
-          tmem_ld_32x16(to + c, o);
+        for (int c = 0; c < p.vdim; c += 32) {
+          uint4 g[4];
+          if (gl != nullptr) {
+#pragma unroll
+            for (int i = 0; i < 4; ++i)
+              if (c + 8 * i < p.vdim) g[i] = *reinterpret_cast<const uint4*>(gl + c + 8 * i);
+          }
+          float o[2][16];
+          tmem_ld_32x16(to + c, o[0]);
+          tmem_ld_32x16(to + (c + 16 < p.vdim ? c + 16 : c), o[1]);
           tmem_ld_wait();
           if (row_ok) {
 #pragma unroll
-            for (int i = 0; i < 16; i += 8)
-              if (c + i < p.vdim) {
+            for (int i = 0; i < 4; ++i) {
+              if (c + 8 * i >= p.vdim) break;
+              float* x = &o[i >> 1][8 * (i & 1)];
 #pragma unroll
-                for (int q = 0; q < 8; ++q) o[i + q] *= f;
-                if (gl != nullptr) {
-                  const uint4 g = *reinterpret_cast<const uint4*>(gl + c + i);
-                  const uint32_t w[4] = {g.x, g.y, g.z, g.w};
+              for (int q = 0; q < 8; ++q) x[q] *= f;
+              if (gl != nullptr) {
+                const uint32_t w[4] = {g[i].x, g[i].y, g[i].z, g[i].w};
 #pragma unroll
-                  for (int q = 0; q < 4; ++q) {
-                    const float2 z = unpack_bf16(w[q]);
-                    o[i + 2 * q] *= fast_sigmoid(z.x);
-                    o[i + 2 * q + 1] *= fast_sigmoid(z.y);
-                  }
+                for (int q = 0; q < 4; ++q) {
+                  const float2 z = unpack_bf16(w[q]);
+                  x[2 * q] *= fast_sigmoid(z.x);
+                  x[2 * q + 1] *= fast_sigmoid(z.y);
                 }
-                *reinterpret_cast<uint4*>(dst + c + i) =
-                    make_uint4(pack_bf16(o[i], o[i + 1]), pack_bf16(o[i + 2], o[i + 3]), pack_bf16(o[i + 4], o[i + 5]),
-                               pack_bf16(o[i + 6], o[i + 7]));
               }
+              *reinterpret_cast<uint4*>(dst + c + 8 * i) =
+                  make_uint4(pack_bf16(x[0], x[1]), pack_bf16(x[2], x[3]), pack_bf16(x[4], x[5]), pack_bf16(x[6], x[7]));
+            }
           }
         }
         tc_fence_before();
@@ -356,7 +396,7 @@ mixer_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_con
   }
   if (warp == 1) {
     tc_fence_after();
-    tmem_dealloc(tmem_base, 512);
+    tmem_dealloc(tmem_base, NB * 256);
   }
 }
 
@@ -377,6 +417,9 @@ bool la_stages(int nk, int nv, int& ks, int& vs) {
 }
 
 int la_boxes(int n) { return (n + 63) / 64; }
+
+// Two CTAs per SM: 227 KB of shared memory in halves, each with the kilobyte the system takes.
+bool la_pair(int nk, int nv, int vdim) { return vdim <= 128 && la_smem(nk, nv, 1, 1) <= 112 * 1024; }
 
 }  // namespace
 
@@ -401,10 +444,19 @@ TRLB_API int trlb_mixer_attn_tc(const void* q, long long q_ld, const void* k, lo
   MixerAttnTc p = {};
   p.cu = cu; p.n_seq = n_seq; p.heads = heads; p.group = heads / kv_heads; p.dim = dim; p.rot = rot; p.vdim = vdim; p.window = window;
   p.nn = la_boxes(dim); p.nr = la_boxes(rot); p.nv = la_boxes(vdim);
-  la_stages(p.nn + p.nr, p.nv, p.k_stages, p.v_stages);
+  const bool pair = la_pair(p.nn + p.nr, p.nv, vdim);
+  if (pair) p.k_stages = p.v_stages = 1;
+  else la_stages(p.nn + p.nr, p.nv, p.k_stages, p.v_stages);
   p.scale_log2 = cap > 0.f ? 1.f : scale * 1.4426950408889634f;
   p.cap_in = cap > 0.f ? scale / cap : 0.f;
   p.cap_out = cap * 1.4426950408889634f;
+  if (cap > 0.f) {
+    const double t[6] = {1.0, -1.0 / 3, 2.0 / 15, -17.0 / 315, 62.0 / 2835, -1382.0 / 155925}, in = (double)scale / cap;
+    double f = (double)cap * 1.4426950408889634 * in;
+    for (int i = 0; i < 6; ++i, f *= in * in) p.poly[i] = (float)(t[i] * f);
+    p.near7 = (float)(0.12 / in);   // the first term left out is below 1e-9 of tanh
+    p.near11 = (float)(0.35 / in);  // below 2e-8
+  }
   p.sink = sink; p.gate_mode = gate_mode; p.gate = gate; p.gate_ld = gate_ld; p.out = (__nv_bfloat16*)out; p.status = status;
   const __nv_bfloat16* qb = (const __nv_bfloat16*)q;
   const int dq = dim + rot;
@@ -419,16 +471,17 @@ TRLB_API int trlb_mixer_attn_tc(const void* q, long long q_ld, const void* k, lo
     if (make_tmap_3d_bf16(&tqr, qb + dim, rot, heads, T, dq, (uint64_t)q_ld, 64, 1, 128)) return -212;
     if (trlb_host::make_tmap_2d_bf16(&tkr, krot, T, rot, (uint64_t)krot_ld, 128, 64)) return -214;
   }
+  using Kern = void (*)(const CUtensorMap, const CUtensorMap, const CUtensorMap, const CUtensorMap, const CUtensorMap, const MixerAttnTc);
+  static const Kern kerns[4] = {mixer_attn_tc_kernel<false, 1>, mixer_attn_tc_kernel<true, 1>, mixer_attn_tc_kernel<false, 2>,
+                                mixer_attn_tc_kernel<true, 2>};
   static bool attr_set = false;
   if (!attr_set) {
-    if (cudaFuncSetAttribute(mixer_attn_tc_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024) != cudaSuccess ||
-        cudaFuncSetAttribute(mixer_attn_tc_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024) != cudaSuccess)
-      return -216;
+    for (Kern k : kerns)
+      if (cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024) != cudaSuccess) return -216;
     attr_set = true;
   }
   const dim3 grid((T + LA_BM - 1) / LA_BM + n_seq, heads);
   const size_t smem = la_smem(p.nn + p.nr, p.nv, p.k_stages, p.v_stages);
-  if (cap > 0.f) mixer_attn_tc_kernel<true><<<grid, LA_THREADS, smem, st>>>(tqn, tqr, tkn, tkr, tv, p);
-  else mixer_attn_tc_kernel<false><<<grid, LA_THREADS, smem, st>>>(tqn, tqr, tkn, tkr, tv, p);
+  kerns[(pair ? 0 : 2) + (cap > 0.f)]<<<grid, LA_THREADS, smem, st>>>(tqn, tqr, tkn, tkr, tv, p);
   return (int)cudaGetLastError();
 }

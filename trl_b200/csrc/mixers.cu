@@ -204,19 +204,25 @@ clamped_glu_kernel(const T* __restrict__ z, T* __restrict__ out, long long total
 }
 
 // Side input of a layer: out[row] = gelu_tanh(z[row]) * table[ids[row], off : off + n].  Z: dtype of z; `clear` zeroes it.
-template <typename T, typename Z>
-__global__ void __launch_bounds__(128)
+template <typename T, typename Z, int VEC>
+__global__ void __launch_bounds__(256)
 side_gate_kernel(Z* __restrict__ z, const long long* __restrict__ ids, const T* __restrict__ table, long long table_ld, int off,
-                 int n, int V, int clear, T* __restrict__ out) {
+                 int n, long long total, int V, int clear, T* __restrict__ out) {
   pdl_launch_dependents();
   pdl_wait();
-  const size_t row = blockIdx.x;
-  const long long id = ids[row];
-  const bool ok = id >= 0 && id < V;
-  for (int j = threadIdx.x; j < n; j += blockDim.x) {
-    const float e = ok ? to_f(table[(size_t)id * table_ld + off + j]) : 0.f;
-    out[row * n + j] = from_f<T>(gelu_tanh_t<T>(to_f(z[row * n + j])) * e);
-    if (clear) z[row * n + j] = from_f<Z>(0.f);
+  const int per = n / VEC;
+  for (long long v = blockIdx.x * (long long)blockDim.x + threadIdx.x; v < total; v += (long long)gridDim.x * blockDim.x) {
+    const long long row = v / per, id = ids[row], at = v * VEC;
+    const bool ok = id >= 0 && id < V;
+    const T* e = table + (size_t)(ok ? id : 0) * table_ld + off + (int)(v % per) * VEC;
+    if (VEC == 4) {
+      const float4 a = load4(z + at), b = ok ? load4(e) : make_float4(0.f, 0.f, 0.f, 0.f);
+      store4(out + at, make_float4(gelu_tanh_t<T>(a.x) * b.x, gelu_tanh_t<T>(a.y) * b.y, gelu_tanh_t<T>(a.z) * b.z, gelu_tanh_t<T>(a.w) * b.w));
+      if (clear) store4(z + at, make_float4(0.f, 0.f, 0.f, 0.f));
+    } else {
+      out[at] = from_f<T>(gelu_tanh_t<T>(to_f(z[at])) * (ok ? to_f(*e) : 0.f));
+      if (clear) z[at] = from_f<Z>(0.f);
+    }
   }
 }
 
@@ -774,10 +780,12 @@ TRLB_API int trlb_clamped_glu(const void* z, void* out, int rows, int n, float l
 TRLB_API int trlb_side_gate(void* z, int z_f32, const long long* ids, const void* table, long long table_ld, int off, int rows,
                             int n, int V, int clear, void* out, int is_bf16, cudaStream_t st) {
   if (rows <= 0 || n <= 0) return 0;
-  const dim3 grid(rows), blk(n >= 128 ? 128 : (n + 31) / 32 * 32);
-#define GO(TT, ZZ) (int)trlb_host::launch_kernel(side_gate_kernel<TT, ZZ>, grid, blk, 0, st, PDL, (ZZ*)z, ids, (const TT*)table, table_ld, off, n, V, clear, (TT*)out)
-  if (is_bf16) return z_f32 ? GO(bf16, float) : GO(bf16, bf16);
-  return GO(float, float);
+  const bool v4 = ((n | off | (int)(table_ld & 3)) & 3) == 0 && (reinterpret_cast<uintptr_t>(table) & 15) == 0;
+  const long long total = (long long)rows * n / (v4 ? 4 : 1);
+#define GO(TT, ZZ, VV) (int)trlb_host::launch_kernel(side_gate_kernel<TT, ZZ, VV>, dim3(grid_for(total, 256)), dim3(256), 0, st, PDL, (ZZ*)z, ids, \
+                                                     (const TT*)table, table_ld, off, n, total, V, clear, (TT*)out)
+  if (is_bf16) return z_f32 ? (v4 ? GO(bf16, float, 4) : GO(bf16, float, 1)) : (v4 ? GO(bf16, bf16, 4) : GO(bf16, bf16, 1));
+  return v4 ? GO(float, float, 4) : GO(float, float, 1);
 #undef GO
 }
 
@@ -797,9 +805,11 @@ TRLB_API int trlb_latent_prep(float* acc, long long ld, int rows, int q_rank, in
   if ((rot & 1) || kr_off < kv_rank || lat_w < kr_off + rot || (cache != nullptr && block_table == nullptr)) return -200;
   LatentPrep p = {acc, ld, q_rank, kv_rank, rot, heads, clear, q_norm, kv_norm, eps, positions, tok_slot,
                   (const float2*)table, table_len, gate, kr_off, lat_w, cache ? block_table : nullptr, max_blocks, block_size};
+  const int widest = q_rank > kv_rank ? q_rank : kv_rank;
+  const dim3 blk(widest > 512 ? 256 : widest > 256 ? 128 : 64);
   if (is_bf16)
-    return (int)trlb_host::launch_kernel(latent_prep_kernel<bf16>, dim3(rows), dim3(256), 0, st, PDL, p, (bf16*)cq, (bf16*)lat, (bf16*)cache);
-  return (int)trlb_host::launch_kernel(latent_prep_kernel<float>, dim3(rows), dim3(256), 0, st, PDL, p, (float*)cq, (float*)lat, (float*)cache);
+    return (int)trlb_host::launch_kernel(latent_prep_kernel<bf16>, dim3(rows), blk, 0, st, PDL, p, (bf16*)cq, (bf16*)lat, (bf16*)cache);
+  return (int)trlb_host::launch_kernel(latent_prep_kernel<float>, dim3(rows), blk, 0, st, PDL, p, (float*)cq, (float*)lat, (float*)cache);
 }
 
 TRLB_API int trlb_rotate_q(void* q, int rows, int heads, int dim, int rot, const int* positions, const float* table,

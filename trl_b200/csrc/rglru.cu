@@ -5,6 +5,8 @@
 //     u_t = conv(x)_t,   log a_t = -decay r_t softplus(lam),   S_t = a_t S_(t-1) + sqrt(1 - a_t^2) i_t u_t,   out_t = S_t gelu(y_t)
 //
 // T is the model dtype; states, gates and decays are fp32.  Compiled without fast-math (csrc/build.py: EXACT_MATH).
+#include <type_traits>
+
 #include "mixers.cuh"
 #include "rglru.cuh"
 
@@ -95,32 +97,57 @@ conv_state_kernel(const T* __restrict__ x, long long ld, const float* __restrict
   }
 }
 
-// One token per slot: x is the slot's share of the input sums (cleared), the kept inputs move up by one.
-template <typename T>
+// One token per slot: x is the slot's share of the input sums (cleared), the kept inputs move up by one.  One thread per slot
+// and VEC channels.
+template <typename T, int VEC>
 __global__ void __launch_bounds__(128)
 conv_step_kernel(float* __restrict__ x, long long ld, const float* __restrict__ xb, const float* __restrict__ w,
                  const float* __restrict__ bias, const int* __restrict__ seq_lens, int C, int taps, float* __restrict__ state,
                  T* __restrict__ u) {
   pdl_launch_dependents();
   pdl_wait();
-  const int b = blockIdx.y, c = blockIdx.x * 128 + threadIdx.x;
+  const int b = blockIdx.y, c = (blockIdx.x * 128 + threadIdx.x) * VEC;
   if (c >= C) return;
-  const float in = x[(size_t)b * ld + c] + xb[c];
-  x[(size_t)b * ld + c] = 0.f;
+  float* st = state + (size_t)b * (taps - 1) * C + c;
+  float* xr = x + (size_t)b * ld + c;
+  const float* wc = w + (size_t)c * taps;
+  auto get = [](const float* p, float (&v)[VEC]) {
+    if (VEC == 4) {
+      const float4 t = load4(p);
+      v[0] = t.x; v[1 % VEC] = t.y; v[2 % VEC] = t.z; v[3 % VEC] = t.w;
+    } else {
+      v[0] = *p;
+    }
+  };
+  auto put = [](auto* p, const float (&v)[VEC]) {
+    if (VEC == 4) store4(p, make_float4(v[0], v[1 % VEC], v[2 % VEC], v[3 % VEC]));
+    else *p = from_f<typename std::remove_reference<decltype(*p)>::type>(v[0]);
+  };
+  float in[VEC], o[VEC], h[VEC], t[VEC];
+  get(xr, in);
+  get(xb + c, t);
+  get(bias + c, o);
+#pragma unroll
+  for (int i = 0; i < VEC; ++i) {
+    in[i] += t[i];
+    t[i] = 0.f;
+  }
+  put(xr, t);
   if (seq_lens[b] < 0) {
-    u[(size_t)b * C + c] = from_f<T>(0.f);
+    put(u + (size_t)b * C + c, t);
     return;
   }
-  float* st = state + (size_t)b * (taps - 1) * C + c;
-  const float* wc = w + (size_t)c * taps;
-  float o = bias[c] + wc[taps - 1] * in;
+#pragma unroll 3
   for (int j = 0; j < taps - 1; ++j) {
-    const float h = st[(size_t)j * C];
-    o += wc[j] * h;
-    if (j > 0) st[(size_t)(j - 1) * C] = h;
+    get(st + (size_t)j * C, h);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) o[i] += wc[(size_t)i * taps + j] * h[i];
+    if (j > 0) put(st + (size_t)(j - 1) * C, h);
   }
-  if (taps > 1) st[(size_t)(taps - 2) * C] = in;
-  u[(size_t)b * C + c] = from_f<T>(o);
+#pragma unroll
+  for (int i = 0; i < VEC; ++i) o[i] += wc[(size_t)i * taps + taps - 1] * in[i];
+  if (taps > 1) put(st + (size_t)(taps - 2) * C, in);
+  put(u + (size_t)b * C + c, o);
 }
 
 // Recurrence over packed prompts: one thread per (sequence, channel).  z [T, 2, C] fp32: logits of r and i without their biases.
@@ -202,9 +229,12 @@ TRLB_API int trlb_conv_step(float* x, long long ld, const float* xb, const float
                             int C, int taps, float* state, void* u, int is_bf16, cudaStream_t st) {
   if (B <= 0 || C <= 0) return 0;
   if (taps < 1) return -261;
-  const dim3 grid((C + 127) / 128, B), blk(128);
-  if (is_bf16) return (int)trlb_host::launch_kernel(conv_step_kernel<bf16>, grid, blk, 0, st, PDL, x, ld, xb, w, bias, seq_lens, C, taps, state, (bf16*)u);
-  return (int)trlb_host::launch_kernel(conv_step_kernel<float>, grid, blk, 0, st, PDL, x, ld, xb, w, bias, seq_lens, C, taps, state, (float*)u);
+  const bool v4 = C % 4 == 0 && ld % 4 == 0 && (reinterpret_cast<uintptr_t>(x) & 15) == 0;
+  const dim3 grid((C / (v4 ? 4 : 1) + 127) / 128, B), blk(128);
+#define GO(TT, VV) (int)trlb_host::launch_kernel(conv_step_kernel<TT, VV>, grid, blk, 0, st, PDL, x, ld, xb, w, bias, seq_lens, C, taps, state, (TT*)u)
+  if (is_bf16) return v4 ? GO(bf16, 4) : GO(bf16, 1);
+  return v4 ? GO(float, 4) : GO(float, 1);
+#undef GO
 }
 
 TRLB_API int trlb_rglru_scan(const float* z, const void* u, const void* y, long long y_ld, const float* lam, const float* gate_bias,

@@ -63,8 +63,8 @@ __device__ __forceinline__ void rg_gates(float zr, float zi, float neg_sp, float
   s = fmaf(x, s, 1.f / 6.f);
   s = fmaf(x, s, 0.5f);
   s = fmaf(x, s, 1.f);
-  const float v = x > -0.25f ? -x * s : fmaf(-a, a, 1.f);
-  w = sqrtf(v) * fast_sigmoid(zi);
+  const float v = fmaxf(x > -0.25f ? -x * s : fmaf(-a, a, 1.f), 1e-37f);
+  w = v * rsqrtf(v) * fast_sigmoid(zi);
 }
 
 __global__ void __launch_bounds__(RG_THREADS, 1)

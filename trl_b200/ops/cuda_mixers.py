@@ -224,6 +224,7 @@ def rglru_scan(z, u, y, m, ctx, seq_slot=None, state=None):
     """Recurrence of packed prompts on the CUDA cores.  z [T, 2, width] fp32 gate logits without their biases, u [T, width], y
     [T, width] GELU branch without its bias (rows may be strided); ``state`` [slots, width] of ``seq_slot`` gets the final one."""
     T, C = u.shape
+    assert z.is_contiguous() and z.dtype == torch.float32 and u.is_contiguous() and y.stride(1) == 1
     out = torch.empty(T, C, dtype=u.dtype, device=u.device)
     cu = ctx.cu_seqlens
     _chk(lib().trlb_rglru_scan(_p(z), _p(u), _p(y), c_longlong(y.stride(0)), _p(m.lam), _p(m.gate_bias), _p(m.y_bias), _p(cu),
@@ -248,6 +249,7 @@ def rglru_prompt_tc(u, y, m, ctx, seq_slot=None, state=None):
 def rglru_step(z, u, y, m, seq_lens, state, out):
     """One token per slot; y: fp32 sums of the GELU branch (zeroed)."""
     B, C = u.shape
+    assert z.is_contiguous() and z.dtype == torch.float32 and u.is_contiguous() and y.stride(1) == 1
     _chk(lib().trlb_rglru_step(_p(z), _p(u), _p(y), c_longlong(y.stride(0)), _p(m.lam), _p(m.gate_bias), _p(m.y_bias), _p(seq_lens),
                                c_int(B), _p(state), c_float(m.decay), c_int(C), _p(out), _b(u), _s()), "rglru_step")
 

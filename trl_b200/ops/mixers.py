@@ -208,7 +208,7 @@ def block_gates(u, gates):
     n, blocks, w, _ = gates.shape
     with _ieee_fp32():
         z = torch.matmul(u.float().view(T, blocks, w).transpose(0, 1), gates.float().transpose(2, 3))  # [2, blocks, T, w]
-    return z.permute(2, 0, 1, 3).reshape(T, n, C)
+    return z.permute(2, 0, 1, 3).reshape(T, n, C).contiguous()
 
 
 def rglru(m, h, ctx, li):
