@@ -70,40 +70,54 @@ __device__ __forceinline__ float la_capped(const MixerAttnTc& p, float v) {
   return v * fmaf(z, t, p.poly[0]);
 }
 
-// Second pass over a row of scores: probabilities, as value and remainder, in place.  LEVEL -1: no cap.  Returns their sum.
-template <int LEVEL>
-__device__ __forceinline__ float la_probs(const MixerAttnTc& p, uint32_t ts, float neg_m, bool full, int key0, int k_min, int k_max) {
-  float sum = 0.f;
-#pragma unroll
-  for (int c = 0; c < 4; ++c) {
+// First pass over a row of scores: the largest visible one and (SPAN) the largest magnitude of any.  Loops over 32 scores stay
+// rolled and tiles without masked keys have code of their own: instruction fetch and count are what limits these passes.
+template <bool SPAN, bool FULL>
+__device__ __forceinline__ float2 la_row_max(uint32_t ts, int first, int last) {
+  float mx[2] = {-INFINITY, -INFINITY}, mn[2] = {INFINITY, INFINITY};
+#pragma unroll 1
+  for (int c = 0; c < 128; c += 32) {
     float v[32];
-    tmem_ld_32x32(ts + 32 * c, v);
+    tmem_ld_32x32(ts + c, v);
     tmem_ld_wait();
+#pragma unroll
+    for (int i = 0; i < 32; ++i) {
+      if (SPAN) mn[i & 1] = fminf(mn[i & 1], FULL ? v[i] : -fabsf(v[i]));
+      mx[i & 1] = fmaxf(mx[i & 1], FULL || (c + i >= first && c + i <= last) ? v[i] : -INFINITY);
+    }
+  }
+  const float m = fmaxf(mx[0], mx[1]);
+  return make_float2(m, SPAN ? fmaxf(m, -fminf(mn[0], mn[1])) : 0.f);
+}
+
+// Second pass: probabilities, as value and remainder, in place.  LEVEL -1: no cap.  Returns their sum.
+template <int LEVEL, bool FULL>
+__device__ __forceinline__ float la_probs(const MixerAttnTc& p, uint32_t ts, float neg_m, int first, int last) {
+  float sum[2] = {0.f, 0.f};
+#pragma unroll 1
+  for (int c = 0; c < 128; c += 32) {
+    float v[32];
+    tmem_ld_32x32(ts + c, v);
+    tmem_ld_wait();
+    uint32_t a[16], b[16];
 #pragma unroll
     for (int i = 0; i < 32; ++i) {
       if (LEVEL < 0) v[i] = fast_exp2(fmaf(v[i], p.scale_log2, neg_m));
       else v[i] = fast_exp2(la_capped<LEVEL < 0 ? 0 : LEVEL>(p, v[i]) + neg_m);
+      if (!FULL) v[i] = c + i >= first && c + i <= last ? v[i] : 0.f;
+      sum[i & 1] += v[i];
     }
-    if (!full) {
-#pragma unroll
-      for (int i = 0; i < 32; ++i) {
-        const int key = key0 + 32 * c + i;
-        if (key < k_min || key > k_max) v[i] = 0.f;
-      }
-    }
-    uint32_t a[16], b[16];
 #pragma unroll
     for (int i = 0; i < 16; ++i) {
-      sum += v[2 * i] + v[2 * i + 1];
       a[i] = pack_bf16(v[2 * i], v[2 * i + 1]);
       const float2 f = unpack_bf16(a[i]);
       b[i] = pack_bf16(v[2 * i] - f.x, v[2 * i + 1] - f.y);
     }
-    tmem_st_32x16(ts + 32 * c, a);
-    tmem_st_32x16(ts + 32 * c + 16, b);
+    tmem_st_32x16(ts + c, a);
+    tmem_st_32x16(ts + c + 16, b);
   }
   tmem_st_wait();
-  return sum;
+  return sum[0] + sum[1];
 }
 
 template <bool CAP, int NB>
@@ -267,32 +281,13 @@ mixer_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_con
       if (!ok) break;
       tc_fence_after();
       const uint32_t ts = tmem_base + lane_off + (uint32_t)s * LA_BN;
-      // first pass: the row's largest score (and with a cap the largest magnitude)
-      float mx = -INFINITY, mn = INFINITY;
-#pragma unroll
-      for (int c = 0; c < 4; c += 2) {
-        float v[2][32];
-        tmem_ld_32x32(ts + 32 * c, v[0]);
-        tmem_ld_32x32(ts + 32 * c + 32, v[1]);
-        tmem_ld_wait();
-#pragma unroll
-        for (int h2 = 0; h2 < 2; ++h2)
-#pragma unroll
-          for (int i = 0; i < 32; ++i) {
-            const int key = key0 + 32 * (c + h2) + i;
-            if (CAP) mn = fminf(mn, v[h2][i]);
-            if (full) mx = fmaxf(mx, v[h2][i]);
-            else {
-              if (CAP) mn = fminf(mn, -v[h2][i]);  // masked scores count for the magnitude
-              if (key >= k_min && key <= k_max) mx = fmaxf(mx, v[h2][i]);
-            }
-          }
-      }
+      const int first = k_min - key0, last = k_max - key0;
+      const float2 top = full ? la_row_max<CAP, true>(ts, first, last) : la_row_max<CAP, false>(ts, first, last);
+      const float mx = top.x;
       int level = -1;
       float m_tile = mx * p.scale_log2;
       if (CAP) {
-        const float top = fmaxf(mx, -mn);
-        level = !__any_sync(0xffffffffu, top > p.near7) ? 0 : !__any_sync(0xffffffffu, top > p.near11) ? 1 : 2;
+        level = !__any_sync(0xffffffffu, top.y > p.near7) ? 0 : !__any_sync(0xffffffffu, top.y > p.near11) ? 1 : 2;
         m_tile = mx == -INFINITY ? mx : level == 0 ? la_capped<0>(p, mx) : level == 1 ? la_capped<1>(p, mx) : la_capped<2>(p, mx);
       }
       float alpha = 1.f;
@@ -322,10 +317,10 @@ mixer_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_con
       l_run *= alpha;
       const float neg_m = m_ref == -INFINITY ? 0.f : -m_ref;
       float sum;
-      if (!CAP) sum = la_probs<-1>(p, ts, neg_m, full, key0, k_min, k_max);
-      else if (level == 0) sum = la_probs<0>(p, ts, neg_m, full, key0, k_min, k_max);
-      else if (level == 1) sum = la_probs<1>(p, ts, neg_m, full, key0, k_min, k_max);
-      else sum = la_probs<2>(p, ts, neg_m, full, key0, k_min, k_max);
+      if (!CAP) sum = full ? la_probs<-1, true>(p, ts, neg_m, first, last) : la_probs<-1, false>(p, ts, neg_m, first, last);
+      else if (level == 0) sum = full ? la_probs<0, true>(p, ts, neg_m, first, last) : la_probs<0, false>(p, ts, neg_m, first, last);
+      else if (level == 1) sum = la_probs<1, false>(p, ts, neg_m, first, last);
+      else sum = la_probs<2, false>(p, ts, neg_m, first, last);
       // P.V(last) completes phase `last` of o_full, and may do so before this thread looks: phase last - 1 has to be seen
       // first.  (With one S buffer the last S was issued after P.V(last - 1), so s_full has shown it.)
       if (NB == 2 && j > 0 && j == n_kv - 1)
