@@ -1,11 +1,12 @@
 """Builds the in-tree native libraries.
 
-    python -m trl_b200.csrc.build [--force] [--verbose] [--part layered]
+    python -m trl_b200.csrc.build [--force] [--verbose] [--part layered [--kinds attention,moe]]
 
 * ``trl_b200/_lib/libtrl_b200_kernels.so``  every ``*.cu`` here, compiled by nvcc for sm_100a only
   (``-gencode arch=compute_100a,code=sm_100a``); works without a GPU (cross-compile).
-* ``trl_b200/_lib/libtrl_b200_layered.so``  with ``--part layered``: only the sources that serving a layered decoder needs
-  (used when the whole kernel library has not been built).
+* ``trl_b200/_lib/libtrl_b200_layered.so``  with ``--part layered``: only the sources that serving a layered decoder with
+  these mixers and feed-forwards needs, and those of earlier such builds (used when the whole kernel library has not been
+  built).
 * ``trl_b200/_lib/libtrl_b200_host.so``     ``*.cpp`` host runtime (scheduler, packing), g++ -O3.
 
 Objects are cached next to the sources' hashes, so unchanged files are not recompiled.
@@ -27,14 +28,17 @@ OBJ = os.path.join(LIB, "obj")
 NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17", "--use_fast_math",
               "-Xcompiler", "-fPIC,-fvisibility=hidden", "-Xptxas", "-v", "--expt-relaxed-constexpr"]
 # sources whose results the fast approximations of exp, tanh, erf, division and square root would show in
-EXACT_MATH = {"grouped_attn.cu", "mixers.cu", "mlstm_chunk_tcgen05.cu", "rglru.cu", "rglru_tcgen05.cu"}
+EXACT_MATH = {"grouped_attn.cu", "layered_moe.cu", "mixers.cu", "mlstm_chunk_tcgen05.cu", "rglru.cu", "rglru_tcgen05.cu"}
 # every source here builds into the one library used at any GPU count (no loads shared across a thread-block cluster)
 
 
-# parts of the kernel library that can be built alone
-PARTS = {"layered": ("decode.cu", "decode_gemm.cu", "grouped_attn.cu", "grouped_decode_tcgen05.cu", "latent_decode_tcgen05.cu",
-                     "mixer_attn_tcgen05.cu", "mixers.cu", "mlstm_chunk_tcgen05.cu", "rglru.cu", "rglru_tcgen05.cu",
-                     "tensormap.cu")}
+# Parts of the kernel library that can be built alone.  "layered": what every layered decoder needs, and the sources of the
+# mixers and feed-forwards it has.
+PARTS = {"layered": ("decode.cu", "decode_gemm.cu", "mixers.cu", "tensormap.cu")}
+_GROUPED = ("grouped_attn.cu", "grouped_decode_tcgen05.cu", "mixer_attn_tcgen05.cu")
+LAYERED_KINDS = {"latent_attention": ("grouped_attn.cu", "latent_decode_tcgen05.cu", "mixer_attn_tcgen05.cu"),
+                 "mlstm": ("mlstm_chunk_tcgen05.cu",), "attention": _GROUPED, "attention_2": _GROUPED,
+                 "rglru": ("rglru.cu", "rglru_tcgen05.cu"), "moe": ("grouped_gemm_tcgen05.cu", "layered_moe.cu")}
 
 
 def _nvcc() -> str:
@@ -77,10 +81,16 @@ def _compile(src: str, force: bool, verbose: bool) -> str:
     return obj
 
 
-def build(force: bool = False, verbose: bool = False, part: str | None = None) -> dict[str, str]:
+def build(force: bool = False, verbose: bool = False, part: str | None = None, kinds=None) -> dict[str, str]:
+    """``kinds`` (with ``part``): the :data:`LAYERED_KINDS` it has to cover, default all of them."""
     os.makedirs(OBJ, exist_ok=True)
-    cus = sorted(os.path.join(HERE, f) for f in os.listdir(HERE)
-                 if f.endswith(".cu") and (part is None or f in PARTS[part]))
+    want = set(os.listdir(HERE))
+    if part is not None:
+        built = {f.split(".cu.")[0] + ".cu" for f in os.listdir(OBJ) if f.endswith(".o")}  # earlier builds' sources stay in
+        some = {f for k in (LAYERED_KINDS if kinds is None else kinds) for f in LAYERED_KINDS.get(k, ())}
+        every = {f for fs in LAYERED_KINDS.values() for f in fs}
+        want &= set(PARTS[part]) | some | (every & built)
+    cus = sorted(os.path.join(HERE, f) for f in want if f.endswith(".cu"))
     cpps = sorted(os.path.join(HERE, f) for f in os.listdir(HERE) if f.endswith(".cpp"))
     with cf.ThreadPoolExecutor(max_workers=min(8, os.cpu_count() or 2)) as ex:
         cu_objs = list(ex.map(lambda s: _compile(s, force, verbose), cus))
@@ -110,8 +120,9 @@ def main():
     ap.add_argument("--force", action="store_true")
     ap.add_argument("--verbose", action="store_true")
     ap.add_argument("--part", choices=sorted(PARTS))
+    ap.add_argument("--kinds", help="comma-separated kinds a layered part covers (default: all)")
     a = ap.parse_args()
-    for k, v in build(a.force, a.verbose, a.part).items():
+    for k, v in build(a.force, a.verbose, a.part, a.kinds.split(",") if a.kinds else None).items():
         print(f"{k}: {v}")
 
 

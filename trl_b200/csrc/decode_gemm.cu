@@ -24,7 +24,8 @@
 //     while other SMs still stream weights, and the consumer waits only on its own counter;
 //   * whole-slab schedules store bf16 directly (+ bias), or apply SwiGLU: gate and up slabs of the same features go
 //     to two accumulators through alternate pipeline stages and the epilogue writes silu(gate) * up (or the clamped
-//     gated unit g sigmoid(alpha g) (u + shift) of g = min(gate, limit), u = up clamped to [-limit, limit]);
+//     gated unit g sigmoid(alpha g) (u + shift) of g = min(gate, limit), u = up clamped to [-limit, limit], or
+//     gelu_tanh(gate) * up);
 //   * W may be stored tile-major ([slab][K block][128][64], each 16 KB tile contiguous), which turns the weight
 //     stream into sequential DRAM bursts; tensor-parallel engines repack their weight slices anyway and use it;
 //   * the kernel is launched with programmatic stream serialization: barrier set-up, TMEM allocation and the first
@@ -42,7 +43,7 @@ constexpr int DG_THREADS = 192;
 constexpr uint32_t DG_W_BYTES = DG_BM * DG_BK * 2;
 constexpr int DG_MAX_PEERS = 7;
 
-enum { DG_ACCUM_F32 = 0, DG_STORE_BF16 = 1, DG_SWIGLU = 2, DG_GELU = 3, DG_CLAMPED_GLU = 4 };
+enum { DG_ACCUM_F32 = 0, DG_STORE_BF16 = 1, DG_SWIGLU = 2, DG_GELU = 3, DG_CLAMPED_GLU = 4, DG_GELU_GLU = 5 };
 
 struct DecodeGemmParams {
   int B, N, K;
@@ -285,6 +286,9 @@ decode_gemm_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_cons
               const float g = fminf(v[i], p.glu_limit), w = fminf(fmaxf(u[i], -p.glu_limit), p.glu_limit);
               v[i] = g * fast_sigmoid(p.glu_alpha * g) * (w + p.glu_shift);
             }
+          } else if (p.mode == DG_GELU_GLU) {
+#pragma unroll
+            for (int i = 0; i < 16; ++i) v[i] = fast_gelu_tanh(v[i]) * u[i];
           } else {
 #pragma unroll
             for (int i = 0; i < 16; ++i) v[i] = v[i] / (1.f + __expf(-v[i])) * u[i];
@@ -390,10 +394,10 @@ int dg_launch(const CUtensorMap& tw, const CUtensorMap& tx, const DecodeGemmPara
   return (int)trlb_host::launch_kernel(kern, dim3(ctas), dim3(DG_THREADS), C::SMEM, st, trlb_host::pdl_enabled(), tw, tx, p);
 }
 
-bool dg_glu(int mode) { return mode == DG_SWIGLU || mode == DG_CLAMPED_GLU; }
+bool dg_glu(int mode) { return mode == DG_SWIGLU || mode == DG_CLAMPED_GLU || mode == DG_GELU_GLU; }
 
 int dg_ctas_per_sm(int B, int mode) {
-  if (mode == DG_GELU || mode == DG_CLAMPED_GLU) return 1;
+  if (mode == DG_GELU || mode == DG_CLAMPED_GLU || mode == DG_GELU_GLU) return 1;
   if (B > 64) return (mode == DG_SWIGLU || g_ctas_per_sm < 2) ? 1 : 2;  // 128-row tiles: 256 / 512 TMEM columns each
   if (mode == DG_SWIGLU) return 1;  // SwiGLU slabs cannot be split along K: one CTA per SM with a deep ring
   return g_ctas_per_sm;
@@ -436,6 +440,7 @@ TRLB_API int trlb_decode_gemm_arrivals(int N) { return 4 * ((N + DG_BM - 1) / DG
 //   mode 3  like mode 1 with the exact GELU of the sum stored
 //   mode 2  W [2N, K] (gate rows, then up rows; N a multiple of 128);  Yb [B, N] bf16 = silu(X Wg^T) * (X Wu^T)
 //   mode 4  W [2N, K] row-major, any N;  Yb [B, N] bf16 = clamped gated unit of both (glu = {limit, alpha, shift})
+//   mode 5  like mode 4;  Yb = gelu_tanh(X Wg^T) * (X Wu^T)
 // max_ctas: 0 = every SM with its resident CTAs, else an upper bound on the grid.
 // Fused all-reduce (mode 0, n_peers > 0): peer_y32[i] is the same buffer on peer i; arrive[0] is this rank's arrival
 // counter and arrive[1 + i] peer i's; stage is a local zeroed fp32 buffer shaped like Y32 and slab_ctr a local zeroed
@@ -447,8 +452,9 @@ TRLB_API int trlb_decode_gemm(const void* X, const void* W, const void* bias, fl
                               float* const* peer_y32, uint32_t* const* arrive, float* stage, uint32_t* slab_ctr,
                               const float* glu, int* status, cudaStream_t st) {
   if (B <= 0 || N <= 0 || K <= 0) return 0;
-  if (B > 128 || (K % 8) != 0 || (ldx % 8) != 0 || mode < 0 || mode > 4) return -150;
-  if (mode == DG_CLAMPED_GLU && (bias != nullptr || tiled || glu == nullptr)) return -150;
+  if (B > 128 || (K % 8) != 0 || (ldx % 8) != 0 || mode < 0 || mode > 5) return -150;
+  if (mode == DG_CLAMPED_GLU && glu == nullptr) return -150;
+  if ((mode == DG_CLAMPED_GLU || mode == DG_GELU_GLU) && (bias != nullptr || tiled)) return -150;
   if (!tiled && (ldw % 8) != 0) return -150;
   if (mode == DG_SWIGLU && (bias != nullptr || (N % DG_BM) != 0)) return -150;
   if (n_peers < 0 || n_peers > DG_MAX_PEERS || (n_peers > 0 && (mode != DG_ACCUM_F32 || !peer_y32 || !arrive))) return -150;

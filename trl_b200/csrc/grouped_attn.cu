@@ -8,105 +8,213 @@
 namespace trlb {
 
 // ------------------------------------------------------------------------------------------------------------
-// From the projections of a layer's input, rows [q | k | v | g] (no k and v in a layer that reads another one's cache):
-// queries divided by their rms per head and multiplied by the temperature of their position, keys divided by their rms,
-// keys and values to the paged cache.  S is the dtype of the rows: T (prompt: q and k are replaced in place, v and g stay
-// where they are) or fp32 sums (decode: q and the gate logits go to buffers, everything read is zeroed).
-// One warp per (row, head of q / k / v / g).
+// From the projections of a layer's input, rows [q | k | v | g] (no k and v in a layer that reads another one's cache, no v
+// where the projected keys are the values, g per element, per head or absent): queries and keys divided by their rms, of a
+// head or (WHOLE) of all heads, times a weight; queries times the temperature of their position; both rotated; keys and
+// values to the paged cache.  S is the dtype of the rows: T (prompt: v and g per element stay where they are, q is replaced in
+// place, k too unless k_out is given) or fp32 sums (decode: q and the gate logits go to buffers, everything read is zeroed).
+// Gates per head leave as sigmoids.  One warp per (row, head of q / k / v / g or all gates of heads); WHOLE: one block per row.
 // ------------------------------------------------------------------------------------------------------------
+enum { GATES_NONE = 0, GATES_HEAD = 1, GATES_ELEMENT = 2 };
+
 struct AttnPrep {
   long long ld;
-  int rows, heads, kv_heads, dim, vdim, has_kv, has_gate;
+  int rows, heads, kv_heads, dim, vdim, has_kv, has_v, gates;
   float eps;
   const int* positions;   // [rows]
   const int* tok_slot;    // [rows] or null (slot = row)
   const float* temp;      // [temp_len] factor of the query by position, or null
   int temp_len;
+  const float* q_w;       // norm weights, [dim] or (WHOLE) [heads dim] / [kv_heads dim]; null: none
+  const float* k_w;
+  int rot, halves;        // rotated elements of a head; pairs (i, i + rot / 2) instead of (2 i, 2 i + 1)
+  const float2* table;    // [table_len, rot / 2] (cos, sin) with the rotation's magnitude folded in
+  int table_len;
+  float* head_gate;       // [rows, heads]
   const int* block_table;  // null: no cache
   int max_blocks, block_size;
 };
 
-template <typename T, typename S>
-__global__ void __launch_bounds__(256)
-attn_prep_kernel(const AttnPrep p, S* __restrict__ src, T* __restrict__ q_out, T* __restrict__ g_out, T* __restrict__ k_cache,
-                 T* __restrict__ v_cache) {
+template <typename T, typename S, bool WHOLE>
+__global__ void __launch_bounds__(WHOLE ? 512 : 256)
+attn_prep_kernel(const AttnPrep p, S* __restrict__ src, T* __restrict__ q_out, T* __restrict__ k_out, T* __restrict__ g_out,
+                 T* __restrict__ k_cache, T* __restrict__ v_cache) {
   constexpr bool SUMS = !(sizeof(T) == 2 && sizeof(S) == 2);  // fp32 models: q_out tells (null: in place)
+  __shared__ float red[WHOLE ? 64 : 1];
   pdl_launch_dependents();
   pdl_wait();
   const int lane = threadIdx.x & 31;
-  const int kv = p.has_kv ? p.kv_heads : 0, units = p.heads + 2 * kv + (p.has_gate && g_out != nullptr ? p.heads : 0);
-  const long long item = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
-  if (item >= (long long)p.rows * units) return;
-  const int row = (int)(item / units), u = (int)(item % units);
-  const int pos = p.positions[row];
   const bool in_place = !SUMS || q_out == nullptr;
+  const int kv = p.has_kv ? p.kv_heads : 0, vv = p.has_v ? kv : 0;
+  const int ge = p.gates == GATES_ELEMENT && !in_place ? p.heads : 0;
+  const int units = p.heads + kv + vv + ge + (p.gates == GATES_HEAD ? 1 : 0);
+  const int q_n = p.heads * p.dim, k_n = kv * p.dim, v_n = vv * p.vdim;
+  int row, u, u_end, u_step;
+  float sq = 0.f, sk = 0.f;  // WHOLE: 1 / rms of all queries, of all keys
+  if (WHOLE) {
+    row = blockIdx.x;
+    u = threadIdx.x >> 5;
+    u_end = units;
+    u_step = blockDim.x >> 5;
+    const S* r = src + (size_t)row * p.ld;
+    const bool v4 = ((q_n | k_n | (int)p.ld) & 3) == 0 && (reinterpret_cast<uintptr_t>(src) & (4 * sizeof(S) - 1)) == 0;
+    if (v4) {
+      for (int j = 4 * threadIdx.x; j < q_n + k_n; j += 4 * blockDim.x) {
+        const float4 v = load4(r + j);
+        const float ss = v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+        if (j < q_n) sq += ss; else sk += ss;
+      }
+    } else {
+      for (int j = threadIdx.x; j < q_n + k_n; j += blockDim.x) {
+        const float v = to_f(r[j]);
+        if (j < q_n) sq += v * v; else sk += v * v;
+      }
+    }
+    const float2 s = block_sum2(sq, sk, red);  // a barrier: the row is replaced below
+    sq = 1.f / sqrtf(s.x / (float)q_n + p.eps);
+    sk = k_n > 0 ? 1.f / sqrtf(s.y / (float)k_n + p.eps) : 0.f;
+  } else {
+    const long long item = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
+    if (item >= (long long)p.rows * units) return;
+    row = (int)(item / units);
+    u = (int)(item % units);
+    u_end = u + 1;
+    u_step = 1;
+  }
+  const int pos = p.positions[row];
   S* r = src + (size_t)row * p.ld;
-  const int q_n = p.heads * p.dim, k_n = kv * p.dim, v_n = kv * p.vdim;
-  S* x;
-  int n;
-  bool normed = false;
-  T* dst = nullptr;    // besides the cache
-  T* paged = nullptr;
-  float mul = 1.f;
   long long at = -1;   // token's row in the cache
-  if (pos >= 0 && p.block_table != nullptr && u >= p.heads && u < p.heads + 2 * kv) {
+  if (pos >= 0 && p.block_table != nullptr) {
     const int slot = p.tok_slot ? p.tok_slot[row] : row;
     if (slot >= 0 && pos / p.block_size < p.max_blocks)
       at = (long long)p.block_table[(size_t)slot * p.max_blocks + pos / p.block_size] * p.block_size + pos % p.block_size;
   }
-  if (u < p.heads) {
-    x = r + (size_t)u * p.dim;
-    n = p.dim;
-    normed = true;
-    if (p.temp != nullptr && pos >= 0 && pos < p.temp_len) mul = p.temp[pos];
-    if (!in_place) dst = q_out + ((size_t)row * p.heads + u) * p.dim;
-  } else if (u < p.heads + kv) {
-    const int h = u - p.heads;
-    x = r + q_n + (size_t)h * p.dim;
-    n = p.dim;
-    normed = true;
-    if (at >= 0) paged = k_cache + (size_t)(at * kv + h) * p.dim;
-  } else if (u < p.heads + 2 * kv) {
-    const int h = u - p.heads - kv;
-    x = r + q_n + k_n + (size_t)h * p.vdim;
-    n = p.vdim;
-    if (at >= 0) paged = v_cache + (size_t)(at * kv + h) * p.vdim;
-  } else {
-    const int h = u - p.heads - 2 * kv;
-    x = r + q_n + k_n + v_n + (size_t)h * p.vdim;
-    n = p.vdim;
-    dst = g_out + ((size_t)row * p.heads + h) * p.vdim;
-  }
-  const bool vec = ((n | (int)p.ld | (int)(x - r)) & 3) == 0 && (reinterpret_cast<uintptr_t>(src) & (4 * sizeof(S) - 1)) == 0;
-  float s = 1.f;
-  if (normed) {
-    float ss = 0.f;
+  const float2* cs = p.rot > 0 && pos >= 0 && pos < p.table_len ? p.table + (size_t)pos * (p.rot / 2) : nullptr;
+  for (; u < u_end; u += u_step) {
+    if (p.gates == GATES_HEAD && u == units - 1) {
+      S* g = r + q_n + k_n + v_n;
+      for (int h = lane; h < p.heads; h += 32) {
+        p.head_gate[(size_t)row * p.heads + h] = sigmoid_f(to_f(g[h]));
+        if (!in_place) g[h] = from_f<S>(0.f);
+      }
+      continue;
+    }
+    S* x;
+    int n;
+    bool normed = false;
+    float mul = 1.f, s = 1.f;
+    const float* w = nullptr;
+    T* dst = nullptr;    // besides the cache
+    T* paged = nullptr;
+    T* raw = nullptr;    // cache row that gets the elements as they are
+    bool put = false;    // back into the row
+    if (u < p.heads) {
+      x = r + (size_t)u * p.dim;
+      n = p.dim;
+      normed = true;
+      w = p.q_w == nullptr ? nullptr : WHOLE ? p.q_w + (size_t)u * p.dim : p.q_w;
+      s = sq;
+      if (p.temp != nullptr && pos >= 0 && pos < p.temp_len) mul = p.temp[pos];
+      if (!in_place) dst = q_out + ((size_t)row * p.heads + u) * p.dim;
+      put = in_place;
+    } else if (u < p.heads + kv) {
+      const int h = u - p.heads;
+      x = r + q_n + (size_t)h * p.dim;
+      n = p.dim;
+      normed = true;
+      w = p.k_w == nullptr ? nullptr : WHOLE ? p.k_w + (size_t)h * p.dim : p.k_w;
+      s = sk;
+      if (k_out != nullptr) dst = k_out + ((size_t)row * kv + h) * p.dim;
+      if (at >= 0) {
+        paged = k_cache + (size_t)(at * kv + h) * p.dim;
+        if (vv == 0) raw = v_cache + (size_t)(at * kv + h) * p.dim;
+      }
+      put = in_place && k_out == nullptr;
+    } else if (u < p.heads + kv + vv) {
+      const int h = u - p.heads - kv;
+      x = r + q_n + k_n + (size_t)h * p.vdim;
+      n = p.vdim;
+      if (at >= 0) paged = v_cache + (size_t)(at * kv + h) * p.vdim;
+    } else {
+      const int h = u - p.heads - kv - vv;
+      x = r + q_n + k_n + v_n + (size_t)h * p.vdim;
+      n = p.vdim;
+      dst = g_out + ((size_t)row * p.heads + h) * p.vdim;
+    }
+    const int rot = normed ? p.rot : 0;
+    const bool vec = ((n | (int)p.ld | (int)(x - r)) & 3) == 0 && (reinterpret_cast<uintptr_t>(src) & (4 * sizeof(S) - 1)) == 0 &&
+                     (rot & (p.halves ? 7 : 3)) == 0;
+    if (normed && !WHOLE) {
+      float ss = 0.f;
+      if (vec) {
+        for (int j = 4 * lane; j < n; j += 128) {
+          const float4 v = load4(x + j);
+          ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+        }
+      } else {
+        for (int j = lane; j < n; j += 32) ss += to_f(x[j]) * to_f(x[j]);
+      }
+      s = 1.f / sqrtf(warp_sum(ss) / (float)n + p.eps);
+    }
+    if (normed) s *= mul; else s = 1.f;
     if (vec) {
-      for (int j = 4 * lane; j < n; j += 128) {
-        const float4 v = load4(x + j);
-        ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+      auto get = [&](int j) {
+        float4 v = load4(x + j);
+        if (raw) store4(raw + j, v);
+        v = make_float4(v.x * s, v.y * s, v.z * s, v.w * s);
+        if (w != nullptr) {
+          const float4 g = load4(w + j);
+          v = make_float4(v.x * g.x, v.y * g.y, v.z * g.z, v.w * g.w);
+        }
+        return v;
+      };
+      auto set = [&](int j, float4 v) {
+        if (dst) store4(dst + j, v);
+        if (paged) store4(paged + j, v);
+        if (!in_place) store4(x + j, make_float4(0.f, 0.f, 0.f, 0.f));
+        else if (put) store4(x + j, v);
+      };
+      if (rot > 0 && p.halves) {
+        const int half = rot / 2;
+        for (int i = 4 * lane; i < half; i += 128) {
+          const float4 a = get(i), b = get(i + half);
+          float2 c[4];
+#pragma unroll
+          for (int k = 0; k < 4; ++k) c[k] = cs != nullptr ? cs[i + k] : make_float2(1.f, 0.f);
+          set(i, make_float4(a.x * c[0].x - b.x * c[0].y, a.y * c[1].x - b.y * c[1].y, a.z * c[2].x - b.z * c[2].y, a.w * c[3].x - b.w * c[3].y));
+          set(i + half, make_float4(b.x * c[0].x + a.x * c[0].y, b.y * c[1].x + a.y * c[1].y, b.z * c[2].x + a.z * c[2].y, b.w * c[3].x + a.w * c[3].y));
+        }
+        for (int j = rot + 4 * lane; j < n; j += 128) set(j, get(j));
+      } else {
+        for (int j = 4 * lane; j < n; j += 128) {
+          float4 v = get(j);
+          if (j < rot && cs != nullptr) {
+            const float2 c0 = cs[j / 2], c1 = cs[j / 2 + 1];
+            v = make_float4(v.x * c0.x - v.y * c0.y, v.y * c0.x + v.x * c0.y, v.z * c1.x - v.w * c1.y, v.w * c1.x + v.z * c1.y);
+          }
+          set(j, v);
+        }
       }
     } else {
-      for (int j = lane; j < n; j += 32) ss += to_f(x[j]) * to_f(x[j]);
-    }
-    s = mul / sqrtf(warp_sum(ss) / (float)n + p.eps);
-  }
-  if (vec) {
-    for (int j = 4 * lane; j < n; j += 128) {
-      float4 v = load4(x + j);
-      v = make_float4(v.x * s, v.y * s, v.z * s, v.w * s);
-      if (dst) store4(dst + j, v);
-      if (paged) store4(paged + j, v);
-      if (!in_place) store4(x + j, make_float4(0.f, 0.f, 0.f, 0.f));
-      else if (normed) store4(x + j, v);
-    }
-  } else {
-    for (int j = lane; j < n; j += 32) {
-      const float v = to_f(x[j]) * s;
-      if (dst) dst[j] = from_f<T>(v);
-      if (paged) paged[j] = from_f<T>(v);
-      if (!in_place) x[j] = from_f<S>(0.f);
-      else if (normed) x[j] = from_f<S>(v);
+      auto get = [&](int j) {
+        const float v = to_f(x[j]);
+        if (raw) raw[j] = from_f<T>(v);
+        return w != nullptr ? v * s * w[j] : v * s;
+      };
+      auto set = [&](int j, float v) {
+        if (dst) dst[j] = from_f<T>(v);
+        if (paged) paged[j] = from_f<T>(v);
+        if (!in_place) x[j] = from_f<S>(0.f);
+        else if (put) x[j] = from_f<S>(v);
+      };
+      for (int i = lane; i < rot / 2; i += 32) {
+        const int ia = p.halves ? i : 2 * i, ib = p.halves ? i + rot / 2 : 2 * i + 1;
+        const float a = get(ia), b = get(ib);
+        const float2 c = cs != nullptr ? cs[i] : make_float2(1.f, 0.f);
+        set(ia, a * c.x - b * c.y);
+        set(ib, b * c.x + a * c.y);
+      }
+      for (int j = rot + lane; j < n; j += 32) set(j, get(j));
     }
   }
 }
@@ -114,10 +222,11 @@ attn_prep_kernel(const AttnPrep p, S* __restrict__ src, T* __restrict__ q_out, T
 // ------------------------------------------------------------------------------------------------------------
 // Prompt attention, any size: one warp per (token, head).  Keys of token t are rows t - min(pos, window - 1) .. t of the
 // packed stream (pos counts from the token's own sequence start), so no sequence table is needed.  Keys may have a second
-// part of `rot` elements shared by the heads; scores may be capped; sink and gate may be null.
+// part of `rot` elements shared by the heads; scores may be capped; sink and gate may be null.  With a window the first `keep`
+// keys of the sequence stay visible: the keys of a token are a list of those before the window, then the window.
 // ------------------------------------------------------------------------------------------------------------
 struct MixerAttn {
-  int T, heads, group, dim, rot, vdim, window;
+  int T, heads, group, dim, rot, vdim, window, keep;
   long long q_ld, k_ld, v_ld, kr_ld, gate_ld;
   float scale, cap;
   const int* positions;
@@ -144,13 +253,14 @@ mixer_attn_kernel(const MixerAttn p, const T* __restrict__ q, const T* __restric
   for (int e = lane; e < p.vdim; e += 32) os[e] = 0.f;
   __syncwarp();
   const int pos = p.positions[t];
-  const int back = p.window > 0 ? min(pos, p.window - 1) : pos;
-  const int k0 = t - back;
+  const int start = t - pos, lo = p.window > 0 ? max(0, pos - p.window + 1) : 0, kept = min(p.keep, lo);
+  const int n_keys = kept + pos - lo + 1;
+  auto key_row = [&](int i) { return start + (i < kept ? i : lo + i - kept); };
   float m = -INFINITY, l = 0.f;
-  for (int base = k0; base <= t; base += 32) {
-    const int key = base + lane;
+  for (int base = 0; base < n_keys; base += 32) {
+    const int key = key_row(base + lane);
     float s = -INFINITY;
-    if (key <= t) {
+    if (base + lane < n_keys) {
       const T* kn = k + (size_t)key * p.k_ld + (size_t)hk * p.dim;
       float acc = 0.f;
       for (int d = 0; d < p.dim; ++d) acc += qs[d] * to_f(kn[d]);
@@ -162,16 +272,16 @@ mixer_attn_kernel(const MixerAttn p, const T* __restrict__ q, const T* __restric
     }
     const float mn = fmaxf(m, warp_max(s));
     const float corr = m == -INFINITY ? 0.f : expf(m - mn);
-    const float pr = key <= t ? expf(s - mn) : 0.f;
+    const float pr = base + lane < n_keys ? expf(s - mn) : 0.f;
     l = l * corr + warp_sum(pr);
     m = mn;
-    const int nk = min(32, t - base + 1);
+    const int nk = min(32, n_keys - base);
     const int e_end = (p.vdim + 31) & ~31;
     for (int e = lane; e < e_end; e += 32) {
       float acc = e < p.vdim ? os[e] * corr : 0.f;
       for (int j = 0; j < nk; ++j) {
         const float w = __shfl_sync(0xffffffffu, pr, j);
-        if (e < p.vdim) acc += w * to_f(v[(size_t)(base + j) * p.v_ld + (size_t)hk * p.vdim + e]);
+        if (e < p.vdim) acc += w * to_f(v[(size_t)key_row(base + j) * p.v_ld + (size_t)hk * p.vdim + e]);
       }
       if (e < p.vdim) os[e] = acc;
     }
@@ -192,10 +302,12 @@ mixer_attn_kernel(const MixerAttn p, const T* __restrict__ q, const T* __restric
 // keys in turn, lanes own dimensions.
 // ------------------------------------------------------------------------------------------------------------
 struct GroupedDecode {
-  int B, heads, kv_heads, dim, vdim, max_blocks, block_size;
+  int B, heads, kv_heads, dim, vdim, max_blocks, block_size, window, keep;
   float scale, cap;
   const int* seq_lens;
   const int* block_table;
+  const float* sink;       // [heads] or null
+  const float* head_gate;  // [B, heads] or null
 };
 
 constexpr int GD_MAX_REG = 32;
@@ -218,7 +330,9 @@ grouped_decode_kernel(const GroupedDecode p, const T* __restrict__ q, const T* _
   float m = -INFINITY, l = 0.f, acc[GD_MAX_REG];
 #pragma unroll
   for (int i = 0; i < GD_MAX_REG; ++i) acc[i] = 0.f;
-  for (int j = warp; j <= pos; j += 4) {
+  const int lo = p.window > 0 ? max(0, pos - p.window + 1) : 0, kept = min(p.keep, lo), n_keys = kept + pos - lo + 1;
+  for (int i = warp; i < n_keys; i += 4) {
+    const int j = i < kept ? i : lo + i - kept;
     const size_t row = ((size_t)bt[j / p.block_size] * p.block_size + j % p.block_size) * p.kv_heads + hk;
     const T* kr = k_cache + row * p.dim;
     const T* vr = v_cache + row * p.vdim;
@@ -243,6 +357,10 @@ grouped_decode_kernel(const GroupedDecode p, const T* __restrict__ q, const T* _
   __syncthreads();
   float mt = ml[0], den = 0.f, f[4];  // warp 0 always has a key
   for (int w = 1; w < 4; ++w) mt = fmaxf(mt, ml[w]);
+  if (p.sink != nullptr) {
+    mt = fmaxf(mt, p.sink[h]);
+    den = expf(p.sink[h] - mt);
+  }
   for (int w = 0; w < 4; ++w) {
     f[w] = ml[w] == -INFINITY ? 0.f : expf(ml[w] - mt);
     den += f[w] * ml[4 + w];
@@ -251,6 +369,7 @@ grouped_decode_kernel(const GroupedDecode p, const T* __restrict__ q, const T* _
     float o = 0.f;
     for (int w = 0; w < 4; ++w) o += f[w] * po[(size_t)w * p.vdim + e];
     o /= den;
+    if (p.head_gate != nullptr) o *= p.head_gate[(size_t)b * p.heads + h];
     const size_t i = ((size_t)b * p.heads + h) * p.vdim + e;
     if (gate != nullptr) o *= sigmoid_f(to_f(gate[i]));
     out[i] = from_f<T>(o);
@@ -276,32 +395,41 @@ using bf16 = __nv_bfloat16;
 
 #define PDL trlb_host::pdl_enabled()
 
-// rows [q | k | v | g] of ld elements; src_f32: fp32 sums (decode: q_out and g_out given), else the model dtype.  temp, tok_slot,
-// block_table may be null.
+// rows [q | k | v | g] of ld elements; src_f32: fp32 sums (decode: q_out and, for gates per element, g_out given), else the model
+// dtype.  temp, q_w, k_w, tok_slot, k_out, block_table may be null; gates: 0 none, 1 per head (to head_gate), 2 per element; rot 0:
+// no rotation; whole: norms over all heads.  Without has_v the keys as projected are the values (prompt: k_out is then required).
 TRLB_API int trlb_attn_prep(void* src, int src_f32, long long ld, int rows, int heads, int kv_heads, int dim, int vdim, int has_kv,
-                            int has_gate, float eps, const int* positions, const int* tok_slot, const float* temp, int temp_len,
-                            void* q_out, void* g_out, void* k_cache, void* v_cache, const int* block_table, int max_blocks,
-                            int block_size, int is_bf16, cudaStream_t st) {
+                            int has_v, int gates, float eps, const int* positions, const int* tok_slot, const float* temp,
+                            int temp_len, int whole, const float* q_w, const float* k_w, int rot, int halves, const float* table,
+                            int table_len, void* q_out, void* k_out, void* g_out, float* head_gate, void* k_cache, void* v_cache,
+                            const int* block_table, int max_blocks, int block_size, int is_bf16, cudaStream_t st) {
   if (rows <= 0) return 0;
   if (heads <= 0 || kv_heads <= 0 || heads % kv_heads || (is_bf16 && src_f32 && q_out == nullptr)) return -250;
-  AttnPrep p = {ld, rows, heads, kv_heads, dim, vdim, has_kv, has_gate, eps, positions, tok_slot, temp, temp_len,
-                k_cache ? block_table : nullptr, max_blocks, block_size};
-  const int units = heads + (has_kv ? 2 * kv_heads : 0) + (has_gate && g_out != nullptr ? heads : 0);
-  const dim3 grid((unsigned)(((long long)rows * units + 7) / 8)), blk(256);
-#define GO(TT, SS) (int)trlb_host::launch_kernel(attn_prep_kernel<TT, SS>, grid, blk, 0, st, PDL, p, (SS*)src, (TT*)q_out, (TT*)g_out, (TT*)k_cache, (TT*)v_cache)
-  if (is_bf16) return src_f32 ? GO(bf16, float) : GO(bf16, bf16);
-  return GO(float, float);
+  if (has_kv && !has_v && (dim != vdim || (q_out == nullptr && k_out == nullptr))) return -250;
+  if (rot < 0 || rot > dim || (rot & 1) || (rot > 0 && table == nullptr)) return -250;
+  if ((gates == GATES_HEAD && head_gate == nullptr) || (gates == GATES_ELEMENT && q_out != nullptr && g_out == nullptr)) return -250;
+  if (k_cache != nullptr && (v_cache == nullptr || block_table == nullptr || block_size <= 0)) return -250;
+  AttnPrep p = {ld, rows, heads, kv_heads, dim, vdim, has_kv, has_kv && has_v, gates, eps, positions, tok_slot, temp, temp_len, q_w,
+                k_w, rot, halves, (const float2*)table, table_len, head_gate, k_cache ? block_table : nullptr, max_blocks, block_size};
+  const int units = heads + (has_kv ? kv_heads * (has_v ? 2 : 1) : 0) + (gates == GATES_ELEMENT && q_out != nullptr ? heads : 0) +
+                    (gates == GATES_HEAD ? 1 : 0);
+  const dim3 grid(whole ? (unsigned)rows : (unsigned)(((long long)rows * units + 7) / 8));
+  const dim3 blk(!whole ? 256 : units >= 16 ? 512 : units >= 8 ? 256 : 128);
+#define GO(TT, SS, WW) (int)trlb_host::launch_kernel(attn_prep_kernel<TT, SS, WW>, grid, blk, 0, st, PDL, p, (SS*)src, (TT*)q_out, (TT*)k_out, \
+                                                     (TT*)g_out, (TT*)k_cache, (TT*)v_cache)
+  if (is_bf16) return src_f32 ? (whole ? GO(bf16, float, true) : GO(bf16, float, false)) : (whole ? GO(bf16, bf16, true) : GO(bf16, bf16, false));
+  return whole ? GO(float, float, true) : GO(float, float, false);
 #undef GO
 }
 
 // Arguments as trlb_mixer_attn_tc (mixer_attn_tcgen05.cu), in either dtype and any size; positions instead of sequence starts.
 TRLB_API int trlb_mixer_attn(const void* q, long long q_ld, const void* k, long long k_ld, const void* v, long long v_ld,
                              const void* krot, long long krot_ld, const int* positions, int T, int heads, int kv_heads, int dim,
-                             int rot, int vdim, int window, float scale, float cap, const float* sink, int gate_mode,
+                             int rot, int vdim, int window, int keep, float scale, float cap, const float* sink, int gate_mode,
                              const void* gate, long long gate_ld, void* out, int is_bf16, cudaStream_t st) {
   if (T <= 0) return 0;
   if (heads <= 0 || kv_heads <= 0 || heads % kv_heads) return -251;
-  MixerAttn p = {T, heads, heads / kv_heads, dim, rot, vdim, window, q_ld, k_ld, v_ld, krot_ld, gate_ld, scale, cap, positions,
+  MixerAttn p = {T, heads, heads / kv_heads, dim, rot, vdim, window, keep, q_ld, k_ld, v_ld, krot_ld, gate_ld, scale, cap, positions,
                  sink, gate_mode, gate_mode == 1 ? (const float*)gate : nullptr};
   const int grid = (int)(((long long)T * heads + 3) / 4);
   const size_t smem = (size_t)4 * (dim + rot + vdim) * 4;
@@ -317,13 +445,15 @@ TRLB_API int trlb_mixer_attn(const void* q, long long q_ld, const void* k, long 
   return (int)cudaGetLastError();
 }
 
-// q [B, heads, dim], k_cache [blocks, block_size, kv_heads, dim], v_cache [.., vdim], gate logits [B, heads, vdim] or null.
-TRLB_API int trlb_grouped_decode(const void* q, const void* k_cache, const void* v_cache, const void* gate, void* out, int B,
-                                 int heads, int kv_heads, int dim, int vdim, float scale, float cap, const int* seq_lens,
+// q [B, heads, dim], k_cache [blocks, block_size, kv_heads, dim], v_cache [.., vdim], gate logits [B, heads, vdim] or null,
+// head_gate (factors) [B, heads] or null, sink [heads] or null.  window <= 0: unlimited, else the first `keep` keys stay visible.
+TRLB_API int trlb_grouped_decode(const void* q, const void* k_cache, const void* v_cache, const void* gate, const float* head_gate,
+                                 const float* sink, void* out, int B, int heads, int kv_heads, int dim, int vdim, int window,
+                                 int keep, float scale, float cap, const int* seq_lens,
                                  const int* block_table, int max_blocks, int block_size, int is_bf16, cudaStream_t st) {
   if (B <= 0) return 0;
   if (heads <= 0 || kv_heads <= 0 || heads % kv_heads || vdim > 32 * GD_MAX_REG) return -253;
-  GroupedDecode p = {B, heads, kv_heads, dim, vdim, max_blocks, block_size, scale, cap, seq_lens, block_table};
+  GroupedDecode p = {B, heads, kv_heads, dim, vdim, max_blocks, block_size, window, keep, scale, cap, seq_lens, block_table, sink, head_gate};
   const size_t smem = (size_t)(dim + 4 * vdim + 8) * 4;
   if (smem > 48 * 1024) return -253;
   const dim3 grid(heads, B), blk(128);

@@ -10,7 +10,9 @@
 // its remainder in columns 8-15 of the same product (which has 16 columns anyway), and the two results are added.  A
 // persistent CTA per SM: warp 0 = TMA producer over a ring of K + V tiles, warp 1 = MMA issuer (S^T double-buffered in TMEM),
 // warps 2-5 = softmax (one thread per token) and output accumulation (one thread per value dimension, SLABS of 128).
-// Scores may be capped (cap tanh(s / cap)); the result may be multiplied by the sigmoid of per-element gate logits.
+// Scores may be capped (cap tanh(s / cap)); the softmax denominator may contain exp(sink[head]); the result may be multiplied by
+// the sigmoid of per-element gate logits or by a factor per head.  With a window only its tiles and those of the first `keep`
+// tokens, which stay visible, are read: the tiles of a slot are a list, kept ones first.
 // Splits leave fp32 partial sums that grouped_combine_kernel merges.
 #include "mixers.cuh"
 
@@ -33,6 +35,9 @@ struct GroupedDecodeTc {
   float* part_o;              // [B, heads, splits, vdim]
   float2* part_ml;            // [B, heads, splits] (maximum in log2 units, sum)
   int* status;
+  int window, keep;           // window 0: unlimited
+  const float* sink;          // [heads] or null
+  const float* head_gate;     // [B, heads] or null
 };
 
 __device__ __forceinline__ bool gt_vote(bool pred) {
@@ -48,8 +53,22 @@ __device__ __forceinline__ bool gt_vote(bool pred) {
   return out != 0;
 }
 
+// What sums of weight L below a maximum m (log2 units) are multiplied by: the sink joins the denominator.
+__device__ __forceinline__ float gt_factor(float m, float L, const float* sink, const float* head_gate, int h, size_t bh) {
+  float f;
+  if (sink != nullptr) {
+    const float sk = sink[h] * 1.4426950408889634f, mt = fmaxf(m, sk), wm = fast_exp2(m - mt);
+    f = wm / (L * wm + fast_exp2(sk - mt));
+  } else {
+    f = L > 0.f ? 1.f / L : 0.f;
+  }
+  return head_gate != nullptr ? f * head_gate[bh] : f;
+}
+
 struct GtItem {
-  int b, kvh, h0, nh, sp, len, t0, t1;
+  int b, kvh, h0, nh, sp, len, t0, t1;  // t0 .. t1: places in the slot's list of tiles
+  int lo, kt;                           // first tile of the window, kept tiles before it
+  __device__ __forceinline__ int tile(int t) const { return t < kt ? t : lo + t - kt; }
 };
 
 __device__ __forceinline__ GtItem gt_item(const GroupedDecodeTc& p, int item) {
@@ -64,7 +83,9 @@ __device__ __forceinline__ GtItem gt_item(const GroupedDecodeTc& p, int item) {
   it.nh = min(8, p.group - g0);
   const int sl = p.seq_lens[it.b];
   it.len = (sl < 0 || sl >= p.max_blocks * p.block_size) ? 0 : sl + 1;  // the new token is in the cache already
-  const int n_t = (it.len + 127) >> 7;
+  it.lo = p.window > 0 ? max(0, it.len - p.window) >> 7 : 0;
+  it.kt = min((p.keep + 127) >> 7, it.lo);
+  const int n_t = it.kt + ((it.len + 127) >> 7) - it.lo;
   it.t0 = n_t * it.sp / p.splits;
   it.t1 = n_t * (it.sp + 1) / p.splits;
   return it;
@@ -152,7 +173,7 @@ grouped_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_
           mbar_expect_tx(&full_bar[stage], (uint32_t)(p.nk + p.nv) * GT_BOX);
           for (int g = 0; g < ppt; ++g) {
             // pages past the sequence's last one: that one again, its scores are masked
-            const int row = bt[min(t * ppt + g, last_page)] * p.block_size;
+            const int row = bt[min(it.tile(t) * ppt + g, last_page)] * p.block_size;
             uint8_t* dst = st + g * p.block_size * 128;
             for (int i = 0; i < p.nk; ++i) tma_load_3d(dst + i * GT_BOX, &tm_k, &full_bar[stage], 64 * i, it.kvh, row);
             for (int i = 0; i < p.nv; ++i) tma_load_3d(dst + k_bytes + i * GT_BOX, &tm_v, &full_bar[stage], 64 * i, it.kvh, row);
@@ -275,7 +296,8 @@ grouped_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_
 #pragma unroll
             for (int g = 0; g < 8; ++g) s[g] = p.cap_out * (far ? tanh_exp(s[g]) : tanh_series(s[g]));
           }
-          const bool valid = t * 128 + row < it.len;
+          const int tok = it.tile(t) * 128 + row;
+          const bool valid = tok < it.len && (p.window == 0 || tok >= it.len - p.window || tok < p.keep);
 #pragma unroll
           for (int g = 0; g < 8; ++g) {
             s[g] = valid ? s[g] * p.scale_log2 : -INFINITY;
@@ -329,12 +351,13 @@ grouped_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_
         if (g >= it.nh) break;
         const size_t bh = (size_t)it.b * p.heads + it.h0 + g;
         const float L = red_l[g] + red_l[8 + g] + red_l[16 + g] + red_l[24 + g];
+        const float f = p.splits == 1 ? gt_factor(mrun[g], L, p.sink, p.head_gate, it.h0 + g, bh) : 0.f;
 #pragma unroll
         for (int sl = 0; sl < SLABS; ++sl) {
           const int d = sl * 128 + row;
           if (d >= p.vdim) continue;
           if (p.splits == 1) {
-            float o = acc[sl][g] / L;
+            float o = acc[sl][g] * f;
             if (p.gate != nullptr) o *= fast_sigmoid(__bfloat162float(p.gate[bh * p.vdim + d]));
             p.out[bh * p.vdim + d] = __float2bfloat16(o);
           } else {
@@ -361,7 +384,8 @@ grouped_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_
 // One block per (head, slot).
 __global__ void __launch_bounds__(128)
 grouped_combine_kernel(const float* __restrict__ part_o, const float2* __restrict__ part_ml, const __nv_bfloat16* __restrict__ gate,
-                       const int* __restrict__ seq_lens, int heads, int vdim, int splits, __nv_bfloat16* __restrict__ out) {
+                       const int* __restrict__ seq_lens, const float* __restrict__ sink, const float* __restrict__ head_gate, int heads,
+                       int vdim, int splits, __nv_bfloat16* __restrict__ out) {
   pdl_launch_dependents();
   pdl_wait();
   const int h = blockIdx.x, b = blockIdx.y;
@@ -373,13 +397,14 @@ grouped_combine_kernel(const float* __restrict__ part_o, const float2* __restric
     const float2 ml = part_ml[bh * splits + s];
     if (ml.y > 0.f) den += ml.y * fast_exp2(ml.x - m);
   }
+  const float f = gt_factor(m, den, sink, head_gate, h, bh);
   for (int d = threadIdx.x; d < vdim; d += 128) {
     float o = 0.f;
     for (int s = 0; s < splits; ++s) {
       const float2 ml = part_ml[bh * splits + s];
       if (ml.y > 0.f) o = fmaf(part_o[(bh * splits + s) * vdim + d], fast_exp2(ml.x - m), o);
     }
-    o = den > 0.f ? o / den : 0.f;
+    o *= f;
     if (gate != nullptr) o *= fast_sigmoid(__bfloat162float(gate[bh * vdim + d]));
     out[bh * vdim + d] = __float2bfloat16(o);
   }
@@ -413,10 +438,11 @@ TRLB_API int trlb_grouped_decode_tc_ok(int heads, int kv_heads, int dim, int vdi
 TRLB_API int trlb_grouped_decode_tc_items(int B, int heads, int kv_heads) { return B * kv_heads * ((heads / kv_heads + 7) / 8); }
 
 // q [B, heads, dim], caches [num_blocks, block_size, kv_heads, dim / vdim], gate logits [B, heads, vdim] or null; one new token per
-// slot, in the cache already.  cap <= 0: none.  splits > 1: part_o [B, heads, splits, vdim], part_ml [B, heads, splits, 2] fp32.
+// slot, in the cache already.  window <= 0: unlimited, else the first `keep` tokens stay visible; cap <= 0: none; sink [heads] and
+// head_gate [B, heads] may be null.  splits > 1: part_o [B, heads, splits, vdim], part_ml [B, heads, splits, 2] fp32.
 TRLB_API int trlb_grouped_decode_tc(const void* q, const void* k_cache, const void* v_cache, const void* gate, void* out,
-                                    int num_blocks, int B, int heads, int kv_heads, int dim, int vdim, float scale, float cap,
-                                    const int* seq_lens, const int* block_table, int max_blocks, int block_size, int splits,
+                                    int num_blocks, int B, int heads, int kv_heads, int dim, int vdim, int window, int keep,
+                                    float scale, float cap, const float* sink, const float* head_gate, const int* seq_lens, const int* block_table, int max_blocks, int block_size, int splits,
                                     float* part_o, float* part_ml, int* status, cudaStream_t st) {
   if (B <= 0) return 0;
   if (!(scale > 0.f) || splits < 1 || !trlb_grouped_decode_tc_ok(heads, kv_heads, dim, vdim, block_size)) return -280;
@@ -431,6 +457,7 @@ TRLB_API int trlb_grouped_decode_tc(const void* q, const void* k_cache, const vo
   p.scale_log2 = cap > 0.f ? 1.f : scale * 1.4426950408889634f;
   p.cap_in = cap > 0.f ? scale / cap : 0.f;
   p.cap_out = cap * 1.4426950408889634f;
+  p.window = window > 0 ? window : 0; p.keep = window > 0 && keep > 0 ? keep : 0; p.sink = sink; p.head_gate = head_gate;
   p.part_o = part_o; p.part_ml = (float2*)part_ml; p.status = status;
   CUtensorMap tk, tv;
   using trlb_host::make_tmap_3d_bf16;
@@ -453,5 +480,5 @@ TRLB_API int trlb_grouped_decode_tc(const void* q, const void* k_cache, const vo
                      : (int)trlb_host::launch_kernel(grouped_decode_tc_kernel<2>, grid, blk, smem, st, pdl, tk, tv, p);
   if (rc || splits == 1) return rc;
   return (int)trlb_host::launch_kernel(grouped_combine_kernel, dim3(heads, B), dim3(128), 0, st, pdl, (const float*)part_o,
-                                       (const float2*)part_ml, p.gate, seq_lens, heads, vdim, splits, p.out);
+                                       (const float2*)part_ml, p.gate, seq_lens, sink, head_gate, heads, vdim, splits, p.out);
 }

@@ -13,12 +13,13 @@
 //     straight from the source rank's buffer over NVLink (no cluster sharing of those tiles), and the output rows are
 //     stored straight into a destination rank's buffer, so the dispatch all-to-all rides on the loads of the first GEMM
 //     and the combine all-to-all on the stores of the second;
-//   * optional SwiGLU epilogue for the gate/up projection: the B tile is 128 gate rows + the matching 128 up rows, the
-//     epilogue writes silu(gate) * up, so the [tokens, 2I] intermediate never reaches memory.
+//   * optional gated epilogue for the gate/up projection: the B tile is 128 gate rows + the matching 128 up rows, the
+//     epilogue writes silu(gate) * up (or the clamped unit g sigmoid(alpha g) (u + shift) of g = min(gate, limit), u = up
+//     clamped to [-limit, limit]), so the [tokens, 2I] intermediate never reaches memory.
 //
 // Replaces the per-expert loop of transformers' MoE blocks that the reference trains through
 // (trl/trainer/grpo_trainer.py forward of Qwen3-MoE style models).
-#include "common.cuh"
+#include "mixers.cuh"
 
 namespace trlb {
 
@@ -34,7 +35,8 @@ struct TmapArray {
 
 struct GroupedParams {
   int E, N, K, n_tiles, k_blocks;
-  int swiglu;          // 1: W is [E, 2*N, K] (gate rows then up rows), C gets N columns
+  int swiglu;          // 1: W is [E, 2*N, K] (gate rows then up rows), C gets N columns; 2: so with the clamped unit
+  float glu_limit, glu_alpha, glu_shift;
   int b_mn;            // 1: W is [E, K, N] (the weight of the forward pass read transposed: input gradient)
   const int* offsets;  // [E + 1] row offsets into A / C (plain mode)
   __nv_bfloat16* C;
@@ -53,6 +55,20 @@ struct GroupedParams {
 };
 
 __device__ __forceinline__ float silu_f(float x) { return x / (1.f + __expf(-x)); }
+
+// In place: g = the gated unit of g and u.
+__device__ __forceinline__ void gg_unit(const GroupedParams& p, float (&g)[32], const float (&u)[32]) {
+  if (p.swiglu == 2) {
+#pragma unroll
+    for (int i = 0; i < 32; ++i) {
+      const float a = fminf(g[i], p.glu_limit), b = fminf(fmaxf(u[i], -p.glu_limit), p.glu_limit);
+      g[i] = a * fast_sigmoid(p.glu_alpha * a) * (b + p.glu_shift);
+    }
+  } else {
+#pragma unroll
+    for (int i = 0; i < 32; ++i) g[i] = silu_f(g[i]) * u[i];
+  }
+}
 
 __global__ void __launch_bounds__(G_THREADS, 1)
 grouped_gemm_kernel(const __grid_constant__ TmapArray tmaps_a, const __grid_constant__ CUtensorMap tmap_b,
@@ -211,19 +227,16 @@ grouped_gemm_kernel(const __grid_constant__ TmapArray tmaps_a, const __grid_cons
           tmem_ld_wait();
           if (row_ok && col0 + c < p.N) {
             __nv_bfloat16* dst = cbase + (long long)(crow0 + r) * p.ldc + col0 + c;
+            gg_unit(p, g, u);
             if (col0 + c + 32 <= p.N && ((reinterpret_cast<uintptr_t>(dst) & 15) == 0)) {
 #pragma unroll
-              for (int i = 0; i < 32; i += 8) {
-                uint4 o;
-                o.x = pack_bf16(silu_f(g[i]) * u[i], silu_f(g[i + 1]) * u[i + 1]);
-                o.y = pack_bf16(silu_f(g[i + 2]) * u[i + 2], silu_f(g[i + 3]) * u[i + 3]);
-                o.z = pack_bf16(silu_f(g[i + 4]) * u[i + 4], silu_f(g[i + 5]) * u[i + 5]);
-                o.w = pack_bf16(silu_f(g[i + 6]) * u[i + 6], silu_f(g[i + 7]) * u[i + 7]);
-                *reinterpret_cast<uint4*>(dst + i) = o;
-              }
+              for (int i = 0; i < 32; i += 8)
+                *reinterpret_cast<uint4*>(dst + i) = make_uint4(pack_bf16(g[i], g[i + 1]), pack_bf16(g[i + 2], g[i + 3]),
+                                                                pack_bf16(g[i + 4], g[i + 5]), pack_bf16(g[i + 6], g[i + 7]));
             } else {
+#pragma unroll
               for (int i = 0; i < 32; ++i)
-                if (col0 + c + i < p.N) dst[i] = __float2bfloat16(silu_f(g[i]) * u[i]);
+                if (col0 + c + i < p.N) dst[i] = __float2bfloat16(g[i]);
             }
           }
         }
@@ -470,14 +483,15 @@ grouped_wgrad_kernel(const __grid_constant__ CUtensorMap tmap_g, const __grid_co
 using namespace trlb;
 
 // A [rows, K] bf16 (row stride lda), rows sorted by expert; W [E, Nw, K] bf16 contiguous with Nw = N (plain) or
-// 2 * N (swiglu: gate rows then up rows); offsets [E + 1] int32 on the device; C [rows, N] bf16 (row stride ldc).
+// 2 * N (swiglu: gate rows then up rows; 2: the clamped unit with glu = {limit, alpha, shift}); offsets [E + 1] int32 on the device; C [rows, N] bf16 (row stride ldc).
 // `rows` is the allocated row count of A and C (an upper bound of offsets[E]).
 // `w_transposed` = 1: W is [E, K, N] and C[r, :] = A[r, :] . W[e] (the forward weight read transposed, for the
 // input gradient); N must then be a multiple of 8 and swiglu 0.
 TRLB_API int trlb_grouped_gemm_bf16(const void* A, const void* W, const int* offsets, void* C, long long rows, int E, int N,
-                                    int K, long long lda, long long ldc, int swiglu, int w_transposed, int* status,
-                                    cudaStream_t st) {
+                                    int K, long long lda, long long ldc, int swiglu, const float* glu, int w_transposed,
+                                    int* status, cudaStream_t st) {
   if (rows <= 0 || E <= 0) return 0;
+  if (swiglu < 0 || swiglu > 2 || (swiglu == 2 && glu == nullptr)) return -130;
   if (E > G_MAX_EXPERTS || (K % 8) != 0 || (lda % 8) != 0) return -130;
   if (w_transposed && (swiglu || (N % 8) != 0)) return -130;
   const long long Nw = swiglu ? 2LL * N : N;
@@ -498,6 +512,7 @@ TRLB_API int trlb_grouped_gemm_bf16(const void* A, const void* W, const int* off
   }
   GroupedParams p = {};
   p.E = E; p.N = N; p.K = K; p.swiglu = swiglu; p.b_mn = w_transposed ? 1 : 0;
+  if (swiglu == 2) { p.glu_limit = glu[0]; p.glu_alpha = glu[1]; p.glu_shift = glu[2]; }
   p.n_tiles = swiglu ? (N + 127) / 128 : (N + GBN - 1) / GBN;
   p.k_blocks = (K + GBK - 1) / GBK;
   p.offsets = offsets; p.C = (__nv_bfloat16*)C; p.ldc = ldc; p.status = status;

@@ -21,7 +21,8 @@
 //   * the softmax denominator may contain exp(sink[head]);
 //   * the output may be multiplied by a gate: one fp32 factor per token and head, or the sigmoid of bf16 logits per
 //     element;
-//   * keys are those of the same sequence, with a window those at distance < window.
+//   * keys are those of the same sequence, with a window those at distance < window and the first `keep` of the sequence: the
+//     tiles of a CTA are those that hold kept keys, then those of the window.
 #include "mixers.cuh"
 
 namespace trlb {
@@ -34,7 +35,7 @@ enum { GATE_NONE = 0, GATE_HEAD = 1, GATE_LOGITS = 2 };
 
 struct MixerAttnTc {
   const int* cu;
-  int n_seq, heads, group, dim, rot, vdim, window;
+  int n_seq, heads, group, dim, rot, vdim, window, keep;
   int nn, nr, nv;      // boxes of the unrotated part, the rotated part and the value
   int k_stages, v_stages;
   float scale_log2;    // CAP: 1 (capped scores are in log2 units already)
@@ -70,20 +71,29 @@ __device__ __forceinline__ float la_capped(const MixerAttnTc& p, float v) {
   return v * fmaf(z, t, p.poly[0]);
 }
 
+// Bits of the 32 scores from column c on that a row sees: first .. last, and the columns before `kept`.
+__device__ __forceinline__ uint32_t la_visible(int c, int first, int last, int kept) {
+  const int n = min(last - c, 31), k = min(kept - 1 - c, n), f = max(first - c, 0);
+  uint32_t m = n >= f ? (0xffffffffu >> (31 - n)) & (0xffffffffu << f) : 0u;
+  if (k >= 0) m |= 0xffffffffu >> (31 - k);
+  return m;
+}
+
 // First pass over a row of scores: the largest visible one and (SPAN) the largest magnitude of any.  Loops over 32 scores stay
 // rolled and tiles without masked keys have code of their own: instruction fetch and count are what limits these passes.
 template <bool SPAN, bool FULL>
-__device__ __forceinline__ float2 la_row_max(uint32_t ts, int first, int last) {
+__device__ __forceinline__ float2 la_row_max(uint32_t ts, int first, int last, int kept) {
   float mx[2] = {-INFINITY, -INFINITY}, mn[2] = {INFINITY, INFINITY};
 #pragma unroll 1
   for (int c = 0; c < 128; c += 32) {
     float v[32];
     tmem_ld_32x32(ts + c, v);
+    const uint32_t seen = FULL ? 0u : la_visible(c, first, last, kept);
     tmem_ld_wait();
 #pragma unroll
     for (int i = 0; i < 32; ++i) {
       if (SPAN) mn[i & 1] = fminf(mn[i & 1], FULL ? v[i] : -fabsf(v[i]));
-      mx[i & 1] = fmaxf(mx[i & 1], FULL || (c + i >= first && c + i <= last) ? v[i] : -INFINITY);
+      mx[i & 1] = fmaxf(mx[i & 1], FULL || (seen >> i & 1u) ? v[i] : -INFINITY);
     }
   }
   const float m = fmaxf(mx[0], mx[1]);
@@ -92,19 +102,20 @@ __device__ __forceinline__ float2 la_row_max(uint32_t ts, int first, int last) {
 
 // Second pass: probabilities, as value and remainder, in place.  LEVEL -1: no cap.  Returns their sum.
 template <int LEVEL, bool FULL>
-__device__ __forceinline__ float la_probs(const MixerAttnTc& p, uint32_t ts, float neg_m, int first, int last) {
+__device__ __forceinline__ float la_probs(const MixerAttnTc& p, uint32_t ts, float neg_m, int first, int last, int kept) {
   float sum[2] = {0.f, 0.f};
 #pragma unroll 1
   for (int c = 0; c < 128; c += 32) {
     float v[32];
     tmem_ld_32x32(ts + c, v);
+    const uint32_t seen = FULL ? 0u : la_visible(c, first, last, kept);
     tmem_ld_wait();
     uint32_t a[16], b[16];
 #pragma unroll
     for (int i = 0; i < 32; ++i) {
       if (LEVEL < 0) v[i] = fast_exp2(fmaf(v[i], p.scale_log2, neg_m));
       else v[i] = fast_exp2(la_capped<LEVEL < 0 ? 0 : LEVEL>(p, v[i]) + neg_m);
-      if (!FULL) v[i] = c + i >= first && c + i <= last ? v[i] : 0.f;
+      if (!FULL) v[i] = seen >> i & 1u ? v[i] : 0.f;
       sum[i & 1] += v[i];
     }
 #pragma unroll
@@ -152,7 +163,9 @@ mixer_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_con
   const int q_last = min(len, q_first + LA_BM) - 1;
   const int hi = q_last / LA_BN;
   const int lo = p.window > 0 ? max(0, q_first - p.window + 1) / LA_BN : 0;
-  const int n_kv = hi - lo + 1;  // >= 1: a token sees itself
+  const int kt = min((p.keep + LA_BN - 1) / LA_BN, lo);  // tiles of kept keys before the window
+  const int n_kv = kt + hi - lo + 1;  // >= 1: a token sees itself
+  auto tile_at = [&](int j) { return j < kt ? j : lo + j - kt; };
 
   if (threadIdx.x == 0) {
     mbar_init(q_full, 1);
@@ -192,7 +205,7 @@ mixer_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_con
         const int s = j % p.k_stages;
         if (!mbar_wait(&k_empty[s], (uint32_t)(((j / p.k_stages) & 1) ^ 1), abort_flag, p.status, 1200 + s)) return false;
         uint8_t* ks = k_s + (size_t)s * k_bytes;
-        const int row = beg + (lo + j) * LA_BN;
+        const int row = beg + tile_at(j) * LA_BN;
         mbar_expect_tx(&k_full[s], k_bytes);
         for (int i = 0; i < p.nn; ++i) tma_load_3d(ks + i * LA_BOX, &tm_kn, &k_full[s], 64 * i, hk, row);
         for (int i = 0; i < p.nr; ++i) tma_load_2d(ks + (p.nn + i) * LA_BOX, &tm_kr, &k_full[s], 64 * i, row);
@@ -206,7 +219,7 @@ mixer_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_con
         if (!mbar_wait(&v_empty[s], (uint32_t)(((j / p.v_stages) & 1) ^ 1), abort_flag, p.status, 1205 + s)) break;
         uint8_t* vs = v_s + (size_t)s * v_bytes;
         mbar_expect_tx(&v_full[s], v_bytes);
-        for (int i = 0; i < p.nv; ++i) tma_load_3d(vs + i * LA_BOX, &tm_v, &v_full[s], 64 * i, hk, beg + (lo + j) * LA_BN);
+        for (int i = 0; i < p.nv; ++i) tma_load_3d(vs + i * LA_BOX, &tm_v, &v_full[s], 64 * i, hk, beg + tile_at(j) * LA_BN);
         if (NB == 1 && j + 1 < n_kv) ok = load_k(j + 1);  // one stage: free only after S(j)
       }
     }
@@ -274,15 +287,15 @@ mixer_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_con
     bool ok = true;
     for (int j = 0; j < n_kv && ok; ++j) {
       const int s = j % NB;
-      const int key0 = (lo + j) * LA_BN;
+      const int key0 = tile_at(j) * LA_BN;
       const bool full = q_first + LA_BM <= len && key0 + LA_BN - 1 <= q_first &&
-                        (p.window <= 0 || key0 >= q_first + LA_BM - p.window);
+                        (p.window <= 0 || key0 >= q_first + LA_BM - p.window || key0 + LA_BN <= p.keep);
       ok = __all_sync(0xffffffffu, mbar_wait(&s_full[s], (uint32_t)((j / NB) & 1), abort_flag, p.status, 1270 + s));
       if (!ok) break;
       tc_fence_after();
       const uint32_t ts = tmem_base + lane_off + (uint32_t)s * LA_BN;
-      const int first = k_min - key0, last = k_max - key0;
-      const float2 top = full ? la_row_max<CAP, true>(ts, first, last) : la_row_max<CAP, false>(ts, first, last);
+      const int first = k_min - key0, last = k_max - key0, kept = p.keep - key0;
+      const float2 top = full ? la_row_max<CAP, true>(ts, first, last, kept) : la_row_max<CAP, false>(ts, first, last, kept);
       const float mx = top.x;
       int level = -1;
       float m_tile = mx * p.scale_log2;
@@ -317,10 +330,10 @@ mixer_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_con
       l_run *= alpha;
       const float neg_m = m_ref == -INFINITY ? 0.f : -m_ref;
       float sum;
-      if (!CAP) sum = full ? la_probs<-1, true>(p, ts, neg_m, first, last) : la_probs<-1, false>(p, ts, neg_m, first, last);
-      else if (level == 0) sum = full ? la_probs<0, true>(p, ts, neg_m, first, last) : la_probs<0, false>(p, ts, neg_m, first, last);
-      else if (level == 1) sum = la_probs<1, false>(p, ts, neg_m, first, last);
-      else sum = la_probs<2, false>(p, ts, neg_m, first, last);
+      if (!CAP) sum = full ? la_probs<-1, true>(p, ts, neg_m, first, last, kept) : la_probs<-1, false>(p, ts, neg_m, first, last, kept);
+      else if (level == 0) sum = full ? la_probs<0, true>(p, ts, neg_m, first, last, kept) : la_probs<0, false>(p, ts, neg_m, first, last, kept);
+      else if (level == 1) sum = la_probs<1, false>(p, ts, neg_m, first, last, kept);
+      else sum = la_probs<2, false>(p, ts, neg_m, first, last, kept);
       // P.V(last) completes phase `last` of o_full, and may do so before this thread looks: phase last - 1 has to be seen
       // first.  (With one S buffer the last S was issued after P.V(last - 1), so s_full has shown it.)
       if (NB == 2 && j > 0 && j == n_kv - 1)
@@ -426,18 +439,19 @@ TRLB_API int trlb_mixer_attn_tc_ok(int heads, int kv_heads, int dim, int rot, in
 }
 
 // q [T rows of q_ld]: heads x (dim + rot), rotated part last; k, v [T rows of k_ld / v_ld]: kv_heads x dim / vdim; krot [T rows
-// of krot_ld]: the shared rotated keys (rot > 0).  All bf16, rows on 16 bytes.  window <= 0: unlimited; cap <= 0: none; scale > 0;
+// of krot_ld]: the shared rotated keys (rot > 0).  All bf16, rows on 16 bytes.  window <= 0: unlimited, else the first `keep` keys stay
+// visible; cap <= 0: none; scale > 0;
 // sink may be null; gate by gate_mode (0 none, 1 fp32 [T, heads], 2 bf16 logits [T rows of gate_ld]).
 TRLB_API int trlb_mixer_attn_tc(const void* q, long long q_ld, const void* k, long long k_ld, const void* v, long long v_ld,
                                 const void* krot, long long krot_ld, const int* cu, int n_seq, int T, int heads, int kv_heads,
-                                int dim, int rot, int vdim, int window, float scale, float cap, const float* sink,
+                                int dim, int rot, int vdim, int window, int keep, float scale, float cap, const float* sink,
                                 int gate_mode, const void* gate, long long gate_ld, void* out, int* status, cudaStream_t st) {
   if (T <= 0 || n_seq <= 0) return 0;
   if (!trlb_mixer_attn_tc_ok(heads, kv_heads, dim, rot, vdim) || (q_ld % 8) || (k_ld % 8) || (v_ld % 8) || !(scale > 0.f)) return -210;
   if (rot > 0 && (krot_ld % 8)) return -210;
   if (gate_mode == GATE_LOGITS && ((gate_ld % 8) || (reinterpret_cast<uintptr_t>(gate) & 15))) return -210;
   MixerAttnTc p = {};
-  p.cu = cu; p.n_seq = n_seq; p.heads = heads; p.group = heads / kv_heads; p.dim = dim; p.rot = rot; p.vdim = vdim; p.window = window;
+  p.cu = cu; p.n_seq = n_seq; p.heads = heads; p.group = heads / kv_heads; p.dim = dim; p.rot = rot; p.vdim = vdim; p.window = window; p.keep = window > 0 && keep > 0 ? keep : 0;
   p.nn = la_boxes(dim); p.nr = la_boxes(rot); p.nv = la_boxes(vdim);
   const bool pair = la_pair(p.nn + p.nr, p.nv, vdim);
   if (pair) p.k_stages = p.v_stages = 1;

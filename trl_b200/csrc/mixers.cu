@@ -34,6 +34,55 @@ embed_scaled_kernel(const long long* __restrict__ ids, const T* __restrict__ emb
     x[(size_t)blockIdx.x * H + j] = (id >= 0 && id < V) ? to_f(emb[(size_t)id * H + j]) * scale : 0.f;
 }
 
+// The same plus a row of a table of token pairs: row (previous * mul_prev + current * mul_cur) mod buckets, or the last row,
+// number `buckets`, at a sequence's first token.  Prompt rows (prev_state is written by a sequence's last row, tok_slot gives
+// the slots; both may be null) take the previous token from ids; decode rows (one per slot, positions negative: idle) from
+// prev_state, which moves on.
+struct PairEmbed {
+  const long long* ids;
+  const int* positions;
+  const int* tok_slot;
+  long long* prev_state;
+  long long mul_prev, mul_cur, buckets;
+  int T, H, V, decode;
+  float scale;
+};
+
+template <typename T>
+__global__ void __launch_bounds__(256)
+embed_pairs_kernel(const PairEmbed p, const T* __restrict__ emb, const T* __restrict__ pairs, float* __restrict__ x) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int r = blockIdx.x, pos = p.positions[r];
+  const long long id = p.ids[r];
+  const bool ok = id >= 0 && id < p.V;
+  long long prev = -1;
+  if (pos > 0) prev = p.decode ? p.prev_state[r] : p.ids[r - 1];
+  long long row = p.buckets;
+  if (prev >= 0) {
+    row = (prev * p.mul_prev + id * p.mul_cur) % p.buckets;
+    if (row < 0) row += p.buckets;
+  }
+  const T* e = emb + (size_t)(ok ? id : 0) * p.H;
+  const T* g = pairs + (size_t)row * p.H;
+  float* o = x + (size_t)r * p.H;
+  if ((p.H & 3) == 0) {
+    for (int j = 4 * threadIdx.x; j < p.H; j += 4 * blockDim.x) {
+      const float4 a = ok ? load4(e + j) : make_float4(0.f, 0.f, 0.f, 0.f), b = load4(g + j);
+      store4(o + j, make_float4(a.x * p.scale + b.x, a.y * p.scale + b.y, a.z * p.scale + b.z, a.w * p.scale + b.w));
+    }
+  } else {
+    for (int j = threadIdx.x; j < p.H; j += blockDim.x) o[j] = (ok ? to_f(e[j]) * p.scale : 0.f) + to_f(g[j]);
+  }
+  if (p.prev_state == nullptr || pos < 0) return;
+  if (p.decode) {
+    __syncthreads();  // everyone has read the old one
+    if (threadIdx.x == 0) p.prev_state[r] = id;
+  } else if (threadIdx.x == 0 && (r + 1 == p.T || p.positions[r + 1] == 0)) {
+    p.prev_state[p.tok_slot[r]] = id;
+  }
+}
+
 // x (+= delta) ; out = tanh(alpha x) w + b.  VEC elements per thread along H (H % VEC == 0).
 template <typename T, int VEC>
 __global__ void __launch_bounds__(256)
@@ -84,9 +133,9 @@ gelu_erf_kernel(const T* __restrict__ z, T* __restrict__ out, long long n) {
 
 // ------------------------------------------------------------------------------------------------------------
 // RMS norms around the residual stream, in one pass over a row:
-//     x += delta                      or, with `post`,   x += delta / rms(delta) * post
-//     out = x / rms(x) * w            or, without `w`,   out = x
-// `clear` zeroes delta behind itself.  One block per row; NV float4 of the row live in each thread's registers.
+//     x += delta                      or, with `post`,   x += delta / rms(delta) * (shift + post) * post_scale
+//     out = x / rms(x) * (shift + w) * gain              or, without `w`,   out = x
+// (no post_scale: 1).  `clear` zeroes delta behind itself.  One block per row; NV float4 of the row live in each thread's registers.
 // ------------------------------------------------------------------------------------------------------------
 struct RmsResidual {
   float* x;
@@ -95,7 +144,19 @@ struct RmsResidual {
   const float* w;      // null: the sum itself is the output
   int H, clear;
   float eps;
+  const float* post_scale;  // null: 1
+  float shift, gain;
 };
+
+__device__ __forceinline__ float4 rms_weight4(const float* w, const float* scale, float shift, float gain, int j) {
+  float4 g = load4(w + j);
+  g = make_float4((shift + g.x) * gain, (shift + g.y) * gain, (shift + g.z) * gain, (shift + g.w) * gain);
+  if (scale != nullptr) {
+    const float4 c = load4(scale + j);
+    g = make_float4(g.x * c.x, g.y * c.y, g.z * c.z, g.w * c.w);
+  }
+  return g;
+}
 
 template <typename T, int NV>
 __global__ void __launch_bounds__(256)
@@ -125,7 +186,7 @@ rms_residual_kernel(const RmsResidual p, T* __restrict__ out) {
     for (int i = 0; i < NV; ++i) {
       const int j = threadIdx.x + i * nt;
       if (j < n4) {
-        const float4 g = p.post != nullptr ? load4(p.post + 4 * j) : make_float4(1.f, 1.f, 1.f, 1.f);
+        const float4 g = p.post != nullptr ? rms_weight4(p.post, p.post_scale, p.shift, 1.f, 4 * j) : make_float4(1.f, 1.f, 1.f, 1.f);
         a[i].x += d[i].x * r * g.x; a[i].y += d[i].y * r * g.y; a[i].z += d[i].z * r * g.z; a[i].w += d[i].w * r * g.w;
         store4(p.x + row + 4 * j, a[i]);
         if (p.clear) store4(p.delta + row + 4 * j, make_float4(0.f, 0.f, 0.f, 0.f));
@@ -143,7 +204,7 @@ rms_residual_kernel(const RmsResidual p, T* __restrict__ out) {
   for (int i = 0; i < NV; ++i) {
     const int j = threadIdx.x + i * nt;
     if (j < n4) {
-      const float4 g = p.w != nullptr ? load4(p.w + 4 * j) : make_float4(1.f, 1.f, 1.f, 1.f);
+      const float4 g = p.w != nullptr ? rms_weight4(p.w, nullptr, p.shift, p.gain, 4 * j) : make_float4(1.f, 1.f, 1.f, 1.f);
       store4(out + row + 4 * j, make_float4(a[i].x * r * g.x, a[i].y * r * g.y, a[i].z * r * g.z, a[i].w * r * g.w));
     }
   }
@@ -168,7 +229,7 @@ rms_residual_any_kernel(const RmsResidual p, T* __restrict__ out) {
   for (int j = threadIdx.x; j < p.H; j += 256) {
     float a = x[j];
     if (d != nullptr) {
-      a += p.post != nullptr ? d[j] * r * p.post[j] : d[j];
+      a += p.post != nullptr ? d[j] * r * (p.shift + p.post[j]) * (p.post_scale != nullptr ? p.post_scale[j] : 1.f) : d[j];
       x[j] = a;
       if (p.clear) d[j] = 0.f;
     }
@@ -176,20 +237,21 @@ rms_residual_any_kernel(const RmsResidual p, T* __restrict__ out) {
   }
   float rx = 1.f;
   if (p.w != nullptr) rx = 1.f / sqrtf(block_sum2(s, 0.f, red).x / (float)p.H + p.eps);
-  for (int j = threadIdx.x; j < p.H; j += 256) out[row + j] = from_f<T>(p.w != nullptr ? x[j] * rx * p.w[j] : x[j]);
+  for (int j = threadIdx.x; j < p.H; j += 256) out[row + j] = from_f<T>(p.w != nullptr ? x[j] * rx * (p.shift + p.w[j]) * p.gain : x[j]);
 }
 
-// Clamped gated linear unit: z [rows, 2 n] = gate | up -> g sigmoid(alpha g) (u + shift), g = min(gate, limit), u = up clamped
-// to [-limit, limit].
-template <typename T, int VEC>
+// Gated linear units, z [rows, 2 n] = gate | up.  GELU: gelu_tanh(gate) up.  Else clamped: g sigmoid(alpha g) (u + shift), g =
+// min(gate, limit), u = up clamped to [-limit, limit].
+template <typename T, int VEC, bool GELU>
 __global__ void __launch_bounds__(256)
-clamped_glu_kernel(const T* __restrict__ z, T* __restrict__ out, long long total, int n, float limit, float alpha, float shift) {
+glu_kernel(const T* __restrict__ z, T* __restrict__ out, long long total, int n, float limit, float alpha, float shift) {
   const int per = n / VEC;
   for (long long v = blockIdx.x * (long long)blockDim.x + threadIdx.x; v < total; v += (long long)gridDim.x * blockDim.x) {
     const long long row = v / per;
     const int j = (int)(v % per) * VEC;
     const T* zr = z + row * 2 * n + j;
     auto act = [&](float g, float u) {
+      if (GELU) return gelu_tanh_t<T>(g) * u;
       g = fminf(g, limit);
       u = fminf(fmaxf(u, -limit), limit);
       return g * sigmoid_t<T>(alpha * g) * (u + shift);
@@ -736,6 +798,19 @@ TRLB_API int trlb_embed_scaled(const long long* ids, const void* emb, float* x, 
   return (int)trlb_host::launch_kernel(embed_scaled_kernel<float>, dim3(T), dim3(256), 0, st, PDL, ids, (const float*)emb, x, H, V, scale);
 }
 
+// pairs [buckets + 1, H] in the dtype of emb; prev_state [slots] (decode: one row per slot) may be null, tok_slot in decode
+TRLB_API int trlb_embed_pairs(const long long* ids, const void* emb, const void* pairs, float* x, int T, int H, int V, float scale,
+                              long long mul_prev, long long mul_cur, long long buckets, const int* positions, const int* tok_slot,
+                              long long* prev_state, int decode, int is_bf16, cudaStream_t st) {
+  if (T <= 0) return 0;
+  if (buckets <= 0 || positions == nullptr || (decode && prev_state == nullptr) || (!decode && prev_state != nullptr && tok_slot == nullptr))
+    return -207;
+  const PairEmbed p = {ids, positions, tok_slot, prev_state, mul_prev, mul_cur, buckets, T, H, V, decode, scale};
+  const dim3 blk(H >= 1024 ? 256 : 64);
+  if (is_bf16) return (int)trlb_host::launch_kernel(embed_pairs_kernel<bf16>, dim3(T), blk, 0, st, PDL, p, (const bf16*)emb, (const bf16*)pairs, x);
+  return (int)trlb_host::launch_kernel(embed_pairs_kernel<float>, dim3(T), blk, 0, st, PDL, p, (const float*)emb, (const float*)pairs, x);
+}
+
 TRLB_API int trlb_dynamic_tanh(float* x, float* delta, const float* alpha, const float* w, const float* b, void* out, int T,
                                int H, int clear, int is_bf16, cudaStream_t st) {
   if (T <= 0) return 0;
@@ -748,11 +823,11 @@ TRLB_API int trlb_dynamic_tanh(float* x, float* delta, const float* alpha, const
 #undef GO
 }
 
-// post, w, delta may be null (see RmsResidual); H: row length
-TRLB_API int trlb_rms_residual(float* x, float* delta, const float* post, const float* w, void* out, int T, int H, float eps,
-                               int clear, int is_bf16, cudaStream_t st) {
+// post, post_scale, w, delta may be null (see RmsResidual); H: row length
+TRLB_API int trlb_rms_residual(float* x, float* delta, const float* post, const float* post_scale, const float* w, void* out, int T,
+                               int H, float eps, float shift, float gain, int clear, int is_bf16, cudaStream_t st) {
   if (T <= 0) return 0;
-  const RmsResidual p = {x, delta, post, w, H, clear, eps};
+  const RmsResidual p = {x, delta, post, w, H, clear, eps, post_scale, shift, gain};
   const int n4 = H / 4;
   const bool regs = H % 4 == 0 && n4 <= 256 * 8;
 #define GO(TT, NN) (int)trlb_host::launch_kernel(rms_residual_kernel<TT, NN>, dim3(T), dim3(n4 >= 256 ? 256 : (n4 + 31) / 32 * 32), 0, st, PDL, p, (TT*)out)
@@ -769,7 +844,19 @@ TRLB_API int trlb_clamped_glu(const void* z, void* out, int rows, int n, float l
   if (rows <= 0 || n <= 0) return 0;
   const bool v4 = n % 4 == 0;
   const long long total = (long long)rows * n / (v4 ? 4 : 1);
-#define GO(TT, VV) clamped_glu_kernel<TT, VV><<<grid_for(total, 256), 256, 0, st>>>((const TT*)z, (TT*)out, total, n, limit, alpha, shift)
+#define GO(TT, VV) glu_kernel<TT, VV, false><<<grid_for(total, 256), 256, 0, st>>>((const TT*)z, (TT*)out, total, n, limit, alpha, shift)
+  if (is_bf16) { if (v4) GO(bf16, 4); else GO(bf16, 1); }
+  else { if (v4) GO(float, 4); else GO(float, 1); }
+#undef GO
+  return (int)cudaGetLastError();
+}
+
+// z [rows, 2 n] = gate | up -> gelu_tanh(gate) up
+TRLB_API int trlb_gelu_glu(const void* z, void* out, int rows, int n, int is_bf16, cudaStream_t st) {
+  if (rows <= 0 || n <= 0) return 0;
+  const bool v4 = n % 4 == 0;
+  const long long total = (long long)rows * n / (v4 ? 4 : 1);
+#define GO(TT, VV) glu_kernel<TT, VV, true><<<grid_for(total, 256), 256, 0, st>>>((const TT*)z, (TT*)out, total, n, 0.f, 0.f, 0.f)
   if (is_bf16) { if (v4) GO(bf16, 4); else GO(bf16, 1); }
   else { if (v4) GO(float, 4); else GO(float, 1); }
 #undef GO

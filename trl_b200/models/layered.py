@@ -16,6 +16,10 @@ Designs
                 ``latent_attention`` (without positions, queries straight from the input) and ``rglru`` (short convolution
                 and real-gated linear recurrence) mixers, clamped gated feed-forward, a per-token input of every layer,
                 tied head.
+    Suposun     RMS norms (weights about zero) and layer scales on the sublayers' outputs only, a table of token pairs beside the
+                embedding, ``attention`` (the projected keys are the values; weighted norms per head, YaRN rotation, window with
+                kept first tokens, capped scores, softmax sink, gate per head) and ``attention_2`` (norms over all heads, rotated
+                halves; a layer may read another one's cache) mixers, GELU-gated or expert feed-forward, tied head with a scale.
 
 The residual stream, norms, gates and recurrent states are fp32 whatever the model dtype.
 """
@@ -37,20 +41,40 @@ from .decoder import CausalLM, SeqCtx
 
 
 @dataclass(frozen=True)
+class AttentionStyle:
+    """What a design fixes about a grouped-query attention mixer."""
+
+    norm_weight: bool = False    # queries and keys over their rms times a weight
+    whole_norm: bool = False     # that norm over all heads at once instead of per head
+    halves: bool = False         # rotated pairs (i, i + dims / 2) instead of (2 i, 2 i + 1)
+    values: bool = True          # a projection of values; without it the projected keys serve as values
+    sink: bool = False           # exp(sink) in the softmax denominator
+    gate: str | None = "element"  # sigmoid gates per "element" or per "head" of the output
+
+
+@dataclass(frozen=True)
 class Design:
     """What a design fixes for all its models."""
 
     norm: str
-    mlp: str
+    mlp: str                     # dense feed-forward
+    moe: str | None = None       # feed-forward of kind 'moe'
+    pre_norm: bool = True        # a norm on the input of every sublayer; without it the sublayers read the stream itself
     post_norm: bool = False      # a norm on the output of every sublayer, before it is added
+    layer_scale: bool = False    # that norm's result times a vector
     latent_sink: bool = False    # latent_attention: exp(sink) in the softmax denominator
     latent_gate: bool = False    # latent_attention: sigmoid gate per head
+    attention: dict = field(default_factory=dict)  # AttentionStyle by mixer kind, where it is not the default one
     tied_head: bool = False
 
 
 DESIGNS: dict[str, Design] = {
     "Zorelorn": Design(norm="dynamic_tanh", mlp="gelu", latent_sink=True, latent_gate=True),
     "Povusun": Design(norm="rms", mlp="clamped_glu", post_norm=True, tied_head=True),
+    "Suposun": Design(norm="rms_about_zero", mlp="gelu_glu", moe="clamped_glu_experts", pre_norm=False, post_norm=True, layer_scale=True,
+                      tied_head=True,
+                      attention={"attention": AttentionStyle(norm_weight=True, values=False, sink=True, gate="head"),
+                                 "attention_2": AttentionStyle(norm_weight=True, whole_norm=True, halves=True, gate=None)}),
 }
 
 
@@ -65,7 +89,7 @@ class LayerSpec:
 
     @property
     def ff(self) -> int:
-        return 0 if self.mlp is None else int(self.mlp["ff"])
+        return 0 if self.mlp is None else int((self.mlp.get("expert") or self.mlp)["ff"])
 
     @property
     def key(self):
@@ -77,6 +101,8 @@ class LayeredArch(ModelArch):
     design: str = ""
     layers: list = field(default_factory=list)  # [LayerSpec]
     side_dim: int = 0  # per-token input of every layer: elements per layer (0: none)
+    pairs: dict | None = None  # table of token pairs: mul_prev, mul_cur, buckets
+    logit_scale: float = 1.0
     source: dict = field(default_factory=dict)  # the config.json this came from
 
     @classmethod
@@ -89,7 +115,7 @@ class LayeredArch(ModelArch):
             if e["type"] not in MIXERS:
                 raise ValueError(f"layer {i}: mixer {e['type']!r} is not registered; known: {sorted(MIXERS)}")
             mlp = e.get("mlp")
-            if mlp is not None and mlp.get("kind", "dense") != "dense":
+            if mlp is not None and mlp.get("kind", "dense") != "dense" and not (mlp["kind"] == "moe" and DESIGNS[name].moe):
                 raise ValueError(f"layer {i}: feed-forward kind {mlp['kind']!r} is not supported")
             owner = i
             if e.get("weights_of") is not None:
@@ -103,11 +129,13 @@ class LayeredArch(ModelArch):
                 raise ValueError(f"layer {i} runs with the weights of layer {owner} but is described differently")
             specs.append(s)
         design = DESIGNS[name]
+        embedding = d.get("embedding") or {}
         heads = max((s.mixer.get("heads", 1) for s in specs), default=1)
         return cls(model_type=name.lower(), design=name, vocab_size=d["vocab"], hidden_size=d["width"],
                    intermediate_size=max((s.ff for s in specs), default=0), num_hidden_layers=len(specs),
                    num_attention_heads=heads, num_key_value_heads=heads, rms_norm_eps=float(d["norm"]["eps"]),
-                   embed_scale=float((d.get("embedding") or {}).get("scale", 1.0)), layers=specs, source=copy.deepcopy(d),
+                   embed_scale=float(embedding.get("scale", 1.0)), layers=specs, source=copy.deepcopy(d),
+                   pairs=dict(embedding["bigram"]) if embedding.get("bigram") else None, logit_scale=float(d.get("logit_scale", 1.0)),
                    side_dim=int((d.get("token_side") or {}).get("dim", 0)), tie_word_embeddings=design.tied_head,
                    attention_bias=False, qk_norm=False, pad_token_id=d.get("pad_token_id"),
                    bos_token_id=d.get("bos_token_id"), eos_token_id=d.get("eos_token_id"))
@@ -155,8 +183,10 @@ def _vec(n=None, fill=0.0, device=None):
 class DynamicTanh(nn.Module):
     """``tanh(alpha x) w + b``: a norm without statistics."""
 
-    def __init__(self, cfg: LayeredArch, device=None):
+    def __init__(self, cfg: LayeredArch, device=None, **kw):
         super().__init__()
+        if kw:
+            raise NotImplementedError(f"Dynamic Tanh with {sorted(kw)}")
         n = cfg.hidden_size
         self.weight, self.bias, self.alpha = _vec(n, 1.0, device), _vec(n, 0.0, device), _vec(None, 0.5, device)
 
@@ -173,20 +203,40 @@ class DynamicTanh(nn.Module):
 
 
 class RmsNorm(nn.Module):
-    """``x / sqrt(mean(x^2) + eps) w``."""
+    """``x / sqrt(mean(x^2) + eps) w gain``; as a norm of a sublayer's output it may carry that sublayer's ``scale`` vector."""
 
-    def __init__(self, cfg: LayeredArch, device=None):
+    shift = 0.0  # added to the weight
+
+    def __init__(self, cfg: LayeredArch, device=None, gain: float = 1.0, scale: bool = False):
         super().__init__()
-        self.weight, self.eps = _vec(cfg.hidden_size, 1.0, device), cfg.rms_norm_eps
+        self.weight, self.eps, self.gain = _vec(cfg.hidden_size, 1.0 - self.shift, device), cfg.rms_norm_eps, gain
+        self.scale = _vec(cfg.hidden_size, 1.0, device) if scale else None
 
     def tensors(self, name):
         return {name: self.weight}
 
     def forward(self, x, out_dtype, delta=None, post=None, **kw):
-        return mx.rms_residual(x, delta, None if post is None else post.weight, self.weight, self.eps, out_dtype, **kw)
+        return mx.rms_residual(x, delta, w=self.weight, eps=self.eps, out_dtype=out_dtype, shift=self.shift, gain=self.gain,
+                               **_weights(post), **kw)
+
+    @staticmethod
+    def stream(x, out_dtype, delta, post, **kw):
+        """The stream itself after the addition of ``delta`` (normed by ``post``), in ``out_dtype``, and in fp32."""
+        eps, shift = (0.0, 0.0) if post is None else (post.eps, post.shift)
+        return mx.rms_residual(x, delta, w=None, eps=eps, out_dtype=out_dtype, shift=shift, **_weights(post), **kw)
 
 
-NORMS = {"dynamic_tanh": DynamicTanh, "rms": RmsNorm}
+class RmsNormAboutZero(RmsNorm):
+    """:class:`RmsNorm` with the weight stored as its distance from one."""
+
+    shift = 1.0
+
+
+def _weights(post):
+    return dict(post=None) if post is None else dict(post=post.weight, post_scale=post.scale)
+
+
+NORMS = {"dynamic_tanh": DynamicTanh, "rms": RmsNorm, "rms_about_zero": RmsNormAboutZero}
 
 
 class LatentAttention(nn.Module):
@@ -283,16 +333,18 @@ class MLstm(nn.Module):
 
 
 class GroupedAttention(nn.Module):
-    """Grouped-query attention without rotation: queries and keys over their rms per head, queries times a temperature that
-    grows with the position, scores capped by tanh, heads times the sigmoid of gates that read the layer input.  With
-    ``kv_from`` the layer has no keys and values of its own and reads those of another layer.  The projections are one
-    matrix (query | key | value | gate)."""
+    """Grouped-query attention: queries and keys over their rms, optionally rotated, queries optionally times a temperature that
+    grows with the position, scores optionally capped by tanh, over all earlier keys or a window and the first tokens, the output
+    optionally times sigmoid gates that read the layer input (what of it a design has: :class:`AttentionStyle` and the layer's
+    sizes).  With ``kv_from`` the layer has no keys and values of its own and reads those of another layer.  The projections are
+    one matrix (query | key | value | gate, with gates per head filled up to whole 16-byte rows)."""
 
     kind = "attention"
 
     def __init__(self, cfg: LayeredArch, m: dict, dtype, device):
         super().__init__()
         kw = dict(dtype=dtype, device=device)
+        style = DESIGNS[cfg.design].attention.get(self.kind, AttentionStyle())
         self.eps = cfg.rms_norm_eps
         self.heads, self.kv_heads, self.dim, self.vdim = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
         if self.heads % self.kv_heads:
@@ -301,22 +353,62 @@ class GroupedAttention(nn.Module):
         self.cap = float(m["softcap"]) if m.get("softcap") else None
         t = m.get("q_temp")
         self.temperature = mx.TemperatureSpec(t["coef"], t["every"]) if t else None
+        mask, rot = m.get("mask") or {}, m.get("rot")
+        self.window = int(mask["size"]) if mask.get("size") else None
+        self.keep = int(mask.get("keep_first") or 0)
+        self.rot, self.rope = (int(rot["dims"]), mx.RotarySpec(rot["dims"], float(rot["base"]), rot.get("scaling"))) if rot else (0, None)
+        if self.rot % 2 or self.rot > self.dim:
+            raise ValueError(f"{self.rot} rotated elements of {self.dim}")
+        self.whole_norm, self.halves, self.values, self.gate = style.whole_norm, style.halves, style.values, style.gate
+        if not self.values and self.vdim != self.dim:
+            raise ValueError("values that are the keys have their size")
         self.kv_from = m.get("kv_from")
         own = self.kv_heads if self.kv_from is None else 0
-        self.parts = [self.heads * self.dim, own * self.dim, own * self.vdim, self.heads * self.vdim]  # rows of w_in
-        h = cfg.hidden_size
-        self.w_in = nn.Parameter(torch.empty(sum(self.parts), h, **kw))
+        gates = {"element": self.heads * self.vdim, "head": self.heads, None: 0}[self.gate]
+        self.parts = [self.heads * self.dim, own * self.dim, own * self.vdim if self.values else 0, gates]  # rows of w_in
+        h, fill = cfg.hidden_size, -sum(self.parts) % 8 if self.gate == "head" else 0
+        self.w_in = nn.Parameter(torch.empty(sum(self.parts) + fill, h, **kw))
+        if fill:
+            self.w_in.data[-fill:].zero_()
         self.o = nn.Parameter(torch.empty(h, self.heads * self.vdim, **kw))
+        self.q_norm = self.k_norm = None
+        if style.norm_weight:
+            self.q_norm = _vec(self.heads * self.dim if self.whole_norm else self.dim, 1.0, device)
+            if own:
+                self.k_norm = _vec(own * self.dim if self.whole_norm else self.dim, 1.0, device)
+        self.sink = _vec(self.heads, 0.0, device) if style.sink else None
+
+    @property
+    def prep(self) -> dict:
+        """How queries and keys are prepared (:func:`~trl_b200.ops.cuda_mixers.attn_prep`)."""
+        return dict(q_norm=self.q_norm, k_norm=self.k_norm, whole_norm=self.whole_norm, rot=self.rot, halves=self.halves,
+                    values=self.values, gates=self.gate)
+
+    @property
+    def sight(self) -> dict:
+        """What a query sees besides the earlier tokens' keys as they are."""
+        return dict(window=self.window, keep=self.keep, sink=self.sink)
 
     def tensors(self, p):
-        q, k, v, g = self.w_in.split(self.parts)
-        out = {p + "q": q, p + "g": g, p + "o": self.o}
+        q, k, v, g = self.w_in[: sum(self.parts)].split(self.parts)
+        out = {p + "q": q, p + "o": self.o}
         if self.kv_from is None:
-            out.update({p + "k": k, p + "v": v})
+            out[p + "k"] = k
+            if self.values:
+                out[p + "v"] = v
+        if self.gate:
+            out[p + "g"] = g
+        out.update({p + n: t for n, t in (("q.norm", self.q_norm), ("k.norm", self.k_norm), ("sink", self.sink)) if t is not None})
         return out
 
     def forward(self, h, ctx: SeqCtx, li: int):
         return mx.attention(self, h, ctx, li)
+
+
+class GroupedAttention2(GroupedAttention):
+    """The other grouped-query attention of a design that has two."""
+
+    kind = "attention_2"
 
 
 class RgLru(nn.Module):
@@ -354,11 +446,16 @@ class RgLru(nn.Module):
         return mx.rglru(self, h, ctx, li)
 
 
-MIXERS = {c.kind: c for c in (LatentAttention, MLstm, GroupedAttention, RgLru)}
+MIXERS = {c.kind: c for c in (LatentAttention, MLstm, GroupedAttention, GroupedAttention2, RgLru)}
 
 
 class DenseMlp(nn.Module):
-    """``down(act(up x))`` with the exact GELU."""
+    """``down(act(up x))`` with the exact GELU.
+
+    ``w_in`` is the first product's weight, ``fused`` names its activation to the weight-streaming product, ``act`` is that
+    activation alone."""
+
+    fused = dict(gelu=True)
 
     def __init__(self, cfg: LayeredArch, spec: dict, dtype, device):
         super().__init__()
@@ -366,37 +463,98 @@ class DenseMlp(nn.Module):
         self.up = nn.Parameter(torch.empty(ff, cfg.hidden_size, dtype=dtype, device=device))
         self.down = nn.Parameter(torch.empty(cfg.hidden_size, ff, dtype=dtype, device=device))
 
+    @property
+    def w_in(self):
+        return self.up
+
     def tensors(self, p):
         return {p + "up": self.up, p + "down": self.down}
 
+    def act(self, z, out=None):
+        return mx.gelu_erf(z, out)
+
     def forward(self, h):
-        return mx.linear_f32(mx.gelu_linear(h, self.up), self.down)
+        return mx.linear_f32(self.act(mx.linear(h, self.w_in)), self.down)
 
 
-class ClampedGluMlp(nn.Module):
-    """``down(g sigmoid(alpha g) (u + shift))`` with ``g = min(gate x, limit)`` and ``u = up x`` within +- limit.  Gate and up
-    projections are one matrix."""
+class GeluGluMlp(DenseMlp):
+    """``down(gelu_tanh(gate x) * up x)``.  Gate and up projections are one matrix."""
+
+    fused = dict(gelu_glu=True)
+
+    def __init__(self, cfg: LayeredArch, spec: dict, dtype, device):
+        nn.Module.__init__(self)
+        self.ff = int(spec["ff"])
+        self.gate_up = nn.Parameter(torch.empty(2 * self.ff, cfg.hidden_size, dtype=dtype, device=device))
+        self.down = nn.Parameter(torch.empty(cfg.hidden_size, self.ff, dtype=dtype, device=device))
+
+    @property
+    def w_in(self):
+        return self.gate_up
+
+    def tensors(self, p):
+        return {p + "gate": self.gate_up[: self.ff], p + "up": self.gate_up[self.ff:], p + "down": self.down}
+
+    def act(self, z, out=None):
+        return mx.gelu_glu(z, out)
+
+
+class ClampedGluMlp(GeluGluMlp):
+    """``down(g sigmoid(alpha g) (u + shift))`` with ``g = min(gate x, limit)`` and ``u = up x`` within +- limit."""
 
     alpha, shift = 1.702, 1.0
 
     def __init__(self, cfg: LayeredArch, spec: dict, dtype, device):
+        super().__init__(cfg, spec, dtype, device)
+        self.limit = float(spec["limit"])
+
+    @property
+    def glu(self):
+        return self.limit, self.alpha, self.shift
+
+    @property
+    def fused(self):
+        return dict(clamped_glu=self.glu)
+
+    def act(self, z, out=None):
+        return mx.clamped_glu(z, *self.glu, out=out)
+
+
+class ExpertMlp(nn.Module):
+    """Mixture of experts, each a clamped gated unit: a token runs the ``top`` experts of the largest sigmoid score plus
+    correction and adds them up with their bare scores as weights.  The experts' matrices are stacked."""
+
+    alpha, shift = 1.702, 1.0
+    renormalize = False  # weights over their sum
+
+    def __init__(self, cfg: LayeredArch, spec: dict, dtype, device):
         super().__init__()
-        self.ff, self.limit = int(spec["ff"]), float(spec["limit"])
-        self.gate_up = nn.Parameter(torch.empty(2 * self.ff, cfg.hidden_size, dtype=dtype, device=device))
-        self.down = nn.Parameter(torch.empty(cfg.hidden_size, self.ff, dtype=dtype, device=device))
+        kw = dict(dtype=dtype, device=device)
+        self.n, self.top = int(spec["router"]["experts"]), int(spec["router"]["top"])
+        self.ff, self.limit = int(spec["expert"]["ff"]), float(spec["expert"]["limit"])
+        if not 1 <= self.top <= self.n <= 1024:
+            raise ValueError(f"{self.top} of {self.n} experts (at most 1024)")
+        h = cfg.hidden_size
+        self.router = nn.Parameter(torch.empty(self.n, h, **kw))
+        self.correction = _vec(self.n, 0.0, device)
+        self.gate_up = nn.Parameter(torch.empty(self.n, 2 * self.ff, h, **kw))
+        self.down = nn.Parameter(torch.empty(self.n, h, self.ff, **kw))
 
     @property
     def glu(self):
         return self.limit, self.alpha, self.shift
 
     def tensors(self, p):
-        return {p + "gate": self.gate_up[: self.ff], p + "up": self.gate_up[self.ff:], p + "down": self.down}
+        out = {p + "router": self.router, p + "correction": self.correction}
+        for e in range(self.n):
+            out.update({f"{p}e{e}.gate": self.gate_up[e, : self.ff], f"{p}e{e}.up": self.gate_up[e, self.ff:], f"{p}e{e}.down": self.down[e]})
+        return out
 
     def forward(self, h):
-        return mx.linear_f32(mx.clamped_glu_linear(h, self.gate_up, *self.glu), self.down)
+        return mx.experts(self, h)
 
 
-MLPS = {"gelu": DenseMlp, "clamped_glu": ClampedGluMlp}
+MLPS = {"gelu": DenseMlp, "gelu_glu": GeluGluMlp, "clamped_glu": ClampedGluMlp, "clamped_glu_experts": ExpertMlp}
 
 
 class TokenSide(nn.Module):
@@ -413,29 +571,26 @@ class TokenSide(nn.Module):
     def tensors(self, p):
         return {p + "gate": self.gate, p + "proj": self.proj, **self.norm.tensors(p + "norm")}
 
-    def stream(self, x, out_dtype, delta, post, **kw):
-        """The stream itself after the addition of ``delta`` (normed by ``post``), in ``out_dtype``, and in fp32."""
-        return mx.rms_residual(x, delta, None if post is None else post.weight, None, self.norm.eps, out_dtype, **kw)
-
     def forward(self, h, ids, table, li: int):
         return mx.side_input(h, ids, table, li * self.dim, self.gate, self.proj)
 
 
 class LayeredBlock(nn.Module):
-    """Pre-norm mixer and (optional) feed-forward around an fp32 residual stream; depending on the design with a norm on each
-    sublayer's output and a per-token input after them."""
+    """Mixer and (optional) feed-forward around an fp32 residual stream; depending on the design with a norm on each sublayer's
+    input (norm1, norm2), on its output (norm1b, norm2b in memory), or both, and a per-token input after them."""
 
     def __init__(self, cfg: LayeredArch, spec: LayerSpec, dtype, device):
         super().__init__()
         design = DESIGNS[cfg.design]
-        norm = NORMS[design.norm]
-        post = norm if design.post_norm else lambda *_: None
-        self.norm1, self.norm1b = norm(cfg, device), post(cfg, device)
+        norm, none = NORMS[design.norm], lambda *_, **__: None
+        pre, post = norm if design.pre_norm else none, norm if design.post_norm else none
+        scale = dict(scale=True) if design.layer_scale else {}
+        self.norm1, self.norm1b = pre(cfg, device), post(cfg, device, **scale)
         self.mixer = MIXERS[spec.kind](cfg, spec.mixer, dtype, device)
         self.norm2 = self.norm2b = self.mlp = None
         if spec.mlp is not None:
-            self.norm2, self.norm2b = norm(cfg, device), post(cfg, device)
-            self.mlp = MLPS[design.mlp](cfg, spec.mlp, dtype, device)
+            self.norm2, self.norm2b = pre(cfg, device), post(cfg, device, **scale)
+            self.mlp = MLPS[design.moe if spec.mlp.get("kind") == "moe" else design.mlp](cfg, spec.mlp, dtype, device)
         self.side = TokenSide(cfg, dtype, device) if cfg.side_dim else None
         self.dtype = dtype
         self.lora = nn.ModuleDict()
@@ -445,27 +600,40 @@ class LayeredBlock(nn.Module):
         return {}  # adapters target the projections of the flat families
 
     def tensors(self, p):
-        out = {**self.norm1.tensors(p + "norm1"), **self.mixer.tensors(p + "mix.")}
-        if self.norm1b is not None:
-            out.update(self.norm1b.tensors(p + "norm1b"))
+        out = self.mixer.tensors(p + "mix.")
         if self.mlp is not None:
-            out.update({**self.norm2.tensors(p + "norm2"), **self.mlp.tensors(p + "mlp.")})
-            if self.norm2b is not None:
-                out.update(self.norm2b.tensors(p + "norm2b"))
+            out.update(self.mlp.tensors(p + "mlp."))
+        for i, pre, post in (("1", self.norm1, self.norm1b), ("2", self.norm2, self.norm2b)):
+            if pre is not None:
+                out.update(pre.tensors(f"{p}norm{i}"))
+            if post is not None:
+                out.update(post.tensors(f"{p}norm{i}" if pre is None else f"{p}norm{i}b"))
+                if post.scale is not None:
+                    out[f"{p}ls{i}"] = post.scale
         if self.side is not None:
             out.update(self.side.tensors(p + "side."))
         return out
 
+    def read_mixer(self, x, delta, post, **kw):
+        """What the mixer reads, and the stream after the addition of the pending ``delta``."""
+        return (RmsNorm.stream if self.norm1 is None else self.norm1)(x, self.dtype, delta, post, **kw)
+
+    def read_mlp(self, x, delta, post, **kw):
+        return (RmsNorm.stream if self.norm2 is None else self.norm2)(x, self.dtype, delta, post, **kw)
+
+    def read_side(self, x, delta, post, **kw):
+        return RmsNorm.stream(x, self.dtype, delta, post, **kw)
+
     def forward(self, x, delta, post, ctx: SeqCtx, li: int, ids=None, side_table=None):
         """(residual, sublayer output not yet added to it, norm of that output) -> the same triple after this layer: every
         addition rides on the norm that follows it."""
-        h, x = self.norm1(x, self.dtype, delta, post)
+        h, x = self.read_mixer(x, delta, post)
         delta, post = self.mixer(h, ctx, li), self.norm1b
         if self.mlp is not None:
-            h, x = self.norm2(x, self.dtype, delta, post)
+            h, x = self.read_mlp(x, delta, post)
             delta, post = self.mlp(h), self.norm2b
         if self.side is not None:
-            h, x = self.side.stream(x, self.dtype, delta, post)
+            h, x = self.read_side(x, delta, post)
             delta, post = self.side(h, ids, side_table, li), self.side.norm
         return x, delta, post
 
@@ -486,10 +654,13 @@ class LayeredLM(CausalLM):
         for i, s in enumerate(cfg.layers):  # a layer that borrows weights IS its owner's block at another place
             blocks.append(blocks[s.owner] if s.owner != i else LayeredBlock(cfg, s, dtype, device))
         self.layers = nn.ModuleList(blocks)
-        self.norm = NORMS[DESIGNS[cfg.design].norm](cfg, device)
+        # the head's scale rides on the norm in front of it
+        self.norm = NORMS[DESIGNS[cfg.design].norm](cfg, device, **(dict(gain=cfg.logit_scale) if cfg.logit_scale != 1.0 else {}))
         self.lm_head = None if cfg.tie_word_embeddings else nn.Parameter(torch.empty(cfg.vocab_size, cfg.hidden_size, dtype=dtype, device=device))
         self.side_embed = (nn.Parameter(torch.empty(cfg.vocab_size, cfg.side_dim * cfg.num_hidden_layers, dtype=dtype, device=device))
                            if cfg.side_dim else None)
+        self.pair_embed = (nn.Parameter(torch.empty(cfg.pairs["buckets"] + 1, cfg.hidden_size, dtype=dtype, device=device))
+                           if cfg.pairs else None)
         self.gradient_checkpointing = False
         self.name_or_path = ""
         self.generation_config = None
@@ -508,6 +679,8 @@ class LayeredLM(CausalLM):
         out = {"embed": self.embed_tokens}
         if self.side_embed is not None:
             out["side.embed"] = self.side_embed
+        if self.pair_embed is not None:
+            out["bigram"] = self.pair_embed
         for i, (s, b) in enumerate(zip(self.config.layers, self.layers)):
             if s.owner == i:
                 out.update(b.tensors(f"l{i}."))
@@ -537,8 +710,14 @@ class LayeredLM(CausalLM):
             dst.copy_(sd[name])
         return [k for k in sd if k not in mine]
 
-    def embed(self, input_ids):
-        return mx.embed_scaled(input_ids, self.embed_tokens, self.config.embed_scale)
+    def embed(self, input_ids, ctx: SeqCtx | None = None):
+        if self.pair_embed is None:
+            return mx.embed_scaled(input_ids, self.embed_tokens, self.config.embed_scale)
+        if ctx is None:
+            raise NotImplementedError("the embedding of this design depends on the tokens' positions in their sequences")
+        where = ctx.kv.last_tokens() if ctx.kv is not None else {}
+        return mx.embed_pairs(input_ids.reshape(-1), self.embed_tokens, self.config.embed_scale, self.pair_embed, self.config.pairs,
+                              ctx.positions, where)
 
     def final_norm(self, x, delta=None, post=None):
         return self.norm(x, self.dtype, delta, post)[0]
@@ -547,7 +726,7 @@ class LayeredLM(CausalLM):
         mx.check_can_run(self.embed_tokens)
         ctx = dataclasses.replace(ctx, shared=dict.fromkeys(self.config.lenders))
         ids = input_ids.reshape(-1)
-        x, delta, post = (self.embed(input_ids) if inputs_embeds is None else inputs_embeds.float()), None, None
+        x, delta, post = (self.embed(input_ids, ctx) if inputs_embeds is None else inputs_embeds.float()), None, None
         for li, layer in enumerate(self.layers):
             x, delta, post = layer(x, delta, post, ctx, li, ids, self.side_embed)
         return self.final_norm(x, delta, post)
@@ -559,3 +738,10 @@ def is_layered_dir(path: str) -> bool:
         return False
     with open(f) as fh:
         return json.load(fh).get("architecture") in DESIGNS
+
+
+def layered_kinds(path: str) -> set:
+    """Mixers and feed-forwards of a model directory whose kernels are built apart (csrc/build.py)."""
+    with open(os.path.join(path, "config.json")) as fh:
+        layers = json.load(fh)["layers"]
+    return {e["type"] for e in layers} | {"moe" for e in layers if (e.get("mlp") or {}).get("kind") == "moe"}

@@ -559,23 +559,24 @@ def attention_varlen_qk(q, k, v, cu_q, cu_k, max_q, max_k):
                        int(max_q), int(max_k), window_size=(-1, 0))
 
 
-def grouped_gemm(a, w, offsets, n_out, swiglu=False, out=None, w_transposed=False):
+def grouped_gemm(a, w, offsets, n_out, swiglu=False, out=None, w_transposed=False, clamped_glu=None):
     """Per-expert GEMM on tcgen05: rows of ``a`` [R, K] are sorted by expert, ``offsets`` [E + 1] int32 on the device,
     ``w`` [E, n_out (or 2 * n_out with swiglu), K].  Returns [R, n_out]; with ``swiglu`` the gate / up halves are
-    combined in the epilogue.  ``w_transposed``: ``w`` is [E, K, n_out] and is read as it lies (the input gradient of
+    combined in the epilogue, with ``clamped_glu=(limit, alpha, shift)`` by the clamped gated unit.  ``w_transposed``: ``w`` is [E, K, n_out] and is read as it lies (the input gradient of
     a layer whose forward weight is ``w``)."""
     R, Kd = a.shape
     E = w.shape[0]
     assert a.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and w.is_contiguous() and a.stride(1) == 1
+    act = 2 if clamped_glu else int(swiglu)
     if w_transposed:
-        assert not swiglu and w.shape[1] == Kd and w.shape[2] == n_out
+        assert not act and w.shape[1] == Kd and w.shape[2] == n_out
     else:
-        assert w.shape[1] == (2 * n_out if swiglu else n_out) and w.shape[2] == Kd
+        assert w.shape[1] == (2 * n_out if act else n_out) and w.shape[2] == Kd
     if out is None:
         out = torch.empty(R, n_out, dtype=torch.bfloat16, device=a.device)
     _chk(lib().trlb_grouped_gemm_bf16(_p(a), _p(w), _p(offsets), _p(out), c_longlong(R), c_int(E), c_int(n_out), c_int(Kd),
-                                      c_longlong(a.stride(0)), c_longlong(out.stride(0)), c_int(int(swiglu)),
-                                      c_int(int(w_transposed)), _p(status_buffer(a.device)), _s()), "grouped_gemm")
+                                      c_longlong(a.stride(0)), c_longlong(out.stride(0)), c_int(act),
+                                      (ctypes.c_float * 3)(*clamped_glu) if clamped_glu else None, c_int(int(w_transposed)), _p(status_buffer(a.device)), _s()), "grouped_gemm")
     return out
 
 
@@ -840,15 +841,15 @@ def set_pdl(on: bool) -> bool:
     return bool(lib().trlb_set_pdl(c_int(int(bool(on)))))
 
 
-def decode_gemm(x, w, bias=None, *, y32=None, out=None, swiglu=False, gelu=False, clamped_glu=None, max_ctas: int = 0,
-                tiled_shape=None, peers=None):
+def decode_gemm(x, w, bias=None, *, y32=None, out=None, swiglu=False, gelu=False, clamped_glu=None, gelu_glu=False,
+                max_ctas: int = 0, tiled_shape=None, peers=None):
     """Weight-streaming tcgen05 GEMM for decode batches (at most 128 rows of ``x``).
 
     ``y32`` given: ``y32[B, N] (fp32) += x @ w^T (+ bias)``, work split stream-K style over every SM; the caller passes
     zeros (the consumer kernels clear the buffer after reading it).  Otherwise bf16 ``out[B, N] = x @ w^T (+ bias)``;
     with ``swiglu`` ``w`` is ``[2N, K]`` (gate rows, then up rows) and ``out = silu(x Wg^T) * (x Wu^T)``; with ``gelu`` the
     exact GELU of the sum is stored; ``clamped_glu=(limit, alpha, shift)`` is the clamped gated unit of a ``[2N, K]``
-    weight (:func:`~trl_b200.ops.cuda_mixers.clamped_glu`).
+    weight (:func:`~trl_b200.ops.cuda_mixers.clamped_glu`), ``gelu_glu`` its ``gelu_tanh(x Wg^T) * (x Wu^T)``.
 
     ``tiled_shape=(rows, K)``: ``w`` is the flat tile-major copy made by :func:`tile_weights` of a ``[rows, K]`` weight.
     ``peers=(peer_y32_ptrs, arrive_ptrs, stage, slab_ctr)``: row-parallel GEMM fused with its all-reduce: partial sums
@@ -865,15 +866,16 @@ def decode_gemm(x, w, bias=None, *, y32=None, out=None, swiglu=False, gelu=False
     else:
         assert w.stride(1) == 1 and w.shape[1] == Kd
         rows, ldw = w.shape[0], w.stride(0)
-    N = rows // 2 if swiglu or clamped_glu else rows
+    glu = bool(swiglu or clamped_glu or gelu_glu)
+    N = rows // 2 if glu else rows
     if y32 is not None:
-        assert y32.dtype == torch.float32 and y32.stride(1) == 1 and tuple(y32.shape) == (B, N) and not swiglu and not clamped_glu
+        assert y32.dtype == torch.float32 and y32.stride(1) == 1 and tuple(y32.shape) == (B, N) and not glu
         mode, ldy, dst32, dstb, ret = 0, y32.stride(0), y32, None, y32
     else:
         if out is None:
             out = torch.empty(B, N, dtype=torch.bfloat16, device=x.device)
         assert out.dtype == torch.bfloat16 and out.stride(1) == 1 and tuple(out.shape) == (B, N)
-        mode, ldy, dst32, dstb, ret = (2 if swiglu else 3 if gelu else 4 if clamped_glu else 1), out.stride(0), None, out, out
+        mode, ldy, dst32, dstb, ret = (2 if swiglu else 3 if gelu else 4 if clamped_glu else 5 if gelu_glu else 1), out.stride(0), None, out, out
     n_peers, peer_arr, arrive_arr, stage, slab_ctr = 0, None, None, None, None
     if peers is not None:
         peer_ptrs, arrive_ptrs, stage, slab_ctr = peers

@@ -1,5 +1,5 @@
-"""ctypes bindings of ``csrc/mixers.cu``, ``csrc/grouped_attn.cu``, ``csrc/rglru.cu`` and of the tensor-core mixer kernels
-(inference only).
+"""ctypes bindings of ``csrc/mixers.cu``, ``csrc/grouped_attn.cu``, ``csrc/rglru.cu``, ``csrc/layered_moe.cu`` and of the
+tensor-core mixer kernels (inference only).
 
 ``model dtype`` below is bf16 or fp32; accumulators, gates, states and norms are fp32 in both."""
 from __future__ import annotations
@@ -40,6 +40,21 @@ def embed_scaled(ids, emb, scale, out=None):
     return out
 
 
+def embed_pairs(ids, emb, scale, pairs, mul_prev, mul_cur, positions, tok_slot=None, prev=None, decode=False, out=None):
+    """``emb[ids] * scale + pairs[row]`` with the row ``(previous * mul_prev + current * mul_cur) mod buckets`` of a table of
+    ``buckets`` + 1 rows, the last one at position 0.  Prompts: ``prev`` (int64 by slot) gets every sequence's last token; decode:
+    one row per slot, ``prev`` is the previous token and moves on where the position is not negative."""
+    T, (V, H) = ids.numel(), emb.shape
+    out = torch.empty(T, H, dtype=torch.float32, device=emb.device) if out is None else out
+    assert ids.dtype == torch.int64 and ids.is_contiguous() and emb.is_contiguous() and pairs.is_contiguous()
+    assert pairs.dtype == emb.dtype and pairs.shape[1] == H and positions.dtype == torch.int32 and positions.numel() >= T
+    assert prev is None or prev.dtype == torch.int64
+    _chk(lib().trlb_embed_pairs(_p(ids), _p(emb), _p(pairs), _p(out), c_int(T), c_int(H), c_int(V), c_float(scale), c_longlong(mul_prev),
+                                c_longlong(mul_cur), c_longlong(pairs.shape[0] - 1), _p(positions), _p(tok_slot), _p(prev),
+                                c_int(int(decode)), _b(emb), _s()), "embed_pairs")
+    return out
+
+
 def dynamic_tanh(x, delta, alpha, w, b, dtype, clear=False, out=None):
     """``x += delta`` (in place; with ``clear`` delta is zeroed), returns ``tanh(alpha x) w + b`` in ``dtype``."""
     T, H = x.shape
@@ -51,15 +66,15 @@ def dynamic_tanh(x, delta, alpha, w, b, dtype, clear=False, out=None):
     return out
 
 
-def rms_residual(x, delta, post, w, eps, dtype, clear=False, out=None):
-    """``x += delta`` or, with ``post``, ``x += delta / rms(delta) * post`` (in place; with ``clear`` delta is zeroed); returns
-    ``x / rms(x) * w`` in ``dtype``, or ``x`` itself without ``w``."""
+def rms_residual(x, delta, post, w, eps, dtype, clear=False, out=None, shift=0.0, post_scale=None, gain=1.0):
+    """``x += delta`` or, with ``post``, ``x += delta / rms(delta) * (shift + post) * post_scale`` (in place; with ``clear`` delta is
+    zeroed); returns ``x / rms(x) * (shift + w) * gain`` in ``dtype``, or ``x`` itself without ``w``."""
     T, H = x.shape
     assert x.dtype == torch.float32 and x.is_contiguous() and (delta is None or (delta.dtype == torch.float32
                                                                                and delta.is_contiguous()))
     out = torch.empty(T, H, dtype=dtype, device=x.device) if out is None else out
-    _chk(lib().trlb_rms_residual(_p(x), _p(delta), _p(post), _p(w), _p(out), c_int(T), c_int(H), c_float(eps),
-                                 c_int(int(clear)), _b(out), _s()), "rms_residual")
+    _chk(lib().trlb_rms_residual(_p(x), _p(delta), _p(post), _p(post_scale), _p(w), _p(out), c_int(T), c_int(H), c_float(eps),
+                                 c_float(shift), c_float(gain), c_int(int(clear)), _b(out), _s()), "rms_residual")
     return out
 
 
@@ -70,6 +85,15 @@ def clamped_glu(z, limit, alpha, shift, out=None):
     out = torch.empty(rows, n, dtype=z.dtype, device=z.device) if out is None else out
     _chk(lib().trlb_clamped_glu(_p(z), _p(out), c_int(rows), c_int(n), c_float(limit), c_float(alpha), c_float(shift), _b(z), _s()),
          "clamped_glu")
+    return out
+
+
+def gelu_glu(z, out=None):
+    """z [rows, 2n] = gate | up -> ``gelu_tanh(gate) * up``."""
+    rows, n = z.shape[0], z.shape[1] // 2
+    assert z.is_contiguous()
+    out = torch.empty(rows, n, dtype=z.dtype, device=z.device) if out is None else out
+    _chk(lib().trlb_gelu_glu(_p(z), _p(out), c_int(rows), c_int(n), _b(z), _s()), "gelu_glu")
     return out
 
 
@@ -123,11 +147,11 @@ def mixer_attn_tc_ok(heads, kv_heads, dim, rot, vdim) -> bool:
     return bool(lib().trlb_mixer_attn_tc_ok(c_int(heads), c_int(kv_heads), c_int(dim), c_int(rot), c_int(vdim)))
 
 
-def mixer_attn(q, k, v, *, heads, kv_heads, scale, ctx, rot=0, krot=None, window=None, cap=None, sink=None, gate=None,
-               gate_logits=None, tensor_cores=True):
+def mixer_attn(q, k, v, *, heads, kv_heads, scale, ctx, rot=0, krot=None, window=None, keep=0, cap=None, sink=None,
+               gate=None, gate_logits=None, tensor_cores=True):
     """Causal attention of packed prompts.  Rows of q: heads x (dim | rot), of k and v: kv_heads x dim / vdim, of krot: the rot
     elements that all heads' keys share (rows may be strided, their elements are dense) -> [T, heads vdim].  Keys at distance <
-    ``window``; scores ``cap tanh(s / cap)``; ``exp(sink)`` in the denominator; ``gate`` (fp32 [T, heads]) or the sigmoid of
+    ``window`` and the first ``keep`` of the sequence; scores ``cap tanh(s / cap)``; ``exp(sink)`` in the denominator; ``gate`` (fp32 [T, heads]) or the sigmoid of
     ``gate_logits`` ([T, heads vdim] in the model dtype) multiplies the result."""
     T, dim, vdim = q.shape[0], k.shape[1] // kv_heads, v.shape[1] // kv_heads
     out = torch.empty(T, heads * vdim, dtype=q.dtype, device=q.device)
@@ -137,7 +161,7 @@ def mixer_attn(q, k, v, *, heads, kv_heads, scale, ctx, rot=0, krot=None, window
     assert mode != 2 or (gate_logits.shape == out.shape and gate_logits.dtype == q.dtype and gate_logits.stride(1) == 1)
     gate = gate_logits if mode == 2 else gate
     rows = [c for t in (q, k, v, krot) for c in (_p(t), c_longlong(0 if t is None else t.stride(0)))]
-    sizes = [c_int(x) for x in (T, heads, kv_heads, dim, rot, vdim, window or 0)] + [c_float(scale), c_float(cap or 0.0)]
+    sizes = [c_int(x) for x in (T, heads, kv_heads, dim, rot, vdim, window or 0, keep)] + [c_float(scale), c_float(cap or 0.0)]
     tail = [_p(sink), c_int(mode), _p(gate), c_longlong(0 if gate is None else gate.stride(0)), _p(out)]
     aligned = all(t is None or (t.data_ptr() % 16 == 0 and t.stride(0) % 8 == 0) for t in (q, k, v, krot)) and (
         mode != 2 or (gate.data_ptr() % 16 == 0 and gate.stride(0) % 8 == 0))
@@ -151,25 +175,40 @@ def mixer_attn(q, k, v, *, heads, kv_heads, scale, ctx, rot=0, krot=None, window
     return out
 
 
-def attn_prep(y, m, positions, temp, *, tok_slot=None, q=None, g=None, k_cache=None, v_cache=None, block_table=None, block_size=0):
-    """Rows ``y`` [q | k | v | g] of an attention mixer's input projection: unit-rms queries (times ``temp`` by position) and
-    keys, keys and values to the paged cache.  Without ``q`` queries and keys are replaced in place; with ``q`` (and ``g`` for
-    the gate logits) ``y`` is fp32 sums, and they are zeroed."""
+GATES = {None: 0, "head": 1, "element": 2}
+
+
+def attn_prep(y, m, positions, temp, *, q_norm=None, k_norm=None, whole_norm=False, table=None, rot=0, halves=False, values=True,
+              gates="element", tok_slot=None, q=None, k=None, g=None, head_gate=None, k_cache=None, v_cache=None, block_table=None,
+              block_size=0):
+    """Rows ``y`` [q | k | v | g] of an attention mixer's input projection: normed queries (times ``temp`` by position) and keys,
+    both rotated by ``table`` (their first ``rot`` elements, in pairs of neighbours or of ``halves``); keys and values to the paged
+    cache; ``gates`` per head as fp32 sigmoids to ``head_gate``.  The norm is per head, with ``whole_norm`` over all heads, and times
+    the weights ``q_norm`` / ``k_norm`` if there are any.  Without ``values`` the keys as projected are the values.  Without
+    ``q`` queries are replaced in place, keys too unless they go to ``k``; with ``q``
+    (and ``g`` for gate logits per element) ``y`` is fp32 sums, and they are zeroed."""
     rows = y.shape[0]
     assert y.stride(1) == 1 and positions.dtype == torch.int32 and (q is None or y.dtype == torch.float32)
+    assert (head_gate is None) == (gates != "head") and (k is None or (k.is_contiguous() and k.dtype == m.o.dtype))
+    assert rot == 0 or (table.dtype == torch.float32 and table.shape[1] * 2 == rot)
     mb = 0 if block_table is None else block_table.shape[1]
     _chk(lib().trlb_attn_prep(_p(y), c_int(int(y.dtype == torch.float32)), c_longlong(y.stride(0)), c_int(rows), c_int(m.heads),
-                              c_int(m.kv_heads), c_int(m.dim), c_int(m.vdim), c_int(int(m.kv_from is None)), c_int(1), c_float(m.eps),
-                              _p(positions), _p(tok_slot), _p(temp), _len(temp), _p(q), _p(g), _p(k_cache), _p(v_cache),
+                              c_int(m.kv_heads), c_int(m.dim), c_int(m.vdim), c_int(int(m.kv_from is None)), c_int(int(values)),
+                              c_int(GATES[gates]), c_float(m.eps), _p(positions), _p(tok_slot), _p(temp), _len(temp),
+                              c_int(int(whole_norm)), _p(q_norm), _p(k_norm), c_int(rot), c_int(int(halves)),
+                              _p(table), _len(table), _p(q), _p(k), _p(g), _p(head_gate), _p(k_cache), _p(v_cache),
                               _p(block_table), c_int(mb), c_int(block_size), _b(m.o), _s()), "attn_prep")
 
 
-def grouped_decode(q, k_cache, v_cache, m, seq_lens, block_table, block_size, out, gate=None):
-    """One token per slot on the CUDA cores: any size, bf16 or fp32.  q [B, heads, dim], gate logits [B, heads vdim]."""
+def grouped_decode(q, k_cache, v_cache, m, seq_lens, block_table, block_size, out, gate=None, *, head_gate=None, window=None, keep=0,
+                   sink=None):
+    """One token per slot on the CUDA cores: any size, bf16 or fp32.  q [B, heads, dim], gate logits [B, heads vdim], factors
+    ``head_gate`` fp32 [B, heads]; ``window``, ``keep`` and ``sink`` as in :func:`mixer_attn`."""
     B = q.shape[0]
-    _chk(lib().trlb_grouped_decode(_p(q), _p(k_cache), _p(v_cache), _p(gate), _p(out), c_int(B), c_int(m.heads), c_int(m.kv_heads),
-                                   c_int(m.dim), c_int(m.vdim), c_float(m.scale), c_float(m.cap or 0.0), _p(seq_lens), _p(block_table),
-                                   c_int(block_table.shape[1]), c_int(block_size), _b(q), _s()), "grouped_decode")
+    _chk(lib().trlb_grouped_decode(_p(q), _p(k_cache), _p(v_cache), _p(gate), _p(head_gate), _p(sink), _p(out), c_int(B), c_int(m.heads),
+                                   c_int(m.kv_heads), c_int(m.dim), c_int(m.vdim), c_int(window or 0), c_int(keep), c_float(m.scale),
+                                   c_float(m.cap or 0.0), _p(seq_lens), _p(block_table), c_int(block_table.shape[1]), c_int(block_size),
+                                   _b(q), _s()), "grouped_decode")
 
 
 def grouped_decode_tc_ok(m, block_size: int) -> bool:
@@ -181,7 +220,8 @@ def grouped_decode_tc_items(B: int, m) -> int:
     return int(lib().trlb_grouped_decode_tc_items(c_int(B), c_int(m.heads), c_int(m.kv_heads)))
 
 
-def grouped_decode_tc(q, k_cache, v_cache, m, seq_lens, block_table, block_size, out, gate=None, splits=1, part_o=None, part_ml=None):
+def grouped_decode_tc(q, k_cache, v_cache, m, seq_lens, block_table, block_size, out, gate=None, splits=1, part_o=None, part_ml=None, *,
+                      head_gate=None, window=None, keep=0, sink=None):
     """:func:`grouped_decode` on the tensor cores (bf16).  With ``splits`` > 1: ``part_o`` [>= B heads splits vdim] and
     ``part_ml`` [>= 2 B heads splits] fp32 scratch."""
     B = q.shape[0]
@@ -190,9 +230,54 @@ def grouped_decode_tc(q, k_cache, v_cache, m, seq_lens, block_table, block_size,
     if splits > 1:
         assert part_o.numel() >= B * m.heads * splits * m.vdim and part_ml.numel() >= 2 * B * m.heads * splits
     _chk(lib().trlb_grouped_decode_tc(_p(q), _p(k_cache), _p(v_cache), _p(gate), _p(out), c_int(k_cache.shape[0]), c_int(B), c_int(m.heads),
-                                      c_int(m.kv_heads), c_int(m.dim), c_int(m.vdim), c_float(m.scale), c_float(m.cap or 0.0), _p(seq_lens),
-                                      _p(block_table), c_int(block_table.shape[1]), c_int(block_size), c_int(splits), _p(part_o), _p(part_ml),
+                                      c_int(m.kv_heads), c_int(m.dim), c_int(m.vdim), c_int(window or 0), c_int(keep), c_float(m.scale),
+                                      c_float(m.cap or 0.0), _p(sink), _p(head_gate), _p(seq_lens), _p(block_table),
+                                      c_int(block_table.shape[1]), c_int(block_size), c_int(splits), _p(part_o), _p(part_ml),
                                       _p(status_buffer(q.device)), _s()), "grouped_decode_tc")
+
+
+def moe_route(z, correction, top, *, positions=None, renormalize=False, clear=False):
+    """fp32 logits z [T, E] (zeroed with ``clear``) -> (choice, rank, weight) [T, top] and counts [E]: the experts of the largest
+    sigmoid score + correction, their place among the expert's tokens, their bare scores (over their sum with ``renormalize``).
+    Rows of negative position choose nothing (-1)."""
+    T, E = z.shape
+    assert z.dtype == torch.float32 and z.is_contiguous() and (correction is None or correction.dtype == torch.float32)
+    i32 = dict(dtype=torch.int32, device=z.device)
+    choice, rank, weight = torch.empty(T, top, **i32), torch.empty(T, top, **i32), torch.empty(T, top, dtype=torch.float32, device=z.device)
+    counts = torch.empty(E, **i32) if T <= 128 else torch.zeros(E, **i32)
+    _chk(lib().trlb_moe_route(_p(z), _p(correction), _p(positions), c_int(T), c_int(E), c_int(top), c_int(int(renormalize)),
+                              c_int(int(clear)), _p(choice), _p(rank), _p(weight), _p(counts), _s()), "moe_route")
+    return choice, rank, weight, counts
+
+
+def moe_gather(h, choice, rank, counts):
+    """Rows of h [T, H] sorted by expert, one per choice -> (x [T top, H], row [T, top] where a choice stands (-1: none), offsets
+    [E + 1]); rows past ``offsets[E]`` mean nothing."""
+    (T, H), top, E = h.shape, choice.shape[1], counts.numel()
+    assert h.is_contiguous()
+    i32 = dict(dtype=torch.int32, device=h.device)
+    x, row, offsets = torch.empty(T * top, H, dtype=h.dtype, device=h.device), torch.empty(T, top, **i32), torch.empty(E + 1, **i32)
+    _chk(lib().trlb_moe_gather(_p(h), _p(choice), _p(rank), _p(counts), c_int(T), c_int(E), c_int(top), c_int(H), _p(x), _p(row),
+                               _p(offsets), _b(h), _s()), "moe_gather")
+    return x, row, offsets
+
+
+def moe_sum(y, row, weight, out=None):
+    """fp32 [T, H]: sum over the choices of ``weight * y[row]``."""
+    (T, top), H = row.shape, y.shape[1]
+    out = torch.empty(T, H, dtype=torch.float32, device=y.device) if out is None else out
+    assert y.is_contiguous() and out.is_contiguous() and out.dtype == torch.float32
+    _chk(lib().trlb_moe_sum(_p(y), _p(row), _p(weight), c_int(T), c_int(top), c_int(H), _p(out), _b(y), _s()), "moe_sum")
+    return out
+
+
+def moe_rows_gemm(a, w, offsets):
+    """``a[r] w[e]^T`` for the rows r of expert e on the CUDA cores: any size, bf16 or fp32."""
+    assert a.is_contiguous() and w.is_contiguous() and a.dtype == w.dtype and a.shape[1] == w.shape[2]
+    out = torch.empty(a.shape[0], w.shape[1], dtype=a.dtype, device=a.device)
+    _chk(lib().trlb_moe_rows_gemm(_p(a), _p(w), _p(offsets), _p(out), c_longlong(a.shape[0]), c_int(w.shape[0]), c_int(w.shape[1]),
+                                  c_int(w.shape[2]), _b(a), _s()), "moe_rows_gemm")
+    return out
 
 
 def conv_prompt(x, m, ctx, seq_slot=None, conv_state=None):

@@ -1,7 +1,7 @@
 """Mechanisms of the layered decoders (models/layered.py) on packed prompts.
 
-CUDA tensors run the kernels of ``csrc/mixers.cu``, ``csrc/grouped_attn.cu``, ``csrc/rglru.cu`` and the tensor-core mixer
-kernels, in bf16 or fp32; CPU tensors run :mod:`trl_b200.oracle.mixers`.  On CUDA the kernels are inference only (prompts,
+CUDA tensors run the kernels of ``csrc/mixers.cu``, ``csrc/grouped_attn.cu``, ``csrc/rglru.cu``, ``csrc/layered_moe.cu`` and the
+tensor-core mixer kernels, in bf16 or fp32; CPU tensors run :mod:`trl_b200.oracle.mixers`.  On CUDA the kernels are inference only (prompts,
 log-probs, generation).
 
 A serving engine passes itself through ``ctx.kv``: ``paged_cache(li)`` and ``recurrent_state(li)`` say where layer ``li``
@@ -24,7 +24,7 @@ def _k():
 
 
 class RotarySpec:
-    """Interleaved rotary positions with optional YaRN scaling.  ``table(n)``: fp32 [n, dims / 2, 2] (cos, sin), the
+    """Rotary positions with optional YaRN scaling.  ``table(n)``: fp32 [n, dims / 2, 2] (cos, sin), the
     magnitude of the scaling folded in; angles are evaluated in fp64 before they are rounded."""
 
     def __init__(self, dims: int, base: float, scaling: dict | None = None):
@@ -117,6 +117,14 @@ def embed_scaled(ids, emb, scale):
     return F.embedding(ids, emb).float() * scale
 
 
+def embed_pairs(ids, emb, scale, pairs, spec, positions, where):
+    """Scaled embeddings plus the rows of a table of token pairs (flat packed ids); ``where``: a serving engine's last tokens."""
+    if emb.is_cuda:
+        return _k().embed_pairs(ids, emb, scale, pairs, spec["mul_prev"], spec["mul_cur"], positions.to(torch.int32), **where)
+    rows = _ref.pair_rows(ids, positions, spec["mul_prev"], spec["mul_cur"], pairs.shape[0] - 1)
+    return F.embedding(ids, emb).float() * scale + F.embedding(rows, pairs).float()
+
+
 def dynamic_tanh(x, delta, alpha, w, b, out_dtype, clear=False, out=None):
     """(norm of ``x + delta`` in ``out_dtype``, ``x + delta``); on CUDA the sum is formed in place."""
     if x.is_cuda:
@@ -125,18 +133,46 @@ def dynamic_tanh(x, delta, alpha, w, b, out_dtype, clear=False, out=None):
     return _ref.dynamic_tanh(x, alpha, w, b).to(out_dtype), x
 
 
-def rms_residual(x, delta, post, w, eps, out_dtype, clear=False, out=None):
+def rms_residual(x, delta, post, w, eps, out_dtype, clear=False, out=None, **kw):
     """(``s / rms(s) * w`` in ``out_dtype``, s) of ``s = x + delta``, where delta over its rms times ``post`` is added when
-    ``post`` is given and s itself is the output when ``w`` is None; on CUDA the sum is formed in place."""
+    ``post`` is given and s itself is the output when ``w`` is None; on CUDA the sum is formed in place.  ``shift`` is added to both
+    weights, ``post_scale`` multiplies ``post``, ``gain`` the output."""
     if x.is_cuda:
-        return _k().rms_residual(x, delta, post, w, eps, out_dtype, clear=clear, out=out), x
-    y, x = _ref.rms_residual(x, delta, post, w, eps)
+        return _k().rms_residual(x, delta, post, w, eps, out_dtype, clear=clear, out=out, **kw), x
+    y, x = _ref.rms_residual(x, delta, post, w, eps, **kw)
     return y.to(out_dtype), x
 
 
-def clamped_glu_linear(h, gate_up, limit, alpha, shift):
-    z = linear(h, gate_up)
-    return _k().clamped_glu(z, limit, alpha, shift) if z.is_cuda else _ref.clamped_glu(z, limit, alpha, shift)
+def clamped_glu(z, limit, alpha, shift, out=None):
+    return _k().clamped_glu(z, limit, alpha, shift, out=out) if z.is_cuda else _ref.clamped_glu(z, limit, alpha, shift)
+
+
+def gelu_glu(z, out=None):
+    return _k().gelu_glu(z, out=out) if z.is_cuda else _ref.gelu_glu(z)
+
+
+def gelu_erf(z, out=None):
+    return _k().gelu_erf(z, out=out) if z.is_cuda else F.gelu(z)
+
+
+def experts(m, h, positions=None, logits=None, out=None):
+    """Mixture of experts: h [T, width] -> fp32 [T, width].  ``positions``: rows where they are negative choose nothing;
+    ``logits``: fp32 sums of the router's product (zeroed), formed here when absent."""
+    if not h.is_cuda:
+        return _ref.experts(m, h.float())
+    K = _k()
+    z = linear_f32(h, m.router) if logits is None else logits
+    choice, rank, weight, counts = K.moe_route(z, m.correction, m.top, positions=positions, renormalize=m.renormalize,
+                                               clear=logits is not None)
+    x, row, offsets = K.moe_gather(h, choice, rank, counts)
+    if h.dtype == torch.bfloat16 and h.shape[1] % 8 == 0 and m.ff % 8 == 0:
+        from . import cuda as KC
+
+        act = KC.grouped_gemm(x, m.gate_up, offsets, m.ff, clamped_glu=m.glu)
+        y = KC.grouped_gemm(act, m.down, offsets, h.shape[1])
+    else:
+        y = K.moe_rows_gemm(K.clamped_glu(K.moe_rows_gemm(x, m.gate_up, offsets), *m.glu), m.down, offsets)
+    return K.moe_sum(y, row, weight, out=out)
 
 
 def side_input(h, ids, table, off, gate, proj):
@@ -145,11 +181,6 @@ def side_input(h, ids, table, off, gate, proj):
     if z.is_cuda:
         return linear_f32(_k().side_gate(z, ids, table, off), proj)
     return linear(F.gelu(z, approximate="tanh") * F.embedding(ids, table)[:, off:off + z.shape[1]].to(z.dtype), proj).float()
-
-
-def gelu_linear(h, up):
-    z = linear(h, up)
-    return _k().gelu_erf(z) if z.is_cuda else F.gelu(z)
 
 
 def latent_attention(m, h, ctx, li):
@@ -189,13 +220,20 @@ def attention(m, h, ctx, li):
         out, kept = _ref.attention(m, h.float(), ctx.positions, ctx.cu_seqlens, kept)
     else:
         K = _k()
+        T, own = h.shape[0], kept is None
         pos = ctx.positions if ctx.positions.dtype == torch.int32 else ctx.positions.to(torch.int32)
         temp = m.temperature.table(ctx.max_seqlen, h.device) if m.temperature is not None else None
+        table = m.rope.table(ctx.max_seqlen, h.device) if m.rot else None
         y = linear(h, m.w_in)
-        K.attn_prep(y, m, pos, temp, **(ctx.kv.paged_cache(li) if ctx.kv is not None else {}))
-        q, k, v, g = y.split(m.parts, 1)
-        kept = (k, v) if kept is None else kept
-        o = K.mixer_attn(q, *kept, heads=m.heads, kv_heads=m.kv_heads, scale=m.scale, cap=m.cap, gate_logits=g, ctx=ctx)
+        q, k, v, g = y[:, : sum(m.parts)].split(m.parts, 1)
+        # projected keys that are also the values stay as they are
+        keys = torch.empty(T, m.kv_heads * m.dim, dtype=h.dtype, device=h.device) if own and not m.values else None
+        gate = torch.empty(T, m.heads, dtype=torch.float32, device=h.device) if m.gate == "head" else None
+        K.attn_prep(y, m, pos, temp, table=table, k=keys, head_gate=gate, **m.prep, **(ctx.kv.paged_cache(li) if ctx.kv is not None else {}))
+        if own:
+            kept = (k, v) if keys is None else (keys, k)
+        o = K.mixer_attn(q, *kept, heads=m.heads, kv_heads=m.kv_heads, scale=m.scale, cap=m.cap, **m.sight, gate=gate,
+                         gate_logits=g if m.gate == "element" else None, ctx=ctx)
         out = linear_f32(o, m.o)
     if li in ctx.shared:
         ctx.shared[li] = kept

@@ -14,17 +14,41 @@ def unit_rms(x, eps):
     return x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps)
 
 
-def rms_residual(x, delta, post, w, eps):
-    """(``x + delta`` (delta over its rms times ``post``, when given)) over its rms times ``w`` (when given), and the sum."""
+def rms_residual(x, delta, post, w, eps, shift=0.0, post_scale=None, gain=1.0):
+    """(``x + delta`` (delta over its rms times ``(shift + post) post_scale``, when given)) over its rms times ``(shift + w) gain``
+    (when given), and the sum."""
     if delta is not None:
-        x = x + (delta if post is None else unit_rms(delta, eps) * post)
-    return (x if w is None else unit_rms(x, eps) * w), x
+        if post is not None:
+            delta = unit_rms(delta, eps) * (shift + post)
+            delta = delta if post_scale is None else delta * post_scale
+        x = x + delta
+    return (x if w is None else unit_rms(x, eps) * ((shift + w) * gain)), x
+
+
+def pair_rows(ids, positions, mul_prev, mul_cur, buckets):
+    """Rows of the table of token pairs for packed sequences: the last one at position 0."""
+    ids = ids.long()
+    row = (ids.roll(1) * mul_prev + ids * mul_cur) % buckets
+    return torch.where(positions > 0, row, torch.full_like(row, buckets))
 
 
 def clamped_glu(z, limit, alpha, shift):
     g, u = z.chunk(2, -1)
     g, u = g.clamp(max=limit), u.clamp(-limit, limit)
     return g * torch.sigmoid(alpha * g) * (u + shift)
+
+
+def gelu_glu(z):
+    g, u = z.chunk(2, -1)
+    return F.gelu(g, approximate="tanh") * u
+
+
+def rotate_halves(x, cos, sin):
+    """x [T, ..., n] with pairs (i, i + n / 2); cos / sin [T, n / 2]."""
+    shape = (x.shape[0],) + (1,) * (x.ndim - 2) + (x.shape[-1] // 2,)
+    c, s = cos.view(shape), sin.view(shape)
+    u, v = x.chunk(2, -1)
+    return torch.cat([u * c - v * s, v * c + u * s], -1)
 
 
 def rotate_pairs(x, cos, sin):
@@ -35,9 +59,10 @@ def rotate_pairs(x, cos, sin):
     return torch.stack([u * c - v * s, v * c + u * s], -1).flatten(-2)
 
 
-def sink_window_attention(q, k, v, scale, window, sink, cu, cap=None):
+def sink_window_attention(q, k, v, scale, window, sink, cu, cap=None, keep=0):
     """q [T, H, D], k [T, G, D], v [T, G, E] (H / G query heads read one key head), packed sequences by ``cu``; scores
-    ``cap tanh(s / cap)``; softmax with ``exp(sink)`` added to the denominator (no such term without a sink)."""
+    ``cap tanh(s / cap)``; softmax with ``exp(sink)`` added to the denominator (no such term without a sink); with a window the first
+    ``keep`` keys of a sequence stay visible."""
     outs, per = [], q.shape[1] // k.shape[1]
     if per > 1:
         k, v = k.repeat_interleave(per, 1), v.repeat_interleave(per, 1)
@@ -48,7 +73,7 @@ def sink_window_attention(q, k, v, scale, window, sink, cu, cap=None):
             s = cap * torch.tanh(s / cap)
         i = torch.arange(n, device=s.device)
         gap = i[:, None] - i[None, :]
-        seen = (gap >= 0) if window is None else (gap >= 0) & (gap < window)
+        seen = (gap >= 0) if window is None else (gap >= 0) & ((gap < window) | (i < keep))
         s = s.masked_fill(~seen, float("-inf"))
         if sink is not None:
             s = torch.cat([s, sink.to(s.dtype)[:, None, None].expand(-1, n, 1)], -1)
@@ -98,16 +123,47 @@ def attention(m, h, positions, cu, kept=None):
     """``m``: a models.layered.GroupedAttention; ``kept``: keys and values of the layer it borrows from.  Returns ([T, width],
     (keys, values))."""
     T, H, G = h.shape[0], m.heads, m.kv_heads
-    y = F.linear(h, m.w_in.to(h.dtype))
-    own = 0 if m.kv_from is not None else G
-    q, k, v, g = y.split([H * m.dim, own * m.dim, own * m.vdim, H * m.vdim], -1)
-    q = unit_rms(q.view(T, H, m.dim), m.eps)
+    q, k, v, g = F.linear(h, m.w_in.to(h.dtype))[:, : sum(m.parts)].split(m.parts, -1)
+
+    def turned(x, n, w):
+        """Norm (of all heads at once, or per head), weight, rotation."""
+        x = unit_rms(x if m.whole_norm else x.view(T, n, m.dim), m.eps)
+        x = (x if w is None else x * w.to(h.dtype)).view(T, n, m.dim)
+        if not m.rot:
+            return x
+        table = m.rope.table(int(positions.max()) + 1 if T else 1, h.device).to(h.dtype)[positions.long()]
+        turn = rotate_halves if m.halves else rotate_pairs
+        return torch.cat([turn(x[..., : m.rot], table[..., 0], table[..., 1]), x[..., m.rot:]], -1)
+
+    q = turned(q, H, m.q_norm)
     if m.temperature is not None:
         q = q * m.temperature.table(int(positions.max()) + 1 if T else 1, h.device).to(h.dtype)[positions.long()][:, None, None]
     if kept is None:
-        kept = unit_rms(k.view(T, G, m.dim), m.eps), v.view(T, G, m.vdim)
-    o = sink_window_attention(q, *kept, m.scale, None, None, cu, m.cap).reshape(T, H * m.vdim)
-    return F.linear(o * torch.sigmoid(g), m.o.to(h.dtype)), kept
+        kept = turned(k, G, m.k_norm), (v if m.values else k).reshape(T, G, m.vdim)
+    o = sink_window_attention(q, *kept, m.scale, m.window, m.sink, cu, m.cap, m.keep)
+    if m.gate == "head":
+        o = o * torch.sigmoid(g)[..., None]
+    o = o.reshape(T, H * m.vdim)
+    return F.linear(o * torch.sigmoid(g) if m.gate == "element" else o, m.o.to(h.dtype)), kept
+
+
+def route(z, correction, top, renormalize=False):
+    """Logits [T, E] -> (experts [T, top], weights [T, top])."""
+    s = torch.sigmoid(z)
+    idx = (s.detach() + correction.to(z.dtype)).topk(top, -1).indices
+    w = s.gather(1, idx)
+    return idx, (w / w.sum(-1, keepdim=True) if renormalize else w)
+
+
+def experts(m, h):
+    """``m``: a models.layered.ExpertMlp; h [T, width] -> [T, width]."""
+    idx, w = route(F.linear(h, m.router.to(h.dtype)), m.correction, m.top, m.renormalize)
+    out = torch.zeros_like(h)
+    for e in range(m.n):
+        t, j = (idx == e).nonzero(as_tuple=True)
+        y = F.linear(clamped_glu(F.linear(h[t], m.gate_up[e].to(h.dtype)), *m.glu), m.down[e].to(h.dtype))
+        out = out.index_add(0, t, y * w[t, j][:, None])
+    return out
 
 
 def causal_conv(x, w, bias, cu):

@@ -7,12 +7,15 @@ reads that layer's instead):
 
     latent_attention   pages of latent rows ``[kv_rank | rotated key]`` behind the engine's block table (the window is a
                        mask: pages stay until the sequence ends)
-    attention          pages of keys (over their rms) and pages of values
+    attention          pages of keys (normed, rotated) and pages of values (the projected keys where those serve as values);
+                       a window is a mask here too
     mlstm              per slot an fp32 matrix state, its normaliser and running maximum
     rglru              per slot an fp32 state vector and the last inputs of the convolution
 
+An embedding of token pairs keeps the last token per slot.
+
 A decode step is one graph: embed, then per layer norm (+ residual) -> input projection -> mixer -> output projection
--> norm (+ residual) -> up / activation -> down (-> stream -> side gate -> side projection), then final norm, head and
+-> norm (+ residual) -> up / activation -> down, or router -> choice -> gather -> experts -> sum (-> stream -> side gate -> side projection), then final norm, head and
 sampler.  Norms on a sublayer's output ride on the norm kernel that follows.  With bf16 weights the projections are the
 weight-streaming tcgen05 kernel; their fp32 sums are consumed and cleared by the next kernel.  fp32 models run the same
 kernels' fp32 forms with library fp32 matrix products."""
@@ -23,7 +26,7 @@ import os
 import torch
 
 from ..models.decoder import SeqCtx
-from ..models.layered import ClampedGluMlp
+from ..models.layered import ExpertMlp
 from ..ops import mixers as mx
 from .engine import RolloutEngine
 
@@ -151,7 +154,7 @@ class _MLstmSlots:
 
 
 class _AttentionSlots:
-    """Decode side of one ``attention`` layer."""
+    """Decode side of one ``attention`` or ``attention_2`` layer."""
 
     def __init__(self, eng: "LayeredRolloutEngine", m, li):
         from ..ops import cuda_mixers as K
@@ -167,15 +170,21 @@ class _AttentionSlots:
             self.k_cache, self.v_cache = lender.k_cache, lender.v_cache
         self.temp = m.temperature.table(eng.max_len + 1, eng.dev) if m.temperature is not None else None
         B = eng.max_seqs
-        self.acc_in = eng.sums("in", m.w_in.shape[0])
+        self.w_in = m.w_in[: sum(m.parts)]
+        self.acc_in = eng.sums("in", sum(m.parts))
         self.q = eng.scratch("q", B, m.heads, m.dim)
-        self.g = eng.scratch("g", B, m.heads * m.vdim)
+        self.table = m.rope.table(eng.max_len + 1, eng.dev) if m.rot else None
+        self.g = eng.scratch("g", B, m.heads * m.vdim) if m.gate == "element" else None
+        self.head_gate = eng.scratch("gate", B, m.heads, dtype=torch.float32) if m.gate == "head" else None
         self.o = eng.scratch("o", B, m.heads * m.vdim)
         # tensor-core decode; other sizes and fp32 run the CUDA-core kernel
         self.tc = eng.dtype == torch.bfloat16 and K.grouped_decode_tc_ok(m, eng.block_size)
         self.splits, self.part_o, self.part_ml = 1, None, None
         if self.tc:
-            self.splits = max(1, min(8, -(-eng.max_len // 128), 148 // K.grouped_decode_tc_items(B, m)))
+            tiles = -(-eng.max_len // 128)
+            if m.window:
+                tiles = min(tiles, -(-m.window // 128) + 1 + -(-m.keep // 128))
+            self.splits = max(1, min(8, tiles, 148 // K.grouped_decode_tc_items(B, m)))
             if self.splits > 1:
                 self.part_o = eng.scratch("part_o", B, m.heads * self.splits * m.vdim, dtype=torch.float32)
                 self.part_ml = eng.scratch("part_ml", B, m.heads * self.splits * 2, dtype=torch.float32)
@@ -199,7 +208,8 @@ class _AttentionSlots:
 
         e = self.e
         where = dict(k_cache=self.k_cache, v_cache=self.v_cache, block_table=e.block_table, block_size=e.block_size) if self.own else {}
-        K.attn_prep(self.acc_in, self.m, e.seq_lens, self.temp, q=self.q, g=self.g, **where)
+        K.attn_prep(self.acc_in, self.m, e.seq_lens, self.temp, table=self.table, q=self.q, g=self.g, head_gate=self.head_gate,
+                    **self.m.prep, **where)
 
     def attend(self):
         from ..ops import cuda_mixers as K
@@ -207,12 +217,12 @@ class _AttentionSlots:
         e = self.e
         args = (self.q, self.k_cache, self.v_cache, self.m, e.seq_lens, e.block_table, e.block_size, self.o, self.g)
         if self.tc:
-            K.grouped_decode_tc(*args, self.splits, self.part_o, self.part_ml)
+            K.grouped_decode_tc(*args, self.splits, self.part_o, self.part_ml, head_gate=self.head_gate, **self.m.sight)
         else:
-            K.grouped_decode(*args)
+            K.grouped_decode(*args, head_gate=self.head_gate, **self.m.sight)
 
     def step(self, h, out):
-        self.e.gemm(h, self.m.w_in, self.acc_in)
+        self.e.gemm(h, self.w_in, self.acc_in)
         self.prepare()
         self.attend()
         self.e.gemm(self.o, self.m.o, out)
@@ -264,7 +274,7 @@ class _RgLruSlots:
         self.e.gemm(self.y, self.m.o, out)
 
 
-SLOTS = {"latent_attention": _LatentSlots, "mlstm": _MLstmSlots, "attention": _AttentionSlots, "rglru": _RgLruSlots}
+SLOTS = {"latent_attention": _LatentSlots, "mlstm": _MLstmSlots, "attention": _AttentionSlots, "attention_2": _AttentionSlots, "rglru": _RgLruSlots}
 
 
 class _Pages:
@@ -277,6 +287,9 @@ class _Pages:
         return self.e.slots[li].prompt_target(self)
 
     recurrent_state = paged_cache
+
+    def last_tokens(self):
+        return dict(tok_slot=self.tok_slot, prev=self.e.last_token)
 
 
 class LayeredRolloutEngine(RolloutEngine):
@@ -313,6 +326,7 @@ class LayeredRolloutEngine(RolloutEngine):
         # weight-streaming GEMM: bf16, at most 128 rows, rows of 16 bytes; other shapes and fp32 use the library
         self._own_gemm = (os.environ.get("TRL_B200_DECODE_GEMM", "own") != "cublas" and self.dtype == torch.bfloat16
                           and B <= 128)
+        self.last_token = torch.zeros(B, dtype=torch.int64, device=self.dev) if cfg.pairs else None
         self.slots: list = []  # a layer may look up an earlier one
         for li, (s, l) in enumerate(zip(cfg.layers, self.model.layers)):
             self.slots.append(SLOTS[s.kind](self, l.mixer, li))
@@ -333,6 +347,8 @@ class LayeredRolloutEngine(RolloutEngine):
     def _copy_slots(self, dst, src):
         for s in self.slots:
             s.copy_slots(dst, src)
+        if self.last_token is not None:
+            self.last_token[dst] = self.last_token[src]
 
     def _head(self, hidden):
         return mx.linear(hidden, self.model.lm_head_weight)
@@ -367,22 +383,31 @@ class LayeredRolloutEngine(RolloutEngine):
         from ..ops import cuda as K
         from ..ops import cuda_mixers as KM
 
-        m, x, h, acc, dt = self.model, self._x, self._h, self._acc, self.dtype
-        KM.embed_scaled(self.next_input, m.embed_tokens, self.cfg.embed_scale, out=x)
+        m, x, h, acc = self.model, self._x, self._h, self._acc
+        if m.pair_embed is None:
+            KM.embed_scaled(self.next_input, m.embed_tokens, self.cfg.embed_scale, out=x)
+        else:
+            p = self.cfg.pairs
+            KM.embed_pairs(self.next_input, m.embed_tokens, self.cfg.embed_scale, m.pair_embed, p["mul_prev"], p["mul_cur"], self.seq_lens,
+                           prev=self.last_token, decode=True, out=x)
         delta = post = None  # sums not yet added to the stream, and the norm they pass first
+        now = dict(clear=True, out=h)
         for li, (layer, slots) in enumerate(zip(m.layers, self.slots)):
-            layer.norm1(x, dt, delta, post, clear=True, out=h)
+            layer.read_mixer(x, delta, post, **now)
             slots.step(h, acc)
             delta, post = acc, layer.norm1b
             if layer.mlp is not None:
-                layer.norm2(x, dt, delta, post, clear=True, out=h)
-                self.gemm(self.mlp_act(h, layer.mlp), layer.mlp.down, acc)
+                layer.read_mlp(x, delta, post, **now)
+                if isinstance(layer.mlp, ExpertMlp):
+                    self.experts(h, layer.mlp, acc)
+                else:
+                    self.gemm(self.mlp_act(h, layer.mlp), layer.mlp.down, acc)
                 post = layer.norm2b
             if layer.side is not None:
-                layer.side.stream(x, dt, delta, post, clear=True, out=h)
+                layer.read_side(x, delta, post, **now)
                 self.gemm(self.side_act(h, layer.side, li), layer.side.proj, acc)
                 post = layer.side.norm
-        m.norm(x, dt, delta, post, clear=True, out=h)
+        m.norm(x, self.dtype, delta, post, **now)
         if self._own_gemm and h.shape[1] % 8 == 0:
             return K.decode_gemm(h, m.lm_head_weight, out=self._logits_buf)
         return mx.linear(h, m.lm_head_weight)
@@ -390,17 +415,17 @@ class LayeredRolloutEngine(RolloutEngine):
     def mlp_act(self, h, mlp):
         """Activation of a feed-forward: fused into the product where the weight-streaming kernel runs."""
         from ..ops import cuda as K
-        from ..ops import cuda_mixers as KM
 
         act = self.scratch("act", self.max_seqs, mlp.down.shape[1])
-        own = self._own_gemm and h.shape[1] % 8 == 0
-        if isinstance(mlp, ClampedGluMlp):
-            if own:
-                return K.decode_gemm(h, mlp.gate_up, out=act, clamped_glu=mlp.glu)
-            return KM.clamped_glu(mx.linear(h, mlp.gate_up), *mlp.glu, out=act)
-        if own:
-            return K.decode_gemm(h, mlp.up, out=act, gelu=True)
-        return KM.gelu_erf(mx.linear(h, mlp.up), out=act)
+        if self._own_gemm and h.shape[1] % 8 == 0:
+            return K.decode_gemm(h, mlp.w_in, out=act, **mlp.fused)
+        return mlp.act(mx.linear(h, mlp.w_in), out=act)
+
+    def experts(self, h, mlp, out):
+        """Mixture of experts of the slots that are live; ``out`` (fp32) is stored to."""
+        z = self.sums("router", mlp.n)
+        self.gemm(h, mlp.router, z)
+        mx.experts(mlp, h, positions=self.seq_lens, logits=z, out=out)
 
     def side_act(self, h, side, li):
         from ..ops import cuda_mixers as KM

@@ -29,10 +29,13 @@ def main(argv=None) -> int:
 
     from .._native import lib_path
     from ..csrc.build import build
-    from ..models.layered import is_layered_dir
+    from ..models.layered import is_layered_dir, layered_kinds
 
     # a fresh checkout compiles what the model needs; an existing complete library is kept up to date
-    build(part="layered" if is_layered_dir(a.model) and not os.path.exists(lib_path("libtrl_b200_kernels.so")) else None)
+    if is_layered_dir(a.model) and not os.path.exists(lib_path("libtrl_b200_kernels.so")):
+        build(part="layered", kinds=layered_kinds(a.model))
+    else:
+        build()
     import torch
 
     from ..models.hf_io import load_model
