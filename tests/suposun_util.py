@@ -67,9 +67,9 @@ ONES = config([attention(heads=1, kv_heads=1, dim=8, mask=(1, 1), rot=(8, 7.0), 
 PLAIN = config([attention(rot=None, mask=None, mlp=ff(24)), attention_2(rot=None, mlp=ff(24))], width=40, pairs=None, scale=2.0)
 
 
-def make(cfg, dtype=torch.float32, device=None, seed=0):
-    """Model with every tensor random (bf16-representable), plus the same tensors in float64 by checkpoint name.  Router choices
-    are kept apart by corrections of a grid that the scores cannot cross by rounding alone too often."""
+def make(cfg, dtype=torch.float32, device=None, seed=0, clear=False):
+    """Model with every tensor random (bf16-representable), plus the same tensors in float64 by checkpoint name.  ``clear``:
+    corrections far apart, so that rounding cannot change which experts are chosen (their weights still vary)."""
     m = build_model(ModelArch.from_hf_dict(cfg), dtype=dtype, device=device).eval().requires_grad_(False)
     g = torch.Generator().manual_seed(seed)
     tensors = {}
@@ -81,7 +81,7 @@ def make(cfg, dtype=torch.float32, device=None, seed=0):
         elif leaf == "router":
             z = 1.5 * z / t.shape[1] ** 0.5
         elif leaf == "correction":
-            z = 0.4 * z
+            z = 2.0 * z.argsort() if clear else 0.4 * z
         elif t.ndim >= 2:
             z = z / t.shape[1] ** 0.5
         elif leaf == "norm" and ".mix." in name:
@@ -102,12 +102,11 @@ def tokens(n, vocab, seed=0):
     return torch.randint(0, vocab, (n,), generator=torch.Generator().manual_seed(seed)).tolist()
 
 
-def rel(got, want, worst=True):
-    """Worst (or middle) row error of centred logits over the typical size of a row."""
+def rel(got, want):
+    """Worst row error of centred logits over the typical size of a row."""
     got, want = got.double().cpu(), want.double()
     d = (got - want) - (got - want).mean(-1, keepdim=True)
-    e = d.pow(2).mean(-1).sqrt()
-    return float((e.max() if worst else e.median()) / want.var(-1).mean().sqrt())
+    return float(d.pow(2).mean(-1).sqrt().max() / want.var(-1).mean().sqrt())
 
 
 def logits(cfg, tensors, toks):

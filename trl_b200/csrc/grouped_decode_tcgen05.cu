@@ -162,6 +162,7 @@ grouped_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_
       GtItem it;
       for (int item = gt_next(p, blockIdx.x, n_items, it); item < n_items && ok; item = gt_next(p, item + gridDim.x, n_items, it)) {
         const int last_page = (it.len - 1) / p.block_size;
+        const int first_page = p.window > 0 ? max(0, it.len - p.window) / p.block_size : 0, kept_page = (p.keep - 1) / p.block_size;
         const int* bt = p.block_table + (size_t)it.b * p.max_blocks;
         for (int t = it.t0; t < it.t1; ++t, ++m) {
           const int stage = m % p.stages;
@@ -172,8 +173,11 @@ grouped_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_
           uint8_t* st = smem + (size_t)stage * stage_bytes;
           mbar_expect_tx(&full_bar[stage], (uint32_t)(p.nk + p.nv) * GT_BOX);
           for (int g = 0; g < ppt; ++g) {
-            // pages past the sequence's last one: that one again, its scores are masked
-            const int row = bt[min(it.tile(t) * ppt + g, last_page)] * p.block_size;
+            // pages past the sequence's last one, past the kept tokens, before the window: the nearest one that holds visible
+            // tokens instead; the scores of such places are masked
+            int page = it.tile(t) * ppt + g;
+            if (page > kept_page && page < first_page) page = t < it.kt ? kept_page : first_page;
+            const int row = bt[min(page, last_page)] * p.block_size;
             uint8_t* dst = st + g * p.block_size * 128;
             for (int i = 0; i < p.nk; ++i) tma_load_3d(dst + i * GT_BOX, &tm_k, &full_bar[stage], 64 * i, it.kvh, row);
             for (int i = 0; i < p.nv; ++i) tma_load_3d(dst + k_bytes + i * GT_BOX, &tm_v, &full_bar[stage], 64 * i, it.kvh, row);

@@ -22,7 +22,8 @@
 //   * the output may be multiplied by a gate: one fp32 factor per token and head, or the sigmoid of bf16 logits per
 //     element;
 //   * keys are those of the same sequence, with a window those at distance < window and the first `keep` of the sequence: the
-//     tiles of a CTA are those that hold kept keys, then those of the window.
+//     tiles of a CTA are those that hold kept keys, then those of the window; the last kept tile is only as wide (in steps of
+//     32 keys) as the kept keys reach.
 #include "mixers.cuh"
 
 namespace trlb {
@@ -82,10 +83,10 @@ __device__ __forceinline__ uint32_t la_visible(int c, int first, int last, int k
 // First pass over a row of scores: the largest visible one and (SPAN) the largest magnitude of any.  Loops over 32 scores stay
 // rolled and tiles without masked keys have code of their own: instruction fetch and count are what limits these passes.
 template <bool SPAN, bool FULL>
-__device__ __forceinline__ float2 la_row_max(uint32_t ts, int first, int last, int kept) {
+__device__ __forceinline__ float2 la_row_max(uint32_t ts, int width, int first, int last, int kept) {
   float mx[2] = {-INFINITY, -INFINITY}, mn[2] = {INFINITY, INFINITY};
 #pragma unroll 1
-  for (int c = 0; c < 128; c += 32) {
+  for (int c = 0; c < (FULL ? LA_BN : width); c += 32) {
     float v[32];
     tmem_ld_32x32(ts + c, v);
     const uint32_t seen = FULL ? 0u : la_visible(c, first, last, kept);
@@ -102,10 +103,10 @@ __device__ __forceinline__ float2 la_row_max(uint32_t ts, int first, int last, i
 
 // Second pass: probabilities, as value and remainder, in place.  LEVEL -1: no cap.  Returns their sum.
 template <int LEVEL, bool FULL>
-__device__ __forceinline__ float la_probs(const MixerAttnTc& p, uint32_t ts, float neg_m, int first, int last, int kept) {
+__device__ __forceinline__ float la_probs(const MixerAttnTc& p, uint32_t ts, int width, float neg_m, int first, int last, int kept) {
   float sum[2] = {0.f, 0.f};
 #pragma unroll 1
-  for (int c = 0; c < 128; c += 32) {
+  for (int c = 0; c < (FULL ? LA_BN : width); c += 32) {
     float v[32];
     tmem_ld_32x32(ts + c, v);
     const uint32_t seen = FULL ? 0u : la_visible(c, first, last, kept);
@@ -166,6 +167,7 @@ mixer_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_con
   const int kt = min((p.keep + LA_BN - 1) / LA_BN, lo);  // tiles of kept keys before the window
   const int n_kv = kt + hi - lo + 1;  // >= 1: a token sees itself
   auto tile_at = [&](int j) { return j < kt ? j : lo + j - kt; };
+  auto width_at = [&](int j) { return j < kt ? min(LA_BN, (p.keep - j * LA_BN + 31) & ~31) : LA_BN; };
 
   if (threadIdx.x == 0) {
     mbar_init(q_full, 1);
@@ -227,7 +229,6 @@ mixer_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_con
   } else if (warp == 1) {
     // ---------------- MMA issuer ----------------
     if (lane == 0) {
-      const uint32_t idesc_s = umma_idesc_bf16_major(LA_BM, LA_BN, false, false);
       const uint32_t idesc_o = umma_idesc_bf16_major(LA_BM, (p.vdim + 15) & ~15, false, true);  // V is MN-major
       const uint64_t q_d = umma_desc_kmajor_sw128(smem_u32(q_s)), k_d = umma_desc_kmajor_sw128(smem_u32(k_s));
       const uint64_t v_d = umma_desc_mnmajor_sw128(smem_u32(v_s), LA_BOX);
@@ -238,6 +239,7 @@ mixer_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_con
         if (!mbar_wait(&k_full[kst], (uint32_t)((j / p.k_stages) & 1), abort_flag, p.status, 1220 + kst)) return false;
         tc_fence_after();
         const uint64_t k_t = desc_at(k_d, (uint32_t)kst * k_bytes);
+        const uint32_t idesc_s = umma_idesc_bf16_major(LA_BM, width_at(j), false, false);
         uint32_t acc = 0;
         for (int i = 0; i < p.nn + p.nr; ++i) {
           const int left = i < p.nn ? p.dim - 64 * i : p.rot - 64 * (i - p.nn);
@@ -261,11 +263,12 @@ mixer_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_con
         if (!mbar_wait(&v_full[s], (uint32_t)((j / p.v_stages) & 1), abort_flag, p.status, 1250 + s)) break;
         tc_fence_after();
         const uint64_t v_t = desc_at(v_d, (uint32_t)s * v_bytes);
+        const int steps = width_at(j) / 16;
         // 32 keys are 16 columns of values and 16 of remainders, 16 keys an MMA step
         for (int half = 0; half < 2; ++half)
 #pragma unroll
           for (int kk = 0; kk < LA_BN / 16; ++kk)
-            umma_bf16_ts(tmem_base + NB * 128, tmem_base + (uint32_t)(sb * LA_BN + (kk >> 1) * 32 + half * 16 + (kk & 1) * 8),
+            if (kk < steps) umma_bf16_ts(tmem_base + NB * 128, tmem_base + (uint32_t)(sb * LA_BN + (kk >> 1) * 32 + half * 16 + (kk & 1) * 8),
                          desc_at(v_t, kk * 2048), idesc_o, (j | half | kk) != 0);
         umma_commit(o_full);
         umma_commit(&v_empty[s]);
@@ -287,15 +290,15 @@ mixer_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_con
     bool ok = true;
     for (int j = 0; j < n_kv && ok; ++j) {
       const int s = j % NB;
-      const int key0 = tile_at(j) * LA_BN;
-      const bool full = q_first + LA_BM <= len && key0 + LA_BN - 1 <= q_first &&
+      const int key0 = tile_at(j) * LA_BN, width = width_at(j);
+      const bool full = width == LA_BN && q_first + LA_BM <= len && key0 + LA_BN - 1 <= q_first &&
                         (p.window <= 0 || key0 >= q_first + LA_BM - p.window || key0 + LA_BN <= p.keep);
       ok = __all_sync(0xffffffffu, mbar_wait(&s_full[s], (uint32_t)((j / NB) & 1), abort_flag, p.status, 1270 + s));
       if (!ok) break;
       tc_fence_after();
       const uint32_t ts = tmem_base + lane_off + (uint32_t)s * LA_BN;
       const int first = k_min - key0, last = k_max - key0, kept = p.keep - key0;
-      const float2 top = full ? la_row_max<CAP, true>(ts, first, last, kept) : la_row_max<CAP, false>(ts, first, last, kept);
+      const float2 top = full ? la_row_max<CAP, true>(ts, width, first, last, kept) : la_row_max<CAP, false>(ts, width, first, last, kept);
       const float mx = top.x;
       int level = -1;
       float m_tile = mx * p.scale_log2;
@@ -330,10 +333,10 @@ mixer_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_con
       l_run *= alpha;
       const float neg_m = m_ref == -INFINITY ? 0.f : -m_ref;
       float sum;
-      if (!CAP) sum = full ? la_probs<-1, true>(p, ts, neg_m, first, last, kept) : la_probs<-1, false>(p, ts, neg_m, first, last, kept);
-      else if (level == 0) sum = full ? la_probs<0, true>(p, ts, neg_m, first, last, kept) : la_probs<0, false>(p, ts, neg_m, first, last, kept);
-      else if (level == 1) sum = la_probs<1, false>(p, ts, neg_m, first, last, kept);
-      else sum = la_probs<2, false>(p, ts, neg_m, first, last, kept);
+      if (!CAP) sum = full ? la_probs<-1, true>(p, ts, width, neg_m, first, last, kept) : la_probs<-1, false>(p, ts, width, neg_m, first, last, kept);
+      else if (level == 0) sum = full ? la_probs<0, true>(p, ts, width, neg_m, first, last, kept) : la_probs<0, false>(p, ts, width, neg_m, first, last, kept);
+      else if (level == 1) sum = la_probs<1, false>(p, ts, width, neg_m, first, last, kept);
+      else sum = la_probs<2, false>(p, ts, width, neg_m, first, last, kept);
       // P.V(last) completes phase `last` of o_full, and may do so before this thread looks: phase last - 1 has to be seen
       // first.  (With one S buffer the last S was issued after P.V(last - 1), so s_full has shown it.)
       if (NB == 2 && j > 0 && j == n_kv - 1)

@@ -278,6 +278,16 @@ PRESETS: dict[str, dict] = {
                 dict(type="attention", mlp=dict(kind="dense", ff=96, limit=6.0),
                      mixer=dict(heads=4, kv_heads=2, dim=16, vdim=16, scale=0.25, softcap=30.0, q_temp=dict(coef=0.1, every=128),
                                 kv_from=0))]),
+    "tiny-suposun": dict(
+        architecture="Suposun", vocab=1024, width=64, norm=dict(eps=1e-5), logit_scale=0.5,
+        embedding=dict(scale=8.0, bigram=dict(buckets=499, mul_prev=23, mul_cur=7)),
+        layers=[dict(type="attention", mlp=dict(kind="moe", expert=dict(ff=32, limit=4.0), router=dict(experts=4, top=2)),
+                     mixer=dict(heads=4, kv_heads=2, dim=16, vdim=16, scale=0.25, softcap=15.0, mask=dict(size=24, keep_first=2),
+                                rot=dict(base=1e4, dims=8, scaling=dict(factor=4.0, original=256, fast=16.0, slow=1.0)))),
+                dict(type="attention_2", mlp=dict(kind="dense", ff=96),
+                     mixer=dict(heads=4, kv_heads=4, dim=16, vdim=16, scale=0.25, rot=dict(base=1e5, dims=16))),
+                dict(type="attention_2", mlp=dict(kind="moe", expert=dict(ff=32, limit=4.0), router=dict(experts=4, top=2)),
+                     mixer=dict(heads=4, kv_heads=4, dim=16, vdim=16, scale=0.25, rot=dict(base=1e5, dims=16), kv_from=1))]),
 }
 
 
