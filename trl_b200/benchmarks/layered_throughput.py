@@ -1,7 +1,7 @@
 """Prompt and decode throughput of a layered design beside the closest flat decoder of the same width, depth and
 parameter count (random weights, bf16, one GPU), through the serving engine.
 
-    python -m trl_b200.benchmarks.layered_throughput [--design zorelorn|povusun] [--sizes small,base] [--kernels]
+    python -m trl_b200.benchmarks.layered_throughput [--design zorelorn|povusun|suposun] [--sizes small,base] [--kernels]
 
 Prompt: packed prompts through the engine's prompt forward into its cache.  Decode: replays of the captured step (CUDA
 graph, sampler included) with every slot at the given context.  CUDA events after warm-up; the weights of a step are
@@ -14,11 +14,14 @@ import os
 
 import torch
 
-# width, heads (attention of every kind), ff; Zorelorn: query latent, mLSTM heads, pairs of layers; Povusun: side input, quads
+# width, heads (attention of every kind), ff; Zorelorn: query latent, mLSTM heads, pairs of layers; Povusun: side input, quads;
+# Suposun: experts of every second layer, of which a token runs `top` of width `eff` (ff = top x eff), quads
 SIZES = {"zorelorn": {"small": dict(width=2048, heads=16, q_rank=768, ff=8192, mheads=4, pairs=4),
                       "base": dict(width=4096, heads=32, q_rank=1536, ff=16384, mheads=8, pairs=4)},
          "povusun": {"small": dict(width=2048, heads=16, ff=6144, side=256, quads=2),
-                     "base": dict(width=4096, heads=32, ff=12288, side=256, quads=2)}}
+                     "base": dict(width=4096, heads=32, ff=12288, side=256, quads=2)},
+         "suposun": {"small": dict(width=2048, heads=16, ff=4096, eff=1024, experts=48, top=4, quads=2),
+                     "base": dict(width=4096, heads=32, ff=8192, eff=2048, experts=32, top=4, quads=2)}}
 VOCAB = 32768
 
 
@@ -44,14 +47,37 @@ def povusun_config(width, heads, ff, side, quads):
     return dict(architecture="Povusun", vocab=VOCAB, width=width, norm=dict(eps=1e-6), token_side=dict(dim=side), layers=layers)
 
 
+def suposun_config(width, heads, ff, eff, experts, top, quads, window=512):
+    dense, moe = dict(kind="dense", ff=ff), dict(kind="moe", expert=dict(ff=eff, limit=7.0), router=dict(experts=experts, top=top))
+    rot = dict(base=5e5, dims=64, scaling=dict(factor=4.0, original=4096, fast=32.0, slow=1.0))
+    near = dict(heads=heads, kv_heads=heads // 4, dim=128, vdim=128, scale=128 ** -0.5, softcap=30.0, mask=dict(size=window, keep_first=4), rot=rot)
+    far = dict(heads=heads, kv_heads=heads // 4, dim=128, vdim=128, scale=128 ** -0.5, rot=dict(base=1e6, dims=128))
+    layers = []
+    for i in range(quads):  # the last layer of every second four reads the cache of the one four layers before
+        own = dict(far, kv_from=4 * i - 1) if i % 2 else far
+        layers += [dict(type="attention", mixer=near, mlp=m) for m in (dense, moe, dense)] + [dict(type="attention_2", mixer=own, mlp=moe)]
+    return dict(architecture="Suposun", vocab=VOCAB, width=width, norm=dict(eps=1e-6), logit_scale=0.5, layers=layers,
+                embedding=dict(scale=1.0, bigram=dict(buckets=8191, mul_prev=131, mul_cur=7)))
+
+
+CONFIGS = {"zorelorn": zorelorn_config, "povusun": povusun_config, "suposun": suposun_config}
+
+
 def layered_config(design, s):
-    return zorelorn_config(**s) if design == "zorelorn" else povusun_config(**s)
+    return CONFIGS[design](**s)
 
 
 def flat_config(s, depth, target, tied):
-    """Llama-type decoder of the same width and depth whose feed-forward width brings it to ``target`` parameters."""
+    """Flat decoder of the same width and depth brought to ``target`` parameters: of the Llama type by the width of its
+    feed-forward, or, where the layered design has experts, of the Qwen3-MoE type with experts in every layer by their number."""
     from ..models.configuration import ModelArch
 
+    if "experts" in s:
+        kw = dict(model_type="qwen3_moe", vocab_size=VOCAB, hidden_size=s["width"], num_hidden_layers=depth, intermediate_size=s["ff"],
+                  num_attention_heads=s["width"] // 128, num_key_value_heads=max(1, s["width"] // 512), head_dim=128, rope_theta=5e5,
+                  tie_word_embeddings=tied, moe_intermediate_size=s["eff"], num_experts_per_tok=s["top"])
+        one, two = (ModelArch(num_experts=n, **kw).num_parameters() for n in (s["top"], s["top"] + 1))
+        return ModelArch(num_experts=s["top"] + max(0, round((target - one) / (two - one))), **kw)
     kw = dict(model_type="llama", vocab_size=VOCAB, hidden_size=s["width"], num_hidden_layers=depth,
               num_attention_heads=s["width"] // 128, num_key_value_heads=max(1, s["width"] // 512), head_dim=128,
               rope_theta=5e5, tie_word_embeddings=tied)
@@ -115,15 +141,16 @@ def run(sizes=("small", "base"), batch=64, prompt=1024, n_prompts=8, design="zor
         s = SIZES[design][name]
         arch = ModelArch.from_hf_dict(layered_config(design, s))
         depth = arch.num_hidden_layers
-        # the per-token table of a side input is looked up, not multiplied with: it does not count as size
-        n = arch.num_parameters() - VOCAB * depth * arch.side_dim
+        # tables of side inputs and token pairs are looked up, not multiplied with: they do not count as size
+        tables = VOCAB * depth * arch.side_dim + (arch.pairs["buckets"] + 1 if arch.pairs else 0) * arch.hidden_size
+        n = arch.num_parameters() - tables
         flat = flat_config(s, depth, n, arch.tie_word_embeddings)
         row = dict(design=design, size=name, layers=depth, width=s["width"], batch=batch, prompt=f"{n_prompts}x{prompt}",
                    decode_context=prompt)
         for key, cfg in (("layered", arch), ("flat", flat)):
             torch.manual_seed(0)
             model = build_model(cfg, dtype=torch.bfloat16, device="cuda").eval().requires_grad_(False)
-            params = sum(p.numel() for p in model.parameters()) - (VOCAB * depth * arch.side_dim if key == "layered" else 0)
+            params = sum(p.numel() for p in model.parameters()) - (tables if key == "layered" else 0)
             row[key] = dict(params_m=round(params / 1e6), **measure(model, batch, prompt, n_prompts))
             del model
             torch.cuda.empty_cache()
@@ -177,10 +204,11 @@ def kernel_table(size="base", batch=64, prompt=1024, n_prompts=8, iters=20, desi
     from ..rollout.engine import make_engine
 
     s = dict(SIZES[design][size], **(dict(pairs=1) if design == "zorelorn" else dict(quads=1)))
+    kernels = {"zorelorn": zorelorn_kernels, "povusun": povusun_kernels, "suposun": suposun_kernels}[design]
     model = build_model(ModelArch.from_hf_dict(layered_config(design, s)), dtype=torch.bfloat16, device="cuda").eval().requires_grad_(False)
     eng = make_engine(model, max_num_seqs=batch, max_model_len=prompt + 64)
     row = KernelTimer(iters)
-    (zorelorn_kernels if design == "zorelorn" else povusun_kernels)(s, model, eng, batch, prompt, n_prompts, row)
+    kernels(s, model, eng, batch, prompt, n_prompts, row)
     flat_kernels(s, batch, prompt, n_prompts, row)
     K.check_status()
     return row.rows
@@ -262,6 +290,102 @@ def povusun_kernels(s, model, eng, batch, prompt, n_prompts, row):
     row("decode gate/up + clamped unit", lambda: eng.mlp_act(hb, mlp), mlp.gate_up.numel() * 2)
     row("decode side gate gemm", lambda: eng.gemm(hb, side.gate, eng.sums("side", side.dim)), side.gate.numel() * 2)
     row("decode side gate", lambda: KM.side_gate(eng.sums("side", side.dim), eng.next_input, model.side_embed, 0, clear=True), B * side.dim * 12)
+
+
+@torch.no_grad()
+def suposun_kernels(s, model, eng, batch, prompt, n_prompts, row):
+    from ..models.decoder import SeqCtx
+    from ..ops import cuda as K
+    from ..ops import cuda_mixers as KM
+    from ..ops import mixers as mx
+
+    near, far, glu, moe = model.layers[0].mixer, model.layers[3].mixer, model.layers[0].mlp, model.layers[1].mlp
+    T, W, dev, bf, B = n_prompts * prompt, s["width"], "cuda", torch.bfloat16, batch
+    ctx = SeqCtx.from_lengths([prompt] * n_prompts, dev)
+    h, post = torch.randn(T, W, device=dev, dtype=bf), model.layers[0].norm1b
+    x, d = torch.randn(T, W, device=dev), torch.randn(T, W, device=dev)
+    slots = torch.arange(n_prompts, device=dev, dtype=torch.int32).repeat_interleave(prompt)
+    pages = eng._page_writer(slots, ctx, None)
+    paged_context(eng, prompt)
+    ids, p = torch.randint(0, VOCAB, (T,), device=dev), model.config.pairs
+    row("prompt embedding + pair embedding", lambda: KM.embed_pairs(ids, model.embed_tokens, 1.0, model.pair_embed, p["mul_prev"], p["mul_cur"], ctx.positions),
+        T * W * 8)
+    row("prompt norm of output + layer scale + residual", lambda: KM.rms_residual(x, d, post.weight, None, post.eps, bf, shift=1.0, post_scale=post.scale), T * W * 14)
+
+    def qkv(m, li, name):
+        y = mx.linear(h, m.w_in)
+        keys = None if m.values else torch.empty(T, m.kv_heads * m.dim, device=dev, dtype=bf)
+        gate = torch.empty(T, m.heads, device=dev) if m.gate else None
+        table = m.rope.table(prompt, dev)
+        kv = m.kv_heads * (m.dim + m.vdim)
+        # in place: queries (and keys) read and written, values read, pages written; keys apart: read once, written twice and copied
+        moved = 2 * m.heads * m.dim + (2 * m.kv_heads * m.dim + m.kv_heads * m.vdim if m.values else 2 * m.kv_heads * m.dim) + kv
+        row(f"prompt preparation of {name}", lambda: KM.attn_prep(y, m, ctx.positions, None, table=table, k=keys, head_gate=gate, **m.prep,
+                                                                  **eng.slots[li].prompt_target(pages)), T * 2 * moved)
+        q, k, v, g = y[:, : sum(m.parts)].split(m.parts, 1)
+        return (q, k, v, None) if m.values else (q, keys, k, gate)
+
+    def attend(m, q, k, v, g, name, window, **kw):
+        win = min(window or prompt, prompt)
+        pairs = n_prompts * (win * (win + 1) / 2 + (prompt - win) * win)
+        row(name, lambda: KM.mixer_attn(q, k, v, heads=m.heads, kv_heads=m.kv_heads, scale=m.scale, window=window, gate=g, ctx=ctx, **kw),
+            T * 2 * (q.shape[1] + k.shape[1] + v.shape[1] + m.heads * m.vdim), 2 * pairs * m.heads * (m.dim + m.vdim))
+
+    t = qkv(near, 0, "attention (keys as values)")
+    attend(near, *t, "prompt windowed attention (capped, sink, gated)", near.window, keep=near.keep, cap=near.cap, sink=near.sink)
+    attend(near, *t, "prompt windowed attention without cap", near.window, keep=near.keep, sink=near.sink)
+    attend(near, *t, "prompt attention without window (capped, sink, gated)", None, cap=near.cap, sink=near.sink)
+    t = qkv(far, 3, "attention_2 (norms over all heads)")
+    attend(far, *t, "prompt attention_2", None)
+    del t
+    z = torch.randn(T, 2 * s["ff"], device=dev, dtype=bf)
+    row("prompt GELU unit", lambda: KM.gelu_glu(z), z.numel() * 3)
+    del z
+    E, top, n = moe.n, moe.top, moe.ff
+    R = T * top
+    zr = mx.linear_f32(h, moe.router)
+    row("prompt router choice", lambda: KM.moe_route(zr, moe.correction, top), T * (E * 4 + top * 12))
+    choice, rank, weight, counts = KM.moe_route(zr, moe.correction, top)
+    row("prompt gather by expert", lambda: KM.moe_gather(h, choice, rank, counts), T * W * 2 + R * W * 2)
+    xs, at, offsets = KM.moe_gather(h, choice, rank, counts)
+    row("prompt experts gate/up + clamped unit", lambda: K.grouped_gemm(xs, moe.gate_up, offsets, n, clamped_glu=moe.glu),
+        moe.gate_up.numel() * 2 + R * (W + n) * 2, 4 * R * W * n)
+    act = K.grouped_gemm(xs, moe.gate_up, offsets, n, clamped_glu=moe.glu)
+    row("prompt experts down", lambda: K.grouped_gemm(act, moe.down, offsets, W), moe.down.numel() * 2 + R * (W + n) * 2, 2 * R * W * n)
+    ys = K.grouped_gemm(act, moe.down, offsets, W)
+    row("prompt weighted sum", lambda: KM.moe_sum(ys, at, weight), R * W * 2 + T * W * 4)
+    row("prompt experts, all of it", lambda: mx.experts(moe, h), moe.gate_up.numel() * 3 + T * W * 6, 6 * R * W * n)
+    del xs, act, ys
+
+    a, r = eng.slots[0], eng.slots[3]
+    hb, xb, db = torch.randn(B, W, device=dev, dtype=bf), torch.randn(B, W, device=dev), torch.randn(B, W, device=dev)
+    row("decode embedding + pair embedding", lambda: KM.embed_pairs(eng.next_input, model.embed_tokens, 1.0, model.pair_embed, p["mul_prev"], p["mul_cur"],
+                                                                    eng.seq_lens, prev=eng.last_token, decode=True, out=xb), B * W * 8)
+    row("decode norm of output + layer scale + residual", lambda: KM.rms_residual(xb, db, post.weight, None, post.eps, bf, clear=True, out=hb, shift=1.0,
+                                                                                 post_scale=post.scale), B * W * 18)
+    kv = near.kv_heads * 256
+    row("decode gemm input attention", lambda: K.decode_gemm(hb, a.w_in, y32=a.acc_in), a.w_in.numel() * 2)
+    row("decode preparation of attention + cache", a.prepare, a.acc_in.numel() * 10)
+    row("decode gemm input attention_2", lambda: K.decode_gemm(hb, r.w_in, y32=r.acc_in), r.w_in.numel() * 2)
+    row("decode preparation of attention_2 + cache", r.prepare, r.acc_in.numel() * 10)
+    seen = min(prompt + 1, near.window + near.keep)
+    row("decode windowed attention (capped, sink, gated)", a.attend, B * seen * kv * 2 + 4 * a.q.numel(), 2 * B * seen * near.heads * 256)
+    row("decode attention_2", r.attend, B * (prompt + 1) * kv * 2 + 4 * r.q.numel(), 2 * B * (prompt + 1) * far.heads * 256)
+    row("decode gate/up + GELU unit", lambda: eng.mlp_act(hb, glu), glu.gate_up.numel() * 2)
+    zb = torch.zeros(B, E, device=dev)
+    row("decode router product", lambda: K.decode_gemm(hb, moe.router, y32=zb), moe.router.numel() * 2)
+    zb = mx.linear_f32(hb, moe.router)
+    row("decode router choice", lambda: KM.moe_route(zb, moe.correction, top, positions=eng.seq_lens), B * (E * 4 + top * 12))
+    choice, rank, weight, counts = KM.moe_route(zb, moe.correction, top)
+    row("decode gather by expert", lambda: KM.moe_gather(hb, choice, rank, counts), B * W * 2 * (1 + top))
+    xs, at, offsets = KM.moe_gather(hb, choice, rank, counts)
+    used = int((counts > 0).sum())
+    row("decode experts gate/up + clamped unit", lambda: K.grouped_gemm(xs, moe.gate_up, offsets, n, clamped_glu=moe.glu), used * 4 * W * n)
+    act = K.grouped_gemm(xs, moe.gate_up, offsets, n, clamped_glu=moe.glu)
+    row("decode experts down", lambda: K.grouped_gemm(act, moe.down, offsets, W), used * 2 * W * n)
+    ys = K.grouped_gemm(act, moe.down, offsets, W)
+    row("decode weighted sum", lambda: KM.moe_sum(ys, at, weight, out=db), B * W * (2 * top + 4))
+    row("decode experts, all of it", lambda: eng.experts(hb, moe, db), used * 6 * W * n)
 
 
 @torch.no_grad()
@@ -368,6 +492,25 @@ def flat_kernels(s, batch, prompt, n_prompts, row):
     gw = torch.randn(2 * s["ff"], W, device=dev, dtype=bf)
     act = torch.empty(batch, s["ff"], device=dev, dtype=bf)
     row("flat: decode gate/up + swiglu", lambda: K.decode_gemm(x, gw, out=act, swiglu=True), gw.numel() * 2)
+    if "experts" in s:
+        flat_moe_kernels(s, batch, T, row)
+
+
+def flat_moe_kernels(s, batch, T, row):
+    from ..ops import cuda as K
+    from ..ops import functional as F_
+
+    dev, bf, W, n, E, top = "cuda", torch.bfloat16, s["width"], s["eff"], s["experts"], s["top"]
+    router, gu, down = (torch.randn(*sh, device=dev, dtype=bf) * 0.02 for sh in ((E, W), (E, 2 * n, W), (E, W, n)))
+    for name, rows in (("prompt", T), ("decode", batch)):
+        R = rows * top
+        h, xs, act = (torch.randn(r, c, device=dev, dtype=bf) for r, c in ((rows, W), (R, W), (R, n)))
+        counts = torch.bincount(torch.randint(0, E, (R,), device=dev), minlength=E)
+        offsets = torch.cat([counts.new_zeros(1), counts.cumsum(0)]).int()
+        used = int((counts > 0).sum())
+        row(f"flat: {name} experts gate/up + swiglu", lambda: K.grouped_gemm(xs, gu, offsets, n, swiglu=True), used * 4 * W * n + R * (W + n) * 2, 4 * R * W * n)
+        row(f"flat: {name} experts down", lambda: K.grouped_gemm(act, down, offsets, W), used * 2 * W * n + R * (W + n) * 2, 2 * R * W * n)
+        row(f"flat: {name} experts, all of it", lambda: F_.moe_mlp(h, router, gu, down, top, True), used * 6 * W * n + rows * W * 4, 6 * R * W * n)
 
 
 def main():
