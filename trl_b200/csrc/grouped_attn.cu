@@ -219,6 +219,174 @@ attn_prep_kernel(const AttnPrep p, S* __restrict__ src, T* __restrict__ q_out, T
   }
 }
 
+// The same for sizes in multiples of 8 with heads of at most 256 elements: one block per row, 2^lanes_log2 threads with 8 elements
+// each per head, so that a row is read once into registers (also for norms over all heads) and moves in 16-byte pieces.  A block
+// takes its row in at most PREP_ROUNDS rounds.
+constexpr int PREP_ROUNDS = 4;
+
+__device__ __forceinline__ void load8(const float* p, float (&v)[8]) {
+  const float4 a = load4(p), b = load4(p + 4);
+  v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
+}
+__device__ __forceinline__ void load8(const __nv_bfloat16* p, float (&v)[8]) {
+  const uint4 u = *reinterpret_cast<const uint4*>(p);
+  const uint32_t w[4] = {u.x, u.y, u.z, u.w};
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const float2 f = unpack_bf16(w[i]);
+    v[2 * i] = f.x;
+    v[2 * i + 1] = f.y;
+  }
+}
+__device__ __forceinline__ void store8(float* p, const float (&v)[8]) {
+  store4(p, make_float4(v[0], v[1], v[2], v[3]));
+  store4(p + 4, make_float4(v[4], v[5], v[6], v[7]));
+}
+__device__ __forceinline__ void store8(__nv_bfloat16* p, const float (&v)[8]) {
+  *reinterpret_cast<uint4*>(p) = make_uint4(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]), pack_bf16(v[4], v[5]), pack_bf16(v[6], v[7]));
+}
+
+template <typename T, typename S, bool WHOLE>
+__global__ void __launch_bounds__(512)
+attn_prep_rows_kernel(const AttnPrep p, int lanes_log2, S* __restrict__ src, T* __restrict__ q_out, T* __restrict__ k_out,
+                      T* __restrict__ g_out, T* __restrict__ k_cache, T* __restrict__ v_cache) {
+  constexpr bool SUMS = !(sizeof(T) == 2 && sizeof(S) == 2);
+  __shared__ float red[WHOLE ? 64 : 1];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int row = blockIdx.x, lanes = 1 << lanes_log2, c = threadIdx.x & (lanes - 1), j0 = 8 * c;
+  const bool in_place = !SUMS || q_out == nullptr;
+  const int kv = p.has_kv ? p.kv_heads : 0, vv = p.has_v ? kv : 0, ge = p.gates == GATES_ELEMENT && !in_place ? p.heads : 0;
+  const int units = p.heads + kv + vv + ge;
+  const int q_n = p.heads * p.dim, k_n = kv * p.dim, v_n = vv * p.vdim;
+  S* r = src + (size_t)row * p.ld;
+  const int per_round = blockDim.x >> lanes_log2, u0 = threadIdx.x >> lanes_log2;
+  // where head u starts in the row
+  auto place = [&](int u) {
+    if (u < p.heads + kv) return u * p.dim;
+    return q_n + k_n + (u - p.heads - kv) * p.vdim;
+  };
+  float x[PREP_ROUNDS][8];
+  float sq = 0.f, sk = 0.f;
+#pragma unroll
+  for (int i = 0; i < PREP_ROUNDS; ++i) {
+    const int u = u0 + i * per_round;
+    const bool on = u < units && j0 < (u < p.heads + kv ? p.dim : p.vdim);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) x[i][e] = 0.f;
+    if (on) load8(r + place(u) + j0, x[i]);
+    if (WHOLE && on && u < p.heads + kv) {
+      float ss = 0.f;
+#pragma unroll
+      for (int e = 0; e < 8; ++e) ss += x[i][e] * x[i][e];
+      if (u < p.heads) sq += ss; else sk += ss;
+    }
+  }
+  if (WHOLE) {
+    const float2 s = block_sum2(sq, sk, red);
+    sq = 1.f / sqrtf(s.x / (float)q_n + p.eps);
+    sk = k_n > 0 ? 1.f / sqrtf(s.y / (float)k_n + p.eps) : 0.f;
+  }
+  const int pos = p.positions[row];
+  long long at = -1;
+  if (pos >= 0 && p.block_table != nullptr) {
+    const int slot = p.tok_slot ? p.tok_slot[row] : row;
+    if (slot >= 0 && pos / p.block_size < p.max_blocks)
+      at = (long long)p.block_table[(size_t)slot * p.max_blocks + pos / p.block_size] * p.block_size + pos % p.block_size;
+  }
+  // this thread's angles are the same in every head
+  const bool turns = j0 < p.rot && pos >= 0 && pos < p.table_len;
+  const int half = p.rot / 2, shift = half / 8;  // halves: the partner is `shift` threads away
+  const bool upper = j0 >= half;
+  float2 cs[8];
+  if (turns) {
+    const float2* t = p.table + (size_t)pos * half + (p.halves ? (upper ? j0 - half : j0) : j0 / 2);
+#pragma unroll
+    for (int e = 0; e < 8; ++e)
+      if (e < 4 || p.halves) cs[e] = t[e];
+  }
+#pragma unroll
+  for (int i = 0; i < PREP_ROUNDS; ++i) {
+    if (i * per_round >= units) break;  // uniform
+    const int u = u0 + i * per_round;
+    const bool normed = u < p.heads + kv, is_q = u < p.heads;
+    const bool on = u < units && j0 < (normed ? p.dim : p.vdim);
+    T* dst = nullptr;
+    T* paged = nullptr;
+    bool put = false;
+    if (on) {
+      if (is_q) {
+        if (!in_place) dst = q_out + ((size_t)row * p.heads + u) * p.dim;
+        put = in_place;
+      } else if (normed) {
+        const int h = u - p.heads;
+        if (k_out != nullptr) dst = k_out + ((size_t)row * kv + h) * p.dim;
+        put = in_place && k_out == nullptr;
+        if (at >= 0) {
+          paged = k_cache + (size_t)(at * kv + h) * p.dim;
+          if (vv == 0) store8(v_cache + (size_t)(at * kv + h) * p.dim + j0, x[i]);
+        }
+      } else if (u < p.heads + kv + vv) {
+        if (at >= 0) paged = v_cache + (size_t)(at * kv + u - p.heads - kv) * p.vdim;
+      } else {
+        dst = g_out + ((size_t)row * p.heads + u - p.heads - kv - vv) * p.vdim;
+      }
+    }
+    float s = WHOLE ? (is_q ? sq : sk) : 1.f;
+    if (!WHOLE) {
+      float ss = 0.f;
+#pragma unroll
+      for (int e = 0; e < 8; ++e) ss += x[i][e] * x[i][e];
+      for (int o = 1; o < lanes; o <<= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+      s = 1.f / sqrtf(ss / (float)p.dim + p.eps);
+    }
+    if (normed) {
+      if (is_q && p.temp != nullptr && pos >= 0 && pos < p.temp_len) s *= p.temp[pos];
+      const float* w = is_q ? p.q_w : p.k_w;
+      if (on && w != nullptr) {
+        float g[8];
+        load8(w + (WHOLE ? (size_t)(is_q ? u : u - p.heads) * p.dim : 0) + j0, g);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) x[i][e] *= s * g[e];
+      } else {
+#pragma unroll
+        for (int e = 0; e < 8; ++e) x[i][e] *= s;
+      }
+    }
+    if (p.rot > 0 && p.halves) {
+#pragma unroll
+      for (int e = 0; e < 8; ++e) {  // every lane takes part
+        const float down = __shfl_down_sync(0xffffffffu, x[i][e], shift, lanes), up = __shfl_up_sync(0xffffffffu, x[i][e], shift, lanes);
+        if (turns && normed) x[i][e] = upper ? x[i][e] * cs[e].x + up * cs[e].y : x[i][e] * cs[e].x - down * cs[e].y;
+      }
+    } else if (turns && normed) {
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const float a = x[i][2 * e], b = x[i][2 * e + 1];
+        x[i][2 * e] = a * cs[e].x - b * cs[e].y;
+        x[i][2 * e + 1] = b * cs[e].x + a * cs[e].y;
+      }
+    }
+    if (on) {
+      if (dst) store8(dst + j0, x[i]);
+      if (paged) store8(paged + j0, x[i]);
+      if (!in_place) {
+        const float zero[8] = {};
+        store8(r + place(u) + j0, zero);
+      } else if (put) {
+        store8(r + place(u) + j0, x[i]);
+      }
+    }
+  }
+  if (p.gates == GATES_HEAD) {
+    S* g = r + q_n + k_n + v_n;
+    for (int h = threadIdx.x; h < p.heads; h += blockDim.x) {
+      p.head_gate[(size_t)row * p.heads + h] = sigmoid_f(to_f(g[h]));
+      if (!in_place) g[h] = from_f<S>(0.f);
+    }
+  }
+}
+
 // ------------------------------------------------------------------------------------------------------------
 // Prompt attention, any size: one warp per (token, head).  Keys of token t are rows t - min(pos, window - 1) .. t of the
 // packed stream (pos counts from the token's own sequence start), so no sequence table is needed.  Keys may have a second
@@ -411,8 +579,24 @@ TRLB_API int trlb_attn_prep(void* src, int src_f32, long long ld, int rows, int 
   if (k_cache != nullptr && (v_cache == nullptr || block_table == nullptr || block_size <= 0)) return -250;
   AttnPrep p = {ld, rows, heads, kv_heads, dim, vdim, has_kv, has_kv && has_v, gates, eps, positions, tok_slot, temp, temp_len, q_w,
                 k_w, rot, halves, (const float2*)table, table_len, head_gate, k_cache ? block_table : nullptr, max_blocks, block_size};
-  const int units = heads + (has_kv ? kv_heads * (has_v ? 2 : 1) : 0) + (gates == GATES_ELEMENT && q_out != nullptr ? heads : 0) +
-                    (gates == GATES_HEAD ? 1 : 0);
+  const int row_units = heads + (has_kv ? kv_heads * (has_v ? 2 : 1) : 0) + (gates == GATES_ELEMENT && q_out != nullptr ? heads : 0);
+  const int widest = dim > vdim ? dim : vdim;
+  int lanes_log2 = 0;
+  while ((8 << lanes_log2) < widest) ++lanes_log2;
+  const int threads = row_units << lanes_log2;  // of one round
+  const auto aligned = [](const void* x) { return (reinterpret_cast<uintptr_t>(x) & 15) == 0; };
+  if (((dim | vdim | (int)(ld & 7)) & 7) == 0 && widest <= 256 && threads <= 512 * PREP_ROUNDS && rot % (halves ? 16 : 8) == 0 && aligned(src) &&
+      aligned(q_out) && aligned(k_out) && aligned(g_out) && aligned(k_cache) && aligned(v_cache) && aligned(q_w) && aligned(k_w)) {
+    const int least = (threads + PREP_ROUNDS - 1) / PREP_ROUNDS;
+    const int want = threads <= 256 ? threads : least <= 256 ? 256 : 512;
+    const dim3 block((want + 31) / 32 * 32);
+#define GO(TT, SS, WW) (int)trlb_host::launch_kernel(attn_prep_rows_kernel<TT, SS, WW>, dim3(rows), block, 0, st, PDL, p, lanes_log2, (SS*)src, (TT*)q_out, \
+                                                     (TT*)k_out, (TT*)g_out, (TT*)k_cache, (TT*)v_cache)
+    if (is_bf16) return src_f32 ? (whole ? GO(bf16, float, true) : GO(bf16, float, false)) : (whole ? GO(bf16, bf16, true) : GO(bf16, bf16, false));
+    return whole ? GO(float, float, true) : GO(float, float, false);
+#undef GO
+  }
+  const int units = row_units + (gates == GATES_HEAD ? 1 : 0);
   const dim3 grid(whole ? (unsigned)rows : (unsigned)(((long long)rows * units + 7) / 8));
   const dim3 blk(!whole ? 256 : units >= 16 ? 512 : units >= 8 ? 256 : 128);
 #define GO(TT, SS, WW) (int)trlb_host::launch_kernel(attn_prep_kernel<TT, SS, WW>, grid, blk, 0, st, PDL, p, (SS*)src, (TT*)q_out, (TT*)k_out, \

@@ -9,10 +9,12 @@
 // Columns 0-7 are the query heads.  Probabilities keep 32-bit precision: P enters as two bf16, the value in columns 0-7 and
 // its remainder in columns 8-15 of the same product (which has 16 columns anyway), and the two results are added.  A
 // persistent CTA per SM: warp 0 = TMA producer over a ring of K + V tiles, warp 1 = MMA issuer (S^T double-buffered in TMEM),
-// warps 2-5 = softmax (one thread per token) and output accumulation (one thread per value dimension, SLABS of 128).
+// warps 2-5 = softmax (one thread per token) and output accumulation (one thread per value dimension, SLABS of 128; HEADS bounds
+// the query heads of an item).  P and O^T have two buffers each: the output of a tile is collected after the probabilities of
+// the next one have been handed over, so that product and softmax overlap.
 // Scores may be capped (cap tanh(s / cap)); the softmax denominator may contain exp(sink[head]); the result may be multiplied by
-// the sigmoid of per-element gate logits or by a factor per head.  With a window only its tiles and those of the first `keep`
-// tokens, which stay visible, are read: the tiles of a slot are a list, kept ones first.
+// the sigmoid of per-element gate logits or by a factor per head.  With a window only its pages and those of the first `keep`
+// tokens, which stay visible, are read: the pages of a slot are a list, kept ones first, that is cut into tiles.
 // Splits leave fp32 partial sums that grouped_combine_kernel merges.
 #include "mixers.cuh"
 
@@ -21,7 +23,7 @@ namespace trlb {
 constexpr int GT_THREADS = 192;
 constexpr int GT_MAX_STAGES = 4;
 constexpr uint32_t GT_BOX = 128 * 64 * 2;  // 128 tokens x 64 dims
-constexpr uint32_t GT_P_BYTES = 4096;      // 2 halves x [16 rows x 64 tok]
+constexpr uint32_t GT_P_BYTES = 4096;      // 2 halves x [16 rows x 64 tok]; two such buffers
 
 struct GroupedDecodeTc {
   const __nv_bfloat16* q;     // [B, heads, dim]
@@ -66,9 +68,9 @@ __device__ __forceinline__ float gt_factor(float m, float L, const float* sink, 
 }
 
 struct GtItem {
-  int b, kvh, h0, nh, sp, len, t0, t1;  // t0 .. t1: places in the slot's list of tiles
-  int lo, kt;                           // first tile of the window, kept tiles before it
-  __device__ __forceinline__ int tile(int t) const { return t < kt ? t : lo + t - kt; }
+  int b, kvh, h0, nh, sp, len, t0, t1;  // t0 .. t1: tiles of the slot's list of pages
+  int lo, kp;                           // first page of the window, kept pages before it
+  __device__ __forceinline__ int page(int i) const { return i < kp ? i : lo + i - kp; }
 };
 
 __device__ __forceinline__ GtItem gt_item(const GroupedDecodeTc& p, int item) {
@@ -83,9 +85,10 @@ __device__ __forceinline__ GtItem gt_item(const GroupedDecodeTc& p, int item) {
   it.nh = min(8, p.group - g0);
   const int sl = p.seq_lens[it.b];
   it.len = (sl < 0 || sl >= p.max_blocks * p.block_size) ? 0 : sl + 1;  // the new token is in the cache already
-  it.lo = p.window > 0 ? max(0, it.len - p.window) >> 7 : 0;
-  it.kt = min((p.keep + 127) >> 7, it.lo);
-  const int n_t = it.kt + ((it.len + 127) >> 7) - it.lo;
+  const int bs = p.block_size;
+  it.lo = p.window > 0 ? max(0, it.len - p.window) / bs : 0;
+  it.kp = min((p.keep + bs - 1) / bs, it.lo);
+  const int n_t = ((it.kp + (it.len + bs - 1) / bs - it.lo) * bs + 127) >> 7;
   it.t0 = n_t * it.sp / p.splits;
   it.t1 = n_t * (it.sp + 1) / p.splits;
   return it;
@@ -101,7 +104,32 @@ __device__ __forceinline__ int gt_next(const GroupedDecodeTc& p, int item, int n
   return item;
 }
 
-template <int SLABS>
+// Maxima over the warp of N values a lane; lane i's result is that of value gt_slot<N>(i).  Each step halves the values a lane
+// holds: N - 1 + log2(32 / N) shuffles.
+template <int N>
+__device__ __forceinline__ int gt_slot(int lane) {
+  return N == 8 ? lane >> 2 & 7 : N == 4 ? lane >> 3 & 3 : N == 2 ? lane >> 4 & 1 : 0;
+}
+template <int N>
+__device__ __forceinline__ float gt_warp_max(const float (&s)[N], int lane) {
+  float v[N];
+#pragma unroll
+  for (int i = 0; i < N; ++i) v[i] = s[i];
+  int o = 16;
+#pragma unroll
+  for (int n = N / 2; n > 0; n >>= 1, o >>= 1) {
+    const bool up = lane & o;
+#pragma unroll
+    for (int i = 0; i < n; ++i) {
+      const float mine = up ? v[i + n] : v[i], other = up ? v[i] : v[i + n];
+      v[i] = fmaxf(mine, __shfl_xor_sync(0xffffffffu, other, o));
+    }
+  }
+  for (; o > 0; o >>= 1) v[0] = fmaxf(v[0], __shfl_xor_sync(0xffffffffu, v[0], o));
+  return v[0];
+}
+
+template <int SLABS, int HEADS>
 __global__ void __launch_bounds__(GT_THREADS, 1)
 grouped_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_constant__ CUtensorMap tm_v,
                          const GroupedDecodeTc p) {
@@ -111,13 +139,13 @@ grouped_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_
   const uint32_t k_bytes = (uint32_t)p.nk * GT_BOX, stage_bytes = k_bytes + 2 * SLABS * GT_BOX, q_bytes = (uint32_t)p.nk * 2048;
   uint8_t* q_s = smem + (size_t)p.stages * stage_bytes;  // two buffers
   uint8_t* p_s = q_s + 2 * q_bytes;
-  uint64_t* bars = reinterpret_cast<uint64_t*>(p_s + GT_P_BYTES);
+  uint64_t* bars = reinterpret_cast<uint64_t*>(p_s + 2 * GT_P_BYTES);
   uint64_t* full_bar = bars;                        // [GT_MAX_STAGES]
   uint64_t* empty_bar = full_bar + GT_MAX_STAGES;   // [GT_MAX_STAGES]
   uint64_t* sfull_bar = empty_bar + GT_MAX_STAGES;  // [2]
-  uint64_t* pfull_bar = sfull_bar + 2;
-  uint64_t* ofull_bar = pfull_bar + 1;
-  uint64_t* qfull_bar = ofull_bar + 1;              // [2]
+  uint64_t* pfull_bar = sfull_bar + 2;              // [2]
+  uint64_t* ofull_bar = pfull_bar + 2;              // [2]
+  uint64_t* qfull_bar = ofull_bar + 2;              // [2]
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(qfull_bar + 2);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
   float* red_m = reinterpret_cast<float*>(tmem_slot + 4);  // [2][4][8]
@@ -134,22 +162,26 @@ grouped_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_
     for (int s = 0; s < 2; ++s) {
       mbar_init(&sfull_bar[s], 1);
       mbar_init(&qfull_bar[s], 128);
+      mbar_init(&pfull_bar[s], 128);
+      mbar_init(&ofull_bar[s], 1);
     }
-    mbar_init(pfull_bar, 128);
-    mbar_init(ofull_bar, 1);
     *abort_flag = 0;
     mbar_fence_init();
     tma_prefetch_desc(&tm_k);
     tma_prefetch_desc(&tm_v);
   }
   if (warp == 1) {
-    tmem_alloc(tmem_slot, 64);  // S^T: 0, 16; O^T: 32, 48
+    tmem_alloc(tmem_slot, 32 + 32 * SLABS <= 64 ? 64 : 128);  // S^T: 0, 16; O^T: 32 + 16 (SLABS buffer + slab)
     tmem_relinquish();
     tc_fence_before();
   }
+  for (int i = threadIdx.x; i < (int)(2 * GT_P_BYTES / 16); i += GT_THREADS)  // rows of heads past HEADS stay zero
+    reinterpret_cast<uint4*>(p_s)[i] = make_uint4(0, 0, 0, 0);
+  fence_proxy_async_smem();
   __syncthreads();
   tc_fence_after();
   const uint32_t tmem_base = *tmem_slot;
+  const int ppt = 128 / p.block_size;
   pdl_launch_dependents();
   pdl_wait();
 
@@ -158,11 +190,9 @@ grouped_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_
     if (lane == 0) {
       int m = 0;
       bool ok = true;
-      const int ppt = 128 / p.block_size;
       GtItem it;
       for (int item = gt_next(p, blockIdx.x, n_items, it); item < n_items && ok; item = gt_next(p, item + gridDim.x, n_items, it)) {
         const int last_page = (it.len - 1) / p.block_size;
-        const int first_page = p.window > 0 ? max(0, it.len - p.window) / p.block_size : 0, kept_page = (p.keep - 1) / p.block_size;
         const int* bt = p.block_table + (size_t)it.b * p.max_blocks;
         for (int t = it.t0; t < it.t1; ++t, ++m) {
           const int stage = m % p.stages;
@@ -173,11 +203,8 @@ grouped_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_
           uint8_t* st = smem + (size_t)stage * stage_bytes;
           mbar_expect_tx(&full_bar[stage], (uint32_t)(p.nk + p.nv) * GT_BOX);
           for (int g = 0; g < ppt; ++g) {
-            // pages past the sequence's last one, past the kept tokens, before the window: the nearest one that holds visible
-            // tokens instead; the scores of such places are masked
-            int page = it.tile(t) * ppt + g;
-            if (page > kept_page && page < first_page) page = t < it.kt ? kept_page : first_page;
-            const int row = bt[min(page, last_page)] * p.block_size;
+            // pages past the sequence's last one: that one again, its scores are masked
+            const int row = bt[min(it.page(t * ppt + g), last_page)] * p.block_size;
             uint8_t* dst = st + g * p.block_size * 128;
             for (int i = 0; i < p.nk; ++i) tma_load_3d(dst + i * GT_BOX, &tm_k, &full_bar[stage], 64 * i, it.kvh, row);
             for (int i = 0; i < p.nv; ++i) tma_load_3d(dst + k_bytes + i * GT_BOX, &tm_v, &full_bar[stage], 64 * i, it.kvh, row);
@@ -218,16 +245,17 @@ grouped_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_
           // with one stage the next K tile arrives only after this tile's products
           if (p.stages > 1 && i + 1 < n && !mma1(m + i + 1, j)) { ok = false; break; }
           const int mm = m + i, stage = mm % p.stages;
-          if (!mbar_wait(pfull_bar, (uint32_t)(mm & 1), abort_flag, p.status, 1830)) { ok = false; break; }
+          if (!mbar_wait(&pfull_bar[mm & 1], (uint32_t)((mm >> 1) & 1), abort_flag, p.status, 1830)) { ok = false; break; }
           tc_fence_after();
 #pragma unroll
           for (int s = 0; s < SLABS; ++s) {
             const uint64_t dv = desc_at(v_d, (uint32_t)stage * stage_bytes + (uint32_t)(2 * s) * GT_BOX);
 #pragma unroll
             for (int kk = 0; kk < 8; ++kk)
-              umma_bf16_ss(tmem_base + 32 + 16 * s, desc_at(dv, kk * 2048), desc_at(p_d, (kk >> 2) * 2048) + 2 * (kk & 3), idesc_o, kk != 0);
+              umma_bf16_ss(tmem_base + 32 + 16 * ((mm & 1) * SLABS + s), desc_at(dv, kk * 2048),
+                           desc_at(p_d, (mm & 1) * GT_P_BYTES + (kk >> 2) * 2048) + 2 * (kk & 3), idesc_o, kk != 0);
           }
-          umma_commit(ofull_bar);
+          umma_commit(&ofull_bar[mm & 1]);
           umma_commit(&empty_bar[stage]);
           if (p.stages == 1 && i + 1 < n && !mma1(m + i + 1, j)) { ok = false; break; }
         }
@@ -273,54 +301,71 @@ grouped_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_
     for (int next; item < n_items && good; item = next, it = nxt, ++j) {
       next = gt_next(p, item + gridDim.x, n_items, nxt);
       if (next < n_items) write_q(nxt, (j + 1) & 1);
-      float mrun[8], lsum[8], acc[SLABS][8];
+      float mrun[HEADS], lsum[HEADS], alpha[HEADS], acc[SLABS][HEADS];
 #pragma unroll
-      for (int g = 0; g < 8; ++g) {
+      for (int g = 0; g < HEADS; ++g) {
         mrun[g] = -INFINITY;
         lsum[g] = 0.f;
+        alpha[g] = 0.f;
 #pragma unroll
         for (int s = 0; s < SLABS; ++s) acc[s][g] = 0.f;
       }
+      // the output of tile m, whose probabilities were formed when alpha was what it is
+      auto collect = [&](int m) -> bool {
+        if (!__all_sync(0xffffffffu, mbar_wait(&ofull_bar[m & 1], (uint32_t)((m >> 1) & 1), abort_flag, p.status, 1850))) return false;
+        tc_fence_after();
+#pragma unroll
+        for (int sl = 0; sl < SLABS; ++sl) {
+          float o[16];
+          tmem_ld_32x16(tmem_base + lane_off + 32 + 16 * ((m & 1) * SLABS + sl), o);
+          tmem_ld_wait();
+#pragma unroll
+          for (int g = 0; g < HEADS; ++g) acc[sl][g] = fmaf(acc[sl][g], alpha[g], o[g] + o[8 + g]);
+        }
+        tc_fence_before();
+        return true;
+      };
       for (int t = it.t0; t < it.t1; ++t, ++m_cnt) {
-        float s[8];
+        float s[HEADS];
         float* rm = red_m + (m_cnt & 1) * 32;
         good = good && __all_sync(0xffffffffu, mbar_wait(&sfull_bar[m_cnt & 1], (uint32_t)((m_cnt >> 1) & 1), abort_flag, p.status, 1840));
         if (good) {
+          float all[8];
           tc_fence_after();
-          tmem_ld_32x8(tmem_base + lane_off + (uint32_t)(m_cnt & 1) * 16, s);
+          tmem_ld_32x8(tmem_base + lane_off + (uint32_t)(m_cnt & 1) * 16, all);
           tmem_ld_wait();
+#pragma unroll
+          for (int g = 0; g < HEADS; ++g) s[g] = all[g];
           if (p.cap_in > 0.f) {
             float top = 0.f;
 #pragma unroll
-            for (int g = 0; g < 8; ++g) {
+            for (int g = 0; g < HEADS; ++g) {
               s[g] *= p.cap_in;
               top = fmaxf(top, fabsf(s[g]));
             }
             const bool far = __any_sync(0xffffffffu, top > CAP_SERIES);
 #pragma unroll
-            for (int g = 0; g < 8; ++g) s[g] = p.cap_out * (far ? tanh_exp(s[g]) : tanh_series(s[g]));
+            for (int g = 0; g < HEADS; ++g) s[g] = p.cap_out * (far ? tanh_exp(s[g]) : tanh_series(s[g]));
           }
-          const int tok = it.tile(t) * 128 + row;
+          const int tok = it.page(t * ppt + row / p.block_size) * p.block_size + row % p.block_size;
           const bool valid = tok < it.len && (p.window == 0 || tok >= it.len - p.window || tok < p.keep);
 #pragma unroll
-          for (int g = 0; g < 8; ++g) {
-            s[g] = valid ? s[g] * p.scale_log2 : -INFINITY;
-            const float wm = warp_max(s[g]);
-            if (lane == 0) rm[quarter * 8 + g] = wm;
-          }
+          for (int g = 0; g < HEADS; ++g) s[g] = valid ? s[g] * p.scale_log2 : -INFINITY;
+          const float wm = gt_warp_max<HEADS>(s, lane);
+          if ((lane & (32 / HEADS - 1)) == 0) rm[quarter * 8 + gt_slot<HEADS>(lane)] = wm;
         }
         good = gt_vote(good);
         if (!good) break;
-        float alpha[8];
-        uint8_t* prow = p_s + (row >> 6) * 2048;  // the [16 x 64 tok] half of this token
+        float next[HEADS];
+        uint8_t* prow = p_s + (m_cnt & 1) * GT_P_BYTES + (row >> 6) * 2048;  // the [16 x 64 tok] half of this token
         const int c = row & 63;
 #pragma unroll
-        for (int g = 0; g < 8; ++g) {
+        for (int g = 0; g < HEADS; ++g) {
           const float mn = fmaxf(mrun[g], fmaxf(fmaxf(rm[g], rm[8 + g]), fmaxf(rm[16 + g], rm[24 + g])));
-          alpha[g] = (mrun[g] == -INFINITY) ? 0.f : fast_exp2(mrun[g] - mn);
+          next[g] = (mrun[g] == -INFINITY) ? 0.f : fast_exp2(mrun[g] - mn);
           const float pv = (s[g] == -INFINITY || g >= it.nh) ? 0.f : fast_exp2(s[g] - mn);
           mrun[g] = mn;
-          lsum[g] = lsum[g] * alpha[g] + pv;
+          lsum[g] = lsum[g] * next[g] + pv;
           const __nv_bfloat16 hi = __float2bfloat16(pv);
           uint8_t* at = prow + g * 128 + ((((c >> 3) ^ g) & 7) << 4) + (c & 7) * 2;
           *reinterpret_cast<__nv_bfloat16*>(at) = hi;
@@ -328,30 +373,21 @@ grouped_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_
         }
         fence_proxy_async_smem();
         tc_fence_before();
-        mbar_arrive(pfull_bar);
-        good = good && __all_sync(0xffffffffu, mbar_wait(ofull_bar, (uint32_t)(m_cnt & 1), abort_flag, p.status, 1850));
-        if (good) {
-          tc_fence_after();
+        mbar_arrive(&pfull_bar[m_cnt & 1]);
+        if (t > it.t0) good = collect(m_cnt - 1);
 #pragma unroll
-          for (int sl = 0; sl < SLABS; ++sl) {
-            float o[16];
-            tmem_ld_32x16(tmem_base + lane_off + 32 + 16 * sl, o);
-            tmem_ld_wait();
-#pragma unroll
-            for (int g = 0; g < 8; ++g) acc[sl][g] = fmaf(acc[sl][g], alpha[g], o[g] + o[8 + g]);
-          }
-          tc_fence_before();
-        }
+        for (int g = 0; g < HEADS; ++g) alpha[g] = next[g];
       }
+      if (good) good = collect(m_cnt - 1);
 #pragma unroll
-      for (int g = 0; g < 8; ++g) {
+      for (int g = 0; g < HEADS; ++g) {
         const float ws = warp_sum(lsum[g]);
         if (lane == 0) red_l[quarter * 8 + g] = ws;
       }
       good = gt_vote(good);  // every softmax thread gets here, also after a failed wait: the vote keeps them together
       if (!good) break;
 #pragma unroll
-      for (int g = 0; g < 8; ++g) {
+      for (int g = 0; g < HEADS; ++g) {
         if (g >= it.nh) break;
         const size_t bh = (size_t)it.b * p.heads + it.h0 + g;
         const float L = red_l[g] + red_l[8 + g] + red_l[16 + g] + red_l[24 + g];
@@ -381,7 +417,7 @@ grouped_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_
   }
   if (warp == 1) {
     tc_fence_after();
-    tmem_dealloc(tmem_base, 64);
+    tmem_dealloc(tmem_base, 32 + 32 * SLABS <= 64 ? 64 : 128);
   }
 }
 
@@ -421,7 +457,7 @@ using namespace trlb;
 namespace {
 
 size_t gt_smem(int nk, int slabs, int stages) {
-  return (size_t)stages * (nk + 2 * slabs) * GT_BOX + 2 * (size_t)nk * 2048 + GT_P_BYTES + 1024 + 1024;
+  return (size_t)stages * (nk + 2 * slabs) * GT_BOX + 2 * (size_t)nk * 2048 + 2 * GT_P_BYTES + 1024 + 1024;
 }
 int gt_stages(int nk, int slabs) {
   for (int s = GT_MAX_STAGES; s > 0; --s)
@@ -468,20 +504,21 @@ TRLB_API int trlb_grouped_decode_tc(const void* q, const void* k_cache, const vo
   const uint64_t rows = (uint64_t)num_blocks * block_size;
   if (make_tmap_3d_bf16(&tk, k_cache, dim, kv_heads, rows, dim, (uint64_t)kv_heads * dim, 64, 1, block_size)) return -281;
   if (make_tmap_3d_bf16(&tv, v_cache, vdim, kv_heads, rows, vdim, (uint64_t)kv_heads * vdim, 64, 1, block_size)) return -282;
+  using Kern = void (*)(const CUtensorMap, const CUtensorMap, const GroupedDecodeTc);
+  static const Kern kerns[2][4] = {{grouped_decode_tc_kernel<1, 1>, grouped_decode_tc_kernel<1, 2>, grouped_decode_tc_kernel<1, 4>, grouped_decode_tc_kernel<1, 8>},
+                                   {grouped_decode_tc_kernel<2, 1>, grouped_decode_tc_kernel<2, 2>, grouped_decode_tc_kernel<2, 4>, grouped_decode_tc_kernel<2, 8>}};
   static bool attr_set = false;
   if (!attr_set) {
-    if (cudaFuncSetAttribute(grouped_decode_tc_kernel<1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024) != cudaSuccess ||
-        cudaFuncSetAttribute(grouped_decode_tc_kernel<2>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024) != cudaSuccess)
-      return -283;
+    for (int i = 0; i < 8; ++i)
+      if (cudaFuncSetAttribute(kerns[i >> 2][i & 3], cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024) != cudaSuccess) return -283;
     attr_set = true;
   }
   const int items = trlb_grouped_decode_tc_items(B, heads, kv_heads) * splits;
   const dim3 grid(items < trlb_host::sm_count() ? items : trlb_host::sm_count()), blk(GT_THREADS);
   const size_t smem = gt_smem(p.nk, slabs, p.stages);
   const bool pdl = trlb_host::pdl_enabled();
-  const int rc = slabs == 1
-                     ? (int)trlb_host::launch_kernel(grouped_decode_tc_kernel<1>, grid, blk, smem, st, pdl, tk, tv, p)
-                     : (int)trlb_host::launch_kernel(grouped_decode_tc_kernel<2>, grid, blk, smem, st, pdl, tk, tv, p);
+  const Kern kern = kerns[slabs - 1][p.group > 4 ? 3 : p.group > 2 ? 2 : p.group > 1 ? 1 : 0];
+  const int rc = (int)trlb_host::launch_kernel(kern, grid, blk, smem, st, pdl, tk, tv, p);
   if (rc || splits == 1) return rc;
   return (int)trlb_host::launch_kernel(grouped_combine_kernel, dim3(heads, B), dim3(128), 0, st, pdl, (const float*)part_o,
                                        (const float2*)part_ml, p.gate, seq_lens, sink, head_gate, heads, vdim, splits, p.out);

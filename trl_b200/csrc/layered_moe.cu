@@ -28,10 +28,10 @@ struct MoeRoute {
   int* counts;   // [E]
 };
 
-template <bool ONE>
+template <bool ONE, int NI>  // NI: experts a lane
 __global__ void __launch_bounds__(ONE ? 1024 : 256)
 moe_route_kernel(const MoeRoute p) {
-  __shared__ int cnt[ONE ? MR_MAX_E : 1];
+  __shared__ int cnt[ONE ? 32 * NI : 1];
   pdl_launch_dependents();
   pdl_wait();
   if (ONE) {
@@ -42,11 +42,10 @@ moe_route_kernel(const MoeRoute p) {
   for (int t = blockIdx.x * per + (threadIdx.x >> 5); t < p.T; t += gridDim.x * per) {
     float* z = p.z + (size_t)t * p.E;
     const bool idle = p.positions != nullptr && p.positions[t] < 0;
-    float sc[MR_MAX_E / 32];   // choice scores of experts lane, lane + 32, ...
+    float sc[NI];   // choice scores of experts lane, lane + 32, ...
 #pragma unroll
-    for (int i = 0; i < MR_MAX_E / 32; ++i) {
+    for (int i = 0; i < NI; ++i) {
       const int e = lane + 32 * i;
-      if (32 * i >= p.E) break;
       sc[i] = -INFINITY;
       if (e < p.E) {
         sc[i] = sigmoid_f(z[e]) + (p.correction != nullptr ? p.correction[e] : 0.f);
@@ -58,8 +57,7 @@ moe_route_kernel(const MoeRoute p) {
       float best = -INFINITY;
       int at = p.E;
 #pragma unroll
-      for (int i = 0; i < MR_MAX_E / 32; ++i) {
-        if (32 * i >= p.E) break;
+      for (int i = 0; i < NI; ++i) {
         if (sc[i] > best) { best = sc[i]; at = lane + 32 * i; }
       }
 #pragma unroll
@@ -69,8 +67,7 @@ moe_route_kernel(const MoeRoute p) {
         if (ob > best || (ob == best && oa < at)) { best = ob; at = oa; }
       }
 #pragma unroll
-      for (int i = 0; i < MR_MAX_E / 32; ++i) {
-        if (32 * i >= p.E) break;
+      for (int i = 0; i < NI; ++i) {
         if (at == lane + 32 * i) sc[i] = -INFINITY;
       }
       if (lane == 0) {
@@ -229,10 +226,13 @@ TRLB_API int trlb_moe_route(float* z, const float* correction, const int* positi
   if (T <= 0) return 0;
   if (E <= 0 || E > MR_MAX_E || top <= 0 || top > E) return -290;
   const MoeRoute p = {z, correction, positions, T, E, top, renorm, clear, choice, rank, weight, counts};
-  if (T <= 128)
-    return (int)trlb_host::launch_kernel(moe_route_kernel<true>, dim3(1), dim3(T >= 32 ? 1024 : T * 32), 0, st, PDL, p);
   const int want = (T + 7) / 8, cap = trlb_host::sm_count() * 8;
-  return (int)trlb_host::launch_kernel(moe_route_kernel<false>, dim3(want < cap ? want : cap), dim3(256), 0, st, PDL, p);
+  const dim3 grid(T <= 128 ? 1 : want < cap ? want : cap), blk(T > 128 ? 256 : T >= 32 ? 1024 : T * 32);
+#define GO(ONE, NI) (int)trlb_host::launch_kernel(moe_route_kernel<ONE, NI>, grid, blk, 0, st, PDL, p)
+#define PICK(NI) (T <= 128 ? GO(true, NI) : GO(false, NI))
+  return E <= 32 ? PICK(1) : E <= 64 ? PICK(2) : E <= 128 ? PICK(4) : E <= 256 ? PICK(8) : PICK(32);
+#undef PICK
+#undef GO
 }
 
 // h [T, H], x [T top, H] in the model dtype; row [T, top], offsets [E + 1]
