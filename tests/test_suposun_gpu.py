@@ -232,7 +232,8 @@ def mixer(H, G, d, e, **kw):
 
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("H,G,d,rot,halves,scaling", [(6, 3, 20, 8, False, None), (4, 1, 128, 32, False, U.yarn()), (3, 3, 9, 4, True, None),
-                                                      (5, 5, 48, 48, True, None), (20, 4, 64, 24, True, U.yarn()), (2, 1, 14, 14, False, None), (8, 2, 16, 0, False, None)])
+                                                      (5, 5, 48, 48, True, None), (20, 4, 64, 24, True, U.yarn()), (2, 1, 14, 14, False, None), (8, 2, 16, 0, False, None),
+                                                      (32, 8, 128, 64, True, None), (72, 8, 128, 40, False, None)])
 @pytest.mark.parametrize("whole", [False, True])
 @pytest.mark.parametrize("kind", ["values", "keys", "borrowed"])
 def test_attention_preparation(H, G, d, rot, halves, scaling, whole, kind, dtype):

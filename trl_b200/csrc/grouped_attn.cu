@@ -221,8 +221,7 @@ attn_prep_kernel(const AttnPrep p, S* __restrict__ src, T* __restrict__ q_out, T
 
 // The same for sizes in multiples of 8 with heads of at most 256 elements: one block per row, 2^lanes_log2 threads with 8 elements
 // each per head, so that a row is read once into registers (also for norms over all heads) and moves in 16-byte pieces.  A block
-// takes its row in at most PREP_ROUNDS rounds.
-constexpr int PREP_ROUNDS = 4;
+// takes its row in at most ROUNDS rounds.
 
 __device__ __forceinline__ void load8(const float* p, float (&v)[8]) {
   const float4 a = load4(p), b = load4(p + 4);
@@ -246,7 +245,7 @@ __device__ __forceinline__ void store8(__nv_bfloat16* p, const float (&v)[8]) {
   *reinterpret_cast<uint4*>(p) = make_uint4(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]), pack_bf16(v[4], v[5]), pack_bf16(v[6], v[7]));
 }
 
-template <typename T, typename S, bool WHOLE>
+template <typename T, typename S, bool WHOLE, int ROUNDS>
 __global__ void __launch_bounds__(512)
 attn_prep_rows_kernel(const AttnPrep p, int lanes_log2, S* __restrict__ src, T* __restrict__ q_out, T* __restrict__ k_out,
                       T* __restrict__ g_out, T* __restrict__ k_cache, T* __restrict__ v_cache) {
@@ -266,10 +265,10 @@ attn_prep_rows_kernel(const AttnPrep p, int lanes_log2, S* __restrict__ src, T* 
     if (u < p.heads + kv) return u * p.dim;
     return q_n + k_n + (u - p.heads - kv) * p.vdim;
   };
-  float x[PREP_ROUNDS][8];
+  float x[ROUNDS][8];
   float sq = 0.f, sk = 0.f;
 #pragma unroll
-  for (int i = 0; i < PREP_ROUNDS; ++i) {
+  for (int i = 0; i < ROUNDS; ++i) {
     const int u = u0 + i * per_round;
     const bool on = u < units && j0 < (u < p.heads + kv ? p.dim : p.vdim);
 #pragma unroll
@@ -306,7 +305,7 @@ attn_prep_rows_kernel(const AttnPrep p, int lanes_log2, S* __restrict__ src, T* 
       if (e < 4 || p.halves) cs[e] = t[e];
   }
 #pragma unroll
-  for (int i = 0; i < PREP_ROUNDS; ++i) {
+  for (int i = 0; i < ROUNDS; ++i) {
     if (i * per_round >= units) break;  // uniform
     const int u = u0 + i * per_round;
     const bool normed = u < p.heads + kv, is_q = u < p.heads;
@@ -585,15 +584,16 @@ TRLB_API int trlb_attn_prep(void* src, int src_f32, long long ld, int rows, int 
   while ((8 << lanes_log2) < widest) ++lanes_log2;
   const int threads = row_units << lanes_log2;  // of one round
   const auto aligned = [](const void* x) { return (reinterpret_cast<uintptr_t>(x) & 15) == 0; };
-  if (((dim | vdim | (int)(ld & 7)) & 7) == 0 && widest <= 256 && threads <= 512 * PREP_ROUNDS && rot % (halves ? 16 : 8) == 0 && aligned(src) &&
+  if (((dim | vdim | (int)(ld & 7)) & 7) == 0 && widest <= 256 && threads <= 2048 && rot % (halves ? 16 : 8) == 0 && aligned(src) &&
       aligned(q_out) && aligned(k_out) && aligned(g_out) && aligned(k_cache) && aligned(v_cache) && aligned(q_w) && aligned(k_w)) {
-    const int least = (threads + PREP_ROUNDS - 1) / PREP_ROUNDS;
-    const int want = threads <= 256 ? threads : least <= 256 ? 256 : 512;
-    const dim3 block((want + 31) / 32 * 32);
-#define GO(TT, SS, WW) (int)trlb_host::launch_kernel(attn_prep_rows_kernel<TT, SS, WW>, dim3(rows), block, 0, st, PDL, p, lanes_log2, (SS*)src, (TT*)q_out, \
-                                                     (TT*)k_out, (TT*)g_out, (TT*)k_cache, (TT*)v_cache)
-    if (is_bf16) return src_f32 ? (whole ? GO(bf16, float, true) : GO(bf16, float, false)) : (whole ? GO(bf16, bf16, true) : GO(bf16, bf16, false));
-    return whole ? GO(float, float, true) : GO(float, float, false);
+    const int rounds = threads <= 256 ? 1 : threads <= 1024 ? 2 : 4;
+    const dim3 block(((threads + rounds - 1) / rounds + 31) / 32 * 32);
+#define GO(TT, SS, WW, RR) (int)trlb_host::launch_kernel(attn_prep_rows_kernel<TT, SS, WW, RR>, dim3(rows), block, 0, st, PDL, p, lanes_log2, (SS*)src, \
+                                                         (TT*)q_out, (TT*)k_out, (TT*)g_out, (TT*)k_cache, (TT*)v_cache)
+#define PICK(TT, SS, WW) (rounds == 1 ? GO(TT, SS, WW, 1) : rounds == 2 ? GO(TT, SS, WW, 2) : GO(TT, SS, WW, 4))
+    if (is_bf16) return src_f32 ? (whole ? PICK(bf16, float, true) : PICK(bf16, float, false)) : (whole ? PICK(bf16, bf16, true) : PICK(bf16, bf16, false));
+    return whole ? PICK(float, float, true) : PICK(float, float, false);
+#undef PICK
 #undef GO
   }
   const int units = row_units + (gates == GATES_HEAD ? 1 : 0);
