@@ -178,7 +178,7 @@ def expert_case(H, n, E, top, dtype, seed=0, limit=0.8):
     r = gen(seed + H + E)
     t = {"router": 2 * r(E, H) / H ** 0.5, "correction": 0.5 * r(E), "gate_up": 2 * r(E, 2 * n, H) / H ** 0.5, "down": r(E, H, n) / n ** 0.5}
     t = {k: v.to(dtype if k != "correction" else torch.float32).double() for k, v in t.items()}
-    m = types.SimpleNamespace(n=E, top=top, ff=n, glu=(limit, 1.702, 1.0), renormalize=False,
+    m = types.SimpleNamespace(n=E, top=top, ff=n, glu=(limit, 1.702, 1.0), routing={},
                               **{k: dev(v, dtype if k != "correction" else torch.float32) for k, v in t.items()})
     w = dict(router=t["router"], correction=t["correction"])
     for e in range(E):

@@ -14,7 +14,8 @@
 // the next one have been handed over, so that product and softmax overlap.
 // Scores may be capped (cap tanh(s / cap)); the softmax denominator may contain exp(sink[head]); the result may be multiplied by
 // the sigmoid of per-element gate logits or by a factor per head.  With a window only its pages and those of the first `keep`
-// tokens, which stay visible, are read: the pages of a slot are a list, kept ones first, that is cut into tiles.
+// tokens, which stay visible, are read: the pages of a slot are a list, kept ones first, that is cut into tiles.  Or tiles of means of
+// the blocks of `pool` tokens before the window come first: the slot has its rows of them beside the pages (grouped_attn.cu).
 // Splits leave fp32 partial sums that grouped_combine_kernel merges.
 #include "mixers.cuh"
 
@@ -40,6 +41,9 @@ struct GroupedDecodeTc {
   int window, keep;           // window 0: unlimited
   const float* sink;          // [heads] or null
   const float* head_gate;     // [B, heads] or null
+  int pool, pool_rows;        // 0: no blocks; rows of means per slot
+  long long out_ld;
+  float out_scale;
 };
 
 __device__ __forceinline__ bool gt_vote(bool pred) {
@@ -70,6 +74,7 @@ __device__ __forceinline__ float gt_factor(float m, float L, const float* sink, 
 struct GtItem {
   int b, kvh, h0, nh, sp, len, t0, t1;  // t0 .. t1: tiles of the slot's list of pages
   int lo, kp;                           // first page of the window, kept pages before it
+  int nb, pt;                           // blocks before the window, tiles of their means (tiles 0 .. pt - 1)
   __device__ __forceinline__ int page(int i) const { return i < kp ? i : lo + i - kp; }
 };
 
@@ -88,7 +93,9 @@ __device__ __forceinline__ GtItem gt_item(const GroupedDecodeTc& p, int item) {
   const int bs = p.block_size;
   it.lo = p.window > 0 ? max(0, it.len - p.window) / bs : 0;
   it.kp = min((p.keep + bs - 1) / bs, it.lo);
-  const int n_t = ((it.kp + (it.len + bs - 1) / bs - it.lo) * bs + 127) >> 7;
+  it.nb = p.pool > 0 ? min(max(0, it.len - p.window) / p.pool, p.pool_rows) : 0;
+  it.pt = (it.nb + 127) >> 7;
+  const int n_t = it.pt + (((it.kp + (it.len + bs - 1) / bs - it.lo) * bs + 127) >> 7);
   it.t0 = n_t * it.sp / p.splits;
   it.t1 = n_t * (it.sp + 1) / p.splits;
   return it;
@@ -132,7 +139,7 @@ __device__ __forceinline__ float gt_warp_max(const float (&s)[N], int lane) {
 template <int SLABS, int HEADS>
 __global__ void __launch_bounds__(GT_THREADS, 1)
 grouped_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_constant__ CUtensorMap tm_v,
-                         const GroupedDecodeTc p) {
+                         const __grid_constant__ CUtensorMap tm_pk, const __grid_constant__ CUtensorMap tm_pv, const GroupedDecodeTc p) {
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   // a slab of O^T reads two boxes of V: the second one may exist only as space
@@ -202,9 +209,15 @@ grouped_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_
           }
           uint8_t* st = smem + (size_t)stage * stage_bytes;
           mbar_expect_tx(&full_bar[stage], (uint32_t)(p.nk + p.nv) * GT_BOX);
+          if (t < it.pt) {
+            const int row = it.b * p.pool_rows + t * 128;  // rows past the slot's blocks: their scores are masked
+            for (int i = 0; i < p.nk; ++i) tma_load_3d(st + i * GT_BOX, &tm_pk, &full_bar[stage], 64 * i, it.kvh, row);
+            for (int i = 0; i < p.nv; ++i) tma_load_3d(st + k_bytes + i * GT_BOX, &tm_pv, &full_bar[stage], 64 * i, it.kvh, row);
+            continue;
+          }
           for (int g = 0; g < ppt; ++g) {
             // pages past the sequence's last one: that one again, its scores are masked
-            const int row = bt[min(it.page(t * ppt + g), last_page)] * p.block_size;
+            const int row = bt[min(it.page((t - it.pt) * ppt + g), last_page)] * p.block_size;
             uint8_t* dst = st + g * p.block_size * 128;
             for (int i = 0; i < p.nk; ++i) tma_load_3d(dst + i * GT_BOX, &tm_k, &full_bar[stage], 64 * i, it.kvh, row);
             for (int i = 0; i < p.nv; ++i) tma_load_3d(dst + k_bytes + i * GT_BOX, &tm_v, &full_bar[stage], 64 * i, it.kvh, row);
@@ -286,7 +299,7 @@ grouped_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_
       for (int item = blockIdx.x; item < n_items; item += gridDim.x) {
         const GtItem it = gt_item(p, item);
         if (it.t1 > it.t0) continue;
-        for (int i = ts; i < it.nh * p.vdim; i += 128) p.out[((size_t)it.b * p.heads + it.h0) * p.vdim + i] = __float2bfloat16(0.f);
+        for (int i = ts; i < it.nh * p.vdim; i += 128) p.out[(size_t)it.b * p.out_ld + (size_t)it.h0 * p.vdim + i] = __float2bfloat16(0.f);
       }
     } else {
       for (int item = blockIdx.x; item < n_items; item += gridDim.x) {
@@ -347,8 +360,8 @@ grouped_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_
 #pragma unroll
             for (int g = 0; g < HEADS; ++g) s[g] = p.cap_out * (far ? tanh_exp(s[g]) : tanh_series(s[g]));
           }
-          const int tok = it.page(t * ppt + row / p.block_size) * p.block_size + row % p.block_size;
-          const bool valid = tok < it.len && (p.window == 0 || tok >= it.len - p.window || tok < p.keep);
+          const int tok = it.page((t - it.pt) * ppt + row / p.block_size) * p.block_size + row % p.block_size;
+          const bool valid = t < it.pt ? t * 128 + row < it.nb : tok < it.len && (p.window == 0 || tok >= it.len - p.window || tok < p.keep);
 #pragma unroll
           for (int g = 0; g < HEADS; ++g) s[g] = valid ? s[g] * p.scale_log2 : -INFINITY;
           const float wm = gt_warp_max<HEADS>(s, lane);
@@ -397,9 +410,9 @@ grouped_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_
           const int d = sl * 128 + row;
           if (d >= p.vdim) continue;
           if (p.splits == 1) {
-            float o = acc[sl][g] * f;
+            float o = acc[sl][g] * f * p.out_scale;
             if (p.gate != nullptr) o *= fast_sigmoid(__bfloat162float(p.gate[bh * p.vdim + d]));
-            p.out[bh * p.vdim + d] = __float2bfloat16(o);
+            p.out[(size_t)it.b * p.out_ld + (size_t)(it.h0 + g) * p.vdim + d] = __float2bfloat16(o);
           } else {
             p.part_o[(bh * p.splits + it.sp) * p.vdim + d] = acc[sl][g];
           }
@@ -425,7 +438,7 @@ grouped_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_
 __global__ void __launch_bounds__(128)
 grouped_combine_kernel(const float* __restrict__ part_o, const float2* __restrict__ part_ml, const __nv_bfloat16* __restrict__ gate,
                        const int* __restrict__ seq_lens, const float* __restrict__ sink, const float* __restrict__ head_gate, int heads,
-                       int vdim, int splits, __nv_bfloat16* __restrict__ out) {
+                       int vdim, int splits, long long out_ld, float out_scale, __nv_bfloat16* __restrict__ out) {
   pdl_launch_dependents();
   pdl_wait();
   const int h = blockIdx.x, b = blockIdx.y;
@@ -437,7 +450,7 @@ grouped_combine_kernel(const float* __restrict__ part_o, const float2* __restric
     const float2 ml = part_ml[bh * splits + s];
     if (ml.y > 0.f) den += ml.y * fast_exp2(ml.x - m);
   }
-  const float f = gt_factor(m, den, sink, head_gate, h, bh);
+  const float f = gt_factor(m, den, sink, head_gate, h, bh) * out_scale;
   for (int d = threadIdx.x; d < vdim; d += 128) {
     float o = 0.f;
     for (int s = 0; s < splits; ++s) {
@@ -446,7 +459,7 @@ grouped_combine_kernel(const float* __restrict__ part_o, const float2* __restric
     }
     o *= f;
     if (gate != nullptr) o *= fast_sigmoid(__bfloat162float(gate[bh * vdim + d]));
-    out[bh * vdim + d] = __float2bfloat16(o);
+    out[(size_t)b * out_ld + (size_t)h * vdim + d] = __float2bfloat16(o);
   }
 }
 
@@ -479,12 +492,15 @@ TRLB_API int trlb_grouped_decode_tc_items(int B, int heads, int kv_heads) { retu
 
 // q [B, heads, dim], caches [num_blocks, block_size, kv_heads, dim / vdim], gate logits [B, heads, vdim] or null; one new token per
 // slot, in the cache already.  window <= 0: unlimited, else the first `keep` tokens stay visible; cap <= 0: none; sink [heads] and
-// head_gate [B, heads] may be null.  splits > 1: part_o [B, heads, splits, vdim], part_ml [B, heads, splits, 2] fp32.
+// head_gate [B, heads] may be null.  pool > 0 (with a window): means pool_k, pool_v [pool_slots, pool_rows, kv_heads, dim / vdim].  out [B
+// rows of out_ld], times out_scale.  splits > 1: part_o [B, heads, splits, vdim], part_ml [B, heads, splits, 2] fp32.
 TRLB_API int trlb_grouped_decode_tc(const void* q, const void* k_cache, const void* v_cache, const void* gate, void* out,
                                     int num_blocks, int B, int heads, int kv_heads, int dim, int vdim, int window, int keep,
                                     float scale, float cap, const float* sink, const float* head_gate, const int* seq_lens, const int* block_table, int max_blocks, int block_size, int splits,
-                                    float* part_o, float* part_ml, int* status, cudaStream_t st) {
+                                    float* part_o, float* part_ml, int pool, int pool_rows, int pool_slots, const void* pool_k,
+                                    const void* pool_v, long long out_ld, float out_scale, int* status, cudaStream_t st) {
   if (B <= 0) return 0;
+  if (pool > 0 && (pool_k == nullptr || pool_v == nullptr || pool_rows <= 0 || pool_slots < B || keep > 0)) return -280;
   if (!(scale > 0.f) || splits < 1 || !trlb_grouped_decode_tc_ok(heads, kv_heads, dim, vdim, block_size)) return -280;
   if (splits > 1 && (part_o == nullptr || part_ml == nullptr)) return -280;
   GroupedDecodeTc p = {};
@@ -499,12 +515,20 @@ TRLB_API int trlb_grouped_decode_tc(const void* q, const void* k_cache, const vo
   p.cap_out = cap * 1.4426950408889634f;
   p.window = window > 0 ? window : 0; p.keep = window > 0 && keep > 0 ? keep : 0; p.sink = sink; p.head_gate = head_gate;
   p.part_o = part_o; p.part_ml = (float2*)part_ml; p.status = status;
-  CUtensorMap tk, tv;
+  p.pool = window > 0 && pool > 0 ? pool : 0; p.pool_rows = pool_rows; p.out_ld = out_ld; p.out_scale = out_scale;
+  CUtensorMap tk, tv, tpk, tpv;
   using trlb_host::make_tmap_3d_bf16;
   const uint64_t rows = (uint64_t)num_blocks * block_size;
   if (make_tmap_3d_bf16(&tk, k_cache, dim, kv_heads, rows, dim, (uint64_t)kv_heads * dim, 64, 1, block_size)) return -281;
   if (make_tmap_3d_bf16(&tv, v_cache, vdim, kv_heads, rows, vdim, (uint64_t)kv_heads * vdim, 64, 1, block_size)) return -282;
-  using Kern = void (*)(const CUtensorMap, const CUtensorMap, const GroupedDecodeTc);
+  tpk = tk;
+  tpv = tv;
+  if (p.pool > 0) {
+    const uint64_t means = (uint64_t)pool_slots * pool_rows;
+    if (make_tmap_3d_bf16(&tpk, pool_k, dim, kv_heads, means, dim, (uint64_t)kv_heads * dim, 64, 1, 128)) return -284;
+    if (make_tmap_3d_bf16(&tpv, pool_v, vdim, kv_heads, means, vdim, (uint64_t)kv_heads * vdim, 64, 1, 128)) return -285;
+  }
+  using Kern = void (*)(const CUtensorMap, const CUtensorMap, const CUtensorMap, const CUtensorMap, const GroupedDecodeTc);
   static const Kern kerns[2][4] = {{grouped_decode_tc_kernel<1, 1>, grouped_decode_tc_kernel<1, 2>, grouped_decode_tc_kernel<1, 4>, grouped_decode_tc_kernel<1, 8>},
                                    {grouped_decode_tc_kernel<2, 1>, grouped_decode_tc_kernel<2, 2>, grouped_decode_tc_kernel<2, 4>, grouped_decode_tc_kernel<2, 8>}};
   static bool attr_set = false;
@@ -518,8 +542,8 @@ TRLB_API int trlb_grouped_decode_tc(const void* q, const void* k_cache, const vo
   const size_t smem = gt_smem(p.nk, slabs, p.stages);
   const bool pdl = trlb_host::pdl_enabled();
   const Kern kern = kerns[slabs - 1][p.group > 4 ? 3 : p.group > 2 ? 2 : p.group > 1 ? 1 : 0];
-  const int rc = (int)trlb_host::launch_kernel(kern, grid, blk, smem, st, pdl, tk, tv, p);
+  const int rc = (int)trlb_host::launch_kernel(kern, grid, blk, smem, st, pdl, tk, tv, tpk, tpv, p);
   if (rc || splits == 1) return rc;
   return (int)trlb_host::launch_kernel(grouped_combine_kernel, dim3(heads, B), dim3(128), 0, st, pdl, (const float*)part_o,
-                                       (const float2*)part_ml, p.gate, seq_lens, sink, head_gate, heads, vdim, splits, p.out);
+                                       (const float2*)part_ml, p.gate, seq_lens, sink, head_gate, heads, vdim, splits, out_ld, out_scale, p.out);
 }

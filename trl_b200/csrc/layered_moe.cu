@@ -12,8 +12,8 @@ namespace trlb {
 constexpr int MR_MAX_E = 1024;
 
 // ------------------------------------------------------------------------------------------------------------
-// Router: scores sigmoid(z); the `top` experts of the largest score + correction (ties: the lower index) with their bare
-// scores as weights (RENORM: over their sum).  One warp per token.  rank: place among the expert's rows.  ONE: a single block
+// Router: scores sigmoid(z), or softmax(z); the `top` experts of the largest score + correction (ties: the lower index) with their
+// bare scores as weights (renorm: over their sum), times gain.  One warp per token.  rank: place among the expert's rows.  ONE: a single block
 // counts in shared memory and stores the counts; else counts are zeros before the launch.  Negative positions mark idle rows,
 // which choose nothing (expert -1).  clear: z is zeroed.
 // ------------------------------------------------------------------------------------------------------------
@@ -21,7 +21,8 @@ struct MoeRoute {
   float* z;  // [T, E]
   const float* correction;  // [E] or null
   const int* positions;     // [T] or null
-  int T, E, top, renorm, clear;
+  int T, E, top, renorm, softmax, clear;
+  float gain;
   int* choice;   // [T, top]
   int* rank;     // [T, top]
   float* weight; // [T, top]
@@ -43,12 +44,21 @@ moe_route_kernel(const MoeRoute p) {
     float* z = p.z + (size_t)t * p.E;
     const bool idle = p.positions != nullptr && p.positions[t] < 0;
     float sc[NI];   // choice scores of experts lane, lane + 32, ...
+    float zmax = -INFINITY, zsum = 1.f;
+    if (p.softmax) {
+      for (int e = lane; e < p.E; e += 32) zmax = fmaxf(zmax, z[e]);
+      zmax = warp_max(zmax);
+      zsum = 0.f;
+      for (int e = lane; e < p.E; e += 32) zsum += expf(z[e] - zmax);
+      zsum = warp_sum(zsum);
+    }
+    auto score = [&](float v) { return p.softmax ? expf(v - zmax) / zsum : sigmoid_f(v); };
 #pragma unroll
     for (int i = 0; i < NI; ++i) {
       const int e = lane + 32 * i;
       sc[i] = -INFINITY;
       if (e < p.E) {
-        sc[i] = sigmoid_f(z[e]) + (p.correction != nullptr ? p.correction[e] : 0.f);
+        sc[i] = score(z[e]) + (p.correction != nullptr ? p.correction[e] : 0.f);
         if (!(sc[i] > -INFINITY)) sc[i] = -3e38f;  // a NaN still has its place in the order
       }
     }
@@ -72,15 +82,15 @@ moe_route_kernel(const MoeRoute p) {
       }
       if (lane == 0) {
         const size_t o = (size_t)t * p.top + j;
-        const float w = sigmoid_f(z[at]);
+        const float w = score(z[at]);
         p.choice[o] = idle ? -1 : at;
-        p.weight[o] = w;
+        p.weight[o] = w * p.gain;
         total += w;
         if (!idle) p.rank[o] = ONE ? atomicAdd(&cnt[at], 1) : atomicAdd(&p.counts[at], 1);
       }
     }
     if (lane == 0 && p.renorm)
-      for (int j = 0; j < p.top; ++j) p.weight[(size_t)t * p.top + j] /= total;
+      for (int j = 0; j < p.top; ++j) p.weight[(size_t)t * p.top + j] /= total + 1e-20f;
     __syncwarp();
     if (p.clear)
       for (int e = lane; e < p.E; e += 32) z[e] = 0.f;
@@ -221,11 +231,11 @@ using bf16 = __nv_bfloat16;
 
 // z [T, E] fp32 logits (zeroed with clear); correction, positions may be null.  choice, rank, weight [T, top]; counts [E]: zeros
 // when T > 128 (they are added to), else any.
-TRLB_API int trlb_moe_route(float* z, const float* correction, const int* positions, int T, int E, int top, int renorm, int clear,
-                            int* choice, int* rank, float* weight, int* counts, cudaStream_t st) {
+TRLB_API int trlb_moe_route(float* z, const float* correction, const int* positions, int T, int E, int top, int renorm, int softmax,
+                            float gain, int clear, int* choice, int* rank, float* weight, int* counts, cudaStream_t st) {
   if (T <= 0) return 0;
   if (E <= 0 || E > MR_MAX_E || top <= 0 || top > E) return -290;
-  const MoeRoute p = {z, correction, positions, T, E, top, renorm, clear, choice, rank, weight, counts};
+  const MoeRoute p = {z, correction, positions, T, E, top, renorm, softmax, clear, gain, choice, rank, weight, counts};
   const int want = (T + 7) / 8, cap = trlb_host::sm_count() * 8;
   const dim3 grid(T <= 128 ? 1 : want < cap ? want : cap), blk(T > 128 ? 256 : T >= 32 ? 1024 : T * 32);
 #define GO(ONE, NI) (int)trlb_host::launch_kernel(moe_route_kernel<ONE, NI>, grid, blk, 0, st, PDL, p)

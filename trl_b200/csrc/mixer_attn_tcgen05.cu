@@ -23,7 +23,9 @@
 //     element;
 //   * keys are those of the same sequence, with a window those at distance < window and the first `keep` of the sequence: the
 //     tiles of a CTA are those that hold kept keys, then those of the window; the last kept tile is only as wide (in steps of
-//     32 keys) as the kept keys reach.
+//     32 keys) as the kept keys reach;
+//   * in place of kept keys there may be means of blocks of `pool` keys and values (tensors of their own, grouped_attn.cu), seen by
+//     the queries whose window begins behind the block: tiles of these means come first.
 #include "mixers.cuh"
 
 namespace trlb {
@@ -36,7 +38,7 @@ enum { GATE_NONE = 0, GATE_HEAD = 1, GATE_LOGITS = 2 };
 
 struct MixerAttnTc {
   const int* cu;
-  int n_seq, heads, group, dim, rot, vdim, window, keep;
+  int n_seq, heads, group, dim, rot, vdim, window, keep, pool;
   int nn, nr, nv;      // boxes of the unrotated part, the rotated part and the value
   int k_stages, v_stages;
   float scale_log2;    // CAP: 1 (capped scores are in log2 units already)
@@ -47,7 +49,9 @@ struct MixerAttnTc {
   int gate_mode;
   const void* gate;    // GATE_HEAD: fp32 [T, heads]; GATE_LOGITS: bf16 [T, gate_ld >= heads vdim]
   long long gate_ld;
-  __nv_bfloat16* out;  // [T, heads, vdim]
+  __nv_bfloat16* out;  // [T rows of out_ld], heads x vdim
+  long long out_ld;
+  float out_scale;
   int* status;
 };
 
@@ -136,7 +140,8 @@ template <bool CAP, int NB>
 __global__ void __launch_bounds__(LA_THREADS, 3 - NB)
 mixer_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_constant__ CUtensorMap tm_qr,
                       const __grid_constant__ CUtensorMap tm_kn, const __grid_constant__ CUtensorMap tm_kr,
-                      const __grid_constant__ CUtensorMap tm_v, const MixerAttnTc p) {
+                      const __grid_constant__ CUtensorMap tm_v, const __grid_constant__ CUtensorMap tm_pk,
+                      const __grid_constant__ CUtensorMap tm_pv, const MixerAttnTc p) {
   int seq, tile;
   if (!la_find_tile(p.cu, p.n_seq, (int)blockIdx.x, seq, tile)) return;  // uniform: before any barrier or TMEM use
   extern __shared__ uint8_t smem_raw[];
@@ -164,10 +169,13 @@ mixer_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_con
   const int q_last = min(len, q_first + LA_BM) - 1;
   const int hi = q_last / LA_BN;
   const int lo = p.window > 0 ? max(0, q_first - p.window + 1) / LA_BN : 0;
-  const int kt = min((p.keep + LA_BN - 1) / LA_BN, lo);  // tiles of kept keys before the window
+  // keys before the window (of the last query, which sees most of them) and their tiles
+  const int before = p.pool > 0 ? max(0, q_last - p.window + 1) / p.pool : p.keep;
+  const int kt = p.pool > 0 ? (before + LA_BN - 1) / LA_BN : min((p.keep + LA_BN - 1) / LA_BN, lo);
   const int n_kv = kt + hi - lo + 1;  // >= 1: a token sees itself
   auto tile_at = [&](int j) { return j < kt ? j : lo + j - kt; };
-  auto width_at = [&](int j) { return j < kt ? min(LA_BN, (p.keep - j * LA_BN + 31) & ~31) : LA_BN; };
+  auto width_at = [&](int j) { return j < kt ? min(LA_BN, (before - j * LA_BN + 31) & ~31) : LA_BN; };
+  const int pool_row = p.pool > 0 ? beg / p.pool : 0;  // where the sequence's blocks begin
 
   if (threadIdx.x == 0) {
     mbar_init(q_full, 1);
@@ -207,9 +215,10 @@ mixer_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_con
         const int s = j % p.k_stages;
         if (!mbar_wait(&k_empty[s], (uint32_t)(((j / p.k_stages) & 1) ^ 1), abort_flag, p.status, 1200 + s)) return false;
         uint8_t* ks = k_s + (size_t)s * k_bytes;
-        const int row = beg + tile_at(j) * LA_BN;
+        const bool mean = p.pool > 0 && j < kt;
+        const int row = (mean ? pool_row : beg) + tile_at(j) * LA_BN;
         mbar_expect_tx(&k_full[s], k_bytes);
-        for (int i = 0; i < p.nn; ++i) tma_load_3d(ks + i * LA_BOX, &tm_kn, &k_full[s], 64 * i, hk, row);
+        for (int i = 0; i < p.nn; ++i) tma_load_3d(ks + i * LA_BOX, mean ? &tm_pk : &tm_kn, &k_full[s], 64 * i, hk, row);
         for (int i = 0; i < p.nr; ++i) tma_load_2d(ks + (p.nn + i) * LA_BOX, &tm_kr, &k_full[s], 64 * i, row);
         return true;
       };
@@ -221,7 +230,9 @@ mixer_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_con
         if (!mbar_wait(&v_empty[s], (uint32_t)(((j / p.v_stages) & 1) ^ 1), abort_flag, p.status, 1205 + s)) break;
         uint8_t* vs = v_s + (size_t)s * v_bytes;
         mbar_expect_tx(&v_full[s], v_bytes);
-        for (int i = 0; i < p.nv; ++i) tma_load_3d(vs + i * LA_BOX, &tm_v, &v_full[s], 64 * i, hk, beg + tile_at(j) * LA_BN);
+        const bool mean = p.pool > 0 && j < kt;
+        const int row = (mean ? pool_row : beg) + tile_at(j) * LA_BN;
+        for (int i = 0; i < p.nv; ++i) tma_load_3d(vs + i * LA_BOX, mean ? &tm_pv : &tm_v, &v_full[s], 64 * i, hk, row);
         if (NB == 1 && j + 1 < n_kv) ok = load_k(j + 1);  // one stage: free only after S(j)
       }
     }
@@ -291,13 +302,15 @@ mixer_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_con
     for (int j = 0; j < n_kv && ok; ++j) {
       const int s = j % NB;
       const int key0 = tile_at(j) * LA_BN, width = width_at(j);
-      const bool full = width == LA_BN && q_first + LA_BM <= len && key0 + LA_BN - 1 <= q_first &&
+      const bool mean = p.pool > 0 && j < kt;
+      const bool full = mean ? q_first + LA_BM <= len && key0 + LA_BN <= max(0, q_first - p.window + 1) / p.pool
+                             : width == LA_BN && q_first + LA_BM <= len && key0 + LA_BN - 1 <= q_first &&
                         (p.window <= 0 || key0 >= q_first + LA_BM - p.window || key0 + LA_BN <= p.keep);
       ok = __all_sync(0xffffffffu, mbar_wait(&s_full[s], (uint32_t)((j / NB) & 1), abort_flag, p.status, 1270 + s));
       if (!ok) break;
       tc_fence_after();
       const uint32_t ts = tmem_base + lane_off + (uint32_t)s * LA_BN;
-      const int first = k_min - key0, last = k_max - key0, kept = p.keep - key0;
+      const int first = (mean ? 0 : k_min) - key0, last = (mean ? (row_ok ? k_min / p.pool : 0) - 1 : k_max) - key0, kept = p.keep - key0;
       const float2 top = full ? la_row_max<CAP, true>(ts, width, first, last, kept) : la_row_max<CAP, false>(ts, width, first, last, kept);
       const float mx = top.x;
       int level = -1;
@@ -357,10 +370,10 @@ mixer_attn_tc_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_con
           const size_t t = (size_t)(beg + q_pos), th = t * p.heads + h;
           const float sk = p.sink != nullptr ? p.sink[h] * 1.4426950408889634f : -INFINITY, mt = fmaxf(m_ref, sk);
           const float wm = fast_exp2(m_ref - mt);
-          f = wm / (l_run * wm + fast_exp2(sk - mt));
+          f = p.out_scale * wm / (l_run * wm + fast_exp2(sk - mt));
           if (p.gate_mode == GATE_HEAD) f *= reinterpret_cast<const float*>(p.gate)[th];
           if (p.gate_mode == GATE_LOGITS) gl = reinterpret_cast<const __nv_bfloat16*>(p.gate) + t * p.gate_ld + (size_t)h * p.vdim;
-          dst = p.out + th * p.vdim;
+          dst = p.out + t * p.out_ld + (size_t)h * p.vdim;
         }
 #pragma unroll 1
         for (int c = 0; c < p.vdim; c += 32) {
@@ -444,17 +457,21 @@ TRLB_API int trlb_mixer_attn_tc_ok(int heads, int kv_heads, int dim, int rot, in
 // q [T rows of q_ld]: heads x (dim + rot), rotated part last; k, v [T rows of k_ld / v_ld]: kv_heads x dim / vdim; krot [T rows
 // of krot_ld]: the shared rotated keys (rot > 0).  All bf16, rows on 16 bytes.  window <= 0: unlimited, else the first `keep` keys stay
 // visible; cap <= 0: none; scale > 0;
-// sink may be null; gate by gate_mode (0 none, 1 fp32 [T, heads], 2 bf16 logits [T rows of gate_ld]).
+// pool > 0 (with a window, without rot and keep): pk, pv [T / pool + 1, kv_heads, dim / vdim], means as trlb_pool_blocks leaves them;
+// out [T rows of out_ld on 16 bytes], times out_scale; sink may be null; gate by gate_mode (0 none, 1 fp32 [T, heads], 2 bf16 logits [T rows of gate_ld]).
 TRLB_API int trlb_mixer_attn_tc(const void* q, long long q_ld, const void* k, long long k_ld, const void* v, long long v_ld,
                                 const void* krot, long long krot_ld, const int* cu, int n_seq, int T, int heads, int kv_heads,
                                 int dim, int rot, int vdim, int window, int keep, float scale, float cap, const float* sink,
-                                int gate_mode, const void* gate, long long gate_ld, void* out, int* status, cudaStream_t st) {
+                                int gate_mode, const void* gate, long long gate_ld, int pool, const void* pk, const void* pv, void* out,
+                                long long out_ld, float out_scale, int* status, cudaStream_t st) {
   if (T <= 0 || n_seq <= 0) return 0;
   if (!trlb_mixer_attn_tc_ok(heads, kv_heads, dim, rot, vdim) || (q_ld % 8) || (k_ld % 8) || (v_ld % 8) || !(scale > 0.f)) return -210;
   if (rot > 0 && (krot_ld % 8)) return -210;
+  if ((out_ld % 8) || (reinterpret_cast<uintptr_t>(out) & 15) || (pool > 0 && (pk == nullptr || pv == nullptr || keep > 0 || rot > 0))) return -210;
   if (gate_mode == GATE_LOGITS && ((gate_ld % 8) || (reinterpret_cast<uintptr_t>(gate) & 15))) return -210;
   MixerAttnTc p = {};
   p.cu = cu; p.n_seq = n_seq; p.heads = heads; p.group = heads / kv_heads; p.dim = dim; p.rot = rot; p.vdim = vdim; p.window = window; p.keep = window > 0 && keep > 0 ? keep : 0;
+  p.pool = window > 0 && pool > 0 ? pool : 0;
   p.nn = la_boxes(dim); p.nr = la_boxes(rot); p.nv = la_boxes(vdim);
   const bool pair = la_pair(p.nn + p.nr, p.nv, vdim);
   if (pair) p.k_stages = p.v_stages = 1;
@@ -469,21 +486,29 @@ TRLB_API int trlb_mixer_attn_tc(const void* q, long long q_ld, const void* k, lo
     p.near7 = (float)(0.12 / in);   // the first term left out is below 1e-9 of tanh
     p.near11 = (float)(0.35 / in);  // below 2e-8
   }
-  p.sink = sink; p.gate_mode = gate_mode; p.gate = gate; p.gate_ld = gate_ld; p.out = (__nv_bfloat16*)out; p.status = status;
+  p.sink = sink; p.gate_mode = gate_mode; p.gate = gate; p.gate_ld = gate_ld; p.out = (__nv_bfloat16*)out; p.out_ld = out_ld; p.out_scale = out_scale; p.status = status;
   const __nv_bfloat16* qb = (const __nv_bfloat16*)q;
   const int dq = dim + rot;
-  CUtensorMap tqn, tqr, tkn, tkr, tv;
+  CUtensorMap tqn, tqr, tkn, tkr, tv, tpk, tpv;
   using trlb_host::make_tmap_3d_bf16;
   if (make_tmap_3d_bf16(&tqn, qb, dim, heads, T, dq, (uint64_t)q_ld, 64, 1, 128)) return -211;
   if (make_tmap_3d_bf16(&tkn, k, dim, kv_heads, T, dim, (uint64_t)k_ld, 64, 1, 128)) return -213;
   if (make_tmap_3d_bf16(&tv, v, vdim, kv_heads, T, vdim, (uint64_t)v_ld, 64, 1, 128)) return -215;
   tqr = tqn;
   tkr = tkn;
+  tpk = tkn;
+  tpv = tv;
+  if (p.pool > 0) {
+    const uint64_t rows = (uint64_t)(T / pool + 1);
+    if (make_tmap_3d_bf16(&tpk, pk, dim, kv_heads, rows, dim, (uint64_t)kv_heads * dim, 64, 1, 128)) return -217;
+    if (make_tmap_3d_bf16(&tpv, pv, vdim, kv_heads, rows, vdim, (uint64_t)kv_heads * vdim, 64, 1, 128)) return -218;
+  }
   if (rot > 0) {
     if (make_tmap_3d_bf16(&tqr, qb + dim, rot, heads, T, dq, (uint64_t)q_ld, 64, 1, 128)) return -212;
     if (trlb_host::make_tmap_2d_bf16(&tkr, krot, T, rot, (uint64_t)krot_ld, 128, 64)) return -214;
   }
-  using Kern = void (*)(const CUtensorMap, const CUtensorMap, const CUtensorMap, const CUtensorMap, const CUtensorMap, const MixerAttnTc);
+  using Kern = void (*)(const CUtensorMap, const CUtensorMap, const CUtensorMap, const CUtensorMap, const CUtensorMap, const CUtensorMap,
+                        const CUtensorMap, const MixerAttnTc);
   static const Kern kerns[4] = {mixer_attn_tc_kernel<false, 1>, mixer_attn_tc_kernel<true, 1>, mixer_attn_tc_kernel<false, 2>,
                                 mixer_attn_tc_kernel<true, 2>};
   static bool attr_set = false;
@@ -494,6 +519,6 @@ TRLB_API int trlb_mixer_attn_tc(const void* q, long long q_ld, const void* k, lo
   }
   const dim3 grid((T + LA_BM - 1) / LA_BM + n_seq, heads);
   const size_t smem = la_smem(p.nn + p.nr, p.nv, p.k_stages, p.v_stages);
-  kerns[(pair ? 0 : 2) + (cap > 0.f)]<<<grid, LA_THREADS, smem, st>>>(tqn, tqr, tkn, tkr, tv, p);
+  kerns[(pair ? 0 : 2) + (cap > 0.f)]<<<grid, LA_THREADS, smem, st>>>(tqn, tqr, tkn, tkr, tv, tpk, tpv, p);
   return (int)cudaGetLastError();
 }

@@ -34,7 +34,46 @@ embed_scaled_kernel(const long long* __restrict__ ids, const T* __restrict__ emb
     x[(size_t)blockIdx.x * H + j] = (id >= 0 && id < V) ? to_f(emb[(size_t)id * H + j]) * scale : 0.f;
 }
 
-// The same plus a row of a table of token pairs: row (previous * mul_prev + current * mul_cur) mod buckets, or the last row,
+// The same over its root mean square, times shift + w; copy (may be null) gets the row too.
+template <typename T>
+__global__ void __launch_bounds__(256)
+embed_normed_kernel(const long long* __restrict__ ids, const T* __restrict__ emb, const float* __restrict__ w, float* __restrict__ x,
+                    float* __restrict__ copy, int H, int V, float scale, float eps, float shift) {
+  __shared__ float red[64];
+  pdl_launch_dependents();
+  pdl_wait();
+  const long long id = ids[blockIdx.x];
+  const bool ok = id >= 0 && id < V, v4 = (H & 3) == 0;
+  const T* e = emb + (size_t)(ok ? id : 0) * H;
+  const size_t row = (size_t)blockIdx.x * H;
+  float s = 0.f;
+  if (v4) {
+    for (int j = 4 * threadIdx.x; j < H; j += 4 * blockDim.x) {
+      const float4 v = load4(e + j);
+      s += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+    }
+  } else {
+    for (int j = threadIdx.x; j < H; j += blockDim.x) s += to_f(e[j]) * to_f(e[j]);
+  }
+  const float ss = block_sum2(s, 0.f, red).x;
+  const float r = ok ? scale / sqrtf(ss * (scale * scale) / (float)H + eps) : 0.f;
+  if (v4) {
+    for (int j = 4 * threadIdx.x; j < H; j += 4 * blockDim.x) {
+      const float4 v = load4(e + j), g = load4(w + j);
+      const float4 o = make_float4(v.x * r * (shift + g.x), v.y * r * (shift + g.y), v.z * r * (shift + g.z), v.w * r * (shift + g.w));
+      store4(x + row + j, o);
+      if (copy != nullptr) store4(copy + row + j, o);
+    }
+  } else {
+    for (int j = threadIdx.x; j < H; j += blockDim.x) {
+      const float o = to_f(e[j]) * r * (shift + w[j]);
+      x[row + j] = o;
+      if (copy != nullptr) copy[row + j] = o;
+    }
+  }
+}
+
+// The same (without the norm) plus a row of a table of token pairs: row (previous * mul_prev + current * mul_cur) mod buckets, or the last row,
 // number `buckets`, at a sequence's first token.  Prompt rows (prev_state is written by a sequence's last row, tok_slot gives
 // the slots; both may be null) take the previous token from ids; decode rows (one per slot, positions negative: idle) from
 // prev_state, which moves on.
@@ -133,8 +172,10 @@ gelu_erf_kernel(const T* __restrict__ z, T* __restrict__ out, long long n) {
 
 // ------------------------------------------------------------------------------------------------------------
 // RMS norms around the residual stream, in one pass over a row:
-//     x += delta                      or, with `post`,   x += delta / rms(delta) * (shift + post) * post_scale
+//     x += mult d                     or, with `post`,   x += mult d / rms(d) * (shift + post) * post_scale
 //     out = x / rms(x) * (shift + w) * gain              or, without `w`,   out = x
+// where d is delta, plus delta2, or plus the sum over the choices c of weight[c] * y[row[c]] (the experts' rows of this token; a
+// negative row: nothing).  x also gets anchor and bump, when given; out2 is the norm with w2 instead of w.
 // (no post_scale: 1).  `clear` zeroes delta behind itself.  One block per row; NV float4 of the row live in each thread's registers.
 // ------------------------------------------------------------------------------------------------------------
 struct RmsResidual {
@@ -145,7 +186,16 @@ struct RmsResidual {
   int H, clear;
   float eps;
   const float* post_scale;  // null: 1
-  float shift, gain;
+  float shift, gain, mult;
+  const float* delta2;      // [T, H] or null
+  const void* y;            // [rows, H] in the dtype of the output, or null
+  const int* row;           // [T, top]
+  const float* weight;      // [T, top]
+  int top;
+  const float* anchor;      // [T, H] or null
+  const float* bump;        // [H] or null
+  const float* w2;          // null: one output
+  void* out2;
 };
 
 __device__ __forceinline__ float4 rms_weight4(const float* w, const float* scale, float shift, float gain, int j) {
@@ -156,6 +206,9 @@ __device__ __forceinline__ float4 rms_weight4(const float* w, const float* scale
     g = make_float4(g.x * c.x, g.y * c.y, g.z * c.z, g.w * c.w);
   }
   return g;
+}
+__device__ __forceinline__ float4 fma4(float s, float4 a, float4 b) {
+  return make_float4(fmaf(s, a.x, b.x), fmaf(s, a.y, b.y), fmaf(s, a.z, b.z), fmaf(s, a.w, b.w));
 }
 
 template <typename T, int NV>
@@ -178,18 +231,44 @@ rms_residual_kernel(const RmsResidual p, T* __restrict__ out) {
     for (int i = 0; i < NV; ++i) {
       const int j = threadIdx.x + i * nt;
       d[i] = j < n4 ? load4(p.delta + row + 4 * j) : make_float4(0.f, 0.f, 0.f, 0.f);
-      sd += d[i].x * d[i].x + d[i].y * d[i].y + d[i].z * d[i].z + d[i].w * d[i].w;
+      if (p.delta2 != nullptr && j < n4) d[i] = fma4(1.f, load4(p.delta2 + row + 4 * j), d[i]);
     }
+    if (p.y != nullptr) {
+      for (int c = 0; c < p.top; ++c) {
+        const int at = p.row[(size_t)blockIdx.x * p.top + c];
+        if (at < 0) continue;
+        const float wt = p.weight[(size_t)blockIdx.x * p.top + c];
+        const T* y = reinterpret_cast<const T*>(p.y) + (size_t)at * p.H;
+#pragma unroll
+        for (int i = 0; i < NV; ++i) {
+          const int j = threadIdx.x + i * nt;
+          if (j < n4) d[i] = fma4(wt, load4(y + 4 * j), d[i]);
+        }
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < NV; ++i) sd += d[i].x * d[i].x + d[i].y * d[i].y + d[i].z * d[i].z + d[i].w * d[i].w;
     float r = 1.f;
     if (p.post != nullptr) r = 1.f / sqrtf(block_sum2(sd, 0.f, red).x / (float)p.H + p.eps);
+    r *= p.mult;
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
       const int j = threadIdx.x + i * nt;
       if (j < n4) {
         const float4 g = p.post != nullptr ? rms_weight4(p.post, p.post_scale, p.shift, 1.f, 4 * j) : make_float4(1.f, 1.f, 1.f, 1.f);
         a[i].x += d[i].x * r * g.x; a[i].y += d[i].y * r * g.y; a[i].z += d[i].z * r * g.z; a[i].w += d[i].w * r * g.w;
-        store4(p.x + row + 4 * j, a[i]);
         if (p.clear) store4(p.delta + row + 4 * j, make_float4(0.f, 0.f, 0.f, 0.f));
+      }
+    }
+  }
+  if (p.delta != nullptr || p.anchor != nullptr || p.bump != nullptr) {
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int j = threadIdx.x + i * nt;
+      if (j < n4) {
+        if (p.anchor != nullptr) a[i] = fma4(1.f, load4(p.anchor + row + 4 * j), a[i]);
+        if (p.bump != nullptr) a[i] = fma4(1.f, load4(p.bump + 4 * j), a[i]);
+        store4(p.x + row + 4 * j, a[i]);
       }
     }
   }
@@ -206,6 +285,10 @@ rms_residual_kernel(const RmsResidual p, T* __restrict__ out) {
     if (j < n4) {
       const float4 g = p.w != nullptr ? rms_weight4(p.w, nullptr, p.shift, p.gain, 4 * j) : make_float4(1.f, 1.f, 1.f, 1.f);
       store4(out + row + 4 * j, make_float4(a[i].x * r * g.x, a[i].y * r * g.y, a[i].z * r * g.z, a[i].w * r * g.w));
+      if (p.w2 != nullptr) {
+        const float4 h = rms_weight4(p.w2, nullptr, p.shift, p.gain, 4 * j);
+        store4(reinterpret_cast<T*>(p.out2) + row + 4 * j, make_float4(a[i].x * r * h.x, a[i].y * r * h.y, a[i].z * r * h.z, a[i].w * r * h.w));
+      }
     }
   }
 }
@@ -220,24 +303,45 @@ rms_residual_any_kernel(const RmsResidual p, T* __restrict__ out) {
   const size_t row = (size_t)blockIdx.x * p.H;
   float* x = p.x + row;
   float* d = p.delta == nullptr ? nullptr : p.delta + row;
+  auto added = [&](int j) {
+    float v = d[j];
+    if (p.delta2 != nullptr) v += p.delta2[row + j];
+    if (p.y != nullptr) {
+      for (int c = 0; c < p.top; ++c) {
+        const int at = p.row[(size_t)blockIdx.x * p.top + c];
+        if (at >= 0) v = fmaf(p.weight[(size_t)blockIdx.x * p.top + c], to_f(reinterpret_cast<const T*>(p.y)[(size_t)at * p.H + j]), v);
+      }
+    }
+    return v;
+  };
   float r = 1.f, s = 0.f;
   if (d != nullptr && p.post != nullptr) {
-    for (int j = threadIdx.x; j < p.H; j += 256) s += d[j] * d[j];
+    for (int j = threadIdx.x; j < p.H; j += 256) {
+      const float v = added(j);
+      s += v * v;
+    }
     r = 1.f / sqrtf(block_sum2(s, 0.f, red).x / (float)p.H + p.eps);
   }
+  r *= p.mult;
   s = 0.f;
   for (int j = threadIdx.x; j < p.H; j += 256) {
     float a = x[j];
     if (d != nullptr) {
-      a += p.post != nullptr ? d[j] * r * (p.shift + p.post[j]) * (p.post_scale != nullptr ? p.post_scale[j] : 1.f) : d[j];
-      x[j] = a;
+      const float v = added(j) * r;
+      a += p.post != nullptr ? v * (p.shift + p.post[j]) * (p.post_scale != nullptr ? p.post_scale[j] : 1.f) : v;
       if (p.clear) d[j] = 0.f;
     }
+    if (p.anchor != nullptr) a += p.anchor[row + j];
+    if (p.bump != nullptr) a += p.bump[j];
+    x[j] = a;
     s += a * a;
   }
   float rx = 1.f;
   if (p.w != nullptr) rx = 1.f / sqrtf(block_sum2(s, 0.f, red).x / (float)p.H + p.eps);
-  for (int j = threadIdx.x; j < p.H; j += 256) out[row + j] = from_f<T>(p.w != nullptr ? x[j] * rx * (p.shift + p.w[j]) * p.gain : x[j]);
+  for (int j = threadIdx.x; j < p.H; j += 256) {
+    out[row + j] = from_f<T>(p.w != nullptr ? x[j] * rx * (p.shift + p.w[j]) * p.gain : x[j]);
+    if (p.w2 != nullptr) reinterpret_cast<T*>(p.out2)[row + j] = from_f<T>(x[j] * rx * (p.shift + p.w2[j]) * p.gain);
+  }
 }
 
 // Gated linear units, z [rows, 2 n] = gate | up.  GELU: gelu_tanh(gate) up.  Else clamped: g sigmoid(alpha g) (u + shift), g =
@@ -798,6 +902,15 @@ TRLB_API int trlb_embed_scaled(const long long* ids, const void* emb, float* x, 
   return (int)trlb_host::launch_kernel(embed_scaled_kernel<float>, dim3(T), dim3(256), 0, st, PDL, ids, (const float*)emb, x, H, V, scale);
 }
 
+// copy may be null
+TRLB_API int trlb_embed_normed(const long long* ids, const void* emb, const float* w, float* x, float* copy, int T, int H, int V, float scale,
+                               float eps, float shift, int is_bf16, cudaStream_t st) {
+  if (T <= 0) return 0;
+  const dim3 blk(H >= 1024 ? 256 : 64);
+  if (is_bf16) return (int)trlb_host::launch_kernel(embed_normed_kernel<bf16>, dim3(T), blk, 0, st, PDL, ids, (const bf16*)emb, w, x, copy, H, V, scale, eps, shift);
+  return (int)trlb_host::launch_kernel(embed_normed_kernel<float>, dim3(T), blk, 0, st, PDL, ids, (const float*)emb, w, x, copy, H, V, scale, eps, shift);
+}
+
 // pairs [buckets + 1, H] in the dtype of emb; prev_state [slots] (decode: one row per slot) may be null, tok_slot in decode
 TRLB_API int trlb_embed_pairs(const long long* ids, const void* emb, const void* pairs, float* x, int T, int H, int V, float scale,
                               long long mul_prev, long long mul_cur, long long buckets, const int* positions, const int* tok_slot,
@@ -823,11 +936,14 @@ TRLB_API int trlb_dynamic_tanh(float* x, float* delta, const float* alpha, const
 #undef GO
 }
 
-// post, post_scale, w, delta may be null (see RmsResidual); H: row length
+// post, post_scale, w, delta, delta2, y, anchor, bump, w2 may be null (see RmsResidual); H: row length
 TRLB_API int trlb_rms_residual(float* x, float* delta, const float* post, const float* post_scale, const float* w, void* out, int T,
-                               int H, float eps, float shift, float gain, int clear, int is_bf16, cudaStream_t st) {
+                               int H, float eps, float shift, float gain, float mult, int clear, const float* delta2, const void* y,
+                               const int* row, const float* weight, int top, const float* anchor, const float* bump, const float* w2,
+                               void* out2, int is_bf16, cudaStream_t st) {
   if (T <= 0) return 0;
-  const RmsResidual p = {x, delta, post, w, H, clear, eps, post_scale, shift, gain};
+  if ((delta == nullptr && (delta2 != nullptr || y != nullptr)) || (w2 != nullptr && (w == nullptr || out2 == nullptr))) return -208;
+  const RmsResidual p = {x, delta, post, w, H, clear, eps, post_scale, shift, gain, mult, delta2, y, row, weight, top, anchor, bump, w2, out2};
   const int n4 = H / 4;
   const bool regs = H % 4 == 0 && n4 <= 256 * 8;
 #define GO(TT, NN) (int)trlb_host::launch_kernel(rms_residual_kernel<TT, NN>, dim3(T), dim3(n4 >= 256 ? 256 : (n4 + 31) / 32 * 32), 0, st, PDL, p, (TT*)out)

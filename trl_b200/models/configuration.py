@@ -288,6 +288,12 @@ PRESETS: dict[str, dict] = {
                      mixer=dict(heads=4, kv_heads=4, dim=16, vdim=16, scale=0.25, rot=dict(base=1e5, dims=16))),
                 dict(type="attention_2", mlp=dict(kind="moe", expert=dict(ff=32, limit=4.0), router=dict(experts=4, top=2)),
                      mixer=dict(heads=4, kv_heads=4, dim=16, vdim=16, scale=0.25, rot=dict(base=1e5, dims=16), kv_from=1))]),
+    "tiny-gerupel": dict(
+        architecture="Gerupel", vocab=1024, width=64, norm=dict(eps=1e-5), residual_mult=0.7, loop=dict(start=1, stop=2, times=2),
+        layers=[dict(type="parallel", mlp=dict(kind="moe", expert=dict(ff=32), router=dict(experts=4, top=2, scale=1.5)),
+                     mixer=dict(left=dict(heads=4, kv_heads=2, dim=16, vdim=16, scale=0.25, mask=dict(size=24, pool=8),
+                                          rot=dict(base=1e4, dims=8, scaling=dict(factor=4.0, low=1.0, high=4.0, original=256))),
+                                right=dict(heads=2, dim=16, vdim=32), left_scale=0.9, right_scale=0.6)) for _ in range(3)]),
 }
 
 

@@ -20,6 +20,10 @@ Designs
                 embedding, ``attention`` (the projected keys are the values; weighted norms per head, YaRN rotation, window with
                 kept first tokens, capped scores, softmax sink, gate per head) and ``attention_2`` (norms over all heads, rotated
                 halves; a layer may read another one's cache) mixers, GELU-gated or expert feed-forward, tied head with a scale.
+    Gerupel     mixer and feed-forward side by side behind a norm each, the residual sum times a constant, a run of layers
+                repeated with the embedding added again, a norm on the embedding, ``parallel`` mixers (``attention`` over a window
+                and pooled blocks before it, Llama-3 frequency scaling, factor per head, one in the softmax denominator, beside
+                ``hgrn2``: linear attention whose forget gate also writes), experts chosen by softmax, tied head.
 
 The residual stream, norms, gates and recurrent states are fp32 whatever the model dtype.
 """
@@ -28,6 +32,7 @@ from __future__ import annotations
 import copy
 import dataclasses
 import json
+import math
 import os
 from dataclasses import dataclass, field
 from typing import Any
@@ -44,11 +49,14 @@ from .decoder import CausalLM, SeqCtx
 class AttentionStyle:
     """What a design fixes about a grouped-query attention mixer."""
 
-    norm_weight: bool = False    # queries and keys over their rms times a weight
+    norm: bool = True            # queries and keys over their rms
+    norm_weight: bool = False    # times a weight
     whole_norm: bool = False     # that norm over all heads at once instead of per head
     halves: bool = False         # rotated pairs (i, i + dims / 2) instead of (2 i, 2 i + 1)
     values: bool = True          # a projection of values; without it the projected keys serve as values
     sink: bool = False           # exp(sink) in the softmax denominator
+    sink_one: bool = False       # the same with exp(sink) = 1 for every head
+    temp: bool = False           # scores times a number per head
     gate: str | None = "element"  # sigmoid gates per "element" or per "head" of the output
 
 
@@ -57,8 +65,11 @@ class Design:
     """What a design fixes for all its models."""
 
     norm: str
-    mlp: str                     # dense feed-forward
+    mlp: str | None              # dense feed-forward
     moe: str | None = None       # feed-forward of kind 'moe'
+    beside: bool = False         # mixer and feed-forward read the same stream, each through its norm, and are added together
+    embed_norm: bool = False     # a norm on the embedding
+    sides: tuple = ()            # mixer 'parallel': the kinds of its left and its right half
     pre_norm: bool = True        # a norm on the input of every sublayer; without it the sublayers read the stream itself
     post_norm: bool = False      # a norm on the output of every sublayer, before it is added
     layer_scale: bool = False    # that norm's result times a vector
@@ -75,17 +86,22 @@ DESIGNS: dict[str, Design] = {
                       tied_head=True,
                       attention={"attention": AttentionStyle(norm_weight=True, values=False, sink=True, gate="head"),
                                  "attention_2": AttentionStyle(norm_weight=True, whole_norm=True, halves=True, gate=None)}),
+    "Gerupel": Design(norm="rms", mlp=None, moe="softmax_experts", beside=True, embed_norm=True, sides=("attention", "hgrn2"), tied_head=True,
+                      attention={"attention": AttentionStyle(norm=False, halves=True, sink_one=True, temp=True, gate=None)}),
 }
 
 
 @dataclass
 class LayerSpec:
-    """One entry of the layer list.  ``owner``: index of the layer whose tensors this one runs with (itself, usually)."""
+    """One layer run.  ``owner``: place of the run whose tensors this one runs with (itself, usually); ``index``: entry of the
+    layer list; ``enters``: number of the loop's pass that begins in front of it."""
 
     kind: str
     mixer: dict
     mlp: dict | None
     owner: int
+    index: int
+    enters: int | None = None
 
     @property
     def ff(self) -> int:
@@ -99,7 +115,9 @@ class LayerSpec:
 @dataclass
 class LayeredArch(ModelArch):
     design: str = ""
-    layers: list = field(default_factory=list)  # [LayerSpec]
+    layers: list = field(default_factory=list)  # [LayerSpec], in the order of computation: a loop is unrolled
+    passes: int = 0  # of the loop (0: none)
+    residual_mult: float = 1.0  # what sublayer outputs are multiplied by when they are added
     side_dim: int = 0  # per-token input of every layer: elements per layer (0: none)
     pairs: dict | None = None  # table of token pairs: mul_prev, mul_cur, buckets
     logit_scale: float = 1.0
@@ -115,26 +133,30 @@ class LayeredArch(ModelArch):
             if e["type"] not in MIXERS:
                 raise ValueError(f"layer {i}: mixer {e['type']!r} is not registered; known: {sorted(MIXERS)}")
             mlp = e.get("mlp")
-            if mlp is not None and mlp.get("kind", "dense") != "dense" and not (mlp["kind"] == "moe" and DESIGNS[name].moe):
-                raise ValueError(f"layer {i}: feed-forward kind {mlp['kind']!r} is not supported")
+            if mlp is not None and not dict(dense=DESIGNS[name].mlp, moe=DESIGNS[name].moe).get(mlp.get("kind", "dense")):
+                raise ValueError(f"layer {i}: feed-forward kind {mlp.get('kind', 'dense')!r} is not supported")
             owner = i
             if e.get("weights_of") is not None:
                 j = int(e["weights_of"])
                 if not 0 <= j < i:
                     raise ValueError(f"layer {i}: weights_of={j} must name an earlier layer")
                 owner = specs[j].owner
-            s = LayerSpec(e["type"], dict(e["mixer"]), None if mlp is None else dict(mlp), owner)
+            s = LayerSpec(e["type"], dict(e["mixer"]), None if mlp is None else dict(mlp), owner, i)
             _check_lender(specs, s, i)
             if owner != i and s.key != specs[owner].key:
                 raise ValueError(f"layer {i} runs with the weights of layer {owner} but is described differently")
             specs.append(s)
+        loop = d.get("loop")
+        if loop:
+            specs = _unrolled(specs, int(loop["start"]), int(loop["stop"]), int(loop["times"]))
         design = DESIGNS[name]
         embedding = d.get("embedding") or {}
-        heads = max((s.mixer.get("heads", 1) for s in specs), default=1)
+        heads = max((h.get("heads", 1) for s in specs for h in (s.mixer, s.mixer.get("left") or {}, s.mixer.get("right") or {})), default=1)
         return cls(model_type=name.lower(), design=name, vocab_size=d["vocab"], hidden_size=d["width"],
                    intermediate_size=max((s.ff for s in specs), default=0), num_hidden_layers=len(specs),
                    num_attention_heads=heads, num_key_value_heads=heads, rms_norm_eps=float(d["norm"]["eps"]),
                    embed_scale=float(embedding.get("scale", 1.0)), layers=specs, source=copy.deepcopy(d),
+                   passes=int(loop["times"]) if loop else 0, residual_mult=float(d.get("residual_mult", 1.0)),
                    pairs=dict(embedding["bigram"]) if embedding.get("bigram") else None, logit_scale=float(d.get("logit_scale", 1.0)),
                    side_dim=int((d.get("token_side") or {}).get("dim", 0)), tie_word_embeddings=design.tied_head,
                    attention_bias=False, qk_norm=False, pad_token_id=d.get("pad_token_id"),
@@ -163,6 +185,21 @@ class LayeredArch(ModelArch):
         return {s.mixer["kv_from"] for s in self.layers if s.mixer.get("kv_from") is not None}
 
 
+def _unrolled(specs: list, start: int, stop: int, times: int) -> list:
+    """Layer runs of a list whose entries ``start`` .. ``stop`` - 1 run ``times`` times in a row with the same weights."""
+    if not 0 <= start < stop <= len(specs) or times < 1:
+        raise ValueError(f"loop over layers {start} .. {stop - 1} of {len(specs)}, {times} times")
+    if any(s.mixer.get("kv_from") is not None for s in specs):
+        raise ValueError("a loop together with layers that read another one's keys and values")
+    out, first = [], {}
+    for t in range(times):
+        out += [(s, t if s.index == start else None) for s in specs[start:stop]]
+    out = [(s, None) for s in specs[:start]] + out + [(s, None) for s in specs[stop:]]
+    for place, (s, _) in enumerate(out):
+        first.setdefault(s.index, place)
+    return [dataclasses.replace(s, owner=first[s.owner], enters=t) for s, t in out]
+
+
 def _check_lender(specs: list, s: LayerSpec, i: int):
     j = s.mixer.get("kv_from")
     if j is None:
@@ -185,8 +222,8 @@ class DynamicTanh(nn.Module):
 
     def __init__(self, cfg: LayeredArch, device=None, **kw):
         super().__init__()
-        if kw:
-            raise NotImplementedError(f"Dynamic Tanh with {sorted(kw)}")
+        if kw or cfg.residual_mult != 1.0:
+            raise NotImplementedError(f"Dynamic Tanh with {sorted(kw) or 'residual_mult'}")
         n = cfg.hidden_size
         self.weight, self.bias, self.alpha = _vec(n, 1.0, device), _vec(n, 0.0, device), _vec(None, 0.5, device)
 
@@ -209,7 +246,7 @@ class RmsNorm(nn.Module):
 
     def __init__(self, cfg: LayeredArch, device=None, gain: float = 1.0, scale: bool = False):
         super().__init__()
-        self.weight, self.eps, self.gain = _vec(cfg.hidden_size, 1.0 - self.shift, device), cfg.rms_norm_eps, gain
+        self.weight, self.eps, self.gain, self.mult = _vec(cfg.hidden_size, 1.0 - self.shift, device), cfg.rms_norm_eps, gain, cfg.residual_mult
         self.scale = _vec(cfg.hidden_size, 1.0, device) if scale else None
 
     def tensors(self, name):
@@ -217,13 +254,13 @@ class RmsNorm(nn.Module):
 
     def forward(self, x, out_dtype, delta=None, post=None, **kw):
         return mx.rms_residual(x, delta, w=self.weight, eps=self.eps, out_dtype=out_dtype, shift=self.shift, gain=self.gain,
-                               **_weights(post), **kw)
+                               mult=self.mult, **_weights(post), **kw)
 
     @staticmethod
-    def stream(x, out_dtype, delta, post, **kw):
+    def stream(x, out_dtype, delta, post, mult=1.0, **kw):
         """The stream itself after the addition of ``delta`` (normed by ``post``), in ``out_dtype``, and in fp32."""
         eps, shift = (0.0, 0.0) if post is None else (post.eps, post.shift)
-        return mx.rms_residual(x, delta, w=None, eps=eps, out_dtype=out_dtype, shift=shift, **_weights(post), **kw)
+        return mx.rms_residual(x, delta, w=None, eps=eps, out_dtype=out_dtype, shift=shift, mult=mult, **_weights(post), **kw)
 
 
 class RmsNormAboutZero(RmsNorm):
@@ -334,18 +371,20 @@ class MLstm(nn.Module):
 
 class GroupedAttention(nn.Module):
     """Grouped-query attention: queries and keys over their rms, optionally rotated, queries optionally times a temperature that
-    grows with the position, scores optionally capped by tanh, over all earlier keys or a window and the first tokens, the output
-    optionally times sigmoid gates that read the layer input (what of it a design has: :class:`AttentionStyle` and the layer's
-    sizes).  With ``kv_from`` the layer has no keys and values of its own and reads those of another layer.  The projections are
-    one matrix (query | key | value | gate, with gates per head filled up to whole 16-byte rows)."""
+    grows with the position or times a number per head, scores optionally capped by tanh, over all earlier keys or a window and
+    the first tokens or the means of the key blocks before it, the output optionally times sigmoid gates that read the layer input
+    (what of it a design has: :class:`AttentionStyle` and the layer's sizes).  With ``kv_from`` the layer has no keys and values
+    of its own and reads those of another layer.  The projections are one matrix (query | key | value | gate, with gates per head
+    filled up to whole 16-byte rows); a ``part`` of another mixer leaves both projections to that one."""
 
     kind = "attention"
+    f32_rows = 0  # rows of the input projection whose fp32 sums are needed
 
-    def __init__(self, cfg: LayeredArch, m: dict, dtype, device):
+    def __init__(self, cfg: LayeredArch, m: dict, dtype, device, part: bool = False):
         super().__init__()
         kw = dict(dtype=dtype, device=device)
         style = DESIGNS[cfg.design].attention.get(self.kind, AttentionStyle())
-        self.eps = cfg.rms_norm_eps
+        self.eps, self.dtype = cfg.rms_norm_eps, dtype
         self.heads, self.kv_heads, self.dim, self.vdim = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
         if self.heads % self.kv_heads:
             raise ValueError(f"{self.heads} query heads over {self.kv_heads} key/value heads")
@@ -356,49 +395,61 @@ class GroupedAttention(nn.Module):
         mask, rot = m.get("mask") or {}, m.get("rot")
         self.window = int(mask["size"]) if mask.get("size") else None
         self.keep = int(mask.get("keep_first") or 0)
+        self.pool = int(mask.get("pool") or 0) if self.window else 0
+        if self.pool and (self.keep or m.get("kv_from") is not None):
+            raise ValueError("pooled blocks together with kept tokens or another layer's cache")
         self.rot, self.rope = (int(rot["dims"]), mx.RotarySpec(rot["dims"], float(rot["base"]), rot.get("scaling"))) if rot else (0, None)
         if self.rot % 2 or self.rot > self.dim:
             raise ValueError(f"{self.rot} rotated elements of {self.dim}")
-        self.whole_norm, self.halves, self.values, self.gate = style.whole_norm, style.halves, style.values, style.gate
+        self.unit, self.whole_norm, self.halves, self.values, self.gate = style.norm, style.whole_norm, style.halves, style.values, style.gate
         if not self.values and self.vdim != self.dim:
             raise ValueError("values that are the keys have their size")
         self.kv_from = m.get("kv_from")
         own = self.kv_heads if self.kv_from is None else 0
         gates = {"element": self.heads * self.vdim, "head": self.heads, None: 0}[self.gate]
         self.parts = [self.heads * self.dim, own * self.dim, own * self.vdim if self.values else 0, gates]  # rows of w_in
-        h, fill = cfg.hidden_size, -sum(self.parts) % 8 if self.gate == "head" else 0
-        self.w_in = nn.Parameter(torch.empty(sum(self.parts) + fill, h, **kw))
-        if fill:
-            self.w_in.data[-fill:].zero_()
-        self.o = nn.Parameter(torch.empty(h, self.heads * self.vdim, **kw))
+        self.rows, self.out_width = sum(self.parts), self.heads * self.vdim
+        h, fill = cfg.hidden_size, -self.rows % 8 if self.gate == "head" else 0
+        if not part:
+            self.w_in = nn.Parameter(torch.empty(self.rows + fill, h, **kw))
+            if fill:
+                self.w_in.data[-fill:].zero_()
+            self.o = nn.Parameter(torch.empty(h, self.out_width, **kw))
         self.q_norm = self.k_norm = None
         if style.norm_weight:
             self.q_norm = _vec(self.heads * self.dim if self.whole_norm else self.dim, 1.0, device)
             if own:
                 self.k_norm = _vec(own * self.dim if self.whole_norm else self.dim, 1.0, device)
-        self.sink = _vec(self.heads, 0.0, device) if style.sink else None
+        self.temp = _vec(self.heads, 1.0, device) if style.temp else None
+        if style.sink_one:
+            self.register_buffer("sink", torch.zeros(self.heads, dtype=torch.float32, device=device), persistent=False)
+        else:
+            self.sink = _vec(self.heads, 0.0, device) if style.sink else None
+        self.sink_learned = style.sink
 
     @property
     def prep(self) -> dict:
         """How queries and keys are prepared (:func:`~trl_b200.ops.cuda_mixers.attn_prep`)."""
-        return dict(q_norm=self.q_norm, k_norm=self.k_norm, whole_norm=self.whole_norm, rot=self.rot, halves=self.halves,
-                    values=self.values, gates=self.gate)
+        return dict(q_norm=self.q_norm, k_norm=self.k_norm, unit=self.unit, whole_norm=self.whole_norm, q_head=self.temp, rot=self.rot,
+                    halves=self.halves, values=self.values, gates=self.gate)
 
     @property
     def sight(self) -> dict:
         """What a query sees besides the earlier tokens' keys as they are."""
         return dict(window=self.window, keep=self.keep, sink=self.sink)
 
-    def tensors(self, p):
-        q, k, v, g = self.w_in[: sum(self.parts)].split(self.parts)
-        out = {p + "q": q, p + "o": self.o}
+    def tensors(self, p, w_in=None, o=None):
+        """``w_in``, ``o``: where a part's projections are."""
+        q, k, v, g = (self.w_in[: self.rows] if w_in is None else w_in).split(self.parts)
+        out = {p + "q": q, p + "o": self.o if o is None else o}
         if self.kv_from is None:
             out[p + "k"] = k
             if self.values:
                 out[p + "v"] = v
         if self.gate:
             out[p + "g"] = g
-        out.update({p + n: t for n, t in (("q.norm", self.q_norm), ("k.norm", self.k_norm), ("sink", self.sink)) if t is not None})
+        out.update({p + n: t for n, t in (("q.norm", self.q_norm), ("k.norm", self.k_norm), ("sink", self.sink if self.sink_learned else None),
+                                          ("temp", self.temp)) if t is not None})
         return out
 
     def forward(self, h, ctx: SeqCtx, li: int):
@@ -446,7 +497,62 @@ class RgLru(nn.Module):
         return mx.rglru(self, h, ctx, li)
 
 
-MIXERS = {c.kind: c for c in (LatentAttention, MLstm, GroupedAttention, GroupedAttention2, RgLru)}
+class HGrn2(nn.Module):
+    """Linear attention in which one gate per head and channel forgets and writes: ``S = diag(f) S + (1 - f) v^T``, ``o = S^T q``
+    with ``f`` between a learned lower bound and one, and an RMS norm per head on the result.  The projections are one matrix
+    (query | value | forget gate); a ``part`` of another mixer leaves both projections to that one."""
+
+    kind = "hgrn2"
+
+    def __init__(self, cfg: LayeredArch, m: dict, dtype, device, part: bool = False):
+        super().__init__()
+        kw = dict(dtype=dtype, device=device)
+        self.eps, self.dtype = cfg.rms_norm_eps, dtype
+        self.heads, self.dim, self.vdim = m["heads"], m["dim"], m["vdim"]
+        qd, vd = self.heads * self.dim, self.heads * self.vdim
+        self.parts, self.rows, self.f32_rows, self.out_width = [qd, vd, qd], qd + vd, qd, vd
+        h = cfg.hidden_size
+        if not part:
+            self.w_in = nn.Parameter(torch.empty(sum(self.parts), h, **kw))
+            self.o = nn.Parameter(torch.empty(h, vd, **kw))
+        self.f_bias, self.lower, self.norm = _vec(qd, 0.0, device), _vec(qd, 0.0, device), _vec(self.vdim, 1.0, device)
+
+    def tensors(self, p, w_in=None, o=None):
+        """``w_in``, ``o``: where a part's projections are."""
+        q, v, f = (self.w_in if w_in is None else w_in).split(self.parts)
+        return {p + "q": q, p + "f": f, p + "f.b": self.f_bias, p + "lower": self.lower, p + "v": v, p + "norm": self.norm,
+                p + "o": self.o if o is None else o}
+
+    def forward(self, h, ctx: SeqCtx, li: int):
+        return mx.hgrn2(self, h, ctx, li)
+
+
+class ParallelMixers(nn.Module):
+    """Two mixers side by side: ``left_scale left(x) + right_scale right(x)``.  Both input projections are one matrix (left's rows
+    | right's rows | rows whose fp32 sums are needed), and so are both output projections; the scales go to the halves' results."""
+
+    kind = "parallel"
+
+    def __init__(self, cfg: LayeredArch, m: dict, dtype, device):
+        super().__init__()
+        kw = dict(dtype=dtype, device=device)
+        self.left, self.right = (MIXERS[k](cfg, m[s], dtype, device, part=True) for k, s in zip(DESIGNS[cfg.design].sides, ("left", "right")))
+        if self.left.f32_rows:
+            raise ValueError("the half with fp32 projections is the right one")
+        self.scales = (float(m["left_scale"]), float(m["right_scale"]))
+        self.rows = self.left.rows + self.right.rows
+        self.w_in = nn.Parameter(torch.empty(self.rows + self.right.f32_rows, cfg.hidden_size, **kw))
+        self.o = nn.Parameter(torch.empty(cfg.hidden_size, self.left.out_width + self.right.out_width, **kw))
+
+    def tensors(self, p):
+        a, b = self.left.rows, self.left.out_width
+        return {**self.left.tensors(p + "left.", self.w_in[:a], self.o[:, :b]), **self.right.tensors(p + "right.", self.w_in[a:], self.o[:, b:])}
+
+    def forward(self, h, ctx: SeqCtx, li: int):
+        return mx.parallel(self, h, ctx, li)
+
+
+MIXERS = {c.kind: c for c in (LatentAttention, MLstm, GroupedAttention, GroupedAttention2, RgLru, HGrn2, ParallelMixers)}
 
 
 class DenseMlp(nn.Module):
@@ -525,18 +631,20 @@ class ExpertMlp(nn.Module):
     correction and adds them up with their bare scores as weights.  The experts' matrices are stacked."""
 
     alpha, shift = 1.702, 1.0
+    scores = "sigmoid"
     renormalize = False  # weights over their sum
+    gain = 1.0           # of the weights
 
     def __init__(self, cfg: LayeredArch, spec: dict, dtype, device):
         super().__init__()
         kw = dict(dtype=dtype, device=device)
         self.n, self.top = int(spec["router"]["experts"]), int(spec["router"]["top"])
-        self.ff, self.limit = int(spec["expert"]["ff"]), float(spec["expert"]["limit"])
+        self.ff, self.limit = int(spec["expert"]["ff"]), float(spec["expert"].get("limit", math.inf))
         if not 1 <= self.top <= self.n <= 1024:
             raise ValueError(f"{self.top} of {self.n} experts (at most 1024)")
         h = cfg.hidden_size
         self.router = nn.Parameter(torch.empty(self.n, h, **kw))
-        self.correction = _vec(self.n, 0.0, device)
+        self.correction = _vec(self.n, 0.0, device) if self.scores == "sigmoid" else None
         self.gate_up = nn.Parameter(torch.empty(self.n, 2 * self.ff, h, **kw))
         self.down = nn.Parameter(torch.empty(self.n, h, self.ff, **kw))
 
@@ -544,17 +652,37 @@ class ExpertMlp(nn.Module):
     def glu(self):
         return self.limit, self.alpha, self.shift
 
+    @property
+    def routing(self) -> dict:
+        return dict(scores=self.scores, renormalize=self.renormalize, gain=self.gain)
+
     def tensors(self, p):
-        out = {p + "router": self.router, p + "correction": self.correction}
+        out = {p + "router": self.router}
+        if self.correction is not None:
+            out[p + "correction"] = self.correction
         for e in range(self.n):
             out.update({f"{p}e{e}.gate": self.gate_up[e, : self.ff], f"{p}e{e}.up": self.gate_up[e, self.ff:], f"{p}e{e}.down": self.down[e]})
         return out
 
-    def forward(self, h):
-        return mx.experts(self, h)
+    def forward(self, h, summed: bool = True):
+        """``summed``: see :func:`~trl_b200.ops.mixers.experts`."""
+        return mx.experts(self, h, summed=summed)
 
 
-MLPS = {"gelu": DenseMlp, "gelu_glu": GeluGluMlp, "clamped_glu": ClampedGluMlp, "clamped_glu_experts": ExpertMlp}
+class SoftmaxExpertMlp(ExpertMlp):
+    """Mixture of SiLU-gated units: the ``top`` experts of the largest softmax score, weighted with their scores over the sum of
+    these, times a constant."""
+
+    alpha, shift = 1.0, 0.0  # the clamped unit without its limit is the SiLU-gated one
+    scores, renormalize = "softmax", True
+
+    def __init__(self, cfg: LayeredArch, spec: dict, dtype, device):
+        super().__init__(cfg, spec, dtype, device)
+        self.gain = float(spec["router"].get("scale", 1.0))
+
+
+MLPS = {"gelu": DenseMlp, "gelu_glu": GeluGluMlp, "clamped_glu": ClampedGluMlp, "clamped_glu_experts": ExpertMlp,
+        "softmax_experts": SoftmaxExpertMlp}
 
 
 class TokenSide(nn.Module):
@@ -577,7 +705,8 @@ class TokenSide(nn.Module):
 
 class LayeredBlock(nn.Module):
     """Mixer and (optional) feed-forward around an fp32 residual stream; depending on the design with a norm on each sublayer's
-    input (norm1, norm2), on its output (norm1b, norm2b in memory), or both, and a per-token input after them."""
+    input (norm1, norm2), on its output (norm1b, norm2b in memory), or both, and a per-token input after them.  With ``beside``
+    both read the same stream, and what is pending after the layer are both outputs."""
 
     def __init__(self, cfg: LayeredArch, spec: LayerSpec, dtype, device):
         super().__init__()
@@ -592,7 +721,7 @@ class LayeredBlock(nn.Module):
             self.norm2, self.norm2b = pre(cfg, device), post(cfg, device, **scale)
             self.mlp = MLPS[design.moe if spec.mlp.get("kind") == "moe" else design.mlp](cfg, spec.mlp, dtype, device)
         self.side = TokenSide(cfg, dtype, device) if cfg.side_dim else None
-        self.dtype = dtype
+        self.dtype, self.mult, self.beside = dtype, cfg.residual_mult, design.beside
         self.lora = nn.ModuleDict()
         self.lora_enabled = True
 
@@ -616,18 +745,35 @@ class LayeredBlock(nn.Module):
 
     def read_mixer(self, x, delta, post, **kw):
         """What the mixer reads, and the stream after the addition of the pending ``delta``."""
-        return (RmsNorm.stream if self.norm1 is None else self.norm1)(x, self.dtype, delta, post, **kw)
+        return self._read(self.norm1, x, delta, post, **kw)
 
     def read_mlp(self, x, delta, post, **kw):
-        return (RmsNorm.stream if self.norm2 is None else self.norm2)(x, self.dtype, delta, post, **kw)
+        return self._read(self.norm2, x, delta, post, **kw)
+
+    def read_both(self, x, delta, post, **kw):
+        """What mixer and feed-forward read (one of the two without a feed-forward) of the same stream."""
+        if self.mlp is not None:
+            kw["w2"] = self.norm2.weight
+        h, x = self.norm1(x, self.dtype, delta, post, **kw)
+        return (h if self.mlp is not None else (h, None)), x
 
     def read_side(self, x, delta, post, **kw):
-        return RmsNorm.stream(x, self.dtype, delta, post, **kw)
+        return self._read(None, x, delta, post, **kw)
 
-    def forward(self, x, delta, post, ctx: SeqCtx, li: int, ids=None, side_table=None):
+    def _read(self, norm, x, delta, post, **kw):
+        if norm is None:
+            return RmsNorm.stream(x, self.dtype, delta, post, mult=self.mult, **kw)
+        return norm(x, self.dtype, delta, post, **kw)
+
+    def forward(self, x, delta, post, ctx: SeqCtx, li: int, ids=None, side_table=None, enter=None):
         """(residual, sublayer output not yet added to it, norm of that output) -> the same triple after this layer: every
-        addition rides on the norm that follows it."""
-        h, x = self.read_mixer(x, delta, post)
+        addition rides on the norm that follows it.  ``enter``: what a loop adds to the stream in front of this layer."""
+        enter = enter or {}
+        if self.beside:
+            (h, h2), x = self.read_both(x, delta, post, **enter)
+            delta = self.mixer(h, ctx, li)
+            return x, (delta if h2 is None else (delta, self.mlp(h2, summed=False))), None
+        h, x = self.read_mixer(x, delta, post, **enter)
         delta, post = self.mixer(h, ctx, li), self.norm1b
         if self.mlp is not None:
             h, x = self.read_mlp(x, delta, post)
@@ -650,6 +796,11 @@ class LayeredLM(CausalLM):
             raise NotImplementedError("layered designs have no classification head")
         self.config = cfg
         self.embed_tokens = nn.Parameter(torch.empty(cfg.vocab_size, cfg.hidden_size, dtype=dtype, device=device))
+        design = DESIGNS[cfg.design]
+        if cfg.passes and design.norm == "dynamic_tanh":
+            raise NotImplementedError("a loop over layers with Dynamic-Tanh norms")
+        self.embed_norm = NORMS[design.norm](cfg, device) if design.embed_norm else None
+        self.loop_step = nn.Parameter(torch.zeros(cfg.passes, cfg.hidden_size, dtype=torch.float32, device=device)) if cfg.passes else None
         blocks: list[LayeredBlock] = []
         for i, s in enumerate(cfg.layers):  # a layer that borrows weights IS its owner's block at another place
             blocks.append(blocks[s.owner] if s.owner != i else LayeredBlock(cfg, s, dtype, device))
@@ -677,13 +828,17 @@ class LayeredLM(CausalLM):
     def named_tensors(self) -> dict[str, torch.Tensor]:
         """Checkpoint name -> parameter or view into a fused parameter."""
         out = {"embed": self.embed_tokens}
+        if self.embed_norm is not None:
+            out.update(self.embed_norm.tensors("embed.norm"))
+        if self.loop_step is not None:
+            out["loop.step"] = self.loop_step
         if self.side_embed is not None:
             out["side.embed"] = self.side_embed
         if self.pair_embed is not None:
             out["bigram"] = self.pair_embed
         for i, (s, b) in enumerate(zip(self.config.layers, self.layers)):
             if s.owner == i:
-                out.update(b.tensors(f"l{i}."))
+                out.update(b.tensors(f"l{s.index}."))
         out.update(self.norm.tensors("final.norm"))
         if self.lm_head is not None:
             out["head"] = self.lm_head
@@ -711,6 +866,9 @@ class LayeredLM(CausalLM):
         return [k for k in sd if k not in mine]
 
     def embed(self, input_ids, ctx: SeqCtx | None = None):
+        if self.embed_norm is not None:
+            n = self.embed_norm
+            return mx.embed_normed(input_ids.reshape(-1), self.embed_tokens, self.config.embed_scale, n.weight, n.eps, n.shift)
         if self.pair_embed is None:
             return mx.embed_scaled(input_ids, self.embed_tokens, self.config.embed_scale)
         if ctx is None:
@@ -727,9 +885,15 @@ class LayeredLM(CausalLM):
         ctx = dataclasses.replace(ctx, shared=dict.fromkeys(self.config.lenders))
         ids = input_ids.reshape(-1)
         x, delta, post = (self.embed(input_ids, ctx) if inputs_embeds is None else inputs_embeds.float()), None, None
+        first = x.clone() if self.config.passes > 1 else None  # the stream moves on in place
         for li, layer in enumerate(self.layers):
-            x, delta, post = layer(x, delta, post, ctx, li, ids, self.side_embed)
+            x, delta, post = layer(x, delta, post, ctx, li, ids, self.side_embed, self.entrance(li, first))
         return self.final_norm(x, delta, post)
+
+    def entrance(self, li: int, first) -> dict:
+        """What the loop adds to the stream in front of layer run ``li``; ``first``: the embedding."""
+        t = self.config.layers[li].enters
+        return {} if t is None else dict(anchor=first if t > 0 else None, bump=self.loop_step[t])
 
 
 def is_layered_dir(path: str) -> bool:
@@ -743,5 +907,7 @@ def is_layered_dir(path: str) -> bool:
 def layered_kinds(path: str) -> set:
     """Mixers and feed-forwards of a model directory whose kernels are built apart (csrc/build.py)."""
     with open(os.path.join(path, "config.json")) as fh:
-        layers = json.load(fh)["layers"]
-    return {e["type"] for e in layers} | {"moe" for e in layers if (e.get("mlp") or {}).get("kind") == "moe"}
+        d = json.load(fh)
+    layers = d["layers"]
+    kinds = {e["type"] for e in layers} | {"moe" for e in layers if (e.get("mlp") or {}).get("kind") == "moe"}
+    return kinds | (set(DESIGNS[d["architecture"]].sides) if "parallel" in kinds else set())

@@ -1,5 +1,5 @@
-"""ctypes bindings of ``csrc/mixers.cu``, ``csrc/grouped_attn.cu``, ``csrc/rglru.cu``, ``csrc/layered_moe.cu`` and of the
-tensor-core mixer kernels (inference only).
+"""ctypes bindings of ``csrc/mixers.cu``, ``csrc/grouped_attn.cu``, ``csrc/rglru.cu``, ``csrc/hgrn2.cu``, ``csrc/layered_moe.cu``
+and of the tensor-core mixer kernels (inference only).
 
 ``model dtype`` below is bf16 or fp32; accumulators, gates, states and norms are fp32 in both."""
 from __future__ import annotations
@@ -40,6 +40,16 @@ def embed_scaled(ids, emb, scale, out=None):
     return out
 
 
+def embed_normed(ids, emb, scale, w, eps, shift=0.0, out=None, copy=None):
+    """fp32 ``emb[ids] * scale`` over its rms times ``shift + w``; ``copy`` gets it too."""
+    T, (V, H) = ids.numel(), emb.shape
+    out = torch.empty(T, H, dtype=torch.float32, device=emb.device) if out is None else out
+    assert ids.dtype == torch.int64 and ids.is_contiguous() and emb.is_contiguous() and (copy is None or copy.shape == out.shape)
+    _chk(lib().trlb_embed_normed(_p(ids), _p(emb), _p(w), _p(out), _p(copy), c_int(T), c_int(H), c_int(V), c_float(scale), c_float(eps),
+                                 c_float(shift), _b(emb), _s()), "embed_normed")
+    return out
+
+
 def embed_pairs(ids, emb, scale, pairs, mul_prev, mul_cur, positions, tok_slot=None, prev=None, decode=False, out=None):
     """``emb[ids] * scale + pairs[row]`` with the row ``(previous * mul_prev + current * mul_cur) mod buckets`` of a table of
     ``buckets`` + 1 rows, the last one at position 0.  Prompts: ``prev`` (int64 by slot) gets every sequence's last token; decode:
@@ -66,16 +76,31 @@ def dynamic_tanh(x, delta, alpha, w, b, dtype, clear=False, out=None):
     return out
 
 
-def rms_residual(x, delta, post, w, eps, dtype, clear=False, out=None, shift=0.0, post_scale=None, gain=1.0):
-    """``x += delta`` or, with ``post``, ``x += delta / rms(delta) * (shift + post) * post_scale`` (in place; with ``clear`` delta is
-    zeroed); returns ``x / rms(x) * (shift + w) * gain`` in ``dtype``, or ``x`` itself without ``w``."""
+def rms_residual(x, delta, post, w, eps, dtype, clear=False, out=None, shift=0.0, post_scale=None, gain=1.0, mult=1.0, anchor=None,
+                 bump=None, w2=None, out2=None):
+    """``x += mult * delta`` or, with ``post``, ``x += mult * delta / rms(delta) * (shift + post) * post_scale``, and ``x += anchor +
+    bump`` (in place; with ``clear`` delta, of a pair the first one, is zeroed); returns ``x / rms(x) * (shift + w) * gain`` in
+    ``dtype``, or ``x`` itself without ``w``, or with ``w2`` a pair.  ``delta``: a tensor, two, or a tensor and
+    :class:`~trl_b200.ops.mixers.ExpertRows`."""
     T, H = x.shape
-    assert x.dtype == torch.float32 and x.is_contiguous() and (delta is None or (delta.dtype == torch.float32
-                                                                               and delta.is_contiguous()))
+
+    def f32(t):
+        return t is None or (t.dtype == torch.float32 and t.is_contiguous())
+
+    more = y = row = weight = None
+    if isinstance(delta, tuple):
+        delta, more = delta
+        if not isinstance(more, torch.Tensor):
+            (y, row, weight), more = more, None
+    assert x.dtype == torch.float32 and x.is_contiguous() and f32(delta) and f32(more) and f32(anchor) and f32(bump)
+    assert y is None or (y.dtype == dtype and y.is_contiguous() and row.shape == weight.shape and row.shape[0] == T and y.shape[1] == H)
     out = torch.empty(T, H, dtype=dtype, device=x.device) if out is None else out
+    if w2 is not None and out2 is None:
+        out2 = torch.empty_like(out)
     _chk(lib().trlb_rms_residual(_p(x), _p(delta), _p(post), _p(post_scale), _p(w), _p(out), c_int(T), c_int(H), c_float(eps),
-                                 c_float(shift), c_float(gain), c_int(int(clear)), _b(out), _s()), "rms_residual")
-    return out
+                                 c_float(shift), c_float(gain), c_float(mult), c_int(int(clear)), _p(more), _p(y), _p(row), _p(weight),
+                                 c_int(0 if y is None else row.shape[1]), _p(anchor), _p(bump), _p(w2), _p(out2), _b(out), _s()), "rms_residual")
+    return out if w2 is None else (out, out2)
 
 
 def clamped_glu(z, limit, alpha, shift, out=None):
@@ -148,13 +173,17 @@ def mixer_attn_tc_ok(heads, kv_heads, dim, rot, vdim) -> bool:
 
 
 def mixer_attn(q, k, v, *, heads, kv_heads, scale, ctx, rot=0, krot=None, window=None, keep=0, cap=None, sink=None,
-               gate=None, gate_logits=None, tensor_cores=True):
+               gate=None, gate_logits=None, pool=0, blocks=None, out=None, out_scale=1.0, tensor_cores=True):
     """Causal attention of packed prompts.  Rows of q: heads x (dim | rot), of k and v: kv_heads x dim / vdim, of krot: the rot
     elements that all heads' keys share (rows may be strided, their elements are dense) -> [T, heads vdim].  Keys at distance <
-    ``window`` and the first ``keep`` of the sequence; scores ``cap tanh(s / cap)``; ``exp(sink)`` in the denominator; ``gate`` (fp32 [T, heads]) or the sigmoid of
-    ``gate_logits`` ([T, heads vdim] in the model dtype) multiplies the result."""
+    ``window`` and the first ``keep`` of the sequence, or the means ``blocks`` of ``pool`` tokens before the window (see
+    :func:`pool_blocks`); scores ``cap tanh(s / cap)``; ``exp(sink)`` in the denominator; ``gate`` (fp32 [T, heads]) or the sigmoid of
+    ``gate_logits`` ([T, heads vdim] in the model dtype), and ``out_scale``, multiply the result (``out``: rows may be strided)."""
     T, dim, vdim = q.shape[0], k.shape[1] // kv_heads, v.shape[1] // kv_heads
-    out = torch.empty(T, heads * vdim, dtype=q.dtype, device=q.device)
+    out = torch.empty(T, heads * vdim, dtype=q.dtype, device=q.device) if out is None else out
+    assert out.shape == (T, heads * vdim) and out.stride(1) == 1 and out.dtype == q.dtype
+    pk, pv = blocks if pool else (None, None)
+    assert not pool or (pk.is_contiguous() and pv.is_contiguous() and pk.shape[0] == pv.shape[0] == T // pool + 1)
     assert q.shape[1] == heads * (dim + rot) and all(t.stride(1) == 1 for t in (q, k, v)) and (rot == 0 or krot.stride(1) == 1)
     mode = 1 if gate is not None else 2 if gate_logits is not None else 0
     assert mode != 1 or (gate.shape == (T, heads) and gate.dtype == torch.float32 and gate.is_contiguous())
@@ -162,8 +191,9 @@ def mixer_attn(q, k, v, *, heads, kv_heads, scale, ctx, rot=0, krot=None, window
     gate = gate_logits if mode == 2 else gate
     rows = [c for t in (q, k, v, krot) for c in (_p(t), c_longlong(0 if t is None else t.stride(0)))]
     sizes = [c_int(x) for x in (T, heads, kv_heads, dim, rot, vdim, window or 0, keep)] + [c_float(scale), c_float(cap or 0.0)]
-    tail = [_p(sink), c_int(mode), _p(gate), c_longlong(0 if gate is None else gate.stride(0)), _p(out)]
-    aligned = all(t is None or (t.data_ptr() % 16 == 0 and t.stride(0) % 8 == 0) for t in (q, k, v, krot)) and (
+    tail = [_p(sink), c_int(mode), _p(gate), c_longlong(0 if gate is None else gate.stride(0)), c_int(pool), _p(pk), _p(pv), _p(out),
+            c_longlong(out.stride(0)), c_float(out_scale)]
+    aligned = all(t is None or (t.data_ptr() % 16 == 0 and t.stride(0) % 8 == 0) for t in (q, k, v, krot, out)) and (
         mode != 2 or (gate.data_ptr() % 16 == 0 and gate.stride(0) % 8 == 0))
     if q.dtype == torch.bfloat16 and tensor_cores and aligned and scale > 0 and mixer_attn_tc_ok(heads, kv_heads, dim, rot, vdim):
         cu = ctx.cu_seqlens
@@ -178,18 +208,41 @@ def mixer_attn(q, k, v, *, heads, kv_heads, scale, ctx, rot=0, krot=None, window
 GATES = {None: 0, "head": 1, "element": 2}
 
 
-def attn_prep(y, m, positions, temp, *, q_norm=None, k_norm=None, whole_norm=False, table=None, rot=0, halves=False, values=True,
+def pool_blocks(k, v, cu, pool, seq_slot=None, pool_k=None, pool_v=None):
+    """Means of blocks of ``pool`` rows of packed keys [T, kv_heads dim] and values: ([T // pool + 1, kv_heads dim], the same of the
+    values); a sequence that starts at token a has its blocks from row ``a // pool`` on, rows of no block are zeros.  With
+    ``seq_slot`` they also go to ``pool_k``, ``pool_v`` [slots, rows, kv_heads, dim / vdim]."""
+    T = k.shape[0]
+    assert k.stride(1) == 1 and v.stride(1) == 1 and k.dtype == v.dtype and cu.dtype == torch.int32
+    pk, pv = (torch.empty(T // pool + 1, t.shape[1], dtype=t.dtype, device=t.device) for t in (k, v))
+    slots, rows = (0, 0) if pool_k is None else pool_k.shape[:2]
+    _chk(lib().trlb_pool_blocks(_p(k), c_longlong(k.stride(0)), c_int(k.shape[1]), _p(v), c_longlong(v.stride(0)), c_int(v.shape[1]), _p(cu),
+                                c_int(cu.numel() - 1), c_int(T), c_int(pool), _p(pk), _p(pv), _p(seq_slot), c_int(slots), c_int(rows),
+                                _p(pool_k), _p(pool_v), _b(k), _s()), "pool_blocks")
+    return pk, pv
+
+
+def _pools(pool, pool_k, pool_v):
+    rows = 0 if pool_k is None else pool_k.shape[1]
+    assert not pool or (pool_k.is_contiguous() and pool_v.is_contiguous() and pool_v.shape[:2] == pool_k.shape[:2])
+    return [c_int(pool), c_int(rows)]
+
+
+def attn_prep(y, m, positions, temp, *, q_norm=None, k_norm=None, unit=True, whole_norm=False, q_head=None, table=None, rot=0, halves=False, values=True,
               gates="element", tok_slot=None, q=None, k=None, g=None, head_gate=None, k_cache=None, v_cache=None, block_table=None,
-              block_size=0):
+              block_size=0, pool=0, pool_k=None, pool_v=None):
     """Rows ``y`` [q | k | v | g] of an attention mixer's input projection: normed queries (times ``temp`` by position) and keys,
     both rotated by ``table`` (their first ``rot`` elements, in pairs of neighbours or of ``halves``); keys and values to the paged
     cache; ``gates`` per head as fp32 sigmoids to ``head_gate``.  The norm is per head, with ``whole_norm`` over all heads, and times
-    the weights ``q_norm`` / ``k_norm`` if there are any.  Without ``values`` the keys as projected are the values.  Without
+    the weights ``q_norm`` / ``k_norm`` if there are any; without ``unit`` there is no norm.  ``q_head``: factors of the queries per
+    head.  With ``pool`` the token that completes a block of that many leaves the block's means in its slot's rows of ``pool_k``,
+    ``pool_v``.  Without ``values`` the keys as projected are the values.  Without
     ``q`` queries are replaced in place, keys too unless they go to ``k``; with ``q``
     (and ``g`` for gate logits per element) ``y`` is fp32 sums, and they are zeroed."""
     rows = y.shape[0]
     assert y.stride(1) == 1 and positions.dtype == torch.int32 and (q is None or y.dtype == torch.float32)
-    assert (head_gate is None) == (gates != "head") and (k is None or (k.is_contiguous() and k.dtype == m.o.dtype))
+    assert (head_gate is None) == (gates != "head") and (k is None or (k.is_contiguous() and k.dtype == (getattr(m, "dtype", None) or m.o.dtype)))
+    dt = getattr(m, "dtype", None) or m.o.dtype
     assert rot == 0 or (table.dtype == torch.float32 and table.shape[1] * 2 == rot)
     mb = 0 if block_table is None else block_table.shape[1]
     _chk(lib().trlb_attn_prep(_p(y), c_int(int(y.dtype == torch.float32)), c_longlong(y.stride(0)), c_int(rows), c_int(m.heads),
@@ -197,17 +250,21 @@ def attn_prep(y, m, positions, temp, *, q_norm=None, k_norm=None, whole_norm=Fal
                               c_int(GATES[gates]), c_float(m.eps), _p(positions), _p(tok_slot), _p(temp), _len(temp),
                               c_int(int(whole_norm)), _p(q_norm), _p(k_norm), c_int(rot), c_int(int(halves)),
                               _p(table), _len(table), _p(q), _p(k), _p(g), _p(head_gate), _p(k_cache), _p(v_cache),
-                              _p(block_table), c_int(mb), c_int(block_size), _b(m.o), _s()), "attn_prep")
+                              _p(block_table), c_int(mb), c_int(block_size), c_int(int(unit)), _p(q_head), *_pools(pool, pool_k, pool_v),
+                              _p(pool_k), _p(pool_v), c_int(int(dt == torch.bfloat16)), _s()), "attn_prep")
 
 
 def grouped_decode(q, k_cache, v_cache, m, seq_lens, block_table, block_size, out, gate=None, *, head_gate=None, window=None, keep=0,
-                   sink=None):
+                   sink=None, pool=0, pool_k=None, pool_v=None, out_scale=1.0):
     """One token per slot on the CUDA cores: any size, bf16 or fp32.  q [B, heads, dim], gate logits [B, heads vdim], factors
-    ``head_gate`` fp32 [B, heads]; ``window``, ``keep`` and ``sink`` as in :func:`mixer_attn`."""
+    ``head_gate`` fp32 [B, heads]; ``window``, ``keep``, ``sink`` and ``out_scale`` as in :func:`mixer_attn`, ``pool`` and its rows as in :func:`attn_prep`; rows
+    of ``out`` [B, heads vdim] may be strided."""
     B = q.shape[0]
+    assert out.shape == (B, m.heads * m.vdim) and out.stride(1) == 1
     _chk(lib().trlb_grouped_decode(_p(q), _p(k_cache), _p(v_cache), _p(gate), _p(head_gate), _p(sink), _p(out), c_int(B), c_int(m.heads),
                                    c_int(m.kv_heads), c_int(m.dim), c_int(m.vdim), c_int(window or 0), c_int(keep), c_float(m.scale),
                                    c_float(m.cap or 0.0), _p(seq_lens), _p(block_table), c_int(block_table.shape[1]), c_int(block_size),
+                                   *_pools(pool, pool_k, pool_v), _p(pool_k), _p(pool_v), c_longlong(out.stride(0)), c_float(out_scale),
                                    _b(q), _s()), "grouped_decode")
 
 
@@ -221,32 +278,33 @@ def grouped_decode_tc_items(B: int, m) -> int:
 
 
 def grouped_decode_tc(q, k_cache, v_cache, m, seq_lens, block_table, block_size, out, gate=None, splits=1, part_o=None, part_ml=None, *,
-                      head_gate=None, window=None, keep=0, sink=None):
+                      head_gate=None, window=None, keep=0, sink=None, pool=0, pool_k=None, pool_v=None, out_scale=1.0):
     """:func:`grouped_decode` on the tensor cores (bf16).  With ``splits`` > 1: ``part_o`` [>= B heads splits vdim] and
     ``part_ml`` [>= 2 B heads splits] fp32 scratch."""
     B = q.shape[0]
     assert q.dtype == torch.bfloat16 and q.is_contiguous() and k_cache.is_contiguous() and v_cache.is_contiguous()
-    assert k_cache.shape[1] == block_size and out.is_contiguous() and (gate is None or gate.is_contiguous())
+    assert k_cache.shape[1] == block_size and out.shape == (B, m.heads * m.vdim) and out.stride(1) == 1 and (gate is None or gate.is_contiguous())
     if splits > 1:
         assert part_o.numel() >= B * m.heads * splits * m.vdim and part_ml.numel() >= 2 * B * m.heads * splits
     _chk(lib().trlb_grouped_decode_tc(_p(q), _p(k_cache), _p(v_cache), _p(gate), _p(out), c_int(k_cache.shape[0]), c_int(B), c_int(m.heads),
                                       c_int(m.kv_heads), c_int(m.dim), c_int(m.vdim), c_int(window or 0), c_int(keep), c_float(m.scale),
                                       c_float(m.cap or 0.0), _p(sink), _p(head_gate), _p(seq_lens), _p(block_table),
                                       c_int(block_table.shape[1]), c_int(block_size), c_int(splits), _p(part_o), _p(part_ml),
-                                      _p(status_buffer(q.device)), _s()), "grouped_decode_tc")
+                                      *_pools(pool, pool_k, pool_v), c_int(0 if pool_k is None else pool_k.shape[0]), _p(pool_k), _p(pool_v),
+                                      c_longlong(out.stride(0)), c_float(out_scale), _p(status_buffer(q.device)), _s()), "grouped_decode_tc")
 
 
-def moe_route(z, correction, top, *, positions=None, renormalize=False, clear=False):
+def moe_route(z, correction, top, *, positions=None, scores="sigmoid", renormalize=False, gain=1.0, clear=False):
     """fp32 logits z [T, E] (zeroed with ``clear``) -> (choice, rank, weight) [T, top] and counts [E]: the experts of the largest
-    sigmoid score + correction, their place among the expert's tokens, their bare scores (over their sum with ``renormalize``).
-    Rows of negative position choose nothing (-1)."""
+    score (sigmoid or softmax) + correction, their place among the expert's tokens, their bare scores (over their sum with
+    ``renormalize``) times ``gain``.  Rows of negative position choose nothing (-1)."""
     T, E = z.shape
     assert z.dtype == torch.float32 and z.is_contiguous() and (correction is None or correction.dtype == torch.float32)
     i32 = dict(dtype=torch.int32, device=z.device)
     choice, rank, weight = torch.empty(T, top, **i32), torch.empty(T, top, **i32), torch.empty(T, top, dtype=torch.float32, device=z.device)
     counts = torch.empty(E, **i32) if T <= 128 else torch.zeros(E, **i32)
     _chk(lib().trlb_moe_route(_p(z), _p(correction), _p(positions), c_int(T), c_int(E), c_int(top), c_int(int(renormalize)),
-                              c_int(int(clear)), _p(choice), _p(rank), _p(weight), _p(counts), _s()), "moe_route")
+                              c_int({"sigmoid": 0, "softmax": 1}[scores]), c_float(gain), c_int(int(clear)), _p(choice), _p(rank), _p(weight), _p(counts), _s()), "moe_route")
     return choice, rank, weight, counts
 
 
@@ -278,6 +336,41 @@ def moe_rows_gemm(a, w, offsets):
     _chk(lib().trlb_moe_rows_gemm(_p(a), _p(w), _p(offsets), _p(out), c_longlong(a.shape[0]), c_int(w.shape[0]), c_int(w.shape[1]),
                                   c_int(w.shape[2]), _b(a), _s()), "moe_rows_gemm")
     return out
+
+
+def hgrn2_prompt(y, z, m, cu, seq_slot=None, state=None):
+    """The recurrence over packed prompts, token by token: rows y [q | v] in the model dtype, z fp32 gate logits without bias ->
+    fp32 [T, heads, vdim]; ``state`` [slots, heads, dim, vdim] of ``seq_slot`` gets the final one."""
+    T, qd = y.shape[0], m.heads * m.dim
+    assert y.stride(1) == 1 and z.stride(1) == 1 and z.dtype == torch.float32 and cu.dtype == torch.int32
+    out = torch.empty(T, m.heads, m.vdim, dtype=torch.float32, device=y.device)
+    _chk(lib().trlb_hgrn2_prompt(_p(y), c_longlong(y.stride(0)), c_int(qd), _p(z), c_longlong(z.stride(0)), _p(m.f_bias), _p(m.lower), _p(cu),
+                                 c_int(cu.numel() - 1), _p(seq_slot if state is not None else None), _p(state),
+                                 c_int(0 if state is None else state.shape[0]), c_int(m.heads), c_int(m.dim), c_int(m.vdim), _p(out), _b(y),
+                                 _s()), "hgrn2_prompt")
+    return out
+
+
+def head_norm(o, w, eps, dtype, out=None, scale=1.0):
+    """o fp32 [T, heads, vdim] over its rms per head times ``w`` [vdim] and ``scale`` -> [T, heads vdim] (rows of ``out`` may be
+    strided)."""
+    T, H, E = o.shape
+    out = torch.empty(T, H * E, dtype=dtype, device=o.device) if out is None else out
+    assert o.is_contiguous() and o.dtype == torch.float32 and out.shape == (T, H * E) and out.stride(1) == 1 and out.dtype == dtype
+    _chk(lib().trlb_head_norm(_p(o), _p(w), c_float(eps), c_int(T), c_int(H), c_int(E), c_float(scale), _p(out), c_longlong(out.stride(0)),
+                              _b(out), _s()), "head_norm")
+    return out
+
+
+def hgrn2_step(sums, m, seq_lens, state, out, scale=1.0):
+    """One token per slot: fp32 sums [B, q | v | z] (zeroed), state [slots, heads, dim, vdim] moves on; out [B, heads vdim] (rows
+    may be strided) = outputs over their rms per head times the norm's weight and ``scale``."""
+    B = sums.shape[0]
+    assert sums.dtype == torch.float32 and sums.stride(1) == 1 and state.is_contiguous() and state.shape[0] >= B
+    assert out.shape == (B, m.heads * m.vdim) and out.stride(1) == 1 and sums.shape[1] >= m.heads * (2 * m.dim + m.vdim)
+    _chk(lib().trlb_hgrn2_step(_p(sums), c_longlong(sums.stride(0)), _p(m.f_bias), _p(m.lower), _p(m.norm), c_float(m.eps), c_float(scale),
+                               _p(seq_lens), c_int(B), _p(state), c_int(m.heads), c_int(m.dim), c_int(m.vdim), _p(out),
+                               c_longlong(out.stride(0)), _b(out), _s()), "hgrn2_step")
 
 
 def conv_prompt(x, m, ctx, seq_slot=None, conv_state=None):

@@ -10,6 +10,7 @@ from __future__ import annotations
 
 import contextlib
 import math
+from typing import NamedTuple
 
 import torch
 import torch.nn.functional as F
@@ -24,8 +25,9 @@ def _k():
 
 
 class RotarySpec:
-    """Rotary positions with optional YaRN scaling.  ``table(n)``: fp32 [n, dims / 2, 2] (cos, sin), the
-    magnitude of the scaling folded in; angles are evaluated in fp64 before they are rounded."""
+    """Rotary positions with optional frequency scaling: YaRN's (``fast``, ``slow``) or Llama 3's (``low``, ``high``).
+    ``table(n)``: fp32 [n, dims / 2, 2] (cos, sin), the magnitude of the scaling folded in; angles are evaluated in fp64 before
+    they are rounded."""
 
     def __init__(self, dims: int, base: float, scaling: dict | None = None):
         self.dims, self.base, self.scaling = dims, base, dict(scaling) if scaling else None
@@ -37,6 +39,11 @@ class RotarySpec:
         if self.scaling is None:
             return f
         s = self.scaling
+        if "low" in s:
+            turns = s["original"] * f / (2.0 * math.pi)  # of a pair in the original context
+            keep = ((turns - s["low"]) / max(s["high"] - s["low"], 1e-9)).clamp(0.0, 1.0)
+            keep = torch.where(turns < s["low"], 0.0, torch.where(turns > s["high"], 1.0, keep))
+            return (1.0 - keep) * f / s["factor"] + keep * f
 
         def turns_to_dim(t):
             return self.dims * math.log(s["original"] / (2.0 * math.pi * t)) / (2.0 * math.log(self.base))
@@ -48,7 +55,7 @@ class RotarySpec:
 
     @property
     def magnitude(self) -> float:
-        return 1.0 if self.scaling is None else 0.1 * math.log(self.scaling["factor"]) + 1.0
+        return 1.0 if self.scaling is None or "low" in self.scaling else 0.1 * math.log(self.scaling["factor"]) + 1.0
 
     def table(self, n: int, device) -> torch.Tensor:
         key = str(device)
@@ -125,6 +132,13 @@ def embed_pairs(ids, emb, scale, pairs, spec, positions, where):
     return F.embedding(ids, emb).float() * scale + F.embedding(rows, pairs).float()
 
 
+def embed_normed(ids, emb, scale, w, eps, shift=0.0):
+    """fp32 embeddings times ``scale``, over their rms times ``shift + w``."""
+    if emb.is_cuda:
+        return _k().embed_normed(ids, emb, scale, w, eps, shift)
+    return _ref.unit_rms(F.embedding(ids, emb).float() * scale, eps) * (shift + w)
+
+
 def dynamic_tanh(x, delta, alpha, w, b, out_dtype, clear=False, out=None):
     """(norm of ``x + delta`` in ``out_dtype``, ``x + delta``); on CUDA the sum is formed in place."""
     if x.is_cuda:
@@ -135,12 +149,24 @@ def dynamic_tanh(x, delta, alpha, w, b, out_dtype, clear=False, out=None):
 
 def rms_residual(x, delta, post, w, eps, out_dtype, clear=False, out=None, **kw):
     """(``s / rms(s) * w`` in ``out_dtype``, s) of ``s = x + delta``, where delta over its rms times ``post`` is added when
-    ``post`` is given and s itself is the output when ``w`` is None; on CUDA the sum is formed in place.  ``shift`` is added to both
-    weights, ``post_scale`` multiplies ``post``, ``gain`` the output."""
+    ``post`` is given and s itself is the output when ``w`` is None; on CUDA the sum is formed in place.  ``shift`` is added to the
+    weights, ``post_scale`` multiplies ``post``, ``gain`` the output.  ``mult`` multiplies delta, which may be a pair (of tensors, or a
+    tensor and :class:`ExpertRows`) to be added up; ``anchor`` [T, H] and ``bump`` [H] are added as well; with a second weight
+    ``w2`` (and ``out2``) the output is a pair."""
     if x.is_cuda:
         return _k().rms_residual(x, delta, post, w, eps, out_dtype, clear=clear, out=out, **kw), x
+    kw.pop("out2", None)
     y, x = _ref.rms_residual(x, delta, post, w, eps, **kw)
-    return y.to(out_dtype), x
+    return (tuple(t.to(out_dtype) for t in y) if isinstance(y, tuple) else y.to(out_dtype)), x
+
+
+class ExpertRows(NamedTuple):
+    """What a mixture of experts gives before it is added up: token t's output is the sum over its choices c of
+    ``weight[t, c] * y[row[t, c]]`` (a negative row: nothing)."""
+
+    y: torch.Tensor
+    row: torch.Tensor
+    weight: torch.Tensor
 
 
 def clamped_glu(z, limit, alpha, shift, out=None):
@@ -155,15 +181,16 @@ def gelu_erf(z, out=None):
     return _k().gelu_erf(z, out=out) if z.is_cuda else F.gelu(z)
 
 
-def experts(m, h, positions=None, logits=None, out=None):
-    """Mixture of experts: h [T, width] -> fp32 [T, width].  ``positions``: rows where they are negative choose nothing;
-    ``logits``: fp32 sums of the router's product (zeroed), formed here when absent."""
+def experts(m, h, positions=None, logits=None, out=None, summed=True):
+    """Mixture of experts: h [T, width] -> fp32 [T, width], or on CUDA without ``summed`` :class:`ExpertRows` for the kernel that
+    adds them to the stream.  ``positions``: rows where they are negative choose nothing; ``logits``: fp32 sums of the router's
+    product (zeroed), formed here when absent."""
     if not h.is_cuda:
         return _ref.experts(m, h.float())
     K = _k()
     z = linear_f32(h, m.router) if logits is None else logits
-    choice, rank, weight, counts = K.moe_route(z, m.correction, m.top, positions=positions, renormalize=m.renormalize,
-                                               clear=logits is not None)
+    choice, rank, weight, counts = K.moe_route(z, m.correction, m.top, positions=positions, clear=logits is not None,
+                                               **m.routing)
     x, row, offsets = K.moe_gather(h, choice, rank, counts)
     if h.dtype == torch.bfloat16 and h.shape[1] % 8 == 0 and m.ff % 8 == 0:
         from . import cuda as KC
@@ -172,7 +199,7 @@ def experts(m, h, positions=None, logits=None, out=None):
         y = KC.grouped_gemm(act, m.down, offsets, h.shape[1])
     else:
         y = K.moe_rows_gemm(K.clamped_glu(K.moe_rows_gemm(x, m.gate_up, offsets), *m.glu), m.down, offsets)
-    return K.moe_sum(y, row, weight, out=out)
+    return K.moe_sum(y, row, weight, out=out) if summed else ExpertRows(y, row, weight)
 
 
 def side_input(h, ids, table, off, gate, proj):
@@ -219,25 +246,65 @@ def attention(m, h, ctx, li):
     if not h.is_cuda:
         out, kept = _ref.attention(m, h.float(), ctx.positions, ctx.cu_seqlens, kept)
     else:
-        K = _k()
-        T, own = h.shape[0], kept is None
-        pos = ctx.positions if ctx.positions.dtype == torch.int32 else ctx.positions.to(torch.int32)
-        temp = m.temperature.table(ctx.max_seqlen, h.device) if m.temperature is not None else None
-        table = m.rope.table(ctx.max_seqlen, h.device) if m.rot else None
-        y = linear(h, m.w_in)
-        q, k, v, g = y[:, : sum(m.parts)].split(m.parts, 1)
-        # projected keys that are also the values stay as they are
-        keys = torch.empty(T, m.kv_heads * m.dim, dtype=h.dtype, device=h.device) if own and not m.values else None
-        gate = torch.empty(T, m.heads, dtype=torch.float32, device=h.device) if m.gate == "head" else None
-        K.attn_prep(y, m, pos, temp, table=table, k=keys, head_gate=gate, **m.prep, **(ctx.kv.paged_cache(li) if ctx.kv is not None else {}))
-        if own:
-            kept = (k, v) if keys is None else (keys, k)
-        o = K.mixer_attn(q, *kept, heads=m.heads, kv_heads=m.kv_heads, scale=m.scale, cap=m.cap, **m.sight, gate=gate,
-                         gate_logits=g if m.gate == "element" else None, ctx=ctx)
+        o, kept = attention_rows(m, linear(h, m.w_in), ctx, ctx.kv.paged_cache(li) if ctx.kv is not None else {}, kept)
         out = linear_f32(o, m.o)
     if li in ctx.shared:
         ctx.shared[li] = kept
     return out
+
+
+def attention_rows(m, y, ctx, where, kept=None, out=None, scale=1.0):
+    """From the rows ``y`` of the input projection (replaced in part) to what the output projection reads, times ``scale``, and the
+    keys and values.  ``where`` (may be empty): the pages and slots that get them; ``kept``: those of the layer it borrows from."""
+    K = _k()
+    T, own, where = y.shape[0], kept is None, dict(where)
+    pos = ctx.positions if ctx.positions.dtype == torch.int32 else ctx.positions.to(torch.int32)
+    temp = m.temperature.table(ctx.max_seqlen, y.device) if m.temperature is not None else None
+    table = m.rope.table(ctx.max_seqlen, y.device) if m.rot else None
+    pools = where.pop("pools", {})
+    q, k, v, g = y[:, : m.rows].split(m.parts, 1)
+    # projected keys that are also the values stay as they are
+    keys = torch.empty(T, m.kv_heads * m.dim, dtype=y.dtype, device=y.device) if own and not m.values else None
+    gate = torch.empty(T, m.heads, dtype=torch.float32, device=y.device) if m.gate == "head" else None
+    K.attn_prep(y, m, pos, temp, table=table, k=keys, head_gate=gate, **m.prep, **where)
+    if own:
+        kept = (k, v) if keys is None else (keys, k)
+    blocks = K.pool_blocks(*kept, ctx.cu_seqlens, m.pool, **pools) if m.pool else None
+    o = K.mixer_attn(q, *kept, heads=m.heads, kv_heads=m.kv_heads, scale=m.scale, cap=m.cap, **m.sight, gate=gate, pool=m.pool, blocks=blocks,
+                     gate_logits=g if m.gate == "element" else None, ctx=ctx, out=out, out_scale=scale)
+    return o, kept
+
+
+def hgrn2(m, h, ctx, li):
+    if not h.is_cuda:
+        return _ref.hgrn2(m, h.float(), ctx.cu_seqlens)
+    where = ctx.kv.recurrent_state(li) if ctx.kv is not None else {}
+    return linear_f32(hgrn2_rows(m, linear(h, m.w_in[: m.rows]), linear_f32(h, m.w_in[m.rows:]), ctx, where), m.o)
+
+
+def hgrn2_rows(m, y, z, ctx, where, out=None, scale=1.0):
+    """From the rows ``y`` (query | value) and ``z`` (forget gate, fp32 sums) of the input projection to what the output projection
+    reads, times ``scale``.  ``where`` (may be empty): the slots that get the final states."""
+    K = _k()
+    return K.head_norm(hgrn2_prompt_scan(m, y, z, ctx, where), m.norm, m.eps, y.dtype, out=out, scale=scale)
+
+
+def hgrn2_prompt_scan(m, y, z, ctx, where, tensor_cores=True):
+    """The recurrence over packed prompts -> fp32 [T, heads, vdim]."""
+    K = _k()
+    return K.hgrn2_prompt(y, z, m, ctx.cu_seqlens, **where)
+
+
+def parallel(m, h, ctx, li):
+    if not h.is_cuda:
+        return _ref.parallel(m, h.float(), ctx.positions, ctx.cu_seqlens)
+    a, b = m.left.rows, m.left.out_width
+    where = ctx.kv.paged_cache(li) if ctx.kv is not None else dict(left={}, right={})
+    y, z = linear(h, m.w_in[: m.rows]), linear_f32(h, m.w_in[m.rows:])
+    o = torch.empty(h.shape[0], m.o.shape[1], dtype=h.dtype, device=h.device)
+    attention_rows(m.left, y[:, :a], ctx, where["left"], out=o[:, :b], scale=m.scales[0])
+    hgrn2_rows(m.right, y[:, a:], z, ctx, where["right"], out=o[:, b:], scale=m.scales[1])
+    return linear_f32(o, m.o)
 
 
 def block_gates(u, gates):

@@ -14,15 +14,23 @@ def unit_rms(x, eps):
     return x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps)
 
 
-def rms_residual(x, delta, post, w, eps, shift=0.0, post_scale=None, gain=1.0):
-    """(``x + delta`` (delta over its rms times ``(shift + post) post_scale``, when given)) over its rms times ``(shift + w) gain``
-    (when given), and the sum."""
+def rms_residual(x, delta, post, w, eps, shift=0.0, post_scale=None, gain=1.0, mult=1.0, anchor=None, bump=None, w2=None):
+    """(``x + mult delta`` (delta over its rms times ``(shift + post) post_scale``, when given) ``+ anchor + bump`` (when given)) over
+    its rms times ``(shift + w) gain`` (when given), with ``w2`` also times ``(shift + w2) gain``, and the sum.  A pair of deltas is
+    their sum."""
     if delta is not None:
+        if isinstance(delta, tuple):
+            delta = delta[0] + delta[1]
         if post is not None:
             delta = unit_rms(delta, eps) * (shift + post)
             delta = delta if post_scale is None else delta * post_scale
-        x = x + delta
-    return (x if w is None else unit_rms(x, eps) * ((shift + w) * gain)), x
+        x = x + mult * delta
+    for more in (anchor, bump):
+        x = x if more is None else x + more
+    y = x if w is None else unit_rms(x, eps)
+    if w2 is not None:
+        return (y * ((shift + w) * gain), y * ((shift + w2) * gain)), x
+    return (y if w is None else y * ((shift + w) * gain)), x
 
 
 def pair_rows(ids, positions, mul_prev, mul_cur, buckets):
@@ -59,25 +67,31 @@ def rotate_pairs(x, cos, sin):
     return torch.stack([u * c - v * s, v * c + u * s], -1).flatten(-2)
 
 
-def sink_window_attention(q, k, v, scale, window, sink, cu, cap=None, keep=0):
+def sink_window_attention(q, k, v, scale, window, sink, cu, cap=None, keep=0, pool=0):
     """q [T, H, D], k [T, G, D], v [T, G, E] (H / G query heads read one key head), packed sequences by ``cu``; scores
     ``cap tanh(s / cap)``; softmax with ``exp(sink)`` added to the denominator (no such term without a sink); with a window the first
-    ``keep`` keys of a sequence stay visible."""
+    ``keep`` keys of a sequence stay visible, or the means of the blocks of ``pool`` tokens that lie before it."""
     outs, per = [], q.shape[1] // k.shape[1]
     if per > 1:
         k, v = k.repeat_interleave(per, 1), v.repeat_interleave(per, 1)
     for a, b in zip(cu[:-1].tolist(), cu[1:].tolist()):
-        n = b - a
-        s = torch.einsum("qhd,khd->hqk", q[a:b], k[a:b]) * scale
+        n, blocks, ks, vs = b - a, 0, k[a:b], v[a:b]
+        if pool and window is not None:
+            blocks = n // pool
+            ks, vs = (torch.cat([x, x[:blocks * pool].reshape(blocks, pool, *x.shape[1:]).mean(1)]) for x in (ks, vs))
+        s = torch.einsum("qhd,khd->hqk", q[a:b], ks) * scale
         if cap is not None:
             s = cap * torch.tanh(s / cap)
         i = torch.arange(n, device=s.device)
         gap = i[:, None] - i[None, :]
         seen = (gap >= 0) if window is None else (gap >= 0) & ((gap < window) | (i < keep))
+        if blocks:
+            ends = torch.arange(blocks, device=s.device) * pool + pool - 1
+            seen = torch.cat([seen, ends[None, :] <= i[:, None] - window], 1)
         s = s.masked_fill(~seen, float("-inf"))
         if sink is not None:
             s = torch.cat([s, sink.to(s.dtype)[:, None, None].expand(-1, n, 1)], -1)
-        outs.append(torch.einsum("hqk,khe->qhe", torch.softmax(s, -1)[..., :n], v[a:b]))
+        outs.append(torch.einsum("hqk,khe->qhe", torch.softmax(s, -1)[..., :n + blocks], vs))
     return torch.cat(outs)
 
 
@@ -122,13 +136,20 @@ def latent_attention(m, h, positions, cu):
 def attention(m, h, positions, cu, kept=None):
     """``m``: a models.layered.GroupedAttention; ``kept``: keys and values of the layer it borrows from.  Returns ([T, width],
     (keys, values))."""
+    o, kept = attention_rows(m, F.linear(h, m.w_in.to(h.dtype))[:, : m.rows], positions, cu, kept)
+    return F.linear(o, m.o.to(h.dtype)), kept
+
+
+def attention_rows(m, h, positions, cu, kept=None):
+    """Rows ``h`` of the input projection -> ([T, heads vdim], (keys, values))."""
     T, H, G = h.shape[0], m.heads, m.kv_heads
-    q, k, v, g = F.linear(h, m.w_in.to(h.dtype))[:, : sum(m.parts)].split(m.parts, -1)
+    q, k, v, g = h.split(m.parts, -1)
 
     def turned(x, n, w):
         """Norm (of all heads at once, or per head), weight, rotation."""
-        x = unit_rms(x if m.whole_norm else x.view(T, n, m.dim), m.eps)
-        x = (x if w is None else x * w.to(h.dtype)).view(T, n, m.dim)
+        if m.unit:
+            x = unit_rms(x if m.whole_norm else x.reshape(T, n, m.dim), m.eps)
+        x = (x if w is None else x * w.to(h.dtype)).reshape(T, n, m.dim)
         if not m.rot:
             return x
         table = m.rope.table(int(positions.max()) + 1 if T else 1, h.device).to(h.dtype)[positions.long()]
@@ -138,26 +159,28 @@ def attention(m, h, positions, cu, kept=None):
     q = turned(q, H, m.q_norm)
     if m.temperature is not None:
         q = q * m.temperature.table(int(positions.max()) + 1 if T else 1, h.device).to(h.dtype)[positions.long()][:, None, None]
+    if m.temp is not None:
+        q = q * m.temp.to(h.dtype)[:, None]
     if kept is None:
         kept = turned(k, G, m.k_norm), (v if m.values else k).reshape(T, G, m.vdim)
-    o = sink_window_attention(q, *kept, m.scale, m.window, m.sink, cu, m.cap, m.keep)
+    o = sink_window_attention(q, *kept, m.scale, m.window, m.sink, cu, m.cap, m.keep, m.pool)
     if m.gate == "head":
         o = o * torch.sigmoid(g)[..., None]
     o = o.reshape(T, H * m.vdim)
-    return F.linear(o * torch.sigmoid(g) if m.gate == "element" else o, m.o.to(h.dtype)), kept
+    return (o * torch.sigmoid(g) if m.gate == "element" else o), kept
 
 
-def route(z, correction, top, renormalize=False):
+def route(z, correction, top, renormalize=False, scores="sigmoid", gain=1.0):
     """Logits [T, E] -> (experts [T, top], weights [T, top])."""
-    s = torch.sigmoid(z)
-    idx = (s.detach() + correction.to(z.dtype)).topk(top, -1).indices
+    s = torch.softmax(z, -1) if scores == "softmax" else torch.sigmoid(z)
+    idx = (s.detach() if correction is None else s.detach() + correction.to(z.dtype)).topk(top, -1).indices
     w = s.gather(1, idx)
-    return idx, (w / w.sum(-1, keepdim=True) if renormalize else w)
+    return idx, (w / (w.sum(-1, keepdim=True) + 1e-20) if renormalize else w) * gain
 
 
 def experts(m, h):
     """``m``: a models.layered.ExpertMlp; h [T, width] -> [T, width]."""
-    idx, w = route(F.linear(h, m.router.to(h.dtype)), m.correction, m.top, m.renormalize)
+    idx, w = route(F.linear(h, m.router.to(h.dtype)), m.correction, m.top, **m.routing)
     out = torch.zeros_like(h)
     for e in range(m.n):
         t, j = (idx == e).nonzero(as_tuple=True)
@@ -213,3 +236,37 @@ def mlstm(m, h, cu):
                        F.logsigmoid(z[:, H:]), cu)
     o = unit_rms(o, m.eps).reshape(T, vd) * m.norm.to(h.dtype) * torch.sigmoid(g)
     return F.linear(o, m.o.to(h.dtype))
+
+
+def hgrn2_scan(q, f, v, cu):
+    """q, f [T, H, D], v [T, H, E] -> [T, H, E]: ``S = diag(f) S + (1 - f) v^T``, ``o = S^T q``."""
+    outs = []
+    for a, b in zip(cu[:-1].tolist(), cu[1:].tolist()):
+        S = torch.zeros(q.shape[1], q.shape[2], v.shape[2], dtype=v.dtype, device=v.device)
+        for t in range(a, b):
+            S = f[t][..., None] * S + (1 - f[t])[..., None] * v[t][:, None]
+            outs.append(torch.einsum("hd,hde->he", q[t], S))
+    return torch.stack(outs)
+
+
+def hgrn2_rows(m, h, cu):
+    """``m``: a models.layered.HGrn2; rows ``h`` of its input projection -> [T, heads vdim]."""
+    T, H = h.shape[0], m.heads
+    q, v, z = h.split(m.parts, -1)
+    low = m.lower.to(h.dtype)
+    f = low + (1 - low) * torch.sigmoid(z + m.f_bias.to(h.dtype))
+    o = hgrn2_scan(F.silu(q).reshape(T, H, m.dim), f.view(T, H, m.dim), v.reshape(T, H, m.vdim), cu)
+    return (unit_rms(o, m.eps) * m.norm.to(h.dtype)).reshape(T, H * m.vdim)
+
+
+def hgrn2(m, h, cu):
+    return F.linear(hgrn2_rows(m, F.linear(h, m.w_in.to(h.dtype)), cu), m.o.to(h.dtype))
+
+
+def parallel(m, h, positions, cu):
+    """``m``: a models.layered.ParallelMixers."""
+    y, a, outs = F.linear(h, m.w_in.to(h.dtype)), m.left.rows, []
+    for side, rows, scale in ((m.left, y[:, :a], m.scales[0]), (m.right, y[:, a:], m.scales[1])):
+        o = attention_rows(side, rows, positions, cu)[0] if side.kind.startswith("attention") else hgrn2_rows(side, rows, cu)
+        outs.append(o * scale)
+    return F.linear(torch.cat(outs, -1), m.o.to(h.dtype))

@@ -2,20 +2,22 @@
 :class:`~trl_b200.rollout.engine.RolloutEngine`'s; this module adds what a layer keeps between tokens and how it takes
 one token further.
 
-Every layer of the list has a cache of its own, also one that runs with another layer's weights (a layer with ``kv_from``
+Every layer run has a cache of its own, also one that runs with another one's weights and every pass of a loop (a layer with ``kv_from``
 reads that layer's instead):
 
     latent_attention   pages of latent rows ``[kv_rank | rotated key]`` behind the engine's block table (the window is a
                        mask: pages stay until the sequence ends)
     attention          pages of keys (normed, rotated) and pages of values (the projected keys where those serve as values);
-                       a window is a mask here too
+                       a window is a mask here too.  With pooled blocks also, per slot, rows of the means of the complete ones
     mlstm              per slot an fp32 matrix state, its normaliser and running maximum
     rglru              per slot an fp32 state vector and the last inputs of the convolution
+    hgrn2              per slot an fp32 matrix state
+    parallel           what its two halves keep
 
 An embedding of token pairs keeps the last token per slot.
 
 A decode step is one graph: embed, then per layer norm (+ residual) -> input projection -> mixer -> output projection
--> norm (+ residual) -> up / activation -> down, or router -> choice -> gather -> experts -> sum (-> stream -> side gate -> side projection), then final norm, head and
+-> norm (+ residual) -> up / activation -> down (mixer and feed-forward side by side: one norm kernel in front of both), or router -> choice -> gather -> experts -> sum (-> stream -> side gate -> side projection), then final norm, head and
 sampler.  Norms on a sublayer's output ride on the norm kernel that follows.  With bf16 weights the projections are the
 weight-streaming tcgen05 kernel; their fp32 sums are consumed and cleared by the next kernel.  fp32 models run the same
 kernels' fp32 forms with library fp32 matrix products."""
@@ -156,7 +158,9 @@ class _MLstmSlots:
 class _AttentionSlots:
     """Decode side of one ``attention`` or ``attention_2`` layer."""
 
-    def __init__(self, eng: "LayeredRolloutEngine", m, li):
+    def __init__(self, eng: "LayeredRolloutEngine", m, li, acc=None, out=None, scale: float = 1.0):
+        """A part of another mixer is given its columns ``acc`` of the input projection's sums, those of the output projection's
+        operand (``out``) and the factor ``scale`` of its output."""
         from ..ops import cuda_mixers as K
 
         self.e, self.m = eng, m
@@ -170,13 +174,18 @@ class _AttentionSlots:
             self.k_cache, self.v_cache = lender.k_cache, lender.v_cache
         self.temp = m.temperature.table(eng.max_len + 1, eng.dev) if m.temperature is not None else None
         B = eng.max_seqs
-        self.w_in = m.w_in[: sum(m.parts)]
-        self.acc_in = eng.sums("in", sum(m.parts))
+        self.w_in = m.w_in[: m.rows] if acc is None else None
+        self.acc_in = eng.sums("in", m.rows) if acc is None else acc
+        self.pools, self.scale = {}, scale
+        if m.pool:
+            shape = (B, eng.max_len // m.pool + 1, m.kv_heads)
+            self.pools = dict(pool_k=torch.zeros(*shape, m.dim, dtype=eng.dtype, device=eng.dev),
+                              pool_v=torch.zeros(*shape, m.vdim, dtype=eng.dtype, device=eng.dev))
         self.q = eng.scratch("q", B, m.heads, m.dim)
         self.table = m.rope.table(eng.max_len + 1, eng.dev) if m.rot else None
         self.g = eng.scratch("g", B, m.heads * m.vdim) if m.gate == "element" else None
         self.head_gate = eng.scratch("gate", B, m.heads, dtype=torch.float32) if m.gate == "head" else None
-        self.o = eng.scratch("o", B, m.heads * m.vdim)
+        self.o = eng.scratch("o", B, m.heads * m.vdim) if out is None else out
         # tensor-core decode; other sizes and fp32 run the CUDA-core kernel
         self.tc = eng.dtype == torch.bfloat16 and K.grouped_decode_tc_ok(m, eng.block_size)
         self.splits, self.part_o, self.part_ml = 1, None, None
@@ -184,6 +193,7 @@ class _AttentionSlots:
             tiles = -(-eng.max_len // 128)
             if m.window:
                 tiles = min(tiles, -(-m.window // 128) + 1 + -(-m.keep // 128))
+                tiles += -(-max(0, eng.max_len - m.window) // (128 * m.pool)) if m.pool else 0
             self.splits = max(1, min(8, tiles, 148 // K.grouped_decode_tc_items(B, m)))
             if self.splits > 1:
                 self.part_o = eng.scratch("part_o", B, m.heads * self.splits * m.vdim, dtype=torch.float32)
@@ -192,22 +202,25 @@ class _AttentionSlots:
     def prompt_target(self, pages: "_Pages") -> dict:
         if not self.own:
             return {}
+        pools = dict(pools=dict(seq_slot=pages.slots, **self.pools)) if self.pools else {}
         return dict(k_cache=self.k_cache, v_cache=self.v_cache, tok_slot=pages.tok_slot, block_table=self.e.block_table,
-                    block_size=self.e.block_size)
+                    block_size=self.e.block_size, **pools)
 
     def copy_pages(self, dst, src):
         for c in (self.k_cache, self.v_cache) if self.own else ():
             c.index_copy_(0, dst, c.index_select(0, src))
 
     def copy_slots(self, dst, src):
-        pass
+        for c in self.pools.values():
+            c.index_copy_(0, dst, c.index_select(0, src))
 
     def prepare(self):
         """``acc_in`` -> queries, gate logits, the new rows of the cache."""
         from ..ops import cuda_mixers as K
 
         e = self.e
-        where = dict(k_cache=self.k_cache, v_cache=self.v_cache, block_table=e.block_table, block_size=e.block_size) if self.own else {}
+        where = dict(k_cache=self.k_cache, v_cache=self.v_cache, block_table=e.block_table, block_size=e.block_size, pool=self.m.pool,
+                     **self.pools) if self.own else {}
         K.attn_prep(self.acc_in, self.m, e.seq_lens, self.temp, table=self.table, q=self.q, g=self.g, head_gate=self.head_gate,
                     **self.m.prep, **where)
 
@@ -216,15 +229,20 @@ class _AttentionSlots:
 
         e = self.e
         args = (self.q, self.k_cache, self.v_cache, self.m, e.seq_lens, e.block_table, e.block_size, self.o, self.g)
+        how = dict(head_gate=self.head_gate, pool=self.m.pool, out_scale=self.scale, **self.pools, **self.m.sight)
         if self.tc:
-            K.grouped_decode_tc(*args, self.splits, self.part_o, self.part_ml, head_gate=self.head_gate, **self.m.sight)
+            K.grouped_decode_tc(*args, self.splits, self.part_o, self.part_ml, **how)
         else:
-            K.grouped_decode(*args, head_gate=self.head_gate, **self.m.sight)
+            K.grouped_decode(*args, **how)
+
+    def mix(self):
+        """Sums of the input projection -> operand of the output projection."""
+        self.prepare()
+        self.attend()
 
     def step(self, h, out):
         self.e.gemm(h, self.w_in, self.acc_in)
-        self.prepare()
-        self.attend()
+        self.mix()
         self.e.gemm(self.o, self.m.o, out)
 
 
@@ -274,7 +292,67 @@ class _RgLruSlots:
         self.e.gemm(self.y, self.m.o, out)
 
 
-SLOTS = {"latent_attention": _LatentSlots, "mlstm": _MLstmSlots, "attention": _AttentionSlots, "attention_2": _AttentionSlots, "rglru": _RgLruSlots}
+class _HGrn2Slots:
+    """Decode side of one ``hgrn2`` layer."""
+
+    def __init__(self, eng: "LayeredRolloutEngine", m, li, acc=None, out=None, scale: float = 1.0):
+        """As :class:`_AttentionSlots`."""
+        self.e, self.m, self.scale = eng, m, scale
+        self.state = torch.zeros(eng.max_seqs, m.heads, m.dim, m.vdim, dtype=torch.float32, device=eng.dev)
+        self.acc_in = eng.sums("in", sum(m.parts)) if acc is None else acc
+        self.y = eng.scratch("o", eng.max_seqs, m.out_width) if out is None else out
+
+    def prompt_target(self, pages: "_Pages") -> dict:
+        return dict(seq_slot=pages.slots, state=self.state)
+
+    def copy_pages(self, dst, src):
+        pass
+
+    def copy_slots(self, dst, src):
+        self.state.index_copy_(0, dst, self.state.index_select(0, src))
+
+    def mix(self):
+        from ..ops import cuda_mixers as K
+
+        K.hgrn2_step(self.acc_in, self.m, self.e.seq_lens, self.state, self.y, self.scale)
+
+    def step(self, h, out):
+        self.e.gemm(h, self.m.w_in, self.acc_in)
+        self.mix()
+        self.e.gemm(self.y, self.m.o, out)
+
+
+class _ParallelSlots:
+    """Decode side of one ``parallel`` layer: one product in front of both halves, one behind them."""
+
+    def __init__(self, eng: "LayeredRolloutEngine", m, li):
+        self.e, self.m = eng, m
+        a, b = m.left.rows, m.left.out_width
+        self.acc_in = eng.sums("in", m.w_in.shape[0])
+        self.o = eng.scratch("o", eng.max_seqs, m.o.shape[1])
+        self.left = SLOTS[m.left.kind](eng, m.left, li, self.acc_in[:, :a], self.o[:, :b], m.scales[0])
+        self.right = SLOTS[m.right.kind](eng, m.right, li, self.acc_in[:, a:], self.o[:, b:], m.scales[1])
+
+    def prompt_target(self, pages: "_Pages") -> dict:
+        return dict(left=self.left.prompt_target(pages), right=self.right.prompt_target(pages))
+
+    def copy_pages(self, dst, src):
+        self.left.copy_pages(dst, src)
+        self.right.copy_pages(dst, src)
+
+    def copy_slots(self, dst, src):
+        self.left.copy_slots(dst, src)
+        self.right.copy_slots(dst, src)
+
+    def step(self, h, out):
+        self.e.gemm(h, self.m.w_in, self.acc_in)
+        self.left.mix()
+        self.right.mix()
+        self.e.gemm(self.o, self.m.o, out)
+
+
+SLOTS = {"latent_attention": _LatentSlots, "mlstm": _MLstmSlots, "attention": _AttentionSlots, "attention_2": _AttentionSlots,
+         "rglru": _RgLruSlots, "hgrn2": _HGrn2Slots, "parallel": _ParallelSlots}
 
 
 class _Pages:
@@ -333,6 +411,8 @@ class LayeredRolloutEngine(RolloutEngine):
         self._x = torch.zeros(B, H, dtype=torch.float32, device=self.dev)
         self._acc = self.sums("out", H)
         self._h = self.scratch("h", B, H)
+        self._h2 = torch.zeros_like(self._h) if any(l.beside for l in self.model.layers) else None
+        self._first = torch.zeros_like(self._x) if cfg.passes > 1 else None  # the embedding, which a loop adds again
         self._logits_buf = torch.zeros(B, cfg.vocab_size, dtype=self.dtype, device=self.dev)
 
     def _reset_sums(self):
@@ -384,7 +464,10 @@ class LayeredRolloutEngine(RolloutEngine):
         from ..ops import cuda_mixers as KM
 
         m, x, h, acc = self.model, self._x, self._h, self._acc
-        if m.pair_embed is None:
+        if m.embed_norm is not None:
+            n = m.embed_norm
+            KM.embed_normed(self.next_input, m.embed_tokens, self.cfg.embed_scale, n.weight, n.eps, n.shift, out=x, copy=self._first)
+        elif m.pair_embed is None:
             KM.embed_scaled(self.next_input, m.embed_tokens, self.cfg.embed_scale, out=x)
         else:
             p = self.cfg.pairs
@@ -393,7 +476,13 @@ class LayeredRolloutEngine(RolloutEngine):
         delta = post = None  # sums not yet added to the stream, and the norm they pass first
         now = dict(clear=True, out=h)
         for li, (layer, slots) in enumerate(zip(m.layers, self.slots)):
-            layer.read_mixer(x, delta, post, **now)
+            if layer.beside:
+                layer.read_both(x, delta, post, **now, out2=self._h2, **m.entrance(li, self._first))
+                rows = None if layer.mlp is None else self.experts(self._h2, layer.mlp)
+                slots.step(h, acc)
+                delta, post = acc if rows is None else (acc, rows), None
+                continue
+            layer.read_mixer(x, delta, post, **now, **m.entrance(li, self._first))
             slots.step(h, acc)
             delta, post = acc, layer.norm1b
             if layer.mlp is not None:
@@ -421,11 +510,12 @@ class LayeredRolloutEngine(RolloutEngine):
             return K.decode_gemm(h, mlp.w_in, out=act, **mlp.fused)
         return mlp.act(mx.linear(h, mlp.w_in), out=act)
 
-    def experts(self, h, mlp, out):
-        """Mixture of experts of the slots that are live; ``out`` (fp32) is stored to."""
+    def experts(self, h, mlp, out=None):
+        """Mixture of experts of the slots that are live; ``out`` (fp32) is stored to.  Without it the experts' rows are returned,
+        not yet added up."""
         z = self.sums("router", mlp.n)
         self.gemm(h, mlp.router, z)
-        mx.experts(mlp, h, positions=self.seq_lens, logits=z, out=out)
+        return mx.experts(mlp, h, positions=self.seq_lens, logits=z, out=out, summed=out is not None)
 
     def side_act(self, h, side, li):
         from ..ops import cuda_mixers as KM
