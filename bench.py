@@ -65,7 +65,7 @@ def parse():
                          "warm-up steps how many layers fit (gradient_checkpointing_kwargs={'num_layers': 'auto'}).  With "
                          "micro-batches of varying length keeping activations did not pay here: the allocator's "
                          "remapping cost what the recomputation saved")
-    ap.add_argument("--layered", nargs="?", const="zorelorn", choices=["zorelorn", "povusun", "suposun"],
+    ap.add_argument("--layered", nargs="?", const="zorelorn", choices=["zorelorn", "povusun", "suposun", "gerupel"],
                     help="instead of the GRPO workload: prompt and decode throughput of a layered design (default Zorelorn) beside "
                          "a flat decoder of equal width, depth and parameter count (with experts where the design has them), and the "
                          "mixers' kernels alone (one GPU)")

@@ -1,7 +1,7 @@
 """Prompt and decode throughput of a layered design beside the closest flat decoder of the same width, depth and
 parameter count (random weights, bf16, one GPU), through the serving engine.
 
-    python -m trl_b200.benchmarks.layered_throughput [--design zorelorn|povusun|suposun] [--sizes small,base] [--kernels]
+    python -m trl_b200.benchmarks.layered_throughput [--design zorelorn|povusun|suposun|gerupel] [--sizes small,base] [--kernels]
 
 Prompt: packed prompts through the engine's prompt forward into its cache.  Decode: replays of the captured step (CUDA
 graph, sampler included) with every slot at the given context.  CUDA events after warm-up; the weights of a step are
@@ -15,13 +15,16 @@ import os
 import torch
 
 # width, heads (attention of every kind), ff; Zorelorn: query latent, mLSTM heads, pairs of layers; Povusun: side input, quads;
-# Suposun: experts of every second layer, of which a token runs `top` of width `eff` (ff = top x eff), quads
+# Suposun: experts of every second layer, of which a token runs `top` of width `eff` (ff = top x eff), quads; Gerupel: heads of the
+# recurrent half (128 x 128), experts of every layer, layers, of which the third and fourth run twice
 SIZES = {"zorelorn": {"small": dict(width=2048, heads=16, q_rank=768, ff=8192, mheads=4, pairs=4),
                       "base": dict(width=4096, heads=32, q_rank=1536, ff=16384, mheads=8, pairs=4)},
          "povusun": {"small": dict(width=2048, heads=16, ff=6144, side=256, quads=2),
                      "base": dict(width=4096, heads=32, ff=12288, side=256, quads=2)},
          "suposun": {"small": dict(width=2048, heads=16, ff=4096, eff=1024, experts=48, top=4, quads=2),
-                     "base": dict(width=4096, heads=32, ff=8192, eff=2048, experts=32, top=4, quads=2)}}
+                     "base": dict(width=4096, heads=32, ff=8192, eff=2048, experts=32, top=4, quads=2)},
+         "gerupel": {"small": dict(width=2048, heads=16, rheads=16, ff=4096, eff=1024, experts=32, top=4, layers=6),
+                     "base": dict(width=4096, heads=32, rheads=32, ff=8192, eff=2048, experts=24, top=4, layers=6)}}
 VOCAB = 32768
 
 
@@ -60,7 +63,16 @@ def suposun_config(width, heads, ff, eff, experts, top, quads, window=512):
                 embedding=dict(scale=1.0, bigram=dict(buckets=8191, mul_prev=131, mul_cur=7)))
 
 
-CONFIGS = {"zorelorn": zorelorn_config, "povusun": povusun_config, "suposun": suposun_config}
+def gerupel_config(width, heads, rheads, ff, eff, experts, top, layers, window=512, pool=16):
+    rot = dict(base=5e5, dims=128, scaling=dict(factor=8.0, original=8192, low=1.0, high=4.0))
+    left = dict(heads=heads, kv_heads=heads // 4, dim=128, vdim=128, scale=128 ** -0.5, mask=dict(size=window, pool=pool), rot=rot)
+    layer = dict(type="parallel", mixer=dict(left=left, right=dict(heads=rheads, dim=128, vdim=128), left_scale=0.9, right_scale=0.7),
+                 mlp=dict(kind="moe", expert=dict(ff=eff), router=dict(experts=experts, top=top, scale=1.5)))
+    return dict(architecture="Gerupel", vocab=VOCAB, width=width, norm=dict(eps=1e-6), residual_mult=0.8, layers=[layer] * layers,
+                loop=dict(start=2, stop=4, times=2) if layers > 3 else None)
+
+
+CONFIGS = {"zorelorn": zorelorn_config, "povusun": povusun_config, "suposun": suposun_config, "gerupel": gerupel_config}
 
 
 def layered_config(design, s):
@@ -203,8 +215,8 @@ def kernel_table(size="base", batch=64, prompt=1024, n_prompts=8, iters=20, desi
     from ..ops import cuda as K
     from ..rollout.engine import make_engine
 
-    s = dict(SIZES[design][size], **(dict(pairs=1) if design == "zorelorn" else dict(quads=1)))
-    kernels = {"zorelorn": zorelorn_kernels, "povusun": povusun_kernels, "suposun": suposun_kernels}[design]
+    s = dict(SIZES[design][size], **{"zorelorn": dict(pairs=1), "gerupel": dict(layers=1)}.get(design, dict(quads=1)))
+    kernels = {"zorelorn": zorelorn_kernels, "povusun": povusun_kernels, "suposun": suposun_kernels, "gerupel": gerupel_kernels}[design]
     model = build_model(ModelArch.from_hf_dict(layered_config(design, s)), dtype=torch.bfloat16, device="cuda").eval().requires_grad_(False)
     eng = make_engine(model, max_num_seqs=batch, max_model_len=prompt + 64)
     row = KernelTimer(iters)
@@ -341,21 +353,7 @@ def suposun_kernels(s, model, eng, batch, prompt, n_prompts, row):
     z = torch.randn(T, 2 * s["ff"], device=dev, dtype=bf)
     row("prompt GELU unit", lambda: KM.gelu_glu(z), z.numel() * 3)
     del z
-    E, top, n = moe.n, moe.top, moe.ff
-    R = T * top
-    zr = mx.linear_f32(h, moe.router)
-    row("prompt router choice", lambda: KM.moe_route(zr, moe.correction, top), T * (E * 4 + top * 12))
-    choice, rank, weight, counts = KM.moe_route(zr, moe.correction, top)
-    row("prompt gather by expert", lambda: KM.moe_gather(h, choice, rank, counts), T * W * 2 + R * W * 2)
-    xs, at, offsets = KM.moe_gather(h, choice, rank, counts)
-    row("prompt experts gate/up + clamped unit", lambda: K.grouped_gemm(xs, moe.gate_up, offsets, n, clamped_glu=moe.glu),
-        moe.gate_up.numel() * 2 + R * (W + n) * 2, 4 * R * W * n)
-    act = K.grouped_gemm(xs, moe.gate_up, offsets, n, clamped_glu=moe.glu)
-    row("prompt experts down", lambda: K.grouped_gemm(act, moe.down, offsets, W), moe.down.numel() * 2 + R * (W + n) * 2, 2 * R * W * n)
-    ys = K.grouped_gemm(act, moe.down, offsets, W)
-    row("prompt weighted sum", lambda: KM.moe_sum(ys, at, weight), R * W * 2 + T * W * 4)
-    row("prompt experts, all of it", lambda: mx.experts(moe, h), moe.gate_up.numel() * 3 + T * W * 6, 6 * R * W * n)
-    del xs, act, ys
+    prompt_expert_kernels(moe, h, row)
 
     a, r = eng.slots[0], eng.slots[3]
     hb, xb, db = torch.randn(B, W, device=dev, dtype=bf), torch.randn(B, W, device=dev), torch.randn(B, W, device=dev)
@@ -372,20 +370,113 @@ def suposun_kernels(s, model, eng, batch, prompt, n_prompts, row):
     row("decode windowed attention (capped, sink, gated)", a.attend, B * seen * kv * 2 + 4 * a.q.numel(), 2 * B * seen * near.heads * 256)
     row("decode attention_2", r.attend, B * (prompt + 1) * kv * 2 + 4 * r.q.numel(), 2 * B * (prompt + 1) * far.heads * 256)
     row("decode gate/up + GELU unit", lambda: eng.mlp_act(hb, glu), glu.gate_up.numel() * 2)
-    zb = torch.zeros(B, E, device=dev)
+    decode_expert_kernels(eng, moe, hb, db, row)
+
+
+@torch.no_grad()
+def prompt_expert_kernels(moe, h, row):
+    from ..ops import cuda as K
+    from ..ops import cuda_mixers as KM
+    from ..ops import mixers as mx
+
+    E, top, n = moe.n, moe.top, moe.ff
+    T, W = h.shape
+    R = T * top
+    zr = mx.linear_f32(h, moe.router)
+    row("prompt router choice", lambda: KM.moe_route(zr, moe.correction, top, **moe.routing), T * (E * 4 + top * 12))
+    choice, rank, weight, counts = KM.moe_route(zr, moe.correction, top, **moe.routing)
+    row("prompt gather by expert", lambda: KM.moe_gather(h, choice, rank, counts), T * W * 2 + R * W * 2)
+    xs, at, offsets = KM.moe_gather(h, choice, rank, counts)
+    row("prompt experts gate/up + gated unit", lambda: K.grouped_gemm(xs, moe.gate_up, offsets, n, clamped_glu=moe.glu),
+        moe.gate_up.numel() * 2 + R * (W + n) * 2, 4 * R * W * n)
+    act = K.grouped_gemm(xs, moe.gate_up, offsets, n, clamped_glu=moe.glu)
+    row("prompt experts down", lambda: K.grouped_gemm(act, moe.down, offsets, W), moe.down.numel() * 2 + R * (W + n) * 2, 2 * R * W * n)
+    ys = K.grouped_gemm(act, moe.down, offsets, W)
+    row("prompt weighted sum", lambda: KM.moe_sum(ys, at, weight), R * W * 2 + T * W * 4)
+    row("prompt experts, all of it", lambda: mx.experts(moe, h), moe.gate_up.numel() * 3 + T * W * 6, 6 * R * W * n)
+
+
+@torch.no_grad()
+def decode_expert_kernels(eng, moe, hb, db, row):
+    from ..ops import cuda as K
+    from ..ops import cuda_mixers as KM
+    from ..ops import mixers as mx
+
+    (B, W), E, top, n = hb.shape, moe.n, moe.top, moe.ff
+    zb = torch.zeros(B, E, device=hb.device)
     row("decode router product", lambda: K.decode_gemm(hb, moe.router, y32=zb), moe.router.numel() * 2)
     zb = mx.linear_f32(hb, moe.router)
-    row("decode router choice", lambda: KM.moe_route(zb, moe.correction, top, positions=eng.seq_lens), B * (E * 4 + top * 12))
-    choice, rank, weight, counts = KM.moe_route(zb, moe.correction, top)
+    row("decode router choice", lambda: KM.moe_route(zb, moe.correction, top, positions=eng.seq_lens, **moe.routing), B * (E * 4 + top * 12))
+    choice, rank, weight, counts = KM.moe_route(zb, moe.correction, top, **moe.routing)
     row("decode gather by expert", lambda: KM.moe_gather(hb, choice, rank, counts), B * W * 2 * (1 + top))
     xs, at, offsets = KM.moe_gather(hb, choice, rank, counts)
     used = int((counts > 0).sum())
-    row("decode experts gate/up + clamped unit", lambda: K.grouped_gemm(xs, moe.gate_up, offsets, n, clamped_glu=moe.glu), used * 4 * W * n)
+    row("decode experts gate/up + gated unit", lambda: K.grouped_gemm(xs, moe.gate_up, offsets, n, clamped_glu=moe.glu), used * 4 * W * n)
     act = K.grouped_gemm(xs, moe.gate_up, offsets, n, clamped_glu=moe.glu)
     row("decode experts down", lambda: K.grouped_gemm(act, moe.down, offsets, W), used * 2 * W * n)
     ys = K.grouped_gemm(act, moe.down, offsets, W)
     row("decode weighted sum", lambda: KM.moe_sum(ys, at, weight, out=db), B * W * (2 * top + 4))
     row("decode experts, all of it", lambda: eng.experts(hb, moe, db), used * 6 * W * n)
+
+
+@torch.no_grad()
+def gerupel_kernels(s, model, eng, batch, prompt, n_prompts, row):
+    from ..models.decoder import SeqCtx
+    from ..ops import cuda as K
+    from ..ops import cuda_mixers as KM
+    from ..ops import mixers as mx
+
+    m, moe, layer = model.layers[0].mixer, model.layers[0].mlp, model.layers[0]
+    at, rg = m.left, m.right
+    T, W, dev, bf, B = n_prompts * prompt, s["width"], "cuda", torch.bfloat16, batch
+    ctx = SeqCtx.from_lengths([prompt] * n_prompts, dev)
+    h = torch.randn(T, W, device=dev, dtype=bf)
+    x, d = torch.randn(T, W, device=dev), torch.randn(T, W, device=dev)
+    of_seq = torch.arange(n_prompts, device=dev, dtype=torch.int32)
+    target = eng.slots[0].prompt_target(eng._page_writer(of_seq.repeat_interleave(prompt), ctx, of_seq))
+    paged_context(eng, prompt)
+    ids = torch.randint(0, VOCAB, (T,), device=dev)
+    row("prompt embedding + norm", lambda: KM.embed_normed(ids, model.embed_tokens, 1.0, model.embed_norm.weight, 1e-6), T * W * 6)
+    ys = mx.experts(moe, h, summed=False)
+    row("prompt experts' sum + residual + both norms", lambda: KM.rms_residual(x, (d, ys), None, layer.norm1.weight, 1e-6, bf, w2=layer.norm2.weight, mult=0.8),
+        T * W * (16 + 2 * moe.top))
+    del ys
+    y, z = mx.linear(h, m.w_in[: m.rows]), mx.linear_f32(h, m.w_in[m.rows:])
+    o = torch.empty(T, m.o.shape[1], device=dev, dtype=bf)
+    ya, yr, (q, k, v, _) = y[:, : at.rows], y[:, at.rows:], y[:, : at.rows].split(at.parts, 1)
+    where = {key: t for key, t in target["left"].items() if key != "pools"}
+    kv = at.kv_heads * (at.dim + at.vdim)
+    row("prompt preparation of attention", lambda: KM.attn_prep(ya, at, ctx.positions, None, table=at.rope.table(prompt, dev), **at.prep, **where),
+        T * 2 * (2 * (at.heads + at.kv_heads) * at.dim + at.kv_heads * at.vdim + kv))
+    row("prompt means of blocks", lambda: KM.pool_blocks(k, v, ctx.cu_seqlens, at.pool, **target["left"]["pools"]), T * kv * 2 * (1 + 2 / at.pool))
+    blocks = KM.pool_blocks(k, v, ctx.cu_seqlens, at.pool)
+    i = torch.arange(prompt, dtype=torch.float64)
+    pairs = n_prompts * float((torch.clamp(i + 1, max=at.window) + torch.floor(torch.clamp(i + 1 - at.window, min=0) / at.pool)).sum())
+    row("prompt windowed attention with blocks (sink)", lambda: KM.mixer_attn(q, k, v, heads=at.heads, kv_heads=at.kv_heads, scale=at.scale, **at.sight, pool=at.pool,
+                                                                             blocks=blocks, ctx=ctx, out=o[:, : at.out_width], out_scale=0.9),
+        T * 2 * (at.rows + at.out_width), 2 * pairs * at.heads * (at.dim + at.vdim))
+    row("prompt hgrn2 recurrence", lambda: mx.hgrn2_prompt_scan(rg, yr, z, ctx, target["right"]),
+        T * rg.heads * (rg.dim * 6 + rg.vdim * 6) + n_prompts * rg.heads * rg.dim * rg.vdim * 4,
+        2 * T * rg.heads * (2 * rg.dim * rg.vdim + 64 * (rg.dim + rg.vdim)))
+    o32 = mx.hgrn2_prompt_scan(rg, yr, z, ctx, {})
+    row("prompt norm per head", lambda: KM.head_norm(o32, rg.norm, 1e-6, bf, out=o[:, at.out_width:], scale=0.7), o32.numel() * 6)
+    del y, z, o, ya, yr, q, k, v, o32
+    prompt_expert_kernels(moe, h, row)
+
+    a = eng.slots[0]
+    hb, xb, db = torch.randn(B, W, device=dev, dtype=bf), torch.randn(B, W, device=dev), torch.randn(B, W, device=dev)
+    row("decode embedding + norm", lambda: KM.embed_normed(eng.next_input, model.embed_tokens, 1.0, model.embed_norm.weight, 1e-6, out=xb), B * W * 6)
+    rows = eng.experts(hb, moe)
+    row("decode experts' sum + residual + both norms", lambda: KM.rms_residual(xb, (db, rows), None, layer.norm1.weight, 1e-6, bf, clear=True, out=hb,
+                                                                              w2=layer.norm2.weight, out2=eng._h2, mult=0.8), B * W * (20 + 2 * moe.top))
+    hb = torch.randn(B, W, device=dev, dtype=bf)
+    row("decode gemm input", lambda: K.decode_gemm(hb, m.w_in, y32=a.acc_in), m.w_in.numel() * 2)
+    row("decode preparation of attention + cache", a.left.prepare, a.left.acc_in.numel() * 10)
+    seen = min(prompt + 1, at.window) + max(0, prompt + 1 - at.window) // at.pool
+    row("decode windowed attention with blocks (sink)", a.left.attend, B * seen * kv * 2 + 4 * a.left.q.numel(), 2 * B * seen * at.heads * (at.dim + at.vdim))
+    row("decode hgrn2 step + norm", a.right.mix, a.right.state.numel() * 8 + B * sum(rg.parts) * 8 + a.right.y.numel() * 2)
+    row("decode gemm output", lambda: K.decode_gemm(a.o, m.o, y32=eng._acc), m.o.numel() * 2)
+    decode_expert_kernels(eng, moe, hb, db, row)
 
 
 @torch.no_grad()
