@@ -28,7 +28,7 @@ OBJ = os.path.join(LIB, "obj")
 NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17", "--use_fast_math",
               "-Xcompiler", "-fPIC,-fvisibility=hidden", "-Xptxas", "-v", "--expt-relaxed-constexpr"]
 # sources whose results the fast approximations of exp, tanh, erf, division and square root would show in
-EXACT_MATH = {"grouped_attn.cu", "hgrn2.cu", "layered_moe.cu", "mixers.cu", "mlstm_chunk_tcgen05.cu", "rglru.cu", "rglru_tcgen05.cu"}
+EXACT_MATH = {"grouped_attn.cu", "hgrn2.cu", "hgrn2_chunk_tcgen05.cu", "layered_moe.cu", "mixers.cu", "mlstm_chunk_tcgen05.cu", "rglru.cu", "rglru_tcgen05.cu"}
 # every source here builds into the one library used at any GPU count (no loads shared across a thread-block cluster)
 
 
@@ -38,7 +38,7 @@ PARTS = {"layered": ("decode.cu", "decode_gemm.cu", "mixers.cu", "tensormap.cu")
 _GROUPED = ("grouped_attn.cu", "grouped_decode_tcgen05.cu", "mixer_attn_tcgen05.cu")
 LAYERED_KINDS = {"latent_attention": ("grouped_attn.cu", "latent_decode_tcgen05.cu", "mixer_attn_tcgen05.cu"),
                  "mlstm": ("mlstm_chunk_tcgen05.cu",), "attention": _GROUPED, "attention_2": _GROUPED,
-                 "rglru": ("rglru.cu", "rglru_tcgen05.cu"), "hgrn2": ("hgrn2.cu",), "moe": ("grouped_gemm_tcgen05.cu", "layered_moe.cu")}
+                 "rglru": ("rglru.cu", "rglru_tcgen05.cu"), "hgrn2": ("hgrn2.cu", "hgrn2_chunk_tcgen05.cu"), "moe": ("grouped_gemm_tcgen05.cu", "layered_moe.cu")}
 
 
 def _nvcc() -> str:

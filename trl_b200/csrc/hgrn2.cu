@@ -2,6 +2,7 @@
 //
 //     f = low + (1 - low) sigmoid(z + bias),   S = diag(f) S + (1 - f) v^T,   o = S^T silu(q),
 //
+// computed with k = 1 - f = (1 - low) sigmoid(-z - bias), which keeps its precision where f is close to one: S += k (v - S).  Here
 // token by token for every size and dtype, the decode step, and the norm per head behind it (prompts on the tensor cores:
 // hgrn2_chunk_tcgen05.cu).
 //
@@ -13,7 +14,7 @@
 namespace trlb {
 
 __device__ __forceinline__ float silu_f(float z) { return z * sigmoid_f(z); }
-__device__ __forceinline__ float forget_f(float z, float low) { return low + (1.f - low) * sigmoid_f(z); }
+__device__ __forceinline__ float write_f(float z, float low) { return (1.f - low) * sigmoid_f(-z); }
 
 // ------------------------------------------------------------------------------------------------------------
 // Prompts: grid (sequence, head, 32-column tile of vdim), 256 threads.  A thread holds NR rows of one column of S in registers;
@@ -38,14 +39,14 @@ hgrn2_prompt_kernel(const Hgrn2 p, const T* __restrict__ y, const float* __restr
   constexpr int ROW = 8 * (NR + 4);  // a lane's rows start on another bank than its neighbours'
   extern __shared__ float sm[];
   float* qs = sm;                        // [HG_STAGE][ROW]
-  float* fs = qs + HG_STAGE * ROW;       // [HG_STAGE][ROW]
-  float* vs = fs + HG_STAGE * ROW;       // [HG_STAGE][32]
+  float* ks = qs + HG_STAGE * ROW;       // [HG_STAGE][ROW]
+  float* vs = ks + HG_STAGE * ROW;       // [HG_STAGE][32]
   const int seq = blockIdx.x, h = blockIdx.y, e0 = blockIdx.z * 32, tid = threadIdx.x, dg = tid & 7, ec = tid >> 3, e = e0 + ec;
   const int t0 = p.cu[seq], len = p.cu[seq + 1] - t0;
   float S[NR];
 #pragma unroll
   for (int i = 0; i < NR; ++i) S[i] = 0.f;
-  for (int i = tid; i < 2 * HG_STAGE * ROW; i += 256) sm[i] = 0.f;  // rows past dim: nothing forgets, writes or reads
+  for (int i = tid; i < 2 * HG_STAGE * ROW; i += 256) sm[i] = 0.f;  // rows past dim write and read nothing
   for (int base = 0; base < len; base += HG_STAGE) {
     const int n = min(HG_STAGE, len - base);
     __syncthreads();
@@ -53,7 +54,7 @@ hgrn2_prompt_kernel(const Hgrn2 p, const T* __restrict__ y, const float* __restr
       const int t = i / p.dim, d = i % p.dim, at = t * ROW + (d / NR) * (NR + 4) + d % NR, hd = h * p.dim + d;
       const size_t row = (size_t)(t0 + base + t);
       qs[at] = silu_f(to_f(y[row * p.y_ld + hd]));
-      fs[at] = forget_f(z[row * p.z_ld + hd] + p.bias[hd], p.low[hd]);
+      ks[at] = write_f(z[row * p.z_ld + hd] + p.bias[hd], p.low[hd]);
     }
     for (int i = tid; i < n * 32; i += 256) {
       const int t = i >> 5, c = e0 + (i & 31);
@@ -62,16 +63,16 @@ hgrn2_prompt_kernel(const Hgrn2 p, const T* __restrict__ y, const float* __restr
     __syncthreads();
     for (int t = 0; t < n; ++t) {
       const float v = vs[t * 32 + ec];
-      const float* f = fs + t * ROW + dg * (NR + 4);
+      const float* k = ks + t * ROW + dg * (NR + 4);
       const float* q = qs + t * ROW + dg * (NR + 4);
       float acc[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
       for (int i = 0; i < NR; i += 4) {
-        const float4 a = load4(f + i), b = load4(q + i);
-        S[i] = fmaf(a.x, S[i] - v, v);
-        S[i + 1] = fmaf(a.y, S[i + 1] - v, v);
-        S[i + 2] = fmaf(a.z, S[i + 2] - v, v);
-        S[i + 3] = fmaf(a.w, S[i + 3] - v, v);
+        const float4 a = load4(k + i), b = load4(q + i);
+        S[i] = fmaf(a.x, v - S[i], S[i]);
+        S[i + 1] = fmaf(a.y, v - S[i + 1], S[i + 1]);
+        S[i + 2] = fmaf(a.z, v - S[i + 2], S[i + 2]);
+        S[i + 3] = fmaf(a.w, v - S[i + 3], S[i + 3]);
         acc[0] = fmaf(S[i], b.x, acc[0]);
         acc[1] = fmaf(S[i + 1], b.y, acc[1]);
         acc[2] = fmaf(S[i + 2], b.z, acc[2]);
@@ -79,7 +80,7 @@ hgrn2_prompt_kernel(const Hgrn2 p, const T* __restrict__ y, const float* __restr
       }
       float o = (acc[0] + acc[1]) + (acc[2] + acc[3]);
 #pragma unroll
-      for (int k = 1; k < 8; k <<= 1) o += __shfl_xor_sync(0xffffffffu, o, k);
+      for (int x = 1; x < 8; x <<= 1) o += __shfl_xor_sync(0xffffffffu, o, x);
       if (dg == 0 && e < p.vdim) out[((size_t)(t0 + base + t) * p.heads + h) * p.vdim + e] = o;
     }
   }
@@ -141,7 +142,7 @@ struct Hgrn2Step {
 template <typename T, int VEC>
 __global__ void __launch_bounds__(256)
 hgrn2_step_kernel(const Hgrn2Step p, T* __restrict__ y) {
-  extern __shared__ float sm[];  // q [dim], f [dim], v [vdim], partial sums [row groups][vdim]
+  extern __shared__ float sm[];  // q [dim], k [dim], v [vdim], partial sums [row groups][vdim]
   __shared__ float red[64];
   pdl_launch_dependents();
   pdl_wait();
@@ -149,15 +150,15 @@ hgrn2_step_kernel(const Hgrn2Step p, T* __restrict__ y) {
   const int rgs = 256 >> p.groups_log2;
   const bool live = p.seq_lens[b] >= 0;
   float* qs = sm;
-  float* fs = qs + p.dim;
-  float* vs = fs + p.dim;
+  float* ks = qs + p.dim;
+  float* vs = ks + p.dim;
   float* part = vs + p.vdim;
   float* q = p.sums + (size_t)b * p.ld + (size_t)h * p.dim;
   float* v = p.sums + (size_t)b * p.ld + (size_t)p.heads * p.dim + (size_t)h * p.vdim;
   float* z = p.sums + (size_t)b * p.ld + (size_t)p.heads * (p.dim + p.vdim) + (size_t)h * p.dim;
   for (int d = tid; d < p.dim; d += 256) {
     qs[d] = silu_f(q[d]);
-    fs[d] = forget_f(z[d] + p.bias[h * p.dim + d], p.low[h * p.dim + d]);
+    ks[d] = write_f(z[d] + p.bias[h * p.dim + d], p.low[h * p.dim + d]);
     q[d] = 0.f;
     z[d] = 0.f;
   }
@@ -187,7 +188,7 @@ hgrn2_step_kernel(const Hgrn2Step p, T* __restrict__ y) {
       }
 #pragma unroll
       for (int i = 0; i < VEC; ++i) {
-        s[i] = fmaf(fs[d], s[i] - w[i], w[i]);
+        s[i] = fmaf(ks[d], w[i] - s[i], s[i]);
         o[i] = fmaf(s[i], qs[d], o[i]);
       }
       if (VEC == 4) store4(at, make_float4(s[0], s[1 % VEC], s[2 % VEC], s[3 % VEC]));

@@ -351,6 +351,28 @@ def hgrn2_prompt(y, z, m, cu, seq_slot=None, state=None):
     return out
 
 
+def hgrn2_chunk_ok(m) -> bool:
+    return bool(lib().trlb_hgrn2_chunk_ok(c_int(m.heads), c_int(m.dim), c_int(m.vdim)))
+
+
+def hgrn2_chunk(y, z, m, cu, seq_slot=None, state=None, normed=None, scale=1.0):
+    """:func:`hgrn2_prompt` in 128-token chunks on the tensor cores (bf16; see ``hgrn2_chunk_ok``).  With ``normed`` [T, heads vdim]
+    (rows may be strided; vdim <= 128) that gets the outputs over their rms per head times the norm's weight and ``scale``, and is
+    returned."""
+    T, n_seq, qd = y.shape[0], cu.numel() - 1, m.heads * m.dim
+    assert y.dtype == torch.bfloat16 and y.stride(1) == 1 and z.stride(1) == 1 and z.dtype == torch.float32 and cu.dtype == torch.int32
+    assert normed is None or (normed.shape == (T, m.heads * m.vdim) and normed.stride(1) == 1 and normed.dtype == torch.bfloat16)
+    out = torch.empty(T, m.heads, m.vdim, dtype=torch.float32, device=y.device) if normed is None else None
+    parts = torch.empty(2, int(lib().trlb_hgrn2_chunks(c_int(T), c_int(n_seq))), m.heads, m.dim, m.vdim, dtype=torch.bfloat16, device=y.device)
+    _chk(lib().trlb_hgrn2_chunk(_p(y), c_longlong(y.stride(0)), c_int(qd), _p(z), c_longlong(z.stride(0)), _p(m.f_bias), _p(m.lower), _p(cu),
+                                c_int(n_seq), c_int(T), _p(seq_slot if state is not None else None), _p(state),
+                                c_int(0 if state is None else state.shape[0]), c_int(m.heads), c_int(m.dim), c_int(m.vdim),
+                                _p(m.norm if normed is not None else None), c_float(m.eps), c_float(scale), _p(normed),
+                                c_longlong(0 if normed is None else normed.stride(0)), _p(out), _p(parts[0]), _p(parts[1]),
+                                _p(status_buffer(y.device)), _s()), "hgrn2_chunk")
+    return out if normed is None else normed
+
+
 def head_norm(o, w, eps, dtype, out=None, scale=1.0):
     """o fp32 [T, heads, vdim] over its rms per head times ``w`` [vdim] and ``scale`` -> [T, heads vdim] (rows of ``out`` may be
     strided)."""
