@@ -321,6 +321,7 @@ attn_prep_rows_kernel(const AttnPrep p, int lanes_log2, S* __restrict__ src, T* 
   const bool turns = j0 < p.rot && pos >= 0 && pos < p.table_len;
   const int half = p.rot / 2, shift = half / 8;  // halves: the partner is `shift` threads away
   const bool upper = j0 >= half;
+  const int partner = (threadIdx.x & 31) + (j0 >= p.rot ? 0 : upper ? -shift : shift);
   float2 cs[8];
   if (turns) {
     const float2* t = p.table + (size_t)pos * half + (p.halves ? (upper ? j0 - half : j0) : j0 / 2);
@@ -380,8 +381,8 @@ attn_prep_rows_kernel(const AttnPrep p, int lanes_log2, S* __restrict__ src, T* 
     if (p.rot > 0 && p.halves) {
 #pragma unroll
       for (int e = 0; e < 8; ++e) {  // every lane takes part
-        const float down = __shfl_down_sync(0xffffffffu, x[i][e], shift, lanes), up = __shfl_up_sync(0xffffffffu, x[i][e], shift, lanes);
-        if (turns && normed) x[i][e] = upper ? x[i][e] * cs[e].x + up * cs[e].y : x[i][e] * cs[e].x - down * cs[e].y;
+        const float other = __shfl_sync(0xffffffffu, x[i][e], partner);
+        if (turns && normed) x[i][e] = x[i][e] * cs[e].x + (upper ? other : -other) * cs[e].y;
       }
     } else if (turns && normed) {
 #pragma unroll
@@ -429,7 +430,7 @@ attn_prep_rows_kernel(const AttnPrep p, int lanes_log2, S* __restrict__ src, T* 
 // ------------------------------------------------------------------------------------------------------------
 // Means of blocks of P rows of packed keys and values (fp32 sums).  The blocks of the sequence that starts at token a are rows
 // a / P + block of pk and pv (no two sequences meet there); rows of no block are zeros.  With slots also to the slots' rows.
-// One block of threads per row; n columns, T of the rows.
+// grid: (rows, slices of the columns).
 // ------------------------------------------------------------------------------------------------------------
 struct PoolBlocks {
   const int* cu;
@@ -457,7 +458,8 @@ pool_blocks_kernel(const PoolBlocks p, const T* __restrict__ k, const T* __restr
   const bool v4 = ((p.k_n | p.v_n | (int)(p.k_ld & 3) | (int)(p.v_ld & 3)) & 3) == 0 &&
                   ((reinterpret_cast<uintptr_t>(k) | reinterpret_cast<uintptr_t>(v)) & (4 * sizeof(T) - 1)) == 0;
   const float inv = 1.f / (float)p.P;
-  for (int c = (v4 ? 4 : 1) * threadIdx.x; c < n; c += (v4 ? 4 : 1) * blockDim.x) {
+  const int vec = v4 ? 4 : 1;
+  for (int c = vec * (blockIdx.y * blockDim.x + threadIdx.x); c < n; c += vec * gridDim.y * blockDim.x) {
     const bool key = c < p.k_n;
     const int j = key ? c : c - p.k_n, m = key ? p.k_n : p.v_n;
     const T* src = (key ? k : v) + t0 * (key ? p.k_ld : p.v_ld) + j;
@@ -467,6 +469,7 @@ pool_blocks_kernel(const PoolBlocks p, const T* __restrict__ k, const T* __restr
     if (v4) {
       float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
       if (seq >= 0) {
+#pragma unroll 8
         for (int t = 0; t < p.P; ++t) {
           const float4 x = load4(src + (size_t)t * ld);
           a = make_float4(a.x + x.x, a.y + x.y, a.z + x.z, a.w + x.w);
@@ -732,7 +735,7 @@ TRLB_API int trlb_pool_blocks(const void* k, long long k_ld, int k_n, const void
   if (T <= 0 || n_seq <= 0) return 0;
   if (P <= 0 || (seq_slot != nullptr && (slot_k == nullptr || slot_v == nullptr))) return -254;
   const PoolBlocks p = {cu, n_seq, P, k_n, v_n, k_ld, v_ld, seq_slot, slots, slot_rows};
-  const int rows = T / P + 1;
+  const dim3 rows(T / P + 1, (k_n + v_n + 511) / 512);
   if (is_bf16) pool_blocks_kernel<bf16><<<rows, 128, 0, st>>>(p, (const bf16*)k, (const bf16*)v, (bf16*)pk, (bf16*)pv, (bf16*)slot_k, (bf16*)slot_v);
   else pool_blocks_kernel<float><<<rows, 128, 0, st>>>(p, (const float*)k, (const float*)v, (float*)pk, (float*)pv, (float*)slot_k, (float*)slot_v);
   return (int)cudaGetLastError();

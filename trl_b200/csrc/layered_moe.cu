@@ -14,14 +14,14 @@ constexpr int MR_MAX_E = 1024;
 // ------------------------------------------------------------------------------------------------------------
 // Router: scores sigmoid(z), or softmax(z); the `top` experts of the largest score + correction (ties: the lower index) with their
 // bare scores as weights (renorm: over their sum), times gain.  One warp per token.  rank: place among the expert's rows.  ONE: a single block
-// counts in shared memory and stores the counts; else counts are zeros before the launch.  Negative positions mark idle rows,
+// stores its counts; else counts are zeros before the launch and blocks of `span` tokens add theirs.  Negative positions mark idle rows,
 // which choose nothing (expert -1).  clear: z is zeroed.
 // ------------------------------------------------------------------------------------------------------------
 struct MoeRoute {
   float* z;  // [T, E]
   const float* correction;  // [E] or null
   const int* positions;     // [T] or null
-  int T, E, top, renorm, softmax, clear;
+  int T, E, top, renorm, softmax, clear, span;
   float gain;
   int* choice;   // [T, top]
   int* rank;     // [T, top]
@@ -30,74 +30,90 @@ struct MoeRoute {
 };
 
 template <bool ONE, int NI>  // NI: experts a lane
-__global__ void __launch_bounds__(ONE ? 1024 : 256)
+__global__ void __launch_bounds__(1024)
 moe_route_kernel(const MoeRoute p) {
-  __shared__ int cnt[ONE ? 32 * NI : 1];
+  __shared__ int cnt[32 * NI];   // tokens of this block per expert
+  __shared__ int base[ONE ? 1 : 32 * NI];
   pdl_launch_dependents();
   pdl_wait();
-  if (ONE) {
-    for (int e = threadIdx.x; e < p.E; e += blockDim.x) cnt[e] = 0;
-    __syncthreads();
-  }
-  const int lane = threadIdx.x & 31, per = blockDim.x >> 5;
-  for (int t = blockIdx.x * per + (threadIdx.x >> 5); t < p.T; t += gridDim.x * per) {
+  for (int e = threadIdx.x; e < p.E; e += blockDim.x) cnt[e] = 0;
+  __syncthreads();
+  const int lane = threadIdx.x & 31, per = blockDim.x >> 5, t_end = min(p.T, (int)(blockIdx.x + 1) * p.span);
+  for (int t = blockIdx.x * p.span + (threadIdx.x >> 5); t < t_end; t += per) {
     float* z = p.z + (size_t)t * p.E;
     const bool idle = p.positions != nullptr && p.positions[t] < 0;
-    float sc[NI];   // choice scores of experts lane, lane + 32, ...
-    float zmax = -INFINITY, zsum = 1.f;
+    float w[NI], sc[NI];   // scores of experts lane, lane + 32, ...: bare and as they are chosen by
+#pragma unroll
+    for (int i = 0; i < NI; ++i) w[i] = lane + 32 * i < p.E ? z[lane + 32 * i] : -INFINITY;
     if (p.softmax) {
-      for (int e = lane; e < p.E; e += 32) zmax = fmaxf(zmax, z[e]);
-      zmax = warp_max(zmax);
-      zsum = 0.f;
-      for (int e = lane; e < p.E; e += 32) zsum += expf(z[e] - zmax);
-      zsum = warp_sum(zsum);
+      float top = -INFINITY, sum = 0.f;
+#pragma unroll
+      for (int i = 0; i < NI; ++i) top = fmaxf(top, w[i]);
+      top = warp_max(top);
+#pragma unroll
+      for (int i = 0; i < NI; ++i) {
+        w[i] = lane + 32 * i < p.E ? expf(w[i] - top) : 0.f;
+        sum += w[i];
+      }
+      sum = warp_sum(sum);
+#pragma unroll
+      for (int i = 0; i < NI; ++i) w[i] /= sum;
+    } else {
+#pragma unroll
+      for (int i = 0; i < NI; ++i) w[i] = sigmoid_f(w[i]);
     }
-    auto score = [&](float v) { return p.softmax ? expf(v - zmax) / zsum : sigmoid_f(v); };
 #pragma unroll
     for (int i = 0; i < NI; ++i) {
       const int e = lane + 32 * i;
       sc[i] = -INFINITY;
       if (e < p.E) {
-        sc[i] = score(z[e]) + (p.correction != nullptr ? p.correction[e] : 0.f);
+        sc[i] = w[i] + (p.correction != nullptr ? p.correction[e] : 0.f);
         if (!(sc[i] > -INFINITY)) sc[i] = -3e38f;  // a NaN still has its place in the order
       }
     }
     float total = 0.f;
     for (int j = 0; j < p.top; ++j) {
-      float best = -INFINITY;
+      float best = -INFINITY, own = 0.f;
       int at = p.E;
 #pragma unroll
       for (int i = 0; i < NI; ++i) {
-        if (sc[i] > best) { best = sc[i]; at = lane + 32 * i; }
+        if (sc[i] > best) { best = sc[i]; at = lane + 32 * i; own = w[i]; }
       }
+      const int mine = at;
 #pragma unroll
       for (int o = 16; o > 0; o >>= 1) {
         const float ob = __shfl_xor_sync(0xffffffffu, best, o);
         const int oa = __shfl_xor_sync(0xffffffffu, at, o);
         if (ob > best || (ob == best && oa < at)) { best = ob; at = oa; }
       }
+      if (mine == at) {  // one lane
+        const size_t o = (size_t)t * p.top + j;
+        p.choice[o] = idle ? -1 : at;
+        p.weight[o] = own * p.gain;
+        if (!idle) p.rank[o] = atomicAdd(&cnt[at], 1);
+      }
+      total += __shfl_sync(0xffffffffu, own, at & 31);
 #pragma unroll
       for (int i = 0; i < NI; ++i) {
         if (at == lane + 32 * i) sc[i] = -INFINITY;
       }
-      if (lane == 0) {
-        const size_t o = (size_t)t * p.top + j;
-        const float w = score(z[at]);
-        p.choice[o] = idle ? -1 : at;
-        p.weight[o] = w * p.gain;
-        total += w;
-        if (!idle) p.rank[o] = ONE ? atomicAdd(&cnt[at], 1) : atomicAdd(&p.counts[at], 1);
-      }
     }
-    if (lane == 0 && p.renorm)
-      for (int j = 0; j < p.top; ++j) p.weight[(size_t)t * p.top + j] /= total + 1e-20f;
     __syncwarp();
+    if (p.renorm)
+      for (int j = lane; j < p.top; j += 32) p.weight[(size_t)t * p.top + j] /= total + 1e-20f;
     if (p.clear)
       for (int e = lane; e < p.E; e += 32) z[e] = 0.f;
   }
+  __syncthreads();
   if (ONE) {
-    __syncthreads();
     for (int e = threadIdx.x; e < p.E; e += blockDim.x) p.counts[e] = cnt[e];
+  } else {  // the block's rows of an expert follow those of the blocks that counted before it
+    for (int e = threadIdx.x; e < p.E; e += blockDim.x) base[e] = cnt[e] > 0 ? atomicAdd(&p.counts[e], cnt[e]) : 0;
+    __syncthreads();
+    for (long long i = (long long)blockIdx.x * p.span * p.top + threadIdx.x; i < (long long)t_end * p.top; i += blockDim.x) {
+      const int e = p.choice[i];
+      if (e >= 0) p.rank[i] += base[e];
+    }
   }
 }
 
@@ -235,9 +251,8 @@ TRLB_API int trlb_moe_route(float* z, const float* correction, const int* positi
                             float gain, int clear, int* choice, int* rank, float* weight, int* counts, cudaStream_t st) {
   if (T <= 0) return 0;
   if (E <= 0 || E > MR_MAX_E || top <= 0 || top > E) return -290;
-  const MoeRoute p = {z, correction, positions, T, E, top, renorm, softmax, clear, gain, choice, rank, weight, counts};
-  const int want = (T + 7) / 8, cap = trlb_host::sm_count() * 8;
-  const dim3 grid(T <= 128 ? 1 : want < cap ? want : cap), blk(T > 128 ? 256 : T >= 32 ? 1024 : T * 32);
+  const MoeRoute p = {z, correction, positions, T, E, top, renorm, softmax, clear, T <= 128 ? T : 32, gain, choice, rank, weight, counts};
+  const dim3 grid(T <= 128 ? 1 : (T + 31) / 32), blk(T > 128 ? (E <= 256 ? 512 : 256) : T >= 32 ? 1024 : T * 32);
 #define GO(ONE, NI) (int)trlb_host::launch_kernel(moe_route_kernel<ONE, NI>, grid, blk, 0, st, PDL, p)
 #define PICK(NI) (T <= 128 ? GO(true, NI) : GO(false, NI))
   return E <= 32 ? PICK(1) : E <= 64 ? PICK(2) : E <= 128 ? PICK(4) : E <= 256 ? PICK(8) : PICK(32);
