@@ -30,10 +30,6 @@ constexpr uint32_t HC_BOX = 128 * 64 * 2;  // 128 rows of 64 elements, 128-byte 
 struct Hgrn2Chunk {
   const int* cu;
   int n_seq, heads, dim, vdim;
-  const __nv_bfloat16* q;  // [T rows of y_ld], heads x dim
-  long long y_ld;
-  const float* z;          // [T rows of z_ld], heads x dim
-  long long z_ld;
   const float* bias;       // [heads dim]
   const float* low;
   __nv_bfloat16* s_hi;     // [chunks, heads, dim, vdim] state in front of a chunk, value and remainder; the first chunk of a
@@ -67,6 +63,25 @@ __device__ __forceinline__ void hc_put8(uint8_t* hi, uint8_t* lo, const float (&
   *reinterpret_cast<uint4*>(lo) = make_uint4(b[0], b[1], b[2], b[3]);
 }
 
+// The same to shared memory (32-bit addresses).
+__device__ __forceinline__ void hc_put8_smem(uint32_t hi, uint32_t lo, const float (&v)[8]) {
+  uint32_t a[4], b[4];
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    a[i] = pack_bf16(v[2 * i], v[2 * i + 1]);
+    const float2 f = unpack_bf16(a[i]);
+    b[i] = pack_bf16(v[2 * i] - f.x, v[2 * i + 1] - f.y);
+  }
+  asm volatile("st.shared.v4.b32 [%0], {%1, %2, %3, %4};" ::"r"(hi), "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]) : "memory");
+  asm volatile("st.shared.v4.b32 [%0], {%1, %2, %3, %4};" ::"r"(lo), "r"(b[0]), "r"(b[1]), "r"(b[2]), "r"(b[3]) : "memory");
+}
+
+// The value, unknown to the compiler: it must not keep partial products of one step in registers for another.
+__device__ __forceinline__ float hc_afresh(float w) {
+  asm volatile("" : "+f"(w));
+  return w;
+}
+
 template <int N>
 struct HcInt {
   static constexpr int value = N;
@@ -76,26 +91,50 @@ struct HcInt {
 template <int THREADS>
 __device__ __forceinline__ void hc_sync() { asm volatile("bar.sync 1, %0;" ::"n"(THREADS) : "memory"); }
 
-// ------------------------------------------------------------------------------------------------------------
-// State pass.  Warps 0-7: thread (channel, half of the tokens) forms the scaled keys, and as (row of S, half of the columns) scales the
-// state; warp 8: TMA; warp 9: MMA.
-// ------------------------------------------------------------------------------------------------------------
-constexpr int HS_THREADS = 320;
-constexpr size_t HS_SMEM = 6 * (size_t)HC_BOX + 1024 + 2048 + 256;
+// Gate logits of channel d at token t of a tile that came as four boxes of 32 channels (rows of 128 bytes, swizzled).
+__device__ __forceinline__ float hc_logit(uint32_t boxes, int d, int t) {
+  const uint32_t w = (uint32_t)d & 31;
+  float v;
+  asm volatile("ld.shared.f32 %0, [%1];"
+               : "=f"(v)
+               : "r"(boxes + (uint32_t)(d >> 5) * HC_BOX + (w & 3) * 4 + (((w >> 2) ^ ((uint32_t)t & 7)) << 4) + (uint32_t)t * 128)
+               : "memory");
+  return v;
+}
+// The same of queries, two boxes of 64 channels.
+__device__ __forceinline__ float hc_query(uint32_t boxes, int d, int t) {
+  const uint32_t w = (uint32_t)d & 63;
+  uint16_t v;
+  asm volatile("ld.shared.u16 %0, [%1];"
+               : "=h"(v)
+               : "r"(boxes + (uint32_t)(d >> 6) * HC_BOX + (w & 7) * 2 + (((w >> 3) ^ ((uint32_t)t & 7)) << 4) + (uint32_t)t * 128)
+               : "memory");
+  return __uint_as_float((uint32_t)v << 16);
+}
 
-__global__ void __launch_bounds__(HS_THREADS, 2)
-hgrn2_state_kernel(const __grid_constant__ CUtensorMap tm_v, const Hgrn2Chunk p) {
+// ------------------------------------------------------------------------------------------------------------
+// State pass.  Warps 0-15: thread (channel, quarter of the tokens) forms the scaled keys, warp (32 rows of S, 32 columns) scales the
+// state; warp 16: TMA; warp 17: MMA.  The gate logits of the next chunk arrive while the products of this one run.
+// ------------------------------------------------------------------------------------------------------------
+constexpr int HC_WORK = 512, HS_THREADS = HC_WORK + 64;
+constexpr size_t HS_SMEM = 12 * (size_t)HC_BOX + 1024 + 4096 + 256;
+
+__global__ void __launch_bounds__(HS_THREADS, 1)
+hgrn2_state_kernel(const __grid_constant__ CUtensorMap tm_z, const __grid_constant__ CUtensorMap tm_v, const Hgrn2Chunk p) {
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
-  uint8_t* k_hi = smem;                // two boxes of 64 tokens, rows are channels
-  uint8_t* k_lo = smem + 2 * HC_BOX;
-  uint8_t* v_s = smem + 4 * HC_BOX;    // two boxes of 64 columns, rows are tokens
-  float* prod = reinterpret_cast<float*>(smem + 6 * HC_BOX);  // [2][2][128] product of the gates of half a chunk
-  uint64_t* bars = reinterpret_cast<uint64_t*>(prod + 512);
-  uint64_t* v_full = bars;
-  uint64_t* ready = bars + 1;
-  uint64_t* acc_full = bars + 2;
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 3);
+  uint8_t* z_s = smem;                 // four boxes of 32 channels, rows are tokens
+  uint8_t* k_s = smem + 4 * HC_BOX;    // keys: two boxes of 64 tokens, rows are channels; then their remainders
+  uint8_t* v_s = smem + 8 * HC_BOX;    // two buffers of two boxes of 64 columns, rows are tokens
+  float* prod = reinterpret_cast<float*>(smem + 12 * HC_BOX);  // [2][4][128] product of the gates of a quarter
+  uint64_t* bars = reinterpret_cast<uint64_t*>(prod + 1024);
+  uint64_t* z_full = bars;
+  uint64_t* z_free = bars + 1;
+  uint64_t* v_full = bars + 2;   // [2]
+  uint64_t* v_free = bars + 4;   // [2]
+  uint64_t* ready = bars + 6;
+  uint64_t* acc_full = bars + 7;
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 8);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
 
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -106,14 +145,20 @@ hgrn2_state_kernel(const __grid_constant__ CUtensorMap tm_v, const Hgrn2Chunk p)
   const int cols = min(128, (p.vdim - e0 + 15) & ~15);
 
   if (tid == 0) {
-    mbar_init(v_full, 1);
-    mbar_init(ready, 256);
+    mbar_init(z_full, 1);
+    mbar_init(z_free, HC_WORK);
+    for (int i = 0; i < 2; ++i) {
+      mbar_init(&v_full[i], 1);
+      mbar_init(&v_free[i], 1);
+    }
+    mbar_init(ready, HC_WORK);
     mbar_init(acc_full, 1);
     *abort_flag = 0;
     mbar_fence_init();
+    tma_prefetch_desc(&tm_z);
     tma_prefetch_desc(&tm_v);
   }
-  if (warp == 9) {
+  if (warp == 17) {
     tmem_alloc(tmem_slot, 128);
     tmem_relinquish();
     tc_fence_before();
@@ -122,77 +167,86 @@ hgrn2_state_kernel(const __grid_constant__ CUtensorMap tm_v, const Hgrn2Chunk p)
   tc_fence_after();
   const uint32_t tmem_base = *tmem_slot;
 
-  if (warp == 8) {
+  if (warp == 16) {
     if (lane == 0) {
       for (int c = 0; c < nc; ++c) {
-        if (c > 0 && !mbar_wait(acc_full, (uint32_t)((c - 1) & 1), abort_flag, p.status, 2000)) break;
-        mbar_expect_tx(v_full, 2 * HC_BOX);
-        for (int i = 0; i < 2; ++i) tma_load_3d(v_s + i * HC_BOX, &tm_v, v_full, e0 + 64 * i, h, beg + c * HC_L);
+        const int b = c & 1;
+        if (c > 0 && !mbar_wait(z_free, (uint32_t)((c - 1) & 1), abort_flag, p.status, 2000)) break;
+        mbar_expect_tx(z_full, 4 * HC_BOX);
+        for (int i = 0; i < 4; ++i) tma_load_3d(z_s + i * HC_BOX, &tm_z, z_full, 64 * i, h, beg + c * HC_L);
+        if (c > 1 && !mbar_wait(&v_free[b], (uint32_t)(((c >> 1) - 1) & 1), abort_flag, p.status, 2001)) break;
+        mbar_expect_tx(&v_full[b], 2 * HC_BOX);
+        for (int i = 0; i < 2; ++i) tma_load_3d(v_s + (2 * b + i) * HC_BOX, &tm_v, &v_full[b], e0 + 64 * i, h, beg + c * HC_L);
       }
     }
     __syncwarp();
-  } else if (warp == 9) {
+  } else if (warp == 17) {
     if (lane == 0) {
       const uint32_t idesc = umma_idesc_bf16_major(128, cols, false, true);
-      const uint64_t ka = umma_desc_kmajor_sw128(smem_u32(k_hi)), vb = umma_desc_mnmajor_sw128(smem_u32(v_s), HC_BOX);
+      const uint64_t ka = umma_desc_kmajor_sw128(smem_u32(k_s)), vb = umma_desc_mnmajor_sw128(smem_u32(v_s), HC_BOX);
       for (int c = 0; c < nc; ++c) {
-        if (!mbar_wait(v_full, (uint32_t)(c & 1), abort_flag, p.status, 2010)) break;
+        const int b = c & 1;
+        if (!mbar_wait(&v_full[b], (uint32_t)((c >> 1) & 1), abort_flag, p.status, 2010)) break;
         if (!mbar_wait(ready, (uint32_t)(c & 1), abort_flag, p.status, 2011)) break;
         tc_fence_after();
+        const uint64_t vd = desc_at(vb, (uint32_t)b * 2 * HC_BOX);
 #pragma unroll
         for (int half = 0; half < 2; ++half)
 #pragma unroll
           for (int kk = 0; kk < HC_L / 16; ++kk)
-            umma_bf16_ss(tmem_base, desc_at(ka, (2 * half + (kk >> 2)) * HC_BOX) + 2 * (kk & 3), desc_at(vb, kk * 2048), idesc,
+            umma_bf16_ss(tmem_base, desc_at(ka, (2 * half + (kk >> 2)) * HC_BOX) + 2 * (kk & 3), desc_at(vd, kk * 2048), idesc,
                          c > 0 || (half | kk) != 0);
+        umma_commit(&v_free[b]);
         umma_commit(acc_full);
       }
     }
     __syncwarp();
   } else {
-    const int d = tid & 127, half = tid >> 7, hd = h * p.dim + d;
+    const int d = tid & 127, qt = tid >> 7, x0 = 32 * qt;  // also: this warp's columns of S
     const bool on = d < p.dim;
-    const float bias = on ? p.bias[hd] : 0.f, room = on ? 1.f - p.low[hd] : 0.f;
-    const uint32_t t_row = tmem_base + ((uint32_t)((warp & 3) * 32) << 16) + (uint32_t)half * 64;
-    uint8_t* hi = k_hi + (size_t)half * HC_BOX + (size_t)d * 128;
-    uint8_t* lo = k_lo + (size_t)half * HC_BOX + (size_t)d * 128;
+    const int hd = h * p.dim + (on ? d : 0);
+    const float bias = p.bias[hd], room = 1.f - p.low[hd];
+    const uint32_t t_row = tmem_base + ((uint32_t)((warp & 3) * 32) << 16) + (uint32_t)x0;
+    uint8_t* keys = k_s + (size_t)(qt >> 1) * HC_BOX + (size_t)d * 128;
     bool ok = true;
     for (int c = 0; c < nc; ++c) {
-      const int t0 = c * HC_L + half * 64;
-      const float* z = p.z + (size_t)(beg + t0) * p.z_ld + hd;
-      float k[64], all = 1.f;
+      const int n = on ? len - c * HC_L - 32 * qt : 0;  // tokens here
+      float k[32], all = 1.f;
+      ok = ok && __all_sync(0xffffffffu, mbar_wait(z_full, (uint32_t)(c & 1), abort_flag, p.status, 2020));
 #pragma unroll
-      for (int i = 0; i < 64; ++i) k[i] = on && t0 + i < len ? z[(size_t)i * p.z_ld] : 0.f;
+      for (int i = 0; i < 32; ++i) k[i] = hc_logit(smem_u32(z_s), d, 32 * qt + i);
 #pragma unroll
-      for (int i = 0; i < 64; ++i) {
-        k[i] = on && t0 + i < len ? __fdividef(room, 1.f + hc_exp(k[i] + bias)) : 0.f;
-        all *= 1.f - k[i];
+      for (int i = 0; i < 32; ++i) {
+        k[i] = i < n ? __fdividef(room, 1.f + hc_exp(k[i] + bias)) : 0.f;
+        all = fmaf(-k[i], all, all);
       }
-      float* pr = prod + (c & 1) * 256;
-      pr[half * 128 + d] = all;
-      hc_sync<256>();
-      const float later = half == 0 ? pr[128 + d] : 1.f, decay = pr[d] * pr[128 + d];
+      mbar_arrive(z_free);
+      float* pr = prod + (c & 1) * 512 + d;
+      pr[128 * qt] = all;
+      hc_sync<HC_WORK>();
+      float w = 1.f;  // the gates of the quarters behind this one
+      for (int i = 3; i > qt; --i) w *= pr[128 * i];
+      const float decay = (pr[0] * pr[128]) * (pr[256] * pr[384]);
       // the products of the chunk before have read the keys and left the state
-      if (c > 0) ok = ok && __all_sync(0xffffffffu, mbar_wait(acc_full, (uint32_t)((c - 1) & 1), abort_flag, p.status, 2020));
+      if (c > 0) ok = ok && __all_sync(0xffffffffu, mbar_wait(acc_full, (uint32_t)((c - 1) & 1), abort_flag, p.status, 2021));
       if (!ok) continue;
       tc_fence_after();
-      float w = later;
 #pragma unroll
-      for (int g = 7; g >= 0; --g) {
+      for (int g = 3; g >= 0; --g) {
         float v[8];
 #pragma unroll
         for (int i = 7; i >= 0; --i) {
           v[i] = k[8 * g + i] * w;
-          w *= 1.f - k[8 * g + i];
+          w = fmaf(-k[8 * g + i], w, w);
         }
-        const int at = (g ^ (d & 7)) << 4;
-        hc_put8(hi + at, lo + at, v);
+        const int at = (((qt & 1) * 4 + g) ^ (d & 7)) << 4;
+        hc_put8(keys + at, keys + 2 * HC_BOX + at, v);
       }
       fence_proxy_async_smem();
-      if (c > 0 && half * 64 < cols) {
-        const size_t row = (((size_t)(chunk0 + c) * p.heads + h) * p.dim + d) * p.vdim + e0 + half * 64;
+      if (c > 0 && x0 < cols) {
+        const size_t row = (((size_t)(chunk0 + c) * p.heads + h) * p.dim + d) * p.vdim + e0 + x0;
 #pragma unroll 1
-        for (int x = 0; x < 64; x += 16) {
+        for (int x = 0; x < 32; x += 16) {
           float s[16];
           tmem_ld_32x16(t_row + x, s);
           tmem_ld_wait();
@@ -202,7 +256,7 @@ hgrn2_state_kernel(const __grid_constant__ CUtensorMap tm_v, const Hgrn2Chunk p)
           tmem_st_32x16(t_row + x, u);
 #pragma unroll
           for (int y = 0; y < 16; y += 8) {
-            if (on && e0 + half * 64 + x + y < p.vdim) {
+            if (on && e0 + x0 + x + y < p.vdim) {
               const float v[8] = {s[y], s[y + 1], s[y + 2], s[y + 3], s[y + 4], s[y + 5], s[y + 6], s[y + 7]};
               hc_put8(reinterpret_cast<uint8_t*>(p.s_hi + row + x + y), reinterpret_cast<uint8_t*>(p.s_lo + row + x + y), v);
             }
@@ -213,20 +267,20 @@ hgrn2_state_kernel(const __grid_constant__ CUtensorMap tm_v, const Hgrn2Chunk p)
       tc_fence_before();
       mbar_arrive(ready);
     }
-    if (ok && nc > 0) {
-      ok = __all_sync(0xffffffffu, mbar_wait(acc_full, (uint32_t)((nc - 1) & 1), abort_flag, p.status, 2030));
+    if (nc > 0) {
+      ok = ok && __all_sync(0xffffffffu, mbar_wait(acc_full, (uint32_t)((nc - 1) & 1), abort_flag, p.status, 2030));
       const int slot = p.seq_slot != nullptr ? p.seq_slot[seq] : -1;
-      if (ok && slot >= 0 && slot < p.slots && half * 64 < cols) {
+      if (ok && slot >= 0 && slot < p.slots && x0 < cols) {
         tc_fence_after();
-        float* dst = p.S + (((size_t)slot * p.heads + h) * p.dim + d) * p.vdim + e0 + half * 64;
+        float* dst = p.S + (((size_t)slot * p.heads + h) * p.dim + d) * p.vdim + e0 + x0;
 #pragma unroll 1
-        for (int x = 0; x < 64; x += 16) {
+        for (int x = 0; x < 32; x += 16) {
           float s[16];
           tmem_ld_32x16(t_row + x, s);
           tmem_ld_wait();
 #pragma unroll
           for (int i = 0; i < 16; i += 4)
-            if (on && e0 + half * 64 + x + i < p.vdim) store4(dst + x + i, make_float4(s[i], s[i + 1], s[i + 2], s[i + 3]));
+            if (on && e0 + x0 + x + i < p.vdim) store4(dst + x + i, make_float4(s[i], s[i + 1], s[i + 2], s[i + 3]));
         }
         tc_fence_before();
       }
@@ -238,27 +292,27 @@ hgrn2_state_kernel(const __grid_constant__ CUtensorMap tm_v, const Hgrn2Chunk p)
     while (globaltimer_ns() - t0 < 200000ull) __nanosleep(1000);
     __syncthreads();
   }
-  if (warp == 9) {
+  if (warp == 17) {
     tc_fence_after();
     tmem_dealloc(tmem_base, 128);
   }
 }
 
 // ------------------------------------------------------------------------------------------------------------
-// Output pass.  Warps 0-15: thread (channel, quarter of the tokens) holds its keys and queries in registers and writes them, scaled,
-// level by level (rows of the operands are channels: eight tokens are one 16-byte store); later warp (32 queries, 32 keys) turns the
-// levels' products into scores, and (32 queries, 32 columns) norms the output.  Warp 16: TMA; warp 17: MMA.  Every barrier is used once.
+// Output pass.  Warps 0-7: thread (channel, half of the tokens) holds its keys and queries in registers and writes them, scaled,
+// level by level (rows of the operands are channels: eight tokens are one 16-byte store); later warp (32 queries, 64 keys) turns the
+// levels' products into scores, and (32 queries, 64 columns) norms the output.  Warp 8: TMA; warp 9: MMA.  Every barrier is used once.
 //
-// Steps: 0 blocks of 8, 1 - 4 levels of 64, 32, 16, 8, 5 queries against the state.  Two slots of shared memory (queries 64 KB, keys
+// Gate logits and queries come to slot 1 and go to registers.  Steps: 0 blocks of 8, 1 - 4 levels of 64, 32, 16, 8, 5 queries against the state.  Two slots of shared memory (queries 64 KB, keys
 // 32 KB, value and remainder each) and 32 KB more for the keys 64 .. 127 of step 0, where v goes later; the state goes where keys were.
 // TMEM: levels [0, 256), blocks of 8 [256, 384), output [384, 512); the scores replace the levels of 64 and 32.
 // ------------------------------------------------------------------------------------------------------------
-constexpr int HO_WORK = 512, HO_THREADS = HO_WORK + 64;
+constexpr int HO_WORK = 256, HO_THREADS = HO_WORK + 64;
 constexpr uint32_t HO_SLOT = 6 * HC_BOX;
-constexpr size_t HO_SMEM = 2 * (size_t)HO_SLOT + 2 * HC_BOX + 1024 + 1536 + 256;
+constexpr size_t HO_SMEM = 2 * (size_t)HO_SLOT + 2 * HC_BOX + 1024 + 512 + 256;
 
 __global__ void __launch_bounds__(HO_THREADS, 1)
-hgrn2_output_kernel(const __grid_constant__ CUtensorMap tm_v, const __grid_constant__ CUtensorMap tm_sh, const __grid_constant__ CUtensorMap tm_sl,
+hgrn2_output_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_z, const __grid_constant__ CUtensorMap tm_v, const __grid_constant__ CUtensorMap tm_sh, const __grid_constant__ CUtensorMap tm_sl,
                     const Hgrn2Chunk p) {
   int seq = -1, c = (int)blockIdx.x;
   for (int s = 0; s < p.n_seq; ++s) {
@@ -271,15 +325,16 @@ hgrn2_output_kernel(const __grid_constant__ CUtensorMap tm_v, const __grid_const
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   // a slot: queries [2 groups of 64 tokens] value, remainder, keys [64 tokens] value, remainder
   uint8_t* x_s = smem + 2 * HO_SLOT;
-  float* prod = reinterpret_cast<float*>(x_s + 2 * HC_BOX);  // [3][128] product of the gates of a quarter
-  uint64_t* bars = reinterpret_cast<uint64_t*>(prod + 384);
+  float* prod = reinterpret_cast<float*>(x_s + 2 * HC_BOX);  // [128] product of the gates of the first half
+  uint64_t* bars = reinterpret_cast<uint64_t*>(prod + 128);
   uint64_t* full = bars;        // [6] operands of a step written
   uint64_t* done = bars + 6;    // [5] its products done
   uint64_t* v_full = bars + 11;
   uint64_t* s_full = bars + 12;
   uint64_t* p_full = bars + 13;
   uint64_t* o_full = bars + 14;
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 15);
+  uint64_t* in_full = bars + 15;
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 16);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
 
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -295,13 +350,16 @@ hgrn2_output_kernel(const __grid_constant__ CUtensorMap tm_v, const __grid_const
     mbar_init(s_full, 1);
     mbar_init(p_full, HO_WORK);
     mbar_init(o_full, 1);
+    mbar_init(in_full, 1);
     *abort_flag = 0;
     mbar_fence_init();
+    tma_prefetch_desc(&tm_q);
+    tma_prefetch_desc(&tm_z);
     tma_prefetch_desc(&tm_v);
     tma_prefetch_desc(&tm_sh);
     tma_prefetch_desc(&tm_sl);
   }
-  if (warp == 17) {
+  if (warp == 9) {
     tmem_alloc(tmem_slot, 512);
     tmem_relinquish();
     tc_fence_before();
@@ -313,8 +371,11 @@ hgrn2_output_kernel(const __grid_constant__ CUtensorMap tm_v, const __grid_const
   uint8_t* s_hi_s = smem + HO_SLOT + 4 * HC_BOX;
   uint8_t* s_lo_s = smem + 4 * HC_BOX;
 
-  if (warp == 16) {
+  if (warp == 8) {
     if (lane == 0) {
+      mbar_expect_tx(in_full, 6 * HC_BOX);
+      for (int i = 0; i < 4; ++i) tma_load_3d(smem + HO_SLOT + i * HC_BOX, &tm_z, in_full, 64 * i, h, row0);
+      for (int i = 0; i < 2; ++i) tma_load_3d(smem + HO_SLOT + (4 + i) * HC_BOX, &tm_q, in_full, 64 * i, h, row0);
       if (mbar_wait(&done[0], 0, abort_flag, p.status, 2100)) {
         mbar_expect_tx(v_full, 2 * HC_BOX);
         for (int i = 0; i < 2; ++i) tma_load_3d(x_s + i * HC_BOX, &tm_v, v_full, e0 + 64 * i, h, row0);
@@ -327,7 +388,7 @@ hgrn2_output_kernel(const __grid_constant__ CUtensorMap tm_v, const __grid_const
       }
     }
     __syncwarp();
-  } else if (warp == 17) {
+  } else if (warp == 9) {
     if (lane == 0) {
       constexpr uint32_t idesc_s = umma_idesc_bf16_major(128, 64, true, true);
       const uint32_t idesc_x = umma_idesc_bf16_major(128, cols, true, true), idesc_o = umma_idesc_bf16_major(128, cols, false, true);
@@ -365,8 +426,7 @@ hgrn2_output_kernel(const __grid_constant__ CUtensorMap tm_v, const __grid_const
           for (int part = 0; part < 3; ++part) {
             const uint64_t da = desc_at(base, HO_SLOT + (part == 2 ? 2 * HC_BOX : 0)), db = desc_at(base, part == 1 ? s_lo : s_hi);
 #pragma unroll 1
-            for (int kk = 0; kk < ksteps; ++kk)
-              umma_bf16_ss(tmem_base + 384, desc_at(da, kk * 2048), desc_at(db, kk * 2048), idesc_x, (part | kk) != 0);
+            for (int kk = 0; kk < ksteps; ++kk) umma_bf16_ss(tmem_base + 384, desc_at(da, kk * 2048), desc_at(db, kk * 2048), idesc_x, (part | kk) != 0);
           }
         }
       }
@@ -384,66 +444,61 @@ hgrn2_output_kernel(const __grid_constant__ CUtensorMap tm_v, const __grid_const
     }
     __syncwarp();
   } else {
-    const int d = tid & 127, qt = tid >> 7, hd = h * p.dim + d;  // the quarter is the same for a whole warp
-    float k[32], q[32];
+    const int d = tid & 127, half = tid >> 7;
+    float k[64], q[64];
+    bool ok = __all_sync(0xffffffffu, mbar_wait(in_full, 0, abort_flag, p.status, 2131));
     {
       const bool on = d < p.dim;
-      const float bias = on ? p.bias[hd] : 0.f, room = on ? 1.f - p.low[hd] : 0.f;
-      const int n = on ? min(32, len - c * HC_L - 32 * qt) : 0;  // tokens here
-      const float* z = p.z + (size_t)(row0 + 32 * qt) * p.z_ld + hd;
-      const __nv_bfloat16* qr = p.q + (size_t)(row0 + 32 * qt) * p.y_ld + hd;
-#pragma unroll
-      for (int i = 0; i < 32; ++i) {
-        k[i] = i < n ? z[(size_t)i * p.z_ld] : 0.f;
-        q[i] = i < n ? __bfloat162float(qr[(size_t)i * p.y_ld]) : 0.f;
-      }
+      const int hd = h * p.dim + (on ? d : 0), n = on ? len - c * HC_L - 64 * half : 0;  // tokens here
+      const float bias = p.bias[hd], room = 1.f - p.low[hd];
       float all = 1.f;
 #pragma unroll
-      for (int i = 0; i < 32; ++i) {  // silu(q) and (1 - low) sigmoid(-z - bias) with one division
-        const float a = 1.f + hc_exp(-q[i]), b = 1.f + hc_exp(k[i] + bias), r = __fdividef(1.f, a * b);
-        q[i] *= r * b;
+      for (int i = 0; i < 64; ++i) {  // silu(q) and (1 - low) sigmoid(-z - bias) with one division
+        const float z = hc_logit(smem_u32(smem) + HO_SLOT, d, 64 * half + i), x = hc_query(smem_u32(smem) + HO_SLOT + 4 * HC_BOX, d, 64 * half + i);
+        const float a = 1.f + hc_exp(-x), b = 1.f + hc_exp(z + bias), r = __fdividef(1.f, a * b);
+        q[i] = i < n ? x * (r * b) : 0.f;
         k[i] = i < n ? room * (r * a) : 0.f;
-        all *= 1.f - k[i];
+        all = fmaf(-k[i], all, all);
       }
-      if (qt < 3) prod[qt * 128 + d] = all;
+      if (half == 0) prod[d] = all;
     }
-    hc_sync<HO_WORK>();
-    const uint32_t sw = (uint32_t)(d & 7), row = (uint32_t)d * 128;
+    hc_sync<HO_WORK>();  // slot 1 is free
+    const uint32_t sw = (uint32_t)(d & 7), row = smem_u32(smem) + (uint32_t)d * 128;
     auto chunk16 = [&](uint32_t g) { return row + ((g ^ sw) << 4); };  // eight tokens, number g of a group of 64
-    // queries i0 .. i0 + n - 1 of this quarter times the gates from i0 on (and w)
-    auto queries = [&](uint8_t* slot, auto i0c, auto nc, float w) {
+    const uint32_t mine = (uint32_t)half * HC_BOX;  // this half's group of queries
+    // queries i0 .. i0 + n - 1 of this half times the gates from i0 on (and w)
+    auto queries = [&](uint32_t slot, auto i0c, auto nc, float w) {
       constexpr int i0 = decltype(i0c)::value, n = decltype(nc)::value;
-      uint8_t* a = slot + (size_t)(qt >> 1) * HC_BOX;
+      w = hc_afresh(w);
 #pragma unroll
       for (int g = 0; g < n / 8; ++g) {
         float v[8];
 #pragma unroll
         for (int i = 0; i < 8; ++i) {
-          w *= 1.f - k[i0 + 8 * g + i];
+          w = fmaf(-k[i0 + 8 * g + i], w, w);
           v[i] = q[i0 + 8 * g + i] * w;
         }
-        const uint32_t at = chunk16((uint32_t)((qt & 1) * 4 + i0 / 8 + g));
-        hc_put8(a + at, a + 2 * HC_BOX + at, v);
+        const uint32_t at = chunk16((uint32_t)(i0 / 8 + g)) + mine + slot;
+        hc_put8_smem(at, at + 2 * HC_BOX, v);
       }
     };
-    // keys i0 .. i0 + n - 1 times the gates behind them up to i0 + n - 1 (and w); g0: where they begin among the 64 of the level
-    auto keys = [&](uint8_t* slot, auto i0c, auto nc, float w, int g0) {
+    // keys i0 .. i0 + n - 1 times the gates behind them up to i0 + n - 1; g0: where they begin among the 64 of the level
+    auto keys = [&](uint32_t slot, auto i0c, auto nc, int g0) {
       constexpr int i0 = decltype(i0c)::value, n = decltype(nc)::value;
-      uint8_t* b = slot + 4 * HC_BOX;
+      float w = hc_afresh(1.f);
 #pragma unroll
       for (int g = n / 8 - 1; g >= 0; --g) {
         float v[8];
 #pragma unroll
         for (int i = 7; i >= 0; --i) {
           v[i] = k[i0 + 8 * g + i] * w;
-          w *= 1.f - k[i0 + 8 * g + i];
+          w = fmaf(-k[i0 + 8 * g + i], w, w);
         }
-        const uint32_t at = chunk16((uint32_t)(g0 + g));
-        hc_put8(b + at, b + HC_BOX + at, v);
+        const uint32_t at = chunk16((uint32_t)(g0 + g)) + slot + 4 * HC_BOX;
+        hc_put8_smem(at, at + HC_BOX, v);
       }
     };
-    uint8_t* slot0 = smem;
-    uint8_t* slot1 = smem + HO_SLOT;
+    constexpr uint32_t slot0 = 0, slot1 = HO_SLOT;
     auto filled = [&](int s) {
       fence_proxy_async_smem();
       mbar_arrive(&full[s]);
@@ -452,105 +507,125 @@ hgrn2_output_kernel(const __grid_constant__ CUtensorMap tm_v, const __grid_const
 
     // step 0: about the middle of every block of 8 (behind its fourth token)
     {
-      uint8_t* a = slot0 + (size_t)(qt >> 1) * HC_BOX;
-      uint8_t* b = qt < 2 ? slot0 + 4 * HC_BOX : x_s;
+      const uint32_t b = half == 0 ? slot0 + 4 * HC_BOX : 2 * HO_SLOT;
 #pragma unroll
-      for (int g = 0; g < 4; ++g) {
-        float f[8], up[8], vq[8], vk[8];  // up: gates from the middle to the token, down to it: their inverse
+      for (int g = 0; g < 8; ++g) {
+        auto gate = [&](int i) { return fmaxf(1.f - hc_afresh(k[8 * g + i]), 5.9604644775390625e-8f); };
+        const uint32_t at = chunk16((uint32_t)g);
+        // products of the gates from the middle to the ends of the block, and their inverses
+        const float low = gate(1) * gate(2) * gate(3), high = gate(4) * gate(5) * gate(6) * gate(7);
+        float v[8], w = __fdividef(1.f, low);
 #pragma unroll
-        for (int i = 1; i < 8; ++i) f[i] = fmaxf(1.f - k[8 * g + i], 5.9604644775390625e-8f);
-        up[3] = 1.f;
-        up[2] = f[3];
-        up[1] = f[3] * f[2];
-        up[0] = up[1] * f[1];
-        up[4] = f[4];
-        up[5] = f[4] * f[5];
-        up[6] = up[5] * f[6];
-        up[7] = up[6] * f[7];
-#pragma unroll
-        for (int i = 0; i < 8; ++i) {
-          const float inv = i == 3 ? 1.f : __fdividef(1.f, up[i]);
-          vq[i] = q[8 * g + i] * (i < 4 ? inv : up[i]);
-          vk[i] = k[8 * g + i] * (i < 4 ? up[i] : inv);
+        for (int i = 0; i < 4; ++i) {
+          v[i] = q[8 * g + i] * w;
+          if (i < 3) w *= gate(i + 1);
         }
-        const uint32_t at = chunk16((uint32_t)((qt & 1) * 4 + g));
-        hc_put8(a + at, a + 2 * HC_BOX + at, vq);
-        hc_put8(b + at, b + HC_BOX + at, vk);
+        w = 1.f;
+#pragma unroll
+        for (int i = 4; i < 8; ++i) {
+          w *= gate(i);
+          v[i] = q[8 * g + i] * w;
+        }
+        hc_put8_smem(at + mine + slot0, at + mine + slot0 + 2 * HC_BOX, v);
+        w = hc_afresh(__fdividef(1.f, high));
+#pragma unroll
+        for (int i = 7; i >= 4; --i) {
+          v[i] = k[8 * g + i] * w;
+          w *= gate(i);
+        }
+        w = hc_afresh(1.f);
+#pragma unroll
+        for (int i = 3; i >= 0; --i) {
+          v[i] = k[8 * g + i] * w;
+          w *= gate(i);
+        }
+        hc_put8_smem(at + b, at + b + HC_BOX, v);
       }
     }
     filled(0);
-    // steps 1 and 2: quarters are queries or keys as a whole
-    if (qt < 2) keys(slot1, HcInt<0>{}, HcInt<32>{}, qt == 0 ? prod[128 + d] : 1.f, 4 * qt);
-    else queries(slot1, HcInt<0>{}, HcInt<32>{}, qt == 3 ? prod[256 + d] : 1.f);
+    // step 1: the halves are keys or queries as a whole
+    if (half == 0) keys(slot1, HcInt<0>{}, HcInt<64>{}, 0);
+    else queries(slot1, HcInt<0>{}, HcInt<64>{}, 1.f);
     filled(1);
-    bool ok = emptied(0);
+    ok = ok && emptied(0);
     if (ok) {
-      if (qt & 1) queries(slot0, HcInt<0>{}, HcInt<32>{}, 1.f);
-      else keys(slot0, HcInt<0>{}, HcInt<32>{}, 1.f, 2 * qt);
+      keys(slot0, HcInt<0>{}, HcInt<32>{}, 4 * half);
+      queries(slot0, HcInt<32>{}, HcInt<32>{}, 1.f);
       filled(2);
       ok = emptied(1);
     }
     if (ok) {
-      keys(slot1, HcInt<0>{}, HcInt<16>{}, 1.f, 2 * qt);
+      keys(slot1, HcInt<0>{}, HcInt<16>{}, 4 * half);
       queries(slot1, HcInt<16>{}, HcInt<16>{}, 1.f);
+      keys(slot1, HcInt<32>{}, HcInt<16>{}, 4 * half + 2);
+      queries(slot1, HcInt<48>{}, HcInt<16>{}, 1.f);
       filled(3);
       ok = emptied(2);
     }
     if (ok) {
-      keys(slot0, HcInt<0>{}, HcInt<8>{}, 1.f, 2 * qt);
+      keys(slot0, HcInt<0>{}, HcInt<8>{}, 4 * half);
       queries(slot0, HcInt<8>{}, HcInt<8>{}, 1.f);
-      keys(slot0, HcInt<16>{}, HcInt<8>{}, 1.f, 2 * qt + 1);
+      keys(slot0, HcInt<16>{}, HcInt<8>{}, 4 * half + 1);
       queries(slot0, HcInt<24>{}, HcInt<8>{}, 1.f);
+      keys(slot0, HcInt<32>{}, HcInt<8>{}, 4 * half + 2);
+      queries(slot0, HcInt<40>{}, HcInt<8>{}, 1.f);
+      keys(slot0, HcInt<48>{}, HcInt<8>{}, 4 * half + 3);
+      queries(slot0, HcInt<56>{}, HcInt<8>{}, 1.f);
       filled(4);
       ok = emptied(3);
     }
     if (ok && carried) {
-      float w = 1.f;
-      for (int i = 0; i < qt; ++i) w *= prod[i * 128 + d];
-      queries(slot1, HcInt<0>{}, HcInt<32>{}, w);
+      queries(slot1, HcInt<0>{}, HcInt<64>{}, half == 0 ? 1.f : prod[d]);
       filled(5);
     }
     if (ok) ok = emptied(4);
-    // scores: warp (queries 32 rq .., keys 32 kq ..)
-    const int rq = warp & 3, kq = warp >> 2;
+    // scores: warp (queries 32 rq .., keys 64 kh ..)
+    const int rq = warp & 3, kh = warp >> 2;
     const uint32_t t_lane = tmem_base + ((uint32_t)(rq * 32) << 16);
-    uint32_t a[16], b[16];
+    uint32_t a[2][16], b[2][16];
     if (ok) {
       tc_fence_after();
-      float v[32];
-      if (kq < rq) {
-        tmem_ld_32x32(t_lane + (uint32_t)(rq >= 2 && kq < 2 ? 32 * kq : 64 + 32 * (rq >> 1)), v);
-        tmem_ld_wait();
-      } else if (kq == rq) {
-        float l16[16], l8[16];
-        tmem_ld_32x32(t_lane + 256 + 32 * rq, v);
-        tmem_ld_32x16(t_lane + 128 + 16 * rq, l16);
-        tmem_ld_32x16(t_lane + 192 + 16 * rq, l8);
-        tmem_ld_wait();
 #pragma unroll
-        for (int x = 0; x < 32; ++x) {
-          float s = v[x];  // same block of 8
-          if ((lane >> 3) != (x >> 3) && (x & 15) < 8) s = l8[8 * (x >> 4) + (x & 7)];
-          if (x < 16 && lane >= 16) s = l16[x & 15];
-          v[x] = x <= lane ? s : 0.f;
+      for (int j = 0; j < 2; ++j) {
+        const int kq = 2 * kh + j;
+        float v[32];
+        if (kq < rq) {
+          tmem_ld_32x32(t_lane + (uint32_t)(rq >= 2 && kq < 2 ? 32 * kq : 64 + 32 * (rq >> 1)), v);
+          tmem_ld_wait();
+        } else if (kq == rq) {
+          float l16[16], l8[16];
+          tmem_ld_32x32(t_lane + 256 + 32 * rq, v);
+          tmem_ld_32x16(t_lane + 128 + 16 * rq, l16);
+          tmem_ld_32x16(t_lane + 192 + 16 * rq, l8);
+          tmem_ld_wait();
+#pragma unroll
+          for (int x = 0; x < 32; ++x) {
+            float s = v[x];  // same block of 8
+            if ((lane >> 3) != (x >> 3) && (x & 15) < 8) s = l8[8 * (x >> 4) + (x & 7)];
+            if (x < 16 && lane >= 16) s = l16[x & 15];
+            v[x] = x <= lane ? s : 0.f;
+          }
+        } else {
+#pragma unroll
+          for (int x = 0; x < 32; ++x) v[x] = 0.f;
         }
-      } else {
 #pragma unroll
-        for (int x = 0; x < 32; ++x) v[x] = 0.f;
-      }
-#pragma unroll
-      for (int i = 0; i < 16; ++i) {
-        a[i] = pack_bf16(v[2 * i], v[2 * i + 1]);
-        const float2 f = unpack_bf16(a[i]);
-        b[i] = pack_bf16(v[2 * i] - f.x, v[2 * i + 1] - f.y);
+        for (int i = 0; i < 16; ++i) {
+          a[j][i] = pack_bf16(v[2 * i], v[2 * i + 1]);
+          const float2 f = unpack_bf16(a[j][i]);
+          b[j][i] = pack_bf16(v[2 * i] - f.x, v[2 * i + 1] - f.y);
+        }
       }
       tc_fence_before();
     }
     hc_sync<HO_WORK>();  // every warp has read what the scores replace
     if (ok) {
       tc_fence_after();
-      tmem_st_32x16(t_lane + 16 * kq, a);
-      tmem_st_32x16(t_lane + 64 + 16 * kq, b);
+#pragma unroll
+      for (int j = 0; j < 2; ++j) {
+        tmem_st_32x16(t_lane + 16 * (2 * kh + j), a[j]);
+        tmem_st_32x16(t_lane + 64 + 16 * (2 * kh + j), b[j]);
+      }
       tmem_st_wait();
       tc_fence_before();
       mbar_arrive(p_full);
@@ -558,40 +633,43 @@ hgrn2_output_kernel(const __grid_constant__ CUtensorMap tm_v, const __grid_const
     }
     {
       tc_fence_after();
-      const int t = c * HC_L + 32 * rq + lane, x0 = 32 * kq;  // this warp's columns
+      const int t = c * HC_L + 32 * rq + lane, x0 = 64 * kh;  // this warp's columns
       const bool row_ok = ok && t < len;
-      float o[32], ss = 0.f;
+      float o[2][32], ss = 0.f;
       if (ok && x0 < cols) {
-        tmem_ld_32x32(t_lane + 384 + x0, o);
+        tmem_ld_32x32(t_lane + 384 + x0, o[0]);
+        tmem_ld_32x32(t_lane + 416 + x0, o[1]);
         tmem_ld_wait();
       }
       if (p.norm != nullptr) {
-        float* red = reinterpret_cast<float*>(smem);  // [4][128]: nothing reads the operands any more
+        float* red = reinterpret_cast<float*>(smem);  // [2][128]: nothing reads the operands any more
         if (ok && x0 < cols) {
 #pragma unroll
-          for (int x = 0; x < 32; ++x) ss += x0 + x < p.vdim ? o[x] * o[x] : 0.f;
+          for (int x = 0; x < 64; ++x) ss += x0 + x < p.vdim ? o[x >> 5][x & 31] * o[x >> 5][x & 31] : 0.f;
         }
-        red[kq * 128 + 32 * rq + lane] = ss;
+        red[kh * 128 + 32 * rq + lane] = ss;
         hc_sync<HO_WORK>();
         const float* r = red + 32 * rq + lane;
-        const float f = p.scale / sqrtf((r[0] + r[128] + r[256] + r[384]) / (float)p.vdim + p.eps);
+        const float f = p.scale / sqrtf((r[0] + r[128]) / (float)p.vdim + p.eps);
         if (row_ok) {
           __nv_bfloat16* y = p.y_out + (size_t)(beg + t) * p.out_ld + (size_t)h * p.vdim + x0;
 #pragma unroll
-          for (int x = 0; x < 32; x += 8) {
+          for (int x = 0; x < 64; x += 8) {
             if (x0 + x < p.vdim) {
+              const float* u = &o[x >> 5][x & 31];
               const float4 g = load4(p.norm + x0 + x), g2 = load4(p.norm + x0 + x + 4);
-              *reinterpret_cast<uint4*>(y + x) =
-                  make_uint4(pack_bf16(o[x] * f * g.x, o[x + 1] * f * g.y), pack_bf16(o[x + 2] * f * g.z, o[x + 3] * f * g.w),
-                             pack_bf16(o[x + 4] * f * g2.x, o[x + 5] * f * g2.y), pack_bf16(o[x + 6] * f * g2.z, o[x + 7] * f * g2.w));
+              *reinterpret_cast<uint4*>(y + x) = make_uint4(pack_bf16(u[0] * f * g.x, u[1] * f * g.y), pack_bf16(u[2] * f * g.z, u[3] * f * g.w),
+                                                            pack_bf16(u[4] * f * g2.x, u[5] * f * g2.y), pack_bf16(u[6] * f * g2.z, u[7] * f * g2.w));
             }
           }
         }
       } else if (row_ok) {
         float* dst = p.out + ((size_t)(beg + t) * p.heads + h) * p.vdim + e0 + x0;
 #pragma unroll
-        for (int x = 0; x < 32; x += 4)
-          if (e0 + x0 + x < p.vdim) store4(dst + x, make_float4(o[x], o[x + 1], o[x + 2], o[x + 3]));
+        for (int x = 0; x < 64; x += 4) {
+          const float* u = &o[x >> 5][x & 31];
+          if (e0 + x0 + x < p.vdim) store4(dst + x, make_float4(u[0], u[1], u[2], u[3]));
+        }
       }
       tc_fence_before();
     }
@@ -602,7 +680,7 @@ hgrn2_output_kernel(const __grid_constant__ CUtensorMap tm_v, const __grid_const
     while (globaltimer_ns() - t0 < 200000ull) __nanosleep(1000);
     __syncthreads();
   }
-  if (warp == 17) {
+  if (warp == 9) {
     tc_fence_after();
     tmem_dealloc(tmem_base, 512);
   }
@@ -613,13 +691,13 @@ hgrn2_output_kernel(const __grid_constant__ CUtensorMap tm_v, const __grid_const
 using namespace trlb;
 
 // 1 when trlb_hgrn2_chunk takes these sizes.
-TRLB_API int trlb_hgrn2_chunk_ok(int heads, int dim, int vdim) { return heads > 0 && dim > 0 && dim <= 128 && vdim > 0 && vdim % 8 == 0; }
+TRLB_API int trlb_hgrn2_chunk_ok(int heads, int dim, int vdim) { return heads > 0 && dim > 0 && dim <= 128 && dim % 8 == 0 && vdim > 0 && vdim % 8 == 0; }
 
 // Chunks (upper bound) of T packed tokens in n_seq sequences: the leading size of s_hi, s_lo [chunks, heads, dim, vdim] bf16.
 TRLB_API int trlb_hgrn2_chunks(int T, int n_seq) { return (T + HC_L - 1) / HC_L + n_seq; }
 
-// y [T rows of y_ld] bf16 on 16 bytes: q at 0, v at v_off (elements, a multiple of 8); z [T rows of z_ld] fp32 gate logits without bias.
-// S [slots, heads, dim, vdim] of seq_slot gets the final states (null: none).  norm [vdim] (vdim <= 128): y_out [T rows of out_ld on 16
+// y [T rows of y_ld] bf16 on 16 bytes: q at 0, v at v_off (elements, a multiple of 8); z [T rows of z_ld] fp32 on 16 bytes, gate logits without
+// bias.  S [slots, heads, dim, vdim] of seq_slot gets the final states (null: none).  norm [vdim] (vdim <= 128): y_out [T rows of out_ld on 16
 // bytes] = outputs over their rms per head times norm and scale, bf16; else out [T, heads, vdim] fp32.
 TRLB_API int trlb_hgrn2_chunk(const void* y, long long y_ld, int v_off, const float* z, long long z_ld, const float* bias, const float* low,
                               const int* cu, int n_seq, int T, const int* seq_slot, float* S, int slots, int heads, int dim, int vdim,
@@ -627,13 +705,16 @@ TRLB_API int trlb_hgrn2_chunk(const void* y, long long y_ld, int v_off, const fl
                               int* status, cudaStream_t st) {
   if (T <= 0 || n_seq <= 0) return 0;
   const auto off16 = [](const void* x) { return (reinterpret_cast<uintptr_t>(x) & 15) != 0; };
-  if (!trlb_hgrn2_chunk_ok(heads, dim, vdim) || (y_ld % 8) || (v_off % 8) || off16(y)) return -310;
+  if (!trlb_hgrn2_chunk_ok(heads, dim, vdim) || (y_ld % 8) || (v_off % 8) || (z_ld % 4) || off16(y) || off16(z)) return -310;
   if (norm != nullptr ? vdim > 128 || y_out == nullptr || (out_ld % 8) || off16(y_out) || off16(norm) : out == nullptr) return -310;
   if (seq_slot != nullptr && S == nullptr) return -310;
   const int chunks = trlb_hgrn2_chunks(T, n_seq);
   const __nv_bfloat16* x = (const __nv_bfloat16*)y;
-  CUtensorMap tv, tsh, tsl;
+  CUtensorMap tq, tz, tv, tsh, tsl;
   using trlb_host::make_tmap_3d_bf16;
+  if (make_tmap_3d_bf16(&tq, x, dim, heads, T, dim, (uint64_t)y_ld, 64, 1, 128)) return -315;
+  // fp32 rows as twice as many 16-bit elements: they are only copied
+  if (make_tmap_3d_bf16(&tz, z, 2 * dim, heads, T, 2 * dim, (uint64_t)z_ld * 2, 64, 1, 128)) return -316;
   if (make_tmap_3d_bf16(&tv, x + v_off, vdim, heads, T, vdim, (uint64_t)y_ld, 64, 1, 128)) return -311;
   if (make_tmap_3d_bf16(&tsh, s_hi, vdim, dim, (uint64_t)chunks * heads, vdim, (uint64_t)dim * vdim, 64, 128, 1)) return -312;
   if (make_tmap_3d_bf16(&tsl, s_lo, vdim, dim, (uint64_t)chunks * heads, vdim, (uint64_t)dim * vdim, 64, 128, 1)) return -313;
@@ -646,11 +727,11 @@ TRLB_API int trlb_hgrn2_chunk(const void* y, long long y_ld, int v_off, const fl
   }
   Hgrn2Chunk p = {};
   p.cu = cu; p.n_seq = n_seq; p.heads = heads; p.dim = dim; p.vdim = vdim;
-  p.q = x; p.y_ld = y_ld; p.z = z; p.z_ld = z_ld; p.bias = bias; p.low = low;
+  p.bias = bias; p.low = low;
   p.s_hi = (__nv_bfloat16*)s_hi; p.s_lo = (__nv_bfloat16*)s_lo; p.S = S; p.seq_slot = seq_slot; p.slots = slots;
   p.norm = norm; p.eps = eps; p.scale = scale; p.y_out = (__nv_bfloat16*)y_out; p.out_ld = out_ld; p.out = out; p.status = status;
   const int tiles = (vdim + 127) / 128;
-  hgrn2_state_kernel<<<dim3(n_seq, heads, tiles), HS_THREADS, HS_SMEM, st>>>(tv, p);
-  hgrn2_output_kernel<<<dim3(chunks, heads, tiles), HO_THREADS, HO_SMEM, st>>>(tv, tsh, tsl, p);
+  hgrn2_state_kernel<<<dim3(n_seq, heads, tiles), HS_THREADS, HS_SMEM, st>>>(tz, tv, p);
+  hgrn2_output_kernel<<<dim3(chunks, heads, tiles), HO_THREADS, HO_SMEM, st>>>(tq, tz, tv, tsh, tsl, p);
   return (int)cudaGetLastError();
 }

@@ -286,22 +286,22 @@ def hgrn2_rows(m, y, z, ctx, where, out=None, scale=1.0):
     """From the rows ``y`` (query | value) and ``z`` (forget gate, fp32 sums) of the input projection to what the output projection
     reads, times ``scale``.  ``where`` (may be empty): the slots that get the final states."""
     K = _k()
-    if m.vdim <= 128 and _hgrn2_tc(m, y, out):
+    if m.vdim <= 128 and _hgrn2_tc(m, z, y, out):
         out = torch.empty(y.shape[0], m.out_width, dtype=y.dtype, device=y.device) if out is None else out
         return K.hgrn2_chunk(y, z, m, ctx.cu_seqlens, normed=out, scale=scale, **where)
     return K.head_norm(hgrn2_prompt_scan(m, y, z, ctx, where), m.norm, m.eps, y.dtype, out=out, scale=scale)
 
 
-def _hgrn2_tc(m, *rows) -> bool:
+def _hgrn2_tc(m, z, *rows) -> bool:
     """Whether the tensor-core kernels take a mixer's sizes and these rows."""
-    return all(t is None or (t.dtype == torch.bfloat16 and t.data_ptr() % 16 == 0 and t.stride(0) % 8 == 0) for t in rows) and (
-        m.heads * m.dim % 8 == 0 and _k().hgrn2_chunk_ok(m))
+    return (all(t is None or (t.dtype == torch.bfloat16 and t.data_ptr() % 16 == 0 and t.stride(0) % 8 == 0) for t in rows)
+            and z.data_ptr() % 16 == 0 and z.stride(0) % 4 == 0 and _k().hgrn2_chunk_ok(m))
 
 
 def hgrn2_prompt_scan(m, y, z, ctx, where, tensor_cores=True):
     """The recurrence over packed prompts -> fp32 [T, heads, vdim]."""
     K = _k()
-    if tensor_cores and _hgrn2_tc(m, y):
+    if tensor_cores and _hgrn2_tc(m, z, y):
         return K.hgrn2_chunk(y, z, m, ctx.cu_seqlens, **where)
     return K.hgrn2_prompt(y, z, m, ctx.cu_seqlens, **where)
 
