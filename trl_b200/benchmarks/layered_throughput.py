@@ -455,12 +455,10 @@ def gerupel_kernels(s, model, eng, batch, prompt, n_prompts, row):
     row("prompt windowed attention with blocks (sink)", lambda: KM.mixer_attn(q, k, v, heads=at.heads, kv_heads=at.kv_heads, scale=at.scale, **at.sight, pool=at.pool,
                                                                              blocks=blocks, ctx=ctx, out=o[:, : at.out_width], out_scale=0.9),
         T * 2 * (at.rows + at.out_width), 2 * pairs * at.heads * (at.dim + at.vdim))
-    row("prompt hgrn2 recurrence", lambda: mx.hgrn2_prompt_scan(rg, yr, z, ctx, target["right"]),
-        T * rg.heads * (rg.dim * 6 + rg.vdim * 6) + n_prompts * rg.heads * rg.dim * rg.vdim * 4,
+    row("prompt hgrn2 (states + outputs + norm per head)", lambda: mx.hgrn2_rows(rg, yr, z, ctx, target["right"], out=o[:, at.out_width:], scale=0.7),
+        T * rg.heads * (rg.dim * 6 + rg.vdim * 4) + n_prompts * rg.heads * rg.dim * rg.vdim * 4,
         2 * T * rg.heads * (2 * rg.dim * rg.vdim + 64 * (rg.dim + rg.vdim)))
-    o32 = mx.hgrn2_prompt_scan(rg, yr, z, ctx, {})
-    row("prompt norm per head", lambda: KM.head_norm(o32, rg.norm, 1e-6, bf, out=o[:, at.out_width:], scale=0.7), o32.numel() * 6)
-    del y, z, o, ya, yr, q, k, v, o32
+    del y, z, o, ya, yr, q, k, v
     prompt_expert_kernels(moe, h, row)
 
     a = eng.slots[0]

@@ -50,21 +50,8 @@ __device__ __forceinline__ int hc_chunks(int len) { return (len + HC_L - 1) / HC
 // exp bounded so that a product of two stays finite
 __device__ __forceinline__ float hc_exp(float x) { return fast_exp2(fminf(1.4426950408889634f * x, 60.f)); }
 
-// Eight values as bf16 and remainders, 16 bytes each.
-__device__ __forceinline__ void hc_put8(uint8_t* hi, uint8_t* lo, const float (&v)[8]) {
-  uint32_t a[4], b[4];
-#pragma unroll
-  for (int i = 0; i < 4; ++i) {
-    a[i] = pack_bf16(v[2 * i], v[2 * i + 1]);
-    const float2 f = unpack_bf16(a[i]);
-    b[i] = pack_bf16(v[2 * i] - f.x, v[2 * i + 1] - f.y);
-  }
-  *reinterpret_cast<uint4*>(hi) = make_uint4(a[0], a[1], a[2], a[3]);
-  *reinterpret_cast<uint4*>(lo) = make_uint4(b[0], b[1], b[2], b[3]);
-}
-
-// The same to shared memory (32-bit addresses).
-__device__ __forceinline__ void hc_put8_smem(uint32_t hi, uint32_t lo, const float (&v)[8]) {
+// Eight values as bf16 and remainders to shared memory, 16 bytes each.
+__device__ __forceinline__ void hc_put8(uint32_t hi, uint32_t lo, const float (&v)[8]) {
   uint32_t a[4], b[4];
 #pragma unroll
   for (int i = 0; i < 4; ++i) {
@@ -114,7 +101,8 @@ __device__ __forceinline__ float hc_query(uint32_t boxes, int d, int t) {
 
 // ------------------------------------------------------------------------------------------------------------
 // State pass.  Warps 0-15: thread (channel, quarter of the tokens) forms the scaled keys, warp (32 rows of S, 32 columns) scales the
-// state; warp 16: TMA; warp 17: MMA.  The gate logits of the next chunk arrive while the products of this one run.
+// state; warp 16: TMA; warp 17: MMA.  The gate logits of the next chunk arrive while the products of this one run.  The state in front
+// of a chunk goes out through the place of the keys, whole lines at a time.
 // ------------------------------------------------------------------------------------------------------------
 constexpr int HC_WORK = 512, HS_THREADS = HC_WORK + 64;
 constexpr size_t HS_SMEM = 12 * (size_t)HC_BOX + 1024 + 4096 + 256;
@@ -207,7 +195,10 @@ hgrn2_state_kernel(const __grid_constant__ CUtensorMap tm_z, const __grid_consta
     const int hd = h * p.dim + (on ? d : 0);
     const float bias = p.bias[hd], room = 1.f - p.low[hd];
     const uint32_t t_row = tmem_base + ((uint32_t)((warp & 3) * 32) << 16) + (uint32_t)x0;
-    uint8_t* keys = k_s + (size_t)(qt >> 1) * HC_BOX + (size_t)d * 128;
+    // eight tokens of this channel's keys, or eight columns of this row of the state: numbers 0 .. 3 of this quarter
+    const uint32_t keys = smem_u32(k_s) + (uint32_t)(qt >> 1) * HC_BOX + (uint32_t)d * 128;
+    auto eight = [&](int g) { return keys + ((((uint32_t)(qt & 1) * 4 + g) ^ ((uint32_t)d & 7)) << 4); };
+    const int per_row = min(16, (p.vdim - e0) >> 3);  // pieces of eight columns
     bool ok = true;
     for (int c = 0; c < nc; ++c) {
       const int n = on ? len - c * HC_L - 32 * qt : 0;  // tokens here
@@ -229,8 +220,38 @@ hgrn2_state_kernel(const __grid_constant__ CUtensorMap tm_z, const __grid_consta
       const float decay = (pr[0] * pr[128]) * (pr[256] * pr[384]);
       // the products of the chunk before have read the keys and left the state
       if (c > 0) ok = ok && __all_sync(0xffffffffu, mbar_wait(acc_full, (uint32_t)((c - 1) & 1), abort_flag, p.status, 2021));
+      if (c > 0) {
+        if (ok && x0 < cols) {
+          tc_fence_after();
+#pragma unroll
+          for (int y = 0; y < 2; ++y) {
+            float s[16];
+            tmem_ld_32x16(t_row + 16 * y, s);
+            tmem_ld_wait();
+            uint32_t u[16];
+#pragma unroll
+            for (int i = 0; i < 16; ++i) u[i] = __float_as_uint(s[i] * decay);
+            tmem_st_32x16(t_row + 16 * y, u);
+#pragma unroll
+            for (int g = 0; g < 2; ++g) {
+              const float v[8] = {s[8 * g], s[8 * g + 1], s[8 * g + 2], s[8 * g + 3], s[8 * g + 4], s[8 * g + 5], s[8 * g + 6], s[8 * g + 7]};
+              hc_put8(eight(2 * y + g), eight(2 * y + g) + 2 * HC_BOX, v);
+            }
+          }
+          tmem_st_wait();
+        }
+        hc_sync<HC_WORK>();
+        const size_t base = ((size_t)(chunk0 + c) * p.heads + h) * p.dim * p.vdim + e0;
+        for (int i = tid; i < p.dim * per_row; i += HC_WORK) {
+          const int r = i / per_row, g = i % per_row;
+          const uint8_t* src = k_s + (size_t)(g >> 3) * HC_BOX + (size_t)r * 128 + (((g & 7) ^ (r & 7)) << 4);
+          const size_t at = base + (size_t)r * p.vdim + 8 * g;
+          *reinterpret_cast<uint4*>(p.s_hi + at) = *reinterpret_cast<const uint4*>(src);
+          *reinterpret_cast<uint4*>(p.s_lo + at) = *reinterpret_cast<const uint4*>(src + 2 * HC_BOX);
+        }
+        hc_sync<HC_WORK>();  // the keys may take the place
+      }
       if (!ok) continue;
-      tc_fence_after();
 #pragma unroll
       for (int g = 3; g >= 0; --g) {
         float v[8];
@@ -239,31 +260,9 @@ hgrn2_state_kernel(const __grid_constant__ CUtensorMap tm_z, const __grid_consta
           v[i] = k[8 * g + i] * w;
           w = fmaf(-k[8 * g + i], w, w);
         }
-        const int at = (((qt & 1) * 4 + g) ^ (d & 7)) << 4;
-        hc_put8(keys + at, keys + 2 * HC_BOX + at, v);
+        hc_put8(eight(g), eight(g) + 2 * HC_BOX, v);
       }
       fence_proxy_async_smem();
-      if (c > 0 && x0 < cols) {
-        const size_t row = (((size_t)(chunk0 + c) * p.heads + h) * p.dim + d) * p.vdim + e0 + x0;
-#pragma unroll 1
-        for (int x = 0; x < 32; x += 16) {
-          float s[16];
-          tmem_ld_32x16(t_row + x, s);
-          tmem_ld_wait();
-          uint32_t u[16];
-#pragma unroll
-          for (int i = 0; i < 16; ++i) u[i] = __float_as_uint(s[i] * decay);
-          tmem_st_32x16(t_row + x, u);
-#pragma unroll
-          for (int y = 0; y < 16; y += 8) {
-            if (on && e0 + x0 + x + y < p.vdim) {
-              const float v[8] = {s[y], s[y + 1], s[y + 2], s[y + 3], s[y + 4], s[y + 5], s[y + 6], s[y + 7]};
-              hc_put8(reinterpret_cast<uint8_t*>(p.s_hi + row + x + y), reinterpret_cast<uint8_t*>(p.s_lo + row + x + y), v);
-            }
-          }
-        }
-        tmem_st_wait();
-      }
       tc_fence_before();
       mbar_arrive(ready);
     }
@@ -303,8 +302,9 @@ hgrn2_state_kernel(const __grid_constant__ CUtensorMap tm_z, const __grid_consta
 // level by level (rows of the operands are channels: eight tokens are one 16-byte store); later warp (32 queries, 64 keys) turns the
 // levels' products into scores, and (32 queries, 64 columns) norms the output.  Warp 8: TMA; warp 9: MMA.  Every barrier is used once.
 //
-// Gate logits and queries come to slot 1 and go to registers.  Steps: 0 blocks of 8, 1 - 4 levels of 64, 32, 16, 8, 5 queries against the state.  Two slots of shared memory (queries 64 KB, keys
-// 32 KB, value and remainder each) and 32 KB more for the keys 64 .. 127 of step 0, where v goes later; the state goes where keys were.
+// Gate logits and queries come to slot 1 and go to registers.  Steps: 0 blocks of 8, 1 - 4 levels of 64, 32, 16, 8, 5 queries against
+// the state.  Two slots of shared memory (queries 64 KB, keys 32 KB, value and remainder each) and 32 KB more for the keys 64 .. 127 of
+// step 0, where v goes later; the state goes where keys were.
 // TMEM: levels [0, 256), blocks of 8 [256, 384), output [384, 512); the scores replace the levels of 64 and 32.
 // ------------------------------------------------------------------------------------------------------------
 constexpr int HO_WORK = 256, HO_THREADS = HO_WORK + 64;
@@ -479,7 +479,7 @@ hgrn2_output_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
           v[i] = q[i0 + 8 * g + i] * w;
         }
         const uint32_t at = chunk16((uint32_t)(i0 / 8 + g)) + mine + slot;
-        hc_put8_smem(at, at + 2 * HC_BOX, v);
+        hc_put8(at, at + 2 * HC_BOX, v);
       }
     };
     // keys i0 .. i0 + n - 1 times the gates behind them up to i0 + n - 1; g0: where they begin among the 64 of the level
@@ -495,7 +495,7 @@ hgrn2_output_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
           w = fmaf(-k[i0 + 8 * g + i], w, w);
         }
         const uint32_t at = chunk16((uint32_t)(g0 + g)) + slot + 4 * HC_BOX;
-        hc_put8_smem(at, at + HC_BOX, v);
+        hc_put8(at, at + HC_BOX, v);
       }
     };
     constexpr uint32_t slot0 = 0, slot1 = HO_SLOT;
@@ -526,7 +526,7 @@ hgrn2_output_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
           w *= gate(i);
           v[i] = q[8 * g + i] * w;
         }
-        hc_put8_smem(at + mine + slot0, at + mine + slot0 + 2 * HC_BOX, v);
+        hc_put8(at + mine + slot0, at + mine + slot0 + 2 * HC_BOX, v);
         w = hc_afresh(__fdividef(1.f, high));
 #pragma unroll
         for (int i = 7; i >= 4; --i) {
@@ -539,7 +539,7 @@ hgrn2_output_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
           v[i] = k[8 * g + i] * w;
           w *= gate(i);
         }
-        hc_put8_smem(at + b, at + b + HC_BOX, v);
+        hc_put8(at + b, at + b + HC_BOX, v);
       }
     }
     filled(0);
@@ -651,17 +651,23 @@ hgrn2_output_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
         hc_sync<HO_WORK>();
         const float* r = red + 32 * rq + lane;
         const float f = p.scale / sqrtf((r[0] + r[128]) / (float)p.vdim + p.eps);
-        if (row_ok) {
-          __nv_bfloat16* y = p.y_out + (size_t)(beg + t) * p.out_ld + (size_t)h * p.vdim + x0;
+        uint8_t* rows = smem + HC_BOX;  // two boxes of 64 columns, rows are tokens
 #pragma unroll
-          for (int x = 0; x < 64; x += 8) {
-            if (x0 + x < p.vdim) {
-              const float* u = &o[x >> 5][x & 31];
-              const float4 g = load4(p.norm + x0 + x), g2 = load4(p.norm + x0 + x + 4);
-              *reinterpret_cast<uint4*>(y + x) = make_uint4(pack_bf16(u[0] * f * g.x, u[1] * f * g.y), pack_bf16(u[2] * f * g.z, u[3] * f * g.w),
-                                                            pack_bf16(u[4] * f * g2.x, u[5] * f * g2.y), pack_bf16(u[6] * f * g2.z, u[7] * f * g2.w));
-            }
+        for (int x = 0; x < 64; x += 8) {
+          if (x0 + x < p.vdim) {
+            const float* u = &o[x >> 5][x & 31];
+            const float4 g = load4(p.norm + x0 + x), g2 = load4(p.norm + x0 + x + 4);
+            *reinterpret_cast<uint4*>(rows + (size_t)kh * HC_BOX + (size_t)(32 * rq + lane) * 128 + (((x >> 3) ^ (lane & 7)) << 4)) =
+                make_uint4(pack_bf16(u[0] * f * g.x, u[1] * f * g.y), pack_bf16(u[2] * f * g.z, u[3] * f * g.w),
+                           pack_bf16(u[4] * f * g2.x, u[5] * f * g2.y), pack_bf16(u[6] * f * g2.z, u[7] * f * g2.w));
           }
+        }
+        hc_sync<HO_WORK>();
+        const int per_row = p.vdim >> 3, n = ok ? min(HC_L, len - c * HC_L) * per_row : 0;
+        for (int i = tid; i < n; i += HO_WORK) {
+          const int r = i / per_row, g = i % per_row;
+          *reinterpret_cast<uint4*>(p.y_out + (size_t)(row0 + r) * p.out_ld + (size_t)h * p.vdim + 8 * g) =
+              *reinterpret_cast<const uint4*>(rows + (size_t)(g >> 3) * HC_BOX + (size_t)r * 128 + (((g & 7) ^ (r & 7)) << 4));
         }
       } else if (row_ok) {
         float* dst = p.out + ((size_t)(beg + t) * p.heads + h) * p.vdim + e0 + x0;
