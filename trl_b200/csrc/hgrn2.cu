@@ -149,6 +149,19 @@ hgrn2_step_kernel(const Hgrn2Step p, T* __restrict__ y) {
   const int h = blockIdx.x, b = blockIdx.y, tid = threadIdx.x, cgs = 1 << p.groups_log2, cg = tid & (cgs - 1), rg = tid >> p.groups_log2;
   const int rgs = 256 >> p.groups_log2;
   const bool live = p.seq_lens[b] >= 0;
+  constexpr int ROWS = 8;  // of S that a thread has under way at a time
+  float* S = p.S + ((size_t)b * p.heads + h) * p.dim * p.vdim;
+  float4 t[ROWS];
+  auto fetch = [&](int e, int d0) {
+#pragma unroll
+    for (int j = 0; j < ROWS; ++j) {
+      const int d = d0 + j * rgs;
+      if (d >= p.dim) continue;
+      if (VEC == 4) t[j] = load4(S + (size_t)d * p.vdim + e);
+      else t[j].x = S[(size_t)d * p.vdim + e];
+    }
+  };
+  if (live && cg * VEC < p.vdim) fetch(cg * VEC, rg);  // while the sums are read
   float* qs = sm;
   float* ks = qs + p.dim;
   float* vs = ks + p.dim;
@@ -168,7 +181,6 @@ hgrn2_step_kernel(const Hgrn2Step p, T* __restrict__ y) {
   }
   if (!live) return;  // uniform
   __syncthreads();
-  float* S = p.S + ((size_t)b * p.heads + h) * p.dim * p.vdim;
   for (int e = cg * VEC; e < p.vdim; e += cgs * VEC) {
     float o[VEC], w[VEC];
 #pragma unroll
@@ -176,23 +188,21 @@ hgrn2_step_kernel(const Hgrn2Step p, T* __restrict__ y) {
       o[i] = 0.f;
       w[i] = vs[e + i];
     }
-#pragma unroll 4
-    for (int d = rg; d < p.dim; d += rgs) {
-      float s[VEC];
-      float* at = S + (size_t)d * p.vdim + e;
-      if (VEC == 4) {
-        const float4 t = load4(at);
-        s[0] = t.x; s[1 % VEC] = t.y; s[2 % VEC] = t.z; s[3 % VEC] = t.w;
-      } else {
-        s[0] = *at;
-      }
+    for (int d0 = rg; d0 < p.dim; d0 += ROWS * rgs) {
+      if (d0 != rg || e != cg * VEC) fetch(e, d0);
 #pragma unroll
-      for (int i = 0; i < VEC; ++i) {
-        s[i] = fmaf(ks[d], w[i] - s[i], s[i]);
-        o[i] = fmaf(s[i], qs[d], o[i]);
+      for (int j = 0; j < ROWS; ++j) {
+        const int d = d0 + j * rgs;
+        if (d >= p.dim) continue;
+        float s[4] = {t[j].x, t[j].y, t[j].z, t[j].w};
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) {
+          s[i] = fmaf(ks[d], w[i] - s[i], s[i]);
+          o[i] = fmaf(s[i], qs[d], o[i]);
+        }
+        if (VEC == 4) store4(S + (size_t)d * p.vdim + e, make_float4(s[0], s[1], s[2], s[3]));
+        else S[(size_t)d * p.vdim + e] = s[0];
       }
-      if (VEC == 4) store4(at, make_float4(s[0], s[1 % VEC], s[2 % VEC], s[3 % VEC]));
-      else *at = s[0];
     }
 #pragma unroll
     for (int i = 0; i < VEC; ++i) part[(size_t)rg * p.vdim + e + i] = o[i];
