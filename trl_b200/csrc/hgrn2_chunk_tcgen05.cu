@@ -242,8 +242,8 @@ hgrn2_state_kernel(const __grid_constant__ CUtensorMap tm_z, const __grid_consta
         }
         hc_sync<HC_WORK>();
         const size_t base = ((size_t)(chunk0 + c) * p.heads + h) * p.dim * p.vdim + e0;
-        for (int i = tid; i < p.dim * per_row; i += HC_WORK) {
-          const int r = i / per_row, g = i % per_row;
+        const int g = tid & 15;
+        for (int r = g < per_row ? tid >> 4 : p.dim; r < p.dim; r += HC_WORK / 16) {
           const uint8_t* src = k_s + (size_t)(g >> 3) * HC_BOX + (size_t)r * 128 + (((g & 7) ^ (r & 7)) << 4);
           const size_t at = base + (size_t)r * p.vdim + 8 * g;
           *reinterpret_cast<uint4*>(p.s_hi + at) = *reinterpret_cast<const uint4*>(src);
@@ -309,7 +309,7 @@ hgrn2_state_kernel(const __grid_constant__ CUtensorMap tm_z, const __grid_consta
 // ------------------------------------------------------------------------------------------------------------
 constexpr int HO_WORK = 256, HO_THREADS = HO_WORK + 64;
 constexpr uint32_t HO_SLOT = 6 * HC_BOX;
-constexpr size_t HO_SMEM = 2 * (size_t)HO_SLOT + 2 * HC_BOX + 1024 + 512 + 256;
+constexpr size_t HO_SMEM = 2 * (size_t)HO_SLOT + 2 * HC_BOX + 1024 + 1024 + 256;
 
 __global__ void __launch_bounds__(HO_THREADS, 1)
 hgrn2_output_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_z, const __grid_constant__ CUtensorMap tm_v, const __grid_constant__ CUtensorMap tm_sh, const __grid_constant__ CUtensorMap tm_sl,
@@ -326,7 +326,8 @@ hgrn2_output_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
   // a slot: queries [2 groups of 64 tokens] value, remainder, keys [64 tokens] value, remainder
   uint8_t* x_s = smem + 2 * HO_SLOT;
   float* prod = reinterpret_cast<float*>(x_s + 2 * HC_BOX);  // [128] product of the gates of the first half
-  uint64_t* bars = reinterpret_cast<uint64_t*>(prod + 128);
+  float* norm = prod + 128;                                  // [128] weights of the norm
+  uint64_t* bars = reinterpret_cast<uint64_t*>(norm + 128);
   uint64_t* full = bars;        // [6] operands of a step written
   uint64_t* done = bars + 6;    // [5] its products done
   uint64_t* v_full = bars + 11;
@@ -390,14 +391,16 @@ hgrn2_output_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
     __syncwarp();
   } else if (warp == 9) {
     if (lane == 0) {
-      constexpr uint32_t idesc_s = umma_idesc_bf16_major(128, 64, true, true);
+      constexpr uint32_t idesc_s = umma_idesc_bf16_major(128, 64, true, true), idesc_0 = umma_idesc_bf16_major(128, 128, true, true);
       const uint32_t idesc_x = umma_idesc_bf16_major(128, cols, true, true), idesc_o = umma_idesc_bf16_major(128, cols, false, true);
       const uint64_t base = umma_desc_mnmajor_sw128(smem_u32(smem), HC_BOX);
+      // step 0 reads keys from two places, 64 tokens each
+      const uint64_t base0 = umma_desc_mnmajor_sw128(smem_u32(smem), 2 * HO_SLOT - 4 * HC_BOX);
       // value x value, value x remainder, remainder x value
-      auto products = [&](uint32_t tmem_d, uint32_t a, uint32_t b, uint32_t lo_a, uint32_t lo_b, uint32_t idesc) {
+      auto products = [&](uint32_t tmem_d, uint32_t slot, uint64_t keys, uint32_t idesc) {
 #pragma unroll 1
         for (int part = 0; part < 3; ++part) {
-          const uint64_t da = desc_at(base, a + (part == 2 ? lo_a : 0)), db = desc_at(base, b + (part == 1 ? lo_b : 0));
+          const uint64_t da = desc_at(base, slot + (part == 2 ? 2 * HC_BOX : 0)), db = desc_at(keys, slot + 4 * HC_BOX + (part == 1 ? HC_BOX : 0));
 #pragma unroll 1
           for (int kk = 0; kk < ksteps; ++kk) umma_bf16_ss(tmem_d, desc_at(da, kk * 2048), desc_at(db, kk * 2048), idesc, (part | kk) != 0);
         }
@@ -408,12 +411,8 @@ hgrn2_output_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
         if (!ok) break;
         tc_fence_after();
         const uint32_t slot = (s & 1) * HO_SLOT;
-        if (s == 0) {
-          products(tmem_base + 256, slot, slot + 4 * HC_BOX, 2 * HC_BOX, HC_BOX, idesc_s);
-          products(tmem_base + 320, slot, 2 * HO_SLOT, 2 * HC_BOX, HC_BOX, idesc_s);
-        } else {
-          products(tmem_base + 64 * (s - 1), slot, slot + 4 * HC_BOX, 2 * HC_BOX, HC_BOX, idesc_s);
-        }
+        if (s == 0) products(tmem_base + 256, slot, base0, idesc_0);
+        else products(tmem_base + 64 * (s - 1), slot, base, idesc_s);
         umma_commit(&done[s]);
       }
       if (ok && carried) {
@@ -461,6 +460,7 @@ hgrn2_output_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
         all = fmaf(-k[i], all, all);
       }
       if (half == 0) prod[d] = all;
+      else if (p.norm != nullptr && d < p.vdim) norm[d] = p.norm[d];
     }
     hc_sync<HO_WORK>();  // slot 1 is free
     const uint32_t sw = (uint32_t)(d & 7), row = smem_u32(smem) + (uint32_t)d * 128;
@@ -656,16 +656,15 @@ hgrn2_output_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
         for (int x = 0; x < 64; x += 8) {
           if (x0 + x < p.vdim) {
             const float* u = &o[x >> 5][x & 31];
-            const float4 g = load4(p.norm + x0 + x), g2 = load4(p.norm + x0 + x + 4);
+            const float4 g = load4(norm + x0 + x), g2 = load4(norm + x0 + x + 4);
             *reinterpret_cast<uint4*>(rows + (size_t)kh * HC_BOX + (size_t)(32 * rq + lane) * 128 + (((x >> 3) ^ (lane & 7)) << 4)) =
                 make_uint4(pack_bf16(u[0] * f * g.x, u[1] * f * g.y), pack_bf16(u[2] * f * g.z, u[3] * f * g.w),
                            pack_bf16(u[4] * f * g2.x, u[5] * f * g2.y), pack_bf16(u[6] * f * g2.z, u[7] * f * g2.w));
           }
         }
         hc_sync<HO_WORK>();
-        const int per_row = p.vdim >> 3, n = ok ? min(HC_L, len - c * HC_L) * per_row : 0;
-        for (int i = tid; i < n; i += HO_WORK) {
-          const int r = i / per_row, g = i % per_row;
+        const int g = tid & 15, n = ok && g < (p.vdim >> 3) ? min(HC_L, len - c * HC_L) : 0;  // pieces of eight columns
+        for (int r = tid >> 4; r < n; r += HO_WORK / 16) {
           *reinterpret_cast<uint4*>(p.y_out + (size_t)(row0 + r) * p.out_ld + (size_t)h * p.vdim + 8 * g) =
               *reinterpret_cast<const uint4*>(rows + (size_t)(g >> 3) * HC_BOX + (size_t)r * 128 + (((g & 7) ^ (r & 7)) << 4));
         }
